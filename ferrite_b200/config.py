@@ -16,6 +16,23 @@ from typing import List, Optional
 
 
 @dataclass
+class LayerSpec:
+    """One layer of a model that lists its layers one by one (`ModelConfig.layers`): the mixer, its sizes and the
+    feed-forward behind it. Layers of one model may differ in all of them."""
+
+    mixer: str = "latent"           # attention over a cached low-rank latent, no positions
+    heads: int = 1
+    dim: int = 0                    # query / key width of a head
+    vdim: int = 0                   # value width of a head
+    q_rank: int = 0                 # the queries come out of a normalised latent of this width
+    kv_rank: int = 0                # width of the cached latent
+    scale: float = 1.0              # scores are (q . k) * scale
+    kv_from: Optional[int] = None   # use the latents that this (earlier) layer caches instead of own ones
+    ff: int = 0                     # feed-forward width, 0 = the layer has none
+    act: str = "relu2"              # its activation
+
+
+@dataclass
 class ModelConfig:
     """Dense hybrid decoder (Gated DeltaNet + gated GQA attention), optionally with MoE FFN or MLA attention."""
 
@@ -57,6 +74,14 @@ class ModelConfig:
     rope_head_dim: int = 0
     nope_head_dim: int = 0
     v_head_dim: int = 0
+    # ---- layers listed one by one (they replace the pattern fields above) ----
+    layers: List[LayerSpec] = field(default_factory=list)
+    out_norm: bool = False          # x + norm(f(x)): norms on the sublayers' outputs, a 32-bit residual stream, plain norm weights
+    embed_scale: float = 1.0
+    gram_buckets: int = 0           # hashed bigram embedding: rows of the table besides the one for a sequence's first token
+    gram_mul_prev: int = 0
+    gram_mul_cur: int = 0
+    logit_softcap: float = 0.0      # logits <- cap * tanh(logits / cap), 0 = off
     # ---- drafter taps ----
     tap_layers: List[int] = field(default_factory=list)
 
@@ -68,12 +93,16 @@ class ModelConfig:
 
     @property
     def layer_kinds(self) -> List[str]:
+        if self.layers:
+            return [l.mixer for l in self.layers]
         if self.kv_lora > 0:
             return ["mla"] * self.n_layers
         return ["attn" if self.is_attn(i) else "gdn" for i in range(self.n_layers)]
 
     @property
     def n_attn(self) -> int:
+        if self.layers:
+            return sum(1 for l in self.layers if l.kv_from is None)
         return sum(1 for k in self.layer_kinds if k != "gdn")
 
     @property
@@ -104,6 +133,12 @@ class ModelConfig:
     def param_count(self) -> int:
         h = self.hidden
         n = self.vocab * h * (1 if self.tie_embeddings else 2)
+        if self.layers:
+            n += (self.gram_buckets + 1) * h if self.gram_buckets else 0
+            for l in self.layers:
+                n += h * l.q_rank + l.q_rank * l.heads * l.dim + l.heads * (l.dim + l.vdim) * l.kv_rank + l.heads * l.vdim * h
+                n += (h * l.kv_rank if l.kv_from is None else 0) + 2 * h * l.ff
+            return n
         for i, kind in enumerate(self.layer_kinds):
             if kind == "gdn":
                 n += h * self.gdn_in_dim + self.lin_v_heads * self.lin_dv * h + self.conv_dim * self.conv_k
@@ -126,6 +161,11 @@ class ModelConfig:
         c = dataclasses.replace(self)
         if world == 1:
             return c
+        if self.layers:
+            assert all(l.heads % world == 0 and l.ff % world == 0 for l in self.layers), \
+                f"heads and feed-forward widths must divide over {world} ranks"
+            c.layers = [dataclasses.replace(l, heads=l.heads // world, ff=l.ff // world) for l in self.layers]
+            return c
         assert self.n_q % world == 0 and self.inter % world == 0
         c.n_q = self.n_q // world
         c.n_kv = max(1, self.n_kv // world)
@@ -144,8 +184,14 @@ class ModelConfig:
     @staticmethod
     def from_hf(path: str | os.PathLike) -> "ModelConfig":
         """Read a Hugging Face `config.json` (the `text_config` block when present), the way the
-        reference does in `crates/fe-model/src/config.rs:44-78`."""
+        reference does in `crates/fe-model/src/config.rs:44-78`. A file that names its `architecture` is read by that
+        architecture's entry in `ARCHITECTURES`."""
         v = json.loads(Path(path).read_text())
+        if "architecture" in v:
+            arch = v["architecture"]
+            if arch not in ARCHITECTURES:
+                raise ValueError(f"unknown architecture {arch!r}: known are {', '.join(sorted(ARCHITECTURES))}")
+            return ARCHITECTURES[arch](v)
         t = v.get("text_config", v)
         rp = t.get("rope_parameters") or {}
         head_dim = int(t["head_dim"])
@@ -167,6 +213,37 @@ class ModelConfig:
             vocab=int(t["vocab_size"]), tie_embeddings=bool(v.get("tie_word_embeddings", False)),
             eos=int(t.get("eos_token_id", 0) if not isinstance(t.get("eos_token_id"), list) else t["eos_token_id"][0]),
         )
+
+
+# ---- architectures by the name their config.json carries ------------------------------------------------------------
+
+def zototar_config(v: dict) -> ModelConfig:
+    """A Zototar config.json: latent attention without positions (latents optionally shared between layers), norms on the
+    sublayers' outputs, squared-relu feed-forwards, a hashed bigram embedding beside the token's, softcapped logits."""
+    layers: List[LayerSpec] = []
+    for i, e in enumerate(v["layers"]):
+        if e["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: mixer type {e['type']!r} is not latent_attention")
+        m, ff = e["mixer"], e.get("mlp")
+        if ff and ff["kind"] != "dense":
+            raise ValueError(f"layer {i}: feed-forward kind {ff['kind']!r} is not dense")
+        src = m.get("kv_from")
+        if src is not None and (not 0 <= src < i or layers[src].kv_from is not None or layers[src].kv_rank != int(m["kv_rank"])):
+            raise ValueError(f"layer {i}: kv_from {src} must name an earlier layer with latents of its own and the same kv_rank")
+        layers.append(LayerSpec(mixer="latent", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                q_rank=int(m["q_rank"]), kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                                kv_from=None if src is None else int(src), ff=int(ff["ff"]) if ff else 0))
+    emb = v["embedding"]
+    gram = emb.get("bigram") or {}
+    return ModelConfig(
+        name="zototar", hidden=int(v["width"]), inter=max([l.ff for l in layers] + [0]), n_layers=len(layers),
+        n_q=layers[0].heads, n_kv=1, head_dim=layers[0].dim, eps=float(v["norm"]["eps"]), vocab=int(v["vocab"]),
+        attn_gate=False, tie_embeddings=False, layers=layers, out_norm=True, embed_scale=float(emb.get("scale", 1.0)),
+        gram_buckets=int(gram.get("buckets", 0)), gram_mul_prev=int(gram.get("mul_prev", 0)),
+        gram_mul_cur=int(gram.get("mul_cur", 0)), logit_softcap=float(v.get("logit_softcap") or 0.0))
+
+
+ARCHITECTURES = {"Zototar": zototar_config}
 
 
 # ---- presets: the five benchmark configurations ----------------------------------------------------
@@ -223,7 +300,32 @@ def tiny_mla(moe: bool = True) -> ModelConfig:
                        v_head_dim=32, **kw)
 
 
+def zototar(width: int, n_layers: int, heads: int, q_rank: int, kv_rank: int, ff: int, vocab: int, dim: int = 128,
+            vdim: int = 128, buckets: int = 65521, name: str = "zototar") -> ModelConfig:
+    """A Zototar model of uniform layers in which every second layer shares the latents of the one before it."""
+    layers = [LayerSpec(heads=heads, dim=dim, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank, scale=dim ** -0.5,
+                        kv_from=None if i % 2 == 0 else i - 1, ff=ff) for i in range(n_layers)]
+    return ModelConfig(name=name, hidden=width, inter=ff, n_layers=n_layers, n_q=heads, n_kv=1, head_dim=dim, eps=1e-6,
+                       vocab=vocab, attn_gate=False, tie_embeddings=False, layers=layers, out_norm=True,
+                       embed_scale=width ** 0.5, gram_buckets=buckets, gram_mul_prev=31, gram_mul_cur=7, logit_softcap=30.0)
+
+
+def tiny_zototar() -> ModelConfig:
+    """5-layer plumbing model of the latent-attention family: unequal layers, sizes off the kernels' tile grid."""
+    c = zototar(200, 5, 4, 72, 80, 224, 300, dim=40, vdim=24, buckets=97, name="tiny-zototar")
+    c.layers[2] = dataclasses.replace(c.layers[2], heads=3, dim=16, vdim=48, q_rank=56, kv_rank=136, scale=0.3, ff=0)
+    c.layers[3] = dataclasses.replace(c.layers[3], kv_from=0, heads=2)
+    c.layers[4] = dataclasses.replace(c.layers[4], kv_from=2, kv_rank=136, ff=104)
+    return c
+
+
+def zototar_7b() -> ModelConfig:
+    """7B-class latent-attention model: 32 layers of width 4096, 32 heads of 128, latents of 512, FFN 16384."""
+    return zototar(4096, 32, 32, 1536, 512, 16384, 129280, name="zototar-7b")
+
+
 PRESETS = {
+    "tiny-zototar": tiny_zototar, "zototar-7b": zototar_7b,
     "tiny": tiny_hybrid, "tiny-mla": tiny_mla, "27b": hybrid_27b, "drafter": drafter_block, "moe80b": moe_80b, "mla671b": mla_671b,
 }
 
@@ -232,6 +334,7 @@ def scaled(cfg: ModelConfig, n_layers: int) -> ModelConfig:
     """Same architecture with fewer layers (for tests that need real widths but little memory)."""
     c = dataclasses.replace(cfg)
     c.n_layers = n_layers
+    c.layers = list(cfg.layers[:n_layers])
     c.tap_layers = [t for t in cfg.tap_layers if t < n_layers]
     return c
 
@@ -244,6 +347,8 @@ class EngineConfig:
     n_slots: int = 4
     max_ctx: int = 4096
     kv_block: int = 64                 # tokens per KV page
+    kv_pool_tokens: int = 0            # tokens the page pool holds over all slots (0 = max_ctx for every slot)
+    compute_dtype: str = "bf16"        # "bf16" | "fp32": activations, weights, cache and products in 32 bits (models of listed layers)
     kv_dtype: str = "bf16"             # "bf16" | "fp8"
     weight_dtype: str = "bf16"         # "bf16" | "nvfp4" | "nvfp4-w4a4" | "nvfp4-a16" | "fp8-block" (e4m3, 128 x 128 blocks) | "exl3[-bits]"
     prefill_chunk: int = 2048          # rows per prompt forward (reference FERRITE_CHUNK)

@@ -117,7 +117,8 @@ int fb_kv_dequant_qn(void* k_out, void* v_out, const void* k_cache, const void* 
 int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                        long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                        const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg, int max_rows,
-                       long q_rows, long cache_rows, int nq, int nkv, int hd, int gated, int* status, cudaStream_t s);
+                       long q_rows, long cache_rows, int nq, int nkv, int hd, int gated, float scale, int exact_p,
+                       long kv_stride, int* status, cudaStream_t s);
 
 // ---- gdn.cu ----
 int fb_gdn_conv(void* out, const void* proj, long proj_stride, const void* conv_w, const void* conv_state,

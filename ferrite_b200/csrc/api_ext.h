@@ -158,6 +158,29 @@ int fb_mla_expand(void* kp, void* vp, const void* kvx, const void* lat, long row
 int fb_mla_qpad(void* qp, const void* q, long q_stride, const void* qabs, long rows, int nq, int dn, int L, int R, int HP,
                 float scale, cudaStream_t s);
 
+// ---- latent.cu ----
+int fb_embed_grams(float* x, void* xb, const void* table, const void* grams, const int* tok, const int* slot, const int* pos,
+                   const int* block_table, int max_blocks, int kv_block, int* tok_pages, int rows, int width, int vocab, float scale,
+                   long buckets, long mul_prev, long mul_cur, int f32, int* status, cudaStream_t s);
+int fb_add_normed(float* x, void* xb, const void* y, int y_f32, const float* w, int rows, int width, int ld, long ldy, float eps,
+                  cudaStream_t s);
+int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps, int f32,
+                 cudaStream_t s);
+int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
+                   const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block, int rows, int q_rank,
+                   int qr, int kv_rank, int lat, float eps, int f32, int* status, cudaStream_t s);
+int fb_softcap(float* y, int rows, int n, long ld, float cap, cudaStream_t s);
+int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaStream_t s);
+int fb_latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
+                   const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat, int nsplit,
+                   float scale, int f32, int* status, cudaStream_t s);
+int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
+                  const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen, const int* block_table,
+                  int max_blocks, int kv_block, int rows, int row_base, int heads, int lat, int nsplit, float scale, int* status,
+                  cudaStream_t s);
+int fb_gemm_f32(float* y, const float* x, const float* w, int M, int N, int K, long ldx, long ldy, int batch, long x_bs, long w_bs,
+                long y_bs, int act, cudaStream_t s);
+
 // ---- drafter_ops.cu ----
 int fb_w4_gemv(void* y, const void* x, const void* qweight, const void* scales, const void* biases, const void* res, int M,
                int N, int K, long ldx, long ldy, cudaStream_t s);

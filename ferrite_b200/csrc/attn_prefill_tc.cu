@@ -74,7 +74,9 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int HD>
+// PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (two TS products per k step, a second
+// P buffer in TMEM), which keeps 16 bits of their mantissa instead of 8.
+template <int HD, bool PX>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
@@ -86,7 +88,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
   constexpr int Q_BYTES = NCH * Q_CH, KV_BYTES = NCH * KV_CH;
-  constexpr uint32_t COL_O = 0, COL_S = HD, COL_P = HD + 2 * FT_BKV;   // TMEM columns: O | S0 S1 | P0 P1
+  constexpr uint32_t COL_O = 0, COL_S = HD, COL_P = HD + 2 * FT_BKV;   // TMEM columns: O | S0 S1 | P0 P1 | remainders
   constexpr uint32_t TMEM_COLS = 512;
   // K runs three tiles ahead at head_dim 256 (S(j+1) is issued a whole tile before PV(j), so with two K buffers a K
   // load had one tile period to arrive and its latency set the pace), four below; V two / three.
@@ -230,6 +232,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int kk = 0; kk < FT_BKV / 16; ++kk)
           tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + s * (FT_BKV / 2) + kk * 8,
                         umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
+        if (PX) {
+#pragma unroll
+          for (int kk = 0; kk < FT_BKV / 16; ++kk)
+            tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + FT_BKV + s * (FT_BKV / 2) + kk * 8,
+                          umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, 1u);
+        }
         tc_commit(&v_empty[st]);
         tc_commit(&p_empty[s]);
       }
@@ -308,7 +316,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         m_ref = m_new;
       }
       const float mr = (m_ref == -INFINITY) ? 0.f : m_ref;
-      uint32_t pr[HC / 2];
+      uint32_t pr[HC / 2], px[PX ? HC / 2 : 1];
       float sum = 0.f;
 #pragma unroll
       for (int c = 0; c < HC / 2; ++c) {
@@ -317,9 +325,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         sum += p0 + p1;
         __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);     // .x (low half) = even key
         pr[c] = *reinterpret_cast<uint32_t*>(&h);
+        if constexpr (PX) px[c] = pack_bf2(p0 - bf_lo(pr[c]), p1 - bf_hi(pr[c]));
       }
       l += sum;
       tmem_st16(tmem + lane_addr + COL_P + s * (FT_BKV / 2) + half * (HC / 2), pr);
+      if constexpr (PX) tmem_st16(tmem + lane_addr + COL_P + FT_BKV + s * (FT_BKV / 2) + half * (HC / 2), px);
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(&p_full[s]);
@@ -378,34 +388,41 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 using namespace fb;
 
-// q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block][nkv*hd] bf16; same outputs as
+// q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block] rows of nkv*hd bf16, kv_stride elements
+// apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; same outputs as
 // fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
 extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                                   long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                                   const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg,
                                   int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int gated,
-                                  int* status, cudaStream_t s) {
+                                  float scale, int exact_p, long kv_stride, int* status, cudaStream_t s) {
   if (nseg <= 0 || max_rows <= 0) return 0;
   if (nq % nkv) return -1;
   if ((hd != 64 && hd != 128 && hd != 256) || kv_block % FT_BKV) return -20;
+  if (kv_stride == 0) kv_stride = (long)nkv * hd;
+  if (kv_stride % 8) return -20;
   CUtensorMap tmQ, tmK, tmV;
   int rc;
   if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, FT_BQ))) return rc;
-  if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)nkv * hd, FT_BKV))) return rc;
-  if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)nkv * hd, FT_BKV))) return rc;
+  if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
+  if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   dim3 grid((max_rows + FT_BQ - 1) / FT_BQ, nq, nseg);
-  const float scale_log2 = 1.4426950408889634f / sqrtf((float)hd);
-#define FB_FT(HDV)                                                                                                 \
+  const float scale_log2 = 1.4426950408889634f * (scale > 0.f ? scale : 1.f / sqrtf((float)hd));
+#define FB_FT(HDV, PXV)                                                                                                 \
   {                                                                                                                \
     const size_t smem = (size_t)(FT_BQ + ((HDV == 256 ? 3 : 4) + (HDV == 256 ? 2 : 3)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
-    auto kern = attn_prefill_tc_kernel<HDV>;                                                                       \
+    auto kern = attn_prefill_tc_kernel<HDV, PXV>;                                                                       \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
     if (e != cudaSuccess) return (int)e;                                                                           \
     launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
                gated, scale_log2, status);                                                                         \
   }
-  if (hd == 256) FB_FT(256) else if (hd == 128) FB_FT(128) else FB_FT(64)
+  if (exact_p) {
+    if (hd == 256) FB_FT(256, true) else if (hd == 128) FB_FT(128, true) else FB_FT(64, true)
+  } else {
+    if (hd == 256) FB_FT(256, false) else if (hd == 128) FB_FT(128, false) else FB_FT(64, false)
+  }
 #undef FB_FT
   return (int)cudaGetLastError();
 }

@@ -552,6 +552,95 @@ void mla_qpad(Tensor qp, Tensor q, Tensor qabs, int64_t nq, int64_t dn, int64_t 
                     (int)L, (int)R, (int)qp.size(-1), (float)scale, cur_stream()), "mla_qpad");
 }
 
+// ---- models of listed layers (latent.cu). The element type of activations and cache (bf16 / fp32) is read off the tensors.
+void* optr(const c10::optional<Tensor>& t) { return t.has_value() ? t->data_ptr() : nullptr; }
+int is_f32(const Tensor& t) {
+  TORCH_CHECK(t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16, "bf16 or fp32 expected");
+  return t.scalar_type() == torch::kFloat32 ? 1 : 0;
+}
+
+void embed_grams(Tensor x, c10::optional<Tensor> xb, Tensor table, c10::optional<Tensor> grams, Tensor tok, Tensor slot, Tensor pos,
+                 Tensor block_table, int64_t kv_block, c10::optional<Tensor> tok_pages, double scale, int64_t buckets,
+                 int64_t mul_prev, int64_t mul_cur, Tensor status) {
+  TORCH_CHECK(x.is_contiguous() && table.is_contiguous() && x.size(1) == table.size(1), "embed_grams: layouts");
+  TORCH_CHECK(!grams || (grams->is_contiguous() && grams->size(0) == buckets + 1 && grams->size(1) == x.size(1) && tok_pages),
+              "embed_grams: bigram table");
+  check(fb_embed_grams(x.data_ptr<float>(), optr(xb), table.data_ptr(), cptr(grams), tok.data_ptr<int>(), slot.data_ptr<int>(),
+                       pos.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block,
+                       (int*)optr(tok_pages), (int)x.size(0), (int)x.size(1), (int)table.size(0), (float)scale, (long)buckets,
+                       (long)mul_prev, (long)mul_cur, is_f32(table), status.data_ptr<int>(), cur_stream()), "embed_grams");
+}
+
+void add_normed(Tensor x, c10::optional<Tensor> xb, Tensor y, Tensor w, int64_t width, double eps) {
+  TORCH_CHECK(x.is_contiguous() && y.stride(1) == 1 && y.size(1) == x.size(1) && w.numel() == x.size(1), "add_normed: layouts");
+  check(fb_add_normed(x.data_ptr<float>(), optr(xb), y.data_ptr(), is_f32(y), w.data_ptr<float>(), (int)x.size(0), (int)width,
+                      (int)x.size(1), (long)y.stride(0), (float)eps, cur_stream()), "add_normed");
+}
+
+void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, int64_t width, double eps) {
+  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && out.size(1) == x.size(1) && w.numel() == x.size(1), "norm_rows: layouts");
+  check(fb_norm_rows(out.data_ptr(), x.data_ptr<float>(), (const int*)cptr(idx), w.data_ptr<float>(), (int)out.size(0), (int)width,
+                     (int)x.size(1), (float)eps, is_f32(out), cur_stream()), "norm_rows");
+}
+
+void latent_prep(Tensor cq, Tensor cache, Tensor proj, Tensor q_norm, c10::optional<Tensor> kv_norm, Tensor row_slot, Tensor row_pos,
+                 Tensor block_table, int64_t kv_block, int64_t q_rank, int64_t kv_rank, double eps, Tensor status) {
+  const int qr = (int)cq.size(1), lat = (int)cache.size(-1);
+  TORCH_CHECK(proj.scalar_type() == torch::kFloat32 && proj.stride(1) == 1 && cq.is_contiguous() && cache.is_contiguous() &&
+              proj.size(1) == qr + (kv_norm ? lat : 0) && cq.scalar_type() == cache.scalar_type(), "latent_prep: layouts");
+  check(fb_latent_prep(cq.data_ptr(), cache.data_ptr(), proj.data_ptr<float>(), (long)proj.stride(0), q_norm.data_ptr<float>(),
+                       (const float*)cptr(kv_norm), row_slot.data_ptr<int>(), row_pos.data_ptr<int>(), block_table.data_ptr<int>(),
+                       (int)block_table.size(1), (int)kv_block, (int)proj.size(0), (int)q_rank, qr, (int)kv_rank, lat, (float)eps,
+                       is_f32(cq), status.data_ptr<int>(), cur_stream()), "latent_prep");
+}
+
+void softcap(Tensor y, double cap) {
+  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.scalar_type() == torch::kFloat32, "softcap: fp32 rows");
+  check(fb_softcap(y.data_ptr<float>(), (int)y.size(0), (int)y.size(1), (long)y.stride(0), (float)cap, cur_stream()), "softcap");
+}
+
+void relu2(Tensor y, Tensor x) {
+  TORCH_CHECK(y.is_contiguous() && x.stride(1) == 1 && y.sizes() == x.sizes(), "relu2: layouts");
+  check(fb_relu2(y.data_ptr(), x.data_ptr(), (long)x.stride(0), (int)x.size(0), (int)x.size(1), cur_stream()), "relu2");
+}
+
+void latent_attn(Tensor out, c10::optional<Tensor> o_part, c10::optional<Tensor> ml_part, Tensor q, Tensor cache, Tensor row_slot,
+                 Tensor row_kvlen, Tensor block_table, int64_t kv_block, int64_t nsplit, double scale, Tensor status) {
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && cache.is_contiguous() && cache.size(-1) == q.size(2) &&
+              (nsplit == 1 || (o_part && ml_part)), "latent_attn: layouts");
+  check(fb_latent_attn(out.data_ptr(), (float*)optr(o_part), (float*)optr(ml_part), q.data_ptr(), cache.data_ptr(),
+                       row_slot.data_ptr<int>(), row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
+                       (int)kv_block, (int)q.size(0), (int)q.size(1), (int)q.size(2), (int)nsplit, (float)scale, is_f32(q),
+                       status.data_ptr<int>(), cur_stream()), "latent_attn");
+}
+
+int64_t latent_mma(Tensor out, c10::optional<Tensor> o_part, c10::optional<Tensor> ml_part, Tensor q, Tensor cache, Tensor seg_slot,
+                   Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, Tensor row_kvlen, Tensor block_table, int64_t kv_block,
+                   int64_t row_base, int64_t nsplit, double scale, Tensor status) {
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && cache.is_contiguous() && cache.size(-1) == q.size(2) &&
+              !is_f32(q) && (nsplit == 1 || (o_part && ml_part)), "latent_mma: layouts");
+  const int rc = fb_latent_mma(out.data_ptr(), (float*)optr(o_part), (float*)optr(ml_part), q.data_ptr(), cache.data_ptr(),
+                               seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), (int)seg_slot.numel(),
+                               (int)max_rows, row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
+                               (int)kv_block, (int)q.size(0), (int)row_base, (int)q.size(1), (int)q.size(2), (int)nsplit,
+                               (float)scale, status.data_ptr<int>(), cur_stream());
+  if (rc == -20) return rc;                     // shape outside this kernel: the caller takes the CUDA-core kernel
+  check(rc, "latent_mma");
+  return 0;
+}
+
+// y [M, N] = act(x [M, K] w [N, K]^T), or per head: x [M, H, K] (unit inner stride), w [H, N, K], y [M, H, N]
+void gemm_f32(Tensor y, Tensor x, Tensor w, int64_t act) {
+  TORCH_CHECK(is_f32(y) && is_f32(x) && is_f32(w) && w.is_contiguous() && x.dim() == w.dim() && y.dim() == w.dim(), "gemm_f32: fp32");
+  const int d = (int)w.dim();
+  TORCH_CHECK((d == 2 || d == 3) && x.stride(d - 1) == 1 && y.stride(d - 1) == 1 && x.size(d - 1) == w.size(d - 1) &&
+              y.size(d - 1) == w.size(d - 2) && x.size(0) == y.size(0), "gemm_f32: shapes");
+  const int batch = d == 3 ? (int)w.size(0) : 1;
+  check(fb_gemm_f32(y.data_ptr<float>(), x.data_ptr<float>(), w.data_ptr<float>(), (int)x.size(0), (int)w.size(d - 2),
+                    (int)w.size(d - 1), (long)x.stride(0), (long)y.stride(0), batch, d == 3 ? (long)x.stride(1) : 0,
+                    d == 3 ? (long)w.stride(0) : 0, d == 3 ? (long)y.stride(1) : 0, (int)act, cur_stream()), "gemm_f32");
+}
+
 void w4_gemv(Tensor y, Tensor x, Tensor qweight, Tensor scales, Tensor biases, c10::optional<Tensor> res) {
   check(fb_w4_gemv(y.data_ptr(), x.data_ptr(), qweight.data_ptr(), scales.data_ptr(), biases.data_ptr(), cptr(res),
                    (int)x.size(0), (int)qweight.size(0), (int)x.size(1), (long)x.stride(0), (long)y.stride(0), cur_stream()),
@@ -623,6 +712,15 @@ void register_ext(pybind11::module_& m) {
   m.def("draft_select", &draft_select);
   m.def("mla_prep", &mla_prep);
   m.def("mla_attn", &mla_attn);
+  m.def("embed_grams", &embed_grams);
+  m.def("add_normed", &add_normed);
+  m.def("norm_rows", &norm_rows);
+  m.def("latent_prep", &latent_prep);
+  m.def("softcap", &softcap);
+  m.def("relu2", &relu2);
+  m.def("latent_attn", &latent_attn);
+  m.def("latent_mma", &latent_mma);
+  m.def("gemm_f32", &gemm_f32);
   m.def("exl3_had", &exl3_had);
   m.def("exl3_gemv", &exl3_gemv);
   m.def("exl3_decode", &exl3_decode);

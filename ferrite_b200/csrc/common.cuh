@@ -45,6 +45,13 @@ __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + __ex
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
 
+// activation a linear's epilogue may apply to its fp32 sums
+enum EpilogueAct : int { ACT_NONE = 0, ACT_RELU2 = 1 };
+__device__ __forceinline__ float epilogue_act(float v, int act) {
+  if (act == ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+  return v;
+}
+
 // unpack two bf16 held in one 32-bit word (low half = element 0)
 __device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }

@@ -74,6 +74,7 @@ struct GemmArgs {
   int fp8;
   const float* scale_m;     // [M]
   const float* scale_n;     // [N] (SwiGLU: [2N], gate features then up features)
+  int act;                  // epilogue activation of the plain (not dual) form
   int out_f32;              // Y is fp32 [M][ldy] instead of bf16 (router logits, lm_head rows)
   void* Y;
   const __nv_bfloat16* res;
@@ -536,7 +537,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 x *= a.scale_n[n + j];
                 if (a.dual) u *= a.scale_n[a.N + n + j];
               }
-              v[j] = a.dual ? siluf_(x) * u : x;
+              v[j] = a.dual ? siluf_(x) * u : epilogue_act(x, a.act);
             }
             if (n + 32 <= a.N) {
               if (a.res) {
@@ -591,6 +592,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                   const float sc = (a.scale_m ? a.scale_m[m] : 1.f);
                   float x = __uint_as_float(r0[j]) * sc * (a.scale_n ? a.scale_n[n] : 1.f);
                   if (a.dual) x = siluf_(x) * (__uint_as_float(r1[j]) * sc * (a.scale_n ? a.scale_n[a.N + n] : 1.f));
+                  else x = epilogue_act(x, a.act);
                   if (a.res) x += bf2f(a.res[(size_t)m * a.ldy + n]);
                   if (a.out_f32) reinterpret_cast<float*>(a.Y)[(size_t)m * a.ldy + n] = x;
                   else Yb[(size_t)m * a.ldy + n] = f2bf(x);
@@ -637,7 +639,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 const float sc = (a.scale_m ? a.scale_m[m] : 1.f);
                 g *= sc * (a.scale_n ? a.scale_n[n] : 1.f);
                 if (a.dual) u *= sc * (a.scale_n ? a.scale_n[a.N + n] : 1.f);
-                float x = a.dual ? siluf_(g) * u : g;
+                float x = a.dual ? siluf_(g) * u : epilogue_act(g, a.act);
                 if (a.res) x += bf2f(a.res[(size_t)m * a.ldy + n]);
                 if (a.out_f32) reinterpret_cast<float*>(a.Y)[(size_t)m * a.ldy + n] = x;
                 else Yb[(size_t)m * a.ldy + n] = f2bf(x);
@@ -736,7 +738,7 @@ struct GemmPlan { GemmArgs a; int grid; size_t smem; };
 
 static int plan_gemm(GemmPlan& p, int M, int N, int K, int mode, int split_k, int sm_count, int fp8 = 0) {
   GemmArgs& a = p.a;
-  a.fp8 = fp8; a.scale_m = nullptr; a.scale_n = nullptr; a.out_f32 = 0;
+  a.fp8 = fp8; a.scale_m = nullptr; a.scale_n = nullptr; a.out_f32 = 0; a.act = ACT_NONE;
   a.M = M; a.N = N; a.K = K;
   a.dual = mode == 1;
   a.swap = M <= 64;

@@ -31,7 +31,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, (M <= 2 ? 4 : (M <= 4 ? 3 : 2)))
         for (int r = 0; r < R; ++r) {
           int nn = n + r;
           if (nn >= row_end) break;
-          float v = acc[r][m];
+          float v = epilogue_act(acc[r][m], a.act);
           if (a.res) v += bf2f(a.res[(size_t)m * a.ldy + nn]);
           if (a.out_f32) reinterpret_cast<float*>(a.Y)[(size_t)m * a.ldy + nn] = v;
           else reinterpret_cast<__nv_bfloat16*>(a.Y)[(size_t)m * a.ldy + nn] = f2bf(v);
@@ -76,7 +76,7 @@ static int launch_gemv(GemvArgs a, int sm_count, cudaStream_t s) {
 
 using namespace fb;
 
-// mode: 0 = plain (optional residual), 1 = SwiGLU (W has 2N rows: gate rows then up rows)
+// mode: 0 = plain (optional residual), 1 = SwiGLU (W has 2N rows: gate rows then up rows), 2 = squared relu
 extern "C" int fb_gemv_bf16(void* Y, const void* X, const void* W, const void* norm_w, const void* res, int M, int N,
                             int K, long ldx, long ldy, float eps, int centred, int out_f32, int mode, int sm_count,
                             cudaStream_t s) {
@@ -86,6 +86,7 @@ extern "C" int fb_gemv_bf16(void* Y, const void* X, const void* W, const void* n
   a.X = (const __nv_bfloat16*)X; a.W = (const __nv_bfloat16*)W; a.norm_w = (const __nv_bfloat16*)norm_w;
   a.res = (const __nv_bfloat16*)res; a.Y = Y; a.M = M; a.N = N; a.K = K; a.ldx = ldx; a.ldy = ldy; a.eps = eps;
   a.centred = centred; a.out_f32 = out_f32; a.rows_per_cta = 0; a.kc = 0;
+  a.act = mode == 2 ? ACT_RELU2 : ACT_NONE;
   if (sm_count <= 0) sm_count = 148;
   if (mode == 1) {
     if (M == 1) return launch_gemv<1, 2, true>(a, sm_count, s);

@@ -32,6 +32,7 @@ struct GemvArgs {
   int out_f32;
   int rows_per_cta;
   int kc;                       // staged chunk length (multiple of GEMV_STEP)
+  int act = ACT_NONE;           // applied to the plain (not SwiGLU) sums before the residual
 };
 
 __host__ __device__ inline int gemv_chunk_len(int M, int K) {

@@ -29,6 +29,7 @@ struct GemvMmaArgs {
   long ldx, ldy;
   float eps;
   int out_f32;
+  int act;                        // epilogue activation of the plain form
   // split-K over blockIdx.y: partial tiles (and partial sums of squares) go to `ws`, the last CTA of a tile to arrive
   // adds them up in split order (deterministic) and runs the epilogue; counters clean themselves
   int split, klen;                // klen = k values per split (multiple of 32)
@@ -252,7 +253,7 @@ __global__ void __launch_bounds__(GM2_WARPS * 32, 2) gemv_mma_kernel(GemvMmaArgs
       gsum *= rs;
       usum *= rs;
     }
-    float v = DUAL ? siluf_(gsum) * usum : gsum;
+    float v = DUAL ? siluf_(gsum) * usum : epilogue_act(gsum, a.act);
     if (a.res) v += bf2f(a.res[(size_t)m * a.ldy + n]);
     if (a.out_f32) reinterpret_cast<float*>(a.y)[(size_t)m * a.ldy + n] = v;
     else reinterpret_cast<__nv_bfloat16*>(a.y)[(size_t)m * a.ldy + n] = f2bf(v);
@@ -315,7 +316,7 @@ static int pick_rt(const GemvMmaArgs& a, int sm_count, float* ws, long ws_floats
 
 using namespace fb;
 
-// mode 1: SwiGLU (W = [gate rows | up rows], 2N rows). M <= 32, K % 32 == 0, ldx % 8 == 0.
+// mode 1: SwiGLU (W = [gate rows | up rows], 2N rows), mode 2: squared relu. M <= 32, K % 32 == 0, ldx % 8 == 0.
 extern "C" int fb_gemv_mma(void* y, const void* x, const void* w, const void* norm_w, const void* res, int M, int N, int K,
                            long ldx, long ldy, float eps, int mode, int out_f32, float* ws, long ws_floats, int* counters,
                            int n_counters, int sm_count, cudaStream_t s) {
@@ -325,6 +326,7 @@ extern "C" int fb_gemv_mma(void* y, const void* x, const void* w, const void* no
   GemvMmaArgs a;
   a.y = y; a.x = (const __nv_bfloat16*)x; a.w = (const __nv_bfloat16*)w; a.norm_w = (const __nv_bfloat16*)norm_w;
   a.res = (const __nv_bfloat16*)res; a.M = M; a.N = N; a.K = K; a.ldx = ldx; a.ldy = ldy; a.eps = eps; a.out_f32 = out_f32;
+  a.act = mode == 2 ? ACT_RELU2 : ACT_NONE;
   a.split = 1; a.klen = K; a.ws = nullptr; a.counters = nullptr;
   const int mt = (M + 7) / 8;
 #define FB_G2(MTT, D) return pick_rt<MTT, D>(a, sm_count, ws, ws_floats, counters, n_counters, s)

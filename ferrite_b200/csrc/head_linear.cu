@@ -23,7 +23,8 @@ __global__ void __launch_bounds__(256, 2) head_linear_kernel(__nv_bfloat16* __re
   const int h = blockIdx.y, t0 = blockIdx.z * ROWS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int chunks = K / 8;
-  const int lpo = chunks < 32 ? chunks : 32;          // lanes per output: a power of two
+  int lpo = 1;                                        // lanes per output: the power of two that covers the chunks, at most 32
+  while (lpo < 32 && lpo < chunks) lpo <<= 1;
   const int per_pass = 32 / lpo;                      // outputs a warp covers in one pass
   const int passes = (HL_OUT / 8) / per_pass > 0 ? (HL_OUT / 8) / per_pass : 1;
   const int sub = lane / lpo, l = lane % lpo;
@@ -38,7 +39,7 @@ __global__ void __launch_bounds__(256, 2) head_linear_kernel(__nv_bfloat16* __re
       const bool ok = live(p0 + u);
 #pragma unroll
       for (int c = 0; c < CPL; ++c)
-        raw[u][c] = ok ? ldg_stream(reinterpret_cast<const uint4*>(Wh + (size_t)out_of(p0 + u) * K) + l + c * lpo)
+        raw[u][c] = ok && l + c * lpo < chunks ? ldg_stream(reinterpret_cast<const uint4*>(Wh + (size_t)out_of(p0 + u) * K) + l + c * lpo)
                        : make_uint4(0, 0, 0, 0);
     }
   };
@@ -52,7 +53,7 @@ __global__ void __launch_bounds__(256, 2) head_linear_kernel(__nv_bfloat16* __re
   for (int r = 0; r < ROWS; ++r) {
 #pragma unroll
     for (int c = 0; c < CPL; ++c) {
-      const uint4 v = t0 + r < T ? *reinterpret_cast<const uint4*>(x + (size_t)(t0 + r) * x_rs + (size_t)h * x_hs + (l + c * lpo) * 8)
+      const uint4 v = t0 + r < T && l + c * lpo < chunks ? *reinterpret_cast<const uint4*>(x + (size_t)(t0 + r) * x_rs + (size_t)h * x_hs + (l + c * lpo) * 8)
                                  : make_uint4(0, 0, 0, 0);
       if constexpr (XF) {
         const uint32_t v4[4] = {v.x, v.y, v.z, v.w};
@@ -112,11 +113,11 @@ using namespace fb;
 extern "C" int fb_head_linear(void* y, const void* x, const void* W, int T, int heads, int N, int K, long x_rs, long x_hs,
                               long y_rs, long y_hs, cudaStream_t s) {
   if (T <= 0 || heads <= 0) return 0;
-  if (K < 8 || K > HL_MAX_K || (K & (K - 1)) || x_rs % 8 || x_hs % 8 || heads > 65535) return -1;
+  if (K < 8 || K > HL_MAX_K || K % 8 || x_rs % 8 || x_hs % 8 || heads > 65535) return -1;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) return -1;
   const int rows = T >= 8 ? 8 : T > 2 ? 4 : T;        // rows per tile: 1, 2, 4 or 8
   dim3 grid((N + HL_OUT - 1) / HL_OUT, heads, (T + rows - 1) / rows);
-  const int chunks = K / 8, cpl = chunks <= 32 ? 1 : chunks / 32;
+  const int chunks = K / 8, cpl = chunks <= 32 ? 1 : chunks <= 64 ? 2 : 4;
 #define FB_HL(C, R)                                                                                                      \
   head_linear_kernel<C, R, (C == 1 ? (R == 8 ? 2 : 4) : C == 2 ? (R == 8 ? 1 : 2) : 1)><<<grid, 256, 0, s>>>(                \
       (__nv_bfloat16*)y, (const __nv_bfloat16*)x, (const __nv_bfloat16*)W, T, N, K, x_rs, x_hs, y_rs, y_hs)

@@ -1,0 +1,714 @@
+// Kernels of the models whose layers are listed one by one: latent attention without positions, RMSNorm on the sublayers'
+// outputs over a 32-bit residual stream, a hashed bigram embedding, softcapped logits.
+//
+//   embed_grams    x = table[token] * scale + grams[(prev * mul_prev + token * mul_cur) mod buckets] in 32 bits. The token of
+//                  every cached position is kept in an int32 page next to the KV pages, so the token before a segment comes
+//                  out of the cache: it moves with the pages (parking, forks, resumed prefixes, rejected drafts) for free.
+//   latent_prep    both latents of a token from one fused projection: RMSNorm of the query latent, RMSNorm of the key / value
+//                  latent into its page
+//   latent_attn    few rows: every head attends the cached latents themselves (key projection folded into the query)
+//   add_normed     x += rms(y) * w on the 32-bit residual stream, plus the copy the next GEMM reads
+//   norm_rows      rms(x[idx]) * w for the rows whose logits are wanted
+//   softcap        logits <- cap * tanh(logits / cap)
+//   gemm_f32       y = x W^T in 32 bits on the CUDA cores, optionally one product per head
+//
+// The row kernels are templates over the element type of activations and cache (bf16, or fp32 for full-precision runs).
+#include "api_ext.h"
+#include "common.cuh"
+
+namespace fb {
+
+template <typename T> struct Elem;
+template <> struct Elem<float> {
+  static __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+  static __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+  static __device__ __forceinline__ float from(float v) { return v; }
+};
+template <> struct Elem<__nv_bfloat16> {
+  static __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf_lo(u.x), bf_hi(u.x), bf_lo(u.y), bf_hi(u.y));
+  }
+  static __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
+  }
+  static __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
+    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(bf_lo(u), bf_hi(u));
+  }
+  static __device__ __forceinline__ __nv_bfloat16 from(float v) { return f2bf(v); }
+};
+
+// ---- embedding -----------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) embed_grams_kernel(float* __restrict__ x, T* __restrict__ xb, const T* __restrict__ table,
+                                                          const T* __restrict__ grams, const int* __restrict__ tok,
+                                                          const int* __restrict__ slot, const int* __restrict__ pos,
+                                                          const int* __restrict__ block_table, int max_blocks, int kv_block,
+                                                          int* tok_pages, int width, int vocab, float scale,
+                                                          unsigned long long buckets, unsigned long long mul_prev,
+                                                          unsigned long long mul_cur, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x;
+  int id = tok[row];
+  if (id < 0 || id >= vocab) { if (threadIdx.x == 0) set_status(status, ST_BOUNDS); id = 0; }
+  const T* gr = nullptr;
+  if (grams) {
+    const int p = pos[row], s = slot[row];
+    const int* bt = block_table + (size_t)s * max_blocks;
+    unsigned long long g = buckets;                       // a sequence's first token has the last row to itself
+    if (p > 0) {
+      int prev;
+      if (row > 0 && slot[row - 1] == s && pos[row - 1] == p - 1) prev = tok[row - 1];
+      else {
+        const int blk = bt[(p - 1) / kv_block];
+        if (blk < 0 && threadIdx.x == 0) set_status(status, ST_BOUNDS);
+        prev = blk < 0 ? 0 : tok_pages[(size_t)blk * kv_block + (p - 1) % kv_block];
+      }
+      g = ((unsigned long long)prev * mul_prev + (unsigned long long)id * mul_cur) % buckets;
+    }
+    gr = grams + (size_t)g * width;
+    if (threadIdx.x == 0) {
+      const int blk = bt[p / kv_block];
+      if (blk < 0) set_status(status, ST_BOUNDS);
+      else tok_pages[(size_t)blk * kv_block + p % kv_block] = id;
+    }
+  }
+  const T* tr = table + (size_t)id * width;
+  for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+    float4 v = Elem<T>::load4(tr + i);
+    v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+    if (gr) {
+      const float4 g = Elem<T>::load4(gr + i);
+      v.x += g.x; v.y += g.y; v.z += g.z; v.w += g.w;
+    }
+    *reinterpret_cast<float4*>(x + (size_t)row * width + i) = v;
+    if (xb) Elem<T>::store4(xb + (size_t)row * width + i, v);
+  }
+}
+
+// ---- row norms -------------------------------------------------------------------------------------------------------
+// Sum of squares of a row of n floats (n % 4 == 0), over the whole CTA.
+template <typename S>
+__device__ __forceinline__ float row_rscale(const S* r, int n, int count, float eps, float* red) {
+  float ss = 0.f;
+  for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+    const float4 v = Elem<S>::load4(r + i);
+    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+  }
+  return 1.f / sqrtf(block_sum(ss, red) / (float)count + eps);
+}
+
+// x[row] += y[row] * rscale * w; xb = x in the GEMM operand type. `width` counts the true columns, `ld` the padded ones
+// (zeros beyond width).
+template <typename T, typename S>
+__global__ void add_normed_kernel(float* __restrict__ x, T* __restrict__ xb, const S* __restrict__ y,
+                                  const float* __restrict__ w, int width, int ld, long ldy, float eps) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const S* yr = y + row * ldy;
+  const float r = row_rscale<S>(yr, ld, width, eps, red);
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    const float4 v = Elem<S>::load4(yr + i), ww = *reinterpret_cast<const float4*>(w + i);
+    float4 a = *reinterpret_cast<const float4*>(x + row * ld + i);
+    a.x += v.x * r * ww.x; a.y += v.y * r * ww.y; a.z += v.z * r * ww.z; a.w += v.w * r * ww.w;
+    *reinterpret_cast<float4*>(x + row * ld + i) = a;
+    if (xb) Elem<T>::store4(xb + row * ld + i, a);
+  }
+}
+
+// out[r] = x[idx ? idx[r] : r] * rscale * w
+template <typename T>
+__global__ void norm_rows_kernel(T* __restrict__ out, const float* __restrict__ x, const int* __restrict__ idx,
+                                 const float* __restrict__ w, int width, int ld, float eps) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * ld;
+  const float r = row_rscale<float>(xr, ld, width, eps, red);
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(xr + i);
+    const float4 ww = *reinterpret_cast<const float4*>(w + i);
+    v.x *= r * ww.x; v.y *= r * ww.y; v.z *= r * ww.z; v.w *= r * ww.w;
+    Elem<T>::store4(out + (size_t)blockIdx.x * ld + i, v);
+  }
+}
+
+// proj row = [query latent (qr columns, q_rank true) | key / value latent (lat columns, kv_rank true)], fp32.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ cq, T* __restrict__ cache, const float* __restrict__ proj,
+                                                          long ldp, const float* __restrict__ q_norm,
+                                                          const float* __restrict__ kv_norm, const int* __restrict__ row_slot,
+                                                          const int* __restrict__ row_pos, const int* __restrict__ block_table,
+                                                          int max_blocks, int kv_block, int q_rank, int qr, int kv_rank, int lat,
+                                                          float eps, int* status) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const float* pr = proj + row * ldp;
+  float r = row_rscale<float>(pr, qr, q_rank, eps, red);
+  for (int i = threadIdx.x * 4; i < qr; i += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(pr + i);
+    const float4 w = *reinterpret_cast<const float4*>(q_norm + i);
+    v.x *= r * w.x; v.y *= r * w.y; v.z *= r * w.z; v.w *= r * w.w;
+    Elem<T>::store4(cq + row * qr + i, v);
+  }
+  if (!kv_norm) return;                                   // the layer reads another layer's latents
+  const int p = row_pos[row];
+  const int blk = block_table[(size_t)row_slot[row] * max_blocks + p / kv_block];
+  if (blk < 0) { if (threadIdx.x == 0) set_status(status, ST_BOUNDS); return; }
+  T* dst = cache + ((size_t)blk * kv_block + p % kv_block) * lat;
+  pr += qr;
+  r = row_rscale<float>(pr, lat, kv_rank, eps, red);
+  for (int i = threadIdx.x * 4; i < lat; i += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(pr + i);
+    const float4 w = *reinterpret_cast<const float4*>(kv_norm + i);
+    v.x *= r * w.x; v.y *= r * w.y; v.z *= r * w.z; v.w *= r * w.w;
+    Elem<T>::store4(dst + i, v);
+  }
+}
+
+__global__ void softcap_kernel(float* __restrict__ y, long ld, int n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  float* r = y + (size_t)blockIdx.y * ld;
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) r[i] = cap * tanhf(r[i] / cap);
+}
+
+// y = relu(x)^2 where the product that made x has no such epilogue (packed weights)
+__global__ void relu2_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ x, long ldx, int n) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float v = fmaxf(bf2f(x[(size_t)blockIdx.y * ldx + i]), 0.f);
+  y[(size_t)blockIdx.y * n + i] = f2bf(v * v);
+}
+
+// ---- attention over the cached latents, CUDA cores ---------------------------------------------------------------------
+// grid (rows, heads, splits), 4 warps striding over the keys with an online softmax; a lane owns columns 64 j + 2 lane, + 1.
+// lat = 64 nl with nl <= NJ. One split writes the normalised output itself, more leave partials for the merge.
+constexpr int LA_WARPS = 4;
+
+template <typename T, int NJ>
+__global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restrict__ out, float* __restrict__ o_part,
+                                                                    float* __restrict__ ml_part, const T* __restrict__ q,
+                                                                    const T* __restrict__ cache, const int* __restrict__ row_slot,
+                                                                    const int* __restrict__ row_kvlen,
+                                                                    const int* __restrict__ block_table, int max_blocks,
+                                                                    int kv_block, int heads, int lat, int nsplit,
+                                                                    float scale_log2, int* status) {
+  extern __shared__ float so[];                            // [warps][lat]
+  __shared__ float sml[LA_WARPS][2];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int nl = lat / 64;
+  const int row = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int kvlen = row_kvlen[row];
+  const int* bt = block_table + (size_t)row_slot[row] * max_blocks;
+  int per = (kvlen + nsplit - 1) / nsplit;
+  per = (per + 31) / 32 * 32;
+  const int lo = split * per, hi = min(kvlen, lo + per);
+  const T* qr = q + ((size_t)row * heads + h) * lat;
+  float2 qf[NJ], o[NJ];
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    o[j] = make_float2(0.f, 0.f);
+    qf[j] = j < nl ? Elem<T>::load2(qr + 64 * j + 2 * lane) : make_float2(0.f, 0.f);
+    qf[j].x *= scale_log2; qf[j].y *= scale_log2;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int t = lo + warp; t < hi; t += LA_WARPS) {
+    const int blk = bt[t / kv_block];
+    if (blk < 0) { if (lane == 0) set_status(status, ST_BOUNDS); break; }
+    const T* kr = cache + ((size_t)blk * kv_block + t % kv_block) * lat + 2 * lane;
+    float2 k[NJ];
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) k[j] = j < nl ? Elem<T>::load2(kr + 64 * j) : make_float2(0.f, 0.f);
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) s = fmaf(qf[j].x, k[j].x, fmaf(qf[j].y, k[j].y, s));
+    s = warp_sum(s);
+    const float mn = fmaxf(m, s);
+    const float a = exp2f(m - mn), p = exp2f(s - mn);
+    l = l * a + p;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) { o[j].x = fmaf(p, k[j].x, o[j].x * a); o[j].y = fmaf(p, k[j].y, o[j].y * a); }
+    m = mn;
+  }
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+    if (j < nl) *reinterpret_cast<float2*>(so + (size_t)warp * lat + 64 * j + 2 * lane) = o[j];
+  if (lane == 0) { sml[warp][0] = m; sml[warp][1] = l; }
+  __syncthreads();
+  float M = -INFINITY, f[LA_WARPS], Ls = 0.f;
+#pragma unroll
+  for (int w = 0; w < LA_WARPS; ++w) M = fmaxf(M, sml[w][0]);
+#pragma unroll
+  for (int w = 0; w < LA_WARPS; ++w) {
+    f[w] = sml[w][0] == -INFINITY ? 0.f : exp2f(sml[w][0] - M);
+    Ls += sml[w][1] * f[w];
+  }
+  const size_t pidx = ((size_t)row * heads + h) * nsplit + split;
+  const float inv = nsplit == 1 ? (Ls > 0.f ? 1.f / Ls : 0.f) : 1.f;
+  for (int d = threadIdx.x; d < lat; d += blockDim.x) {
+    float acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < LA_WARPS; ++w) acc += so[(size_t)w * lat + d] * f[w];
+    if (nsplit == 1) out[((size_t)row * heads + h) * lat + d] = Elem<T>::from(acc * inv);
+    else o_part[pidx * lat + d] = acc;
+  }
+  if (nsplit > 1 && threadIdx.x == 0) { ml_part[pidx * 2] = M; ml_part[pidx * 2 + 1] = Ls; }
+}
+
+// merge of the splits in split order; grid (rows, heads)
+template <typename T>
+__global__ void __launch_bounds__(128) latent_merge_kernel(T* __restrict__ out, const float* __restrict__ o_part,
+                                                           const float* __restrict__ ml_part, int heads, int nsplit, int lat) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t rh = (size_t)blockIdx.x * heads + blockIdx.y, pbase = rh * nsplit;
+  float M = -INFINITY;
+  for (int s = 0; s < nsplit; ++s) M = fmaxf(M, ml_part[(pbase + s) * 2]);
+  float Ls = 0.f;
+  for (int s = 0; s < nsplit; ++s) {
+    const float ms = ml_part[(pbase + s) * 2];
+    if (ms != -INFINITY) Ls += ml_part[(pbase + s) * 2 + 1] * exp2f(ms - M);
+  }
+  const float inv = Ls > 0.f ? 1.f / Ls : 0.f;
+  for (int d = threadIdx.x * 4; d < lat; d += blockDim.x * 4) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < nsplit; ++s) {
+      const float ms = ml_part[(pbase + s) * 2];
+      if (ms == -INFINITY) continue;                       // an empty split wrote no rows
+      const float f = exp2f(ms - M);
+      const float4 v = *reinterpret_cast<const float4*>(o_part + (pbase + s) * lat + d);
+      acc.x = fmaf(v.x, f, acc.x); acc.y = fmaf(v.y, f, acc.y); acc.z = fmaf(v.z, f, acc.z); acc.w = fmaf(v.w, f, acc.w);
+    }
+    acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
+    Elem<T>::store4(out + rh * lat + d, acc);
+  }
+}
+
+// ---- attention over the cached latents, tensor cores ---------------------------------------------------------------------
+// bf16. The M dimension is (row of the segment, head): all of them read the same latents, so one pass over a key tile
+// serves 64 of them. grid (segments x M tiles, splits), 8 warps. Scores: warp = 16 M rows x 32 of the tile's 64 keys over the
+// whole latent. Values are the same shared-memory tile read transposed: warp = all 64 M rows x lat / 8 columns. The softmax
+// weights go through shared memory as a bf16 value plus its bf16 remainder, two products each, so they keep 16 bits of mantissa
+// instead of 8; scores, maxima, exponentials and row sums are 32-bit.
+constexpr int LM_M = 64, LM_KEYS = 64, LM_THREADS = 256, LM_LDP = LM_KEYS + 8;
+
+__device__ __forceinline__ void lm_cp16(void* smem, const void* gmem, bool valid) {
+  const int sz = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem)), "l"(gmem), "r"(sz) : "memory");
+}
+__device__ __forceinline__ void lm_ldsm(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void lm_ldsm_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <int NJ>
+struct Lm {
+  static constexpr int LAT = NJ * 64, LD = LAT + 8;
+  static constexpr size_t SMEM = (size_t)(LM_M + 2 * LM_KEYS) * LD * 2 + (size_t)2 * LM_M * LM_LDP * 2 + 4 * LM_M * 4;
+};
+
+template <int NJ>
+__global__ void __launch_bounds__(LM_THREADS, 1)
+latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, float* __restrict__ ml_part,
+                  const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache, const int* __restrict__ seg_slot,
+                  const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows, const int* __restrict__ row_kvlen,
+                  const int* __restrict__ block_table, int max_blocks, int kv_block, int heads, int row_base, int tiles_per_seg,
+                  int nsplit, float scale_log2, int* status) {
+  constexpr int LAT = Lm<NJ>::LAT, LD = Lm<NJ>::LD, CPR = LAT / 8;
+  extern __shared__ __align__(16) unsigned char lm_smem[];
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [M][LD]
+  __nv_bfloat16* sK = sQ + LM_M * LD;                                      // [2][KEYS][LD]
+  __nv_bfloat16* sP = sK + 2 * LM_KEYS * LD;                               // [value | remainder][M][LDP]
+  float* smx = reinterpret_cast<float*>(sP + 2 * LM_M * LM_LDP);           // [2][M] maxima of the two key halves, then sums
+  float* sfac = smx + 2 * LM_M;                                            // [M] rescale factor of the tile
+  float* sinv = sfac + LM_M;                                               // [M] 1 / row sum
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int seg = blockIdx.x / tiles_per_seg, tile_m = blockIdx.x % tiles_per_seg, split = blockIdx.y;
+  const int n = seg_nrows[seg], m_all = n * heads, m0 = tile_m * LM_M;
+  if (m0 >= m_all) return;
+  const int valid_m = min(LM_M, m_all - m0);
+  const int row0 = seg_row0[seg];
+  const int* bt = block_table + (size_t)seg_slot[seg] * max_blocks;
+  const int kv_end = row_kvlen[row0 + (m0 + valid_m - 1) / heads - row_base];          // rows of a segment see ever more keys
+  int per = (kv_end + nsplit - 1) / nsplit;
+  per = (per + LM_KEYS - 1) / LM_KEYS * LM_KEYS;
+  const int lo = split * per, hi = min(kv_end, lo + per);
+  // (row, head) flat index of an M row in q / out, which start at row row_base of the step
+  const size_t flat0 = (size_t)(row0 - row_base) * heads + m0;
+  if (lo >= hi) {
+    if (nsplit > 1)
+      for (int m = tid; m < valid_m; m += LM_THREADS) {
+        float* ml = ml_part + ((flat0 + m) * nsplit + split) * 2;
+        ml[0] = -INFINITY; ml[1] = 0.f;
+      }
+    return;
+  }
+  for (int c = tid; c < LM_M * CPR; c += LM_THREADS) {
+    const int m = c / CPR, cc = c % CPR;
+    const bool ok = m < valid_m;
+    lm_cp16(sQ + m * LD + cc * 8, q + (flat0 + (ok ? m : 0)) * LAT + cc * 8, ok);
+  }
+  auto load_tile = [&](int t0, int stage) {
+    for (int c = tid; c < LM_KEYS * CPR; c += LM_THREADS) {
+      const int r = c / CPR, cc = c % CPR, t = t0 + r;
+      bool ok = t < hi;
+      const int blk = ok ? bt[t / kv_block] : 0;
+      if (blk < 0) { ok = false; set_status(status, ST_BOUNDS); }
+      lm_cp16(sK + (stage * LM_KEYS + r) * LD + cc * 8,
+              cache + (ok ? ((size_t)blk * kv_block + t % kv_block) * LAT + cc * 8 : 0), ok);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load_tile(lo, 0);
+
+  const int mw = warp & 3, nw = warp >> 2;                   // score role
+  const int r_lo = mw * 16 + lane / 4;                       // this thread's two M rows: r_lo, r_lo + 8
+  int kvl[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int m = r_lo + 8 * h;
+    kvl[h] = m < valid_m ? row_kvlen[row0 + (m0 + m) / heads - row_base] : 0;
+  }
+  float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+  float o[4][NJ][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) { o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f; }
+  const int ntiles = (hi - lo + LM_KEYS - 1) / LM_KEYS;
+  const bool score_on = mw * 16 < valid_m;
+
+  for (int tile = 0; tile < ntiles; ++tile) {
+    const int stage = tile & 1;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                         // the tile has landed; everyone is done with the other buffer
+    if (tile + 1 < ntiles) load_tile(lo + (tile + 1) * LM_KEYS, stage ^ 1);
+    const __nv_bfloat16* K = sK + stage * LM_KEYS * LD;
+    float s[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
+    float mx[2] = {-INFINITY, -INFINITY};
+    if (score_on) {
+#pragma unroll 4
+      for (int ks = 0; ks < LAT / 16; ++ks) {
+        uint32_t a[4], b[4];
+        lm_ldsm(a, sQ + (mw * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          lm_ldsm(b, K + (nw * 32 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * LD + ks * 16 + ((lane >> 3) & 1) * 8);
+          lm_mma(s[np * 2], a, b[0], b[1]);
+          lm_mma(s[np * 2 + 1], a, b[2], b[3]);
+        }
+      }
+      const int kbase = lo + tile * LM_KEYS + nw * 32 + (lane & 3) * 2;
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = kbase + nt * 8 + (e & 1), h = e >> 1;
+          const float v = (t < kvl[h] && t < hi) ? s[nt][e] * scale_log2 : -INFINITY;
+          s[nt][e] = v;
+          mx[h] = fmaxf(mx[h], v);
+        }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+        if ((lane & 3) == 0) smx[nw * LM_M + r_lo + 8 * h] = mx[h];
+      }
+    }
+    __syncthreads();
+    if (score_on) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int r = r_lo + 8 * h;
+        const float mn = fmaxf(mrow[h], fmaxf(smx[r], smx[LM_M + r]));
+        const float f = mn == -INFINITY ? 1.f : exp2f(mrow[h] - mn);
+        mrow[h] = mn;
+        float ls = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) {
+          const float p0 = mn == -INFINITY ? 0.f : exp2f(s[nt][2 * h] - mn);
+          const float p1 = mn == -INFINITY ? 0.f : exp2f(s[nt][2 * h + 1] - mn);
+          ls += p0 + p1;
+          const uint32_t v = pack_bf2(p0, p1);
+          const int at = r * LM_LDP + nw * 32 + nt * 8 + (lane & 3) * 2;
+          *reinterpret_cast<uint32_t*>(sP + at) = v;
+          *reinterpret_cast<uint32_t*>(sP + LM_M * LM_LDP + at) = pack_bf2(p0 - bf_lo(v), p1 - bf_hi(v));
+        }
+        lrow[h] = lrow[h] * f + ls;
+        if (nw == 0 && (lane & 3) == 0) sfac[r] = f;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int mt = 0; mt < 4; ++mt) {
+      if (mt * 16 >= valid_m) break;
+      const float f0 = sfac[mt * 16 + lane / 4], f1 = sfac[mt * 16 + lane / 4 + 8];
+      if (!__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) continue;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) { o[mt][j][0] *= f0; o[mt][j][1] *= f0; o[mt][j][2] *= f1; o[mt][j][3] *= f1; }
+    }
+#pragma unroll
+    for (int kp = 0; kp < 2; ++kp) {
+      uint32_t b[NJ][4];                                     // 8 columns x 32 keys each: two k steps
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) lm_ldsm_t(b[j], K + (kp * 32 + lane) * LD + (warp * NJ + j) * 8);
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt) {
+        if (mt * 16 >= valid_m) break;
+#pragma unroll
+        for (int k2 = 0; k2 < 2; ++k2) {
+#pragma unroll
+          for (int part = 0; part < 2; ++part) {
+            uint32_t a[4];
+            lm_ldsm(a, sP + (part * LM_M + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LM_LDP + (kp * 2 + k2) * 16 + (lane >> 4) * 8);
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) lm_mma(o[mt][j], a, b[j][2 * k2], b[j][2 * k2 + 1]);
+          }
+        }
+      }
+    }
+  }
+  __syncthreads();                                           // the maxima buffer takes the row sums now
+  if (score_on) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      lrow[h] += __shfl_xor_sync(0xffffffffu, lrow[h], 1);
+      lrow[h] += __shfl_xor_sync(0xffffffffu, lrow[h], 2);
+      if ((lane & 3) == 0) smx[nw * LM_M + r_lo + 8 * h] = lrow[h];
+    }
+  }
+  __syncthreads();
+  if (score_on && nw == 0 && (lane & 3) == 0) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = r_lo + 8 * h;
+      if (r >= valid_m) continue;
+      const float l = smx[r] + smx[LM_M + r];
+      if (nsplit == 1) sinv[r] = l > 0.f ? 1.f / l : 0.f;
+      else {
+        float* ml = ml_part + ((flat0 + r) * nsplit + split) * 2;
+        ml[0] = mrow[h]; ml[1] = l;
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = mt * 16 + lane / 4 + 8 * h;
+      if (r >= valid_m) continue;
+      const float inv = nsplit == 1 ? sinv[r] : 1.f;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (warp * NJ + j) * 8 + (lane & 3) * 2;
+        if (nsplit == 1)
+          *reinterpret_cast<uint32_t*>(out + (flat0 + r) * LAT + d) = pack_bf2(o[mt][j][2 * h] * inv, o[mt][j][2 * h + 1] * inv);
+        else
+          *reinterpret_cast<float2*>(o_part + ((flat0 + r) * nsplit + split) * LAT + d) = make_float2(o[mt][j][2 * h], o[mt][j][2 * h + 1]);
+      }
+    }
+}
+
+// ---- y = x W^T in 32 bits -----------------------------------------------------------------------------------------------
+// 64 x 64 tile per CTA of 256 threads (4 x 4 outputs each), K in steps of 16; grid.z = batch (one product per head).
+__global__ void __launch_bounds__(256) gemm_f32_kernel(float* __restrict__ y, const float* __restrict__ x,
+                                                       const float* __restrict__ w, int M, int N, int K, long ldx, long ldy,
+                                                       long x_bs, long w_bs, long y_bs, int act) {
+  __shared__ float sx[16][64 + 4], sw[16][64 + 4];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
+  x += (size_t)blockIdx.z * x_bs; w += (size_t)blockIdx.z * w_bs; y += (size_t)blockIdx.z * y_bs;
+  const int lr = tid / 4, lk = (tid % 4) * 4;                // loader: row of the tile, 4 k values
+  const int tx = tid % 16, ty = tid / 16;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+    if (m0 + lr < M && k0 + lk < K) a = *reinterpret_cast<const float4*>(x + (size_t)(m0 + lr) * ldx + k0 + lk);
+    if (n0 + lr < N && k0 + lk < K) b = *reinterpret_cast<const float4*>(w + (size_t)(n0 + lr) * K + k0 + lk);
+    __syncthreads();
+    sx[lk][lr] = a.x; sx[lk + 1][lr] = a.y; sx[lk + 2][lr] = a.z; sx[lk + 3][lr] = a.w;
+    sw[lk][lr] = b.x; sw[lk + 1][lr] = b.y; sw[lk + 2][lr] = b.z; sw[lk + 3][lr] = b.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      const float4 av = *reinterpret_cast<const float4*>(&sx[k][ty * 4]), bv = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+      const float am[4] = {av.x, av.y, av.z, av.w}, bn[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(am[i], bn[j], acc[i][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (m < M && n < N) y[(size_t)m * ldy + n] = epilogue_act(acc[i][j], act);
+    }
+}
+
+}  // namespace fb
+
+using namespace fb;
+using bf16 = __nv_bfloat16;
+
+static int row_threads(int width) { return width >= 4096 ? 512 : width >= 1024 ? 256 : 128; }
+
+extern "C" int fb_embed_grams(float* x, void* xb, const void* table, const void* grams, const int* tok, const int* slot,
+                              const int* pos, const int* block_table, int max_blocks, int kv_block, int* tok_pages, int rows,
+                              int width, int vocab, float scale, long buckets, long mul_prev, long mul_cur, int f32, int* status,
+                              cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (width % 4 || (grams && (buckets <= 0 || !tok_pages))) return -1;
+  if (f32)
+    return (int)launch_pdl(embed_grams_kernel<float>, dim3(rows), dim3(256), 0, s, x, (float*)xb, (const float*)table,
+                           (const float*)grams, tok, slot, pos, block_table, max_blocks, kv_block, tok_pages, width, vocab, scale,
+                           (unsigned long long)buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, status);
+  return (int)launch_pdl(embed_grams_kernel<bf16>, dim3(rows), dim3(256), 0, s, x, (bf16*)xb, (const bf16*)table, (const bf16*)grams,
+                         tok, slot, pos, block_table, max_blocks, kv_block, tok_pages, width, vocab, scale,
+                         (unsigned long long)buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, status);
+}
+
+// y: fp32 (y_f32) or bf16 rows of stride ldy; xb: bf16 copy of x, or null
+extern "C" int fb_add_normed(float* x, void* xb, const void* y, int y_f32, const float* w, int rows, int width, int ld, long ldy,
+                             float eps, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (ld % 4 || ldy % 4) return -1;
+  const dim3 g(rows), b(row_threads(ld));
+  if (y_f32) return (int)launch_pdl(add_normed_kernel<bf16, float>, g, b, 0, s, x, (bf16*)xb, (const float*)y, w, width, ld, ldy, eps);
+  return (int)launch_pdl(add_normed_kernel<bf16, bf16>, g, b, 0, s, x, (bf16*)xb, (const bf16*)y, w, width, ld, ldy, eps);
+}
+
+extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps,
+                            int f32, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (ld % 4) return -1;
+  const dim3 g(rows), b(row_threads(ld));
+  if (f32) return (int)launch_pdl(norm_rows_kernel<float>, g, b, 0, s, (float*)out, x, idx, w, width, ld, eps);
+  return (int)launch_pdl(norm_rows_kernel<bf16>, g, b, 0, s, (bf16*)out, x, idx, w, width, ld, eps);
+}
+
+extern "C" int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
+                              const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block,
+                              int rows, int q_rank, int qr, int kv_rank, int lat, float eps, int f32, int* status, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (qr % 4 || lat % 4 || ldp % 4) return -1;
+  const dim3 g(rows), b(qr + lat >= 512 ? 256 : 128);
+  if (f32)
+    return (int)launch_pdl(latent_prep_kernel<float>, g, b, 0, s, (float*)cq, (float*)cache, proj, ldp, q_norm, kv_norm, row_slot,
+                           row_pos, block_table, max_blocks, kv_block, q_rank, qr, kv_rank, lat, eps, status);
+  return (int)launch_pdl(latent_prep_kernel<bf16>, g, b, 0, s, (bf16*)cq, (bf16*)cache, proj, ldp, q_norm, kv_norm, row_slot, row_pos,
+                         block_table, max_blocks, kv_block, q_rank, qr, kv_rank, lat, eps, status);
+}
+
+extern "C" int fb_softcap(float* y, int rows, int n, long ld, float cap, cudaStream_t s) {
+  if (rows <= 0 || n <= 0) return 0;
+  if (rows > 65535) return -1;
+  return (int)launch_pdl(softcap_kernel, dim3((n + 255) / 256, rows), dim3(256), 0, s, y, ld, n, cap);
+}
+
+extern "C" int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaStream_t s) {
+  if (rows <= 0 || n <= 0) return 0;
+  if (rows > 65535) return -1;
+  relu2_kernel<<<dim3((n + 255) / 256, rows), 256, 0, s>>>((bf16*)y, (const bf16*)x, ldx, n);
+  return (int)cudaGetLastError();
+}
+
+template <typename T>
+static int latent_merge(void* out, const float* o_part, const float* ml_part, int rows, int heads, int nsplit, int lat, cudaStream_t s) {
+  return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128), 0, s, (T*)out, o_part, ml_part, heads, nsplit, lat);
+}
+
+template <typename T>
+static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
+                       const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat,
+                       int nsplit, float scale_log2, int* status, cudaStream_t s) {
+  const dim3 grid(rows, heads, nsplit);
+  const size_t smem = (size_t)LA_WARPS * lat * 4;
+  auto go = [&](auto kern) {
+    return (int)launch_pdl(kern, grid, dim3(LA_WARPS * 32), smem, s, (T*)out, o_part, ml_part, (const T*)q, (const T*)cache, row_slot,
+                           row_kvlen, block_table, max_blocks, kv_block, heads, lat, nsplit, scale_log2, status);
+  };
+  int rc;
+  if (lat <= 128) rc = go(latent_attn_kernel<T, 2>);
+  else if (lat <= 256) rc = go(latent_attn_kernel<T, 4>);
+  else if (lat <= 512) rc = go(latent_attn_kernel<T, 8>);
+  else rc = go(latent_attn_kernel<T, 16>);
+  if (rc || nsplit == 1) return rc;
+  return latent_merge<T>(out, o_part, ml_part, rows, heads, nsplit, lat, s);
+}
+
+// out [rows][heads][lat]; partials (nsplit > 1): o_part rows * heads * nsplit * lat floats, ml_part two per record
+extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
+                              const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat,
+                              int nsplit, float scale, int f32, int* status, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 65535) return -1;
+  const float sl = scale * 1.4426950408889634f;
+  return f32 ? latent_attn<float>(out, o_part, ml_part, q, cache, row_slot, row_kvlen, block_table, max_blocks, kv_block, rows, heads,
+                                  lat, nsplit, sl, status, s)
+             : latent_attn<bf16>(out, o_part, ml_part, q, cache, row_slot, row_kvlen, block_table, max_blocks, kv_block, rows, heads,
+                                 lat, nsplit, sl, status, s);
+}
+
+// The same on tensor cores for bf16 and lat <= 512 (-20 otherwise). Rows come in segments (consecutive rows of one slot);
+// seg_row0 counts the rows of the step, of which q / out / row_kvlen hold those from row_base on.
+extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
+                             const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen,
+                             const int* block_table, int max_blocks, int kv_block, int rows, int row_base, int heads, int lat,
+                             int nsplit, float scale, int* status, cudaStream_t s) {
+  if (rows <= 0 || nseg <= 0) return 0;
+  if (lat % 64 || lat > 512) return -20;
+  if (nsplit < 1 || nsplit > 65535) return -1;
+  const int tps = (max_rows * heads + LM_M - 1) / LM_M;
+  const dim3 grid(nseg * tps, nsplit);
+  const float sl = scale * 1.4426950408889634f;
+  int rc = 0;
+#define FB_LM(NJ)                                                                                                              \
+  case NJ: {                                                                                                                   \
+    auto kern = latent_mma_kernel<NJ>;                                                                                         \
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Lm<NJ>::SMEM);                \
+    if (e != cudaSuccess) return (int)e;                                                                                       \
+    rc = (int)launch_pdl(kern, grid, dim3(LM_THREADS), Lm<NJ>::SMEM, s, (bf16*)out, o_part, ml_part, (const bf16*)q,           \
+                         (const bf16*)cache, seg_slot, seg_row0, seg_nrows, row_kvlen, block_table, max_blocks, kv_block, heads, \
+                         row_base, tps, nsplit, sl, status);                                                                   \
+    break;                                                                                                                     \
+  }
+  switch (lat / 64) { FB_LM(1) FB_LM(2) FB_LM(3) FB_LM(4) FB_LM(5) FB_LM(6) FB_LM(7) FB_LM(8) }
+#undef FB_LM
+  if (rc || nsplit == 1) return rc;
+  return latent_merge<bf16>(out, o_part, ml_part, rows, heads, nsplit, lat, s);
+}
+
+// y [batch][M][N] = act(x [batch][M][K] w [batch][N][K]^T); row strides ldx / ldy, batch strides x_bs / w_bs / y_bs (elements)
+extern "C" int fb_gemm_f32(float* y, const float* x, const float* w, int M, int N, int K, long ldx, long ldy, int batch, long x_bs,
+                           long w_bs, long y_bs, int act, cudaStream_t s) {
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
+  if (K % 4 || ldx % 4 || x_bs % 4 || w_bs % 4 || batch > 65535 || (M + 63) / 64 > 65535) return -1;
+  gemm_f32_kernel<<<dim3((N + 63) / 64, (M + 63) / 64, batch), 256, 0, s>>>(y, x, w, M, N, K, ldx, ldy, x_bs, w_bs, y_bs, act);
+  return (int)cudaGetLastError();
+}

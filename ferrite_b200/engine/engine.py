@@ -11,7 +11,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..config import EngineConfig, ModelConfig
-from ..models.weights import Weights, init_weights, shard_weights
+from ..models.weights import Weights, init_weights, pack_latent, shard_weights
 from .executor import Executor, Segment, StepBatch
 
 
@@ -40,7 +40,13 @@ class Engine:
             device = "cuda" if torch.cuda.is_available() else "cpu"
         self.device = torch.device(device)
         on_gpu = self.device.type == "cuda"
-        self.dtype = torch.bfloat16 if on_gpu else torch.float32
+        if self.ecfg.compute_dtype not in ("bf16", "fp32"):
+            raise ValueError(f"compute_dtype {self.ecfg.compute_dtype!r}: expected bf16 or fp32")
+        if self.ecfg.compute_dtype == "fp32" and on_gpu and (not cfg.layers or self.ecfg.weight_dtype != "bf16"):
+            raise ValueError("compute_dtype fp32 on a GPU: models of listed layers with unpacked weights only")
+        if cfg.layers and self.ecfg.kv_dtype != "bf16":
+            raise ValueError(f"kv_dtype {self.ecfg.kv_dtype!r}: latent caches are kept in the compute dtype")
+        self.dtype = torch.bfloat16 if on_gpu and self.ecfg.compute_dtype == "bf16" else torch.float32
         world = tp.world if tp is not None else 1
         rank = tp.rank if tp is not None else 0
         if weights is None:
@@ -59,7 +65,8 @@ class Engine:
             weights = shard_weights(cfg, weights, rank, world)
         from ..formats.packed import is_packed
         weights = {k: (v if (is_packed(v) or not isinstance(v, torch.Tensor)) else
-                       v.to(self.device) if v.dtype == torch.float32 and k.endswith(("A_log", "dt_bias", "router_bias"))
+                       v.to(self.device) if v.dtype == torch.float32 and (k.endswith(("A_log", "dt_bias", "router_bias")) or
+                                                                                 (cfg.out_norm and k.endswith("norm")))
                        else v.to(self.device, self.dtype)) for k, v in weights.items()}
         # linears that arrived packed from a quantised checkpoint (ModelOpt NVFP4 / FP8, EXL3) become the kernels' weight
         # objects here, after the tensor-parallel cut; on the CPU they are dequantised for the fp32 oracle
@@ -68,10 +75,12 @@ class Engine:
             for k in list(weights.keys()):
                 if is_packed(weights[k]):
                     weights[k] = from_packed(weights[k], self.device, self.dtype, on_gpu)
+        if cfg.layers:
+            weights = pack_latent(cfg.shard(world), weights)
         is_t = lambda v: isinstance(v, torch.Tensor)
         if self.ecfg.weight_dtype in ("nvfp4", "nvfp4-a16", "nvfp4-w4a4"):
             from ..ops.qweight import quantize_experts, quantize_weight
-            big = ("in_proj", "out_proj", "gate_up", "down", "lm_head")
+            big = ("in_proj", "out_proj", "gate_up", "up", "down", "lm_head")
             for k in list(weights.keys()):
                 if not is_t(weights[k]):
                     continue
@@ -83,7 +92,7 @@ class Engine:
                     weights[k] = quantize_experts(weights[k])
         elif self.ecfg.weight_dtype == "fp8-block":
             from ..ops.qweight import quantize_weight
-            big = ("in_proj", "out_proj", "gate_up", "down")
+            big = ("in_proj", "out_proj", "gate_up", "up", "down")
             for k in list(weights.keys()):
                 if is_t(weights[k]) and k.split(".")[-1] in big and weights[k].dim() == 2:
                     weights[k] = quantize_weight(weights[k], "fp8b", keep_dense=True, dense_dtype=self.dtype)

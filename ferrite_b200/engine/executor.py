@@ -22,7 +22,8 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from ..config import EngineConfig, ModelConfig
-from ..models.weights import Weights
+from ..models.weights import Weights, latent_dims
+from ..ops.latent import seg_groups
 from ..ops.qweight import QWeight
 
 
@@ -49,7 +50,7 @@ class Segment:
     slot: int
     pos0: int
     tokens: List[int]
-    want_logits: str = "last"       # "last" | "all" | "none"
+    want_logits: object = "last"    # "last" | "all" | "none" | row indices inside the segment, in the order wanted
     # verify tree: parent row of every row inside the segment (-1 for row 0, parents before children). A row sits at
     # position pos0 + depth, sees the committed context plus its own ancestors, and is stored at cache row pos0 + index.
     parents: Optional[List[int]] = None
@@ -136,7 +137,8 @@ class Executor:
         c = cfg
         self.kinds = c.layer_kinds
         self.max_blocks = (ecfg.max_ctx + ecfg.kv_block - 1) // ecfg.kv_block
-        n_blocks = ecfg.n_slots * self.max_blocks + (int(ecfg.park_gb * (1 << 30) / max(1, self.kv_block_bytes())) if ecfg.park_gb > 0 else 0)
+        pool_blocks = (ecfg.kv_pool_tokens + ecfg.kv_block - 1) // ecfg.kv_block if ecfg.kv_pool_tokens else ecfg.n_slots * self.max_blocks
+        n_blocks = pool_blocks + (int(ecfg.park_gb * (1 << 30) / max(1, self.kv_block_bytes())) if ecfg.park_gb > 0 else 0)
         self.pool = BlockPool(n_blocks)
         dev, dt = self.device, self.dtype
         # quantised caches: byte codes + fp32 scales. "fp8": e4m3, one scale per (token, kv head); "int4" / "int6": 4- /
@@ -169,9 +171,18 @@ class Executor:
                 # one latent row [kv_lora | rope] per token; the value cache slot stays empty
                 self.k_cache[i] = torch.zeros(n_blocks, ecfg.kv_block, 1, c.kv_lora + c.rope_head_dim, dtype=dt, device=dev)
                 self.v_cache[i] = torch.zeros(n_blocks, 0, dtype=dt, device=dev)
+            elif kind == "latent":
+                # one latent row per token, in the layers that have latents of their own
+                if c.layers[i].kv_from is None:
+                    self.k_cache[i] = torch.zeros(n_blocks, ecfg.kv_block, latent_dims(c, i).lat, dtype=dt, device=dev)
+                    self.v_cache[i] = torch.zeros(n_blocks, 0, dtype=dt, device=dev)
             elif kind == "gdn":
                 self.rec_state[i] = torch.zeros(ecfg.n_slots, c.lin_v_heads, c.lin_dk, c.lin_dv, dtype=torch.float32, device=dev)
                 self.conv_state[i] = torch.zeros(ecfg.n_slots, c.conv_k - 1, c.conv_dim, dtype=dt, device=dev)
+        # the token at every cached position, paged like the latents: the token before a segment (bigram embeddings) is read
+        # from here, so it follows the pages through parking, forks, resumed prefixes and rejected drafts
+        self.tok_pages = torch.zeros(n_blocks, ecfg.kv_block, dtype=torch.int32, device=dev) if c.gram_buckets else None
+        self.latent_dims = {i: latent_dims(c, i) for i, kind in enumerate(self.kinds) if kind == "latent"}
         self.block_table_host = torch.full((ecfg.n_slots, self.max_blocks), -1, dtype=torch.int32)
         self.block_table = self.block_table_host.to(dev)
         self.slot_blocks: List[List[int]] = [[] for _ in range(ecfg.n_slots)]
@@ -303,6 +314,10 @@ class Executor:
             per = 2 * e.kv_block * c.n_kv * (c.head_dim * int(kd[3]) // 8 + c.head_dim // 32 * 4)
         if c.kv_lora > 0:
             per = e.kv_block * (c.kv_lora + c.rope_head_dim) * 2
+        if c.layers:
+            item = torch.empty(0, dtype=self.dtype).element_size()
+            return e.kv_block * (item * sum(latent_dims(c, i).lat for i, l in enumerate(c.layers) if l.kv_from is None)
+                                 + (4 if c.gram_buckets else 0))
         return per * max(1, self.cfg.n_attn)
 
     # ---- block tables -----------------------------------------------------------------------------
@@ -377,6 +392,8 @@ class Executor:
             self.v_cache[i][d] = self.v_cache[i][s]
             if i in self.kv_scale:
                 self.kv_scale[i][d] = self.kv_scale[i][s]
+        if self.tok_pages is not None:
+            self.tok_pages[d] = self.tok_pages[s]
 
     def copy_slot(self, src: int, dst: int, n_tokens: int) -> None:
         """Fork: copy KV pages covering n_tokens and the GDN state from one slot to another
@@ -384,14 +401,7 @@ class Executor:
         self.reset_slot(dst)
         self.ensure_capacity(dst, n_tokens)
         nb = (n_tokens + self.ecfg.kv_block - 1) // self.ecfg.kv_block
-        if nb:
-            s = torch.tensor(self.slot_blocks[src][:nb], device=self.device, dtype=torch.long)
-            d = torch.tensor(self.slot_blocks[dst][:nb], device=self.device, dtype=torch.long)
-            for i in self.k_cache:
-                self.k_cache[i][d] = self.k_cache[i][s]
-                self.v_cache[i][d] = self.v_cache[i][s]
-                if i in self.kv_scale:
-                    self.kv_scale[i][d] = self.kv_scale[i][s]
+        self.copy_blocks(self.slot_blocks[src][:nb], self.slot_blocks[dst][:nb])
         for t in self.rec_state.values():
             t[dst].copy_(t[src])
         for t in self.conv_state.values():
@@ -453,8 +463,18 @@ class Executor:
             elif sg.want_logits == "last":
                 logit_rows.append(r + n - 1)
             r += n
+        picked = any(not isinstance(sg.want_logits, str) for sg in batch.segments)
+        if picked:                                        # some segment names its rows
+            logit_rows, r = [], 0
+            for sg in batch.segments:
+                n, want = len(sg.tokens), sg.want_logits
+                inside = range(n) if want == "all" else [n - 1] if want == "last" else [] if want == "none" else [int(i) for i in want]
+                assert all(0 <= i < n for i in inside), "want_logits: row outside its segment"
+                logit_rows.extend(r + i for i in inside)
+                r += n
+            assert len(logit_rows) <= T, "want_logits: more rows than the step has"
         nl = len(logit_rows)
-        if hn is None:
+        if hn is None or picked:
             lrow[:nl] = torch.tensor(logit_rows, dtype=torch.int32) if nl else lrow[:0]
         used = 5 * T + 4 * S
         self.meta_i32[:used].copy_(h[:used], non_blocking=True)
@@ -547,6 +567,62 @@ class Executor:
             return ops.moe_experts(h, ids, wts, w[p + "experts_gate_up"], w[p + "experts_down"], e_lo, e_hi, shared, sgate, x)
         part = ops.moe_experts(h, ids, wts, w[p + "experts_gate_up"], w[p + "experts_down"], e_lo, e_hi, shared, sgate, None)
         return self.tp.allreduce_rows(ops, part, x)
+
+    # ---- models of listed layers: norms on the sublayers' outputs, 32-bit residual stream ---------------------------
+    def _sum_ranks(self, x_in, w):
+        """Row-parallel product without a residual: 32-bit sums on one rank, reduced over the ranks otherwise."""
+        if self.tp is None or self.tp.world == 1:
+            return self.ops.linear(x_in, w, out_f32=True)
+        return self.tp.linear_allreduce(self.ops, x_in, w, None)
+
+    def _mix_latent(self, xb, i, mv, groups, nsplit, gathered):
+        """Latent attention of layer i over operand rows xb: rows of prompt segments attend keys and values expanded from the
+        latents, the others the latents themselves."""
+        w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{i}.", self.latent_dims[i]
+        cache, T = self.k_cache[d.source], xb.shape[0]
+        proj = ops.linear(xb, w[p + "in_proj"], out_f32=True)
+        cq = ops.latent_prep(proj, d, w[p + "q_a_norm"], w.get(p + "kv_a_norm"), mv["slot"], mv["pos"], self.block_table, cache, kvb,
+                             self.cfg.eps)
+        q = ops.linear(cq, w[p + "q_b"])
+        o = None
+        for g in groups:
+            segs = tuple(mv[k][g.seg_lo:g.seg_hi] for k in ("sslot", "srow0", "snrows", "spos0"))
+            if g.prompt and d.hp <= 256:
+                o = torch.empty_like(q) if o is None else o
+                key = (d.source, g.row_lo)
+                if key not in gathered:                  # shared by the layers that share the latents
+                    gathered[key] = ops.latent_rows(cache, g, kvb)
+                ops.latent_attention_prompt(q, gathered[key], w[p + "kv_up"], d, g, segs, kvb, o)
+                continue
+            a, b = g.row_lo, g.row_hi
+            qabs = ops.head_linear(q[a:b].view(b - a, d.heads, d.hp), w[p + "k_abs"])
+            ol = ops.latent_attention(qabs, cache, g, mv["slot"][a:b], mv["kvlen"][a:b], segs, self.block_table, kvb, d.scale, nsplit)
+            if a == 0 and b == T:
+                o = ops.head_linear(ol, w[p + "v_up"]).reshape(T, -1)
+            else:
+                o = torch.empty_like(q) if o is None else o
+                ops.head_linear(ol, w[p + "v_up"], out=o[a:b].view(b - a, d.heads, d.hp))
+        return self._sum_ranks(o, w[p + "out_proj"])
+
+    def _layers_out_norm(self, x, xb, mv, T, nseg, max_seg_rows, nsplit):
+        """x <- x + norm(mixer(x)), x <- x + norm(ff(x)): x is the 32-bit residual stream (updated in place), xb its copy in the
+        GEMM operand type. Returns the last copy."""
+        c, w, ops = self.cfg, self.w, self.ops
+        self.taps = []
+        groups = seg_groups(self._step_segments if ops.name == "cuda" and self.dtype == torch.bfloat16 else None, nseg, T,
+                            max_seg_rows, FLASH_MIN_ROWS, self.block_table, self.ecfg.kv_block, self.device)
+        gathered: Dict[tuple, torch.Tensor] = {}
+        for i, l in enumerate(c.layers):
+            p = f"l{i}."
+            xb = ops.add_normed(x, self._mix_latent(xb, i, mv, groups, nsplit, gathered), w[p + "mix_norm"], c.hidden, c.eps)
+            if l.ff:
+                act = ops.linear(xb, w[p + "up"], act=l.act)
+                xb = ops.add_normed(x, self._sum_ranks(act, w[p + "down"]), w[p + "ffn_norm"], c.hidden, c.eps)
+            if i in c.tap_layers:
+                self.taps.append(xb[:, :c.hidden].clone() if xb is x else xb[:, :c.hidden])
+            if self.dump_layers:
+                self._dump_layer(i, x[:, :c.hidden], False, T)
+        return xb
 
     def _layers(self, x, mv, T, nseg, max_seg_rows, nsplit, commit, tv=None):
         c, w, ops = self.cfg, self.w, self.ops
@@ -722,6 +798,14 @@ class Executor:
         c, w, ops = self.cfg, self.w, self.ops
         if nlog == 0:
             return None, None
+        if c.out_norm:
+            rows = ops.norm_rows(x, mv["lrow"], w["final_norm"], c.hidden, c.eps)
+            logits = ops.linear(rows, w["lm_head"], out_f32=True)
+            if c.logit_softcap:
+                logits = ops.softcap(logits, c.logit_softcap)
+            if self.tp is not None and self.tp.world > 1:
+                return self.tp.gather_logits(ops, logits, greedy, self.tp.rank * ((c.vocab + self.tp.world - 1) // self.tp.world), c.vocab)
+            return logits, ops.argmax(logits) if greedy else None
         rows = x[mv["lrow"].long()] if nlog != x.shape[0] else x
         head = w["embed"] if c.tie_embeddings else w["lm_head"]
         if self.tp is not None and self.tp.world > 1:
@@ -740,6 +824,14 @@ class Executor:
     def _run(self, T, nseg, nlog, max_seg_rows, nsplit, commit, greedy, x_add=None, tree=False):
         mv = self._meta_views(T, nseg, nlog)
         self._last_meta = (mv, max_seg_rows)
+        if self.cfg.out_norm:
+            c, w = self.cfg, self.w
+            assert x_add is None and not tree, "models of listed layers: no injected rows, no verify trees"
+            x, xb = self.ops.embed_grams(w["embed"], w.get("bigram"), mv["tok"], mv["slot"], mv["pos"], self.block_table,
+                                         self.tok_pages, self.ecfg.kv_block, c.embed_scale, c.gram_buckets, c.gram_mul_prev,
+                                         c.gram_mul_cur)
+            self.last_hidden = self._layers_out_norm(x, xb, mv, T, nseg, max_seg_rows, nsplit)[:, :c.hidden]
+            return self._head(x, mv, nlog, greedy)
         x = self.ops.embed(self.w["embed"], mv["tok"])
         if x_add is not None and self.input_rows:
             x = x_add.to(x.dtype)                            # MTP head: the caller computed the input rows itself
@@ -884,12 +976,12 @@ class Executor:
         nseg = len(batch.segments)
         max_seg_rows = max(len(s.tokens) for s in batch.segments)
         max_kvlen = max(s.pos0 + len(s.tokens) for s in batch.segments)
-        nsplit = self.attn_splits(max_kvlen) if max_seg_rows <= FLASH_MIN_ROWS else 1
+        nsplit = self.attn_splits(max_kvlen) if max_seg_rows <= FLASH_MIN_ROWS or self.cfg.layers else 1
         use_graph = (self.ecfg.use_graphs and self.device.type == "cuda" and T <= self.ecfg.decode_rows_max
                      and self.profile is None and x_add is None and not self.dump_layers)
         tree = batch.tree
         if tree:
-            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and "mla" not in self.kinds, \
+            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and not {"mla", "latent"} & set(self.kinds), \
                 "verify trees: commit=False, at most TREE_MAX_ROWS rows per segment, attention / GDN layers"
             assert self.tp is None or self.tp.world == 1 or not self.tp.sp_ready(T)
         logit_rows = self._upload(batch)

@@ -52,12 +52,35 @@ def _take(w, index: torch.Tensor):
     raise TypeError(f"{type(w).__name__} rows cannot be regrouped")
 
 
+def _load_zototar(st: SafeTensors, cfg: ModelConfig, dtype) -> Dict[str, torch.Tensor]:
+    """A Zototar checkpoint under engine names; every tensor's shape is checked against the configuration."""
+    top = {"embed": "embed", "bigram": "bigram", "final_norm": "final.norm", "lm_head": "head"}
+    sub = {"mix_norm": "norm1", "ffn_norm": "norm2", "q_a": "mix.dq", "q_a_norm": "mix.dq.norm", "q_b": "mix.uq",
+           "kv_a": "mix.dkv", "kv_a_norm": "mix.dkv.norm", "k_b": "mix.uk", "v_b": "mix.uv", "out_proj": "mix.o",
+           "up": "mlp.up", "down": "mlp.down"}
+    w: Dict[str, torch.Tensor] = {}
+    for name, shape in weight_shapes(cfg).items():
+        layer, _, base = name.rpartition(".")
+        src = f"{layer}.{sub[base]}" if layer else top[base]
+        if not st.has(src):
+            raise KeyError(f"{src} is missing from the checkpoint")
+        t = st.get(src)
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"{src}: shape {tuple(t.shape)}, the configuration says {tuple(shape)}")
+        w[name] = t if base.endswith("norm") else t.to(dtype)
+    return w
+
+
 def load_model_weights(model_dir: str, cfg: ModelConfig, dtype=torch.bfloat16, dense: bool = False) -> Dict[str, torch.Tensor]:
     st = SafeTensors(model_dir)
     _dense = lambda st_, base, dt: _linear(st_, base, dt, dense)
     names = set(st.names())
     if "embed" in names and "final_norm" in names:                    # native layout
         return {k: st.get(k) for k in weight_shapes(cfg) if st.has(k)}
+    if cfg.layers:
+        w = _load_zototar(st, cfg, dtype)
+        st.close()
+        return w
     pre = "model.language_model." if any(n.startswith("model.language_model.") for n in names) else "model."
     w: Dict[str, torch.Tensor] = {}
     w["embed"] = st.get(pre + "embed_tokens.weight").to(dtype)

@@ -12,6 +12,7 @@ RMSNorm weights are stored zero-centred (effective weight 1 + w), the GDN gated-
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Dict, List
 
 import torch
@@ -22,9 +23,27 @@ from ..formats.packed import cat_rows
 Weights = Dict[str, torch.Tensor]
 
 
+def latent_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
+    """Latent attention with norms on the sublayers' outputs (`LayerSpec`)."""
+    l, h, p = cfg.layers[i], cfg.hidden, f"l{i}."
+    out: Dict[str, tuple] = {p + "mix_norm": (h,), p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,),
+                             p + "q_b": (l.heads * l.dim, l.q_rank)}
+    if l.kv_from is None:
+        out[p + "kv_a"] = (l.kv_rank, h)
+        out[p + "kv_a_norm"] = (l.kv_rank,)
+    out[p + "k_b"] = (l.heads * l.dim, l.kv_rank)
+    out[p + "v_b"] = (l.heads * l.vdim, l.kv_rank)
+    out[p + "out_proj"] = (h, l.heads * l.vdim)
+    if l.ff:
+        out.update({p + "ffn_norm": (h,), p + "up": (l.ff, h), p + "down": (h, l.ff)})
+    return out
+
+
 def layer_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
     h = cfg.hidden
     p = f"l{i}."
+    if cfg.layers:
+        return latent_weight_shapes(cfg, i)
     out: Dict[str, tuple] = {p + "input_norm": (h,), p + "post_norm": (h,)}
     kind = cfg.layer_kinds[i]
     if kind == "gdn":
@@ -70,6 +89,8 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
     out: Dict[str, tuple] = {"embed": (cfg.vocab, cfg.hidden), "final_norm": (cfg.hidden,)}
     if not cfg.tie_embeddings:
         out["lm_head"] = (cfg.vocab, cfg.hidden)
+    if cfg.gram_buckets:
+        out["bigram"] = (cfg.gram_buckets + 1, cfg.hidden)
     for i in range(cfg.n_layers):
         out.update(layer_weight_shapes(cfg, i))
     return out
@@ -88,9 +109,9 @@ def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="c
     w: Weights = {}
     for name, shape in weight_shapes(cfg).items():
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32) * std
-        if name.endswith("gnorm_w"):
+        if name.endswith("gnorm_w") or (cfg.out_norm and name.endswith("norm")):
             t = t + 1.0
-        keep32 = name.endswith(_F32_NAMES)
+        keep32 = name.endswith(_F32_NAMES) or (cfg.out_norm and name.endswith("norm"))
         t = t if keep32 else t.to(dtype)
         w[name] = post(name, t) if post is not None else t
     return w
@@ -160,6 +181,8 @@ def shard_weights(cfg: ModelConfig, w: Weights, rank: int, world: int) -> Weight
                 per = cfg.lin_v_heads // world * cfg.lin_dv
             elif kind == "attn":
                 per = cfg.n_q // world * cfg.head_dim
+            elif kind == "latent":
+                per = t.shape[1] // world
             else:
                 per = cfg.n_q // world * cfg.v_head_dim
             out[name] = t[:, rank * per:(rank + 1) * per].contiguous()
@@ -174,6 +197,9 @@ def shard_weights(cfg: ModelConfig, w: Weights, rank: int, world: int) -> Weight
             # expert parallel: whole experts per rank
             per = cfg.n_experts // world
             out[name] = t[rank * per:(rank + 1) * per].contiguous()
+        elif base in ("k_b", "v_b", "up"):
+            per = t.shape[0] // world
+            out[name] = t[rank * per:(rank + 1) * per].contiguous()
         elif base == "q_b":
             per = t.shape[0] // world
             out[name] = t[rank * per:(rank + 1) * per].contiguous()
@@ -182,4 +208,84 @@ def shard_weights(cfg: ModelConfig, w: Weights, rank: int, world: int) -> Weight
             out[name] = t[rank * per:(rank + 1) * per].contiguous()
         else:
             out[name] = t
+    return out
+
+
+# ---- kernel layout of latent-attention layers ------------------------------------------------------------------------
+
+def round_up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass(frozen=True)
+class LatentDims:
+    """Sizes of one latent-attention layer as its kernels see them. Every dimension is padded with zeros to the tile grid
+    of the GEMMs (64 columns) and the head width to one the tensor-core prompt kernel takes (64 / 128 / 256; wider heads
+    go up in steps of 64 and keep to the latent form). Norms divide by the true sizes."""
+
+    heads: int
+    q_rank: int
+    kv_rank: int
+    qr: int           # padded q_rank
+    lat: int          # padded kv_rank = cache row
+    hp: int           # padded head width, keys and values alike
+    scale: float
+    source: int       # layer whose cache holds the latents
+
+
+def latent_dims(cfg: ModelConfig, i: int) -> LatentDims:
+    l = cfg.layers[i]
+    hd = max(l.dim, l.vdim)
+    hp = next((w for w in (64, 128, 256) if hd <= w), round_up(hd, 64))
+    return LatentDims(l.heads, l.q_rank, l.kv_rank, round_up(l.q_rank, 64), round_up(l.kv_rank, 64), hp, l.scale,
+                      i if l.kv_from is None else l.kv_from)
+
+
+def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
+    if tuple(t.shape) == shape:
+        return t.contiguous()
+    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
+    out[tuple(slice(0, n) for n in t.shape)] = t
+    return out
+
+
+def pack_latent(cfg: ModelConfig, w: Weights) -> Weights:
+    """Engine weights of a latent-attention model in the kernels' layout (see `LatentDims`):
+
+    * in_proj  rows = [q_a | kv_a]           one product for both latents of a token
+    * q_b      [heads * hp, qr]              per head zero-padded rows, so queries come out at the padded width
+    * kv_up    [2 * heads * hp, lat]         key rows of every head, then value rows: expands latents for prompt rows
+    * k_abs    [heads, lat, hp]              W_uk^T per head: folds the key projection into a decode row's query
+    * v_up     [heads, hp, lat]              W_uv per head (a view of kv_up): latent-space outputs to values
+    * out_proj [width, heads * hp]
+
+    Norm weights become 32-bit."""
+    W = round_up(cfg.hidden, 64)
+    out: Weights = {"embed": _pad(w["embed"], cfg.vocab, W), "lm_head": _pad(w["lm_head"], w["lm_head"].shape[0], W),
+                    "final_norm": _pad(w["final_norm"].float(), W)}
+    if cfg.gram_buckets:
+        out["bigram"] = _pad(w["bigram"], cfg.gram_buckets + 1, W)
+    for i, l in enumerate(cfg.layers):
+        p, d = f"l{i}.", latent_dims(cfg, i)
+        parts = [_pad(w[p + "q_a"], d.qr, W)]
+        out[p + "q_a_norm"] = _pad(w[p + "q_a_norm"].float(), d.qr)
+        if l.kv_from is None:
+            parts.append(_pad(w[p + "kv_a"], d.lat, W))
+            out[p + "kv_a_norm"] = _pad(w[p + "kv_a_norm"].float(), d.lat)
+        out[p + "in_proj"] = torch.cat(parts)
+        q_b = _pad(w[p + "q_b"].view(l.heads, l.dim, l.q_rank), l.heads, d.hp, d.qr)
+        out[p + "q_b"] = q_b.view(l.heads * d.hp, d.qr)
+        k = _pad(w[p + "k_b"].view(l.heads, l.dim, l.kv_rank), l.heads, d.hp, d.lat)
+        v = _pad(w[p + "v_b"].view(l.heads, l.vdim, l.kv_rank), l.heads, d.hp, d.lat)
+        out[p + "kv_up"] = torch.cat([k.view(-1, d.lat), v.view(-1, d.lat)])
+        out[p + "k_abs"] = k.transpose(1, 2).contiguous()
+        out[p + "v_up"] = out[p + "kv_up"][l.heads * d.hp:].view(l.heads, d.hp, d.lat)
+        o = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp)
+        out[p + "out_proj"] = o.view(W, l.heads * d.hp)
+        out[p + "mix_norm"] = _pad(w[p + "mix_norm"].float(), W)
+        if l.ff:
+            F = round_up(l.ff, 64)
+            out[p + "up"] = _pad(w[p + "up"], F, W)
+            out[p + "down"] = _pad(w[p + "down"], W, F)
+            out[p + "ffn_norm"] = _pad(w[p + "ffn_norm"].float(), W)
     return out

@@ -16,6 +16,7 @@ import torch
 
 from .._ext import load
 from .extras import CudaExtras
+from .latent import CudaLatent
 from .qweight import Exl3Weight, ExpertsFP4, GgufWeight, QWeight, StackWeight
 
 GEMV_MAX_ROWS = 8
@@ -23,14 +24,15 @@ MOE_PAIR_ROWS = 64     # up to this many rows (the largest graph-captured step) 
                        # beyond as grouped GEMMs, which read the per-expert row counts on the host
 
 
-class CudaOps(CudaExtras):
+class CudaOps(CudaLatent, CudaExtras):
     name = "cuda"
 
     def __init__(self, device, dtype=torch.bfloat16):
         self.C = load()
         self.device = torch.device(device)
         self.dtype = dtype
-        assert dtype == torch.bfloat16, "the sm_100a kernels take bf16 activations"
+        # fp32: the kernels of the models of listed layers (`ops/latent.py`); the other families' kernels take bf16 only
+        assert dtype in (torch.bfloat16, torch.float32), "the sm_100a kernels take bf16 or fp32 activations"
         cap = torch.cuda.get_device_capability(self.device)
         if cap != (10, 0) and not os.environ.get("FB_SKIP_ARCH_CHECK"):
             # the extension holds sm_100a code only: on any other GPU every launch would fail with "no kernel image"
@@ -154,7 +156,20 @@ class CudaOps(CudaExtras):
         s = max(1, min(kblocks // 4, want))
         return s
 
-    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, out=None):
+    def relu2(self, x):
+        y = self.empty(x.shape[0], x.shape[1], dtype=self.dtype, device=self.device)
+        self.launches += 1
+        self.C.relu2(y, x)
+        return y
+
+    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, out=None, act=None):
+        """`act`: activation of the epilogue ("relu2": squared relu), not together with SwiGLU."""
+        if self.dtype == torch.float32:
+            assert norm_w is None and res is None and not swiglu, "fp32 linears have an activation epilogue only"
+            return self.linear_f32(x, w, act, out)
+        if act is not None and not isinstance(w, torch.Tensor):
+            assert act == "relu2" and not swiglu and not out_f32
+            return self.relu2(self.linear(x, w, norm_w=norm_w, eps=eps, res=res))      # packed weights: a pass of its own
         if isinstance(w, (Exl3Weight, StackWeight, GgufWeight)):
             # EXL3 / GGUF blocks (and stacks of differently stored parts): the norm runs once, each part fills its column
             # range, the SwiGLU / residual run on the joined output. The trellis kernels rotate their own input.
@@ -222,7 +237,7 @@ class CudaOps(CudaExtras):
             # a few rows (concurrent decode streams, speculative verify): weights streamed once into mma.sync fragments
             y = out if out is not None else self.empty(M, N, dtype=torch.float32 if out_f32 else self.dtype, device=self.device)
             self.launches += 1
-            self.C.gemv_mma(y, x, w, norm_w, res, eps, 1 if swiglu else 0, self._workspace(8 << 20), self._counters)
+            self.C.gemv_mma(y, x, w, norm_w, res, eps, 1 if swiglu else 2 if act else 0, self._workspace(8 << 20), self._counters)
             return y
         if M <= GEMV_MAX_ROWS or self.force_gemv_chunks:
             y = out if out is not None else self.empty(M, N, dtype=torch.float32 if out_f32 else self.dtype, device=self.device)
@@ -230,7 +245,7 @@ class CudaOps(CudaExtras):
                 r1 = min(M, r0 + GEMV_MAX_ROWS)
                 self.launches += 1
                 self.C.gemv(y[r0:r1], x[r0:r1], w, norm_w, None if res is None else res[r0:r1], eps, True,
-                            1 if swiglu else 0)
+                            1 if swiglu else 2 if act else 0)
             return y
         if norm_w is not None:
             x, _ = self.rmsnorm(x, norm_w, eps, True)
@@ -244,7 +259,7 @@ class CudaOps(CudaExtras):
             ws = self._workspace(nb)
             cnt = self._counters
         self.launches += 1
-        self.C.gemm(y, x, w, res, (1 if swiglu else 0) | (2 if out_f32 else 0), split, ws, cnt, self.status_word)
+        self.C.gemm(y, x, w, res, (1 if swiglu else 0) | (2 if out_f32 else 0) | (4 if act else 0), split, ws, cnt, self.status_word)
         return y
 
     # ---- FP8 (e4m3) weights and activations -----------------------------------------------------------
@@ -710,6 +725,8 @@ class CudaOps(CudaExtras):
         GEMM (every head a group of T rows)."""
         T, nh, K = x.shape
         N = W.shape[1]
+        if self.dtype == torch.float32:
+            return self.linear_f32(x, W, None, out)
         y = out if out is not None else self.empty(T, nh, N, dtype=self.dtype, device=self.device)
         if T <= 8 or K % 64 or N % 8 or nh * T < 256 or nh * N < 256:      # the GEMM's 128/256-row boxes fit the operands
             self.launches += 1

@@ -13,13 +13,14 @@ import torch
 import torch.nn.functional as F
 
 from .extras import TorchExtras
+from .latent import TORCH_ACTS, TorchLatent
 
 
 def _softplus(x):
     return torch.where(x > 20, x, torch.log1p(torch.exp(torch.clamp(x, max=20.0))))
 
 
-class TorchOps(TorchExtras):
+class TorchOps(TorchLatent, TorchExtras):
     name = "torch"
 
     def __init__(self, device="cpu", dtype=torch.float32):
@@ -40,8 +41,8 @@ class TorchOps(TorchExtras):
         wf = w.float() + 1.0 if centred else w.float()
         return (xf * r * wf).to(self.dtype), x
 
-    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False):
-        """y = x W^T with optional RMSNorm(1+w) prologue, SwiGLU (W = [gate|up]) or residual epilogue."""
+    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, act=None):
+        """y = x W^T with optional RMSNorm(1+w) prologue, SwiGLU (W = [gate|up]), activation or residual epilogue."""
         if hasattr(w, "dense"):
             w = w.dense                      # quantised weight: the oracle multiplies by its dequantised values
         xf = x.float()
@@ -52,6 +53,7 @@ class TorchOps(TorchExtras):
         if swiglu:
             i = y.shape[-1] // 2
             y = F.silu(y[:, :i]) * y[:, i:]
+        y = TORCH_ACTS[act](y)
         if res is not None:
             y = y + res.float()
         return y if out_f32 else y.to(self.dtype)
