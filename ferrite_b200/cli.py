@@ -15,7 +15,7 @@ Launched under `python -m torch.distributed.run --nproc-per-node N` every rank r
 tensor-parallel engine (greedy picks are the same on every rank); rank 0 prints.
 
 Common: `--device cuda|cpu`, `--layers N` (cut the model), `--weights bf16|nvfp4|...`, `--spec N` (draft depth for the
-scheduler commands). `--model DIR` loads a checkpoint directory (safetensors bf16 / ModelOpt NVFP4 / EXL3 / GGUF) and its
+scheduler commands), `--compute fp32` (full precision on the GPU), `--kv-tokens N` (size of the page pool). `--model DIR` loads a checkpoint directory (safetensors bf16 / ModelOpt NVFP4 / EXL3 / GGUF) and its
 tokenizer; without it the weights are seeded random and ids stand for text.
 
 Counterpart of the reference's `ferrite selftest | gemm-bench | generate | logits | bench | sched-test | park-test |
@@ -91,7 +91,7 @@ def build_engine(a, n_slots: int = 1, max_ctx: int = 4096, tap_layers=None):
     if tap_layers == "thirds" and not cfg.tap_layers:
         cfg.tap_layers = sorted({max(0, cfg.n_layers * (i + 1) // 4 - 1) for i in range(3)})
     tp = tp_from_env(a)
-    ecfg = EngineConfig(n_slots=n_slots, max_ctx=max_ctx, weight_dtype=a.weights)
+    ecfg = EngineConfig(n_slots=n_slots, max_ctx=max_ctx, weight_dtype=a.weights, kv_pool_tokens=a.kv_tokens, compute_dtype=a.compute)
     eng = Engine(cfg, weights, ecfg, device=a.device or None, seed=a.seed, tp=tp)
     return cfg, eng, tok
 
@@ -514,10 +514,13 @@ def main(argv: Optional[List[str]] = None) -> int:
     sub = ap.add_subparsers(dest="cmd", required=True)
 
     def common(p, max_tokens: int):
-        p.add_argument("--preset", default="tiny", help="tiny | tiny-mla | 27b | moe80b | mla671b | drafter")
+        p.add_argument("--preset", default="tiny", help="tiny | tiny-mla | tiny-zototar | 27b | moe80b | mla671b | zototar-7b | drafter")
         p.add_argument("--model", default="", help="checkpoint directory (config.json + safetensors, or a .gguf)")
         p.add_argument("--layers", type=int, default=0)
         p.add_argument("--weights", default="bf16")
+        p.add_argument("--compute", default="bf16", choices=["bf16", "fp32"], help="fp32: 32-bit activations, weights and cache on the "
+                       "GPU (models of listed layers)")
+        p.add_argument("--kv-tokens", type=int, default=0, help="tokens the page pool holds over all slots (0: max-ctx for every slot)")
         p.add_argument("--device", default="")
         p.add_argument("--seed", type=int, default=0)
         p.add_argument("--max-ctx", type=int, default=4096)

@@ -378,6 +378,8 @@ class EngineConfig:
             return int(e[name]) if name in e and e[name] != "" else cur
         c.n_slots = geti("FERRITE_SLOTS", c.n_slots)
         c.max_ctx = geti("FERRITE_CTX", c.max_ctx)
+        c.kv_pool_tokens = geti("FERRITE_KV_TOKENS", c.kv_pool_tokens)
+        c.compute_dtype = e.get("FERRITE_COMPUTE", "") or c.compute_dtype
         c.prefill_chunk = geti("FERRITE_CHUNK", c.prefill_chunk)
         c.spec_depth = geti("FE_SPEC", c.spec_depth)
         c.graph_max = geti("FE_GRAPH_MAX", c.graph_max)

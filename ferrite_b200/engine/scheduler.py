@@ -376,12 +376,40 @@ class Scheduler:
         sc.clear()
 
     def _reclaim(self) -> bool:
-        """Evict the least recently used parked sequence and return its pages to the pool."""
+        """Evict the least recently used parked sequence and return its pages to the pool; with none left, drop what a free
+        slot still keeps of its last conversation."""
         ev = self.park.evict_lru()
-        if ev is None:
-            return False
-        self.eng.ex.pool.release(ev.blocks)
-        return True
+        if ev is not None:
+            self.eng.ex.pool.release(ev.blocks)
+            return True
+        for s in self.free:
+            if self.eng.ex.slot_blocks[s]:
+                self.eng.reset_slot(s)
+                self.slot_cache[s].clear()
+                return True
+        return False
+
+    def _pages(self, n_tokens: int) -> int:
+        return (n_tokens + self.eng.ecfg.kv_block - 1) // self.eng.ecfg.kv_block
+
+    def _make_room(self, wants: Sequence[Tuple[int, int]]) -> None:
+        """Reclaim pages until every (slot, tokens) of `wants` can be covered. Done before the step, so that under tensor
+        parallelism the releases reach the other ranks before the step that needs them."""
+        need = sum(max(0, self._pages(n) - len(self.eng.ex.slot_blocks[s])) for s, n in wants)
+        while self.eng.ex.pool.n_free < need and self._reclaim():
+            pass
+
+    def _forward(self, segs: List[Segment], **kw):
+        self._make_room([(s.slot, s.pos0 + len(s.tokens)) for s in segs])
+        return self.eng.forward(segs, **kw)
+
+    def _fits(self, req: Request) -> bool:
+        """A page pool smaller than slots x max_ctx: admit a request only while the pages that it and the running ones may
+        come to need exist, so no running request is ever cut short. A request that runs alone is always admitted."""
+        def most(r: Request) -> int:
+            room = DECODE_ROWS if self.opts.spec > 0 or self.drafter else 1
+            return self._pages(min(len(r.prompt) + r.sampling.max_tokens + room, self.eng.ecfg.max_ctx))
+        return not self.active or most(req) + sum(most(a.req) for a in self.active.values()) <= self.eng.ex.pool.n_blocks
 
     # ---- shared prefill: a request whose prompt starts like one that is being prefilled waits for it --------------
     def _share_point(self, prompt: Sequence[int], a: Active) -> int:
@@ -418,6 +446,8 @@ class Scheduler:
             if self._should_wait(self.backlog[i]):
                 i += 1
                 continue
+            if not self._fits(self.backlog[i]):
+                break                                  # first come, first served: later requests do not overtake it
             req = self.backlog.pop(i)
             if req.cancel.is_set():
                 if req.sink:
@@ -435,6 +465,7 @@ class Scheduler:
                 src, fs = fork
                 self._park_slot(slot) if sc.tokens else self.eng.reset_slot(slot)
                 nb = (fs.pos + self.eng.ecfg.kv_block - 1) // self.eng.ecfg.kv_block
+                self._make_room([(slot, fs.pos)])
                 self.eng.ex.ensure_capacity(slot, fs.pos)
                 self.eng.ex.copy_blocks(self.eng.ex.slot_blocks[src.slot][:nb], self.eng.ex.slot_blocks[slot][:nb])
                 self.eng.ex.state_restore(slot, fs.state["gdn"])
@@ -451,6 +482,7 @@ class Scheduler:
                 self._park_slot(slot) if sc.tokens else self.eng.reset_slot(slot)
                 nb = (ps.pos + self.eng.ecfg.kv_block - 1) // self.eng.ecfg.kv_block
                 if pe.shared:
+                    self._make_room([(slot, ps.pos)])
                     self.eng.ex.ensure_capacity(slot, ps.pos)
                     self.eng.ex.copy_blocks(pe.blocks[:nb], self.eng.ex.slot_blocks[slot][:nb])
                     self.park.touch(pe)
@@ -550,7 +582,7 @@ class Scheduler:
             return self._decode_step(decoders), self._prefill_step(a, budget)
         segs = [Segment(d.slot, d.pos, [d.next_token], "last") for d in decoders]
         segs.append(Segment(a.slot, a.pos, toks, "last" if last else "none"))
-        logits, picks, rows = self.eng.forward(segs, commit=True, greedy=True)
+        logits, picks, rows = self._forward(segs, commit=True, greedy=True)
         ids = picks[0].tolist()
         if self.opts.finite_check and not bool(picks[1].all()):
             for d in decoders + [a]:
@@ -582,7 +614,7 @@ class Scheduler:
             return self._prefill_step(group[0][0], group[0][1])
         segs = [Segment(a.slot, a.pos, toks, "last" if last else "none") for a, _, toks, last, _ in group]
         all_greedy = all(g for _, _, _, last, g in group if last)
-        logits, picks, _ = self.eng.forward(segs, greedy=all_greedy)
+        logits, picks, _ = self._forward(segs, greedy=all_greedy)
         ids = picks[0].tolist() if (all_greedy and picks is not None) else None
         k = r = n = 0
         for a, cut, toks, last, _ in group:
@@ -607,7 +639,7 @@ class Scheduler:
     def _prefill_step(self, a: Active, budget: int) -> int:
         """Run the next chunk of a prompt on its own."""
         cut, toks, last, greedy = self._prefill_cut(a, budget)
-        logits, picks, _ = self.eng.forward([Segment(a.slot, a.pos, toks, "last" if last else "none")], greedy=greedy)
+        logits, picks, _ = self._forward([Segment(a.slot, a.pos, toks, "last" if last else "none")], greedy=greedy)
         tok = None
         if last:
             tok = int(picks[0][0]) if greedy else a.sampler.sample(logits[0], first=not a.out)
@@ -690,7 +722,7 @@ class Scheduler:
             segs.append(Segment(a.slot, a.pos, [a.next_token] + d, "all", parents=par))
         spec = any(drafts)
         all_greedy = all(a.req.sampling.greedy for a in decoders)
-        logits, picks, rows = self.eng.forward(segs, commit=not spec, greedy=all_greedy)
+        logits, picks, rows = self._forward(segs, commit=not spec, greedy=all_greedy)
         ids = picks[0].tolist() if all_greedy else None
         if self.opts.finite_check:
             finite = bool(picks[1].all()) if all_greedy else bool(torch.isfinite(logits).all())

@@ -47,6 +47,8 @@ class MtpDrafter(Drafter):
 
     def __init__(self, target: Engine, n_slots: int, max_ctx: int, seed: int = 1, weights=None, depth: int = 4):
         tcfg = target.full_cfg
+        if tcfg.layers:
+            raise ValueError("the MTP head shares a target's plain embedding table: models of listed layers have none")
         assert tcfg.tap_layers and tcfg.tap_layers[-1] == tcfg.n_layers - 1, "the target must tap its last layer"
         self.target = target
         self.depth = depth

@@ -81,6 +81,7 @@ class RefState:
     def __init__(self, cfg: ModelConfig):
         self.cfg = cfg
         self.pos = 0
+        self.prev: Optional[int] = None          # last token (hashed bigram embeddings)
         self.k: List[List[torch.Tensor]] = [[] for _ in range(cfg.n_layers)]
         self.v: List[List[torch.Tensor]] = [[] for _ in range(cfg.n_layers)]
         self.conv = [torch.zeros(cfg.conv_dim, cfg.conv_k - 1) for _ in range(cfg.n_layers)]
@@ -88,7 +89,7 @@ class RefState:
 
     def clone(self) -> "RefState":
         s = RefState(self.cfg)
-        s.pos = self.pos
+        s.pos, s.prev = self.pos, self.prev
         s.k = [list(x) for x in self.k]
         s.v = [list(x) for x in self.v]
         s.conv = [x.clone() for x in self.conv]
@@ -190,6 +191,33 @@ class RefModel:
         o = torch.einsum("ht,thd->hd", pr, vv)
         return w[p + "out_proj"] @ o.reshape(-1)
 
+    def _latent(self, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """Latent attention without positions; a layer with `kv_from` reads the rows that layer appended for this token."""
+        l, w, p, eps = self.cfg.layers[i], self.w, f"l{i}.", self.cfg.eps
+        q = (w[p + "q_b"] @ rmsnorm(w[p + "q_a"] @ x, w[p + "q_a_norm"], eps, False)).view(l.heads, l.dim)
+        if l.kv_from is None:
+            st.k[i].append(rmsnorm(w[p + "kv_a"] @ x, w[p + "kv_a_norm"], eps, False))
+        lat = torch.stack(st.k[i if l.kv_from is None else l.kv_from], 0)                  # [T, kv_rank]
+        k = (lat @ w[p + "k_b"].t()).view(-1, l.heads, l.dim)
+        v = (lat @ w[p + "v_b"].t()).view(-1, l.heads, l.vdim)
+        pr = torch.softmax(torch.einsum("hd,thd->ht", q, k) * l.scale, -1)
+        return w[p + "out_proj"] @ torch.einsum("ht,thv->hv", pr, v).reshape(-1)
+
+    def _token_out_norm(self, t: int, st: RefState, tap: list) -> torch.Tensor:
+        """One token through a model with norms on the sublayers' outputs: the row before the final norm."""
+        c, w = self.cfg, self.w
+        x = w["embed"][t] * c.embed_scale
+        if c.gram_buckets:
+            x = x + w["bigram"][c.gram_buckets if st.prev is None else (st.prev * c.gram_mul_prev + t * c.gram_mul_cur) % c.gram_buckets]
+        st.prev = t
+        for i, l in enumerate(c.layers):
+            x = x + rmsnorm(self._latent(i, x, st), w[f"l{i}.mix_norm"], c.eps, False)
+            if l.ff:
+                x = x + rmsnorm(w[f"l{i}.down"] @ torch.relu(w[f"l{i}.up"] @ x).square(), w[f"l{i}.ffn_norm"], c.eps, False)
+            if i in c.tap_layers:
+                tap.append(x.clone())
+        return x
+
     def _ffn(self, i: int, x: torch.Tensor) -> torch.Tensor:
         c, w = self.cfg, self.w
         p = f"l{i}."
@@ -212,8 +240,15 @@ class RefModel:
         logits, taps = [], []
         head = w["embed"] if c.tie_embeddings else w["lm_head"]
         for t in list(tokens):
-            x = w["embed"][int(t)].clone()
             tap = []
+            if c.out_norm:
+                x = self._token_out_norm(int(t), st, tap)
+                st.pos += 1
+                y = head @ rmsnorm(x, w["final_norm"], c.eps, False)
+                logits.append(c.logit_softcap * torch.tanh(y / c.logit_softcap) if c.logit_softcap else y)
+                taps.append(tap)
+                continue
+            x = w["embed"][int(t)].clone()
             for i, kind in enumerate(c.layer_kinds):
                 h = rmsnorm(x, w[f"l{i}.input_norm"], c.eps)
                 if kind == "gdn":

@@ -44,7 +44,8 @@ def build_engine(args, tok):
         elif not cfg.tap_layers:
             cfg.tap_layers = sorted({max(0, cfg.n_layers * (i + 1) // 4 - 1) for i in range(3)})
     ecfg = EngineConfig.from_env(n_slots=args.slots, max_ctx=args.max_model_len, prefill_chunk=args.prefill_chunk,
-                                 weight_dtype=args.weights)
+                                 weight_dtype=args.weights, kv_pool_tokens=getattr(args, "kv_tokens", None),
+                                 compute_dtype=getattr(args, "compute", None))
     weights = None
     if args.model_dir and any(f.endswith(".safetensors") for f in os.listdir(args.model_dir)):
         from ..formats.loader import load_model_weights
@@ -124,6 +125,8 @@ def main(argv=None) -> int:
     ap.add_argument("--preset", default="tiny", choices=sorted(PRESETS))
     ap.add_argument("--layers", type=int, default=0)
     ap.add_argument("--weights", default=os.environ.get("FERRITE_WEIGHTS", "bf16"))
+    ap.add_argument("--compute", default=None, choices=["bf16", "fp32"], help="fp32: models of listed layers in full precision")
+    ap.add_argument("--kv-tokens", type=int, default=None, help="tokens the page pool holds over all slots (default: max context per slot)")
     ap.add_argument("--device", default="")
     ap.add_argument("--slots", type=int, default=int(os.environ.get("FERRITE_SLOTS", "4")))
     ap.add_argument("--prefill-chunk", type=int, default=int(os.environ.get("FERRITE_CHUNK", "2048")))
