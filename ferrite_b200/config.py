@@ -313,7 +313,7 @@ def zototar(width: int, n_layers: int, heads: int, q_rank: int, kv_rank: int, ff
 def tiny_zototar() -> ModelConfig:
     """5-layer plumbing model of the latent-attention family: unequal layers, sizes off the kernels' tile grid."""
     c = zototar(200, 5, 4, 72, 80, 224, 300, dim=40, vdim=24, buckets=97, name="tiny-zototar")
-    c.layers[2] = dataclasses.replace(c.layers[2], heads=3, dim=16, vdim=48, q_rank=56, kv_rank=136, scale=0.3, ff=0)
+    c.layers[2] = dataclasses.replace(c.layers[2], heads=6, dim=16, vdim=48, q_rank=56, kv_rank=136, scale=0.3, ff=0)
     c.layers[3] = dataclasses.replace(c.layers[3], kv_from=0, heads=2)
     c.layers[4] = dataclasses.replace(c.layers[4], kv_from=2, kv_rank=136, ff=104)
     return c

@@ -1,0 +1,383 @@
+"""The kernels and the engine of the Zototar design on the GPU, in bf16 and in fp32, against plain statements of the same
+arithmetic: every kernel alone (sizes on and off its tiles, keys at page borders, keys just inside and just outside what a row
+sees), then whole models in prompts, portions, decoding, mixed batches and through the scheduler."""
+import math
+
+import pytest
+import torch
+
+import plain_latent as plain
+from ferrite_b200.engine.executor import Segment
+from ferrite_b200.engine.sampler import Sampling
+from ferrite_b200.engine.scheduler import SchedOptions, Scheduler, generate
+from ferrite_b200.models.weights import LatentDims
+from ferrite_b200.ops.latent import SegGroup, seg_groups
+from ferrite_b200.ops.torch_ops import TorchOps
+from zototar_cases import CASES, config, engine, error, layer, run_cuts, tokens, weights, write
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda"
+BF, F32 = torch.bfloat16, torch.float32
+LIM = {"fp32": 3e-5, "bf16": 6e-2}
+
+
+@pytest.fixture(scope="module")
+def cops(ext):
+    from ferrite_b200.ops.cuda_ops import CudaOps
+    return {BF: CudaOps(DEV), F32: CudaOps(DEV, F32)}
+
+
+def gen(seed):
+    g = torch.Generator(device=DEV).manual_seed(seed)
+    return lambda *s, sc=1.0, dt=F32: (torch.randn(*s, generator=g, device=DEV) * sc).to(dt)
+
+
+def i32(v):
+    return torch.tensor(v, dtype=torch.int32, device=DEV)
+
+
+# ---- kernels ------------------------------------------------------------------------------------------------------------
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("width", [64, 320, 4096])
+def test_embedding_norms_softcap(cops, dt, width):
+    ops, tops, r = cops[dt], TorchOps(DEV, dt), gen(width)
+    kvb, V, B = 64, 50, 37
+    table, grams = r(V, width, dt=dt), r(B + 1, width, dt=dt)
+    bt = torch.randperm(6, device=DEV).to(torch.int32).view(2, 3)
+    pa, pb = torch.zeros(6, kvb, dtype=torch.int32, device=DEV), torch.zeros(6, kvb, dtype=torch.int32, device=DEV)
+    for lo, hi, lo1, hi1 in ((0, 64, 0, 1), (64, 65, 1, 3), (65, 130, 3, 70)):           # segments that start at page borders too
+        tok = torch.randint(0, V, (hi - lo + hi1 - lo1,), device=DEV).to(torch.int32)
+        slot, pos = i32([1] * (hi - lo) + [0] * (hi1 - lo1)), i32(list(range(lo, hi)) + list(range(lo1, hi1)))
+        for mul in ((31, 7), (1 << 31, (1 << 31) - 1)):                                  # products beyond 32 bits
+            x, xb = ops.embed_grams(table, grams, tok, slot, pos, bt, pa, kvb, 1.7, B, *mul)
+            y, _ = tops.embed_grams(table, grams, tok, slot, pos, bt, pb, kvb, 1.7, B, *mul)
+            assert torch.allclose(x, y, atol=1e-5, rtol=1e-6) and torch.equal(xb, x.to(dt)) and torch.equal(pa, pb)
+    x, _ = ops.embed_grams(table, None, tok, slot, pos, bt, None, kvb, 1.7, 0, 0, 0)
+    assert torch.allclose(x, table[tok.long()].float() * 1.7)
+    x, w = r(9, width), r(width)
+    true = width - 5
+    w[true:] = 0
+    for y in (r(9, width, sc=4.0), r(9, width, dt=BF)):
+        y[:, true:] = 0
+        x1 = x.clone()
+        xb = ops.add_normed(x1, y, w, true, 1e-5)
+        want = x.double() + plain.rms_norm(y[:, :true].double(), w[:true].double(), 1e-5).new_zeros(9, width)
+        want[:, :true] += plain.rms_norm(y[:, :true].double(), w[:true].double(), 1e-5)
+        assert torch.allclose(x1.double(), want, atol=2e-5, rtol=1e-5) and torch.equal(xb, x1.to(dt))
+    idx = i32([8, 0, 3])
+    got = ops.norm_rows(x, idx, w, width, 1e-5)
+    assert torch.allclose(got.double(), plain.rms_norm(x[idx.long()].double(), w.double(), 1e-5), atol=1e-5 if dt == F32 else 5e-2)
+    z = r(3, 515, sc=60.0)[:, :511]
+    assert torch.allclose(ops.softcap(z.clone(), 25.0), plain.softcap(z, 25.0), atol=1e-4)
+    assert ops.status() == 0
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("q_rank,kv_rank,own", [(72, 100, True), (1536, 512, True), (64, 576, True), (40, 200, False)])
+def test_latent_prep(cops, dt, q_rank, kv_rank, own):
+    ops, r, kvb = cops[dt], gen(q_rank), 64
+    up = lambda n: (n + 63) // 64 * 64
+    d = LatentDims(1, q_rank, kv_rank, up(q_rank), up(kv_rank), 64, 1.0, 0)
+    proj = torch.zeros(7, d.qr + (d.lat if own else 0), device=DEV)
+    qn, kn = torch.zeros(d.qr, device=DEV), torch.zeros(d.lat, device=DEV)
+    proj[:, :q_rank], qn[:q_rank], kn[:kv_rank] = r(7, q_rank, sc=3.0), r(q_rank), r(kv_rank)
+    if own:
+        proj[:, d.qr:d.qr + kv_rank] = r(7, kv_rank, sc=0.01)
+    cache = torch.full((4, kvb, d.lat), 5.0, dtype=dt, device=DEV)
+    bt, slot, pos = i32([[3, 1], [0, 2]]), i32([0, 0, 0, 1, 1, 1, 1]), i32([62, 63, 64, 0, 1, 2, 127])
+    cq = ops.latent_prep(proj, d, qn, kn if own else None, slot, pos, bt, cache, kvb, 1e-4)
+    tol = 1e-5 if dt == F32 else 3e-2
+    assert torch.allclose(cq[:, :q_rank].float(), plain.rms_norm(proj[:, :q_rank], qn[:q_rank], 1e-4), atol=tol, rtol=tol)
+    assert cq[:, q_rank:].float().abs().sum() == 0
+    rows = cache[bt[slot.long(), pos.long() // kvb].long(), pos.long() % kvb].float()
+    if own:
+        want = plain.rms_norm(proj[:, d.qr:d.qr + kv_rank], kn[:kv_rank], 1e-4)
+        assert torch.allclose(rows[:, :kv_rank], want, atol=tol, rtol=tol) and rows[:, kv_rank:].abs().sum() == 0
+        assert int((cache != 5.0).any(-1).sum()) == 7
+    else:
+        assert bool((cache == 5.0).all())
+    assert ops.status() == 0
+
+
+def paged(lat, lens, dt, seed, kvb=64):
+    r = gen(seed)
+    nb = [(n + kvb - 1) // kvb for n in lens]
+    perm = torch.randperm(sum(nb) + 2, generator=torch.Generator().manual_seed(seed)).tolist()
+    bt = torch.full((len(lens), max(nb)), -1, dtype=torch.int32)
+    k = 0
+    for s, n in enumerate(nb):
+        for j in range(n):
+            bt[s, j] = perm[k]
+            k += 1
+    return r(sum(nb) + 2, kvb, lat, dt=dt), bt.to(DEV)
+
+
+def attend_case(ops, dt, lat, heads, segs, nsplit, scale, seed, plant=None):
+    """segs: (rows, context length after the segment). Returns (kernel's rows, plain rows)."""
+    kvb, r = 64, gen(seed + 1)
+    cache, bt = paged(lat, [n for _, n in segs], dt, seed)
+    slot = i32([s for s, (m, _) in enumerate(segs) for _ in range(m)])
+    kvlen = i32([n - m + j + 1 for m, n in segs for j in range(m)])
+    row0 = [sum(m for m, _ in segs[:s]) for s in range(len(segs))]
+    q = r(slot.numel(), heads, lat, dt=dt)
+    if plant is not None:
+        plant(q, cache, bt, kvb)
+    ms = max(m for m, _ in segs)
+    tables = (i32(list(range(len(segs)))), i32(row0), i32([m for m, _ in segs]))
+    got = ops.latent_attention(q, cache, SegGroup(0, len(segs), 0, slot.numel(), ms), slot, kvlen, tables, bt, kvb, scale, nsplit)
+    want = TorchOps(DEV, F32).latent_attention(q, cache, None, slot, kvlen, None, bt, kvb, scale)
+    assert ops.status() == 0
+    return got.float(), want
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("lat,heads", [(64, 1), (64, 16), (128, 3), (192, 5), (256, 33), (320, 2), (384, 8), (448, 4), (512, 128), (512, 16),
+                                       (576, 3), (1024, 2)])
+def test_latent_attention_sizes(cops, dt, lat, heads):
+    for nsplit in (1, 3, 64):
+        segs = [(1, 1), (1, 63), (1, 64), (1, 65), (1, 400)]
+        got, want = attend_case(cops[dt], dt, lat, heads, segs, nsplit, 2.0 * lat ** -0.5, lat + heads)
+        assert torch.allclose(got, want, atol=2e-5 if dt == F32 else 2e-2, rtol=1e-2 if dt == BF else 1e-4), (nsplit, (got - want).abs().max())
+    segs = [(7, 130), (2, 2), (1, 321), (30, 96), (3, 66)]
+    got, want = attend_case(cops[dt], dt, lat, heads, segs, 8, 2.0 * lat ** -0.5, lat + heads)
+    assert torch.allclose(got, want, atol=2e-5 if dt == F32 else 2e-2, rtol=1e-2 if dt == BF else 1e-4)
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("at", [0, 1, 63, 64, 127, 128, 298, 299])
+@pytest.mark.parametrize("nsplit", [1, 4])
+def test_one_latent_stands_out(cops, dt, at, nsplit):
+    """One latent that all queries point at among hundreds: rows at or after it return it, rows before it do not see it."""
+    def plant(q, cache, bt, kvb):
+        q.fill_(1.0)
+        cache.mul_(0.1)
+        cache[int(bt[0, at // kvb]), at % kvb] = 2.0
+    got, want = attend_case(cops[dt], dt, 128, 6, [(3, 300)], nsplit, 0.5, 7, plant)
+    for j, kvlen in enumerate((298, 299, 300)):
+        assert bool((got[j] - 2.0).abs().max() < 1e-3) == (at < kvlen)
+        assert torch.allclose(got[j], want[j], atol=1e-2)
+
+
+def test_softmax_weights_keep_more_than_16_bit_operands(cops):
+    """Two keys whose weighted values nearly cancel: weights rounded to bf16 would be off by up to 2^-9 of the values."""
+    x, a0 = 0.3, 64.0
+
+    def plant(q, cache, bt, kvb):
+        q.zero_(); q[:, :, 0] = 1.0
+        cache.zero_()
+        cache[int(bt[0, 0]), 0, 0], cache[int(bt[0, 0]), 0, 1], cache[int(bt[0, 0]), 1, 1] = x, a0, -a0 * 1.34375
+    for seed in range(2):
+        got, want = attend_case(cops[BF], BF, 64, 4, [(1, 2)], 1, 1.0, seed, plant)
+        assert float((got[:, :, 1] - want[:, :, 1]).abs().max()) < a0 * 2.0 ** -12 and float(want[:, :, 1].abs().max()) < 0.5
+
+
+@pytest.mark.parametrize("hp,heads,lat,scale", [(64, 3, 64, 0.2), (128, 4, 512, 0.088), (256, 2, 576, 0.05), (64, 1, 192, 0.5)])
+def test_prompt_attention_expanded(cops, hp, heads, lat, scale):
+    """Prompt segments (a fresh one, one that continues a cached context off the page grid, one of 33 rows) against keys and
+    values written out in 32 bits from the same latents; values near cancelling keep their 32-bit weights."""
+    ops, r, kvb = cops[BF], gen(hp + heads), 64
+    segs = [(0, 0, 150), (1, 70, 90), (2, 127, 33)]
+    cache, bt = paged(lat, [p + n for _, p, n in segs], BF, hp)
+    T = sum(n for _, _, n in segs)
+    q = r(T, heads * hp, dt=BF)
+    kv_up = r(2 * heads * hp, lat, sc=lat ** -0.5, dt=BF)
+    d = LatentDims(heads, 64, lat, 64, lat, hp, scale, 0)
+    (g,) = seg_groups(segs, 3, T, 150, 32, bt, kvb, torch.device(DEV))
+    assert g.prompt
+    tables = (i32([0, 1, 2]), i32([0, 150, 240]), i32([150, 90, 33]), i32([0, 70, 127]))
+    out = torch.empty_like(q)
+    ops.latent_attention_prompt(q, ops.latent_rows(cache, g, kvb), kv_up, d, g, tables, kvb, out)
+    r0 = 0
+    for s, p, n in segs:
+        c = cache[bt[s, :(p + n + kvb - 1) // kvb].long()].reshape(-1, lat)[:p + n].float()
+        kv = (c @ kv_up.float().t()).to(BF).float()
+        k, v = kv[:, :heads * hp].reshape(-1, heads, hp), kv[:, heads * hp:].reshape(-1, heads, hp)
+        sc = torch.einsum("ihd,jhd->hij", q[r0:r0 + n].float().view(n, heads, hp), k) * scale
+        seen = torch.arange(p + n, device=DEV)[None, :] <= p + torch.arange(n, device=DEV)[:, None]
+        want = torch.einsum("hij,jhd->ihd", torch.softmax(sc.masked_fill(~seen, -math.inf), -1), v).reshape(n, -1)
+        assert torch.allclose(out[r0:r0 + n].float(), want, atol=1e-2, rtol=1e-2), (s, (out[r0:r0 + n].float() - want).abs().max())
+        r0 += n
+    assert ops.status() == 0
+
+
+@pytest.mark.parametrize("at", [0, 63, 64, 127, 128, 199])
+def test_prompt_attention_one_key_stands_out(cops, at):
+    ops, kvb, hp, lat = cops[BF], 64, 64, 64
+    cache, bt = paged(lat, [200], BF, at)
+    cache.mul_(0.1)
+    cache[int(bt[0, at // kvb]), at % kvb] = 2.0
+    kv_up = torch.cat([torch.eye(64), torch.eye(64)]).to(DEV, BF)
+    q = torch.ones(200, hp, dtype=BF, device=DEV)
+    d = LatentDims(1, 64, lat, 64, lat, hp, 0.5, 0)
+    (g,) = seg_groups([(0, 0, 200)], 1, 200, 200, 32, bt, kvb, torch.device(DEV))
+    out = ops.latent_attention_prompt(q, ops.latent_rows(cache, g, kvb), kv_up, d, g, (i32([0]), i32([0]), i32([200]), i32([0])), kvb,
+                                      torch.empty_like(q))
+    hit = (out.float() - 2.0).abs().amax(1) < 1e-2
+    assert bool(hit[at:].all()) and not bool(hit[:at].any())
+
+
+def test_prompt_attention_weights_keep_more_than_16_bit_operands(cops):
+    ops, hp = cops[BF], 64
+    cache, bt = paged(64, [64], BF, 3)
+    cache.zero_()
+    page = cache[int(bt[0, 0])]
+    page[0, 0], page[0, 1], page[1, 1] = 0.3, 64.0, -86.0
+    page[2:, 0] = -60.0                                          # later keys: no weight
+    kv_up = torch.cat([torch.eye(64), torch.eye(64)]).to(DEV, BF)
+    q = torch.zeros(40, hp, dtype=BF, device=DEV)
+    q[:, 0] = 1.0
+    d = LatentDims(1, 64, 64, 64, 64, hp, 1.0, 0)
+    (g,) = seg_groups([(0, 0, 40)], 1, 40, 40, 32, bt, 64, torch.device(DEV))
+    out = ops.latent_attention_prompt(q, ops.latent_rows(cache, g, 64), kv_up, d, g, (i32([0]), i32([0]), i32([40]), i32([0])), 64,
+                                      torch.empty_like(q))
+    p = torch.softmax(torch.tensor([float(page[0, 0]), 0.0], dtype=torch.float64), 0)
+    want = float(p[0] * 64.0 - p[1] * 86.0)
+    assert float((out[1:, 1].double() - want).abs().max()) < 64 * 2.0 ** -12 and abs(want) < 0.5
+
+
+@pytest.mark.parametrize("M,N,K", [(1, 7, 64), (5, 200, 320), (70, 131, 64), (300, 64, 1024)])
+def test_fp32_products(cops, M, N, K):
+    ops, r = cops[F32], gen(M * N)
+    x, w = r(M, K), r(N, K)
+    want = x.double() @ w.double().t()
+    assert float((ops.linear(x, w).double() - want).abs().max()) < 1e-4 * K ** 0.5
+    assert float((ops.linear(x, w, act="relu2").double() - plain.relu_squared(want)).abs().max()) < 2e-3 * K ** 0.5
+    xh, wh = r(M, 3, K + 64)[:, :, :K], r(3, N, K)
+    y = torch.full((M, 3, N + 5), 7.0, device=DEV)
+    ops.head_linear(xh, wh, out=y[:, :, :N])
+    assert float((y[:, :, :N].double() - torch.einsum("thk,hnk->thn", xh.double(), wh.double())).abs().max()) < 1e-4 * K ** 0.5
+    assert bool((y[:, :, N:] == 7.0).all())
+
+
+@pytest.mark.parametrize("M", [1, 2, 7, 8, 20, 33, 64, 65, 300])
+def test_squared_relu_epilogue_and_fp32_output_of_every_linear_kernel(cops, M):
+    ops, r = cops[BF], gen(M)
+    for N, K in ((192, 256), (1000, 640), (257, 64)):
+        x, w = r(M, K, dt=BF), r(N, K, sc=K ** -0.5, dt=BF)
+        want = x.float() @ w.float().t()
+        assert torch.allclose(ops.linear(x, w, act="relu2").float(), plain.relu_squared(want), atol=1e-2, rtol=1e-2)
+        assert torch.allclose(ops.linear(x, w, out_f32=True), want, atol=1e-4, rtol=1e-4)
+    assert ops.status() == 0
+
+
+@pytest.mark.parametrize("T", [1, 3, 8, 40, 200])
+@pytest.mark.parametrize("nh,N,K", [(3, 64, 192), (4, 64, 576), (2, 320, 320), (16, 128, 384)])
+def test_per_head_products_of_any_width(cops, T, nh, N, K):
+    ops, r = cops[BF], gen(T + K)
+    x, w = r(T, nh, K, dt=BF), r(nh, N, K, sc=K ** -0.5, dt=BF)
+    want = torch.einsum("thk,hnk->thn", x.float(), w.float())
+    assert torch.allclose(ops.head_linear(x, w).float(), want, atol=2e-2, rtol=1e-2)
+
+
+# ---- models --------------------------------------------------------------------------------------------------------------
+
+@pytest.fixture(scope="module")
+def models(tmp_path_factory):
+    root = tmp_path_factory.mktemp("zototar")
+    out = {}
+    for j, (name, cfg) in enumerate(CASES.items()):
+        w = weights(cfg, seed=j)
+        ids = tokens(cfg, 420, 11)
+        out[name] = (cfg, w, write(cfg, w, root / name), ids, plain.forward(cfg, w, ids)[0])
+    return out
+
+
+@pytest.mark.parametrize("compute", ["fp32", "bf16"])
+@pytest.mark.parametrize("name", list(CASES))
+@pytest.mark.parametrize("cuts", [[1000], [301, 1], [2], [63, 2, 1, 64, 33, 3, 65, 100, 2, 32]], ids=["whole", "decode", "pairs", "mixed"])
+def test_sequence_in_portions(ext, models, compute, name, cuts):
+    cfg, w, d, ids, want = models[name]
+    eng = engine(d, DEV, compute)
+    err = error(run_cuts(eng, ids, cuts), want)
+    eng.check()
+    assert err < LIM[compute], err
+
+
+@pytest.mark.parametrize("compute", ["fp32", "bf16"])
+def test_portions_and_batches_agree_beyond_rounding_only(ext, models, compute):
+    """Requests together (prompt portions beside decoded tokens, long segments beside short ones, a tight pool, slots and pages
+    that go round) against the plain rows of each."""
+    for name in ("grid", "ragged", "wide"):
+        cfg, w, d, ids, want = models[name]
+        eng = engine(d, DEV, compute, max_ctx=448, pool=1024)
+        seqs = {"a": (ids, want)}
+        for k, n in (("b", 90), ("c", 3), ("d", 200), ("e", 65), ("f", 1)):
+            s = tokens(cfg, n, 50 + n)
+            seqs[k] = (s, plain.forward(cfg, w, s)[0])
+        slot, at, got, free = {}, {k: 0 for k in seqs}, {k: [] for k in seqs}, [0, 1, 2, 3]
+        for st in (dict(a=100, b=2), dict(b=40, a=1, c=3), dict(a=50, d=1), dict(b=48, d=100, a=1), dict(a=200, d=2), dict(d=97, a=2, f=1),
+                   dict(e=64, a=33), dict(a=33, e=1)):
+            segs = []
+            for k, n in st.items():
+                if k not in slot:
+                    slot[k] = free.pop(0)
+                segs.append((k, Segment(slot[k], at[k], seqs[k][0][at[k]:at[k] + n], "all")))
+            lg, _, _ = eng.forward([s for _, s in segs], greedy=False)
+            lg, r = lg.float().cpu().clone(), 0
+            for k, s in segs:
+                got[k].append(lg[r:r + len(s.tokens)])
+                r += len(s.tokens)
+                at[k] += len(s.tokens)
+                if at[k] == len(seqs[k][0]):
+                    eng.reset_slot(slot[k])
+                    free.append(slot.pop(k))
+        eng.check()
+        assert eng.ex.pool.n_free == eng.ex.pool.n_blocks
+        for k in seqs:
+            e = error(torch.cat(got[k]), seqs[k][1])
+            assert e < LIM[compute], (name, k, e)
+
+
+def test_residual_rows_after_every_layer(ext, models):
+    cfg, w, d, ids, _ = models["ragged"]
+    _, after = plain.forward(cfg, w, ids[:50])
+    for compute, tol in (("fp32", 1e-4), ("bf16", 4e-2)):
+        eng = engine(d, DEV, compute)
+        eng.cfg.tap_layers[:] = range(len(cfg["layers"]))
+        eng.forward([Segment(0, 0, ids[:50], "none")])
+        for got, want in zip(eng.taps, after):
+            assert float((got.cpu().double() - want).pow(2).mean().sqrt()) < tol * float(want.pow(2).mean().sqrt())
+
+
+def test_greedy_generation_and_scheduler(ext, models):
+    cfg, w, d, _, _ = models["grid"]
+    prompts = [tokens(cfg, n, 30 + n) for n in (5, 70, 33, 1)]
+    prompts += [prompts[1] + tokens(cfg, 9, 77), (tokens(cfg, 6, 78) * 6)[:34]]
+    want = [plain.greedy(cfg, w, p, 8) for p in prompts]
+    assert engine(d, DEV, "fp32", slots=1, max_ctx=128).generate(prompts[1], 8) == want[1]
+    for spec, pool in ((0, 0), (0, 320), (4, 0)):
+        eng = engine(d, DEV, "fp32", slots=3, max_ctx=192, pool=pool, prefill_chunk=32)
+        sched = Scheduler(eng, SchedOptions(spec=spec, arrival_ms=0, share_min=32))
+        assert generate(sched, prompts, Sampling(max_tokens=8), snapshots=[[64] if len(p) > 64 else [] for p in prompts]) == want
+        assert generate(sched, [prompts[4]], Sampling(max_tokens=8), snapshots=[[64]])[0] == want[4]
+        eng.check()
+    # bf16: every generated token is the plain model's choice, or one that rounding cannot tell from it
+    eng = engine(d, DEV, "bf16", slots=3, max_ctx=192)
+    for p, out in zip(prompts, generate(Scheduler(eng, SchedOptions(arrival_ms=0)), prompts, Sampling(max_tokens=8))):
+        lg = plain.forward(cfg, w, p + out[:-1])[0][len(p) - 1:]
+        gap = lg.amax(-1) - lg.gather(1, torch.tensor(out)[:, None])[:, 0]
+        assert float(gap.max()) < 3 * LIM["bf16"] * float(lg.std())
+
+
+@pytest.mark.parametrize("fmt", ["nvfp4-a16", "nvfp4", "fp8-block"])
+def test_packed_weights(ext, tmp_path, fmt):
+    """Quantised projections (activation as a pass of its own) against the plain model with the same dequantised weights."""
+    cfg = config(256, 128, [layer(4, 64, 64, 128, 128, 512), layer(4, 64, 64, 128, 128, 256, kv_from=0)])
+    w = weights(cfg, gain=1.0)
+    eng = engine(write(cfg, w, tmp_path / "m"), DEV, "bf16", weight_dtype=fmt)
+    deq = lambda t: t.dense.float().cpu() if hasattr(t, "dense") else t.float().cpu()
+    w = dict(w, head=deq(eng.ex.w["lm_head"]))
+    for i in range(2):
+        for a, b in (("mix.o", "out_proj"), ("mlp.up", "up"), ("mlp.down", "down")):
+            w[f"l{i}.{a}"] = deq(eng.ex.w[f"l{i}.{b}"])
+        ip = deq(eng.ex.w[f"l{i}.in_proj"])
+        w[f"l{i}.mix.dq"] = ip[:128]
+        if i == 0:
+            w["l0.mix.dkv"] = ip[128:]
+    ids = tokens(cfg, 90, 1)
+    want = plain.forward(cfg, w, ids)[0]
+    for cuts in ([90], [70, 1], [5]):
+        err = error(run_cuts(eng, ids, cuts), want)
+        assert err < 0.1, (cuts, err)
+    eng.check()
