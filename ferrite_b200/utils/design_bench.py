@@ -1,0 +1,203 @@
+"""Two latent-attention designs side by side: Zototar (no positions, output norms on a 32-bit residual stream, latents shared by
+pairs of layers) and the dense MLA model of the same width, heads, latent and parameter count, with random weights.
+
+`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()` times every
+kernel of the first beside the kernel that does the same job for the second and gives both as fractions of their rooflines.
+Both print nothing and return plain dictionaries; `bench.py --design zototar` and `microbench latent` print them.
+"""
+from __future__ import annotations
+
+import statistics
+from typing import Dict, List
+
+import torch
+
+from ..config import EngineConfig, ModelConfig, zototar
+from .microbench import Timer, graph_time, peaks, rnd
+
+SIZES = {       # name: width, heads, query latent, feed-forward width, layers
+    "2k": (2048, 16, 768, 8192, 16),
+    "4k": (4096, 32, 1536, 16384, 8),
+    "7k": (7168, 128, 1536, 27648, 4),
+}
+KV_RANK, DIM, ROPE, VOCAB = 512, 128, 64, 65536
+
+
+def pair(size: str):
+    """(Zototar model, dense MLA model) of one size: the feed-forward of the second has three matrices instead of two."""
+    w, h, qr, ff, n = SIZES[size]
+    a = zototar(w, n, h, qr, KV_RANK, ff, VOCAB, DIM, DIM, name=f"zototar-{size}")
+    b = ModelConfig(name=f"mla-{size}", hidden=w, inter=(2 * ff // 3 + 127) // 128 * 128, n_layers=n, head_dim=DIM + ROPE, n_q=h,
+                    n_kv=h, rotary_dim=ROPE, rope_theta=1e4, attn_gate=False, vocab=VOCAB, tie_embeddings=False, kv_lora=KV_RANK,
+                    q_lora=qr, rope_head_dim=ROPE, nope_head_dim=DIM, v_head_dim=DIM)
+    return a, b
+
+
+def run_model(cfg: ModelConfig, ctx: int, prompts: List[int], streams: List[int], steps: int, warmup: int, dev) -> Dict:
+    from ..engine.engine import Engine
+    from ..engine.executor import Segment
+    n = max(streams)
+    eng = Engine(cfg, None, EngineConfig(n_slots=n, max_ctx=max(max(prompts), ctx + steps * 8 + 128), prefill_chunk=2048), device=str(dev))
+    g = torch.Generator().manual_seed(0)
+    toks = lambda k: torch.randint(0, cfg.vocab, (k,), generator=g).tolist()
+    out: Dict = {"params": cfg.param_count(), "cache_bytes_per_token": eng.ex.kv_block_bytes() // eng.ecfg.kv_block}
+    for p in prompts:
+        ids, times = toks(p), []
+        for rep in range(5):
+            eng.reset_slot(0)
+            torch.cuda.synchronize(dev)
+            e0, e1 = torch.cuda.Event(True), torch.cuda.Event(True)
+            e0.record()
+            eng.prefill(0, ids)
+            e1.record()
+            torch.cuda.synchronize(dev)
+            times.append(e0.elapsed_time(e1))
+        out[f"prefill_{p}_tok_s"] = round(p / statistics.median(times[2:]) * 1e3, 1)
+    ids = toks(ctx)
+    for s in range(n):
+        eng.reset_slot(s)
+        eng.prefill(s, ids)
+    for m in streams:
+        def step():
+            eng.forward([Segment(s, eng.slot_len[s], [ids[s]], "last") for s in range(m)])
+        for _ in range(max(3, warmup)):
+            step()
+        torch.cuda.synchronize(dev)
+        e0, e1 = torch.cuda.Event(True), torch.cuda.Event(True)
+        e0.record()
+        for _ in range(steps):
+            step()
+        e1.record()
+        torch.cuda.synchronize(dev)
+        ms = e0.elapsed_time(e1) / steps
+        out[f"decode_{m}_tok_s"], out[f"decode_{m}_ms"] = round(m / ms * 1e3, 1), round(ms, 4)
+    eng.check()
+    del eng
+    torch.cuda.empty_cache()
+    return out
+
+
+def models(sizes: List[str], steps: int, warmup: int, dev, ctx: int = 2048) -> Dict:
+    out = {}
+    for size in sizes:
+        a, b = pair(size)
+        ra = run_model(a, ctx, [2048, 8192], [1, 4, 16], steps, warmup, dev)
+        rb = run_model(b, ctx, [2048, 8192], [1, 4, 16], steps, warmup, dev)
+        out[size] = {"zototar": ra, "mla_dense": rb, "ratio": {k: round(ra[k] / rb[k], 3) for k in ra if k.endswith("tok_s")}}
+    return out
+
+
+def kernels(dev, heads: int = 32, width: int = 4096, ctx: int = 4096, prompt: int = 2048) -> List[Dict]:
+    """[{kernel, like, ms, like_ms, frac, like_frac}]: times in a CUDA graph of calls over buffers that together exceed L2."""
+    from ..models.weights import LatentDims
+    from ..ops.cuda_ops import CudaOps
+    from ..ops.latent import SegGroup, seg_groups
+    ops, t = CudaOps(dev), Timer(dev, 3, 20, flush=False)
+    hbm, tf, _ = peaks()
+    L, R, D, QR, kvb = KV_RANK, ROPE, DIM, 1536, 64
+    rows: List[Dict] = []
+
+    def timed(fn, nbytes: float, flops: float, bufs: int):
+        reps = max(4, min(40, int(-(-(400 << 20) // max(1, nbytes)))), bufs)
+        ms = graph_time(t, lambda: [fn(j % bufs) for j in range(reps)], reps)
+        return ms, max(nbytes / (hbm * 1e6), flops / (tf * 1e9)) / ms
+
+    def add(name, new, like_name, like):
+        (ms, fr), (lms, lfr) = timed(*new), timed(*like)
+        rows.append({"kernel": name, "ms": round(ms, 5), "frac": round(fr, 3), "like": like_name, "like_ms": round(lms, 5),
+                     "like_frac": round(lfr, 3)})
+
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    inv = torch.rand(R // 2, device=dev)
+    for m in (1, 4, 16):
+        nb = ctx // kvb
+        bufs = max(1, min(8, (400 << 20) // (m * ctx * L * 2)))
+        c0, c1 = [rnd(m * nb, kvb, L) for _ in range(bufs)], [rnd(m * nb, kvb, L + R) for _ in range(bufs)]
+        bt, slot = torch.arange(m * nb, dtype=torch.int32, device=dev).view(m, nb), torch.arange(m, dtype=torch.int32, device=dev)
+        kvlen, ones = torch.full((m,), ctx, dtype=torch.int32, device=dev), torch.ones(m, dtype=torch.int32, device=dev)
+        q0, q1 = rnd(m, heads, L), rnd(m, heads, L + R)
+        grp = SegGroup(0, m, 0, m, 1)
+        add(f"latent_mma + merge, {m} rows, {heads} heads, {ctx} keys",
+            (lambda j: ops.latent_attention(q0, c0[j], grp, slot, kvlen, (slot, slot, ones), bt, kvb, 0.088, 64), m * ctx * L * 2.0,
+             4.0 * m * heads * ctx * L, bufs), "mla_attn + combine",
+            (lambda j: ops.mla_attention(q1, c1[j], slot, kvlen, bt, kvb, heads, L, R, 0.07, nsplit=64), m * ctx * (L + R) * 2.0,
+             2.0 * m * heads * ctx * (2 * L + R), bufs))
+        del c0, c1
+    for m in (1, 16, prompt):
+        bufs = max(1, min(8, (400 << 20) // (m * width * 4)))
+        x0, y0 = [rnd(m, width, dtype=torch.float32) for _ in range(bufs)], [rnd(m, width, dtype=torch.float32) for _ in range(bufs)]
+        xb, yb = [rnd(m, width) for _ in range(bufs)], [rnd(m, width) for _ in range(bufs)]
+        w32, w16 = torch.ones(width, device=dev), rnd(width)
+        add(f"add_normed, {m} rows", (lambda j: ops.add_normed(x0[j], y0[j], w32, width, 1e-6), m * width * 14.0, 0.0, bufs),
+            "rmsnorm + residual", (lambda j: ops.rmsnorm(xb[j], w16, 1e-6, True, res=yb[j]), m * width * 8.0, 0.0, bufs))
+        add(f"norm_rows, {m} rows", (lambda j: ops.norm_rows(x0[j], None, w32, width, 1e-6), m * width * 6.0, 0.0, bufs),
+            "rmsnorm", (lambda j: ops.rmsnorm(xb[j], w16, 1e-6, True), m * width * 4.0, 0.0, bufs))
+        nb = max(1, m // kvb)
+        slot = torch.zeros(m, dtype=torch.int32, device=dev) if m > kvb else torch.arange(m, dtype=torch.int32, device=dev)
+        pos = torch.arange(m, dtype=torch.int32, device=dev) if m > kvb else torch.zeros(m, dtype=torch.int32, device=dev)
+        bt = torch.arange((1 if m > kvb else m) * nb, dtype=torch.int32, device=dev).view(-1, nb)
+        d = LatentDims(heads, QR, L, QR, L, D, 0.088, 0)
+        pb = 8 if m > kvb else 32
+        proj = [rnd(m, QR + L, dtype=torch.float32) for _ in range(pb)]
+        cl = torch.zeros(m * kvb if m <= kvb else m, L, dtype=torch.bfloat16, device=dev).view(-1, kvb, L)
+        cm = torch.zeros(cl.shape[0], kvb, L + R, dtype=torch.bfloat16, device=dev)
+        kva, qq, qa, qn, kn = [rnd(m, L + R) for _ in range(pb)], rnd(m, heads * (D + R)), [rnd(m, QR) for _ in range(pb)], rnd(QR), rnd(L)
+
+        def mla_norms(j):
+            ops.rmsnorm(qa[j], qn, 1e-6, True)
+            ops.mla_prep(qq, kva[j], kn, None, inv, slot, pos, bt, cm, kvb, heads, D, L, R, 1e-6, absorb=False)
+        add(f"latent_prep, {m} rows", (lambda j: ops.latent_prep(proj[j], d, w32[:QR], w32[:L], slot, pos, bt, cl, kvb, 1e-6),
+                                       m * (QR + L) * 6.0, 0.0, pb),
+            "rmsnorm + mla_prep", (mla_norms, m * (QR * 4.0 + (L + R) * 4.0 + heads * R * 4.0), 0.0, pb))
+        tab, gr = rnd(VOCAB, width), rnd(65522, width)
+        tok = [torch.randint(0, VOCAB, (m,), device=dev).to(torch.int32) for _ in range(8)]
+        tp = torch.zeros(cl.shape[0], kvb, dtype=torch.int32, device=dev)
+        add(f"embed_grams, {m} rows", (lambda j: ops.embed_grams(tab, gr, tok[j], slot, pos, bt, tp, kvb, 64.0, 65521, 31, 7),
+                                       m * width * 10.0, 0.0, 8), "embed", (lambda j: ops.embed(tab, tok[j]), m * width * 4.0, 0.0, 8))
+        del tab, gr, x0, y0, xb, yb
+    for m in (1, 16):
+        z = [rnd(m, 129280, dtype=torch.float32) for _ in range(8)]
+        add(f"softcap, {m} rows of 129280", (lambda j: ops.softcap(z[j], 30.0), m * 129280 * 8.0, 0.0, 8), "argmax",
+            (lambda j: ops.argmax(z[j]), m * 129280 * 4.0, 0.0, 8))
+    ff, inter = 4 * width, (8 * width // 3 + 127) // 128 * 128
+    for m in (1, 4, 16, prompt):
+        x, xw = rnd(m, width), m * width * 2.0
+        up, gu = [rnd(ff, width, scale=0.02) for _ in range(4)], [rnd(2 * inter, width, scale=0.02) for _ in range(4)]
+        add(f"linear + relu^2, {m} rows, {width} -> {ff}", (lambda j: ops.linear(x, up[j], act="relu2"), ff * width * 2.0 + xw + m * ff * 2.0,
+                                                            2.0 * m * ff * width, 4), "linear + SwiGLU",
+            (lambda j: ops.linear(x, gu[j], swiglu=True), inter * width * 4.0 + xw + m * inter * 2.0, 4.0 * m * inter * width, 4))
+        wo = [rnd(width, heads * D, scale=0.02) for _ in range(8)]
+        o, res = rnd(m, heads * D), rnd(m, width)
+        add(f"linear, fp32 sums, {m} rows, {heads * D} -> {width}",
+            (lambda j: ops.linear(o, wo[j], out_f32=True), width * heads * D * 2.0 + m * (heads * D * 2.0 + width * 4.0),
+             2.0 * m * width * heads * D, 8), "linear + residual",
+            (lambda j: ops.linear(o, wo[j], res=res), width * heads * D * 2.0 + m * (heads * D * 2.0 + width * 4.0), 2.0 * m * width * heads * D, 8))
+        del up, gu, wo
+    # prompt attention: expansion GEMM and flash kernel of one whole prompt
+    T, nb = prompt, prompt // kvb
+    perm = torch.randperm(nb, device=dev).to(torch.int32).view(1, nb)
+    c0, c1 = rnd(nb, kvb, L), rnd(nb, kvb, L + R)
+    kv_up, kv_b = rnd(2 * heads * D, L, scale=L ** -0.5), rnd(2 * heads * D, L, scale=L ** -0.5)
+    q0, q1, qabs = rnd(T, heads * D), rnd(T, heads * (D + R)), rnd(T, heads, L + R)
+    (grp,) = seg_groups([(0, 0, T)], 1, T, T, 32, perm, kvb, dev)
+    s0 = (i32([0]), i32([0]), i32([T]), i32([0]))
+    d = LatentDims(heads, QR, L, QR, L, D, 0.088, 0)
+    out = torch.empty_like(q0)
+    work = 2.0 * T * L * 2 * heads * D
+    tri = T * (T + 1) / 2.0
+    torch.cuda.synchronize(dev)
+    ms = t.run(lambda: ops.latent_attention_prompt(q0, ops.latent_rows(c0, grp, kvb), kv_up, d, grp, s0, kvb, out))
+    lms = t.run(lambda: ops.mla_attention_prefill(q1, qabs, c1, kv_b, [(0, 0, T)], s0[1], s0[2], s0[3], perm, kvb, heads, D, D, L, R))
+    fl, lfl = work + tri * heads * 4 * D, work + tri * heads * 2 * (2 * D + R)
+    rows.append({"kernel": f"prompt attention (gather, expansion GEMM, flash with 16-bit weight remainders), {T} rows", "ms": round(ms, 5),
+                 "frac": round(fl / (tf * 1e9) / ms, 3), "like": "mla prompt attention (gather, GEMM, packing, flash)",
+                 "like_ms": round(lms, 5), "like_frac": round(lfl / (tf * 1e9) / lms, 3)})
+    kv = ops.linear(ops.latent_rows(c0, grp, kvb), kv_up).view(-1, kvb, 2, heads, D)
+
+    def flash(exact):
+        return lambda j: ops.C.attn_prefill_tc(out, q0, kv[:, :, 0], kv[:, :, 1], q0, grp.own, s0[1], s0[2], s0[3], grp.table, kvb, T, heads,
+                                               heads, D, False, ops.status_word, scale=0.088, exact_p=exact)
+    add(f"flash, softmax weights as value + remainder, {T} rows, {heads} heads of {D}", (flash(True), 0.0, tri * heads * 4 * D, 1),
+        "flash, bf16 softmax weights", (flash(False), 0.0, tri * heads * 4 * D, 1))
+    assert ops.status() == 0
+    return rows

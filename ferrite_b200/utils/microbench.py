@@ -159,7 +159,9 @@ def graph_time(t, chain, reps):
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("what", choices=["gemv", "gemm", "layer", "attn_decode", "attn_prefill", "gdn", "moe", "exl3",
-                                     "head_linear", "ffn_fp4", "select"])
+                                     "head_linear", "ffn_fp4", "select", "latent"])
+    ap.add_argument("--heads", type=int, default=32, help="latent: heads")
+    ap.add_argument("--width", type=int, default=4096, help="latent: model width")
     ap.add_argument("--kv", default="bf16", help="attn_decode: cache form (bf16 | fp8 | int6 | int4)")
     ap.add_argument("--m", type=int, default=1)
     ap.add_argument("--n", type=int, default=5120)
@@ -254,6 +256,11 @@ def main():
             ms = graph_time(t, lambda: [ops.head_linear(x, W) for W in Ws], reps)
             report(f"head_linear rows{a.m} {nh} heads N{N} K{K} ({label})", ms, wbytes + a.m * nh * (N + K) * 2,
                    2.0 * a.m * nh * N * K)
+    elif a.what == "latent":
+        # the Zototar kernels beside the dense MLA model's, both as fractions of their rooflines
+        from .design_bench import kernels
+        for r in kernels(dev, a.heads, a.width, a.ctx):
+            print(json.dumps(r), flush=True)
     elif a.what == "ffn_fp4":
         # dense FFN block of the 27B model on prompt rows, NVFP4 weights and activations: gate|up + SwiGLU + down with the
         # activation re-quantised in the first GEMM's epilogue, against the same block through a bf16 activation
