@@ -266,39 +266,60 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
   if (nsplit > 1 && threadIdx.x == 0) { ml_part[pidx * 2] = M; ml_part[pidx * 2 + 1] = Ls; }
 }
 
-// merge of the splits in split order; grid (rows, heads)
+// Merge of the splits; grid (rows, heads). LG_GROUPS groups of 128 threads take every LG_GROUPS-th split each (all loads of a
+// group in flight together) and are added in group order, so the result does not depend on scheduling.
+constexpr int LG_GROUPS = 4;
+
 template <typename T>
-__global__ void __launch_bounds__(128) latent_merge_kernel(T* __restrict__ out, const float* __restrict__ o_part,
-                                                           const float* __restrict__ ml_part, int heads, int nsplit, int lat) {
+__global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __restrict__ out, const float* __restrict__ o_part,
+                                                                       const float* __restrict__ ml_part, int heads, int nsplit,
+                                                                       int lat) {
+  extern __shared__ float sf[];                            // [nsplit] factors, then [groups][lat] partial sums
+  __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   const size_t rh = (size_t)blockIdx.x * heads + blockIdx.y, pbase = rh * nsplit;
-  float M = -INFINITY;
-  for (int s = 0; s < nsplit; ++s) M = fmaxf(M, ml_part[(pbase + s) * 2]);
-  float Ls = 0.f;
-  for (int s = 0; s < nsplit; ++s) {
+  const int tid = threadIdx.x, grp = tid / 128, col = (tid % 128) * 4;
+  float M = -INFINITY, Ls = 0.f;
+  for (int s = tid; s < nsplit; s += blockDim.x) M = fmaxf(M, ml_part[(pbase + s) * 2]);
+  M = block_max(M, red);
+  for (int s = tid; s < nsplit; s += blockDim.x) {
     const float ms = ml_part[(pbase + s) * 2];
-    if (ms != -INFINITY) Ls += ml_part[(pbase + s) * 2 + 1] * exp2f(ms - M);
+    const float f = ms == -INFINITY ? 0.f : exp2f(ms - M);          // an empty split wrote no rows
+    sf[s] = f;
+    Ls += f == 0.f ? 0.f : ml_part[(pbase + s) * 2 + 1] * f;
   }
+  Ls = block_sum(Ls, red);                                 // (its barriers publish the factors)
   const float inv = Ls > 0.f ? 1.f / Ls : 0.f;
-  for (int d = threadIdx.x * 4; d < lat; d += blockDim.x * 4) {
+  float* sums = sf + nsplit;
+  for (int d = col; d < lat; d += 512) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < nsplit; ++s) {
-      const float ms = ml_part[(pbase + s) * 2];
-      if (ms == -INFINITY) continue;                       // an empty split wrote no rows
-      const float f = exp2f(ms - M);
+#pragma unroll 8
+    for (int s = grp; s < nsplit; s += LG_GROUPS) {
+      const float f = sf[s];
+      if (f == 0.f) continue;
       const float4 v = *reinterpret_cast<const float4*>(o_part + (pbase + s) * lat + d);
       acc.x = fmaf(v.x, f, acc.x); acc.y = fmaf(v.y, f, acc.y); acc.z = fmaf(v.z, f, acc.z); acc.w = fmaf(v.w, f, acc.w);
     }
-    acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
-    Elem<T>::store4(out + rh * lat + d, acc);
+    float* p = sums + grp * lat + d;
+    p[0] = acc.x; p[1] = acc.y; p[2] = acc.z; p[3] = acc.w;
   }
+  __syncthreads();
+  if (tid < lat / 4)
+    for (int d = tid * 4; d < lat; d += 512 * 4) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int g = 0; g < LG_GROUPS; ++g)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] += sums[g * lat + d + e];
+      Elem<T>::store4(out + rh * lat + d, make_float4(v[0] * inv, v[1] * inv, v[2] * inv, v[3] * inv));
+    }
 }
 
 // ---- attention over the cached latents, tensor cores ---------------------------------------------------------------------
 // bf16. The M dimension is (row of the segment, head): all of them read the same latents, so one pass over a key tile
 // serves 64 of them. grid (segments x M tiles, splits), 8 warps. Scores: warp = 16 M rows x 32 of the tile's 64 keys over the
-// whole latent. Values are the same shared-memory tile read transposed: warp = all 64 M rows x lat / 8 columns. The softmax
+// whole latent (16 keys when at most 32 M rows are in use, so that no warp idles). Values are the same shared-memory tile read transposed: warp = all 64 M rows x lat / 8 columns. The softmax
 // weights go through shared memory as a bf16 value plus its bf16 remainder, two products each, so they keep 16 bits of mantissa
 // instead of 8; scores, maxima, exponentials and row sums are 32-bit.
 constexpr int LM_M = 64, LM_KEYS = 64, LM_THREADS = 256, LM_LDP = LM_KEYS + 8;
@@ -316,15 +337,15 @@ __device__ __forceinline__ void lm_ldsm_t(uint32_t (&r)[4], const void* p) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
 }
 __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
 template <int NJ>
 struct Lm {
   static constexpr int LAT = NJ * 64, LD = LAT + 8;
-  static constexpr size_t SMEM = (size_t)(LM_M + 2 * LM_KEYS) * LD * 2 + (size_t)2 * LM_M * LM_LDP * 2 + 4 * LM_M * 4;
+  static constexpr size_t SMEM = (size_t)(LM_M + 2 * LM_KEYS) * LD * 2 + (size_t)2 * LM_M * LM_LDP * 2 + 6 * LM_M * 4;
 };
 
 template <int NJ>
@@ -339,8 +360,8 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [M][LD]
   __nv_bfloat16* sK = sQ + LM_M * LD;                                      // [2][KEYS][LD]
   __nv_bfloat16* sP = sK + 2 * LM_KEYS * LD;                               // [value | remainder][M][LDP]
-  float* smx = reinterpret_cast<float*>(sP + 2 * LM_M * LM_LDP);           // [2][M] maxima of the two key halves, then sums
-  float* sfac = smx + 2 * LM_M;                                            // [M] rescale factor of the tile
+  float* smx = reinterpret_cast<float*>(sP + 2 * LM_M * LM_LDP);           // [4][M] maxima of the key groups, then sums
+  float* sfac = smx + 4 * LM_M;                                            // [M] rescale factor of the tile
   float* sinv = sfac + LM_M;                                               // [M] 1 / row sum
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -369,20 +390,25 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
     const bool ok = m < valid_m;
     lm_cp16(sQ + m * LD + cc * 8, q + (flat0 + (ok ? m : 0)) * LAT + cc * 8, ok);
   }
-  auto load_tile = [&](int t0, int stage) {
+  auto load_tile = [&](int t0, int stage) {                  // a tile lies in one page: both start on multiples of 64 keys
+    const int blk = bt[t0 / kv_block];
+    if (blk < 0 && tid == 0) set_status(status, ST_BOUNDS);
+    const int live = blk < 0 ? 0 : min(LM_KEYS, hi - t0);
+    const __nv_bfloat16* src = cache + (blk < 0 ? 0 : ((size_t)blk * kv_block + t0 % kv_block) * LAT);
+    __nv_bfloat16* dst = sK + stage * LM_KEYS * LD;
+#pragma unroll 4
     for (int c = tid; c < LM_KEYS * CPR; c += LM_THREADS) {
-      const int r = c / CPR, cc = c % CPR, t = t0 + r;
-      bool ok = t < hi;
-      const int blk = ok ? bt[t / kv_block] : 0;
-      if (blk < 0) { ok = false; set_status(status, ST_BOUNDS); }
-      lm_cp16(sK + (stage * LM_KEYS + r) * LD + cc * 8,
-              cache + (ok ? ((size_t)blk * kv_block + t % kv_block) * LAT + cc * 8 : 0), ok);
+      const int r = c / CPR, cc = c % CPR;
+      lm_cp16(dst + r * LD + cc * 8, src + (r < live ? c * 8 : 0), r < live);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load_tile(lo, 0);
 
-  const int mw = warp & 3, nw = warp >> 2;                   // score role
+  // score role: 16 M rows at mw * 16, keys [key0, key0 + 16 npairs) of the tile
+  const bool few = valid_m <= 32;
+  const int mw = few ? warp & 1 : warp & 3, nw = few ? warp >> 1 : warp >> 2, kgroups = few ? 4 : 2;
+  const int npairs = few ? 1 : 2, key0 = nw * 16 * npairs;
   const int r_lo = mw * 16 + lane / 4;                       // this thread's two M rows: r_lo, r_lo + 8
   int kvl[2];
 #pragma unroll
@@ -410,24 +436,35 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
     for (int i = 0; i < 4; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
     float mx[2] = {-INFINITY, -INFINITY};
     if (score_on) {
+      // fragments are loaded one k step ahead of the products
+      const __nv_bfloat16* pa = sQ + (mw * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8;
+      const __nv_bfloat16* pb = K + (key0 + (lane >> 4) * 8 + (lane & 7)) * LD + ((lane >> 3) & 1) * 8;
+      uint32_t a[2][4], b[2][2][4];
+      lm_ldsm(a[0], pa);
+      lm_ldsm(b[0][0], pb);
+      if (!few) lm_ldsm(b[0][1], pb + 16 * LD);
 #pragma unroll 4
       for (int ks = 0; ks < LAT / 16; ++ks) {
-        uint32_t a[4], b[4];
-        lm_ldsm(a, sQ + (mw * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          lm_ldsm(b, K + (nw * 32 + np * 16 + (lane >> 4) * 8 + (lane & 7)) * LD + ks * 16 + ((lane >> 3) & 1) * 8);
-          lm_mma(s[np * 2], a, b[0], b[1]);
-          lm_mma(s[np * 2 + 1], a, b[2], b[3]);
+        const int cur = ks & 1;
+        if (ks + 1 < LAT / 16) {
+          lm_ldsm(a[cur ^ 1], pa + (ks + 1) * 16);
+          lm_ldsm(b[cur ^ 1][0], pb + (ks + 1) * 16);
+          if (!few) lm_ldsm(b[cur ^ 1][1], pb + 16 * LD + (ks + 1) * 16);
+        }
+        lm_mma(s[0], a[cur], b[cur][0][0], b[cur][0][1]);
+        lm_mma(s[1], a[cur], b[cur][0][2], b[cur][0][3]);
+        if (!few) {
+          lm_mma(s[2], a[cur], b[cur][1][0], b[cur][1][1]);
+          lm_mma(s[3], a[cur], b[cur][1][2], b[cur][1][3]);
         }
       }
-      const int kbase = lo + tile * LM_KEYS + nw * 32 + (lane & 3) * 2;
+      const int kbase = lo + tile * LM_KEYS + key0 + (lane & 3) * 2;
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = kbase + nt * 8 + (e & 1), h = e >> 1;
-          const float v = (t < kvl[h] && t < hi) ? s[nt][e] * scale_log2 : -INFINITY;
+          const float v = (nt < 2 * npairs && t < kvl[h] && t < hi) ? s[nt][e] * scale_log2 : -INFINITY;
           s[nt][e] = v;
           mx[h] = fmaxf(mx[h], v);
         }
@@ -443,17 +480,19 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         const int r = r_lo + 8 * h;
-        const float mn = fmaxf(mrow[h], fmaxf(smx[r], smx[LM_M + r]));
+        float mn = fmaxf(mrow[h], fmaxf(smx[r], smx[LM_M + r]));
+        if (few) mn = fmaxf(mn, fmaxf(smx[2 * LM_M + r], smx[3 * LM_M + r]));
         const float f = mn == -INFINITY ? 1.f : exp2f(mrow[h] - mn);
         mrow[h] = mn;
         float ls = 0.f;
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
+          if (nt >= 2 * npairs) break;
           const float p0 = mn == -INFINITY ? 0.f : exp2f(s[nt][2 * h] - mn);
           const float p1 = mn == -INFINITY ? 0.f : exp2f(s[nt][2 * h + 1] - mn);
           ls += p0 + p1;
           const uint32_t v = pack_bf2(p0, p1);
-          const int at = r * LM_LDP + nw * 32 + nt * 8 + (lane & 3) * 2;
+          const int at = r * LM_LDP + key0 + nt * 8 + (lane & 3) * 2;
           *reinterpret_cast<uint32_t*>(sP + at) = v;
           *reinterpret_cast<uint32_t*>(sP + LM_M * LM_LDP + at) = pack_bf2(p0 - bf_lo(v), p1 - bf_hi(v));
         }
@@ -506,7 +545,8 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
     for (int h = 0; h < 2; ++h) {
       const int r = r_lo + 8 * h;
       if (r >= valid_m) continue;
-      const float l = smx[r] + smx[LM_M + r];
+      float l = 0.f;
+      for (int g = 0; g < kgroups; ++g) l += smx[g * LM_M + r];
       if (nsplit == 1) sinv[r] = l > 0.f ? 1.f / l : 0.f;
       else {
         float* ml = ml_part + ((flat0 + r) * nsplit + split) * 2;
@@ -640,7 +680,8 @@ extern "C" int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaS
 
 template <typename T>
 static int latent_merge(void* out, const float* o_part, const float* ml_part, int rows, int heads, int nsplit, int lat, cudaStream_t s) {
-  return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128), 0, s, (T*)out, o_part, ml_part, heads, nsplit, lat);
+  return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128 * LG_GROUPS), (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out,
+                         o_part, ml_part, heads, nsplit, lat);
 }
 
 template <typename T>
@@ -667,7 +708,7 @@ extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const vo
                               const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat,
                               int nsplit, float scale, int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 65535) return -1;
+  if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
   const float sl = scale * 1.4426950408889634f;
   return f32 ? latent_attn<float>(out, o_part, ml_part, q, cache, row_slot, row_kvlen, block_table, max_blocks, kv_block, rows, heads,
                                   lat, nsplit, sl, status, s)
@@ -675,15 +716,15 @@ extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const vo
                                  lat, nsplit, sl, status, s);
 }
 
-// The same on tensor cores for bf16 and lat <= 512 (-20 otherwise). Rows come in segments (consecutive rows of one slot);
+// The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in segments (consecutive rows of one slot);
 // seg_row0 counts the rows of the step, of which q / out / row_kvlen hold those from row_base on.
 extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
                              const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen,
                              const int* block_table, int max_blocks, int kv_block, int rows, int row_base, int heads, int lat,
                              int nsplit, float scale, int* status, cudaStream_t s) {
   if (rows <= 0 || nseg <= 0) return 0;
-  if (lat % 64 || lat > 512) return -20;
-  if (nsplit < 1 || nsplit > 65535) return -1;
+  if (lat % 64 || lat > 512 || kv_block % LM_KEYS) return -20;
+  if (nsplit < 1 || nsplit > 4096) return -1;
   const int tps = (max_rows * heads + LM_M - 1) / LM_M;
   const dim3 grid(nseg * tps, nsplit);
   const float sl = scale * 1.4426950408889634f;

@@ -120,11 +120,11 @@ class CudaLatent:
     def latent_attention(self, qabs, cache, group, slot, kvlen, segs, block_table, kv_block, scale, nsplit=1):
         """Rows of one slot form a segment (`segs` = slots, first rows, row counts), so its rows and heads share every pass over
         the latents on the tensor cores; fp32 and latents wider than 512 take the CUDA-core kernel. `nsplit` bounds the key
-        splits; what is left of it is what fills the GPU about twice."""
+        splits; what is left of it is what fills the GPU."""
         rows, heads, lat = qabs.shape
         mma = qabs.dtype == torch.bfloat16 and lat <= 512
         ctas = rows * heads if not mma else max(1, (group.seg_hi - group.seg_lo) * ((group.max_rows * heads + 63) // 64))
-        nsplit = max(1, min(nsplit, (2 if mma else 8) * self.sm_count // ctas))
+        nsplit = max(1, min(nsplit, (8 if not mma else 2 if lat <= 192 else 1) * self.sm_count // ctas))     # (wide latents: one CTA per SM)
         out = self.empty(rows, heads, lat, dtype=qabs.dtype, device=self.device)
         o_part = ml_part = None
         if nsplit > 1:
