@@ -414,7 +414,7 @@ def cmd_selftest(a) -> int:
     ids = torch.randint(1, full.vocab, (48,), generator=g).tolist()
     checks = {}
     if a.model == "" and full.n_layers <= 12 and full.hidden <= 512:
-        ref = RefModel(full, init_weights(full, seed=a.seed))
+        ref = RefModel(full, init_weights(full, seed=a.seed, dtype=eng.dtype, device=eng.device))     # the engine's own draw
         want = ref.forward(ids, ref.new_state())
         want = want[0] if isinstance(want, tuple) else want
         got = torch.cat([scheduled_logits(eng, ids[:40], 32, "plain")] +

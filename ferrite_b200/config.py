@@ -218,7 +218,7 @@ class ModelConfig:
 # ---- architectures by the name their config.json carries ------------------------------------------------------------
 
 def zototar_config(v: dict) -> ModelConfig:
-    """A Zototar config.json: latent attention without positions (latents optionally shared between layers), norms on the
+    """A Zototar config.json: position-free latent attention (latents optionally shared between layers), norms on the
     sublayers' outputs, squared-relu feed-forwards, a hashed bigram embedding beside the token's, softcapped logits."""
     layers: List[LayerSpec] = []
     for i, e in enumerate(v["layers"]):

@@ -407,7 +407,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   dim3 grid((max_rows + FT_BQ - 1) / FT_BQ, nq, nseg);
-  const float scale_log2 = 1.4426950408889634f * (scale > 0.f ? scale : 1.f / sqrtf((float)hd));
+  const float scale_log2 = 1.4426950408889634f * (scale != 0.f ? scale : 1.f / sqrtf((float)hd));
 #define FB_FT(HDV, PXV)                                                                                                 \
   {                                                                                                                \
     const size_t smem = (size_t)(FT_BQ + ((HDV == 256 ? 3 : 4) + (HDV == 256 ? 2 : 3)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \

@@ -1,4 +1,4 @@
-// Kernels of the models whose layers are listed one by one: latent attention without positions, RMSNorm on the sublayers'
+// Kernels of the models whose layers are listed one by one: position-free latent attention, RMSNorm on the sublayers'
 // outputs over a 32-bit residual stream, a hashed bigram embedding, softcapped logits.
 //
 //   embed_grams    x = table[token] * scale + grams[(prev * mul_prev + token * mul_cur) mod buckets] in 32 bits. The token of
@@ -319,9 +319,10 @@ __global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __rest
 // ---- attention over the cached latents, tensor cores ---------------------------------------------------------------------
 // bf16. The M dimension is (row of the segment, head): all of them read the same latents, so one pass over a key tile
 // serves 64 of them. grid (segments x M tiles, splits), 8 warps. Scores: warp = 16 M rows x 32 of the tile's 64 keys over the
-// whole latent (16 keys when at most 32 M rows are in use, so that no warp idles). Values are the same shared-memory tile read transposed: warp = all 64 M rows x lat / 8 columns. The softmax
-// weights go through shared memory as a bf16 value plus its bf16 remainder, two products each, so they keep 16 bits of mantissa
-// instead of 8; scores, maxima, exponentials and row sums are 32-bit.
+// whole latent (16 keys when at most 32 M rows are in use, so that no warp idles). Values are the same shared-memory tile read
+// transposed: warp = all 64 M rows x lat / 8 columns. The softmax weights go through shared memory as a bf16 value plus its bf16
+// remainder, two products each, so they keep 16 bits of mantissa instead of 8; scores, maxima, exponentials and row sums are
+// 32-bit.
 constexpr int LM_M = 64, LM_KEYS = 64, LM_THREADS = 256, LM_LDP = LM_KEYS + 8;
 
 __device__ __forceinline__ void lm_cp16(void* smem, const void* gmem, bool valid) {
@@ -680,8 +681,8 @@ extern "C" int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaS
 
 template <typename T>
 static int latent_merge(void* out, const float* o_part, const float* ml_part, int rows, int heads, int nsplit, int lat, cudaStream_t s) {
-  return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128 * LG_GROUPS), (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out,
-                         o_part, ml_part, heads, nsplit, lat);
+  return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128 * LG_GROUPS),
+                         (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out, o_part, ml_part, heads, nsplit, lat);
 }
 
 template <typename T>
@@ -716,8 +717,8 @@ extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const vo
                                  lat, nsplit, sl, status, s);
 }
 
-// The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in segments (consecutive rows of one slot);
-// seg_row0 counts the rows of the step, of which q / out / row_kvlen hold those from row_base on.
+// The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in
+// segments (consecutive rows of one slot); seg_row0 counts the rows of the step, of which q / out / row_kvlen hold those from row_base on.
 extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
                              const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen,
                              const int* block_table, int max_blocks, int kv_block, int rows, int row_base, int heads, int lat,

@@ -42,8 +42,9 @@ class Engine:
         on_gpu = self.device.type == "cuda"
         if self.ecfg.compute_dtype not in ("bf16", "fp32"):
             raise ValueError(f"compute_dtype {self.ecfg.compute_dtype!r}: expected bf16 or fp32")
-        if self.ecfg.compute_dtype == "fp32" and on_gpu and (not cfg.layers or self.ecfg.weight_dtype != "bf16"):
-            raise ValueError("compute_dtype fp32 on a GPU: models of listed layers with unpacked weights only")
+        if self.ecfg.compute_dtype == "fp32" and on_gpu and (
+                not cfg.layers or self.ecfg.weight_dtype != "bf16" or (tp is not None and tp.world > 1)):
+            raise ValueError("compute_dtype fp32 on a GPU: models of listed layers with unpacked weights on one GPU only")
         if cfg.layers and self.ecfg.kv_dtype != "bf16":
             raise ValueError(f"kv_dtype {self.ecfg.kv_dtype!r}: latent caches are kept in the compute dtype")
         self.dtype = torch.bfloat16 if on_gpu and self.ecfg.compute_dtype == "bf16" else torch.float32

@@ -192,7 +192,7 @@ class RefModel:
         return w[p + "out_proj"] @ o.reshape(-1)
 
     def _latent(self, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
-        """Latent attention without positions; a layer with `kv_from` reads the rows that layer appended for this token."""
+        """Position-free latent attention; a layer with `kv_from` reads the rows that layer appended for this token."""
         l, w, p, eps = self.cfg.layers[i], self.w, f"l{i}.", self.cfg.eps
         q = (w[p + "q_b"] @ rmsnorm(w[p + "q_a"] @ x, w[p + "q_a_norm"], eps, False)).view(l.heads, l.dim)
         if l.kv_from is None:

@@ -1,4 +1,4 @@
-"""Ops of the models whose layers are listed one by one: latent attention without positions, norms on the sublayers'
+"""Ops of the models whose layers are listed one by one: position-free latent attention, norms on the sublayers'
 outputs over a 32-bit residual stream, hashed bigram embeddings, softcapped logits. `TorchLatent` states each op in plain
 PyTorch for the fp32 CPU engine, `CudaLatent` runs the kernels of `csrc/latent.cu` and the tcgen05 prompt attention; both have
 the same signatures and work on the same paged caches.
@@ -30,29 +30,29 @@ class SegGroup:
     own: Optional[torch.Tensor] = None
 
 
-def _prev_tokens(tok, slot, pos, block_table, tok_pages, kv_block) -> List[int]:
+def _prev_tokens(ids, row_slot, row_pos, block_table, tok_pages, kv_block) -> List[int]:
     """Token before every row (-1 at a sequence's start): the row before it in the step, or the cached one."""
     out = []
-    for r in range(tok.numel()):
-        p, s = int(pos[r]), int(slot[r])
+    for r in range(ids.numel()):
+        p, s = int(row_pos[r]), int(row_slot[r])
         if p == 0:
             out.append(-1)
-        elif r > 0 and int(slot[r - 1]) == s and int(pos[r - 1]) == p - 1:
-            out.append(int(tok[r - 1]))
+        elif r > 0 and int(row_slot[r - 1]) == s and int(row_pos[r - 1]) == p - 1:
+            out.append(int(ids[r - 1]))
         else:
             out.append(int(tok_pages[int(block_table[s, (p - 1) // kv_block]), (p - 1) % kv_block]))
     return out
 
 
 class TorchLatent:
-    def embed_grams(self, table, grams, tok, slot, pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
+    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
         """Scaled token embedding plus the hashed bigram's row: (x fp32 [T, width], the same rows as GEMM operand)."""
-        x = table[tok.long()].float() * scale
+        x = table[ids.long()].float() * scale
         if grams is not None:
-            prev = _prev_tokens(tok, slot, pos, block_table, tok_pages, kv_block)
-            rows = [buckets if p < 0 else (p * mul_prev + int(t) * mul_cur) % buckets for p, t in zip(prev, tok)]
+            prev = _prev_tokens(ids, row_slot, row_pos, block_table, tok_pages, kv_block)
+            rows = [buckets if p < 0 else (p * mul_prev + int(t) * mul_cur) % buckets for p, t in zip(prev, ids)]
             x = x + grams[torch.tensor(rows, dtype=torch.long, device=x.device)].float()
-            tok_pages[block_table[slot.long(), pos.long() // kv_block].long(), pos.long() % kv_block] = tok.to(tok_pages.dtype)
+            tok_pages[block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block] = ids.to(tok_pages.dtype)
         return x, x.to(self.dtype)
 
     @staticmethod
@@ -68,19 +68,19 @@ class TorchLatent:
     def norm_rows(self, x, idx, w, width, eps):
         return self._rms(x if idx is None else x[idx.long()], w, width, eps).to(self.dtype)
 
-    def latent_prep(self, proj, d, q_norm, kv_norm, slot, pos, block_table, cache, kv_block, eps):
+    def latent_prep(self, proj, d, q_norm, kv_norm, row_slot, row_pos, block_table, cache, kv_block, eps):
         """Both latents of a token from the fused projection: returns the normalised query latent, writes the normalised key /
         value latent into its page (`kv_norm` None: the layer reads another layer's)."""
         if kv_norm is not None:
             c = self._rms(proj[:, d.qr:], kv_norm, d.kv_rank, eps)
-            cache[block_table[slot.long(), pos.long() // kv_block].long(), pos.long() % kv_block] = c.to(cache.dtype)
+            cache[block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block] = c.to(cache.dtype)
         return self._rms(proj[:, :d.qr], q_norm, d.q_rank, eps).to(self.dtype)
 
-    def latent_attention(self, qabs, cache, group, slot, kvlen, segs, block_table, kv_block, scale, nsplit=1):
+    def latent_attention(self, qabs, cache, group, row_slot, row_kvlen, segs, block_table, kv_block, scale, nsplit=1):
         """Every head attends the cached latents: qabs [rows, heads, lat] of the group's rows -> [rows, heads, lat]."""
         out = torch.zeros(qabs.shape, dtype=torch.float32, device=qabs.device)
         for r in range(qabs.shape[0]):
-            n, s = int(kvlen[r]), int(slot[r])
+            n, s = int(row_kvlen[r]), int(row_slot[r])
             keys = cache[block_table[s, :(n + kv_block - 1) // kv_block].long()].reshape(-1, qabs.shape[2])[:n].float()
             out[r] = torch.softmax((qabs[r].float() @ keys.t()) * scale, -1) @ keys
         return out.to(self.dtype)
@@ -90,11 +90,11 @@ class TorchLatent:
 
 
 class CudaLatent:
-    def embed_grams(self, table, grams, tok, slot, pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
-        x = self.empty(tok.numel(), table.shape[1], dtype=torch.float32, device=self.device)
+    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
+        x = self.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=self.device)
         xb = None if self.dtype == torch.float32 else self.empty(*x.shape, dtype=self.dtype, device=self.device)
         self.launches += 1
-        self.C.embed_grams(x, xb, table, grams, tok, slot, pos, block_table, kv_block, tok_pages, scale, buckets, mul_prev, mul_cur,
+        self.C.embed_grams(x, xb, table, grams, ids, row_slot, row_pos, block_table, kv_block, tok_pages, scale, buckets, mul_prev, mul_cur,
                            self.status_word)
         return x, (x if xb is None else xb)
 
@@ -110,31 +110,32 @@ class CudaLatent:
         self.C.norm_rows(out, x, idx, w, width, eps)
         return out
 
-    def latent_prep(self, proj, d, q_norm, kv_norm, slot, pos, block_table, cache, kv_block, eps):
+    def latent_prep(self, proj, d, q_norm, kv_norm, row_slot, row_pos, block_table, cache, kv_block, eps):
         cq = self.empty(proj.shape[0], d.qr, dtype=self.dtype, device=self.device)
         self.launches += 1
-        self.C.latent_prep(cq, cache, proj, q_norm, kv_norm, slot, pos, block_table, kv_block, d.q_rank, d.kv_rank, eps,
+        self.C.latent_prep(cq, cache, proj, q_norm, kv_norm, row_slot, row_pos, block_table, kv_block, d.q_rank, d.kv_rank, eps,
                            self.status_word)
         return cq
 
-    def latent_attention(self, qabs, cache, group, slot, kvlen, segs, block_table, kv_block, scale, nsplit=1):
+    def latent_attention(self, qabs, cache, group, row_slot, row_kvlen, segs, block_table, kv_block, scale, nsplit=1):
         """Rows of one slot form a segment (`segs` = slots, first rows, row counts), so its rows and heads share every pass over
         the latents on the tensor cores; fp32 and latents wider than 512 take the CUDA-core kernel. `nsplit` bounds the key
         splits; what is left of it is what fills the GPU."""
         rows, heads, lat = qabs.shape
         mma = qabs.dtype == torch.bfloat16 and lat <= 512
         ctas = rows * heads if not mma else max(1, (group.seg_hi - group.seg_lo) * ((group.max_rows * heads + 63) // 64))
-        nsplit = max(1, min(nsplit, (8 if not mma else 2 if lat <= 192 else 1) * self.sm_count // ctas))     # (wide latents: one CTA per SM)
+        per_sm = 8 if not mma else 2 if lat <= 192 else 1          # CTAs; a tile of wide latents fills an SM's shared memory
+        nsplit = max(1, min(nsplit, per_sm * self.sm_count // ctas))
         out = self.empty(rows, heads, lat, dtype=qabs.dtype, device=self.device)
         o_part = ml_part = None
         if nsplit > 1:
             o_part = self.empty(rows * heads * nsplit * lat, dtype=torch.float32, device=self.device)
             ml_part = self.empty(rows * heads * nsplit * 2, dtype=torch.float32, device=self.device)
         self.launches += 1 if nsplit == 1 else 2
-        if mma and self.C.latent_mma(out, o_part, ml_part, qabs, cache, segs[0], segs[1], segs[2], group.max_rows, kvlen,
+        if mma and self.C.latent_mma(out, o_part, ml_part, qabs, cache, segs[0], segs[1], segs[2], group.max_rows, row_kvlen,
                                      block_table, kv_block, group.row_lo, nsplit, scale, self.status_word) == 0:
             return out
-        self.C.latent_attn(out, o_part, ml_part, qabs, cache, slot, kvlen, block_table, kv_block, nsplit, scale, self.status_word)
+        self.C.latent_attn(out, o_part, ml_part, qabs, cache, row_slot, row_kvlen, block_table, kv_block, nsplit, scale, self.status_word)
         return out
 
     def latent_rows(self, cache, group, kv_block):

@@ -2,18 +2,17 @@
 
     trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N [--device cuda|cpu]
 
-Nothing is sampled. The trace's steps run through the engine the server and the command line use (`Engine.forward` over
-segments, its paged cache and slots), so a recorded schedule (portions of prompts beside single decoded tokens, requests that
-pause and go on) can be repeated and its logits compared between builds, schedules or precisions. A step is one JSON line on
-standard input:
+Logits only: every token comes from the trace. Steps go through the engine that the server and the command line use
+(`Engine.forward` over segments, its paged cache and slots), so a recorded schedule (portions of prompts beside single decoded tokens,
+requests that pause and go on) can be repeated and its logits compared between builds, schedules or precisions. Standard input holds
+one JSON object per line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "q", "tokens": [11, 4], "want": [1]}, {"id": "p", "tokens": [9], "want": []}], "end": ["p"]}
 
-`entries`: each request's next tokens and the places among them whose logits are wanted; a request is admitted at its first
-entry. `end`: requests that are finished after the step; their pages and slot are given back. Steps with wanted logits write
-DIR/<step>.f32 (little-endian fp32 [wanted, vocab], in the order of the entries); every step prints `done <step>`.
-
-`--max-tokens` sizes the page pool: the most tokens live requests hold at any time, each rounded up to whole pages of 64.
+An entry feeds a request its next tokens and names the ones (by place in `tokens`) whose logits to write; a request takes a slot with
+its first entry. Requests listed under `end` give back their pages and slot when the step is done. Wanted logits go to
+DIR/<step>.f32 (little-endian fp32 rows of the vocabulary, entries in order, places in order); after each step `done <step>` is
+printed. `--max-tokens` is the size of the page pool in tokens, counted in whole pages of 64 per request.
 """
 from __future__ import annotations
 

@@ -37,7 +37,7 @@ def _limits(ex) -> Dict[str, Tuple[int, int, str]]:
 
 # (op name, parameter) pairs whose limit depends on the op rather than on the parameter's name
 def _special(ex, op: str, param: str, bound: Dict[str, Any]) -> Optional[Tuple[int, int, str]]:
-    if op == "embed" and param == "ids":
+    if op in ("embed", "embed_grams") and param == "ids":
         return 0, int(bound["table"].shape[0]), "rows of the embedding table"
     if op in ("moe_experts",) and param == "ids":
         return 0, max(1, ex.full_cfg.n_experts) + 1, "experts (+ the shared expert's stack entry)"
