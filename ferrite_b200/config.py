@@ -20,7 +20,9 @@ class LayerSpec:
     """One layer of a model that lists its layers one by one (`ModelConfig.layers`): the mixer, its sizes and the
     feed-forward behind it. Layers of one model may differ in all of them."""
 
-    mixer: str = "latent"           # attention over a cached low-rank latent, no positions
+    # "latent": attention over a cached low-rank latent, no positions. "gqa": grouped-query attention over cached keys and
+    # values. "cdelta": gated delta rule with one decay per key channel (recurrent state, no cache)
+    mixer: str = "latent"
     heads: int = 1
     dim: int = 0                    # query / key width of a head
     vdim: int = 0                   # value width of a head
@@ -29,7 +31,32 @@ class LayerSpec:
     scale: float = 1.0              # scores are (q . k) * scale
     kv_from: Optional[int] = None   # use the latents that this (earlier) layer caches instead of own ones
     ff: int = 0                     # feed-forward width, 0 = the layer has none
-    act: str = "relu2"              # its activation
+    act: str = "relu2"              # its activation; "swiglu": silu(gate) * up
+    kv_heads: int = 0               # gqa, cdelta: key / value (cdelta: query / key) heads, each serving heads / kv_heads heads
+    bias: bool = False              # gqa: biases on the query, key and output projections
+    sink: bool = False              # gqa: a learned number per head in every softmax denominator
+    key_values: bool = False        # gqa: the values are the projected keys, before rotation and norm
+    qk_norm: bool = False           # gqa: queries and keys divided by their root mean square after the rotation
+    rot_dims: int = 0               # gqa: rotated columns of a head, pairs (0, 1), (2, 3), ...
+    rot_base: float = 1e4
+    rot_scaling: Optional[dict] = None   # long wavelengths stretched: factor, low, high, original
+    conv: int = 0                   # cdelta: taps of the short convolutions
+    decay_rank: int = 0             # cdelta: width between the two decay projections (0: the checkpoint says)
+    gate_rank: int = 0              # cdelta: ... and between the two output gate projections
+
+    @property
+    def cached(self) -> bool:
+        """The layer keeps rows of its own in the page pool."""
+        return self.mixer != "cdelta" and self.kv_from is None
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer. Looped layers run several times with the same weights; every run has its own cache or state."""
+
+    index: int                      # place in the order of execution: names the run's cache or state
+    layer: int                      # whose weights
+    enter: Optional[int] = None     # this run opens pass number `enter` of the loop
 
 
 @dataclass
@@ -77,6 +104,10 @@ class ModelConfig:
     # ---- layers listed one by one (they replace the pattern fields above) ----
     layers: List[LayerSpec] = field(default_factory=list)
     out_norm: bool = False          # x + norm(f(x)): norms on the sublayers' outputs, a 32-bit residual stream, plain norm weights
+    pre_norm: bool = False          # ... and norms on the sublayers' inputs as well: x + norm(f(norm(x)))
+    residual_mult: float = 1.0      # x + residual_mult * norm(f(..))
+    loop: Optional[List[int]] = None     # [start, stop, times]: layers start .. stop - 1 run `times` times in a row
+    logit_scale: float = 1.0
     embed_scale: float = 1.0
     gram_buckets: int = 0           # hashed bigram embedding: rows of the table besides the one for a sequence's first token
     gram_mul_prev: int = 0
@@ -100,9 +131,22 @@ class ModelConfig:
         return ["attn" if self.is_attn(i) else "gdn" for i in range(self.n_layers)]
 
     @property
+    def layer_runs(self) -> List[LayerRun]:
+        """Layers in the order they run."""
+        n = self.n_layers
+        if not self.loop:
+            return [LayerRun(i, i) for i in range(n)]
+        a, b, times = self.loop
+        order = [(i, None) for i in range(a)]
+        for t in range(times):
+            order += [(i, t if i == a else None) for i in range(a, b)]
+        order += [(i, None) for i in range(b, n)]
+        return [LayerRun(r, i, t) for r, (i, t) in enumerate(order)]
+
+    @property
     def n_attn(self) -> int:
         if self.layers:
-            return sum(1 for l in self.layers if l.kv_from is None)
+            return sum(1 for r in self.layer_runs if self.layers[r.layer].cached)
         return sum(1 for k in self.layer_kinds if k != "gdn")
 
     @property
@@ -135,7 +179,16 @@ class ModelConfig:
         n = self.vocab * h * (1 if self.tie_embeddings else 2)
         if self.layers:
             n += (self.gram_buckets + 1) * h if self.gram_buckets else 0
+            n += 2 * h * h if self.loop else 0
             for l in self.layers:
+                if l.mixer == "gqa":
+                    n += h * (2 * l.heads + l.kv_heads * (1 if l.key_values else 2)) * l.dim
+                elif l.mixer == "cdelta":
+                    n += h * (2 * l.kv_heads * l.dim + 2 * l.heads * l.vdim + l.heads) + (2 * l.kv_heads * l.dim + l.heads * l.vdim) * l.conv
+                    n += l.decay_rank * (h + l.heads * l.dim) + l.gate_rank * (h + l.heads * l.vdim)
+                if l.mixer != "latent":
+                    n += (3 if l.act == "swiglu" else 2) * h * l.ff
+                    continue
                 n += h * l.q_rank + l.q_rank * l.heads * l.dim + l.heads * (l.dim + l.vdim) * l.kv_rank + l.heads * l.vdim * h
                 n += (h * l.kv_rank if l.kv_from is None else 0) + 2 * h * l.ff
             return n
@@ -162,9 +215,9 @@ class ModelConfig:
         if world == 1:
             return c
         if self.layers:
-            assert all(l.heads % world == 0 and l.ff % world == 0 for l in self.layers), \
+            assert all(l.heads % world == 0 and l.kv_heads % world == 0 and l.ff % world == 0 for l in self.layers), \
                 f"heads and feed-forward widths must divide over {world} ranks"
-            c.layers = [dataclasses.replace(l, heads=l.heads // world, ff=l.ff // world) for l in self.layers]
+            c.layers = [dataclasses.replace(l, heads=l.heads // world, kv_heads=l.kv_heads // world, ff=l.ff // world) for l in self.layers]
             return c
         assert self.n_q % world == 0 and self.inter % world == 0
         c.n_q = self.n_q // world
@@ -243,7 +296,41 @@ def zototar_config(v: dict) -> ModelConfig:
         gram_mul_cur=int(gram.get("mul_cur", 0)), logit_softcap=float(v.get("logit_softcap") or 0.0))
 
 
-ARCHITECTURES = {"Zototar": zototar_config}
+def dofunex_config(v: dict) -> ModelConfig:
+    """A Dofunex config.json: grouped-query attention whose values are the projected keys (interleaved rotation, normed queries and
+    keys, a sink) and gated delta rules with a decay per channel, norms before and after every sublayer, looped layers."""
+    layers: List[LayerSpec] = []
+    for i, e in enumerate(v["layers"]):
+        kind, m, ff = e["type"], e["mixer"], e.get("mlp")
+        if kind not in ("attention", "channel_delta"):
+            raise ValueError(f"layer {i}: mixer type {kind!r} is neither attention nor channel_delta")
+        if ff and ff["kind"] != "dense":
+            raise ValueError(f"layer {i}: feed-forward kind {ff['kind']!r} is not dense")
+        kw = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                  ff=int(ff["ff"]) if ff else 0, act="swiglu")
+        if kw["heads"] % kw["kv_heads"]:
+            raise ValueError(f"layer {i}: {kw['heads']} heads do not divide over {kw['kv_heads']} key heads")
+        if kind == "attention":
+            if kw["dim"] != kw["vdim"]:
+                raise ValueError(f"layer {i}: the values are the keys, so vdim {kw['vdim']} must be dim {kw['dim']}")
+            rot = m.get("rot") or {}
+            s = rot.get("scaling")
+            layers.append(LayerSpec(mixer="gqa", scale=float(m["scale"]), bias=True, sink=True, key_values=True, qk_norm=True,
+                                    rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 1e4)),
+                                    rot_scaling={k: float(s[k]) for k in ("factor", "low", "high", "original")} if s else None, **kw))
+        else:
+            layers.append(LayerSpec(mixer="cdelta", conv=int(m["conv"]), **kw))
+    lp = v.get("loop")
+    if lp and not 0 <= lp["start"] < lp["stop"] <= len(layers):
+        raise ValueError(f"loop {lp['start']} .. {lp['stop']} lies outside the {len(layers)} layers")
+    return ModelConfig(
+        name="dofunex", hidden=int(v["width"]), inter=max([l.ff for l in layers] + [0]), n_layers=len(layers), n_q=layers[0].heads,
+        n_kv=layers[0].kv_heads, head_dim=layers[0].dim, eps=float(v["norm"]["eps"]), vocab=int(v["vocab"]), attn_gate=False,
+        tie_embeddings=False, layers=layers, out_norm=True, pre_norm=True, residual_mult=float(v.get("residual_mult", 1.0)),
+        loop=[int(lp[k]) for k in ("start", "stop", "times")] if lp else None, logit_scale=float(v.get("logit_scale", 1.0)))
+
+
+ARCHITECTURES = {"Zototar": zototar_config, "Dofunex": dofunex_config}
 
 
 # ---- presets: the five benchmark configurations ----------------------------------------------------
@@ -324,7 +411,35 @@ def zototar_7b() -> ModelConfig:
     return zototar(4096, 32, 32, 1536, 512, 16384, 129280, name="zototar-7b")
 
 
+def dofunex(width: int, n_layers: int, heads: int, kv_heads: int, ff: int, vocab: int, dim: int = 128, every: int = 4,
+            rank: int = 128, loop: Optional[List[int]] = None, name: str = "dofunex") -> ModelConfig:
+    """A Dofunex model of equal layers, every `every`-th one attention, the others delta rules with `heads` heads of `dim`."""
+    scaling = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192.0}
+    attn = LayerSpec(mixer="gqa", heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, ff=ff, act="swiglu", bias=True,
+                     sink=True, key_values=True, qk_norm=True, rot_dims=dim, rot_base=5e5, rot_scaling=scaling)
+    delta = LayerSpec(mixer="cdelta", heads=heads, kv_heads=heads, dim=dim, vdim=dim, ff=ff, act="swiglu", conv=4, decay_rank=rank,
+                      gate_rank=rank)
+    layers = [dataclasses.replace(attn if i % every == every - 1 else delta) for i in range(n_layers)]
+    return ModelConfig(name=name, hidden=width, inter=ff, n_layers=n_layers, n_q=heads, n_kv=kv_heads, head_dim=dim, eps=1e-6, vocab=vocab,
+                       attn_gate=False, tie_embeddings=False, layers=layers, out_norm=True, pre_norm=True, loop=loop)
+
+
+def tiny_dofunex() -> ModelConfig:
+    """4-layer plumbing model of the channel-delta family: unequal layers, sizes off the kernels' tile grid, two layers looped."""
+    c = dofunex(136, 4, 4, 2, 168, 300, dim=40, every=2, rank=20, loop=[1, 3, 3], name="tiny-dofunex")
+    c.residual_mult, c.logit_scale = 0.6, 1.5
+    c.layers[0] = dataclasses.replace(c.layers[0], dim=24, vdim=56, kv_heads=2, conv=3, ff=0)
+    c.layers[3] = dataclasses.replace(c.layers[3], heads=6, kv_heads=6, rot_dims=16, rot_scaling=None, ff=72)
+    return c
+
+
+def dofunex_7b() -> ModelConfig:
+    """7B-class channel-delta model: 32 layers of width 4096 (every fourth attention), 32 heads of 128, FFN 11008."""
+    return dofunex(4096, 32, 32, 8, 11008, 129280, name="dofunex-7b")
+
+
 PRESETS = {
+    "tiny-dofunex": tiny_dofunex, "dofunex-7b": dofunex_7b,
     "tiny-zototar": tiny_zototar, "zototar-7b": zototar_7b,
     "tiny": tiny_hybrid, "tiny-mla": tiny_mla, "27b": hybrid_27b, "drafter": drafter_block, "moe80b": moe_80b, "mla671b": mla_671b,
 }
@@ -335,6 +450,9 @@ def scaled(cfg: ModelConfig, n_layers: int) -> ModelConfig:
     c = dataclasses.replace(cfg)
     c.n_layers = n_layers
     c.layers = list(cfg.layers[:n_layers])
+    if cfg.loop:
+        a, b = cfg.loop[0], min(cfg.loop[1], n_layers)
+        c.loop = [a, b, cfg.loop[2]] if a < b else None
     c.tap_layers = [t for t in cfg.tap_layers if t < n_layers]
     return c
 

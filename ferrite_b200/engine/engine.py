@@ -11,7 +11,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..config import EngineConfig, ModelConfig
-from ..models.weights import Weights, init_weights, pack_latent, shard_weights
+from ..models.weights import Weights, init_weights, keeps_f32, pack_listed, shard_weights
 from .executor import Executor, Segment, StepBatch
 
 
@@ -46,7 +46,7 @@ class Engine:
                 not cfg.layers or self.ecfg.weight_dtype != "bf16" or (tp is not None and tp.world > 1)):
             raise ValueError("compute_dtype fp32 on a GPU: models of listed layers with unpacked weights on one GPU only")
         if cfg.layers and self.ecfg.kv_dtype != "bf16":
-            raise ValueError(f"kv_dtype {self.ecfg.kv_dtype!r}: latent caches are kept in the compute dtype")
+            raise ValueError(f"kv_dtype {self.ecfg.kv_dtype!r}: caches of models of listed layers are kept in the compute dtype")
         self.dtype = torch.bfloat16 if on_gpu and self.ecfg.compute_dtype == "bf16" else torch.float32
         world = tp.world if tp is not None else 1
         rank = tp.rank if tp is not None else 0
@@ -66,9 +66,7 @@ class Engine:
             weights = shard_weights(cfg, weights, rank, world)
         from ..formats.packed import is_packed
         weights = {k: (v if (is_packed(v) or not isinstance(v, torch.Tensor)) else
-                       v.to(self.device) if v.dtype == torch.float32 and (k.endswith(("A_log", "dt_bias", "router_bias")) or
-                                                                                 (cfg.out_norm and k.endswith("norm")))
-                       else v.to(self.device, self.dtype)) for k, v in weights.items()}
+                       v.to(self.device) if v.dtype == torch.float32 and keeps_f32(cfg, k) else v.to(self.device, self.dtype)) for k, v in weights.items()}
         # linears that arrived packed from a quantised checkpoint (ModelOpt NVFP4 / FP8, EXL3) become the kernels' weight
         # objects here, after the tensor-parallel cut; on the CPU they are dequantised for the fp32 oracle
         if any(is_packed(v) for v in weights.values()):
@@ -77,7 +75,7 @@ class Engine:
                 if is_packed(weights[k]):
                     weights[k] = from_packed(weights[k], self.device, self.dtype, on_gpu)
         if cfg.layers:
-            weights = pack_latent(cfg.shard(world), weights)
+            weights = pack_listed(cfg.shard(world), weights)
         is_t = lambda v: isinstance(v, torch.Tensor)
         if self.ecfg.weight_dtype in ("nvfp4", "nvfp4-a16", "nvfp4-w4a4"):
             from ..ops.qweight import quantize_experts, quantize_weight

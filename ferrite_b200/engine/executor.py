@@ -6,7 +6,8 @@ primitives `:1846-2141`): rows in, logits out, commit, slot copy / snapshot. Pol
 
 A row is (token, slot, position). Rows of one slot form a segment (contiguous, increasing positions): a decode
 row, a chain of verify rows, or a prompt chunk. State per slot: paged KV for the attention layers (a block
-table per slot), and for every Gated DeltaNet layer an fp32 recurrent state plus a 3-tap conv tail.
+table per slot), and for every Gated DeltaNet layer an fp32 recurrent state plus a 3-tap conv tail. Models of listed layers keep
+caches and states per run of a layer (looped layers run several times).
 """
 from __future__ import annotations
 
@@ -22,8 +23,8 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from ..config import EngineConfig, ModelConfig
-from ..models.weights import Weights, latent_dims
-from ..ops.latent import seg_groups
+from ..models.weights import Weights, delta_dims, gqa_dims, latent_dims
+from ..ops.latent import SegGroup, seg_groups
 from ..ops.qweight import QWeight
 
 
@@ -171,18 +172,31 @@ class Executor:
                 # one latent row [kv_lora | rope] per token; the value cache slot stays empty
                 self.k_cache[i] = torch.zeros(n_blocks, ecfg.kv_block, 1, c.kv_lora + c.rope_head_dim, dtype=dt, device=dev)
                 self.v_cache[i] = torch.zeros(n_blocks, 0, dtype=dt, device=dev)
-            elif kind == "latent":
-                # one latent row per token, in the layers that have latents of their own
-                if c.layers[i].kv_from is None:
-                    self.k_cache[i] = torch.zeros(n_blocks, ecfg.kv_block, latent_dims(c, i).lat, dtype=dt, device=dev)
-                    self.v_cache[i] = torch.zeros(n_blocks, 0, dtype=dt, device=dev)
             elif kind == "gdn":
                 self.rec_state[i] = torch.zeros(ecfg.n_slots, c.lin_v_heads, c.lin_dk, c.lin_dv, dtype=torch.float32, device=dev)
                 self.conv_state[i] = torch.zeros(ecfg.n_slots, c.conv_k - 1, c.conv_dim, dtype=dt, device=dev)
+        # models of listed layers: caches and states belong to runs of layers (a looped layer has one per pass)
+        self.runs = c.layer_runs if c.layers else []
+        self.run_dims: Dict[int, object] = {}
+        for r in self.runs:
+            l, zeros = c.layers[r.layer], lambda *s, t=dt: torch.zeros(*s, dtype=t, device=dev)
+            if l.mixer == "latent":
+                # one latent row per token, in the layers that have latents of their own
+                d = self.run_dims[r.index] = latent_dims(c, r.layer)
+                if l.kv_from is None:
+                    self.k_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.lat)
+                    self.v_cache[r.index] = zeros(n_blocks, 0)
+            elif l.mixer == "gqa":
+                d = self.run_dims[r.index] = gqa_dims(c, r.layer)
+                self.k_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
+                self.v_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
+            else:
+                d = self.run_dims[r.index] = delta_dims(c, r.layer)
+                self.rec_state[r.index] = zeros(ecfg.n_slots, d.heads, d.dim, d.vdim, t=torch.float32)
+                self.conv_state[r.index] = zeros(ecfg.n_slots, d.conv - 1, d.channels)
         # the token at every cached position, paged like the latents: the token before a segment (bigram embeddings) is read
         # from here, so it follows the pages through parking, forks, resumed prefixes and rejected drafts
         self.tok_pages = torch.zeros(n_blocks, ecfg.kv_block, dtype=torch.int32, device=dev) if c.gram_buckets else None
-        self.latent_dims = {i: latent_dims(c, i) for i, kind in enumerate(self.kinds) if kind == "latent"}
         self.block_table_host = torch.full((ecfg.n_slots, self.max_blocks), -1, dtype=torch.int32)
         self.block_table = self.block_table_host.to(dev)
         self.slot_blocks: List[List[int]] = [[] for _ in range(ecfg.n_slots)]
@@ -316,8 +330,9 @@ class Executor:
             per = e.kv_block * (c.kv_lora + c.rope_head_dim) * 2
         if c.layers:
             item = torch.empty(0, dtype=self.dtype).element_size()
-            return e.kv_block * (item * sum(latent_dims(c, i).lat for i, l in enumerate(c.layers) if l.kv_from is None)
-                                 + (4 if c.gram_buckets else 0))
+            dims = [(gqa_dims if c.layers[r.layer].mixer == "gqa" else latent_dims)(c, r.layer) for r in c.layer_runs if c.layers[r.layer].cached]
+            row = sum(2 * d.kv_heads * d.hp if hasattr(d, "kv_heads") else d.lat for d in dims)
+            return e.kv_block * (item * row + (4 if c.gram_buckets else 0))
         return per * max(1, self.cfg.n_attn)
 
     # ---- block tables -----------------------------------------------------------------------------
@@ -349,14 +364,15 @@ class Executor:
             t[slot].zero_()
 
     # ---- snapshots (prompt-cache primitives) ---------------------------------------------------------
-    def state_save(self, slot: int) -> Dict[str, torch.Tensor]:
-        """Copy of the GDN recurrent + conv state of a slot (a `Snap`, reference `pcache.rs`); KV stays in place."""
-        return {
-            "rec": torch.stack([t[slot] for t in self.rec_state.values()]).clone() if self.rec_state else torch.empty(0),
-            "conv": torch.stack([t[slot] for t in self.conv_state.values()]).clone() if self.conv_state else torch.empty(0),
-        }
+    def state_save(self, slot: int) -> Dict[str, Sequence[torch.Tensor]]:
+        """Copy of the recurrent + conv state of a slot (a `Snap`, reference `pcache.rs`), layer by layer; KV stays in place."""
+        def copies(states):
+            ts = [t[slot] for t in states.values()]
+            # layers of one size are copied by one launch; those of listed models may differ
+            return torch.stack(ts) if len({t.shape for t in ts}) == 1 else [t.clone() for t in ts]
+        return {"rec": copies(self.rec_state), "conv": copies(self.conv_state)}
 
-    def state_restore(self, slot: int, snap: Dict[str, torch.Tensor]) -> None:
+    def state_restore(self, slot: int, snap: Dict[str, Sequence[torch.Tensor]]) -> None:
         for j, t in enumerate(self.rec_state.values()):
             t[slot].copy_(snap["rec"][j])
         for j, t in enumerate(self.conv_state.values()):
@@ -575,10 +591,10 @@ class Executor:
             return self.ops.linear(x_in, w, out_f32=True)
         return self.tp.linear_allreduce(self.ops, x_in, w, None)
 
-    def _mix_latent(self, xb, i, mv, groups, nsplit, gathered):
-        """Latent attention of layer i over operand rows xb: rows of prompt segments attend keys and values expanded from the
-        latents, the others the latents themselves."""
-        w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{i}.", self.latent_dims[i]
+    def _mix_latent(self, xb, run, mv, groups, nsplit, gathered):
+        """Latent attention over operand rows xb: rows of prompt segments attend keys and values expanded from the latents, the
+        others the latents themselves."""
+        w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{run.layer}.", self.run_dims[run.index]
         cache, T = self.k_cache[d.source], xb.shape[0]
         proj = ops.linear(xb, w[p + "in_proj"], out_f32=True)
         cq = ops.latent_prep(proj, d, w[p + "q_a_norm"], w.get(p + "kv_a_norm"), mv["slot"], mv["pos"], self.block_table, cache, kvb,
@@ -604,22 +620,74 @@ class Executor:
                 ops.head_linear(ol, w[p + "v_up"], out=o[a:b].view(b - a, d.heads, d.hp))
         return self._sum_ranks(o, w[p + "out_proj"])
 
-    def _layers_out_norm(self, x, xb, mv, T, nseg, max_seg_rows, nsplit):
-        """x <- x + norm(mixer(x)), x <- x + norm(ff(x)): x is the 32-bit residual stream (updated in place), xb its copy in the
-        GEMM operand type. Returns the last copy."""
+    def _mix_gqa(self, h, run, mv, groups, nsplit):
+        """Grouped-query attention over operand rows h: prompt segments on the flash kernel, the others split over the keys."""
+        w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{run.layer}.", self.run_dims[run.index]
+        kc, vc = self.k_cache[run.index], self.v_cache[run.index]
+        proj = ops.linear(h, w[p + "in_proj"], out_f32=True)
+        q = ops.gqa_prep(proj, d, w.get(p + "in_bias"), w[p + "inv_freq"], mv["slot"], mv["pos"], self.block_table, kc, vc, kvb, self.cfg.eps)
+        o = torch.empty_like(q)
+        for g in groups:
+            segs = tuple(mv[k][g.seg_lo:g.seg_hi] for k in ("sslot", "srow0", "snrows", "spos0"))
+            ops.gqa_attention(q, d, kc, vc, w.get(p + "sink"), g, mv["slot"], mv["kvlen"], segs, self.block_table, kvb, nsplit, o)
+        return self._sum_ranks(o.view(o.shape[0], -1), w[p + "out_proj"])
+
+    def _mix_cdelta(self, h, run, mv, groups, commit):
+        """Delta rule with a decay per channel over operand rows h; verify rows keep their projections for the replay."""
+        w, p = self.w, f"l{run.layer}."
+        proj = self.ops.linear(h, w[p + "in_proj"])
+        if not commit:
+            self.verify_proj[run.index] = proj
+        return self._sum_ranks(self._cdelta(proj, run, mv, groups, commit), w[p + "out_proj"])
+
+    def _cdelta(self, proj, run, mv, groups, commit):
+        p, r = f"l{run.layer}.", run.index
+        names = ("decay_up", "gate_up_lr", "conv", "A_log", "dt_bias", "gnorm_w")
+        return self.ops.cdelta(proj, self.run_dims[r], {n: self.w[p + n] for n in names}, self.rec_state[r], self.conv_state[r], groups,
+                               mv["sslot"], mv["srow0"], mv["snrows"], self.cfg.eps, commit)
+
+    def _layers_listed(self, x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit):
+        """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), with `pre_norm` also a norm ahead of the mixer and the feed-forward: x is
+        the 32-bit residual stream (updated in place), xb its copy in the GEMM operand type. The pass over the rows that adds a
+        sublayer's output also makes the operand of whatever comes next. `loop_rows` [T, 2 width]: operand of the product that opens
+        a pass of the loop, the embedding output in its right half. Returns the last copy of x."""
         c, w, ops = self.cfg, self.w, self.ops
         self.taps = []
-        groups = seg_groups(self._step_segments if ops.name == "cuda" and self.dtype == torch.bfloat16 else None, nseg, T,
-                            max_seg_rows, FLASH_MIN_ROWS, self.block_table, self.ecfg.kv_block, self.device)
+        kinds = {l.mixer for l in c.layers}
+        groups = seg_groups(self._step_segments if ops.name == "cuda" and (self.dtype == torch.bfloat16 or "cdelta" in kinds) else None, nseg, T,
+                            max_seg_rows, FLASH_MIN_ROWS, self.block_table, self.ecfg.kv_block, self.device, "latent" in kinds)
         gathered: Dict[tuple, torch.Tensor] = {}
-        for i, l in enumerate(c.layers):
+        W = x.shape[1]
+        last_run = {r.layer: r.index for r in self.runs}
+
+        def after(j):
+            """Operand that run j starts from: (weight of a norm, buffer)."""
+            if j < len(self.runs) and self.runs[j].enter is not None:
+                return None, loop_rows[:, :W]
+            return (w[f"l{self.runs[j].layer}.pre_norm"] if c.pre_norm and j < len(self.runs) else None), None
+
+        for run in self.runs:
+            i, l = run.layer, c.layers[run.layer]
             p = f"l{i}."
-            xb = ops.add_normed(x, self._mix_latent(xb, i, mv, groups, nsplit, gathered), w[p + "mix_norm"], c.hidden, c.eps)
+            if run.enter is not None:
+                y = ops.linear(loop_rows, w["loop_in"], out_f32=True)
+                xb = ops.add_normed(x, y, None, c.hidden, c.eps, bias=w["loop_step"][run.enter], next_w=w.get(p + "pre_norm"))
+            elif run.index == 0 and c.pre_norm:
+                xb = ops.norm_rows(x, None, w[p + "pre_norm"], c.hidden, c.eps)
+            if l.mixer == "latent":
+                y = self._mix_latent(xb, run, mv, groups, nsplit, gathered)
+            elif l.mixer == "gqa":
+                y = self._mix_gqa(xb, run, mv, groups, nsplit)
+            else:
+                y = self._mix_cdelta(xb, run, mv, groups, commit)
+            nxt, buf = (w.get(p + "ffn_pre_norm"), None) if l.ff else after(run.index + 1)
+            xb = ops.add_normed(x, y, w[p + "mix_norm"], c.hidden, c.eps, bias=w.get(p + "out_bias"), next_w=nxt, out=buf)
             if l.ff:
-                act = ops.linear(xb, w[p + "up"], act=l.act)
-                xb = ops.add_normed(x, self._sum_ranks(act, w[p + "down"]), w[p + "ffn_norm"], c.hidden, c.eps)
-            if i in c.tap_layers:
-                self.taps.append(xb[:, :c.hidden].clone() if xb is x else xb[:, :c.hidden])
+                act = ops.linear(xb, w[p + "gate_up"], swiglu=True) if l.act == "swiglu" else ops.linear(xb, w[p + "up"], act=l.act)
+                nxt, buf = after(run.index + 1)
+                xb = ops.add_normed(x, self._sum_ranks(act, w[p + "down"]), w[p + "ffn_norm"], c.hidden, c.eps, next_w=nxt, out=buf)
+            if i in c.tap_layers and run.index == last_run[i]:
+                self.taps.append(x[:, :c.hidden].to(self.dtype, copy=True) if c.pre_norm or xb is x else xb[:, :c.hidden])
             if self.dump_layers:
                 self._dump_layer(i, x[:, :c.hidden], False, T)
         return xb
@@ -827,10 +895,11 @@ class Executor:
         if self.cfg.out_norm:
             c, w = self.cfg, self.w
             assert x_add is None and not tree, "models of listed layers: no injected rows, no verify trees"
+            loop_rows = torch.empty(T, 2 * w["embed"].shape[1], dtype=self.dtype, device=self.device) if c.loop else None
             x, xb = self.ops.embed_grams(w["embed"], w.get("bigram"), mv["tok"], mv["slot"], mv["pos"], self.block_table,
                                          self.tok_pages, self.ecfg.kv_block, c.embed_scale, c.gram_buckets, c.gram_mul_prev,
-                                         c.gram_mul_cur)
-            self.last_hidden = self._layers_out_norm(x, xb, mv, T, nseg, max_seg_rows, nsplit)[:, :c.hidden]
+                                         c.gram_mul_cur, **({"out": loop_rows} if c.loop else {}))
+            self.last_hidden = self._layers_listed(x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit)[:, :c.hidden]
             return self._head(x, mv, nlog, greedy)
         x = self.ops.embed(self.w["embed"], mv["tok"])
         if x_add is not None and self.input_rows:
@@ -866,8 +935,8 @@ class Executor:
         c, w, ops = self.cfg, self.w, self.ops
         mv["snrows"].copy_(torch.tensor(list(keep), dtype=torch.int32), non_blocking=False)
         mr = max(max(keep), 1)
-        if (self._last_graph_key is not None and self.profile is None and self._replay_fused(mr)
-                and any(k == "gdn" for k in self.kinds)):
+        if (self._last_graph_key is not None and self.profile is None
+                and ((self._replay_fused(mr) and "gdn" in self.kinds) or "cdelta" in self.kinds)):
             # The verify step ran as a CUDA graph, so the projections it saved sit in that graph's buffers: the replay
             # (one fused launch per GDN layer, the kept counts are device data) is captured once per forward graph and
             # replayed with it. Eager verify steps allocate fresh projections every time and replay eagerly.
@@ -888,6 +957,10 @@ class Executor:
 
     def _replay_layers(self, mv, mr: int) -> None:
         c, w, ops = self.cfg, self.w, self.ops
+        for run in self.runs:
+            if c.layers[run.layer].mixer == "cdelta":
+                proj = self.verify_proj[run.index]
+                self._cdelta(proj, run, mv, [SegGroup(0, mv["sslot"].numel(), 0, proj.shape[0], mr)], True)
         for i, kind in enumerate(self.kinds):
             if kind != "gdn":
                 continue
@@ -981,7 +1054,7 @@ class Executor:
                      and self.profile is None and x_add is None and not self.dump_layers)
         tree = batch.tree
         if tree:
-            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and not {"mla", "latent"} & set(self.kinds), \
+            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and not {"mla", "latent", "gqa", "cdelta"} & set(self.kinds), \
                 "verify trees: commit=False, at most TREE_MAX_ROWS rows per segment, attention / GDN layers"
             assert self.tp is None or self.tp.world == 1 or not self.tp.sp_ready(T)
         logit_rows = self._upload(batch)

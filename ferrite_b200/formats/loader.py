@@ -14,7 +14,7 @@ from typing import Dict, Optional
 import torch
 
 from ..config import ModelConfig
-from ..models.weights import weight_shapes
+from ..models.weights import keeps_f32, weight_shapes
 from . import exl3, modelopt
 from .packed import PackedEXL3, PackedLinear, cat_rows, dense_of
 from .safetensors_io import SafeTensors, save_file
@@ -52,22 +52,37 @@ def _take(w, index: torch.Tensor):
     raise TypeError(f"{type(w).__name__} rows cannot be regrouped")
 
 
-def _load_zototar(st: SafeTensors, cfg: ModelConfig, dtype) -> Dict[str, torch.Tensor]:
-    """A Zototar checkpoint under engine names; every tensor's shape is checked against the configuration."""
-    top = {"embed": "embed", "bigram": "bigram", "final_norm": "final.norm", "lm_head": "head"}
-    sub = {"mix_norm": "norm1", "ffn_norm": "norm2", "q_a": "mix.dq", "q_a_norm": "mix.dq.norm", "q_b": "mix.uq",
-           "kv_a": "mix.dkv", "kv_a_norm": "mix.dkv.norm", "k_b": "mix.uk", "v_b": "mix.uv", "out_proj": "mix.o",
-           "up": "mlp.up", "down": "mlp.down"}
+_LISTED_TOP = {"embed": "embed", "bigram": "bigram", "final_norm": "final.norm", "lm_head": "head", "loop_in": "loop.in",
+               "loop_step": "loop.step"}
+_LISTED_SUB = {
+    "zototar": {"mix_norm": "norm1", "ffn_norm": "norm2", "q_a": "mix.dq", "q_a_norm": "mix.dq.norm", "q_b": "mix.uq", "kv_a": "mix.dkv",
+                "kv_a_norm": "mix.dkv.norm", "k_b": "mix.uk", "v_b": "mix.uv", "out_proj": "mix.o", "up": "mlp.up", "down": "mlp.down"},
+    "dofunex": {"pre_norm": "norm1", "mix_norm": "norm1b", "ffn_pre_norm": "norm2", "ffn_norm": "norm2b", "out_proj": "mix.o",
+                "out_bias": "mix.o.b", "gnorm_w": "mix.norm", "gate": "mlp.gate", "up": "mlp.up", "down": "mlp.down",
+                **{n: f"mix.{n}" for n in ("q", "k", "v", "b", "sink", "A_log", "dt_bias", "a1", "a2", "g1", "g2")},
+                **{n + "_bias": f"mix.{n}.b" for n in "qk"}, **{n + "_conv": f"mix.{n}.conv" for n in "qkv"}},
+}
+
+
+def _load_listed(st: SafeTensors, cfg: ModelConfig, dtype) -> Dict[str, torch.Tensor]:
+    """A checkpoint of a model of listed layers under engine names; every tensor's shape is checked against the configuration.
+    Widths that only the tensors tell (the low ranks of channel-delta layers) are filled into it."""
+    sub = _LISTED_SUB["zototar" if any(l.mixer == "latent" for l in cfg.layers) else "dofunex"]
+    for i, l in enumerate(cfg.layers):
+        if l.mixer == "cdelta":
+            for field, base in (("decay_rank", "a1"), ("gate_rank", "g1")):
+                if not getattr(l, field) and st.has(f"l{i}.{sub[base]}"):
+                    setattr(l, field, int(st.get(f"l{i}.{sub[base]}").shape[0]))
     w: Dict[str, torch.Tensor] = {}
     for name, shape in weight_shapes(cfg).items():
         layer, _, base = name.rpartition(".")
-        src = f"{layer}.{sub[base]}" if layer else top[base]
+        src = f"{layer}.{sub[base]}" if layer else _LISTED_TOP[base]
         if not st.has(src):
             raise KeyError(f"{src} is missing from the checkpoint")
         t = st.get(src)
         if tuple(t.shape) != tuple(shape):
             raise ValueError(f"{src}: shape {tuple(t.shape)}, the configuration says {tuple(shape)}")
-        w[name] = t if base.endswith("norm") else t.to(dtype)
+        w[name] = t.float() if keeps_f32(cfg, name) else t.to(dtype)
     return w
 
 
@@ -78,7 +93,7 @@ def load_model_weights(model_dir: str, cfg: ModelConfig, dtype=torch.bfloat16, d
     if "embed" in names and "final_norm" in names:                    # native layout
         return {k: st.get(k) for k in weight_shapes(cfg) if st.has(k)}
     if cfg.layers:
-        w = _load_zototar(st, cfg, dtype)
+        w = _load_listed(st, cfg, dtype)
         st.close()
         return w
     pre = "model.language_model." if any(n.startswith("model.language_model.") for n in names) else "model."

@@ -12,6 +12,7 @@ RMSNorm weights are stored zero-centred (effective weight 1 + w), the GDN gated-
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Dict, List
 
@@ -23,19 +24,44 @@ from ..formats.packed import cat_rows
 Weights = Dict[str, torch.Tensor]
 
 
-def latent_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
-    """Latent attention with norms on the sublayers' outputs (`LayerSpec`)."""
+def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
+    """A layer of a model that lists its layers (`LayerSpec`): norms on the sublayers' outputs and, with `pre_norm`, inputs."""
     l, h, p = cfg.layers[i], cfg.hidden, f"l{i}."
-    out: Dict[str, tuple] = {p + "mix_norm": (h,), p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,),
-                             p + "q_b": (l.heads * l.dim, l.q_rank)}
-    if l.kv_from is None:
-        out[p + "kv_a"] = (l.kv_rank, h)
-        out[p + "kv_a_norm"] = (l.kv_rank,)
-    out[p + "k_b"] = (l.heads * l.dim, l.kv_rank)
-    out[p + "v_b"] = (l.heads * l.vdim, l.kv_rank)
-    out[p + "out_proj"] = (h, l.heads * l.vdim)
+    out: Dict[str, tuple] = {p + "pre_norm": (h,)} if cfg.pre_norm else {}
+    out[p + "mix_norm"] = (h,)
+    if l.mixer == "latent":
+        out.update({p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,), p + "q_b": (l.heads * l.dim, l.q_rank)})
+        if l.kv_from is None:
+            out[p + "kv_a"] = (l.kv_rank, h)
+            out[p + "kv_a_norm"] = (l.kv_rank,)
+        out[p + "k_b"] = (l.heads * l.dim, l.kv_rank)
+        out[p + "v_b"] = (l.heads * l.vdim, l.kv_rank)
+        out[p + "out_proj"] = (h, l.heads * l.vdim)
+    elif l.mixer == "gqa":
+        for n, heads, d in (("q", l.heads, l.dim), ("k", l.kv_heads, l.dim)) + (() if l.key_values else (("v", l.kv_heads, l.vdim),)):
+            out[p + n] = (heads * d, h)
+            if l.bias:
+                out[p + n + "_bias"] = (heads * d,)
+        if l.sink:
+            out[p + "sink"] = (l.heads,)
+        out[p + "out_proj"] = (h, l.heads * l.vdim)
+        if l.bias:
+            out[p + "out_bias"] = (h,)
+    else:
+        nk, nv = l.kv_heads * l.dim, l.heads * l.vdim
+        for n, rows in (("q", nk), ("k", nk), ("v", nv)):
+            out[p + n] = (rows, h)
+            out[p + n + "_conv"] = (rows, l.conv)
+        out.update({p + "b": (l.heads, h), p + "A_log": (l.heads,), p + "dt_bias": (l.heads * l.dim,), p + "gnorm_w": (l.vdim,),
+                    p + "a1": (l.decay_rank, h), p + "a2": (l.heads * l.dim, l.decay_rank), p + "g1": (l.gate_rank, h),
+                    p + "g2": (nv, l.gate_rank), p + "out_proj": (h, nv)})
     if l.ff:
-        out.update({p + "ffn_norm": (h,), p + "up": (l.ff, h), p + "down": (h, l.ff)})
+        if cfg.pre_norm:
+            out[p + "ffn_pre_norm"] = (h,)
+        out[p + "ffn_norm"] = (h,)
+        if l.act == "swiglu":
+            out[p + "gate"] = (l.ff, h)
+        out.update({p + "up": (l.ff, h), p + "down": (h, l.ff)})
     return out
 
 
@@ -43,7 +69,7 @@ def layer_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
     h = cfg.hidden
     p = f"l{i}."
     if cfg.layers:
-        return latent_weight_shapes(cfg, i)
+        return listed_weight_shapes(cfg, i)
     out: Dict[str, tuple] = {p + "input_norm": (h,), p + "post_norm": (h,)}
     kind = cfg.layer_kinds[i]
     if kind == "gdn":
@@ -91,12 +117,21 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
         out["lm_head"] = (cfg.vocab, cfg.hidden)
     if cfg.gram_buckets:
         out["bigram"] = (cfg.gram_buckets + 1, cfg.hidden)
+    if cfg.loop:
+        out["loop_in"] = (cfg.hidden, 2 * cfg.hidden)
+        out["loop_step"] = (cfg.loop[2], cfg.hidden)
     for i in range(cfg.n_layers):
         out.update(layer_weight_shapes(cfg, i))
     return out
 
 
 _F32_NAMES = ("A_log", "dt_bias", "router_bias")
+_F32_LISTED = ("norm", "gnorm_w", "_bias", "sink", "_conv", "loop_step")     # ... of models of listed layers
+
+
+def keeps_f32(cfg: ModelConfig, name: str) -> bool:
+    """Small tensors that enter 32-bit arithmetic and stay in 32 bits whatever the engine computes in."""
+    return name.endswith(_F32_NAMES) or (cfg.out_norm and name.endswith(_F32_LISTED))
 
 
 def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="cpu", std: float = 0.02, post=None) -> Weights:
@@ -111,8 +146,9 @@ def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="c
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32) * std
         if name.endswith("gnorm_w") or (cfg.out_norm and name.endswith("norm")):
             t = t + 1.0
-        keep32 = name.endswith(_F32_NAMES) or (cfg.out_norm and name.endswith("norm"))
-        t = t if keep32 else t.to(dtype)
+        if cfg.out_norm and name.endswith("_conv"):
+            t = t / std * shape[1] ** -0.5
+        t = t if keeps_f32(cfg, name) else t.to(dtype)
         w[name] = post(name, t) if post is not None else t
     return w
 
@@ -121,6 +157,20 @@ def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="c
 
 def _rows(t: torch.Tensor, lo: int, hi: int) -> torch.Tensor:
     return t[lo:hi]
+
+
+_BY_ROWS = ("q", "k", "v", "q_bias", "k_bias", "v_bias", "sink", "q_conv", "k_conv", "v_conv", "b", "A_log", "dt_bias", "a2", "g2", "gate", "up")
+
+
+def _shard_listed(base: str, t: torch.Tensor, rank: int, world: int) -> torch.Tensor:
+    """gqa / cdelta layers and their feed-forwards: heads (rows of what makes them, columns of what reads them) divide evenly."""
+    if base in _BY_ROWS:
+        per = t.shape[0] // world
+        return t[rank * per:(rank + 1) * per].contiguous()
+    if base in ("out_proj", "down"):
+        per = t.shape[1] // world
+        return t[:, rank * per:(rank + 1) * per].contiguous()
+    return t
 
 
 def shard_weights(cfg: ModelConfig, w: Weights, rank: int, world: int) -> Weights:
@@ -137,7 +187,9 @@ def shard_weights(cfg: ModelConfig, w: Weights, rank: int, world: int) -> Weight
         base = name.split(".")[-1]
         li = int(name[1:name.index(".")]) if name.startswith("l") and "." in name else -1
         kind = cfg.layer_kinds[li] if li >= 0 else ""
-        if name == "lm_head":
+        if kind in ("gqa", "cdelta"):
+            out[name] = _shard_listed(base, t, rank, world)
+        elif name == "lm_head":
             per = (cfg.vocab + world - 1) // world
             out[name] = t[rank * per:min(cfg.vocab, (rank + 1) * per)].contiguous()
         elif base == "in_proj" and kind == "gdn":
@@ -235,8 +287,7 @@ class LatentDims:
 
 def latent_dims(cfg: ModelConfig, i: int) -> LatentDims:
     l = cfg.layers[i]
-    hd = max(l.dim, l.vdim)
-    hp = next((w for w in (64, 128, 256) if hd <= w), round_up(hd, 64))
+    hp = head_width(max(l.dim, l.vdim))
     return LatentDims(l.heads, l.q_rank, l.kv_rank, round_up(l.q_rank, 64), round_up(l.kv_rank, 64), hp, l.scale,
                       i if l.kv_from is None else l.kv_from)
 
@@ -249,43 +300,168 @@ def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
     return out
 
 
-def pack_latent(cfg: ModelConfig, w: Weights) -> Weights:
-    """Engine weights of a latent-attention model in the kernels' layout (see `LatentDims`):
+@dataclass(frozen=True)
+class GqaDims:
+    """Sizes of one grouped-query attention layer as its kernels see them. Cache rows and attention operands have heads of `hp`
+    columns, zeros beyond `dim`: 64 / 128 / 256 are what the tensor-core kernels take, wider heads run on the CUDA cores."""
 
-    * in_proj  rows = [q_a | kv_a]           one product for both latents of a token
+    heads: int
+    kv_heads: int
+    dim: int
+    hp: int
+    scale: float
+    rot_dims: int
+    v_off: int        # column of the projection where the values start (the keys' column when they are the values)
+    qk_norm: bool
+
+
+def head_width(d: int) -> int:
+    return next((w for w in (64, 128, 256) if d <= w), round_up(d, 64))
+
+
+def gqa_dims(cfg: ModelConfig, i: int) -> GqaDims:
+    l = cfg.layers[i]
+    assert l.dim == l.vdim, "keys and values of one width"
+    return GqaDims(l.heads, l.kv_heads, l.dim, head_width(l.dim), l.scale, l.rot_dims,
+                   (l.heads + (0 if l.key_values else l.kv_heads)) * l.dim, l.qk_norm)
+
+
+def rope_frequencies(l) -> torch.Tensor:
+    """Angle per position of every rotated pair of a gqa layer. With `rot_scaling` wavelengths beyond original / low are stretched
+    by `factor`, those below original / high stay, the ones between are blended."""
+    f = l.rot_base ** (-torch.arange(0, l.rot_dims, 2, dtype=torch.float64) / max(1, l.rot_dims))
+    s = l.rot_scaling
+    if s:
+        turns = s["original"] * f / (2 * math.pi)                            # of the pair over the original context
+        if s["high"] != s["low"]:
+            t = ((turns - s["low"]) / (s["high"] - s["low"])).clamp(0, 1)
+        else:
+            t = (turns >= s["low"]).double()
+        f = (1 - t) * f / s["factor"] + t * f
+    return f
+
+
+@dataclass(frozen=True)
+class DeltaDims:
+    """Sizes of one channel-delta layer as its kernels see them: columns of the fused projection [a1 | g1 | q | k | v | b]
+    (the two low-rank inputs first, so that they are aligned operands of their own) and the padded width of the mixer's output."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    ra: int           # padded decay rank
+    rg: int           # padded gate rank
+    ko: int           # padded heads * vdim
+
+    @property
+    def q_off(self) -> int:
+        return self.ra + self.rg
+
+    @property
+    def channels(self) -> int:
+        """Columns that pass the short convolutions: q | k | v."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def b_off(self) -> int:
+        return self.q_off + self.channels
+
+
+def delta_dims(cfg: ModelConfig, i: int) -> DeltaDims:
+    l = cfg.layers[i]
+    return DeltaDims(l.heads, l.kv_heads, l.dim, l.vdim, l.conv, round_up(l.decay_rank, 64), round_up(l.gate_rank, 64),
+                     round_up(l.heads * l.vdim, 64))
+
+
+def _pack_latent(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
+    """* in_proj  rows = [q_a | kv_a]           one product for both latents of a token
     * q_b      [heads * hp, qr]              per head zero-padded rows, so queries come out at the padded width
     * kv_up    [2 * heads * hp, lat]         key rows of every head, then value rows: expands latents for prompt rows
     * k_abs    [heads, lat, hp]              W_uk^T per head: folds the key projection into a decode row's query
     * v_up     [heads, hp, lat]              W_uv per head (a view of kv_up): latent-space outputs to values
-    * out_proj [width, heads * hp]
+    * out_proj [width, heads * hp]"""
+    l, p, d = cfg.layers[i], f"l{i}.", latent_dims(cfg, i)
+    parts = [_pad(w[p + "q_a"], d.qr, W)]
+    out[p + "q_a_norm"] = _pad(w[p + "q_a_norm"].float(), d.qr)
+    if l.kv_from is None:
+        parts.append(_pad(w[p + "kv_a"], d.lat, W))
+        out[p + "kv_a_norm"] = _pad(w[p + "kv_a_norm"].float(), d.lat)
+    out[p + "in_proj"] = torch.cat(parts)
+    q_b = _pad(w[p + "q_b"].view(l.heads, l.dim, l.q_rank), l.heads, d.hp, d.qr)
+    out[p + "q_b"] = q_b.view(l.heads * d.hp, d.qr)
+    k = _pad(w[p + "k_b"].view(l.heads, l.dim, l.kv_rank), l.heads, d.hp, d.lat)
+    v = _pad(w[p + "v_b"].view(l.heads, l.vdim, l.kv_rank), l.heads, d.hp, d.lat)
+    out[p + "kv_up"] = torch.cat([k.view(-1, d.lat), v.view(-1, d.lat)])
+    out[p + "k_abs"] = k.transpose(1, 2).contiguous()
+    out[p + "v_up"] = out[p + "kv_up"][l.heads * d.hp:].view(l.heads, d.hp, d.lat)
+    o = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp)
+    out[p + "out_proj"] = o.view(W, l.heads * d.hp)
 
-    Norm weights become 32-bit."""
+
+def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
+    """* in_proj  rows = [q | k (| v)] of all heads at their true width; in_bias the same
+    * out_proj [width, heads * hp]"""
+    l, p, d = cfg.layers[i], f"l{i}.", gqa_dims(cfg, i)
+    names = ("q", "k") if l.key_values else ("q", "k", "v")
+    rows = torch.cat([w[p + n] for n in names])
+    out[p + "in_proj"] = _pad(rows, rows.shape[0], W)
+    if l.bias:
+        out[p + "in_bias"] = torch.cat([w[p + n + "_bias"].float() for n in names])
+        out[p + "out_bias"] = _pad(w[p + "out_bias"].float(), W)
+    if l.sink:
+        out[p + "sink"] = w[p + "sink"].float().contiguous()
+    out[p + "out_proj"] = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp).view(W, -1)
+    out[p + "inv_freq"] = rope_frequencies(l).to(rows.device)
+
+
+def _pack_cdelta(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
+    """* in_proj  rows = [a1 | g1 | q | k | v | b] (see `DeltaDims`)
+    * conv     [channels, taps], decay_up [heads * dim, ra], gate_up_lr [heads * vdim, rg]
+    * out_proj [width, ko]"""
+    l, p, d = cfg.layers[i], f"l{i}.", delta_dims(cfg, i)
+    rows = torch.cat([_pad(w[p + "a1"], d.ra, cfg.hidden), _pad(w[p + "g1"], d.rg, cfg.hidden)] + [w[p + n] for n in ("q", "k", "v", "b")])
+    out[p + "in_proj"] = _pad(rows, rows.shape[0], W)
+    out[p + "conv"] = torch.cat([w[p + n + "_conv"].float() for n in ("q", "k", "v")]).contiguous()
+    out[p + "decay_up"] = _pad(w[p + "a2"], l.heads * l.dim, d.ra)
+    out[p + "gate_up_lr"] = _pad(w[p + "g2"], l.heads * l.vdim, d.rg)
+    for n in ("A_log", "dt_bias", "gnorm_w"):
+        out[p + n] = w[p + n].float().contiguous()
+    out[p + "out_proj"] = _pad(w[p + "out_proj"], W, d.ko)
+
+
+_PACK = {"latent": _pack_latent, "gqa": _pack_gqa, "cdelta": _pack_cdelta}
+
+
+def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
+    """Engine weights of a model of listed layers in the kernels' layout (see `LatentDims`, `GqaDims`, `DeltaDims`): sizes padded
+    with zeros, projections that share an input joined, norm weights in 32 bits with the residual's and the logits' multipliers in
+    them."""
     W = round_up(cfg.hidden, 64)
+    vec = lambda n, f=1.0: _pad(w[n].float() * f, W)
     out: Weights = {"embed": _pad(w["embed"], cfg.vocab, W), "lm_head": _pad(w["lm_head"], w["lm_head"].shape[0], W),
-                    "final_norm": _pad(w["final_norm"].float(), W)}
+                    "final_norm": vec("final_norm", cfg.logit_scale)}
     if cfg.gram_buckets:
         out["bigram"] = _pad(w["bigram"], cfg.gram_buckets + 1, W)
+    if cfg.loop:
+        out["loop_in"] = _pad(w["loop_in"].view(cfg.hidden, 2, cfg.hidden), W, 2, W).view(W, 2 * W)
+        out["loop_step"] = _pad(w["loop_step"].float(), cfg.loop[2], W)
     for i, l in enumerate(cfg.layers):
-        p, d = f"l{i}.", latent_dims(cfg, i)
-        parts = [_pad(w[p + "q_a"], d.qr, W)]
-        out[p + "q_a_norm"] = _pad(w[p + "q_a_norm"].float(), d.qr)
-        if l.kv_from is None:
-            parts.append(_pad(w[p + "kv_a"], d.lat, W))
-            out[p + "kv_a_norm"] = _pad(w[p + "kv_a_norm"].float(), d.lat)
-        out[p + "in_proj"] = torch.cat(parts)
-        q_b = _pad(w[p + "q_b"].view(l.heads, l.dim, l.q_rank), l.heads, d.hp, d.qr)
-        out[p + "q_b"] = q_b.view(l.heads * d.hp, d.qr)
-        k = _pad(w[p + "k_b"].view(l.heads, l.dim, l.kv_rank), l.heads, d.hp, d.lat)
-        v = _pad(w[p + "v_b"].view(l.heads, l.vdim, l.kv_rank), l.heads, d.hp, d.lat)
-        out[p + "kv_up"] = torch.cat([k.view(-1, d.lat), v.view(-1, d.lat)])
-        out[p + "k_abs"] = k.transpose(1, 2).contiguous()
-        out[p + "v_up"] = out[p + "kv_up"][l.heads * d.hp:].view(l.heads, d.hp, d.lat)
-        o = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp)
-        out[p + "out_proj"] = o.view(W, l.heads * d.hp)
-        out[p + "mix_norm"] = _pad(w[p + "mix_norm"].float(), W)
+        p = f"l{i}."
+        _PACK[l.mixer](cfg, w, i, W, out)
+        out[p + "mix_norm"] = vec(p + "mix_norm", cfg.residual_mult)
+        if cfg.pre_norm:
+            out[p + "pre_norm"] = vec(p + "pre_norm")
         if l.ff:
             F = round_up(l.ff, 64)
-            out[p + "up"] = _pad(w[p + "up"], F, W)
+            up = _pad(w[p + "up"], F, W)
+            if l.act == "swiglu":
+                out[p + "gate_up"] = torch.cat([_pad(w[p + "gate"], F, W), up])
+            else:
+                out[p + "up"] = up
             out[p + "down"] = _pad(w[p + "down"], W, F)
-            out[p + "ffn_norm"] = _pad(w[p + "ffn_norm"].float(), W)
+            out[p + "ffn_norm"] = vec(p + "ffn_norm", cfg.residual_mult)
+            if cfg.pre_norm:
+                out[p + "ffn_pre_norm"] = vec(p + "ffn_pre_norm")
     return out

@@ -45,14 +45,18 @@ def _prev_tokens(ids, row_slot, row_pos, block_table, tok_pages, kv_block) -> Li
 
 
 class TorchLatent:
-    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
-        """Scaled token embedding plus the hashed bigram's row: (x fp32 [T, width], the same rows as GEMM operand)."""
+    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur, out=None):
+        """Scaled token embedding plus the hashed bigram's row: (x fp32 [T, width], the same rows as GEMM operand). `out`: a buffer
+        [T, k * width] whose k blocks of columns all take the operand."""
         x = table[ids.long()].float() * scale
         if grams is not None:
             prev = _prev_tokens(ids, row_slot, row_pos, block_table, tok_pages, kv_block)
             rows = [buckets if p < 0 else (p * mul_prev + int(t) * mul_cur) % buckets for p, t in zip(prev, ids)]
             x = x + grams[torch.tensor(rows, dtype=torch.long, device=x.device)].float()
             tok_pages[block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block] = ids.to(tok_pages.dtype)
+        if out is not None:
+            for j in range(0, out.shape[1], x.shape[1]):
+                out[:, j:j + x.shape[1]] = x.to(self.dtype)
         return x, x.to(self.dtype)
 
     @staticmethod
@@ -60,10 +64,19 @@ class TorchLatent:
         xf = x.float()
         return xf / torch.sqrt(xf.pow(2).sum(-1, keepdim=True) / width + eps) * w
 
-    def add_normed(self, x, y, w, width, eps):
-        """x += rms(y) * w in place; returns x as GEMM operand."""
-        x += self._rms(y, w, width, eps)
-        return x.to(self.dtype)
+    def add_normed(self, x, y, w, width, eps, bias=None, next_w=None, out=None):
+        """x += rms(y + bias) * w in place (x = y + bias with w None). Returns the next GEMM operand: rms(x) * next_w, or x itself
+        with next_w None; written to `out` (rows may lie apart) when given."""
+        y = y.float() if bias is None else y.float() + bias
+        if w is None:
+            x.copy_(y)
+        else:
+            x += self._rms(y, w, width, eps)
+        h = x if next_w is None else self._rms(x, next_w, width, eps)
+        if out is not None:
+            out.copy_(h)
+            return out
+        return h.to(self.dtype)
 
     def norm_rows(self, x, idx, w, width, eps):
         return self._rms(x if idx is None else x[idx.long()], w, width, eps).to(self.dtype)
@@ -90,18 +103,20 @@ class TorchLatent:
 
 
 class CudaLatent:
-    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur):
+    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur, out=None):
         x = self.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=self.device)
-        xb = None if self.dtype == torch.float32 else self.empty(*x.shape, dtype=self.dtype, device=self.device)
+        xb = out if out is not None else None if self.dtype == torch.float32 else self.empty(*x.shape, dtype=self.dtype, device=self.device)
         self.launches += 1
         self.C.embed_grams(x, xb, table, grams, ids, row_slot, row_pos, block_table, kv_block, tok_pages, scale, buckets, mul_prev, mul_cur,
                            self.status_word)
         return x, (x if xb is None else xb)
 
-    def add_normed(self, x, y, w, width, eps):
-        xb = None if self.dtype == torch.float32 else self.empty(*x.shape, dtype=self.dtype, device=self.device)
+    def add_normed(self, x, y, w, width, eps, bias=None, next_w=None, out=None):
+        xb = out
+        if out is None and (self.dtype != torch.float32 or next_w is not None):
+            xb = self.empty(*x.shape, dtype=self.dtype, device=self.device)
         self.launches += 1
-        self.C.add_normed(x, xb, y, w, width, eps)
+        self.C.add_normed(x, xb, y, w, width, eps, bias, next_w)
         return x if xb is None else xb
 
     def norm_rows(self, x, idx, w, width, eps):
@@ -178,9 +193,10 @@ TORCH_ACTS = {None: lambda x: x, "relu2": relu2}
 
 
 def seg_groups(segments: Optional[List[Tuple[int, int, int]]], n_seg: int, n_rows: int, max_rows: int, flash_min: int, block_table,
-               kv_block: int, device) -> List[SegGroup]:
+               kv_block: int, device, gather: bool = True) -> List[SegGroup]:
     """Cut a step into runs of prompt segments (more than `flash_min` rows) and runs of the others. `segments`: host view
-    (slot, first position, rows) of an eager step, None inside a graph, whose launches must not depend on it."""
+    (slot, first position, rows) of an eager step, None inside a graph, whose launches must not depend on it. `gather`: prompt groups
+    carry the page lists of the expanded latent form."""
     if segments is None:
         return [SegGroup(0, n_seg, 0, n_rows, max_rows)]
     out: List[SegGroup] = []
@@ -194,7 +210,7 @@ def seg_groups(segments: Optional[List[Tuple[int, int, int]]], n_seg: int, n_row
             out.append(SegGroup(i, i + 1, row, row + n, n, prompt))
         row += n
     for g in out:
-        if not g.prompt:
+        if not g.prompt or not gather:
             continue
         counts = [(p + n + kv_block - 1) // kv_block for _, p, n in segments[g.seg_lo:g.seg_hi]]
         g.pages = torch.cat([block_table[s, :nb] for (s, _, _), nb in zip(segments[g.seg_lo:g.seg_hi], counts)])

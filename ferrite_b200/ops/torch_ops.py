@@ -14,13 +14,14 @@ import torch.nn.functional as F
 
 from .extras import TorchExtras
 from .latent import TORCH_ACTS, TorchLatent
+from .mixers import TorchMixers
 
 
 def _softplus(x):
     return torch.where(x > 20, x, torch.log1p(torch.exp(torch.clamp(x, max=20.0))))
 
 
-class TorchOps(TorchLatent, TorchExtras):
+class TorchOps(TorchLatent, TorchMixers, TorchExtras):
     name = "torch"
 
     def __init__(self, device="cpu", dtype=torch.float32):

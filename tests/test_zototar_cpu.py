@@ -15,7 +15,7 @@ from ferrite_b200.engine.executor import Segment
 from ferrite_b200.engine.sampler import Sampling
 from ferrite_b200.engine.scheduler import SchedOptions, Scheduler, generate
 from ferrite_b200.formats.loader import load_model_weights
-from ferrite_b200.models.weights import init_weights, latent_dims, pack_latent
+from ferrite_b200.models.weights import init_weights, latent_dims, pack_listed
 from ferrite_b200.ops.torch_ops import TorchOps
 from zototar_cases import CASES, engine, error, run_cuts, tokens, weights, write
 
@@ -83,7 +83,7 @@ def test_checkpoint_shapes_are_checked(tmp_path):
 def test_kernel_layout_pads_with_zeros():
     cfg = tiny_zototar()
     w = init_weights(cfg, seed=3)
-    pk = pack_latent(cfg, w)
+    pk = pack_listed(cfg, w)
     for i, l in enumerate(cfg.layers):
         d, p = latent_dims(cfg, i), f"l{i}."
         assert d.qr % 64 == d.lat % 64 == 0 and d.hp in (64, 128, 256)
