@@ -159,11 +159,11 @@ int fb_mla_qpad(void* qp, const void* q, long q_stride, const void* qabs, long r
                 float scale, cudaStream_t s);
 
 // ---- latent.cu ----
-int fb_embed_grams(float* x, void* xb, const void* table, const void* grams, const int* tok, const int* slot, const int* pos,
+int fb_embed_grams(float* x, void* xb, int copies, const void* table, const void* grams, const int* tok, const int* slot, const int* pos,
                    const int* block_table, int max_blocks, int kv_block, int* tok_pages, int rows, int width, int vocab, float scale,
                    long buckets, long mul_prev, long mul_cur, int f32, int* status, cudaStream_t s);
-int fb_add_normed(float* x, void* xb, const void* y, int y_f32, const float* w, int rows, int width, int ld, long ldy, float eps,
-                  cudaStream_t s);
+int fb_add_normed(float* x, void* xb, int xb_f32, long ldb, const void* y, int y_f32, const float* bias, const float* w,
+                  const float* next_w, int rows, int width, int ld, long ldy, float eps, cudaStream_t s);
 int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps, int f32,
                  cudaStream_t s);
 int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
@@ -178,6 +178,34 @@ int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const
                   const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen, const int* block_table,
                   int max_blocks, int kv_block, int rows, int row_base, int heads, int lat, int nsplit, float scale, int* status,
                   cudaStream_t s);
+int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache, const float* sink,
+                const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
+                int kv_heads, int hd, int nsplit, float scale, int f32, int* status, cudaStream_t s);
+int fb_attn_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int hd,
+                  cudaStream_t s);
+
+// ---- gqa.cu ----
+int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* bias, const double* inv_freq,
+                const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
+                int kv_heads, int dim, int hp, int rot, int v_off, int norm, float eps, int f32, int* status, cudaStream_t s);
+
+// ---- cdelta.cu, cdelta_chunk.cu ----
+int fb_cd_lowrank(float* out, const void* proj, long ldp, const void* wa, int na, int ra, const void* wg, int ng, int rg, int rows,
+                  int f32, cudaStream_t s);
+int fb_cd_step(void* out, int ko, float* rec, void* tail, const void* proj, long ldp, const float* decay, long ldd, const float* gate,
+               long ldg, const float* conv_w, const float* A_log, const float* dt_bias, const float* norm_w, const int* seg_slot,
+               const int* seg_row0, const int* seg_nrows, int nseg, int heads, int kv_heads, int dim, int vdim, int taps, int q_off,
+               float eps, int commit, int f32, cudaStream_t s);
+int fb_cd_tail(void* tail, const void* proj, long ldp, const int* seg_slot, const int* seg_row0, const int* seg_nrows, int nseg, int heads,
+               int kv_heads, int dim, int vdim, int taps, int q_off, int f32, cudaStream_t s);
+int fb_cd_rec(float* y, float* rec, void* qkv, const void* tail, const void* proj, long ldp, const float* decay, long ldd,
+              const float* conv_w, const float* A_log, const float* dt_bias, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
+              int nseg, int max_rows, int heads, int kv_heads, int dim, int vdim, int taps, int q_off, int commit, int f32, cudaStream_t s);
+long fb_cd_chunk_scratch_bytes(int rows, int nseg, int heads, int dim);
+int fb_cd_chunk(float* y, float* rec, float* scratch, const void* tail, const void* proj, long ldp, const float* decay, long ldd,
+                const float* conv_w, const float* A_log, const float* dt_bias, const int* seg_slot, const int* seg_row0,
+                const int* seg_nrows, int nseg, int max_rows, int heads, int kv_heads, int dim, int vdim, int taps, int q_off, int sm_count,
+                int f32, cudaStream_t s);
 int fb_gemm_f32(float* y, const float* x, const float* w, int M, int N, int K, long ldx, long ldy, int batch, long x_bs, long w_bs,
                 long y_bs, int act, cudaStream_t s);
 

@@ -64,7 +64,8 @@ __device__ __forceinline__ void dm_e4m3x16_to_bf16(const uint4& c, uint4& lo, ui
 // KV8: e4m3 cache (codes [..][HD] bytes, scales [token * nkv + head][2] fp32 for K and V). The byte tiles stream through
 // a two-stage cp.async ring and are expanded to bf16 tiles in shared memory before the MMAs; the per-key scales are
 // applied to the scores (K) and to P (V) instead of to every element.
-template <int HD, bool KV8>
+// PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (16 bits of mantissa instead of 8).
+template <int HD, bool KV8, bool PX>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, const __nv_bfloat16* __restrict__ q,
                        const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
@@ -72,7 +73,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
                        const int* __restrict__ seg_nrows, const int* __restrict__ row_kvlen,
                        const int* __restrict__ row_base, const unsigned long long* __restrict__ row_mask,
                        const int* __restrict__ block_table, int max_blocks, int kv_block, int nq, int nkv, int nsplit,
-                       int groups_per_seg, float scale_log2) {
+                       int groups_per_seg, int row_first, float scale_log2) {
   constexpr int LD = HD + 8;                    // padded row (elements): conflict-free ldmatrix
   constexpr int CPR = HD / 8;                   // 16-byte chunks per row
   extern __shared__ __align__(16) unsigned char dm_smem[];
@@ -94,7 +95,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
   if (r_first >= n) return;
   const int rows_here = min(RG, n - r_first);
   const int valid_m = rows_here * G;            // M rows in use: m = local row * G + head of the group
-  const int row0 = seg_row0[seg] + r_first, slot = seg_slot[seg];
+  const int row0 = seg_row0[seg] - row_first + r_first, slot = seg_slot[seg];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   const int* bt = block_table + (size_t)slot * max_blocks;
   int kv_end = 0;
@@ -238,7 +239,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
         mrow[h] = mn;
       }
       float ls[2] = {0.f, 0.f};
-      uint32_t pa[2][4];
+      uint32_t pa[2][4], pr[PX ? 2 : 1][4];
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt) {
         const float p0 = (mrow[0] == -INFINITY) ? 0.f : exp2f(s[nt][0] - mrow[0]);
@@ -250,6 +251,11 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
         if (KV8) { v0 = tsc[((lane & 3) * 2 + nt * 8) * 2 + 1]; v1 = tsc[((lane & 3) * 2 + nt * 8 + 1) * 2 + 1]; }
         pa[nt >> 1][(nt & 1) * 2 + 0] = pack_bf2(p0 * v0, p1 * v1);
         pa[nt >> 1][(nt & 1) * 2 + 1] = pack_bf2(p2 * v0, p3 * v1);
+        if constexpr (PX) {
+          const uint32_t a0 = pa[nt >> 1][(nt & 1) * 2], a1 = pa[nt >> 1][(nt & 1) * 2 + 1];
+          pr[nt >> 1][(nt & 1) * 2 + 0] = pack_bf2(p0 - bf_lo(a0), p1 - bf_hi(a0));
+          pr[nt >> 1][(nt & 1) * 2 + 1] = pack_bf2(p2 - bf_lo(a1), p3 - bf_hi(a1));
+        }
       }
 #pragma unroll
       for (int h = 0; h < 2; ++h) lrow[h] = lrow[h] * sc[h] + ls[h];
@@ -263,6 +269,10 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
           dm_ldsm_t(b, V + (ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LD + np * 16 + (lane >> 4) * 8);
           dm_mma(o[np * 2], pa[ks], b[0], b[1]);
           dm_mma(o[np * 2 + 1], pa[ks], b[2], b[3]);
+          if constexpr (PX) {
+            dm_mma(o[np * 2], pr[ks], b[0], b[1]);
+            dm_mma(o[np * 2 + 1], pr[ks], b[2], b[3]);
+          }
         }
       }
     }
@@ -293,14 +303,15 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
 using namespace fb;
 
 // Same outputs as fb_attn_decode (bf16 cache) / fb_attn_decode_kv8 (kv_scale != null: e4m3 cache); rows are addressed
-// through their segments (rows of one segment share a slot). Returns -20 for shapes this kernel does not take (the
-// caller uses the SIMT kernel).
+// through their segments (rows of one segment share a slot). scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as
+// value + remainder (bf16 cache); row_first: row of the step that q / out / row_kvlen start at; out null: the split records stay for
+// the caller to merge. Returns -20 for shapes this kernel does not take (the caller uses the SIMT kernel).
 extern "C" int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache,
                                   const void* v_cache, const float* kv_scale, const void* proj, long proj_stride,
                                   const int* seg_slot, const int* seg_row0, const int* seg_nrows, const int* row_kvlen,
                                   const int* row_base, const unsigned long long* row_mask, const int* block_table,
                                   int max_blocks, int kv_block, int nseg, int max_rows, int rows, int nq, int nkv, int hd,
-                                  int nsplit, int gated, cudaStream_t s) {
+                                  int nsplit, int gated, float scale, int exact_p, int row_first, cudaStream_t s) {
   if (nseg <= 0 || rows <= 0) return 0;
   if (nq % nkv) return -1;
   const int G = nq / nkv;
@@ -308,25 +319,27 @@ extern "C" int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, cons
   const int RG = DM_BM / G;
   const int gps = (max_rows + RG - 1) / RG;
   dim3 grid(nseg * gps, nkv, nsplit);
-  const float scale_log2 = 1.4426950408889634f / sqrtf((float)hd);
-#define FB_DM(HDV, K8)                                                                                              \
+  const float scale_log2 = 1.4426950408889634f * (scale != 0.f ? scale : 1.f / sqrtf((float)hd));
+#define FB_DM(HDV, K8, PXV)                                                                                              \
   {                                                                                                                 \
     const size_t smem = K8 ? (size_t)(DM_BM + 2 * DM_BKV) * (HDV + 8) * 2 + (size_t)4 * DM_BKV * HDV + 4 * DM_BKV * 4 * 2 \
                            : (size_t)(DM_BM + 4 * DM_BKV) * (HDV + 8) * 2;                                          \
-    auto kern = attn_decode_mma_kernel<HDV, K8>;                                                                    \
+    auto kern = attn_decode_mma_kernel<HDV, K8, PXV>;                                                               \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
     if (e != cudaSuccess) return (int)e;                                                                            \
     launch_pdl(kern, grid, dim3(DM_WARPS * 32), smem, s, o_part, ml_part, (const __nv_bfloat16*)q,                   \
                (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, kv_scale, seg_slot, seg_row0, seg_nrows, \
-               row_kvlen, row_base, row_mask, block_table, max_blocks, kv_block, nq, nkv, nsplit, gps, scale_log2);  \
+               row_kvlen, row_base, row_mask, block_table, max_blocks, kv_block, nq, nkv, nsplit, gps, row_first, scale_log2);  \
   }
   if (kv_scale) {
-    if (hd == 256) FB_DM(256, true) else if (hd == 128) FB_DM(128, true) else FB_DM(64, true)
+    if (hd == 256) FB_DM(256, true, false) else if (hd == 128) FB_DM(128, true, false) else FB_DM(64, true, false)
+  } else if (exact_p) {
+    if (hd == 256) FB_DM(256, false, true) else if (hd == 128) FB_DM(128, false, true) else FB_DM(64, false, true)
   } else {
-    if (hd == 256) FB_DM(256, false) else if (hd == 128) FB_DM(128, false) else FB_DM(64, false)
+    if (hd == 256) FB_DM(256, false, false) else if (hd == 128) FB_DM(128, false, false) else FB_DM(64, false, false)
   }
 #undef FB_DM
   int rc = (int)cudaGetLastError();
-  if (rc) return rc;
+  if (rc || !out) return rc;
   return fb_attn_combine(out, o_part, ml_part, proj, proj_stride, rows, nq, hd, nsplit, gated, s);
 }

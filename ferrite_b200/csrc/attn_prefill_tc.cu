@@ -83,7 +83,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                        const __nv_bfloat16* __restrict__ proj, long proj_stride, const int* __restrict__ seg_slot,
                        const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows,
                        const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
-                       int kv_block, int nq, int nkv, int gated, float scale_log2, int* status) {
+                       int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink,
+                       int* status) {
   constexpr int NCH = HD / 64;                     // 64-element (128-byte) chunks of the head dim
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
@@ -345,7 +346,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     asm volatile("bar.sync 1, 256;" ::: "memory");
     if (!fail_s[2]) {
       tc_fence_after();
-      const float lt = l + l_s[half ^ 1][row];
+      float lt = l + l_s[half ^ 1][row];
+      if (sink) lt += exp2f(sink[qh] * 1.4426950408889634f - m_ref);
       const float inv = lt > 0.f ? 1.f / lt : 0.f;
       const bool valid = q0 + row < n;
       const size_t grow = (size_t)(row0 + q0 + row);
@@ -389,13 +391,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 using namespace fb;
 
 // q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block] rows of nkv*hd bf16, kv_stride elements
-// apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; same outputs as
-// fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
+// apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; sink: a number per q head
+// that joins the softmax denominator, or null; same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
 extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                                   long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                                   const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg,
                                   int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int gated,
-                                  float scale, int exact_p, long kv_stride, int* status, cudaStream_t s) {
+                                  float scale, int exact_p, long kv_stride, const float* sink, int* status, cudaStream_t s) {
   if (nseg <= 0 || max_rows <= 0) return 0;
   if (nq % nkv) return -1;
   if ((hd != 64 && hd != 128 && hd != 256) || kv_block % FT_BKV) return -20;
@@ -416,7 +418,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
     if (e != cudaSuccess) return (int)e;                                                                           \
     launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
-               gated, scale_log2, status);                                                                         \
+               gated, scale_log2, sink, status);                                                                   \
   }
   if (exact_p) {
     if (hd == 256) FB_FT(256, true) else if (hd == 128) FB_FT(128, true) else FB_FT(64, true)

@@ -562,19 +562,153 @@ int is_f32(const Tensor& t) {
 void embed_grams(Tensor x, c10::optional<Tensor> xb, Tensor table, c10::optional<Tensor> grams, Tensor tok, Tensor slot, Tensor pos,
                  Tensor block_table, int64_t kv_block, c10::optional<Tensor> tok_pages, double scale, int64_t buckets,
                  int64_t mul_prev, int64_t mul_cur, Tensor status) {
-  TORCH_CHECK(x.is_contiguous() && table.is_contiguous() && x.size(1) == table.size(1), "embed_grams: layouts");
+  TORCH_CHECK(x.is_contiguous() && table.is_contiguous() && x.size(1) == table.size(1) &&
+              (!xb || (xb->is_contiguous() && xb->size(1) % x.size(1) == 0)), "embed_grams: layouts");
   TORCH_CHECK(!grams || (grams->is_contiguous() && grams->size(0) == buckets + 1 && grams->size(1) == x.size(1) && tok_pages),
               "embed_grams: bigram table");
-  check(fb_embed_grams(x.data_ptr<float>(), optr(xb), table.data_ptr(), cptr(grams), tok.data_ptr<int>(), slot.data_ptr<int>(),
+  check(fb_embed_grams(x.data_ptr<float>(), optr(xb), xb ? (int)(xb->size(1) / x.size(1)) : 0, table.data_ptr(), cptr(grams), tok.data_ptr<int>(), slot.data_ptr<int>(),
                        pos.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block,
                        (int*)optr(tok_pages), (int)x.size(0), (int)x.size(1), (int)table.size(0), (float)scale, (long)buckets,
                        (long)mul_prev, (long)mul_cur, is_f32(table), status.data_ptr<int>(), cur_stream()), "embed_grams");
 }
 
-void add_normed(Tensor x, c10::optional<Tensor> xb, Tensor y, Tensor w, int64_t width, double eps) {
-  TORCH_CHECK(x.is_contiguous() && y.stride(1) == 1 && y.size(1) == x.size(1) && w.numel() == x.size(1), "add_normed: layouts");
-  check(fb_add_normed(x.data_ptr<float>(), optr(xb), y.data_ptr(), is_f32(y), w.data_ptr<float>(), (int)x.size(0), (int)width,
+void add_normed(Tensor x, c10::optional<Tensor> xb, Tensor y, c10::optional<Tensor> w, int64_t width, double eps,
+                c10::optional<Tensor> bias, c10::optional<Tensor> next_w) {
+  auto row_ok = [&](const c10::optional<Tensor>& t) { return !t || (t->numel() == x.size(1) && t->is_contiguous() && is_f32(*t)); };
+  TORCH_CHECK(x.is_contiguous() && y.stride(1) == 1 && y.sizes() == x.sizes() && row_ok(w) && row_ok(bias) && row_ok(next_w) &&
+              (!xb || (xb->stride(1) == 1 && xb->sizes() == x.sizes())), "add_normed: layouts");
+  check(fb_add_normed(x.data_ptr<float>(), optr(xb), xb ? is_f32(*xb) : 0, xb ? (long)xb->stride(0) : 0, y.data_ptr(), is_f32(y),
+                      (const float*)cptr(bias), (const float*)cptr(w), (const float*)cptr(next_w), (int)x.size(0), (int)width,
                       (int)x.size(1), (long)y.stride(0), (float)eps, cur_stream()), "add_normed");
+}
+
+void silu_mul_f32(Tensor out, Tensor gu) {
+  TORCH_CHECK(is_f32(out) && is_f32(gu) && out.is_contiguous() && gu.is_contiguous() && gu.size(1) == 2 * out.size(1), "silu_mul_f32: layouts");
+  check(fb_silu_mul_f32(out.data_ptr<float>(), gu.data_ptr<float>(), (int)out.size(0), (int)out.size(1), cur_stream()), "silu_mul_f32");
+}
+
+void gqa_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::optional<Tensor> bias, Tensor inv_freq, Tensor row_slot,
+              Tensor row_pos, Tensor block_table, int64_t kv_block, int64_t dim, int64_t rot, int64_t v_off, bool norm, double eps,
+              Tensor status) {
+  const int heads = (int)q.size(1), kvh = (int)k_cache.size(2), hp = (int)q.size(2);
+  TORCH_CHECK(q.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.sizes() == v_cache.sizes() &&
+              k_cache.size(3) == hp && k_cache.size(1) == kv_block && is_f32(proj) && proj.stride(1) == 1 &&
+              q.scalar_type() == k_cache.scalar_type() && q.scalar_type() == v_cache.scalar_type() &&
+              proj.size(1) >= (heads + kvh) * dim && proj.size(1) >= v_off + kvh * dim && inv_freq.scalar_type() == torch::kFloat64 &&
+              inv_freq.numel() * 2 >= rot && (!bias || (is_f32(*bias) && bias->numel() >= v_off + kvh * dim && bias->numel() >= (heads + kvh) * dim)),
+              "gqa_prep: layouts");
+  check(fb_gqa_prep(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), proj.data_ptr<float>(), (long)proj.stride(0),
+                    (const float*)cptr(bias), inv_freq.data_ptr<double>(), row_slot.data_ptr<int>(), row_pos.data_ptr<int>(),
+                    block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block, (int)q.size(0), heads, kvh, (int)dim, hp, (int)rot,
+                    (int)v_off, norm ? 1 : 0, (float)eps, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_prep");
+}
+
+// Few rows of grouped-query attention: q, out [rows, heads, hd]; tensor cores for bf16 (segments of consecutive rows of one slot, the
+// step's row row_first first), CUDA cores otherwise.
+void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cache, Tensor v_cache, c10::optional<Tensor> sink,
+              Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, Tensor row_slot, Tensor row_kvlen, Tensor block_table,
+              int64_t kv_block, int64_t row_first, int64_t nsplit, double scale, bool cuda_cores, Tensor status) {
+  const int rows = (int)q.size(0), heads = (int)q.size(1), hd = (int)q.size(2), kvh = (int)k_cache.size(2);
+  const long recs = (long)rows * heads * nsplit;
+  TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.size(3) == hd &&
+              o_part.numel() >= recs * hd && ml_part.numel() >= recs * 2 && row_slot.numel() == rows && row_kvlen.numel() == rows &&
+              (!sink || sink->numel() == heads), "gqa_attn: layouts");
+  const float* sk = (const float*)cptr(sink);
+  if (!cuda_cores) {
+    check(fb_attn_decode_mma(nullptr, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                             nullptr, nullptr, 0, seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(),
+                             row_kvlen.data_ptr<int>(), nullptr, nullptr, block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block,
+                             (int)seg_slot.numel(), (int)max_rows, rows, heads, kvh, hd, (int)nsplit, 0, (float)scale, 1, (int)row_first,
+                             cur_stream()), "attn_decode_mma");
+    check(fb_attn_merge(out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), sk, rows, heads, (int)nsplit, hd, cur_stream()),
+          "attn_merge");
+    return;
+  }
+  check(fb_gqa_attn(out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                    sk, row_slot.data_ptr<int>(), row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
+                    (int)kv_block, rows, heads, kvh, hd, (int)nsplit, (float)scale, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_attn");
+}
+
+// Channel-delta layers. sizes: heads, kv_heads, dim, vdim, taps, first convolved column of the projection.
+struct CdArgs { int heads, kvh, dim, vdim, taps, q_off; };
+CdArgs cd_args(const std::vector<int64_t>& v, const Tensor& proj, const Tensor& rec, const Tensor& tail, const Tensor& conv_w) {
+  TORCH_CHECK(v.size() == 6, "cdelta: six sizes");
+  CdArgs a{(int)v[0], (int)v[1], (int)v[2], (int)v[3], (int)v[4], (int)v[5]};
+  const int ch = 2 * a.kvh * a.dim + a.heads * a.vdim;
+  TORCH_CHECK(proj.stride(1) == 1 && proj.size(1) >= a.q_off + ch + a.heads && rec.is_contiguous() && tail.is_contiguous() && is_f32(rec) &&
+              rec.size(1) == a.heads && rec.size(2) == a.dim && rec.size(3) == a.vdim && tail.size(1) == a.taps - 1 && tail.size(2) == ch &&
+              tail.scalar_type() == proj.scalar_type() && conv_w.is_contiguous() && conv_w.size(0) == ch && conv_w.size(1) == a.taps &&
+              is_f32(conv_w), "cdelta: layouts");
+  return a;
+}
+
+void cd_lowrank(Tensor out, Tensor proj, Tensor wa, Tensor wg) {
+  TORCH_CHECK(out.is_contiguous() && is_f32(out) && proj.stride(1) == 1 && wa.is_contiguous() && wg.is_contiguous() &&
+              wa.scalar_type() == proj.scalar_type() && wg.scalar_type() == proj.scalar_type() && out.size(1) == wa.size(0) + wg.size(0) &&
+              proj.size(1) >= wa.size(1) + wg.size(1), "cd_lowrank: layouts");
+  check(fb_cd_lowrank(out.data_ptr<float>(), proj.data_ptr(), (long)proj.stride(0), wa.data_ptr(), (int)wa.size(0), (int)wa.size(1),
+                      wg.data_ptr(), (int)wg.size(0), (int)wg.size(1), (int)proj.size(0), is_f32(proj), cur_stream()), "cd_lowrank");
+}
+
+int64_t cd_step(Tensor out, Tensor rec, Tensor tail, Tensor proj, Tensor decay, Tensor gate, Tensor conv_w, Tensor A_log, Tensor dt_bias,
+                Tensor norm_w, Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, std::vector<int64_t> sizes, double eps, bool commit) {
+  const CdArgs a = cd_args(sizes, proj, rec, tail, conv_w);
+  TORCH_CHECK(out.is_contiguous() && out.scalar_type() == proj.scalar_type() && decay.stride(1) == 1 && gate.stride(1) == 1 && is_f32(decay) &&
+              is_f32(gate), "cd_step: layouts");
+  const int rc = fb_cd_step(out.data_ptr(), (int)out.size(1), rec.data_ptr<float>(), tail.data_ptr(), proj.data_ptr(), (long)proj.stride(0),
+                            decay.data_ptr<float>(), (long)decay.stride(0), gate.data_ptr<float>(), (long)gate.stride(0),
+                            conv_w.data_ptr<float>(), A_log.data_ptr<float>(), dt_bias.data_ptr<float>(), norm_w.data_ptr<float>(),
+                            seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), (int)seg_slot.numel(), a.heads, a.kvh,
+                            a.dim, a.vdim, a.taps, a.q_off, (float)eps, commit ? 1 : 0, is_f32(proj), cur_stream());
+  if (rc == -20) return rc;                     // sizes for the split form
+  check(rc, "cd_step");
+  return 0;
+}
+
+void cd_tail(Tensor rec, Tensor tail, Tensor proj, Tensor conv_w, Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, std::vector<int64_t> sizes) {
+  const CdArgs a = cd_args(sizes, proj, rec, tail, conv_w);
+  check(fb_cd_tail(tail.data_ptr(), proj.data_ptr(), (long)proj.stride(0), seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(),
+                   seg_nrows.data_ptr<int>(), (int)seg_slot.numel(), a.heads, a.kvh, a.dim, a.vdim, a.taps, a.q_off, is_f32(proj),
+                   cur_stream()), "cd_tail");
+}
+
+void cd_rec(Tensor y, Tensor rec, Tensor qkv, Tensor tail, Tensor proj, Tensor decay, Tensor conv_w, Tensor A_log, Tensor dt_bias,
+            Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, std::vector<int64_t> sizes, bool commit) {
+  const CdArgs a = cd_args(sizes, proj, rec, tail, conv_w);
+  TORCH_CHECK(y.is_contiguous() && is_f32(y) && qkv.is_contiguous() && qkv.scalar_type() == proj.scalar_type() && is_f32(decay) &&
+              decay.stride(1) == 1, "cd_rec: layouts");
+  check(fb_cd_rec(y.data_ptr<float>(), rec.data_ptr<float>(), qkv.data_ptr(), tail.data_ptr(), proj.data_ptr(), (long)proj.stride(0),
+                  decay.data_ptr<float>(), (long)decay.stride(0), conv_w.data_ptr<float>(), A_log.data_ptr<float>(), dt_bias.data_ptr<float>(),
+                  seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), (int)seg_slot.numel(), (int)max_rows, a.heads,
+                  a.kvh, a.dim, a.vdim, a.taps, a.q_off, commit ? 1 : 0, is_f32(proj), cur_stream()), "cd_rec");
+}
+
+int64_t cd_chunk_scratch_bytes(int64_t rows, int64_t nseg, int64_t heads, int64_t dim) {
+  return fb_cd_chunk_scratch_bytes((int)rows, (int)nseg, (int)heads, (int)dim);
+}
+
+int64_t cd_chunk(Tensor y, Tensor rec, Tensor scratch, Tensor tail, Tensor proj, Tensor decay, Tensor conv_w, Tensor A_log, Tensor dt_bias,
+                 Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, std::vector<int64_t> sizes) {
+  const CdArgs a = cd_args(sizes, proj, rec, tail, conv_w);
+  TORCH_CHECK(y.is_contiguous() && is_f32(y) && is_f32(decay) && decay.stride(1) == 1 &&
+              scratch.numel() * scratch.element_size() >= fb_cd_chunk_scratch_bytes((int)proj.size(0), (int)seg_slot.numel(), a.heads, a.dim),
+              "cd_chunk: layouts");
+  const int rc = fb_cd_chunk(y.data_ptr<float>(), rec.data_ptr<float>(), (float*)scratch.data_ptr(), tail.data_ptr(), proj.data_ptr(),
+                             (long)proj.stride(0), decay.data_ptr<float>(), (long)decay.stride(0), conv_w.data_ptr<float>(),
+                             A_log.data_ptr<float>(), dt_bias.data_ptr<float>(), seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(),
+                             seg_nrows.data_ptr<int>(), (int)seg_slot.numel(), (int)max_rows, a.heads, a.kvh, a.dim, a.vdim, a.taps, a.q_off,
+                             at::cuda::getCurrentDeviceProperties()->multiProcessorCount, is_f32(proj), cur_stream());
+  if (rc == -20) return rc;                     // heads wider than the kernel takes
+  check(rc, "cd_chunk");
+  return 0;
+}
+
+void gated_norm_sigmoid(Tensor out, Tensor y, Tensor z, Tensor w, double eps) {
+  const int heads = (int)y.size(1), dv = (int)y.size(2);
+  TORCH_CHECK(out.is_contiguous() && y.is_contiguous() && z.stride(1) == 1 && is_f32(y) && is_f32(z) && is_f32(w) && w.numel() == dv &&
+              z.size(1) == heads * dv, "gated_norm_sigmoid: layouts");
+  check(fb_gated_norm_sigmoid(out.data_ptr(), (int)out.size(1), y.data_ptr<float>(), z.data_ptr<float>(), (long)z.stride(0),
+                              w.data_ptr<float>(), (int)y.size(0), heads, dv, (float)eps, is_f32(out), cur_stream()), "gated_norm_sigmoid");
 }
 
 void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, int64_t width, double eps) {
@@ -721,6 +855,16 @@ void register_ext(pybind11::module_& m) {
   m.def("latent_attn", &latent_attn);
   m.def("latent_mma", &latent_mma);
   m.def("gemm_f32", &gemm_f32);
+  m.def("silu_mul_f32", &silu_mul_f32);
+  m.def("gqa_prep", &gqa_prep);
+  m.def("gqa_attn", &gqa_attn);
+  m.def("cd_lowrank", &cd_lowrank);
+  m.def("cd_step", &cd_step);
+  m.def("cd_tail", &cd_tail);
+  m.def("cd_rec", &cd_rec);
+  m.def("cd_chunk", &cd_chunk);
+  m.def("cd_chunk_scratch_bytes", &cd_chunk_scratch_bytes);
+  m.def("gated_norm_sigmoid", &gated_norm_sigmoid);
   m.def("exl3_had", &exl3_had);
   m.def("exl3_gemv", &exl3_gemv);
   m.def("exl3_decode", &exl3_decode);

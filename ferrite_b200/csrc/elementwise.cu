@@ -4,6 +4,7 @@
 // `fe_add_bf16` (`kernels/k-core/src/misc.rs:7-179`) and `fe_gdn_norm` (`kernels/k-core/src/gdn.rs:417`).
 #include "api.h"
 #include "common.cuh"
+#include "elem.cuh"
 
 namespace fb {
 
@@ -74,6 +75,15 @@ __global__ void rmsnorm_kernel(__nv_bfloat16* __restrict__ out, __nv_bfloat16* _
   }
 }
 
+// The same in fp32
+__global__ void silu_mul_f32_kernel(float* __restrict__ out, const float* __restrict__ gu, int inter) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= inter) return;
+  const float* r = gu + (size_t)blockIdx.y * 2 * inter;
+  const float g = r[i];
+  out[(size_t)blockIdx.y * inter + i] = g / (1.f + expf(-g)) * r[inter + i];
+}
+
 // out[r][i] = silu(gu[r][i]) * gu[r][inter + i]
 __global__ void silu_mul_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu, int inter,
                                 float clamp) {
@@ -96,10 +106,11 @@ __global__ void silu_mul_kernel(__nv_bfloat16* __restrict__ out, const __nv_bflo
 }
 
 // Gated per-head RMSNorm of the GDN output: out[r][h][d] = bf16( y * rsqrt(mean_d y^2 + eps) * w[d] * silu(z) ).
-// y is fp32 [rows][heads][dv]; z is a bf16 column block of the fused projection (row stride z_stride).
-__global__ void gated_norm_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ y,
-                                  const __nv_bfloat16* __restrict__ z, long z_stride,
-                                  const __nv_bfloat16* __restrict__ w, int heads, int dv, float eps) {
+// y is fp32 [rows][heads][dv]; z is a column block of the fused projection (row stride z_stride). SIG: gated by sigmoid(z) instead.
+// Output rows are ldo wide, zeros beyond the heads.
+template <typename T, typename Z, bool SIG>
+__global__ void gated_norm_kernel(T* __restrict__ out, int ldo, const float* __restrict__ y, const Z* __restrict__ z, long z_stride,
+                                  const Z* __restrict__ w, int heads, int dv, float eps) {
   pdl_launch_dependents();
   pdl_wait();
   int row = blockIdx.x;
@@ -111,12 +122,14 @@ __global__ void gated_norm_kernel(__nv_bfloat16* __restrict__ out, const float* 
     for (int d = lane; d < dv; d += 32) { float v = yp[d]; ss += v * v; }
     ss = warp_sum(ss);
     float r = rsqrtf(ss / (float)dv + eps);
-    const __nv_bfloat16* zp = z + (size_t)row * z_stride + (size_t)h * dv;
+    const Z* zp = z + (size_t)row * z_stride + (size_t)h * dv;
     for (int d = lane; d < dv; d += 32) {
-      float v = yp[d] * r * bf2f(w[d]) * siluf_(bf2f(zp[d]));
-      out[((size_t)row * heads + h) * dv + d] = f2bf(v);
+      const float zv = Elem<Z>::to(zp[d]);
+      const float v = yp[d] * r * Elem<Z>::to(w[d]) * (SIG ? 1.f / (1.f + expf(-zv)) : siluf_(zv));
+      out[(size_t)row * ldo + h * dv + d] = Elem<T>::from(v);
     }
   }
+  for (int c = heads * dv + threadIdx.x; c < ldo; c += blockDim.x) out[(size_t)row * ldo + c] = Elem<T>::from(0.f);
 }
 
 __global__ void gather_rows_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ in,
@@ -173,13 +186,33 @@ extern "C" int fb_silu_mul(void* out, const void* gu, int rows, int inter, float
   return (int)cudaGetLastError();
 }
 
+extern "C" int fb_silu_mul_f32(float* out, const float* gu, int rows, int inter, cudaStream_t s) {
+  if (rows <= 0 || inter <= 0) return 0;
+  if (rows > 65535) return -1;
+  silu_mul_f32_kernel<<<dim3((inter + 255) / 256, rows), 256, 0, s>>>(out, gu, inter);
+  return (int)cudaGetLastError();
+}
+
 extern "C" int fb_gated_norm(void* out, const float* y, const void* z, long z_stride, const void* w, int rows,
                              int heads, int dv, float eps, cudaStream_t s) {
   if (rows <= 0) return 0;
   int threads = heads >= 8 ? 256 : 32 * heads;
-  launch_pdl(gated_norm_kernel, dim3(rows), dim3(threads), (size_t)(0), s, (__nv_bfloat16*)out, y, (const __nv_bfloat16*)z, z_stride,
-                                             (const __nv_bfloat16*)w, heads, dv, eps);
+  launch_pdl(gated_norm_kernel<__nv_bfloat16, __nv_bfloat16, false>, dim3(rows), dim3(threads), (size_t)(0), s, (__nv_bfloat16*)out,
+             heads * dv, y, (const __nv_bfloat16*)z, z_stride, (const __nv_bfloat16*)w, heads, dv, eps);
   return (int)cudaGetLastError();
+}
+
+// Gate sigmoid(z), z and w fp32, out bf16 or fp32 (f32) rows of ldo columns
+extern "C" int fb_gated_norm_sigmoid(void* out, int ldo, const float* y, const float* z, long z_stride, const float* w, int rows, int heads,
+                                     int dv, float eps, int f32, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (ldo < heads * dv) return -1;
+  const dim3 b(heads >= 8 ? 256 : 32 * heads);
+  if (f32)
+    return (int)launch_pdl(gated_norm_kernel<float, float, true>, dim3(rows), b, (size_t)0, s, (float*)out, ldo, y, z, z_stride, w, heads, dv,
+                           eps);
+  return (int)launch_pdl(gated_norm_kernel<__nv_bfloat16, float, true>, dim3(rows), b, (size_t)0, s, (__nv_bfloat16*)out, ldo, y, z, z_stride,
+                         w, heads, dv, eps);
 }
 
 extern "C" int fb_gather_rows(void* out, const void* in, const int* idx, int rows, int width, cudaStream_t s) {

@@ -1,0 +1,106 @@
+// Grouped-query attention of the models of listed layers: what happens between the fused projection and the attention kernels
+// (`attn_prefill_tc.cu` for prompt segments, `attn_decode_mma.cu` for few rows, `latent.cu` in 32 bits).
+//
+//   proj row = [q heads | k heads (| v heads)] of `dim` columns each, fp32 sums without their biases; with v_off at the keys the
+//   values are the projected keys themselves, before rotation and norm.
+//
+// One warp per head: bias, rotation of the pairs (0, 1), (2, 3), ... of the first `rot` columns, division by the root mean square
+// over `dim` (no weight), q to [row][head][hp], k and v into their page rows [kv head][hp]; columns dim .. hp - 1 are zeros.
+// Angles are formed and reduced to one turn in double: a position of millions keeps all its bits.
+#include "api_ext.h"
+#include "common.cuh"
+#include "elem.cuh"
+
+namespace fb {
+
+constexpr int GP_WARPS = 8;
+
+// NP: pairs of a head per lane (dim <= 64 NP)
+template <typename T, int NP>
+__global__ void __launch_bounds__(GP_WARPS * 32)
+gqa_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ proj, long ldp,
+                const float* __restrict__ bias, const double* __restrict__ inv_freq, const int* __restrict__ row_slot,
+                const int* __restrict__ row_pos, const int* __restrict__ block_table, int max_blocks, int kv_block, int heads,
+                int kv_heads, int dim, int hp, int rot, int v_off, int norm, float eps, int* status) {
+  extern __shared__ float2 gp_turn[];                       // (cos, sin) of every rotated pair
+  pdl_launch_dependents();
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_wait();
+  const int pos = row_pos[row];
+  for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+    constexpr double TURN = 6.283185307179586476925;
+    double a = (double)pos * inv_freq[i];
+    a -= TURN * rint(a / TURN);
+    float s, c;
+    sincosf((float)a, &s, &c);
+    gp_turn[i] = make_float2(c, s);
+  }
+  __syncthreads();
+  const int h = blockIdx.y * GP_WARPS + warp;
+  if (h >= heads + kv_heads) return;
+  const int col = h * dim;                                  // q heads, then k heads
+  const float* src = proj + (size_t)row * ldp + col;
+  const bool is_q = h < heads;
+  float2 v[NP];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int d = 2 * (lane + 32 * j);
+    float2 x = make_float2(0.f, 0.f);
+    if (d < dim) x.x = src[d] + (bias ? bias[col + d] : 0.f);
+    if (d + 1 < dim) x.y = src[d + 1] + (bias ? bias[col + d + 1] : 0.f);
+    if (d < rot) {
+      const float2 t = gp_turn[d / 2];
+      x = make_float2(x.x * t.x - x.y * t.y, x.y * t.x + x.x * t.y);
+    }
+    v[j] = x;
+    ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
+  }
+  ss = warp_sum(ss);
+  const float r = norm ? 1.f / sqrtf(ss / (float)dim + eps) : 1.f;
+  T* dst;
+  if (is_q) {
+    dst = q_out + ((size_t)row * heads + h) * hp;
+  } else {
+    const int blk = block_table[(size_t)row_slot[row] * max_blocks + pos / kv_block];
+    if (blk < 0) { if (lane == 0) set_status(status, ST_BOUNDS); return; }
+    const size_t at = (((size_t)blk * kv_block + pos % kv_block) * kv_heads + (h - heads)) * hp;
+    dst = k_cache + at;
+    const int vc = v_off + (h - heads) * dim;
+    const float* vs = proj + (size_t)row * ldp + vc;
+    for (int d = 2 * lane; d < hp; d += 64) {
+      const float a = d < dim ? vs[d] + (bias ? bias[vc + d] : 0.f) : 0.f;
+      const float b = d + 1 < dim ? vs[d + 1] + (bias ? bias[vc + d + 1] : 0.f) : 0.f;
+      Elem<T>::store2(v_cache + at + d, a, b);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int d = 2 * (lane + 32 * j);
+    if (d < hp) Elem<T>::store2(dst + d, v[j].x * r, v[j].y * r);
+  }
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* bias,
+                           const double* inv_freq, const int* row_slot, const int* row_pos, const int* block_table, int max_blocks,
+                           int kv_block, int rows, int heads, int kv_heads, int dim, int hp, int rot, int v_off, int norm, float eps,
+                           int f32, int* status, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (dim < 1 || dim > hp || hp % 64 || hp > 1024 || rot % 2 || rot > dim || (rot && !inv_freq)) return -1;
+  const dim3 grid(rows, (heads + kv_heads + GP_WARPS - 1) / GP_WARPS);
+  const size_t smem = (size_t)(rot / 2 + 1) * sizeof(float2);
+  auto go = [&](auto kern, auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    return (int)launch_pdl(kern, grid, dim3(GP_WARPS * 32), smem, s, (T*)q_out, (T*)k_cache, (T*)v_cache, proj, ldp, bias, inv_freq,
+                           row_slot, row_pos, block_table, max_blocks, kv_block, heads, kv_heads, dim, hp, rot, v_off, norm, eps, status);
+  };
+  using B = __nv_bfloat16;
+  if (hp <= 64) return f32 ? go(gqa_prep_kernel<float, 1>, (float*)0) : go(gqa_prep_kernel<B, 1>, (B*)0);
+  if (hp <= 128) return f32 ? go(gqa_prep_kernel<float, 2>, (float*)0) : go(gqa_prep_kernel<B, 2>, (B*)0);
+  if (hp <= 256) return f32 ? go(gqa_prep_kernel<float, 4>, (float*)0) : go(gqa_prep_kernel<B, 4>, (B*)0);
+  return f32 ? go(gqa_prep_kernel<float, 16>, (float*)0) : go(gqa_prep_kernel<B, 16>, (B*)0);
+}

@@ -6,8 +6,10 @@
 //                  out of the cache: it moves with the pages (parking, forks, resumed prefixes, rejected drafts) for free.
 //   latent_prep    both latents of a token from one fused projection: RMSNorm of the query latent, RMSNorm of the key / value
 //                  latent into its page
-//   latent_attn    few rows: every head attends the cached latents themselves (key projection folded into the query)
-//   add_normed     x += rms(y) * w on the 32-bit residual stream, plus the copy the next GEMM reads
+//   latent_attn    few rows: every head attends the cached latents themselves (key projection folded into the query); the same
+//                  kernel over separate keys and values of grouped heads, with a sink, is what grouped-query attention runs in 32
+//                  bits and at head widths the tensor-core kernels do not take
+//   add_normed     x += rms(y + bias) * w on the 32-bit residual stream, plus the next GEMM's operand: the new x or its norm
 //   norm_rows      rms(x[idx]) * w for the rows whose logits are wanted
 //   softcap        logits <- cap * tanh(logits / cap)
 //   gemm_f32       y = x W^T in 32 bits on the CUDA cores, optionally one product per head
@@ -15,34 +17,13 @@
 // The row kernels are templates over the element type of activations and cache (bf16, or fp32 for full-precision runs).
 #include "api_ext.h"
 #include "common.cuh"
+#include "elem.cuh"
 
 namespace fb {
 
-template <typename T> struct Elem;
-template <> struct Elem<float> {
-  static __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-  static __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-  static __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
-  static __device__ __forceinline__ float from(float v) { return v; }
-};
-template <> struct Elem<__nv_bfloat16> {
-  static __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(bf_lo(u.x), bf_hi(u.x), bf_lo(u.y), bf_hi(u.y));
-  }
-  static __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
-  }
-  static __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
-    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
-    return make_float2(bf_lo(u), bf_hi(u));
-  }
-  static __device__ __forceinline__ __nv_bfloat16 from(float v) { return f2bf(v); }
-};
-
 // ---- embedding -----------------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(256) embed_grams_kernel(float* __restrict__ x, T* __restrict__ xb, const T* __restrict__ table,
+__global__ void __launch_bounds__(256) embed_grams_kernel(float* __restrict__ x, T* __restrict__ xb, int copies, const T* __restrict__ table,
                                                           const T* __restrict__ grams, const int* __restrict__ tok,
                                                           const int* __restrict__ slot, const int* __restrict__ pos,
                                                           const int* __restrict__ block_table, int max_blocks, int kv_block,
@@ -85,7 +66,7 @@ __global__ void __launch_bounds__(256) embed_grams_kernel(float* __restrict__ x,
       v.x += g.x; v.y += g.y; v.z += g.z; v.w += g.w;
     }
     *reinterpret_cast<float4*>(x + (size_t)row * width + i) = v;
-    if (xb) Elem<T>::store4(xb + (size_t)row * width + i, v);
+    for (int c = 0; c < copies; ++c) Elem<T>::store4(xb + ((size_t)row * copies + c) * width + i, v);
   }
 }
 
@@ -101,23 +82,49 @@ __device__ __forceinline__ float row_rscale(const S* r, int n, int count, float 
   return 1.f / sqrtf(block_sum(ss, red) / (float)count + eps);
 }
 
-// x[row] += y[row] * rscale * w; xb = x in the GEMM operand type. `width` counts the true columns, `ld` the padded ones
-// (zeros beyond width).
+// x[row] += rms(y[row] + bias) * w (no w: x[row] = y[row] + bias); xb = the next operand: rms(x) * next_w, or x with next_w null. The
+// row waits in shared memory between the passes (every thread reads what it wrote itself). `width` counts the true columns, `ld` the
+// padded ones (zeros beyond width).
 template <typename T, typename S>
-__global__ void add_normed_kernel(float* __restrict__ x, T* __restrict__ xb, const S* __restrict__ y,
-                                  const float* __restrict__ w, int width, int ld, long ldy, float eps) {
+__global__ void add_normed_kernel(float* __restrict__ x, T* __restrict__ xb, long ldb, const S* __restrict__ y,
+                                  const float* __restrict__ bias, const float* __restrict__ w, const float* __restrict__ next_w,
+                                  int width, int ld, long ldy, float eps) {
+  extern __shared__ __align__(16) float an_row[];
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   const size_t row = blockIdx.x;
   const S* yr = y + row * ldy;
-  const float r = row_rscale<S>(yr, ld, width, eps, red);
+  float ss = 0.f;
   for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-    const float4 v = Elem<S>::load4(yr + i), ww = *reinterpret_cast<const float4*>(w + i);
-    float4 a = *reinterpret_cast<const float4*>(x + row * ld + i);
-    a.x += v.x * r * ww.x; a.y += v.y * r * ww.y; a.z += v.z * r * ww.z; a.w += v.w * r * ww.w;
+    float4 v = Elem<S>::load4(yr + i);
+    if (bias) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + i);
+      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+    }
+    *reinterpret_cast<float4*>(an_row + i) = v;
+    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+  }
+  const float r = w ? 1.f / sqrtf(block_sum(ss, red) / (float)width + eps) : 0.f;
+  ss = 0.f;
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    float4 a = *reinterpret_cast<const float4*>(an_row + i);
+    if (w) {
+      const float4 ww = *reinterpret_cast<const float4*>(w + i), xx = *reinterpret_cast<const float4*>(x + row * ld + i);
+      a.x = xx.x + a.x * r * ww.x; a.y = xx.y + a.y * r * ww.y; a.z = xx.z + a.z * r * ww.z; a.w = xx.w + a.w * r * ww.w;
+    }
     *reinterpret_cast<float4*>(x + row * ld + i) = a;
-    if (xb) Elem<T>::store4(xb + row * ld + i, a);
+    if (next_w) *reinterpret_cast<float4*>(an_row + i) = a;
+    else if (xb) Elem<T>::store4(xb + row * ldb + i, a);
+    ss = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, ss))));
+  }
+  if (!next_w) return;
+  const float r2 = 1.f / sqrtf(block_sum(ss, red) / (float)width + eps);
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(an_row + i);
+    const float4 ww = *reinterpret_cast<const float4*>(next_w + i);
+    v.x *= r2 * ww.x; v.y *= r2 * ww.y; v.z *= r2 * ww.z; v.w *= r2 * ww.w;
+    Elem<T>::store4(xb + row * ldb + i, v);
   }
 }
 
@@ -191,16 +198,20 @@ __global__ void relu2_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16*
 
 // ---- attention over the cached latents, CUDA cores ---------------------------------------------------------------------
 // grid (rows, heads, splits), 4 warps striding over the keys with an online softmax; a lane owns columns 64 j + 2 lane, + 1.
-// lat = 64 nl with nl <= NJ. One split writes the normalised output itself, more leave partials for the merge.
+// lat = 64 nl with nl <= NJ. One split writes the normalised output itself, more leave partials for the merge. KV: cache rows are
+// [kv_heads][lat] of keys with the values in v_cache (else one latent row, keys and values alike); sink: a number per head that
+// joins the denominator.
 constexpr int LA_WARPS = 4;
+constexpr float LOG2E = 1.4426950408889634f;
 
-template <typename T, int NJ>
+template <typename T, int NJ, bool KV>
 __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restrict__ out, float* __restrict__ o_part,
                                                                     float* __restrict__ ml_part, const T* __restrict__ q,
-                                                                    const T* __restrict__ cache, const int* __restrict__ row_slot,
+                                                                    const T* __restrict__ cache, const T* __restrict__ v_cache,
+                                                                    const float* __restrict__ sink, const int* __restrict__ row_slot,
                                                                     const int* __restrict__ row_kvlen,
                                                                     const int* __restrict__ block_table, int max_blocks,
-                                                                    int kv_block, int heads, int lat, int nsplit,
+                                                                    int kv_block, int heads, int kv_heads, int lat, int nsplit,
                                                                     float scale_log2, int* status) {
   extern __shared__ float so[];                            // [warps][lat]
   __shared__ float sml[LA_WARPS][2];
@@ -226,7 +237,9 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
   for (int t = lo + warp; t < hi; t += LA_WARPS) {
     const int blk = bt[t / kv_block];
     if (blk < 0) { if (lane == 0) set_status(status, ST_BOUNDS); break; }
-    const T* kr = cache + ((size_t)blk * kv_block + t % kv_block) * lat + 2 * lane;
+    size_t at = (size_t)blk * kv_block + t % kv_block;
+    if constexpr (KV) at = at * kv_heads + h / (heads / kv_heads);
+    const T* kr = cache + at * lat + 2 * lane;
     float2 k[NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) k[j] = j < nl ? Elem<T>::load2(kr + 64 * j) : make_float2(0.f, 0.f);
@@ -237,6 +250,11 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
     const float mn = fmaxf(m, s);
     const float a = exp2f(m - mn), p = exp2f(s - mn);
     l = l * a + p;
+    if constexpr (KV) {
+      const T* vr = v_cache + at * lat + 2 * lane;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) k[j] = j < nl ? Elem<T>::load2(vr + 64 * j) : make_float2(0.f, 0.f);
+    }
 #pragma unroll
     for (int j = 0; j < NJ; ++j) { o[j].x = fmaf(p, k[j].x, o[j].x * a); o[j].y = fmaf(p, k[j].y, o[j].y * a); }
     m = mn;
@@ -255,7 +273,8 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
     Ls += sml[w][1] * f[w];
   }
   const size_t pidx = ((size_t)row * heads + h) * nsplit + split;
-  const float inv = nsplit == 1 ? (Ls > 0.f ? 1.f / Ls : 0.f) : 1.f;
+  const float den = Ls + (sink && nsplit == 1 ? exp2f(sink[h] * LOG2E - M) : 0.f);
+  const float inv = nsplit == 1 ? (den > 0.f ? 1.f / den : 0.f) : 1.f;
   for (int d = threadIdx.x; d < lat; d += blockDim.x) {
     float acc = 0.f;
 #pragma unroll
@@ -272,8 +291,8 @@ constexpr int LG_GROUPS = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __restrict__ out, const float* __restrict__ o_part,
-                                                                       const float* __restrict__ ml_part, int heads, int nsplit,
-                                                                       int lat) {
+                                                                       const float* __restrict__ ml_part,
+                                                                       const float* __restrict__ sink, int heads, int nsplit, int lat) {
   extern __shared__ float sf[];                            // [nsplit] factors, then [groups][lat] partial sums
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -290,6 +309,7 @@ __global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __rest
     Ls += f == 0.f ? 0.f : ml_part[(pbase + s) * 2 + 1] * f;
   }
   Ls = block_sum(Ls, red);                                 // (its barriers publish the factors)
+  if (sink) Ls += exp2f(sink[blockIdx.y] * LOG2E - M);
   const float inv = Ls > 0.f ? 1.f / Ls : 0.f;
   float* sums = sf + nsplit;
   for (int d = col; d < lat; d += 512) {
@@ -619,29 +639,42 @@ using bf16 = __nv_bfloat16;
 
 static int row_threads(int width) { return width >= 4096 ? 512 : width >= 1024 ? 256 : 128; }
 
-extern "C" int fb_embed_grams(float* x, void* xb, const void* table, const void* grams, const int* tok, const int* slot,
+extern "C" int fb_embed_grams(float* x, void* xb, int copies, const void* table, const void* grams, const int* tok, const int* slot,
                               const int* pos, const int* block_table, int max_blocks, int kv_block, int* tok_pages, int rows,
                               int width, int vocab, float scale, long buckets, long mul_prev, long mul_cur, int f32, int* status,
                               cudaStream_t s) {
   if (rows <= 0) return 0;
   if (width % 4 || (grams && (buckets <= 0 || !tok_pages))) return -1;
   if (f32)
-    return (int)launch_pdl(embed_grams_kernel<float>, dim3(rows), dim3(256), 0, s, x, (float*)xb, (const float*)table,
+    return (int)launch_pdl(embed_grams_kernel<float>, dim3(rows), dim3(256), 0, s, x, (float*)xb, copies, (const float*)table,
                            (const float*)grams, tok, slot, pos, block_table, max_blocks, kv_block, tok_pages, width, vocab, scale,
                            (unsigned long long)buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, status);
-  return (int)launch_pdl(embed_grams_kernel<bf16>, dim3(rows), dim3(256), 0, s, x, (bf16*)xb, (const bf16*)table, (const bf16*)grams,
+  return (int)launch_pdl(embed_grams_kernel<bf16>, dim3(rows), dim3(256), 0, s, x, (bf16*)xb, copies, (const bf16*)table, (const bf16*)grams,
                          tok, slot, pos, block_table, max_blocks, kv_block, tok_pages, width, vocab, scale,
                          (unsigned long long)buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, status);
 }
 
-// y: fp32 (y_f32) or bf16 rows of stride ldy; xb: bf16 copy of x, or null
-extern "C" int fb_add_normed(float* x, void* xb, const void* y, int y_f32, const float* w, int rows, int width, int ld, long ldy,
-                             float eps, cudaStream_t s) {
+// y: fp32 (y_f32) or bf16 rows of stride ldy; xb: rows of stride ldb in the operand type (xb_f32), or null; bias, w, next_w: ld
+// floats or null
+extern "C" int fb_add_normed(float* x, void* xb, int xb_f32, long ldb, const void* y, int y_f32, const float* bias, const float* w,
+                             const float* next_w, int rows, int width, int ld, long ldy, float eps, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (ld % 4 || ldy % 4) return -1;
+  if (ld % 4 || ldy % 4 || ldb % 4 || (next_w && !xb) || ld > 49152) return -1;
   const dim3 g(rows), b(row_threads(ld));
-  if (y_f32) return (int)launch_pdl(add_normed_kernel<bf16, float>, g, b, 0, s, x, (bf16*)xb, (const float*)y, w, width, ld, ldy, eps);
-  return (int)launch_pdl(add_normed_kernel<bf16, bf16>, g, b, 0, s, x, (bf16*)xb, (const bf16*)y, w, width, ld, ldy, eps);
+  const size_t smem = (size_t)ld * 4;
+  auto go = [&](auto kern, auto* xo, const auto* yi) {
+    if (smem > 40 * 1024) {
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return (int)e;
+    }
+    return (int)launch_pdl(kern, g, b, smem, s, x, xo, ldb, yi, bias, w, next_w, width, ld, ldy, eps);
+  };
+  if (xb_f32) {
+    if (!y_f32) return -1;
+    return go(add_normed_kernel<float, float>, (float*)xb, (const float*)y);
+  }
+  if (y_f32) return go(add_normed_kernel<bf16, float>, (bf16*)xb, (const float*)y);
+  return go(add_normed_kernel<bf16, bf16>, (bf16*)xb, (const bf16*)y);
 }
 
 extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps,
@@ -680,28 +713,30 @@ extern "C" int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaS
 }
 
 template <typename T>
-static int latent_merge(void* out, const float* o_part, const float* ml_part, int rows, int heads, int nsplit, int lat, cudaStream_t s) {
+static int latent_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int lat,
+                        cudaStream_t s) {
   return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128 * LG_GROUPS),
-                         (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out, o_part, ml_part, heads, nsplit, lat);
+                         (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out, o_part, ml_part, sink, heads, nsplit, lat);
 }
 
-template <typename T>
-static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
-                       const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat,
-                       int nsplit, float scale_log2, int* status, cudaStream_t s) {
+template <typename T, bool KV>
+static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const void* v_cache, const float* sink,
+                       const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
+                       int kv_heads, int lat, int nsplit, float scale_log2, int* status, cudaStream_t s) {
   const dim3 grid(rows, heads, nsplit);
   const size_t smem = (size_t)LA_WARPS * lat * 4;
   auto go = [&](auto kern) {
-    return (int)launch_pdl(kern, grid, dim3(LA_WARPS * 32), smem, s, (T*)out, o_part, ml_part, (const T*)q, (const T*)cache, row_slot,
-                           row_kvlen, block_table, max_blocks, kv_block, heads, lat, nsplit, scale_log2, status);
+    return (int)launch_pdl(kern, grid, dim3(LA_WARPS * 32), smem, s, (T*)out, o_part, ml_part, (const T*)q, (const T*)cache,
+                           (const T*)v_cache, sink, row_slot, row_kvlen, block_table, max_blocks, kv_block, heads, kv_heads, lat, nsplit,
+                           scale_log2, status);
   };
   int rc;
-  if (lat <= 128) rc = go(latent_attn_kernel<T, 2>);
-  else if (lat <= 256) rc = go(latent_attn_kernel<T, 4>);
-  else if (lat <= 512) rc = go(latent_attn_kernel<T, 8>);
-  else rc = go(latent_attn_kernel<T, 16>);
+  if (lat <= 128) rc = go(latent_attn_kernel<T, 2, KV>);
+  else if (lat <= 256) rc = go(latent_attn_kernel<T, 4, KV>);
+  else if (lat <= 512) rc = go(latent_attn_kernel<T, 8, KV>);
+  else rc = go(latent_attn_kernel<T, 16, KV>);
   if (rc || nsplit == 1) return rc;
-  return latent_merge<T>(out, o_part, ml_part, rows, heads, nsplit, lat, s);
+  return latent_merge<T>(out, o_part, ml_part, sink, rows, heads, nsplit, lat, s);
 }
 
 // out [rows][heads][lat]; partials (nsplit > 1): o_part rows * heads * nsplit * lat floats, ml_part two per record
@@ -711,10 +746,32 @@ extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const vo
   if (rows <= 0) return 0;
   if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
   const float sl = scale * 1.4426950408889634f;
-  return f32 ? latent_attn<float>(out, o_part, ml_part, q, cache, row_slot, row_kvlen, block_table, max_blocks, kv_block, rows, heads,
-                                  lat, nsplit, sl, status, s)
-             : latent_attn<bf16>(out, o_part, ml_part, q, cache, row_slot, row_kvlen, block_table, max_blocks, kv_block, rows, heads,
-                                 lat, nsplit, sl, status, s);
+  return f32 ? latent_attn<float, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
+                                         kv_block, rows, heads, 1, lat, nsplit, sl, status, s)
+             : latent_attn<bf16, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
+                                        kv_block, rows, heads, 1, lat, nsplit, sl, status, s);
+}
+
+// The same over separate keys and values: caches [page][kv_block][kv_heads][hd], q / out [rows][heads][hd]; sink: heads floats or null
+extern "C" int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache,
+                           const float* sink, const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks,
+                           int kv_block, int rows, int heads, int kv_heads, int hd, int nsplit, float scale, int f32, int* status,
+                           cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (hd % 64 || hd > 1024 || heads > 65535 || kv_heads <= 0 || heads % kv_heads || nsplit < 1 || nsplit > 4096) return -1;
+  const float sl = scale * LOG2E;
+  return f32 ? latent_attn<float, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
+                                        kv_block, rows, heads, kv_heads, hd, nsplit, sl, status, s)
+             : latent_attn<bf16, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
+                                       kv_block, rows, heads, kv_heads, hd, nsplit, sl, status, s);
+}
+
+// Merge of key splits alone (records as fb_attn_decode_mma leaves them), sink: heads floats or null
+extern "C" int fb_attn_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit,
+                             int hd, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (hd % 64 || hd > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
+  return latent_merge<bf16>(out, o_part, ml_part, sink, rows, heads, nsplit, hd, s);
 }
 
 // The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in
@@ -743,7 +800,7 @@ extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const voi
   switch (lat / 64) { FB_LM(1) FB_LM(2) FB_LM(3) FB_LM(4) FB_LM(5) FB_LM(6) FB_LM(7) FB_LM(8) }
 #undef FB_LM
   if (rc || nsplit == 1) return rc;
-  return latent_merge<bf16>(out, o_part, ml_part, rows, heads, nsplit, lat, s);
+  return latent_merge<bf16>(out, o_part, ml_part, nullptr, rows, heads, nsplit, lat, s);
 }
 
 // y [batch][M][N] = act(x [batch][M][K] w [batch][N][K]^T); row strides ldx / ldy, batch strides x_bs / w_bs / y_bs (elements)

@@ -406,7 +406,7 @@ def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> Non
     l, p, d = cfg.layers[i], f"l{i}.", gqa_dims(cfg, i)
     names = ("q", "k") if l.key_values else ("q", "k", "v")
     rows = torch.cat([w[p + n] for n in names])
-    out[p + "in_proj"] = _pad(rows, rows.shape[0], W)
+    out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     if l.bias:
         out[p + "in_bias"] = torch.cat([w[p + n + "_bias"].float() for n in names])
         out[p + "out_bias"] = _pad(w[p + "out_bias"].float(), W)
@@ -422,7 +422,7 @@ def _pack_cdelta(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> 
     * out_proj [width, ko]"""
     l, p, d = cfg.layers[i], f"l{i}.", delta_dims(cfg, i)
     rows = torch.cat([_pad(w[p + "a1"], d.ra, cfg.hidden), _pad(w[p + "g1"], d.rg, cfg.hidden)] + [w[p + n] for n in ("q", "k", "v", "b")])
-    out[p + "in_proj"] = _pad(rows, rows.shape[0], W)
+    out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     out[p + "conv"] = torch.cat([w[p + n + "_conv"].float() for n in ("q", "k", "v")]).contiguous()
     out[p + "decay_up"] = _pad(w[p + "a2"], l.heads * l.dim, d.ra)
     out[p + "gate_up_lr"] = _pad(w[p + "g2"], l.heads * l.vdim, d.rg)

@@ -17,6 +17,7 @@ import torch
 from .._ext import load
 from .extras import CudaExtras
 from .latent import CudaLatent
+from .mixers import CudaMixers
 from .qweight import Exl3Weight, ExpertsFP4, GgufWeight, QWeight, StackWeight
 
 GEMV_MAX_ROWS = 8
@@ -24,7 +25,7 @@ MOE_PAIR_ROWS = 64     # up to this many rows (the largest graph-captured step) 
                        # beyond as grouped GEMMs, which read the per-expert row counts on the host
 
 
-class CudaOps(CudaLatent, CudaExtras):
+class CudaOps(CudaLatent, CudaMixers, CudaExtras):
     name = "cuda"
 
     def __init__(self, device, dtype=torch.bfloat16):
@@ -165,8 +166,9 @@ class CudaOps(CudaLatent, CudaExtras):
     def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, out=None, act=None):
         """`act`: activation of the epilogue ("relu2": squared relu), not together with SwiGLU."""
         if self.dtype == torch.float32:
-            assert norm_w is None and res is None and not swiglu, "fp32 linears have an activation epilogue only"
-            return self.linear_f32(x, w, act, out)
+            assert norm_w is None and res is None, "fp32 linears have an activation epilogue only"
+            y = self.linear_f32(x, w, act, out)
+            return self.silu_mul_f32(y) if swiglu else y
         if act is not None and not isinstance(w, torch.Tensor):
             assert act == "relu2" and not swiglu and not out_f32
             return self.relu2(self.linear(x, w, norm_w=norm_w, eps=eps, res=res))      # packed weights: a pass of its own

@@ -174,6 +174,12 @@ class CudaLatent:
         self.C.softcap(logits, cap)
         return logits
 
+    def silu_mul_f32(self, gu):
+        y = self.empty(gu.shape[0], gu.shape[1] // 2, dtype=torch.float32, device=self.device)
+        self.launches += 1
+        self.C.silu_mul_f32(y, gu)
+        return y
+
     def linear_f32(self, x, w, act=None, out=None):
         """y = x W^T in 32 bits; 3-d operands: one product per head."""
         y = out if out is not None else self.empty(*x.shape[:-1], w.shape[-2], dtype=torch.float32, device=self.device)

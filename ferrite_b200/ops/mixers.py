@@ -11,6 +11,7 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as F
 
+LOWRANK_ROWS = 64     # up to this many rows (the largest graph-captured step) the low-rank products are one SIMT launch
 UNIT_EPS = 1e-6       # inside the root of the delta rule's unit queries and keys
 
 
@@ -81,3 +82,80 @@ class TorchMixers:
                 rec_state[slot] = S
                 conv_state[slot] = x[n:].to(conv_state.dtype)
         return y.to(self.dtype)
+
+
+class CudaMixers:
+    def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps):
+        q = self.empty(proj.shape[0], d.heads, d.hp, dtype=self.dtype, device=self.device)
+        self.launches += 1
+        self.C.gqa_prep(q, k_cache, v_cache, proj, bias, inv_freq, row_slot, row_pos, block_table, kv_block, d.dim, d.rot_dims, d.v_off,
+                        d.qk_norm, eps, self.status_word)
+        return q
+
+    def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out):
+        """Prompt groups go to the tcgen05 flash kernel (softmax weights as value + remainder); the others are split over their keys on
+        the mma.sync kernel. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
+        key splits; what is left of it is what fills the GPU."""
+        a, b = group.row_lo, group.row_hi
+        tc = self.dtype == torch.bfloat16 and d.hp in (64, 128, 256)
+        if group.prompt and tc and kv_block % 64 == 0:
+            self.launches += 1
+            flat = q.view(q.shape[0], -1)
+            rc = self.C.attn_prefill_tc(out, flat, k_cache, v_cache, flat, segs[0], segs[1], segs[2], segs[3], block_table, kv_block,
+                                        group.max_rows, d.heads, d.kv_heads, d.hp, False, self.status_word, scale=d.scale, exact_p=True, sink=sink)
+            assert rc == 0, "prompt attention: shape outside the tensor-core kernel"
+            return out
+        mma = tc and d.heads // d.kv_heads <= 64
+        per_group = max(1, 64 // max(1, d.heads // d.kv_heads))
+        ctas = (group.seg_hi - group.seg_lo) * -(-group.max_rows // per_group) * d.kv_heads if mma else (b - a) * d.heads
+        nsplit = max(1, min(nsplit, (4 if mma else 8) * self.sm_count // max(1, ctas)))
+        o_part = self.empty((b - a) * d.heads * nsplit * d.hp, dtype=torch.float32, device=self.device)
+        ml_part = self.empty((b - a) * d.heads * nsplit * 2, dtype=torch.float32, device=self.device)
+        self.launches += 2 if mma or nsplit > 1 else 1
+        self.C.gqa_attn(out[a:b], o_part, ml_part, q[a:b], k_cache, v_cache, sink, segs[0], segs[1], segs[2], group.max_rows, row_slot[a:b],
+                        row_kvlen[a:b], block_table, kv_block, a, nsplit, d.scale, not mma, self.status_word)
+        return out
+
+    def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
+        """Few rows: both low-rank products in one launch, then one launch per group for the whole mixer. Prompt groups: two GEMMs,
+        the chunked scan, the gated norm. Sizes beyond the fused kernels (heads wider than 128) run conv, recurrence and norm apart."""
+        T = proj.shape[0]
+        sizes = [d.heads, d.kv_heads, d.dim, d.vdim, d.conv, d.q_off]
+        na = d.heads * d.dim
+        if T <= LOWRANK_ROWS:
+            up = self.empty(T, na + d.heads * d.vdim, dtype=torch.float32, device=self.device)
+            self.launches += 1
+            self.C.cd_lowrank(up, proj, w["decay_up"], w["gate_up_lr"])
+            decay, gate = up[:, :na], up[:, na:]
+        else:
+            decay = self.linear(proj[:, :d.ra], w["decay_up"], out_f32=True)
+            gate = self.linear(proj[:, d.ra:d.q_off], w["gate_up_lr"], out_f32=True)
+        out = self.empty(T, d.ko, dtype=self.dtype, device=self.device)
+        par = (w["conv"], w["A_log"], w["dt_bias"])
+        y = qkv = None
+        for g in groups:
+            segs = tuple(t[g.seg_lo:g.seg_hi] for t in (seg_slot, seg_row0, seg_nrows))
+            a, b = g.row_lo, g.row_hi
+            fused = max(d.dim, d.vdim) <= 128 and not (g.prompt and commit)
+            if fused:
+                self.launches += 1
+                self.C.cd_step(out, rec_state, conv_state, proj, decay, gate, *par, w["gnorm_w"], *segs, sizes, eps, commit)
+            else:
+                if y is None:
+                    y = self.empty(T, d.heads, d.vdim, dtype=torch.float32, device=self.device)
+                if g.prompt and commit and d.dim <= 128:
+                    nb = self.C.cd_chunk_scratch_bytes(T, g.seg_hi - g.seg_lo, d.heads, d.dim)
+                    self.launches += 2
+                    self.C.cd_chunk(y, rec_state, self.scratch("cd_chunk", nb // 4, torch.float32), conv_state, proj, decay, *par, *segs,
+                                    g.max_rows, sizes)
+                else:
+                    if qkv is None:
+                        qkv = self.empty(T, d.channels, dtype=self.dtype, device=self.device)
+                    self.launches += 2
+                    self.C.cd_rec(y, rec_state, qkv, conv_state, proj, decay, *par, *segs, g.max_rows, sizes, commit)
+                self.launches += 1
+                self.C.gated_norm_sigmoid(out[a:b], y[a:b], gate[a:b], w["gnorm_w"], eps)
+            if commit and not (fused and d.heads == d.kv_heads):
+                self.launches += 1
+                self.C.cd_tail(rec_state, conv_state, proj, w["conv"], *segs, sizes)
+        return out
