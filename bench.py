@@ -100,10 +100,11 @@ def main():
     ap.add_argument("--model", default="27b", choices=["27b", "moe80b", "mla671b"],
                     help="27b: the headline model. moe80b (80B-A3B hybrid MoE, fits one GPU with --dtype nvfp4) and mla671b "
                          "(needs --layers on one GPU) measure the same plain decode + 2K prefill on the MoE families")
-    ap.add_argument("--design", default="", choices=["", "zototar"],
-                    help="zototar: instead of the headline workload, prefill and decode throughput of the Zototar design beside the dense "
-                         "MLA model of equal size (random weights), at the sizes of --sizes; one JSON line")
-    ap.add_argument("--sizes", default="2k,4k,7k", help="with --design: sizes to measure (2k | 4k | 7k: model width)")
+    ap.add_argument("--design", default="", choices=["", "zototar", "dofunex"],
+                    help="instead of the headline workload, prefill and decode throughput of a design of listed layers beside the closest "
+                         "other model of equal size (random weights; zototar: the dense MLA model, dofunex: the dense Gated DeltaNet hybrid), "
+                         "at the sizes of --sizes; one JSON line")
+    ap.add_argument("--sizes", default="", help="with --design: sizes to measure (model widths; zototar 2k,4k,7k, dofunex 2k,4k,5k)")
     ap.add_argument("--fused-layers", default="auto", choices=["auto", "on", "off"],
                     help="plain decode rows: one persistent kernel per layer (auto = when tensor parallel)")
     ap.add_argument("--no-extras", action="store_true", help="only the headline decode measurement and the 2K prefill")
@@ -138,11 +139,12 @@ def main():
     assert world == args.gpus, f"--gpus {args.gpus} but WORLD_SIZE {world}: launch with torch.distributed.run"
 
     if args.design:
-        from ferrite_b200.utils.design_bench import models
+        from ferrite_b200.utils.design_bench import DESIGNS, models
         sampler = ClockSampler(local)
         sampler.start()
-        res = models([x for x in args.sizes.split(",") if x], args.steps, args.warmup, dev, args.ctx)
-        print(json.dumps({"design": args.design, "beside": "dense MLA model of equal width, heads, latent and parameter count", "steps": args.steps,
+        sizes = args.sizes or DESIGNS[args.design][3]
+        res = models([x for x in sizes.split(",") if x], args.steps, args.warmup, dev, args.ctx, args.design)
+        print(json.dumps({"design": args.design, "beside": DESIGNS[args.design][2], "steps": args.steps,
                           "warmup": args.warmup, "ctx": args.ctx, "dtype": "bf16", "data": "synthetic, random-init weights",
                           "l2": "every step streams all weights (> 1 GB)", "clocks": sampler.stop(), "sizes": res}))
         return 0

@@ -17,7 +17,7 @@ import torch
 import torch.nn.functional as F
 
 from ..config import ModelConfig
-from .weights import Weights
+from .weights import Weights, rope_frequencies
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, centred: bool = True) -> torch.Tensor:
@@ -86,6 +86,7 @@ class RefState:
         self.v: List[List[torch.Tensor]] = [[] for _ in range(cfg.n_layers)]
         self.conv = [torch.zeros(cfg.conv_dim, cfg.conv_k - 1) for _ in range(cfg.n_layers)]
         self.rec = [torch.zeros(cfg.lin_v_heads, cfg.lin_dk, cfg.lin_dv) for _ in range(cfg.n_layers)]
+        self.run: Dict[tuple, object] = {}       # rows and states of the runs of listed layers, by (what, run)
 
     def clone(self) -> "RefState":
         s = RefState(self.cfg)
@@ -94,6 +95,7 @@ class RefState:
         s.v = [list(x) for x in self.v]
         s.conv = [x.clone() for x in self.conv]
         s.rec = [x.clone() for x in self.rec]
+        s.run = {k: list(x) if isinstance(x, list) else x for k, x in self.run.items()}
         return s
 
 
@@ -203,18 +205,67 @@ class RefModel:
         pr = torch.softmax(torch.einsum("hd,thd->ht", q, k) * l.scale, -1)
         return w[p + "out_proj"] @ torch.einsum("ht,thv->hv", pr, v).reshape(-1)
 
+    def _gqa(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """Grouped-query attention of listed layers; run r's keys and values are its own."""
+        l, w, p = self.cfg.layers[i], self.w, f"l{i}."
+        proj = {n: w[p + n] @ x + (w[p + n + "_bias"] if l.bias else 0.0) for n in ("q", "k") + (() if l.key_values else ("v",))}
+        ang = st.pos * rope_frequencies(l)
+        c, s = ang.cos().float(), ang.sin().float()
+
+        def turned(z):
+            z = z.clone()
+            a, b = z[:, 0:l.rot_dims:2].clone(), z[:, 1:l.rot_dims:2].clone()
+            z[:, 0:l.rot_dims:2], z[:, 1:l.rot_dims:2] = a * c - b * s, b * c + a * s
+            return z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + self.cfg.eps) if l.qk_norm else z
+        q, k = turned(proj["q"].view(l.heads, l.dim)), proj["k"].view(l.kv_heads, l.dim)
+        st.run.setdefault(("k", r), []).append(turned(k))
+        st.run.setdefault(("v", r), []).append(k if l.key_values else proj["v"].view(l.kv_heads, l.vdim))
+        own = torch.arange(l.heads) // (l.heads // l.kv_heads)
+        K, V = torch.stack(st.run["k", r])[:, own], torch.stack(st.run["v", r])[:, own]
+        e = torch.exp(torch.einsum("hd,thd->ht", q, K) * l.scale)
+        pr = e / (e.sum(-1, keepdim=True) + (torch.exp(w[p + "sink"])[:, None] if l.sink else 0.0))
+        return w[p + "out_proj"] @ torch.einsum("ht,thd->hd", pr, V).reshape(-1) + (w[p + "out_bias"] if l.bias else 0.0)
+
+    def _cdelta(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """Delta rule with a decay per key channel; run r's state and convolution inputs are its own."""
+        l, w, p = self.cfg.layers[i], self.w, f"l{i}."
+        H, G, D, V = l.heads, l.kv_heads, l.dim, l.vdim
+        out = {}
+        for n in "qkv":
+            buf = st.run.setdefault((n + "_conv", r), [])
+            buf.append(w[p + n] @ x)
+            out[n] = F.silu(sum(z * w[p + n + "_conv"][:, l.conv - 1 - j] for j, z in enumerate(reversed(buf[-l.conv:]))))
+        own = torch.arange(H) // (H // G)
+        unit = lambda z: z * torch.rsqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6)
+        q, k = unit(out["q"].view(G, D))[own] / math.sqrt(D), unit(out["k"].view(G, D))[own]
+        g = torch.exp(-torch.exp(w[p + "A_log"])[:, None] * softplus(w[p + "a2"] @ (w[p + "a1"] @ x) + w[p + "dt_bias"]).view(H, D))
+        S = st.run.get(("rec", r), torch.zeros(H, D, V)) * g[:, :, None]
+        u = torch.sigmoid(w[p + "b"] @ x)[:, None] * (out["v"].view(H, V) - torch.einsum("hdv,hd->hv", S, k))
+        S = st.run["rec", r] = S + k[:, :, None] * u[:, None, :]
+        o = rmsnorm(torch.einsum("hdv,hd->hv", S, q), w[p + "gnorm_w"], self.cfg.eps, False)
+        return w[p + "out_proj"] @ (o * torch.sigmoid(w[p + "g2"] @ (w[p + "g1"] @ x)).view(H, V)).reshape(-1)
+
     def _token_out_norm(self, t: int, st: RefState, tap: list) -> torch.Tensor:
         """One token through a model with norms on the sublayers' outputs: the row before the final norm."""
         c, w = self.cfg, self.w
         x = w["embed"][t] * c.embed_scale
         if c.gram_buckets:
             x = x + w["bigram"][c.gram_buckets if st.prev is None else (st.prev * c.gram_mul_prev + t * c.gram_mul_cur) % c.gram_buckets]
-        st.prev = t
-        for i, l in enumerate(c.layers):
-            x = x + rmsnorm(self._latent(i, x, st), w[f"l{i}.mix_norm"], c.eps, False)
+        st.prev, x0 = t, x
+        before = lambda name: rmsnorm(x, w[name], c.eps, False) if c.pre_norm else x
+        for run in c.layer_runs:
+            i, l = run.layer, c.layers[run.layer]
+            p = f"l{i}."
+            if run.enter is not None:
+                x = w["loop_in"] @ torch.cat([x, x0]) + w["loop_step"][run.enter]
+            h = before(p + "pre_norm")
+            y = self._latent(i, h, st) if l.mixer == "latent" else (self._gqa if l.mixer == "gqa" else self._cdelta)(run.index, i, h, st)
+            x = x + c.residual_mult * rmsnorm(y, w[p + "mix_norm"], c.eps, False)
             if l.ff:
-                x = x + rmsnorm(w[f"l{i}.down"] @ torch.relu(w[f"l{i}.up"] @ x).square(), w[f"l{i}.ffn_norm"], c.eps, False)
-            if i in c.tap_layers:
+                h = before(p + "ffn_pre_norm")
+                act = F.silu(w[p + "gate"] @ h) * (w[p + "up"] @ h) if l.act == "swiglu" else torch.relu(w[p + "up"] @ h).square()
+                x = x + c.residual_mult * rmsnorm(w[p + "down"] @ act, w[p + "ffn_norm"], c.eps, False)
+            if i in c.tap_layers and not any(q.layer == i and q.index > run.index for q in c.layer_runs):
                 tap.append(x.clone())
         return x
 
@@ -244,7 +295,7 @@ class RefModel:
             if c.out_norm:
                 x = self._token_out_norm(int(t), st, tap)
                 st.pos += 1
-                y = head @ rmsnorm(x, w["final_norm"], c.eps, False)
+                y = head @ rmsnorm(x, w["final_norm"], c.eps, False) * c.logit_scale
                 logits.append(c.logit_softcap * torch.tanh(y / c.logit_softcap) if c.logit_softcap else y)
                 taps.append(tap)
                 continue

@@ -1,9 +1,10 @@
-"""Two latent-attention designs side by side: Zototar (no positions, output norms on a 32-bit residual stream, latents shared by
-pairs of layers) and the dense MLA model of the same width, heads, latent and parameter count, with random weights.
+"""Designs of listed layers, each beside the framework's closest other model of the same width, heads and parameter count, with
+random weights: Zototar (latent attention without positions) beside the dense MLA model, Dofunex (delta rules with a decay per
+channel, every fourth layer attention) beside the dense Gated DeltaNet hybrid.
 
-`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()` times every
-kernel of the first beside the kernel that does the same job for the second and gives both as fractions of their rooflines.
-Both print nothing and return plain dictionaries; `bench.py --design zototar` and `microbench latent` print them.
+`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()` /
+`kernels_dofunex()` time every kernel of the first beside the kernel that does the same job for the second and give both as fractions
+of their rooflines. They print nothing and return plain dictionaries; `bench.py --design ...` and `microbench latent|cdelta` print them.
 """
 from __future__ import annotations
 
@@ -12,7 +13,7 @@ from typing import Dict, List
 
 import torch
 
-from ..config import EngineConfig, ModelConfig, zototar
+from ..config import EngineConfig, ModelConfig, dofunex, zototar
 from .microbench import Timer, graph_time, peaks, rnd
 
 SIZES = {       # name: width, heads, query latent, feed-forward width, layers
@@ -31,6 +32,26 @@ def pair(size: str):
                     n_kv=h, rotary_dim=ROPE, rope_theta=1e4, attn_gate=False, vocab=VOCAB, tie_embeddings=False, kv_lora=KV_RANK,
                     q_lora=qr, rope_head_dim=ROPE, nope_head_dim=DIM, v_head_dim=DIM)
     return a, b
+
+
+def pair_dofunex(size: str):
+    """(Dofunex model, dense hybrid of Gated DeltaNet and gated attention layers) of one size, every fourth layer attention; the
+    feed-forward of the second makes up for its wider gates."""
+    w, h, kv, ff, n = SIZES_DOFUNEX[size]
+    a = dofunex(w, n, h, kv, ff, VOCAB, name=f"dofunex-{size}")
+    kw = dict(name=f"hybrid-{size}", hidden=w, n_layers=n, full_attn_every=4, head_dim=DIM, n_q=h, n_kv=kv, rotary_dim=DIM, lin_k_heads=h,
+              lin_v_heads=h, lin_dk=DIM, lin_dv=DIM, vocab=VOCAB, tie_embeddings=False)
+    spare = a.param_count() - ModelConfig(inter=0, **kw).param_count()
+    return a, ModelConfig(inter=max(256, round(spare / (3 * w * n) / 256) * 256), **kw)
+
+
+SIZES_DOFUNEX = {       # name: width, heads, key / value heads of the attention layers, feed-forward width, layers
+    "2k": (2048, 16, 4, 6144, 16),
+    "4k": (4096, 32, 8, 11008, 8),
+    "5k": (5120, 40, 8, 17408, 8),
+}
+DESIGNS = {"zototar": (pair, "mla_dense", "dense MLA model of equal width, heads, latent and parameter count", "2k,4k,7k"),
+           "dofunex": (pair_dofunex, "hybrid_dense", "dense Gated DeltaNet hybrid of equal width, heads and parameter count", "2k,4k,5k")}
 
 
 def run_model(cfg: ModelConfig, ctx: int, prompts: List[int], streams: List[int], steps: int, warmup: int, dev) -> Dict:
@@ -77,35 +98,43 @@ def run_model(cfg: ModelConfig, ctx: int, prompts: List[int], streams: List[int]
     return out
 
 
-def models(sizes: List[str], steps: int, warmup: int, dev, ctx: int = 2048) -> Dict:
+def models(sizes: List[str], steps: int, warmup: int, dev, ctx: int = 2048, design: str = "zototar") -> Dict:
     out = {}
+    of, other = DESIGNS[design][:2]
     for size in sizes:
-        a, b = pair(size)
+        a, b = of(size)
         ra = run_model(a, ctx, [2048, 8192], [1, 4, 16], steps, warmup, dev)
         rb = run_model(b, ctx, [2048, 8192], [1, 4, 16], steps, warmup, dev)
-        out[size] = {"zototar": ra, "mla_dense": rb, "ratio": {k: round(ra[k] / rb[k], 3) for k in ra if k.endswith("tok_s")}}
+        out[size] = {design: ra, other: rb, "ratio": {k: round(ra[k] / rb[k], 3) for k in ra if k.endswith("tok_s")}}
     return out
 
 
+class _Rows:
+    """Collects {kernel, like, ms, like_ms, frac, like_frac}: times in a CUDA graph of calls over buffers that together exceed L2."""
+
+    def __init__(self, dev):
+        self.t, self.rows = Timer(dev, 3, 20, flush=False), []
+        self.hbm, self.tf, _ = peaks()
+
+    def timed(self, fn, nbytes: float, flops: float, bufs: int):
+        reps = max(4, min(40, int(-(-(400 << 20) // max(1, nbytes)))), bufs)
+        ms = graph_time(self.t, lambda: [fn(j % bufs) for j in range(reps)], reps)
+        return ms, max(nbytes / (self.hbm * 1e6), flops / (self.tf * 1e9)) / ms
+
+    def add(self, name, new, like_name, like):
+        (ms, fr), (lms, lfr) = self.timed(*new), self.timed(*like)
+        self.rows.append({"kernel": name, "ms": round(ms, 5), "frac": round(fr, 4), "like": like_name, "like_ms": round(lms, 5),
+                          "like_frac": round(lfr, 4)})
+
+
 def kernels(dev, heads: int = 32, width: int = 4096, ctx: int = 4096, prompt: int = 2048) -> List[Dict]:
-    """[{kernel, like, ms, like_ms, frac, like_frac}]: times in a CUDA graph of calls over buffers that together exceed L2."""
+    """Zototar's kernels beside those of the dense MLA model."""
     from ..models.weights import LatentDims
     from ..ops.cuda_ops import CudaOps
     from ..ops.latent import SegGroup, seg_groups
-    ops, t = CudaOps(dev), Timer(dev, 3, 20, flush=False)
-    hbm, tf, _ = peaks()
+    ops, acc = CudaOps(dev), _Rows(dev)
+    t, hbm, tf, rows, add = acc.t, acc.hbm, acc.tf, acc.rows, acc.add
     L, R, D, QR, kvb = KV_RANK, ROPE, DIM, 1536, 64
-    rows: List[Dict] = []
-
-    def timed(fn, nbytes: float, flops: float, bufs: int):
-        reps = max(4, min(40, int(-(-(400 << 20) // max(1, nbytes)))), bufs)
-        ms = graph_time(t, lambda: [fn(j % bufs) for j in range(reps)], reps)
-        return ms, max(nbytes / (hbm * 1e6), flops / (tf * 1e9)) / ms
-
-    def add(name, new, like_name, like):
-        (ms, fr), (lms, lfr) = timed(*new), timed(*like)
-        rows.append({"kernel": name, "ms": round(ms, 5), "frac": round(fr, 3), "like": like_name, "like_ms": round(lms, 5),
-                     "like_frac": round(lfr, 3)})
 
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
     inv = torch.rand(R // 2, device=dev)
@@ -201,3 +230,106 @@ def kernels(dev, heads: int = 32, width: int = 4096, ctx: int = 4096, prompt: in
         "flash, bf16 softmax weights", (flash(False), 0.0, tri * heads * 4 * D, 1))
     assert ops.status() == 0
     return rows
+
+
+def kernels_dofunex(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, ctx: int = 4096, prompt: int = 2048) -> List[Dict]:
+    """Dofunex's kernels beside those of the dense hybrid (heads of 128 columns, four taps, ranks of 128)."""
+    from ..models.weights import DeltaDims, GqaDims
+    from ..ops.cuda_ops import CudaOps
+    from ..ops.latent import SegGroup
+    ops, acc = CudaOps(dev), _Rows(dev)
+    add = acc.add
+    D, kvb, K, R, H, G = DIM, 64, 4, 128, heads, kv_heads
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    inv, inv64 = torch.rand(D // 2, device=dev), torch.rand(D // 2, device=dev, dtype=torch.float64)
+    gd, sink = GqaDims(H, G, D, D, D ** -0.5, D, H * D, True), f32(H)
+    nw = rnd(D)
+    # rows between the products
+    for m in (1, 16, prompt):
+        bufs = max(1, min(8, (400 << 20) // (m * width * 4)))
+        x0, y0 = [f32(m, width) for _ in range(bufs)], [f32(m, width) for _ in range(bufs)]
+        xb, yb = [rnd(m, width) for _ in range(bufs)], [rnd(m, width) for _ in range(bufs)]
+        w32, w16 = torch.ones(width, device=dev), rnd(width)
+        add(f"add_normed (bias, norm of y, add, next norm), {m} rows", (lambda j: ops.add_normed(x0[j], y0[j], w32, width, 1e-6, bias=w32, next_w=w32),
+                                                                          m * width * 14.0, 0.0, bufs),
+            "rmsnorm + residual", (lambda j: ops.rmsnorm(xb[j], w16, 1e-6, True, res=yb[j]), m * width * 8.0, 0.0, bufs))
+        # attention: projection to operands
+        nb = max(1, m // kvb)
+        many = m > kvb
+        slot = torch.zeros(m, dtype=torch.int32, device=dev) if many else torch.arange(m, dtype=torch.int32, device=dev)
+        pos = torch.arange(m, dtype=torch.int32, device=dev) if many else torch.zeros(m, dtype=torch.int32, device=dev)
+        bt = torch.arange((1 if many else m) * nb, dtype=torch.int32, device=dev).view(-1, nb)
+        kc, vc = rnd(bt.numel(), kvb, G, D), rnd(bt.numel(), kvb, G, D)
+        pb = 8 if many else 32
+        proj, bias = [f32(m, (H + G) * D) for _ in range(pb)], f32((H + G) * D)
+        pq = [rnd(m, (2 * H + 2 * G) * D) for _ in range(pb)]
+        add(f"gqa_prep, {m} rows, {H} / {G} heads", (lambda j: ops.gqa_prep(proj[j], gd, bias, inv64, slot, pos, bt, kc, vc, kvb, 1e-6),
+                                                      m * D * ((H + G) * 4.0 + (H + 2 * G) * 2.0), 0.0, pb),
+            "attn_prep", (lambda j: ops.attn_prep(pq[j], nw, nw, inv, slot, pos, bt, kc, vc, kvb, H, G, D, D, True, 1e-6),
+                          m * D * (H + 2 * G) * 4.0, 0.0, pb))
+        del x0, y0, xb, yb, proj, pq
+    for m in (1, 4, 16):
+        nb = ctx // kvb
+        bufs = max(1, min(8, (400 << 20) // (m * ctx * G * D * 4)))
+        kc, vc = [rnd(m * nb, kvb, G, D) for _ in range(bufs)], [rnd(m * nb, kvb, G, D) for _ in range(bufs)]
+        bt, slot = torch.arange(m * nb, dtype=torch.int32, device=dev).view(m, nb), torch.arange(m, dtype=torch.int32, device=dev)
+        kvlen, ones = torch.full((m,), ctx, dtype=torch.int32, device=dev), torch.ones(m, dtype=torch.int32, device=dev)
+        q, out, pj = rnd(m, H, D), rnd(m, H, D), rnd(m, 2 * H * D)
+        grp = SegGroup(0, m, 0, m, 1)
+        work = (m * ctx * G * D * 4.0, 4.0 * m * H * ctx * D, bufs)
+        add(f"decode attention + merge with sink, weights as value + remainder, {m} rows, {ctx} keys",
+            (lambda j: ops.gqa_attention(q, gd, kc[j], vc[j], sink, grp, slot, kvlen, (slot, slot, ones), bt, kvb, 64, out), *work), "attention + combine",
+            (lambda j: ops.attention(q, pj, kc[j], vc[j], slot, kvlen, bt, kvb, H, G, D, True, nsplit=64, segs=(slot, slot, ones, 1)), *work))
+        del kc, vc
+    T, nb = prompt, prompt // kvb
+    perm = torch.randperm(nb, device=dev).to(torch.int32).view(1, nb)
+    kc, vc, q, out, pj = rnd(nb, kvb, G, D), rnd(nb, kvb, G, D), rnd(T, H, D), rnd(T, H, D), rnd(T, 2 * H * D)
+    s0 = (i32([0]), i32([0]), i32([T]), i32([0]))
+    rslot, rlen = torch.zeros(T, dtype=torch.int32, device=dev), torch.arange(1, T + 1, dtype=torch.int32, device=dev)
+    grp = SegGroup(0, 1, 0, T, T, True)
+    work = (0.0, T * (T + 1) / 2.0 * H * 4 * D, 1)
+    add(f"prompt attention with sink, weights as value + remainder, {T} rows",
+        (lambda j: ops.gqa_attention(q, gd, kc, vc, sink, grp, rslot, rlen, s0, perm, kvb, 1, out), *work), "prompt attention, bf16 weights",
+        (lambda j: ops.attention_prefill(q, pj, kc, vc, *s0, perm, kvb, H, G, D, True, T), *work))
+    # delta rule
+    d = DeltaDims(H, H, D, D, K, R, R, H * D)
+    sizes = [H, H, D, D, K, d.q_off]
+    w = dict(decay_up=rnd(H * D, R, scale=R ** -0.5), gate_up_lr=rnd(H * D, R, scale=R ** -0.5), conv=f32(d.channels, K), A_log=f32(H),
+             dt_bias=f32(H * D) - 3, gnorm_w=f32(D))
+    cw, A, dtb, gw = rnd(3 * H * D, K), f32(H), f32(H), rnd(D)
+    for m in (1, 4, 16):
+        bufs = max(2, min(64, (400 << 20) // (m * H * D * D * 4)))
+        rec, tail = [f32(m, H, D, D) for _ in range(bufs)], [rnd(m, K - 1, d.channels) for _ in range(bufs)]
+        proj, pg = rnd(m, d.b_off + H), rnd(m, 4 * H * D + 2 * H)
+        up = f32(m, 2 * H * D)
+        slot, ones, out = torch.arange(m, dtype=torch.int32, device=dev), torch.ones(m, dtype=torch.int32, device=dev), rnd(m, H * D)
+        state = m * H * D * D * 8.0
+        add(f"cd_step, {m} rows, {H} heads", (lambda j: ops.C.cd_step(out, rec[j], tail[j], proj, up[:, :H * D], up[:, H * D:], w["conv"], w["A_log"],
+                                                                       w["dt_bias"], w["gnorm_w"], slot, slot, ones, sizes, 1e-6, True),
+                                               state + m * H * D * 24.0, 0.0, bufs), "gdn_step",
+            (lambda j: ops.gdn_step(pg, cw, rec[j], tail[j], A, dtb, gw, slot, slot, ones, H, H, D, D, 1e-6), state + m * H * D * 20.0, 0.0, bufs))
+        ups = [(rnd(H * D, R), rnd(H * D, R)) for _ in range(32)]
+        wo = [rnd(2 * H * D, R) for _ in range(32)]
+        xr = rnd(m, R)
+        add(f"cd_lowrank, {m} rows", (lambda j: ops.C.cd_lowrank(up, proj, *ups[j]), H * D * R * 4.0 + m * H * D * 8.0, 4.0 * m * H * D * R, 32),
+            "linear of the same bytes", (lambda j: ops.linear(xr, wo[j], out_f32=True), H * D * R * 4.0 + m * H * D * 8.0, 4.0 * m * H * D * R, 32))
+        del rec, tail
+    rec, tail = f32(1, H, D, D), rnd(1, K - 1, d.channels)
+    proj, pg = rnd(T, d.b_off + H), rnd(T, 4 * H * D + 2 * H)
+    decay = f32(T, H * D)
+    scratch = ops.scratch("cd_chunk", ops.C.cd_chunk_scratch_bytes(T, 1, H, D) // 4, torch.float32)
+    y, gate = f32(T, H, D), f32(T, H * D)
+    # 64-row chunks: the Gram products, the solve and the five products with the state, per head
+    fl = T / 64 * H * (4 * 64 * 64 * D + 64 * 64 * 64 / 3 + 6 * 64 * D * D + 4 * 64 * 64 * D)
+    one = (i32([0]), i32([0]), i32([T]))
+    add(f"cd_chunk (prep + scan), {T} rows, {H} heads",
+        (lambda j: ops.C.cd_chunk(y, rec, scratch, tail, proj, decay, w["conv"], w["A_log"], w["dt_bias"], *one, T, sizes), T * H * D * 14.0, fl, 1),
+        "gdn_conv + gdn_chunk",
+        (lambda j: ops.gdn_rec(ops.gdn_conv(pg, cw, tail, *one, 3 * H * D, T), pg, rec, tail, A, dtb, *one, H, H, D, D, 1e-6, chunked=True, max_rows=T),
+         T * H * D * 10.0, fl, 1))
+    gout = rnd(T, H * D)
+    add(f"gated head norm, {T} rows", (lambda j: ops.C.gated_norm_sigmoid(gout, y, gate, w["gnorm_w"], 1e-6), T * H * D * 10.0, 0.0, 1), "gated_norm",
+        (lambda j: ops.gated_norm(y.view(T, H * D), pg, 3 * H * D, gw, H, D, 1e-6), T * H * D * 8.0, 0.0, 1))
+    assert ops.status() == 0
+    return acc.rows
