@@ -50,7 +50,7 @@ __global__ void __launch_bounds__(256) cd_lowrank_kernel(float* __restrict__ out
 // form the decays. State: thread (col = tid % DVP, part = tid / DVP) holds DKP / PARTS rows of column col across the segment.
 constexpr int CD_THREADS = 512;
 
-template <typename T, int DKP, int DVP>
+template <typename T, int DKP, int DVP, int NT>
 __global__ void __launch_bounds__(CD_THREADS)
 cd_step_kernel(T* __restrict__ out, int ko, float* __restrict__ rec_state, T* __restrict__ conv_state, const T* __restrict__ proj, long ldp,
                const float* __restrict__ decay, long ldd, const float* __restrict__ gate, long ldg, const float* __restrict__ conv_w,
@@ -70,7 +70,7 @@ cd_step_kernel(T* __restrict__ out, int ko, float* __restrict__ rec_state, T* __
   const int idx = role == 0 ? tid : role == 1 ? tid - DKP : role == 2 ? tid - 2 * DKP : tid - 2 * DKP - DVP;
   const bool live = role < 4 && idx < (role == 2 ? L.vdim : L.dim);
   const int ch = role == 0 ? kh * L.dim + idx : role == 1 ? (L.kv_heads + kh) * L.dim + idx : 2 * L.kv_heads * L.dim + h * L.vdim + idx;
-  float w[CD_TAPS], win[CD_TAPS - 1], dtb = 0.f, expA = 0.f;
+  float w[NT], win[NT - 1], dtb = 0.f, expA = 0.f;
   if (live && role < 3) cd_load_taps(w, conv_w, ch, L.taps);
   if (live && role == 3) { dtb = dt_bias[h * L.dim + idx]; expA = expf(A_log[h]); }
   const float nw = col < L.vdim ? norm_w[col] : 0.f;
@@ -81,8 +81,8 @@ cd_step_kernel(T* __restrict__ out, int ko, float* __restrict__ rec_state, T* __
   T* tail = conv_state + (size_t)slot * (L.taps - 1) * C;
   if (live && role < 3)
 #pragma unroll
-    for (int j = 0; j < CD_TAPS - 1; ++j)
-      win[j] = cd_input(proj, ldp, L.q_off, tail, C, L.taps, row0, j - (CD_TAPS - 1), ch);
+    for (int j = 0; j < NT - 1; ++j)
+      win[j] = cd_input(proj, ldp, L.q_off, tail, C, L.taps, row0, j - (NT - 1), ch);
   float* Sg = rec_state + ((size_t)slot * L.heads + h) * L.dim * L.vdim;
   float S[RP];
 #pragma unroll
@@ -106,12 +106,12 @@ cd_step_kernel(T* __restrict__ out, int ko, float* __restrict__ rec_state, T* __
     const RowIn cur = nxt;
     if (r + 1 < n) nxt = fetch(r + 1);
     if (role < 2) {
-      const float cv = live ? cd_conv_step<T>(w, win, cur.x) : 0.f;
+      const float cv = live ? cd_conv_step<T, NT>(w, win, cur.x) : 0.f;
       (role == 0 ? qs : ks)[idx] = cv;
       const float sq = warp_sum(cv * cv);
       if ((tid & 31) == 0) ssq[role][idx >> 5] = sq;
     } else if (role == 2) {
-      vs[idx] = live ? cd_conv_step<T>(w, win, cur.x) : 0.f;
+      vs[idx] = live ? cd_conv_step<T, NT>(w, win, cur.x) : 0.f;
     } else if (role == 3) {
       gs[idx] = live ? expf(cd_log_decay(expA, cur.x + dtb)) : 0.f;
     }
@@ -176,8 +176,8 @@ cd_step_kernel(T* __restrict__ out, int ko, float* __restrict__ rec_state, T* __
   // every q / k channel belongs to one CTA only when heads do not share them; cd_tail writes the tail otherwise
   if (L.heads == L.kv_heads && live && role < 3)
 #pragma unroll
-    for (int j = 0; j < CD_TAPS - 1; ++j) {
-      const int i = j - (CD_TAPS - L.taps);
+    for (int j = 0; j < NT - 1; ++j) {
+      const int i = j - (NT - L.taps);
       if (i >= 0) tail[(size_t)i * C + ch] = Elem<T>::from(win[j]);
     }
 }
@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(256) cd_conv_kernel(T* __restrict__ out, const
   for (int j = 0; j < CD_TAPS - 1; ++j) win[j] = cd_input(proj, ldp, L.q_off, tail, C, L.taps, row0, r0 + j - (CD_TAPS - 1), c);
   for (int r = r0; r < min(n, r0 + 32); ++r)
     out[(size_t)(row0 + r) * C + c] =
-        Elem<T>::from(cd_conv_step<T>(w, win, Elem<T>::to(proj[(size_t)(row0 + r) * ldp + L.q_off + c])));
+        Elem<T>::from(cd_conv_step<T, CD_TAPS>(w, win, Elem<T>::to(proj[(size_t)(row0 + r) * ldp + L.q_off + c])));
 }
 
 // y [rows][heads][vdim] fp32. grid (ceil(vdim / 32), heads, segments), 8 warps: warp p holds rows p, p + 8, ... of 32 state columns
@@ -327,8 +327,12 @@ static int cd_step(void* out, int ko, float* rec, void* tail, const void* proj, 
     return (int)launch_pdl(kern, dim3(L.heads, nseg), dim3(CD_THREADS), 0, s, (T*)out, ko, rec, (T*)tail, (const T*)proj, ldp, decay, ldd,
                            gate, ldg, conv_w, A_log, dt_bias, norm_w, seg_slot, seg_row0, seg_nrows, L, eps, commit);
   };
-  if (L.dim <= 64) return L.vdim <= 64 ? go(cd_step_kernel<T, 64, 64>) : go(cd_step_kernel<T, 64, 128>);
-  return L.vdim <= 64 ? go(cd_step_kernel<T, 128, 64>) : go(cd_step_kernel<T, 128, 128>);
+  if (L.taps <= 4) {
+    if (L.dim <= 64) return L.vdim <= 64 ? go(cd_step_kernel<T, 64, 64, 4>) : go(cd_step_kernel<T, 64, 128, 4>);
+    return L.vdim <= 64 ? go(cd_step_kernel<T, 128, 64, 4>) : go(cd_step_kernel<T, 128, 128, 4>);
+  }
+  if (L.dim <= 64) return L.vdim <= 64 ? go(cd_step_kernel<T, 64, 64, CD_TAPS>) : go(cd_step_kernel<T, 64, 128, CD_TAPS>);
+  return L.vdim <= 64 ? go(cd_step_kernel<T, 128, 64, CD_TAPS>) : go(cd_step_kernel<T, 128, 128, CD_TAPS>);
 }
 
 template <typename T>

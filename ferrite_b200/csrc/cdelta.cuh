@@ -10,7 +10,7 @@
 
 namespace fb {
 
-constexpr int CD_TAPS = 8;              // most taps of a short convolution
+constexpr int CD_TAPS = 8;              // most taps of a short convolution; kernels come with room for NT = 4 and for all of them
 constexpr float CD_UNIT_EPS = 1e-6f;
 
 // Columns of the fused projection row [a1 (ra) | g1 (rg) | q (kv_heads dim) | k | v (heads vdim) | b (heads)]
@@ -28,11 +28,12 @@ __device__ __forceinline__ float cd_silu(float x) { return x / (1.f + expf(-x));
 // log of a decay
 __device__ __forceinline__ float cd_log_decay(float expA, float z) { return -expA * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))); }
 
-// Taps of channel c, right-aligned in CD_TAPS registers
-__device__ __forceinline__ void cd_load_taps(float (&w)[CD_TAPS], const float* conv_w, int c, int taps) {
+// Taps of channel c, right-aligned in NT registers
+template <int NT>
+__device__ __forceinline__ void cd_load_taps(float (&w)[NT], const float* conv_w, int c, int taps) {
 #pragma unroll
-  for (int j = 0; j < CD_TAPS; ++j) {
-    const int i = j - (CD_TAPS - taps);
+  for (int j = 0; j < NT; ++j) {
+    const int i = j - (NT - taps);
     w[j] = i >= 0 ? conv_w[(size_t)c * taps + i] : 0.f;
   }
 }
@@ -43,14 +44,14 @@ __device__ __forceinline__ float cd_input(const T* proj, long ldp, int q_off, co
   return r >= 1 - taps ? Elem<T>::to(tail[(size_t)(taps - 1 + r) * channels + c]) : 0.f;
 }
 // One step of the sliding window: the activated convolution, rounded to the type that the prompt kernels keep it in
-template <typename T>
-__device__ __forceinline__ float cd_conv_step(const float (&w)[CD_TAPS], float (&win)[CD_TAPS - 1], float x) {
-  float a = w[CD_TAPS - 1] * x;
+template <typename T, int NT>
+__device__ __forceinline__ float cd_conv_step(const float (&w)[NT], float (&win)[NT - 1], float x) {
+  float a = w[NT - 1] * x;
 #pragma unroll
-  for (int j = 0; j < CD_TAPS - 1; ++j) a = fmaf(w[j], win[j], a);
+  for (int j = 0; j < NT - 1; ++j) a = fmaf(w[j], win[j], a);
 #pragma unroll
-  for (int j = 0; j < CD_TAPS - 2; ++j) win[j] = win[j + 1];
-  win[CD_TAPS - 2] = x;
+  for (int j = 0; j < NT - 2; ++j) win[j] = win[j + 1];
+  win[NT - 2] = x;
   return Elem<T>::to(Elem<T>::from(cd_silu(a)));
 }
 

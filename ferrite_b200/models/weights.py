@@ -408,7 +408,7 @@ def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> Non
     rows = torch.cat([w[p + n] for n in names])
     out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     if l.bias:
-        out[p + "in_bias"] = torch.cat([w[p + n + "_bias"].float() for n in names])
+        out[p + "in_bias"] = _pad(torch.cat([w[p + n + "_bias"].float() for n in names]), round_up(rows.shape[0], 8))
         out[p + "out_bias"] = _pad(w[p + "out_bias"].float(), W)
     if l.sink:
         out[p + "sink"] = w[p + "sink"].float().contiguous()

@@ -11,7 +11,7 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as F
 
-LOWRANK_ROWS = 64     # up to this many rows (the largest graph-captured step) the low-rank products are one SIMT launch
+LOWRANK_ROWS = 4      # up to this many rows the low-rank products are one SIMT launch, beyond two of the row or GEMM kernels
 UNIT_EPS = 1e-6       # inside the root of the delta rule's unit queries and keys
 
 
@@ -117,7 +117,7 @@ class CudaMixers:
         return out
 
     def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
-        """Few rows: both low-rank products in one launch, then one launch per group for the whole mixer. Prompt groups: two GEMMs,
+        """A few rows: both low-rank products in one launch, then one launch per group for the whole mixer. Prompt groups: two GEMMs,
         the chunked scan, the gated norm. Sizes beyond the fused kernels (heads wider than 128) run conv, recurrence and norm apart."""
         T = proj.shape[0]
         sizes = [d.heads, d.kv_heads, d.dim, d.vdim, d.conv, d.q_off]

@@ -237,6 +237,7 @@ def kernels_dofunex(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     from ..models.weights import DeltaDims, GqaDims
     from ..ops.cuda_ops import CudaOps
     from ..ops.latent import SegGroup
+    from ..ops.mixers import LOWRANK_ROWS
     ops, acc = CudaOps(dev), _Rows(dev)
     add = acc.add
     D, kvb, K, R, H, G = DIM, 64, 4, 128, heads, kv_heads
@@ -312,8 +313,15 @@ def kernels_dofunex(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
         ups = [(rnd(H * D, R), rnd(H * D, R)) for _ in range(32)]
         wo = [rnd(2 * H * D, R) for _ in range(32)]
         xr = rnd(m, R)
-        add(f"cd_lowrank, {m} rows", (lambda j: ops.C.cd_lowrank(up, proj, *ups[j]), H * D * R * 4.0 + m * H * D * 8.0, 4.0 * m * H * D * R, 32),
-            "linear of the same bytes", (lambda j: ops.linear(xr, wo[j], out_f32=True), H * D * R * 4.0 + m * H * D * 8.0, 4.0 * m * H * D * R, 32))
+
+        def low_rank(j):
+            if m <= LOWRANK_ROWS:
+                ops.C.cd_lowrank(up, proj, *ups[j])
+            else:
+                ops.linear(proj[:, :R], ups[j][0], out_f32=True)
+                ops.linear(proj[:, R:2 * R], ups[j][1], out_f32=True)
+        work = (H * D * R * 4.0 + m * H * D * 8.0, 4.0 * m * H * D * R, 32)
+        add(f"low-rank products, {m} rows", (low_rank, *work), "linear of the same bytes", (lambda j: ops.linear(xr, wo[j], out_f32=True), *work))
         del rec, tail
     rec, tail = f32(1, H, D, D), rnd(1, K - 1, d.channels)
     proj, pg = rnd(T, d.b_off + H), rnd(T, 4 * H * D + 2 * H)

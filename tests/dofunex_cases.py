@@ -39,6 +39,8 @@ CASES = {
     "bare": config(64, 96, [delta(1, 1, 16, 24, 1, 48), delta(2, 1, 32, 8, 2, None)], eps=1e-3),
     # attention without positions between rotated layers, loop over everything
     "round": config(72, 130, [attn(3, 3, 24, 40, rot=0), attn(4, 1, 32, None, rot=8, scaling=(16.0, 2.0, 2.5, 40))], (0, 2, 3), mult=0.6, scale=0.25),
+    # odd widths throughout
+    "odd": config(70, 101, [delta(3, 3, 13, 27, 2, 51), attn(3, 1, 21, 35, rot=10), delta(5, 1, 65, 3, 4, None)], (1, 2, 2), mult=0.9),
     # heads wider than the tensor-core and fused kernels take
     "broad": config(96, 120, [attn(2, 1, 272, 64), delta(2, 2, 160, 136, 4, 64), delta(1, 1, 40, 264, 3, None)], (2, 3, 2)),
 }
@@ -66,6 +68,9 @@ def weights(cfg, seed=0, ranks=(20, 28)):
         else:
             for n, rows in (("q", G * D), ("k", G * D), ("v", H * V)):
                 w[x + n], w[x + n + ".conv"] = mat(rows, W), r(rows, m["conv"]) * m["conv"] ** -0.5
+            # queries near their keys: the first read of a head is sign(q k) v after its norm, and at right angles 16-bit operands
+            # would pick the sign
+            w[x + "q"], w[x + "q.conv"] = 0.6 * w[x + "q"] + 0.8 * w[x + "k"], 0.3 * w[x + "q.conv"] + 0.9 * w[x + "k.conv"]
             w[x + "b"], w[x + "norm"] = mat(H, W, 2.0), nrm(V)
             w[x + "A_log"], w[x + "dt_bias"] = u(-3.0, 3.5, H), u(-7.0, 2.0, H * D)
             w[x + "a1"], w[x + "a2"] = mat(ranks[0], W), mat(H * D, ranks[0], 2.0)

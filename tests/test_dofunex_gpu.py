@@ -331,8 +331,7 @@ def test_sequence_in_portions(ext, models, compute, name, cuts):
 @pytest.mark.parametrize("compute", ["fp32", "bf16"])
 def test_portions_and_batches_agree_beyond_rounding_only(ext, models, compute):
     """Requests together (prompt portions beside decoded tokens, long segments beside short ones, a tight pool, slots and pages
-    that go round) against the plain rows of each. (The first read of a head is sign(q k) v after its norm: sequences that start with
-    q and k at right angles, where 16-bit operands pick the sign, are not among these.)"""
+    that go round) against the plain rows of each."""
     for name in CASES:
         cfg, w, d, ids, want = models[name, compute]
         eng = engine(d, DEV, compute, max_ctx=448, pool=1024)
