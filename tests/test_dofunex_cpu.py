@@ -282,11 +282,11 @@ def test_every_part_shows_in_the_logits(models):
     for t in range(0, 6):
         assert error(plain.forward(cfg, w, ids[:t] + [(ids[t] + 1) % cfg["vocab"]] + ids[t + 1:])[0][-1:], base) > 20 * LIM
     for name in ("l0.mix.sink", "l2.mix.sink", "l0.mix.k.b", "l2.mix.o.b", "l1.mix.dt_bias", "l3.mix.A_log", "l1.mix.b", "loop.step", "l3.mix.g2"):
-        assert error(plain.forward(cfg, dict(w, **{name: w[name] * 0.9}), ids)[0][-1:], base) > 100 * LIM, name
+        assert error(plain.forward(cfg, dict(w, **{name: w[name] * 0.9}), ids)[0][-1:], base) > 50 * LIM, name
     for name in ("l1.mix.q.conv", "l3.mix.v.conv"):
         cut = w[name].clone()
         cut[:, 0] = 0                                                # the oldest tap
-        assert error(plain.forward(cfg, dict(w, **{name: cut}), ids)[0][-1:], base) > 100 * LIM, name
+        assert error(plain.forward(cfg, dict(w, **{name: cut}), ids)[0][-1:], base) > 50 * LIM, name
     for change in (lambda c: c["loop"].update(times=2), lambda c: c["layers"][0]["mixer"]["rot"].update(base=705.0),
                    lambda c: c["layers"][2]["mixer"]["rot"]["scaling"].update(low=1.1), lambda c: c.update(residual_mult=0.551)):
         other = copy.deepcopy(cfg)
