@@ -311,7 +311,8 @@ cd_chunk_prep_kernel(float* __restrict__ scratch, const T* __restrict__ proj, lo
 }
 
 // ---- scan --------------------------------------------------------------------------------------------------------------------
-// grid (ceil(vdim / W), heads, segments), 16 W threads. A thread's tile: rows of one row group x 4 columns. Kt and Qt of the next chunk
+// grid (ceil(vdim / W), heads, segments), 8 W threads. A thread's tile: two rows of the chunk x 4 columns (shared-memory reads per FMA
+// set the pace). Kt and Qt of the next chunk
 // are fetched while the current one is past them, Kh, T', P T', eC likewise, and so are the raw inputs of v.
 template <int DKP, int W>
 struct ScanSmem {
@@ -320,14 +321,14 @@ struct ScanSmem {
 };
 
 template <typename T, int DKP, int W, int NT>
-__global__ void __launch_bounds__(16 * W)
+__global__ void __launch_bounds__(8 * W)
 cd_chunk_scan_kernel(float* __restrict__ y, float* __restrict__ rec_state, const float* __restrict__ scratch, const T* __restrict__ proj,
                      long ldp, const float* __restrict__ conv_w, const T* __restrict__ conv_state, const int* __restrict__ seg_slot,
                      const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows, CdLayer L) {
   using M = ScanSmem<DKP, W>;
-  constexpr int NTH = 16 * W, LDK = M::LDK, LDT = M::LDT, CG = W / 4, RG = NTH / CG;         // RG = C: a row of the chunk per row group
+  constexpr int NTH = 8 * W, LDK = M::LDK, LDT = M::LDT, CG = W / 4, RG = NTH / CG, R = CC / RG;       // rows rg, rg + RG of the chunk
   constexpr int R3 = DKP / RG;                                                              // state rows per thread
-  static_assert(RG == CC && R3 >= 1, "tiles");
+  static_assert(R == 2 && R3 >= 2, "tiles");
   extern __shared__ __align__(16) float cs_smem[];
   float* KQ = cs_smem;                                      // [2 C][LDK]: K~ rows, then Q~ rows
   float* Kh = KQ + 2 * CC * LDK;                            // [C][LDK]
@@ -367,7 +368,7 @@ cd_chunk_scan_kernel(float* __restrict__ y, float* __restrict__ rec_state, const
   load_kq(rec);
   load_rest(rec);
 
-  // this thread's share of v: one column, four rows of every chunk and the NT - 1 inputs ahead of them
+  // this thread's share of v: one column, eight rows of every chunk and the NT - 1 inputs ahead of them
   constexpr int VR = CC * W / NTH;
   const int vc = tid % W, vt = tid / W * VR, vcol = min(col0 + vc, L.vdim - 1), vch = 2 * L.kv_heads * L.dim + h * L.vdim + vcol;
   const T* tail = conv_state + (size_t)slot * (L.taps - 1) * C;
@@ -400,48 +401,75 @@ cd_chunk_scan_kernel(float* __restrict__ y, float* __restrict__ rec_state, const
     }
     cc_wait<1>();                                           // K~, Q~ have landed (Kh and the rest may still be on their way)
     __syncthreads();                                        // ... for everyone, V too, and the state slice is complete
-    float u[4] = {}, o[4] = {};                             // row rg of K~ S and of Q~ S
-#pragma unroll 4
+    float u[R][4] = {}, o[R][4] = {};                       // this thread's rows of K~ S and of Q~ S
+#pragma unroll 2
     for (int k = 0; k < DKP; k += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(KQ + rg * LDK + k), b = *reinterpret_cast<const float4*>(KQ + (CC + rg) * LDK + k);
-      const float ax[4] = {a.x, a.y, a.z, a.w}, bx[4] = {b.x, b.y, b.z, b.w};
+      float4 sv[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float4 s = *reinterpret_cast<const float4*>(Ss + (k + e) * W + cg);
-        u[0] = fmaf(ax[e], s.x, u[0]); u[1] = fmaf(ax[e], s.y, u[1]); u[2] = fmaf(ax[e], s.z, u[2]); u[3] = fmaf(ax[e], s.w, u[3]);
-        o[0] = fmaf(bx[e], s.x, o[0]); o[1] = fmaf(bx[e], s.y, o[1]); o[2] = fmaf(bx[e], s.z, o[2]); o[3] = fmaf(bx[e], s.w, o[3]);
+      for (int e = 0; e < 4; ++e) sv[e] = *reinterpret_cast<const float4*>(Ss + (k + e) * W + cg);
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const float4 a = *reinterpret_cast<const float4*>(KQ + (rg + i * RG) * LDK + k);
+        const float4 b = *reinterpret_cast<const float4*>(KQ + (CC + rg + i * RG) * LDK + k);
+        const float ax[4] = {a.x, a.y, a.z, a.w}, bx[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float4 v = sv[e];
+          u[i][0] = fmaf(ax[e], v.x, u[i][0]); u[i][1] = fmaf(ax[e], v.y, u[i][1]);
+          u[i][2] = fmaf(ax[e], v.z, u[i][2]); u[i][3] = fmaf(ax[e], v.w, u[i][3]);
+          o[i][0] = fmaf(bx[e], v.x, o[i][0]); o[i][1] = fmaf(bx[e], v.y, o[i][1]);
+          o[i][2] = fmaf(bx[e], v.z, o[i][2]); o[i][3] = fmaf(bx[e], v.w, o[i][3]);
+        }
       }
     }
-    {
-      const float4 v = *reinterpret_cast<const float4*>(Vs + rg * W + cg);
-      *reinterpret_cast<float4*>(Bs + rg * W + cg) = make_float4(v.x - u[0], v.y - u[1], v.z - u[2], v.w - u[3]);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const float4 v = *reinterpret_cast<const float4*>(Vs + (rg + i * RG) * W + cg);
+      *reinterpret_cast<float4*>(Bs + (rg + i * RG) * W + cg) = make_float4(v.x - u[i][0], v.y - u[i][1], v.z - u[i][2], v.w - u[i][3]);
     }
     cc_wait<0>();                                           // Kh, T', P T', eC
     __syncthreads();                                        // ... and B; K~ and Q~ are free
     if (chn + 1 < nchunks) load_kq(rec + (size_t)(chn + 1) * rec_stride);
-    // D = T' B, O = Q~ S + P T' B (both lower triangular, zeros above)
-    float d[4] = {};
-    const int last = (rg | 7) + 1;                          // the same bound for all rows of a warp or two
-#pragma unroll 2
-    for (int k = 0; k < last; k += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(Ts + rg * LDT + k), b = *reinterpret_cast<const float4*>(Ps + rg * LDT + k);
-      const float ax[4] = {a.x, a.y, a.z, a.w}, bx[4] = {b.x, b.y, b.z, b.w};
+    // D = T' B, O = Q~ S + P T' B (both lower triangular, zeros above); past its own diagonal the first row is done
+    float d[R][4] = {};
+    auto triangle = [&](int k, auto first) {
+      constexpr int I0 = decltype(first)::value;
+      float4 sv[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float4 s = *reinterpret_cast<const float4*>(Bs + (k + e) * W + cg);
-        d[0] = fmaf(ax[e], s.x, d[0]); d[1] = fmaf(ax[e], s.y, d[1]); d[2] = fmaf(ax[e], s.z, d[2]); d[3] = fmaf(ax[e], s.w, d[3]);
-        o[0] = fmaf(bx[e], s.x, o[0]); o[1] = fmaf(bx[e], s.y, o[1]); o[2] = fmaf(bx[e], s.z, o[2]); o[3] = fmaf(bx[e], s.w, o[3]);
+      for (int e = 0; e < 4; ++e) sv[e] = *reinterpret_cast<const float4*>(Bs + (k + e) * W + cg);
+#pragma unroll
+      for (int i = I0; i < R; ++i) {
+        const float4 a = *reinterpret_cast<const float4*>(Ts + (rg + i * RG) * LDT + k);
+        const float4 b = *reinterpret_cast<const float4*>(Ps + (rg + i * RG) * LDT + k);
+        const float ax[4] = {a.x, a.y, a.z, a.w}, bx[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float4 v = sv[e];
+          d[i][0] = fmaf(ax[e], v.x, d[i][0]); d[i][1] = fmaf(ax[e], v.y, d[i][1]);
+          d[i][2] = fmaf(ax[e], v.z, d[i][2]); d[i][3] = fmaf(ax[e], v.w, d[i][3]);
+          o[i][0] = fmaf(bx[e], v.x, o[i][0]); o[i][1] = fmaf(bx[e], v.y, o[i][1]);
+          o[i][2] = fmaf(bx[e], v.z, o[i][2]); o[i][3] = fmaf(bx[e], v.w, o[i][3]);
+        }
       }
-    }
-    *reinterpret_cast<float4*>(Ds + rg * W + cg) = make_float4(d[0], d[1], d[2], d[3]);
-    if (rg < valid) {
-      float* dst = y + ((size_t)(seg0 + r0 + rg) * L.heads + h) * L.vdim + col0 + cg;
-      if (L.vdim % 4 == 0 && col0 + cg < L.vdim) {
-        *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
-      } else {
+    };
+#pragma unroll 2
+    for (int k = 0; k < RG; k += 4) triangle(k, std::integral_constant<int, 0>());
+    const int last = RG + (rg | 7) + 1;                     // the same bound for all rows of a warp
+#pragma unroll 2
+    for (int k = RG; k < last; k += 4) triangle(k, std::integral_constant<int, 1>());
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (col0 + cg + e < L.vdim) dst[e] = o[e];
+    for (int i = 0; i < R; ++i) {
+      const int t = rg + i * RG;
+      *reinterpret_cast<float4*>(Ds + t * W + cg) = make_float4(d[i][0], d[i][1], d[i][2], d[i][3]);
+      if (t < valid) {
+        float* dst = y + ((size_t)(seg0 + r0 + t) * L.heads + h) * L.vdim + col0 + cg;
+        if (L.vdim % 4 == 0 && col0 + cg < L.vdim) {
+          *reinterpret_cast<float4*>(dst) = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (col0 + cg + e < L.vdim) dst[e] = o[i][e];
+        }
       }
     }
     __syncthreads();
@@ -459,12 +487,10 @@ cd_chunk_scan_kernel(float* __restrict__ y, float* __restrict__ rec_state, const
       for (int t = 0; t < CC; ++t) {
         const float4 dd = *reinterpret_cast<const float4*>(Ds + t * W + cg);
         float kx[R3];
-        if constexpr (R3 == 2) {
-          const float2 a = *reinterpret_cast<const float2*>(Kh + t * LDK + rg * R3);
-          kx[0] = a.x; kx[1] = a.y;
-        } else {
 #pragma unroll
-          for (int i = 0; i < R3; ++i) kx[i] = Kh[t * LDK + rg * R3 + i];
+        for (int i = 0; i < R3; i += 2) {
+          const float2 a = *reinterpret_cast<const float2*>(Kh + t * LDK + rg * R3 + i);
+          kx[i] = a.x; kx[i + 1] = a.y;
         }
 #pragma unroll
         for (int i = 0; i < R3; ++i) {
@@ -498,7 +524,7 @@ static int cd_chunk(float* y, float* rec, float* scratch, const void* tail, cons
     e = launch_pdl(prep, dim3((max_rows + CC - 1) / CC, L.heads, nseg), dim3(CP_THREADS), psm, s, scratch, (const T*)proj, ldp, decay, ldd,
                    conv_w, A_log, dt_bias, (const T*)tail, seg_slot, seg_row0, seg_nrows, L);
   if (e == cudaSuccess)
-    e = launch_pdl(scan, dim3((L.vdim + W - 1) / W, L.heads, nseg), dim3(16 * W), ssm, s, y, rec, (const float*)scratch, (const T*)proj,
+    e = launch_pdl(scan, dim3((L.vdim + W - 1) / W, L.heads, nseg), dim3(8 * W), ssm, s, y, rec, (const float*)scratch, (const T*)proj,
                    ldp, conv_w, (const T*)tail, seg_slot, seg_row0, seg_nrows, L);
   return (int)e;
 }
