@@ -32,11 +32,23 @@ class LayerSpec:
     kv_from: Optional[int] = None   # use the latents that this (earlier) layer caches instead of own ones
     ff: int = 0                     # feed-forward width, 0 = the layer has none
     act: str = "relu2"              # its activation; "swiglu": silu(gate) * up
+    experts: int = 0                # the feed-forward is a mixture of this many swiglu experts of width `ff` ...
+    top: int = 0                    # ... of which a token takes the `top` best (sigmoid scores) ...
+    groups: int = 1                 # ... among the best `keep_groups` of `groups` groups of neighbours ...
+    keep_groups: int = 1
+    route_scale: float = 1.0        # ... weighted by their share of the chosen scores times this
     kv_heads: int = 0               # gqa, cdelta: key / value (cdelta: query / key) heads, each serving heads / kv_heads heads
     bias: bool = False              # gqa: biases on the query, key and output projections
     sink: bool = False              # gqa: a learned number per head in every softmax denominator
     key_values: bool = False        # gqa: the values are the projected keys, before rotation and norm
     qk_norm: bool = False           # gqa: queries and keys divided by their root mean square after the rotation
+    row_norm: bool = False          # gqa: RMS norms with weights over a whole row of queries and of keys, before the rotation
+    softcap: float = 0.0            # gqa: scores <- cap * tanh(scores / cap), 0 = off
+    window: int = 0                 # gqa: a row sees itself and the window - 1 positions before it, 0 = all of them
+    chunk: int = 0                  # gqa: a row sees the positions of its own chunk of this many, counted from 0
+    maps: int = 1                   # gqa: 2 = differential: two softmax maps per head over shared values, their weighted difference
+    diff: float = 0.0               # gqa, two maps: constant of the difference's weight; 1 - diff scales its normed rows
+    out_gate: bool = False          # gqa: the heads' outputs are multiplied by the sigmoid of a projection of the mixer's input
     rot_dims: int = 0               # gqa: rotated columns of a head, pairs (0, 1), (2, 3), ...
     rot_base: float = 1e4
     rot_scaling: Optional[dict] = None   # long wavelengths stretched: factor, low, high, original
@@ -105,8 +117,10 @@ class ModelConfig:
     layers: List[LayerSpec] = field(default_factory=list)
     out_norm: bool = False          # x + norm(f(x)): norms on the sublayers' outputs, a 32-bit residual stream, plain norm weights
     pre_norm: bool = False          # ... and norms on the sublayers' inputs as well: x + norm(f(norm(x)))
+    parallel: bool = False          # x + (mixer(norm(x)) + f(norm(x))): one layer norm (with bias) ahead of both sublayers, none behind
     residual_mult: float = 1.0      # x + residual_mult * norm(f(..))
     loop: Optional[List[int]] = None     # [start, stop, times]: layers start .. stop - 1 run `times` times in a row
+    loop_input: bool = True         # a pass of the loop opens with a product of [x | embedding] and a bias per pass
     logit_scale: float = 1.0
     embed_scale: float = 1.0
     gram_buckets: int = 0           # hashed bigram embedding: rows of the table besides the one for a sequence's first token
@@ -179,13 +193,16 @@ class ModelConfig:
         n = self.vocab * h * (1 if self.tie_embeddings else 2)
         if self.layers:
             n += (self.gram_buckets + 1) * h if self.gram_buckets else 0
-            n += 2 * h * h if self.loop else 0
+            n += 2 * h * h if self.loop and self.loop_input else 0
             for l in self.layers:
                 if l.mixer == "gqa":
-                    n += h * (2 * l.heads + l.kv_heads * (1 if l.key_values else 2)) * l.dim
+                    n += h * (l.maps * l.dim * (l.heads + l.kv_heads) + l.vdim * ((2 if l.out_gate else 1) * l.heads + (0 if l.key_values else l.kv_heads)))
                 elif l.mixer == "cdelta":
                     n += h * (2 * l.kv_heads * l.dim + 2 * l.heads * l.vdim + l.heads) + (2 * l.kv_heads * l.dim + l.heads * l.vdim) * l.conv
                     n += l.decay_rank * (h + l.heads * l.dim) + l.gate_rank * (h + l.heads * l.vdim)
+                if l.experts:
+                    n += l.experts * (h + 3 * h * l.ff)
+                    continue
                 if l.mixer != "latent":
                     n += (3 if l.act == "swiglu" else 2) * h * l.ff
                     continue
@@ -215,6 +232,8 @@ class ModelConfig:
         if world == 1:
             return c
         if self.layers:
+            if self.parallel:
+                raise ValueError("models of parallel blocks run on one rank: their query and key norms span all heads")
             assert all(l.heads % world == 0 and l.kv_heads % world == 0 and l.ff % world == 0 for l in self.layers), \
                 f"heads and feed-forward widths must divide over {world} ranks"
             c.layers = [dataclasses.replace(l, heads=l.heads // world, kv_heads=l.kv_heads // world, ff=l.ff // world) for l in self.layers]
@@ -330,7 +349,54 @@ def dofunex_config(v: dict) -> ModelConfig:
         loop=[int(lp[k]) for k in ("start", "stop", "times")] if lp else None, logit_scale=float(v.get("logit_scale", 1.0)))
 
 
-ARCHITECTURES = {"Zototar": zototar_config, "Dofunex": dofunex_config}
+def rakizen_config(v: dict) -> ModelConfig:
+    """A Rakizen config.json: parallel blocks under one layer norm; "attention" takes the difference of two softmax maps over chunks of
+    the sequence, with gated outputs and no positions, "attention_2" normed and rotated queries and keys under a sliding window, both
+    with softcapped scores; dense or routed swiglu feed-forwards; layers may loop, with a cache per pass."""
+    layers: List[LayerSpec] = []
+    for i, e in enumerate(v["layers"]):
+        kind, m, ff = e["type"], e["mixer"], e.get("mlp")
+        if kind not in ("attention", "attention_2"):
+            raise ValueError(f"layer {i}: mixer type {kind!r} is neither attention nor attention_2")
+        size = int(m["mask"]["size"])
+        if size < 1 or float(m["softcap"]) <= 0:
+            raise ValueError(f"layer {i}: mask size {size} and softcap {m['softcap']} must be positive")
+        kw = dict(mixer="gqa", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                  scale=float(m["scale"]), softcap=float(m["softcap"]), act="swiglu")
+        if kw["heads"] % kw["kv_heads"]:
+            raise ValueError(f"layer {i}: {kw['heads']} heads do not divide over {kw['kv_heads']} key heads")
+        if kind == "attention":
+            kw.update(chunk=size, maps=2, diff=float(m["diff"]), out_gate=True)
+        else:
+            rot = m.get("rot") or {}
+            kw.update(window=size, row_norm=True, rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 1e4)))
+            if kw["rot_dims"] % 2 or kw["rot_dims"] > kw["dim"]:
+                raise ValueError(f"layer {i}: {kw['rot_dims']} rotated dimensions of {kw['dim']}")
+        if ff and ff["kind"] == "dense":
+            kw["ff"] = int(ff["ff"])
+        elif ff and ff["kind"] == "moe":
+            r = ff["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            kw.update(ff=int(ff["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=int(g["count"]),
+                      keep_groups=int(g["keep"]), route_scale=float(r["scale"]))
+            if kw["experts"] % kw["groups"] or not 1 <= kw["keep_groups"] <= kw["groups"]:
+                raise ValueError(f"layer {i}: {kw['experts']} experts in {kw['groups']} groups, of which {kw['keep_groups']} are kept")
+            if not 1 <= kw["top"] <= kw["experts"] // kw["groups"] * kw["keep_groups"]:
+                raise ValueError(f"layer {i}: {kw['top']} experts per token cannot come out of {kw['keep_groups']} groups")
+        elif ff:
+            raise ValueError(f"layer {i}: feed-forward kind {ff['kind']!r} is neither dense nor moe")
+        layers.append(LayerSpec(**kw))
+    lp = v.get("loop")
+    if lp and not (0 <= lp["start"] <= lp["stop"] <= len(layers) and lp["times"] >= 1):
+        raise ValueError(f"loop {lp['start']} .. {lp['stop']}, {lp['times']} times, over {len(layers)} layers")
+    return ModelConfig(
+        name="rakizen", hidden=int(v["width"]), inter=max([l.ff for l in layers] + [0]), n_layers=len(layers), n_q=layers[0].heads,
+        n_kv=layers[0].kv_heads, head_dim=layers[0].dim, eps=float(v["norm"]["eps"]), vocab=int(v["vocab"]), attn_gate=False,
+        tie_embeddings=False, layers=layers, pre_norm=True, parallel=True,
+        loop=[int(lp[k]) for k in ("start", "stop", "times")] if lp else None, loop_input=False)
+
+
+ARCHITECTURES = {"Zototar": zototar_config, "Dofunex": dofunex_config, "Rakizen": rakizen_config}
 
 
 # ---- presets: the five benchmark configurations ----------------------------------------------------
@@ -438,7 +504,38 @@ def dofunex_7b() -> ModelConfig:
     return dofunex(4096, 32, 32, 8, 11008, 129280, name="dofunex-7b")
 
 
+def rakizen(width: int, n_layers: int, heads: int, kv_heads: int, ff: int, vocab: int, dim: int = 128, window: int = 1024,
+            chunk: int = 2048, experts: int = 0, top: int = 0, groups: int = 1, keep: int = 1, expert_ff: int = 0, every: int = 4,
+            loop: Optional[List[int]] = None, name: str = "rakizen") -> ModelConfig:
+    """A Rakizen model in which every `every`-th layer takes the difference of two maps (half the heads, twice the value width), the
+    others a window; with `experts`, every second layer has a routed feed-forward."""
+    common = dict(mixer="gqa", act="swiglu", softcap=50.0)
+    win = LayerSpec(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, window=window, row_norm=True, rot_dims=dim,
+                    rot_base=1e6, ff=ff, **common)
+    two = LayerSpec(heads=heads // 2, kv_heads=max(1, kv_heads // 2), dim=dim // 2, vdim=dim, scale=(dim // 2) ** -0.5, chunk=chunk, maps=2,
+                    diff=0.6, out_gate=True, ff=ff, **common)
+    moe = dict(ff=expert_ff, experts=experts, top=top, groups=groups, keep_groups=keep, route_scale=1.5) if experts else {}
+    layers = [dataclasses.replace(two if i % every == every - 1 else win, **(moe if i % 2 else {})) for i in range(n_layers)]
+    return ModelConfig(name=name, hidden=width, inter=ff, n_layers=n_layers, n_q=heads, n_kv=kv_heads, head_dim=dim, eps=1e-6, vocab=vocab,
+                       attn_gate=False, tie_embeddings=False, layers=layers, pre_norm=True, parallel=True, loop=loop, loop_input=False)
+
+
+def tiny_rakizen() -> ModelConfig:
+    """4-layer plumbing model of the parallel-block family: unequal layers, sizes off the kernels' tile grid, two layers looped."""
+    c = rakizen(136, 4, 4, 2, 104, 300, dim=40, window=24, chunk=56, experts=6, top=2, groups=3, keep=2, expert_ff=44, every=2, loop=[1, 3, 2],
+                name="tiny-rakizen")
+    c.layers[0] = dataclasses.replace(c.layers[0], dim=24, vdim=56, kv_heads=1, rot_dims=10, rot_base=500.0)
+    c.layers[2] = dataclasses.replace(c.layers[2], heads=6, kv_heads=3, ff=0)
+    return c
+
+
+def rakizen_7b() -> ModelConfig:
+    """7B-class parallel-block model: 32 layers of width 4096, 32 heads of 128, dense feed-forwards of 12288."""
+    return rakizen(4096, 32, 32, 8, 12288, 129280, name="rakizen-7b")
+
+
 PRESETS = {
+    "tiny-rakizen": tiny_rakizen, "rakizen-7b": rakizen_7b,
     "tiny-dofunex": tiny_dofunex, "dofunex-7b": dofunex_7b,
     "tiny-zototar": tiny_zototar, "zototar-7b": zototar_7b,
     "tiny": tiny_hybrid, "tiny-mla": tiny_mla, "27b": hybrid_27b, "drafter": drafter_block, "moe80b": moe_80b, "mla671b": mla_671b,

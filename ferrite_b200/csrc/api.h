@@ -5,6 +5,13 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+// What a row sees of the keys up to its own, and the softcap of its scores (0 = none). window: the row and the window - 1 positions
+// before it; chunk: the positions of its own chunk, counted from 0 (0 = all, at most one of the two).
+typedef struct KeyBounds {
+  int window, chunk;
+  float cap;
+} KeyBounds;
+
 #ifdef __cplusplus
 extern "C" {
 #endif
@@ -14,7 +21,7 @@ int fb_embed(void* out, const void* table, const int* ids, int rows, int hidden,
 int fb_rmsnorm(void* out, void* x_out, const void* x, const void* res, const void* w, int rows, int hidden, float eps,
                int centred, cudaStream_t s);
 int fb_silu_mul(void* out, const void* gu, int rows, int inter, float clamp, cudaStream_t s);
-int fb_silu_mul_f32(float* out, const float* gu, int rows, int inter, cudaStream_t s);
+int fb_silu_mul_f32(float* out, long ldo, const float* gu, int rows, int inter, cudaStream_t s);
 int fb_gated_norm_sigmoid(void* out, int ldo, const float* y, const float* z, long z_stride, const float* w, int rows, int heads, int dv,
                           float eps, int f32, cudaStream_t s);
 int fb_gated_norm(void* out, const float* y, const void* z, long z_stride, const void* w, int rows, int heads, int dv,
@@ -90,7 +97,7 @@ int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, const void* q, 
                        const float* kv_scale, const void* proj, long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                        const int* row_kvlen, const int* row_base, const unsigned long long* row_mask,
                        const int* block_table, int max_blocks, int kv_block, int nseg, int max_rows, int rows, int nq,
-                       int nkv, int hd, int nsplit, int gated, float scale, int exact_p, int row_first, cudaStream_t s);
+                       int nkv, int hd, int nsplit, int gated, float scale, int exact_p, const KeyBounds* kb, int row_first, cudaStream_t s);
 // 4-bit KV cache: codes [..][hd/2] bytes, scales [..][2 * hd/32] fp32 per (token, kv head) row (K groups, V groups)
 int fb_attn_prep_q4(void* q_out, void* k_cache4, void* v_cache4, float* kv_scale, const void* proj, long proj_stride,
                     const void* q_norm, const void* k_norm, const float* inv_freq, const int* row_slot, const int* row_pos,
@@ -121,7 +128,7 @@ int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void
                        long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                        const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg, int max_rows,
                        long q_rows, long cache_rows, int nq, int nkv, int hd, int gated, float scale, int exact_p,
-                       long kv_stride, const float* sink, int* status, cudaStream_t s);
+                       long kv_stride, const float* sink, const KeyBounds* kb, long ldo, int out_f32, int* status, cudaStream_t s);
 
 // ---- gdn.cu ----
 int fb_gdn_conv(void* out, const void* proj, long proj_stride, const void* conv_w, const void* conv_state,

@@ -3,6 +3,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "api.h"
+
 #ifdef __cplusplus
 extern "C" {
 #endif
@@ -100,6 +102,8 @@ int fb_moe_gate_up_fp4(void* act, const void* x, const void* wq, const void* ws,
 int fb_moe_down_fp4(float* yp, const void* act, const void* wq, const void* ws, float gscale, const int* ids, int pairs,
                     int hidden, int inter, int e_lo, int e_hi, cudaStream_t s);
 int fb_nvfp4_dequant(void* out, const void* wq, const void* ws, float gscale, long elements, cudaStream_t s);
+int fb_expert_rows_f32(float* yp, float* act, const float* x, const float* w_gu, const float* w_down, const int* ids, int pairs, int top_k,
+                       int hidden, int inter, int n_exp, cudaStream_t s);
 int fb_moe_combine(void* out, const float* yp, const float* wts, const void* shared, const float* shared_gate,
                    const void* res, int rows, int top_k, int hidden, int out_f32, cudaStream_t s);
 
@@ -127,7 +131,7 @@ int fb_head_linear(void* y, const void* x, const void* W, int T, int heads, int 
 long fb_ep_workspace_bytes(int n_experts, int hidden, long cap_rows);
 long fb_ep_recv_offset(int n_experts, int hidden, long cap_rows);
 long fb_ep_out_offset(int n_experts, int hidden, long cap_rows);
-int fb_ep_moe(void* out, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
+int fb_ep_moe(void* out, int out_f32, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
               const void* shared, const float* shared_gate, const void* res, void* act, int* plan, int rows, int top_k,
               int n_experts, int hidden, int inter, long cap_rows, const void* const* peers, int rank, int world,
               uint32_t* ctr, int* status, unsigned spin_limit, int sm_count, cudaStream_t s);
@@ -164,8 +168,10 @@ int fb_embed_grams(float* x, void* xb, int copies, const void* table, const void
                    long buckets, long mul_prev, long mul_cur, int f32, int* status, cudaStream_t s);
 int fb_add_normed(float* x, void* xb, int xb_f32, long ldb, const void* y, int y_f32, const float* bias, const float* w,
                   const float* next_w, int rows, int width, int ld, long ldy, float eps, cudaStream_t s);
-int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps, int f32,
+int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int rows, int width, int ld, float eps, int f32,
                  cudaStream_t s);
+int fb_add_layer_norm(float* x, void* xb, int f32, const void* y, int y_f32, long ldy, const float* yp, const float* wts, int top,
+                      const float* next_w, const float* next_b, int rows, int width, int ld, float eps, cudaStream_t s);
 int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
                    const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block, int rows, int q_rank,
                    int qr, int kv_rank, int lat, float eps, int f32, int* status, cudaStream_t s);
@@ -180,14 +186,22 @@ int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const
                   cudaStream_t s);
 int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache, const float* sink,
                 const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
-                int kv_heads, int hd, int nsplit, float scale, int f32, int* status, cudaStream_t s);
-int fb_attn_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int hd,
+                int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb, long ldo, int f32, int* status, cudaStream_t s);
+int fb_attn_merge(void* out, long ldo, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int hd,
                   cudaStream_t s);
+int fb_attn_merge_mix(void* out, long ldo, const float* o_part, const float* ml_part, const float* lam, const float* gate, long ldg,
+                      float mix_scale, int maps, int rows, int heads, int nsplit, int vdim, int hd, float eps, int f32, cudaStream_t s);
+int fb_head_mix(void* out, long ldo, const float* in, const float* lam, const float* gate, long ldg, float mix_scale, int maps, int rows,
+                int heads, int vdim, int hd, float eps, int f32, cudaStream_t s);
 
 // ---- gqa.cu ----
 int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* bias, const double* inv_freq,
                 const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
                 int kv_heads, int dim, int hp, int rot, int v_off, int norm, float eps, int f32, int* status, cudaStream_t s);
+int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* q_norm, const float* k_norm,
+                    const double* inv_freq, const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block,
+                    int rows, int heads, int kv_heads, int maps, int dim, int vdim, int hp, int rot, int v_off, float eps, int f32, int* status,
+                    cudaStream_t s);
 
 // ---- cdelta.cu, cdelta_chunk.cu ----
 int fb_cd_lowrank(float* out, const void* proj, long ldp, const void* wa, int na, int ra, const void* wg, int ng, int rg, int rows,

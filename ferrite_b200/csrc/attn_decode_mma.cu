@@ -65,7 +65,9 @@ __device__ __forceinline__ void dm_e4m3x16_to_bf16(const uint4& c, uint4& lo, ui
 // a two-stage cp.async ring and are expanded to bf16 tiles in shared memory before the MMAs; the per-key scales are
 // applied to the scores (K) and to P (V) instead of to every element.
 // PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (16 bits of mantissa instead of 8).
-template <int HD, bool KV8, bool PX>
+// BND: rows see a window or a chunk of the keys up to their own, scores are softcapped (cap_log2 = cap * log2 e; scale_log2 then leads to
+// the argument of tanh_of_2log2); the splits share the keys that some row of the CTA sees.
+template <int HD, bool KV8, bool PX, bool BND>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, const __nv_bfloat16* __restrict__ q,
                        const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
@@ -73,7 +75,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
                        const int* __restrict__ seg_nrows, const int* __restrict__ row_kvlen,
                        const int* __restrict__ row_base, const unsigned long long* __restrict__ row_mask,
                        const int* __restrict__ block_table, int max_blocks, int kv_block, int nq, int nkv, int nsplit,
-                       int groups_per_seg, int row_first, float scale_log2) {
+                       int groups_per_seg, int row_first, float scale_log2, int window, int chunk, float cap_log2) {
   constexpr int LD = HD + 8;                    // padded row (elements): conflict-free ldmatrix
   constexpr int CPR = HD / 8;                   // 16-byte chunks per row
   extern __shared__ __align__(16) unsigned char dm_smem[];
@@ -100,13 +102,15 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
   const int* bt = block_table + (size_t)slot * max_blocks;
   int kv_end = 0;
   for (int r = 0; r < rows_here; ++r) kv_end = max(kv_end, row_kvlen[row0 + r]);
-  int per = (kv_end + nsplit - 1) / nsplit;
+  // rows of a segment follow one another, so the first row sees the earliest key
+  const int kv_lo = BND ? first_key(row_kvlen[row0] - 1, window, chunk) / DM_BKV * DM_BKV : 0;
+  int per = (kv_end - kv_lo + nsplit - 1) / nsplit;
   per = (per + DM_BKV - 1) / DM_BKV * DM_BKV;
-  const int lo = split * per, hi = min(kv_end, lo + per);
+  const int lo = kv_lo + split * per, hi = min(kv_end, lo + per);
 
   // this thread's two M rows
   const int m_lo = warp * 16 + lane / 4, m_hi = m_lo + 8;
-  int kvl[2] = {0, 0}, base[2] = {0, 0};
+  int kvl[2] = {0, 0}, base[2] = {0, 0}, klo[2] = {0, 0};
   unsigned long long msk[2] = {0ull, 0ull};
   size_t pidx[2] = {0, 0};
 #pragma unroll
@@ -115,6 +119,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
     if (m < valid_m) {
       const int grow = row0 + m / G, qh = kvh * G + m % G;
       kvl[h] = row_kvlen[grow];
+      if (BND) klo[h] = first_key(kvl[h] - 1, window, chunk);
       base[h] = row_base ? row_base[grow] : kvl[h];
       msk[h] = row_mask ? row_mask[grow] : 0ull;
       pidx[h] = ((size_t)grow * nq + qh) * nsplit + split;
@@ -220,11 +225,13 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = kbase + nt * 8 + (e & 1), h = e >> 1;
-          bool vis = t < kvl[h] && t < hi;
+          bool vis = t < kvl[h] && t < hi && (!BND || t >= klo[h]);
           if (vis && t >= base[h]) vis = ((msk[h] >> (t - base[h])) & 1ull) != 0ull;
           float sv = s[nt][e];
           if (KV8) sv *= tsc[((lane & 3) * 2 + nt * 8 + (e & 1)) * 2];
-          const float v = vis ? sv * scale_log2 : -INFINITY;
+          sv *= scale_log2;
+          if (BND && cap_log2 > 0.f) sv = cap_log2 * tanh_of_2log2(sv);
+          const float v = vis ? sv : -INFINITY;
           s[nt][e] = v;
           mx[h] = fmaxf(mx[h], v);
         }
@@ -304,14 +311,14 @@ using namespace fb;
 
 // Same outputs as fb_attn_decode (bf16 cache) / fb_attn_decode_kv8 (kv_scale != null: e4m3 cache); rows are addressed
 // through their segments (rows of one segment share a slot). scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as
-// value + remainder (bf16 cache); row_first: row of the step that q / out / row_kvlen start at; out null: the split records stay for
+// value + remainder (bf16 cache); kb: window, chunk and softcap (with exact_p), or null; row_first: row of the step that q / out / row_kvlen start at; out null: the split records stay for
 // the caller to merge. Returns -20 for shapes this kernel does not take (the caller uses the SIMT kernel).
 extern "C" int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache,
                                   const void* v_cache, const float* kv_scale, const void* proj, long proj_stride,
                                   const int* seg_slot, const int* seg_row0, const int* seg_nrows, const int* row_kvlen,
                                   const int* row_base, const unsigned long long* row_mask, const int* block_table,
                                   int max_blocks, int kv_block, int nseg, int max_rows, int rows, int nq, int nkv, int hd,
-                                  int nsplit, int gated, float scale, int exact_p, int row_first, cudaStream_t s) {
+                                  int nsplit, int gated, float scale, int exact_p, const KeyBounds* kb, int row_first, cudaStream_t s) {
   if (nseg <= 0 || rows <= 0) return 0;
   if (nq % nkv) return -1;
   const int G = nq / nkv;
@@ -319,24 +326,31 @@ extern "C" int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, cons
   const int RG = DM_BM / G;
   const int gps = (max_rows + RG - 1) / RG;
   dim3 grid(nseg * gps, nkv, nsplit);
-  const float scale_log2 = 1.4426950408889634f * (scale != 0.f ? scale : 1.f / sqrtf((float)hd));
-#define FB_DM(HDV, K8, PXV)                                                                                              \
+  if (kb && (kv_scale || !exact_p)) return -20;
+  if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
+  constexpr float LOG2E = 1.4426950408889634f;
+  const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
+  const float scale_log2 = LOG2E * raw_scale * (cap > 0.f ? 2.f / cap : 1.f);
+#define FB_DM(HDV, K8, PXV, BNDV)                                                                                              \
   {                                                                                                                 \
     const size_t smem = K8 ? (size_t)(DM_BM + 2 * DM_BKV) * (HDV + 8) * 2 + (size_t)4 * DM_BKV * HDV + 4 * DM_BKV * 4 * 2 \
                            : (size_t)(DM_BM + 4 * DM_BKV) * (HDV + 8) * 2;                                          \
-    auto kern = attn_decode_mma_kernel<HDV, K8, PXV>;                                                               \
+    auto kern = attn_decode_mma_kernel<HDV, K8, PXV, BNDV>;                                                               \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
     if (e != cudaSuccess) return (int)e;                                                                            \
     launch_pdl(kern, grid, dim3(DM_WARPS * 32), smem, s, o_part, ml_part, (const __nv_bfloat16*)q,                   \
                (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, kv_scale, seg_slot, seg_row0, seg_nrows, \
-               row_kvlen, row_base, row_mask, block_table, max_blocks, kv_block, nq, nkv, nsplit, gps, row_first, scale_log2);  \
+               row_kvlen, row_base, row_mask, block_table, max_blocks, kv_block, nq, nkv, nsplit, gps, row_first, scale_log2, \
+               kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E);                                               \
   }
   if (kv_scale) {
-    if (hd == 256) FB_DM(256, true, false) else if (hd == 128) FB_DM(128, true, false) else FB_DM(64, true, false)
+    if (hd == 256) FB_DM(256, true, false, false) else if (hd == 128) FB_DM(128, true, false, false) else FB_DM(64, true, false, false)
+  } else if (kb) {
+    if (hd == 256) FB_DM(256, false, true, true) else if (hd == 128) FB_DM(128, false, true, true) else FB_DM(64, false, true, true)
   } else if (exact_p) {
-    if (hd == 256) FB_DM(256, false, true) else if (hd == 128) FB_DM(128, false, true) else FB_DM(64, false, true)
+    if (hd == 256) FB_DM(256, false, true, false) else if (hd == 128) FB_DM(128, false, true, false) else FB_DM(64, false, true, false)
   } else {
-    if (hd == 256) FB_DM(256, false, false) else if (hd == 128) FB_DM(128, false, false) else FB_DM(64, false, false)
+    if (hd == 256) FB_DM(256, false, false, false) else if (hd == 128) FB_DM(128, false, false, false) else FB_DM(64, false, false, false)
   }
 #undef FB_DM
   int rc = (int)cudaGetLastError();

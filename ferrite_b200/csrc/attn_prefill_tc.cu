@@ -76,15 +76,17 @@ __device__ __forceinline__ float fast_exp2(float x) {
 
 // PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (two TS products per k step, a second
 // P buffer in TMEM), which keeps 16 bits of their mantissa instead of 8.
-template <int HD, bool PX>
+// BND: rows see a window or a chunk of the keys, scores are softcapped (cap_log2 = cap * log2 e, scale_log2 then leads to the argument of
+// tanh_of_2log2). Key tiles that no row of the CTA sees are skipped; out_f32: rows of floats.
+template <int HD, bool PX, bool BND>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
                        const __nv_bfloat16* __restrict__ proj, long proj_stride, const int* __restrict__ seg_slot,
                        const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows,
                        const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
-                       int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink,
-                       int* status) {
+                       int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink, int window, int chunk,
+                       float cap_log2, long ldo, int out_f32, int* status) {
   constexpr int NCH = HD / 64;                     // 64-element (128-byte) chunks of the head dim
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
@@ -129,7 +131,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int row0 = seg_row0[seg], pos0 = seg_pos0[seg], slot = seg_slot[seg];
   const int kvh = qh / (nq / nkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int nt = (pos0 + min(q0 + FT_BQ, n) + FT_BKV - 1) / FT_BKV;   // key tiles the last query row of the tile sees
+  const int tile0 = BND ? first_key(pos0 + q0, window, chunk) / FT_BKV : 0;   // first key tile that a row of the CTA sees
+  const int nt = (pos0 + min(q0 + FT_BQ, n) + FT_BKV - 1) / FT_BKV - tile0;   // key tiles up to the one the last query row ends in
   volatile int* abort_flag = abort_p;
 
   if (threadIdx.x == 0) {
@@ -163,7 +166,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       int k_armed = 0, v_armed = 0;                           // tiles whose K / V loads were issued
       bool ok = true;
       auto tile_row = [&](int j) -> int {
-        const int t0 = j * FT_BKV;
+        const int t0 = (tile0 + j) * FT_BKV;
         const int blk = bt[t0 / kv_block];
         return blk < 0 ? -1 : blk * kv_block + t0 % kv_block;
       };
@@ -255,6 +258,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int row = quad * 32 + lane;
     const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
     const int qpos = pos0 + q0 + row;
+    const int klo = BND ? first_key(qpos, window, chunk) : 0;
+    const int klo_last = BND ? first_key(pos0 + q0 + FT_BQ - 1, window, chunk) : 0;
     constexpr int HC = FT_BKV / 2;                          // keys per thread and tile
     constexpr int OC = HD / 2;                              // O columns per thread (rescale, epilogue)
     float m_ref = -INFINITY, l = 0.f;
@@ -272,12 +277,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_wait();
         tc_fence_before();
         mbar_arrive(&s_empty[s]);
-        const int t0 = j * FT_BKV + half * HC;
-        const bool need_mask = t0 + HC - 1 > pos0 + q0;
+        const int t0 = (tile0 + j) * FT_BKV + half * HC;
+        const bool need_mask = t0 + HC - 1 > pos0 + q0 || (BND && t0 < klo_last);
 #pragma unroll
         for (int c = 0; c < HC; ++c) {
           float v = __uint_as_float(sr[c]) * scale_log2;
-          if (need_mask && t0 + c > qpos) v = -INFINITY;
+          if (BND && cap_log2 > 0.f) v = cap_log2 * tanh_of_2log2(v);
+          if (need_mask && (t0 + c > qpos || (BND && t0 + c < klo))) v = -INFINITY;
           sr[c] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -351,14 +357,21 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const float inv = lt > 0.f ? 1.f / lt : 0.f;
       const bool valid = q0 + row < n;
       const size_t grow = (size_t)(row0 + q0 + row);
-      __nv_bfloat16* dst = out + grow * (size_t)nq * HD + (size_t)qh * HD + half * OC;
+      __nv_bfloat16* dst = out + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
+      float* dst32 = reinterpret_cast<float*>(out) + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
       const __nv_bfloat16* gate = proj + grow * proj_stride + (size_t)qh * 2 * HD + HD + half * OC;
 #pragma unroll 1
       for (int c0 = 0; c0 < OC; c0 += 32) {
         uint32_t o[32];
         tmem_ld32(tmem + lane_addr + COL_O + half * OC + c0, o);
         tmem_ld_wait();
-        if (valid) {
+        if (BND && valid && out_f32) {
+#pragma unroll
+          for (int v4 = 0; v4 < 8; ++v4)
+            *reinterpret_cast<float4*>(dst32 + c0 + v4 * 4) =
+                make_float4(__uint_as_float(o[v4 * 4]) * inv, __uint_as_float(o[v4 * 4 + 1]) * inv, __uint_as_float(o[v4 * 4 + 2]) * inv,
+                            __uint_as_float(o[v4 * 4 + 3]) * inv);
+        } else if (valid) {
 #pragma unroll
           for (int v4 = 0; v4 < 4; ++v4) {
             uint32_t w[4];
@@ -392,12 +405,14 @@ using namespace fb;
 
 // q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block] rows of nkv*hd bf16, kv_stride elements
 // apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; sink: a number per q head
-// that joins the softmax denominator, or null; same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
+// that joins the softmax denominator, or null; kb: window, chunk and softcap, or null (only with exact_p and a bounded call: fp32 rows,
+// out_f32); ldo: elements between rows of out (0: dense); same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
 extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                                   long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                                   const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg,
                                   int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int gated,
-                                  float scale, int exact_p, long kv_stride, const float* sink, int* status, cudaStream_t s) {
+                                  float scale, int exact_p, long kv_stride, const float* sink, const KeyBounds* kb, long ldo,
+                                  int out_f32, int* status, cudaStream_t s) {
   if (nseg <= 0 || max_rows <= 0) return 0;
   if (nq % nkv) return -1;
   if ((hd != 64 && hd != 128 && hd != 256) || kv_block % FT_BKV) return -20;
@@ -409,21 +424,29 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   dim3 grid((max_rows + FT_BQ - 1) / FT_BQ, nq, nseg);
-  const float scale_log2 = 1.4426950408889634f * (scale != 0.f ? scale : 1.f / sqrtf((float)hd));
-#define FB_FT(HDV, PXV)                                                                                                 \
+  if ((kb || out_f32) && (!exact_p || gated)) return -20;
+  if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
+  if (ldo == 0) ldo = (long)nq * hd;
+  if (ldo % 8) return -20;
+  constexpr float LOG2E = 1.4426950408889634f;
+  const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
+  const float scale_log2 = LOG2E * raw_scale * (cap > 0.f ? 2.f / cap : 1.f);
+#define FB_FT(HDV, PXV, BNDV)                                                                                                 \
   {                                                                                                                \
     const size_t smem = (size_t)(FT_BQ + ((HDV == 256 ? 3 : 4) + (HDV == 256 ? 2 : 3)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
-    auto kern = attn_prefill_tc_kernel<HDV, PXV>;                                                                       \
+    auto kern = attn_prefill_tc_kernel<HDV, PXV, BNDV>;                                                                       \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
     if (e != cudaSuccess) return (int)e;                                                                           \
     launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
-               gated, scale_log2, sink, status);                                                                   \
+               gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, status);                                                                   \
   }
-  if (exact_p) {
-    if (hd == 256) FB_FT(256, true) else if (hd == 128) FB_FT(128, true) else FB_FT(64, true)
+  if (kb || out_f32) {
+    if (hd == 256) FB_FT(256, true, true) else if (hd == 128) FB_FT(128, true, true) else FB_FT(64, true, true)
+  } else if (exact_p) {
+    if (hd == 256) FB_FT(256, true, false) else if (hd == 128) FB_FT(128, true, false) else FB_FT(64, true, false)
   } else {
-    if (hd == 256) FB_FT(256, false) else if (hd == 128) FB_FT(128, false) else FB_FT(64, false)
+    if (hd == 256) FB_FT(256, false, false) else if (hd == 128) FB_FT(128, false, false) else FB_FT(64, false, false)
   }
 #undef FB_FT
   return (int)cudaGetLastError();

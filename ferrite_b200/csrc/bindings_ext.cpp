@@ -353,13 +353,18 @@ EpHandle make_ep_comm(std::vector<int64_t> peer_ptrs, int64_t rank, int64_t n_ex
   return c;
 }
 
+int is_f32(const Tensor& t) {
+  TORCH_CHECK(t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16, "bf16 or fp32 expected");
+  return t.scalar_type() == torch::kFloat32 ? 1 : 0;
+}
+
 void ep_moe(const EpHandle& c, Tensor out, Tensor x, Tensor ids, Tensor wts, Tensor w_gu, Tensor w_down,
             c10::optional<Tensor> shared, c10::optional<Tensor> shared_gate, c10::optional<Tensor> res, Tensor act,
             Tensor plan) {
   int rows = (int)x.size(0), top_k = (int)ids.size(1), inter = (int)w_down.size(2);
   TORCH_CHECK(plan.numel() >= (int64_t)rows * top_k + 3 * c.n_experts + 8, "ep_moe: plan scratch too small");
   TORCH_CHECK(act.numel() >= c.cap_rows * inter, "ep_moe: activation scratch too small");
-  check(fb_ep_moe(out.data_ptr(), x.data_ptr(), ids.data_ptr<int>(), wts.data_ptr<float>(), w_gu.data_ptr(),
+  check(fb_ep_moe(out.data_ptr(), is_f32(out), x.data_ptr(), ids.data_ptr<int>(), wts.data_ptr<float>(), w_gu.data_ptr(),
                   w_down.data_ptr(), cptr(shared), shared_gate.has_value() ? shared_gate->data_ptr<float>() : nullptr,
                   cptr(res), act.data_ptr(), plan.data_ptr<int>(), rows, top_k, c.n_experts, c.hidden, inter, c.cap_rows,
                   c.peers.data(), c.rank, c.world, (uint32_t*)c.ctr.data_ptr(), c.status.data_ptr<int>(), c.spin_limit,
@@ -554,10 +559,6 @@ void mla_qpad(Tensor qp, Tensor q, Tensor qabs, int64_t nq, int64_t dn, int64_t 
 
 // ---- models of listed layers (latent.cu). The element type of activations and cache (bf16 / fp32) is read off the tensors.
 void* optr(const c10::optional<Tensor>& t) { return t.has_value() ? t->data_ptr() : nullptr; }
-int is_f32(const Tensor& t) {
-  TORCH_CHECK(t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16, "bf16 or fp32 expected");
-  return t.scalar_type() == torch::kFloat32 ? 1 : 0;
-}
 
 void embed_grams(Tensor x, c10::optional<Tensor> xb, Tensor table, c10::optional<Tensor> grams, Tensor tok, Tensor slot, Tensor pos,
                  Tensor block_table, int64_t kv_block, c10::optional<Tensor> tok_pages, double scale, int64_t buckets,
@@ -582,9 +583,23 @@ void add_normed(Tensor x, c10::optional<Tensor> xb, Tensor y, c10::optional<Tens
                       (int)x.size(1), (long)y.stride(0), (float)eps, cur_stream()), "add_normed");
 }
 
+void add_layer_norm(Tensor x, c10::optional<Tensor> xb, Tensor y, c10::optional<Tensor> yp, c10::optional<Tensor> wts, c10::optional<Tensor> next_w,
+                    c10::optional<Tensor> next_b, int64_t width, double eps) {
+  auto row_ok = [&](const c10::optional<Tensor>& t) { return !t || (t->numel() == x.size(1) && t->is_contiguous() && is_f32(*t)); };
+  TORCH_CHECK(x.is_contiguous() && is_f32(x) && y.stride(1) == 1 && y.sizes() == x.sizes() && row_ok(next_w) && row_ok(next_b) &&
+              (!xb || (xb->is_contiguous() && xb->sizes() == x.sizes())) && next_w.has_value() == next_b.has_value() &&
+              next_w.has_value() == xb.has_value() && yp.has_value() == wts.has_value(), "add_layer_norm: layouts");
+  const int top = wts ? (int)wts->size(1) : 0;
+  TORCH_CHECK(!yp || (yp->is_contiguous() && wts->is_contiguous() && is_f32(*yp) && is_f32(*wts) && wts->size(0) == x.size(0) &&
+              yp->size(0) == x.size(0) * top && yp->size(1) == x.size(1)), "add_layer_norm: expert rows");
+  check(fb_add_layer_norm(x.data_ptr<float>(), optr(xb), xb ? is_f32(*xb) : is_f32(y), y.data_ptr(), is_f32(y), (long)y.stride(0), (const float*)cptr(yp),
+                          (const float*)cptr(wts), top, (const float*)cptr(next_w), (const float*)cptr(next_b), (int)x.size(0), (int)width,
+                          (int)x.size(1), (float)eps, cur_stream()), "add_layer_norm");
+}
+
 void silu_mul_f32(Tensor out, Tensor gu) {
-  TORCH_CHECK(is_f32(out) && is_f32(gu) && out.is_contiguous() && gu.is_contiguous() && gu.size(1) == 2 * out.size(1), "silu_mul_f32: layouts");
-  check(fb_silu_mul_f32(out.data_ptr<float>(), gu.data_ptr<float>(), (int)out.size(0), (int)out.size(1), cur_stream()), "silu_mul_f32");
+  TORCH_CHECK(is_f32(out) && is_f32(gu) && out.stride(1) == 1 && gu.is_contiguous() && gu.size(1) == 2 * out.size(1), "silu_mul_f32: layouts");
+  check(fb_silu_mul_f32(out.data_ptr<float>(), (long)out.stride(0), gu.data_ptr<float>(), (int)out.size(0), (int)out.size(1), cur_stream()), "silu_mul_f32");
 }
 
 void gqa_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::optional<Tensor> bias, Tensor inv_freq, Tensor row_slot,
@@ -603,14 +618,78 @@ void gqa_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::option
                     (int)v_off, norm ? 1 : 0, (float)eps, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_prep");
 }
 
-// Few rows of grouped-query attention: q, out [rows, heads, hd]; tensor cores for bf16 (segments of consecutive rows of one slot, the
+// sizes: heads, maps, dim, vdim, rotated columns, first column of the values
+void gqa_row_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::optional<Tensor> q_norm, c10::optional<Tensor> k_norm, Tensor inv_freq,
+                  Tensor row_slot, Tensor row_pos, Tensor block_table, int64_t kv_block, std::vector<int64_t> sizes, double eps, Tensor status) {
+  TORCH_CHECK(sizes.size() == 6, "gqa_row_prep: six sizes");
+  const int64_t heads = sizes[0], maps = sizes[1], dim = sizes[2], vdim = sizes[3], rot = sizes[4], v_off = sizes[5];
+  const int64_t kvh = k_cache.size(2), hp = q.size(2);
+  TORCH_CHECK(q.is_contiguous() && q.size(1) == heads * maps && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.sizes() == v_cache.sizes() &&
+              k_cache.size(3) == hp && k_cache.size(1) == kv_block && is_f32(proj) && proj.stride(1) == 1 && proj.size(0) == q.size(0) &&
+              q.scalar_type() == k_cache.scalar_type() && q.scalar_type() == v_cache.scalar_type() && v_off >= (heads + kvh) * maps * dim &&
+              proj.size(1) >= v_off + kvh * vdim && inv_freq.scalar_type() == torch::kFloat64 && inv_freq.numel() * 2 >= rot &&
+              (!q_norm || (is_f32(*q_norm) && q_norm->numel() == heads * maps * dim)) &&
+              (!k_norm || (is_f32(*k_norm) && k_norm->numel() == kvh * maps * dim)), "gqa_row_prep: layouts");
+  check(fb_gqa_row_prep(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), proj.data_ptr<float>(), (long)proj.stride(0),
+                        (const float*)cptr(q_norm), (const float*)cptr(k_norm), inv_freq.data_ptr<double>(), row_slot.data_ptr<int>(),
+                        row_pos.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block, (int)q.size(0), (int)heads,
+                        (int)kvh, (int)maps, (int)dim, (int)vdim, (int)hp, (int)rot, (int)v_off, (float)eps, is_f32(q), status.data_ptr<int>(),
+                        cur_stream()), "gqa_row_prep");
+}
+
+// Two maps per head, output gates: out [rows, heads, hd] from in [rows, heads * maps, hd]
+void head_mix(Tensor out, Tensor in, c10::optional<Tensor> lam, c10::optional<Tensor> gate, double scale, int64_t maps, int64_t vdim, double eps) {
+  const int64_t heads = out.size(1), hd = out.size(2);
+  TORCH_CHECK(out.stride(2) == 1 && out.stride(1) == hd && in.is_contiguous() && is_f32(in) && in.size(0) == out.size(0) &&
+              in.size(1) == heads * maps && in.size(2) == hd && (!gate || (is_f32(*gate) && gate->stride(1) == 1 && gate->size(1) == heads * vdim &&
+              gate->size(0) == out.size(0))) && (maps == 1 || (lam && is_f32(*lam))), "head_mix: layouts");
+  check(fb_head_mix(out.data_ptr(), (long)out.stride(0), in.data_ptr<float>(), (const float*)cptr(lam), (const float*)cptr(gate),
+                    gate ? (long)gate->stride(0) : 0, (float)scale, (int)maps, (int)out.size(0), (int)heads, (int)vdim, (int)hd, (float)eps,
+                    is_f32(out), cur_stream()), "head_mix");
+}
+
+// Rows of every (token, pick)'s expert: x [rows, hidden], w_gu [experts, 2 inter, hidden], w_down [experts, hidden, inter]
+void expert_rows(Tensor yp, Tensor act, Tensor x, Tensor w_gu, Tensor w_down, Tensor ids) {
+  const int pairs = (int)ids.numel(), top = (int)ids.size(1), hidden = (int)x.size(1), inter = (int)w_down.size(2), ne = (int)w_down.size(0);
+  TORCH_CHECK(x.is_contiguous() && w_gu.is_contiguous() && w_down.is_contiguous() && ids.is_contiguous() && yp.is_contiguous() &&
+              act.is_contiguous() && is_f32(yp) && yp.size(0) == pairs && yp.size(1) == hidden && act.size(0) == pairs && act.size(1) == inter &&
+              w_gu.size(0) == ne && w_gu.size(1) == 2 * inter && w_gu.size(2) == hidden && w_down.size(1) == hidden &&
+              act.scalar_type() == x.scalar_type() && w_gu.scalar_type() == x.scalar_type() && w_down.scalar_type() == x.scalar_type() &&
+              ids.size(0) == x.size(0), "expert_rows: layouts");
+  if (is_f32(x)) {
+    check(fb_expert_rows_f32(yp.data_ptr<float>(), act.data_ptr<float>(), x.data_ptr<float>(), w_gu.data_ptr<float>(), w_down.data_ptr<float>(),
+                             ids.data_ptr<int>(), pairs, top, hidden, inter, ne, cur_stream()), "expert_rows_f32");
+    return;
+  }
+  check(fb_moe_gate_up(act.data_ptr(), x.data_ptr(), w_gu.data_ptr(), ids.data_ptr<int>(), pairs, top, hidden, inter, 0, ne, cur_stream()),
+        "moe_gate_up");
+  check(fb_moe_down(yp.data_ptr<float>(), act.data_ptr(), w_down.data_ptr(), ids.data_ptr<int>(), pairs, hidden, inter, 0, ne, cur_stream()),
+        "moe_down");
+}
+
+// Few rows of grouped-query attention: q [rows, queries, hd], out [rows, heads, hd] (rows may lie apart; queries = maps * heads); with lam or
+// gate what follows the attention rides on the merge of the splits; tensor cores for bf16 (segments of consecutive rows of one slot, the
 // step's row row_first first), CUDA cores otherwise.
 void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cache, Tensor v_cache, c10::optional<Tensor> sink,
               Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, Tensor row_slot, Tensor row_kvlen, Tensor block_table,
-              int64_t kv_block, int64_t row_first, int64_t nsplit, double scale, bool cuda_cores, Tensor status) {
+              int64_t kv_block, int64_t row_first, int64_t nsplit, double scale, bool cuda_cores, Tensor status, int64_t window, int64_t chunk,
+              double softcap, c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t maps, int64_t vdim, double eps) {
   const int rows = (int)q.size(0), heads = (int)q.size(1), hd = (int)q.size(2), kvh = (int)k_cache.size(2);
   const long recs = (long)rows * heads * nsplit;
-  TORCH_CHECK(q.is_contiguous() && out.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.size(3) == hd &&
+  const bool mixed = lam.has_value() || gate.has_value();
+  const KeyBounds kb{(int)window, (int)chunk, (float)softcap};
+  const KeyBounds* kbp = window || chunk || softcap != 0.0 ? &kb : nullptr;
+  TORCH_CHECK(out.dim() == 3 && out.stride(2) == 1 && out.stride(1) == hd && out.size(1) * maps == heads && out.size(2) == hd &&
+              out.scalar_type() == q.scalar_type() && (maps == 1 || (maps == 2 && lam && is_f32(*lam))) && (!mixed || (!sink && vdim > 0)) &&
+              (!gate || (is_f32(*gate) && gate->stride(1) == 1 && gate->size(0) == rows && gate->size(1) == out.size(1) * vdim)),
+              "gqa_attn: outputs");
+  const long ldo = (long)out.stride(0);
+  auto finish = [&]() {
+    check(fb_attn_merge_mix(out.data_ptr(), ldo, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), (const float*)cptr(lam),
+                            (const float*)cptr(gate), gate ? (long)gate->stride(0) : 0, (float)mix_scale, (int)maps, rows, (int)out.size(1),
+                            (int)nsplit, (int)vdim, hd, (float)eps, is_f32(out), cur_stream()), "attn_merge_mix");
+  };
+  TORCH_CHECK(q.is_contiguous() && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.size(3) == hd &&
               o_part.numel() >= recs * hd && ml_part.numel() >= recs * 2 && row_slot.numel() == rows && row_kvlen.numel() == rows &&
               (!sink || sink->numel() == heads), "gqa_attn: layouts");
   const float* sk = (const float*)cptr(sink);
@@ -618,15 +697,17 @@ void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cach
     check(fb_attn_decode_mma(nullptr, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                              nullptr, nullptr, 0, seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(),
                              row_kvlen.data_ptr<int>(), nullptr, nullptr, block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block,
-                             (int)seg_slot.numel(), (int)max_rows, rows, heads, kvh, hd, (int)nsplit, 0, (float)scale, 1, (int)row_first,
+                             (int)seg_slot.numel(), (int)max_rows, rows, heads, kvh, hd, (int)nsplit, 0, (float)scale, 1, kbp, (int)row_first,
                              cur_stream()), "attn_decode_mma");
-    check(fb_attn_merge(out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), sk, rows, heads, (int)nsplit, hd, cur_stream()),
+    if (mixed) return finish();
+    check(fb_attn_merge(out.data_ptr(), ldo, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), sk, rows, heads, (int)nsplit, hd, cur_stream()),
           "attn_merge");
     return;
   }
-  check(fb_gqa_attn(out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+  check(fb_gqa_attn(mixed ? nullptr : out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                     sk, row_slot.data_ptr<int>(), row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
-                    (int)kv_block, rows, heads, kvh, hd, (int)nsplit, (float)scale, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_attn");
+                    (int)kv_block, rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, ldo, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_attn");
+  if (mixed) finish();
 }
 
 // Channel-delta layers. sizes: heads, kv_heads, dim, vdim, taps, first convolved column of the projection.
@@ -711,9 +792,10 @@ void gated_norm_sigmoid(Tensor out, Tensor y, Tensor z, Tensor w, double eps) {
                               w.data_ptr<float>(), (int)y.size(0), heads, dv, (float)eps, is_f32(out), cur_stream()), "gated_norm_sigmoid");
 }
 
-void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, int64_t width, double eps) {
-  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && out.size(1) == x.size(1) && w.numel() == x.size(1), "norm_rows: layouts");
-  check(fb_norm_rows(out.data_ptr(), x.data_ptr<float>(), (const int*)cptr(idx), w.data_ptr<float>(), (int)out.size(0), (int)width,
+void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, c10::optional<Tensor> bias, int64_t width, double eps) {
+  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && out.size(1) == x.size(1) && w.numel() == x.size(1) && is_f32(w) &&
+              (!bias || (bias->numel() == x.size(1) && is_f32(*bias))), "norm_rows: layouts");
+  check(fb_norm_rows(out.data_ptr(), x.data_ptr<float>(), (const int*)cptr(idx), w.data_ptr<float>(), (const float*)cptr(bias), (int)out.size(0), (int)width,
                      (int)x.size(1), (float)eps, is_f32(out), cur_stream()), "norm_rows");
 }
 
@@ -857,7 +939,16 @@ void register_ext(pybind11::module_& m) {
   m.def("gemm_f32", &gemm_f32);
   m.def("silu_mul_f32", &silu_mul_f32);
   m.def("gqa_prep", &gqa_prep);
-  m.def("gqa_attn", &gqa_attn);
+  m.def("gqa_attn", &gqa_attn, pybind11::arg("out"), pybind11::arg("o_part"), pybind11::arg("ml_part"), pybind11::arg("q"), pybind11::arg("k_cache"), pybind11::arg("v_cache"),
+        pybind11::arg("sink"), pybind11::arg("seg_slot"), pybind11::arg("seg_row0"), pybind11::arg("seg_nrows"), pybind11::arg("max_rows"), pybind11::arg("row_slot"),
+        pybind11::arg("row_kvlen"), pybind11::arg("block_table"), pybind11::arg("kv_block"), pybind11::arg("row_first"), pybind11::arg("nsplit"), pybind11::arg("scale"),
+        pybind11::arg("cuda_cores"), pybind11::arg("status"), pybind11::arg("window") = 0, pybind11::arg("chunk") = 0, pybind11::arg("softcap") = 0.0,
+        pybind11::arg("lam") = pybind11::none(), pybind11::arg("gate") = pybind11::none(), pybind11::arg("mix_scale") = 1.0, pybind11::arg("maps") = 1, pybind11::arg("vdim") = 0,
+        pybind11::arg("eps") = 0.0);
+  m.def("gqa_row_prep", &gqa_row_prep);
+  m.def("head_mix", &head_mix);
+  m.def("expert_rows", &expert_rows);
+  m.def("add_layer_norm", &add_layer_norm);
   m.def("cd_lowrank", &cd_lowrank);
   m.def("cd_step", &cd_step);
   m.def("cd_tail", &cd_tail);

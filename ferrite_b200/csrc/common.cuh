@@ -42,6 +42,17 @@ __device__ __forceinline__ void set_status(int* status, int code) {
 __device__ __forceinline__ float bf2f(__nv_bfloat16 x) { return __bfloat162float(x); }
 __device__ __forceinline__ __nv_bfloat16 f2bf(float x) { return __float2bfloat16_rn(x); }
 __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + __expf(-x)); }
+// First key that the row at `pos` sees under a window or a chunk (0 = neither).
+__host__ __device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  if (window > 0) return pos >= window ? pos - window + 1 : 0;
+  return chunk > 0 ? pos - pos % chunk : 0;
+}
+// tanh(x) = 1 - 2 / (e^2x + 1), given x * 2 log2(e); off by a few 2^-23 of one
+__device__ __forceinline__ float tanh_of_2log2(float x) {
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x));
+  return 1.f - __fdividef(2.f, e + 1.f);
+}
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
 

@@ -76,12 +76,12 @@ __global__ void rmsnorm_kernel(__nv_bfloat16* __restrict__ out, __nv_bfloat16* _
 }
 
 // The same in fp32
-__global__ void silu_mul_f32_kernel(float* __restrict__ out, const float* __restrict__ gu, int inter) {
+__global__ void silu_mul_f32_kernel(float* __restrict__ out, long ldo, const float* __restrict__ gu, int inter) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= inter) return;
   const float* r = gu + (size_t)blockIdx.y * 2 * inter;
   const float g = r[i];
-  out[(size_t)blockIdx.y * inter + i] = g / (1.f + expf(-g)) * r[inter + i];
+  out[(size_t)blockIdx.y * ldo + i] = g / (1.f + expf(-g)) * r[inter + i];
 }
 
 // out[r][i] = silu(gu[r][i]) * gu[r][inter + i]
@@ -186,10 +186,10 @@ extern "C" int fb_silu_mul(void* out, const void* gu, int rows, int inter, float
   return (int)cudaGetLastError();
 }
 
-extern "C" int fb_silu_mul_f32(float* out, const float* gu, int rows, int inter, cudaStream_t s) {
+extern "C" int fb_silu_mul_f32(float* out, long ldo, const float* gu, int rows, int inter, cudaStream_t s) {
   if (rows <= 0 || inter <= 0) return 0;
   if (rows > 65535) return -1;
-  silu_mul_f32_kernel<<<dim3((inter + 255) / 256, rows), 256, 0, s>>>(out, gu, inter);
+  silu_mul_f32_kernel<<<dim3((inter + 255) / 256, rows), 256, 0, s>>>(out, ldo, gu, inter);
   return (int)cudaGetLastError();
 }
 

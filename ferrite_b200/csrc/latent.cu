@@ -10,7 +10,8 @@
 //                  kernel over separate keys and values of grouped heads, with a sink, is what grouped-query attention runs in 32
 //                  bits and at head widths the tensor-core kernels do not take
 //   add_normed     x += rms(y + bias) * w on the 32-bit residual stream, plus the next GEMM's operand: the new x or its norm
-//   norm_rows      rms(x[idx]) * w for the rows whose logits are wanted
+//   norm_rows      rms(x[idx]) * w for the rows whose logits are wanted; layer_norm_rows the same with the mean off and a bias
+//   add_layer_norm x += y + weighted expert rows, plus the next GEMM's operand, the layer norm of the new x (parallel blocks)
 //   softcap        logits <- cap * tanh(logits / cap)
 //   gemm_f32       y = x W^T in 32 bits on the CUDA cores, optionally one product per head
 //
@@ -145,6 +146,85 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const float* __restrict__ 
   }
 }
 
+// ---- layer norms (mean off, bias): rows of `width` true columns, zeros up to ld ------------------------------------------
+// The row waits in shared memory (every thread reads what it wrote itself); mean first, then the squared deviations of the true columns.
+__device__ __forceinline__ float2 ln_stats(const float* row, float sum, int width, int ld, float eps, float* red) {
+  const float mean = block_sum(sum, red) / (float)width;
+  float ss = 0.f;
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    const float4 v = *reinterpret_cast<const float4*>(row + i);
+    const float a = v.x - mean, b = v.y - mean, c = v.z - mean, d = v.w - mean;
+    if (i + 3 < width) {
+      ss = fmaf(a, a, fmaf(b, b, fmaf(c, c, fmaf(d, d, ss))));
+    } else {
+      if (i < width) ss = fmaf(a, a, ss);
+      if (i + 1 < width) ss = fmaf(b, b, ss);
+      if (i + 2 < width) ss = fmaf(c, c, ss);
+    }
+  }
+  return make_float2(mean, 1.f / sqrtf(block_sum(ss, red) / (float)width + eps));
+}
+template <typename T>
+__device__ __forceinline__ void ln_store(T* out, const float* row, float2 st, const float* w, const float* b, int ld) {
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(row + i);
+    const float4 ww = *reinterpret_cast<const float4*>(w + i), bb = *reinterpret_cast<const float4*>(b + i);
+    v.x = (v.x - st.x) * st.y * ww.x + bb.x; v.y = (v.y - st.x) * st.y * ww.y + bb.y;
+    v.z = (v.z - st.x) * st.y * ww.z + bb.z; v.w = (v.w - st.x) * st.y * ww.w + bb.w;
+    Elem<T>::store4(out + i, v);
+  }
+}
+
+// x[row] += y[row] + sum over `top` picks of wts[row][k] * yp[row * top + k]; xb = layer norm of the new x (no w: none)
+template <typename T, typename S>
+__global__ void add_layer_norm_kernel(float* __restrict__ x, T* __restrict__ xb, const S* __restrict__ y, long ldy, const float* __restrict__ yp,
+                                      const float* __restrict__ wts, int top, const float* __restrict__ w, const float* __restrict__ b,
+                                      int width, int ld, float eps) {
+  extern __shared__ __align__(16) float al_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const S* yr = y + row * ldy;
+  float* xr = x + row * ld;
+  float sum = 0.f;
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    float4 a = *reinterpret_cast<const float4*>(xr + i);
+    const float4 v = Elem<S>::load4(yr + i);
+    float4 s = v;
+    for (int k = 0; k < top; ++k) {
+      const float g = wts[row * top + k];
+      const float4 e = *reinterpret_cast<const float4*>(yp + (row * top + k) * ld + i);
+      s.x = fmaf(g, e.x, s.x); s.y = fmaf(g, e.y, s.y); s.z = fmaf(g, e.z, s.z); s.w = fmaf(g, e.w, s.w);
+    }
+    a.x += s.x; a.y += s.y; a.z += s.z; a.w += s.w;
+    *reinterpret_cast<float4*>(xr + i) = a;
+    if (w) *reinterpret_cast<float4*>(al_row + i) = a;
+    sum += (a.x + a.y) + (a.z + a.w);
+  }
+  if (!w) return;
+  const float2 st = ln_stats(al_row, sum, width, ld, eps, red);
+  ln_store<T>(xb + row * ld, al_row, st, w, b, ld);
+}
+
+template <typename T>
+__global__ void layer_norm_rows_kernel(T* __restrict__ out, const float* __restrict__ x, const int* __restrict__ idx,
+                                       const float* __restrict__ w, const float* __restrict__ b, int width, int ld, float eps) {
+  extern __shared__ __align__(16) float al_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * ld;
+  float sum = 0.f;
+  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
+    const float4 v = *reinterpret_cast<const float4*>(xr + i);
+    *reinterpret_cast<float4*>(al_row + i) = v;
+    sum += (v.x + v.y) + (v.z + v.w);
+  }
+  const float2 st = ln_stats(al_row, sum, width, ld, eps, red);
+  ln_store<T>(out + (size_t)blockIdx.x * ld, al_row, st, w, b, ld);
+}
+
 // proj row = [query latent (qr columns, q_rank true) | key / value latent (lat columns, kv_rank true)], fp32.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ cq, T* __restrict__ cache, const float* __restrict__ proj,
@@ -200,7 +280,8 @@ __global__ void relu2_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16*
 // grid (rows, heads, splits), 4 warps striding over the keys with an online softmax; a lane owns columns 64 j + 2 lane, + 1.
 // lat = 64 nl with nl <= NJ. One split writes the normalised output itself, more leave partials for the merge. KV: cache rows are
 // [kv_heads][lat] of keys with the values in v_cache (else one latent row, keys and values alike); sink: a number per head that
-// joins the denominator.
+// joins the denominator; window / chunk bound the keys a row sees, cap > 0 softcaps the scores (scale_log2 is then scale / cap).
+// `records`: one split leaves its partial as well. Rows of out are ldo elements apart.
 constexpr int LA_WARPS = 4;
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -212,7 +293,8 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
                                                                     const int* __restrict__ row_kvlen,
                                                                     const int* __restrict__ block_table, int max_blocks,
                                                                     int kv_block, int heads, int kv_heads, int lat, int nsplit,
-                                                                    float scale_log2, int* status) {
+                                                                    float scale_log2, int window, int chunk, float cap, long ldo, int records,
+                                                                    int* status) {
   extern __shared__ float so[];                            // [warps][lat]
   __shared__ float sml[LA_WARPS][2];
   pdl_launch_dependents();
@@ -222,9 +304,10 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kvlen = row_kvlen[row];
   const int* bt = block_table + (size_t)row_slot[row] * max_blocks;
-  int per = (kvlen + nsplit - 1) / nsplit;
+  const int kv_lo = KV ? first_key(kvlen - 1, window, chunk) : 0;
+  int per = (kvlen - kv_lo + nsplit - 1) / nsplit;
   per = (per + 31) / 32 * 32;
-  const int lo = split * per, hi = min(kvlen, lo + per);
+  const int lo = kv_lo + split * per, hi = min(kvlen, lo + per);
   const T* qr = q + ((size_t)row * heads + h) * lat;
   float2 qf[NJ], o[NJ];
 #pragma unroll
@@ -247,6 +330,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
 #pragma unroll
     for (int j = 0; j < NJ; ++j) s = fmaf(qf[j].x, k[j].x, fmaf(qf[j].y, k[j].y, s));
     s = warp_sum(s);
+    if constexpr (KV) { if (cap > 0.f) s = cap * LOG2E * tanhf(s); }
     const float mn = fmaxf(m, s);
     const float a = exp2f(m - mn), p = exp2f(s - mn);
     l = l * a + p;
@@ -274,15 +358,16 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
   }
   const size_t pidx = ((size_t)row * heads + h) * nsplit + split;
   const float den = Ls + (sink && nsplit == 1 ? exp2f(sink[h] * LOG2E - M) : 0.f);
-  const float inv = nsplit == 1 ? (den > 0.f ? 1.f / den : 0.f) : 1.f;
+  const bool final_rows = nsplit == 1 && !records;
+  const float inv = final_rows ? (den > 0.f ? 1.f / den : 0.f) : 1.f;
   for (int d = threadIdx.x; d < lat; d += blockDim.x) {
     float acc = 0.f;
 #pragma unroll
     for (int w = 0; w < LA_WARPS; ++w) acc += so[(size_t)w * lat + d] * f[w];
-    if (nsplit == 1) out[((size_t)row * heads + h) * lat + d] = Elem<T>::from(acc * inv);
+    if (final_rows) out[(size_t)row * ldo + (size_t)h * lat + d] = Elem<T>::from(acc * inv);
     else o_part[pidx * lat + d] = acc;
   }
-  if (nsplit > 1 && threadIdx.x == 0) { ml_part[pidx * 2] = M; ml_part[pidx * 2 + 1] = Ls; }
+  if (!final_rows && threadIdx.x == 0) { ml_part[pidx * 2] = M; ml_part[pidx * 2 + 1] = Ls; }
 }
 
 // Merge of the splits; grid (rows, heads). LG_GROUPS groups of 128 threads take every LG_GROUPS-th split each (all loads of a
@@ -290,7 +375,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
 constexpr int LG_GROUPS = 4;
 
 template <typename T>
-__global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __restrict__ out, const float* __restrict__ o_part,
+__global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __restrict__ out, long ldo, const float* __restrict__ o_part,
                                                                        const float* __restrict__ ml_part,
                                                                        const float* __restrict__ sink, int heads, int nsplit, int lat) {
   extern __shared__ float sf[];                            // [nsplit] factors, then [groups][lat] partial sums
@@ -332,8 +417,124 @@ __global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __rest
       for (int g = 0; g < LG_GROUPS; ++g)
 #pragma unroll
         for (int e = 0; e < 4; ++e) v[e] += sums[g * lat + d + e];
-      Elem<T>::store4(out + rh * lat + d, make_float4(v[0] * inv, v[1] * inv, v[2] * inv, v[3] * inv));
+      Elem<T>::store4(out + (size_t)blockIdx.x * ldo + (size_t)blockIdx.y * lat + d, make_float4(v[0] * inv, v[1] * inv, v[2] * inv, v[3] * inv));
     }
+}
+
+// ---- heads' outputs: difference of two maps, norm, output gate -----------------------------------------------------------
+// o = a1 - lam a2, divided by its root mean square over vdim and scaled (two maps), times sigmoid(gate): from the records of key splits
+// (one CTA per row and head; half of it per map) or from normalised rows (one warp per row and head).
+constexpr int MX_THREADS = 256;
+
+template <typename T, int MAPS>
+__global__ void __launch_bounds__(MX_THREADS) attn_merge_mix_kernel(T* __restrict__ out, long ldo, const float* __restrict__ o_part,
+                                                                    const float* __restrict__ ml_part, const float* __restrict__ lam,
+                                                                    const float* __restrict__ gate, long ldg, float mix_scale, int heads,
+                                                                    int nsplit, int vdim, int hd, float eps) {
+  constexpr int PER = MX_THREADS / MAPS;                   // threads of a map
+  extern __shared__ __align__(16) float mx_s[];            // [MAPS][nsplit] factors, [MAPS] 1 / row sum, [MAPS][groups][hd] sums
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, map = tid / PER, t = tid % PER, warp = tid >> 5, lane = tid & 31;
+  const size_t row = blockIdx.x;
+  const int h = blockIdx.y;
+  const size_t pbase = ((row * heads + h) * MAPS + map) * nsplit;
+  float* fac = mx_s + map * nsplit;
+  float* inv = mx_s + MAPS * nsplit;
+  float* sums = mx_s + (MAPS * nsplit + MAPS + 3) / 4 * 4;
+  if (warp < MAPS) {                                       // one warp per map turns the maxima into factors
+    const size_t pb = ((row * heads + h) * MAPS + warp) * nsplit;
+    float M = -INFINITY, L = 0.f;
+    for (int s = lane; s < nsplit; s += 32) M = fmaxf(M, ml_part[(pb + s) * 2]);
+    M = warp_max(M);
+    for (int s = lane; s < nsplit; s += 32) {
+      const float ms = ml_part[(pb + s) * 2];
+      const float f = ms == -INFINITY ? 0.f : exp2f(ms - M);         // an empty split wrote no rows
+      mx_s[warp * nsplit + s] = f;
+      if (f != 0.f) L += ml_part[(pb + s) * 2 + 1] * f;
+    }
+    L = warp_sum(L);
+    if (lane == 0) inv[warp] = L > 0.f ? 1.f / L : 0.f;
+  }
+  __syncthreads();
+  const int cols = hd / 4, groups = max(1, PER / cols);    // groups of threads take every groups-th split
+  for (int i = t; i < cols * groups; i += PER) {
+    const int g = i / cols, d = (i % cols) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = g; s < nsplit; s += groups) {
+      const float f = fac[s];
+      if (f == 0.f) continue;
+      const float4 v = *reinterpret_cast<const float4*>(o_part + (pbase + s) * hd + d);
+      acc.x = fmaf(v.x, f, acc.x); acc.y = fmaf(v.y, f, acc.y); acc.z = fmaf(v.z, f, acc.z); acc.w = fmaf(v.w, f, acc.w);
+    }
+    *reinterpret_cast<float4*>(sums + ((size_t)map * groups + g) * hd + d) = acc;
+  }
+  __syncthreads();
+  const float l2 = MAPS == 2 ? lam[0] : 0.f;
+  float ss = 0.f;
+  for (int d = tid; d < hd; d += MX_THREADS) {
+    float a[MAPS];
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+      a[m] = 0.f;
+      for (int g = 0; g < groups; ++g) a[m] += sums[((size_t)m * groups + g) * hd + d];
+      a[m] *= inv[m];
+    }
+    const float o = MAPS == 2 ? a[0] - l2 * a[MAPS - 1] : a[0];
+    sums[d] = o;                                           // this thread's own column of group 0
+    ss = fmaf(o, o, ss);
+  }
+  const float r = MAPS == 2 ? mix_scale / sqrtf(block_sum(ss, red) / (float)vdim + eps) : 1.f;
+  for (int d = tid; d < hd; d += MX_THREADS) {
+    float o = sums[d] * r;
+    if (gate && d < vdim) o *= 1.f / (1.f + expf(-gate[row * ldg + (size_t)h * vdim + d]));
+    out[row * ldo + (size_t)h * hd + d] = Elem<T>::from(o);
+  }
+}
+
+// in [rows][heads * MAPS][hd] fp32, zeros beyond vdim
+template <typename T, int MAPS>
+__global__ void __launch_bounds__(256) head_mix_kernel(T* __restrict__ out, long ldo, const float* __restrict__ in, const float* __restrict__ lam,
+                                                       const float* __restrict__ gate, long ldg, float mix_scale, int heads, int vdim, int hd,
+                                                       float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= heads) return;
+  const float* a = in + (row * heads + h) * MAPS * hd;
+  T* dst = out + row * ldo + (size_t)h * hd;
+  const float l2 = MAPS == 2 ? lam[0] : 0.f;
+  float ss = 0.f;
+  auto value = [&](int d) {
+    float4 v = *reinterpret_cast<const float4*>(a + d);
+    if constexpr (MAPS == 2) {
+      const float4 b = *reinterpret_cast<const float4*>(a + hd + d);
+      v.x -= l2 * b.x; v.y -= l2 * b.y; v.z -= l2 * b.z; v.w -= l2 * b.w;
+    }
+    return v;
+  };
+  float r = 1.f;
+  if constexpr (MAPS == 2) {
+    for (int d = lane * 4; d < hd; d += 128) {
+      const float4 v = value(d);
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+    r = mix_scale / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  }
+  for (int d = lane * 4; d < hd; d += 128) {
+    const float4 v = value(d);
+    float o[4] = {v.x * r, v.y * r, v.z * r, v.w * r};
+    if (gate) {
+      const float* g = gate + row * ldg + (size_t)h * vdim + d;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (d + e < vdim) o[e] *= 1.f / (1.f + expf(-g[e]));
+    }
+    Elem<T>::store4(dst + d, make_float4(o[0], o[1], o[2], o[3]));
+  }
 }
 
 // ---- attention over the cached latents, tensor cores ---------------------------------------------------------------------
@@ -677,13 +878,42 @@ extern "C" int fb_add_normed(float* x, void* xb, int xb_f32, long ldb, const voi
   return go(add_normed_kernel<bf16, bf16>, (bf16*)xb, (const bf16*)y);
 }
 
-extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, int rows, int width, int ld, float eps,
+template <typename Kern>
+static int row_smem(Kern kern, size_t smem) {
+  return smem > 40 * 1024 ? (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : 0;
+}
+
+// b: bias of a layer norm, or null for the root mean square norm
+extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int rows, int width, int ld, float eps,
                             int f32, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (ld % 4) return -1;
+  if (ld % 4 || ld > 49152) return -1;
+  const dim3 g(rows), t(row_threads(ld));
+  if (b) {
+    auto go = [&](auto kern, auto* o) {
+      if (const int e = row_smem(kern, (size_t)ld * 4)) return e;
+      return (int)launch_pdl(kern, g, t, (size_t)ld * 4, s, o, x, idx, w, b, width, ld, eps);
+    };
+    return f32 ? go(layer_norm_rows_kernel<float>, (float*)out) : go(layer_norm_rows_kernel<bf16>, (bf16*)out);
+  }
+  if (f32) return (int)launch_pdl(norm_rows_kernel<float>, g, t, 0, s, (float*)out, x, idx, w, width, ld, eps);
+  return (int)launch_pdl(norm_rows_kernel<bf16>, g, t, 0, s, (bf16*)out, x, idx, w, width, ld, eps);
+}
+
+// y: fp32 (y_f32) or bf16 rows of stride ldy; yp / wts: rows of a token's `top` experts and their weights (top 0: none); next_w, next_b:
+// ld floats, or null for no operand
+extern "C" int fb_add_layer_norm(float* x, void* xb, int f32, const void* y, int y_f32, long ldy, const float* yp, const float* wts, int top,
+                                 const float* next_w, const float* next_b, int rows, int width, int ld, float eps, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (ld % 4 || ldy % 4 || ld > 49152 || (next_w && (!xb || !next_b)) || (top && (!yp || !wts)) || (f32 && !y_f32)) return -1;
   const dim3 g(rows), b(row_threads(ld));
-  if (f32) return (int)launch_pdl(norm_rows_kernel<float>, g, b, 0, s, (float*)out, x, idx, w, width, ld, eps);
-  return (int)launch_pdl(norm_rows_kernel<bf16>, g, b, 0, s, (bf16*)out, x, idx, w, width, ld, eps);
+  auto go = [&](auto kern, auto* xo, const auto* yi) {
+    if (const int e = row_smem(kern, (size_t)ld * 4)) return e;
+    return (int)launch_pdl(kern, g, b, (size_t)ld * 4, s, x, xo, yi, ldy, yp, wts, top, next_w, next_b, width, ld, eps);
+  };
+  if (f32) return go(add_layer_norm_kernel<float, float>, (float*)xb, (const float*)y);
+  if (y_f32) return go(add_layer_norm_kernel<bf16, float>, (bf16*)xb, (const float*)y);
+  return go(add_layer_norm_kernel<bf16, bf16>, (bf16*)xb, (const bf16*)y);
 }
 
 extern "C" int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
@@ -713,30 +943,35 @@ extern "C" int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaS
 }
 
 template <typename T>
-static int latent_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int lat,
+static int latent_merge(void* out, long ldo, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int lat,
                         cudaStream_t s) {
   return (int)launch_pdl(latent_merge_kernel<T>, dim3(rows, heads), dim3(128 * LG_GROUPS),
-                         (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out, o_part, ml_part, sink, heads, nsplit, lat);
+                         (size_t)(nsplit + LG_GROUPS * lat) * 4, s, (T*)out, ldo, o_part, ml_part, sink, heads, nsplit, lat);
 }
 
 template <typename T, bool KV>
 static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const void* v_cache, const float* sink,
                        const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
-                       int kv_heads, int lat, int nsplit, float scale_log2, int* status, cudaStream_t s) {
+                       int kv_heads, int lat, int nsplit, float scale, const KeyBounds* kb, long ldo, bool records, int* status,
+                       cudaStream_t s) {
+  const KeyBounds none{0, 0, 0.f};
+  const KeyBounds& b = kb ? *kb : none;
+  if (b.window < 0 || b.chunk < 0 || (b.window && b.chunk) || b.cap < 0.f) return -1;
+  const float scale_log2 = b.cap > 0.f ? scale / b.cap : scale * LOG2E;
   const dim3 grid(rows, heads, nsplit);
   const size_t smem = (size_t)LA_WARPS * lat * 4;
   auto go = [&](auto kern) {
     return (int)launch_pdl(kern, grid, dim3(LA_WARPS * 32), smem, s, (T*)out, o_part, ml_part, (const T*)q, (const T*)cache,
                            (const T*)v_cache, sink, row_slot, row_kvlen, block_table, max_blocks, kv_block, heads, kv_heads, lat, nsplit,
-                           scale_log2, status);
+                           scale_log2, b.window, b.chunk, b.cap, ldo, records ? 1 : 0, status);
   };
   int rc;
   if (lat <= 128) rc = go(latent_attn_kernel<T, 2, KV>);
   else if (lat <= 256) rc = go(latent_attn_kernel<T, 4, KV>);
   else if (lat <= 512) rc = go(latent_attn_kernel<T, 8, KV>);
   else rc = go(latent_attn_kernel<T, 16, KV>);
-  if (rc || nsplit == 1) return rc;
-  return latent_merge<T>(out, o_part, ml_part, sink, rows, heads, nsplit, lat, s);
+  if (rc || nsplit == 1 || records) return rc;
+  return latent_merge<T>(out, ldo, o_part, ml_part, sink, rows, heads, nsplit, lat, s);
 }
 
 // out [rows][heads][lat]; partials (nsplit > 1): o_part rows * heads * nsplit * lat floats, ml_part two per record
@@ -745,33 +980,64 @@ extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const vo
                               int nsplit, float scale, int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
-  const float sl = scale * 1.4426950408889634f;
+  const long ldo = (long)heads * lat;
   return f32 ? latent_attn<float, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
-                                         kv_block, rows, heads, 1, lat, nsplit, sl, status, s)
+                                         kv_block, rows, heads, 1, lat, nsplit, scale, nullptr, ldo, false, status, s)
              : latent_attn<bf16, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
-                                        kv_block, rows, heads, 1, lat, nsplit, sl, status, s);
+                                        kv_block, rows, heads, 1, lat, nsplit, scale, nullptr, ldo, false, status, s);
 }
 
-// The same over separate keys and values: caches [page][kv_block][kv_heads][hd], q / out [rows][heads][hd]; sink: heads floats or null
+// The same over separate keys and values: caches [page][kv_block][kv_heads][hd], q / out [rows][heads][hd] (rows of out ldo elements
+// apart); sink: heads floats or null; kb: window, chunk, softcap, or null; out null: the records of the splits stay for the caller
 extern "C" int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache,
                            const float* sink, const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks,
-                           int kv_block, int rows, int heads, int kv_heads, int hd, int nsplit, float scale, int f32, int* status,
-                           cudaStream_t s) {
+                           int kv_block, int rows, int heads, int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb, long ldo,
+                           int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (hd % 64 || hd > 1024 || heads > 65535 || kv_heads <= 0 || heads % kv_heads || nsplit < 1 || nsplit > 4096) return -1;
-  const float sl = scale * LOG2E;
+  if (ldo % 4 || (!out && sink)) return -1;
   return f32 ? latent_attn<float, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
-                                        kv_block, rows, heads, kv_heads, hd, nsplit, sl, status, s)
+                                        kv_block, rows, heads, kv_heads, hd, nsplit, scale, kb, ldo, !out, status, s)
              : latent_attn<bf16, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
-                                       kv_block, rows, heads, kv_heads, hd, nsplit, sl, status, s);
+                                       kv_block, rows, heads, kv_heads, hd, nsplit, scale, kb, ldo, !out, status, s);
 }
 
 // Merge of key splits alone (records as fb_attn_decode_mma leaves them), sink: heads floats or null
-extern "C" int fb_attn_merge(void* out, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit,
+extern "C" int fb_attn_merge(void* out, long ldo, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit,
                              int hd, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (hd % 64 || hd > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
-  return latent_merge<bf16>(out, o_part, ml_part, sink, rows, heads, nsplit, hd, s);
+  if (hd % 64 || hd > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096 || ldo % 4) return -1;
+  return latent_merge<bf16>(out, ldo, o_part, ml_part, sink, rows, heads, nsplit, hd, s);
+}
+
+// Merge of key splits with what follows it: maps 2: the difference of a head's two maps (records [rows][heads][2]), its norm over vdim,
+// mix_scale; gate: rows of heads * vdim logits ldg floats apart, or null. out [rows][heads][hd], rows ldo elements apart.
+extern "C" int fb_attn_merge_mix(void* out, long ldo, const float* o_part, const float* ml_part, const float* lam, const float* gate, long ldg,
+                                 float mix_scale, int maps, int rows, int heads, int nsplit, int vdim, int hd, float eps, int f32,
+                                 cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (hd % 64 || hd > 1024 || heads > 65535 || nsplit < 1 || nsplit > 256 || maps < 1 || maps > 2 || (maps == 2 && !lam) || vdim < 1 ||
+      vdim > hd) return -1;
+  const int per = MX_THREADS / maps, groups = per / (hd / 4) > 1 ? per / (hd / 4) : 1;
+  const size_t smem = ((size_t)(maps * nsplit + maps + 3) / 4 * 4 + (size_t)maps * groups * hd) * 4;
+  auto go = [&](auto kern, auto* o) {
+    return (int)launch_pdl(kern, dim3(rows, heads), dim3(MX_THREADS), smem, s, o, ldo, o_part, ml_part, lam, gate, ldg, mix_scale, heads, nsplit,
+                           vdim, hd, eps);
+  };
+  if (f32) return maps == 2 ? go(attn_merge_mix_kernel<float, 2>, (float*)out) : go(attn_merge_mix_kernel<float, 1>, (float*)out);
+  return maps == 2 ? go(attn_merge_mix_kernel<bf16, 2>, (bf16*)out) : go(attn_merge_mix_kernel<bf16, 1>, (bf16*)out);
+}
+
+// The same for rows that need no merge: in [rows][heads * maps][hd] fp32
+extern "C" int fb_head_mix(void* out, long ldo, const float* in, const float* lam, const float* gate, long ldg, float mix_scale, int maps,
+                           int rows, int heads, int vdim, int hd, float eps, int f32, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (hd % 64 || ldo % 4 || maps < 1 || maps > 2 || (maps == 2 && !lam) || vdim < 1 || vdim > hd || (heads + 7) / 8 > 65535) return -1;
+  auto go = [&](auto kern, auto* o) {
+    return (int)launch_pdl(kern, dim3(rows, (heads + 7) / 8), dim3(256), 0, s, o, ldo, in, lam, gate, ldg, mix_scale, heads, vdim, hd, eps);
+  };
+  if (f32) return maps == 2 ? go(head_mix_kernel<float, 2>, (float*)out) : go(head_mix_kernel<float, 1>, (float*)out);
+  return maps == 2 ? go(head_mix_kernel<bf16, 2>, (bf16*)out) : go(head_mix_kernel<bf16, 1>, (bf16*)out);
 }
 
 // The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in
@@ -800,7 +1066,7 @@ extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const voi
   switch (lat / 64) { FB_LM(1) FB_LM(2) FB_LM(3) FB_LM(4) FB_LM(5) FB_LM(6) FB_LM(7) FB_LM(8) }
 #undef FB_LM
   if (rc || nsplit == 1) return rc;
-  return latent_merge<bf16>(out, o_part, ml_part, nullptr, rows, heads, nsplit, lat, s);
+  return latent_merge<bf16>(out, (long)heads * lat, o_part, ml_part, nullptr, rows, heads, nsplit, lat, s);
 }
 
 // y [batch][M][N] = act(x [batch][M][K] w [batch][N][K]^T); row strides ldx / ldy, batch strides x_bs / w_bs / y_bs (elements)

@@ -20,7 +20,7 @@ constexpr int RT_MAXPL = 32;      // experts per lane (up to 1024 experts)
 __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float* __restrict__ wts,
                                                    const float* __restrict__ logits, const float* __restrict__ bias,
                                                    int n_exp, int top_k, int mode, int n_groups, int topk_groups,
-                                                   float scale, int ld, int shared_col, int shared_id) {
+                                                   float scale, int ld, int shared_col, int shared_id, int lane_groups) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x, lane = threadIdx.x;
@@ -48,7 +48,30 @@ __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float*
       sc[j] = e < n_exp ? sigmoidf_(sc[j]) : 0.f;
       sel[j] = e < n_exp ? sc[j] + (bias ? bias[e] : 0.f) : -INFINITY;
     }
-    if (n_groups > 1 && topk_groups < n_groups) {
+    if (n_groups > 1 && topk_groups < n_groups && !lane_groups) {
+      // groups that do not fall on a power of two of whole lanes: every lane scores its groups out of shared memory
+      extern __shared__ float rt_s[];                // [n_exp] scores, [n_groups] group scores
+      float* gs = rt_s + n_exp;
+      const int size = n_exp / n_groups;
+      for (int j = 0; j < per; ++j)
+        if (lane * per + j < n_exp) rt_s[lane * per + j] = sel[j];
+      __syncwarp();
+      for (int g = lane; g < n_groups; g += 32) {
+        float b1 = -INFINITY, b2 = -INFINITY;
+        for (int i = 0; i < size; ++i) { const float v = rt_s[g * size + i]; if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v; }
+        gs[g] = size > 1 ? b1 + b2 : b1;
+      }
+      __syncwarp();
+      for (int j = 0; j < per; ++j) {
+        const int e = lane * per + j;
+        if (e >= n_exp) continue;
+        const int g = e / size;
+        int better = 0;
+        for (int og = 0; og < n_groups; ++og)
+          if (gs[og] > gs[g] || (gs[og] == gs[g] && og < g)) ++better;
+        if (better >= topk_groups) sel[j] = -INFINITY;
+      }
+    } else if (n_groups > 1 && topk_groups < n_groups) {
       // a group spans gl = (experts per group) / (experts per lane) lanes; its score is the sum of its two best
       // biased scores
       const int gl = (n_exp / n_groups) / per;
@@ -198,6 +221,33 @@ moe_down_kernel(float* __restrict__ yp, const __nv_bfloat16* __restrict__ act, c
   }
 }
 
+// The same in 32 bits, one warp per output: GU: out[p][j] = silu(W[e][j] . x[t]) * (W[e][N + j] . x[t]), else out[p][j] = W[e][j] . x[p]
+template <bool GU>
+__global__ void __launch_bounds__(256) expert_f32_kernel(float* __restrict__ out, const float* __restrict__ x, const float* __restrict__ w,
+                                                         const int* __restrict__ ids, int p0, int top_k, int K, int N, int n_exp) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int p = p0 + blockIdx.y, e = ids[p], lane = threadIdx.x & 31;
+  const int j = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (j >= N) return;
+  float a = 0.f, b = 0.f;
+  if (e >= 0 && e < n_exp) {
+    const float* xr = x + (size_t)(GU ? p / top_k : p) * K;
+    const float* w0 = w + ((size_t)e * (GU ? 2 : 1) * N + j) * K;
+    for (int k = lane * 4; k < K; k += 128) {
+      const float4 xv = *reinterpret_cast<const float4*>(xr + k), v = *reinterpret_cast<const float4*>(w0 + k);
+      a = fmaf(xv.x, v.x, fmaf(xv.y, v.y, fmaf(xv.z, v.z, fmaf(xv.w, v.w, a))));
+      if (GU) {
+        const float4 u = *reinterpret_cast<const float4*>(w0 + (size_t)N * K + k);
+        b = fmaf(xv.x, u.x, fmaf(xv.y, u.y, fmaf(xv.z, u.z, fmaf(xv.w, u.w, b))));
+      }
+    }
+  }
+  a = warp_sum(a);
+  if (GU) b = warp_sum(b);
+  if (lane == 0) out[(size_t)p * N + j] = GU ? a / (1.f + expf(-a)) * b : a;
+}
+
 // out[t] = (res[t]) + sum_k wts[t][k] * yp[t*K + k]  (pick order) + shared[t] * gate[t]; fp32 or bf16 out
 __global__ void moe_combine_kernel(void* __restrict__ out, const float* __restrict__ yp, const float* __restrict__ wts,
                                    const __nv_bfloat16* __restrict__ shared, const float* __restrict__ shared_gate,
@@ -225,15 +275,31 @@ extern "C" int fb_moe_route(int* ids, float* wts, const float* logits, const flo
   if (rows <= 0) return 0;
   if (ld < n_exp || shared_col >= ld) return -1;
   if (n_exp > 32 * RT_MAXPL || top_k > 32 || top_k > n_exp) return -1;
+  int lane_groups = 1;
   if (mode == 1 && n_groups > 1) {
-    // a group must cover a power-of-two number of whole lanes
-    const int per = (n_exp + 31) / 32;
-    if (n_exp % n_groups || (n_exp / n_groups) % per) return -2;
-    const int gl = (n_exp / n_groups) / per;
-    if (gl < 1 || (gl & (gl - 1)) || n_groups * gl > 32) return -2;
+    if (n_exp % n_groups || topk_groups < 1 || top_k > (long)n_exp / n_groups * topk_groups) return -2;
+    // groups of several experts that cover a power-of-two number of whole lanes are scored with shuffles
+    const int per = (n_exp + 31) / 32, size = n_exp / n_groups, gl = size / per;
+    lane_groups = size > 1 && size % per == 0 && gl >= 1 && !(gl & (gl - 1)) && n_groups * gl <= 32;
   }
-  return (int)launch_pdl(route_kernel, dim3(rows), dim3(32), 0, s, ids, wts, logits, bias, n_exp, top_k, mode,
-                         n_groups, topk_groups, scale, ld, shared_col, shared_id);
+  const size_t smem = lane_groups ? 0 : (size_t)(n_exp + n_groups) * 4;
+  return (int)launch_pdl(route_kernel, dim3(rows), dim3(32), smem, s, ids, wts, logits, bias, n_exp, top_k, mode,
+                         n_groups, topk_groups, scale, ld, shared_col, shared_id, lane_groups);
+}
+
+// The pair products in 32 bits: act and yp as fb_moe_gate_up / fb_moe_down leave them; ids outside [0, n_exp) give zero rows.
+extern "C" int fb_expert_rows_f32(float* yp, float* act, const float* x, const float* w_gu, const float* w_down, const int* ids, int pairs,
+                                  int top_k, int hidden, int inter, int n_exp, cudaStream_t s) {
+  if (pairs <= 0) return 0;
+  if (hidden % 4 || inter % 4) return -1;
+  for (int p0 = 0; p0 < pairs; p0 += 32768) {              // grid.y; a multiple of top_k is not needed: pairs are counted from 0
+    const int n = pairs - p0 < 32768 ? pairs - p0 : 32768;
+    int rc = (int)launch_pdl(expert_f32_kernel<true>, dim3((inter + 7) / 8, n), dim3(256), 0, s, act, x, w_gu, ids, p0, top_k, hidden, inter, n_exp);
+    if (!rc) rc = (int)launch_pdl(expert_f32_kernel<false>, dim3((hidden + 7) / 8, n), dim3(256), 0, s, yp, (const float*)act, w_down, ids, p0,
+                                  top_k, inter, hidden, n_exp);
+    if (rc) return rc;
+  }
+  return 0;
 }
 
 extern "C" int fb_moe_gate_up(void* act, const void* x, const void* w_gu, const int* ids, int pairs, int top_k,

@@ -168,7 +168,8 @@ __global__ void ep_signal_kernel(EpComm c) {
 
 // ---- 6. combine ------------------------------------------------------------------------------------------------
 // grid = local tokens; out[t] = res[t] + shared[t] * sigmoid(gate[t]) + sum_k wts[t][k] * result_row(t, k), pick order
-__global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16* __restrict__ out,
+// With `acc` the sum is added to its fp32 rows instead of being written to out.
+__global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16* __restrict__ out, float* __restrict__ acc32,
                                                          const int* __restrict__ ids, const float* __restrict__ wts,
                                                          const int* __restrict__ pos, const int* __restrict__ send_off,
                                                          const __nv_bfloat16* __restrict__ shared,
@@ -210,6 +211,13 @@ __global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16
 #pragma unroll
         for (int j = 0; j < 4; ++j) { acc[2 * j] += bf_lo(u[j]); acc[2 * j + 1] += bf_hi(u[j]); }
       }
+      if (acc32) {
+        float4* a = reinterpret_cast<float4*>(acc32 + (size_t)t * H + i * 8);
+        const float4 a0 = a[0], a1 = a[1];
+        a[0] = make_float4(a0.x + acc[0], a0.y + acc[1], a0.z + acc[2], a0.w + acc[3]);
+        a[1] = make_float4(a1.x + acc[4], a1.y + acc[5], a1.z + acc[6], a1.w + acc[7]);
+        continue;
+      }
       reinterpret_cast<uint4*>(out + (size_t)t * H)[i] =
           make_uint4(pack_bf2(acc[0], acc[1]), pack_bf2(acc[2], acc[3]), pack_bf2(acc[4], acc[5]), pack_bf2(acc[6], acc[7]));
     }
@@ -249,8 +257,9 @@ extern "C" long fb_ep_recv_offset(int n_experts, int hidden, long cap_rows) { re
 extern "C" long fb_ep_out_offset(int n_experts, int hidden, long cap_rows) { return ep_layout(n_experts, hidden, cap_rows).out_off; }
 
 // One expert-parallel MoE block over this rank's `rows` tokens. `act` is scratch [cap_rows][inter] bf16; `plan` is int
-// scratch of rows * top_k + 3 * n_experts + 8 entries. w_gu / w_down hold only the experts this rank owns.
-extern "C" int fb_ep_moe(void* out, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
+// scratch of rows * top_k + 3 * n_experts + 8 entries. w_gu / w_down hold only the experts this rank owns. out_f32: `out` holds
+// fp32 rows to which the experts' sum is added.
+extern "C" int fb_ep_moe(void* out, int out_f32, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
                          const void* shared, const float* shared_gate, const void* res, void* act, int* plan, int rows,
                          int top_k, int n_experts, int hidden, int inter, long cap_rows, const void* const* peers, int rank,
                          int world, uint32_t* ctr, int* status, unsigned spin_limit, int sm_count, cudaStream_t s) {
@@ -281,7 +290,7 @@ extern "C" int fb_ep_moe(void* out, const void* x, const int* ids, const float* 
                        hidden, inter, inter, hidden, 0, status, sm_count, s);
   if (rc) return rc;
   ep_signal_kernel<<<1, 32, 0, s>>>(c);
-  ep_combine_kernel<<<rows > 0 ? rows : 1, 256, 0, s>>>(c, (__nv_bfloat16*)out, ids, wts, pos, send_off,
+  ep_combine_kernel<<<rows > 0 ? rows : 1, 256, 0, s>>>(c, (__nv_bfloat16*)out, out_f32 ? (float*)out : nullptr, ids, wts, pos, send_off,
                                                         (const __nv_bfloat16*)shared, shared_gate,
                                                         (const __nv_bfloat16*)res, rows, top_k);
   return (int)cudaGetLastError();

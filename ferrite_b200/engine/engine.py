@@ -80,8 +80,10 @@ class Engine:
         if self.ecfg.weight_dtype in ("nvfp4", "nvfp4-a16", "nvfp4-w4a4"):
             from ..ops.qweight import quantize_experts, quantize_weight
             big = ("in_proj", "out_proj", "gate_up", "up", "down", "lm_head")
+            # routed layers of listed models stay in 16 bits where a router's logits come out of the product, and in their experts
+            routed = {f"l{i}.{n}" for i, l in enumerate(cfg.layers) if l.experts for n in ("in_proj", "experts_gate_up", "experts_down")}
             for k in list(weights.keys()):
-                if not is_t(weights[k]):
+                if not is_t(weights[k]) or k in routed:
                     continue
                 if k.split(".")[-1] in big and weights[k].dim() == 2 and weights[k].shape[1] % 32 == 0:
                     weights[k] = quantize_weight(weights[k], "nvfp4", keep_dense=True, dense_dtype=self.dtype)
@@ -155,6 +157,13 @@ class Engine:
             from ..parallel.ep import ExpertParallel
             self.ex.ep = ExpertParallel(tp if world > 1 else None, self.device, cfg.n_experts, cfg.hidden,
                                         cap_rows=self.ecfg.max_step_rows * cfg.top_k)
+        if on_gpu and self.dtype == torch.bfloat16:
+            # prompt-sized steps of routed layers of listed models: the same kernels, one set of buffers per number of experts
+            from ..parallel.ep import ExpertParallel
+            for n in sorted({l.experts for l in cfg.layers if l.experts}):
+                top = max(l.top for l in cfg.layers if l.experts == n)
+                self.ex.ep_listed[n] = ExpertParallel(None, self.device, n, weights["embed"].shape[1], cap_rows=max(256, self.ecfg.max_step_rows * top),
+                                                          status=ops.status_word)
         self.slot_len: List[int] = [0] * self.ecfg.n_slots
         if self.ex.heat:
             import atexit

@@ -247,15 +247,17 @@ class Executor:
         # `crates/fe-dsc/src/engine.rs:2251-2315`).
         self.heat_path = os.environ.get("FE_EXPERT_HEAT", "")
         self.heat: Dict[int, torch.Tensor] = {}
-        if self.heat_path and cfg.n_experts > 0:
+        if self.heat_path:
             for i in range(cfg.n_layers):
-                if cfg.is_moe(i):
-                    self.heat[i] = torch.zeros((full_cfg or cfg).n_experts + 1, dtype=torch.int64, device=self.device)
+                n_exp = cfg.layers[i].experts if cfg.layers else (full_cfg or cfg).n_experts if cfg.is_moe(i) else 0
+                if n_exp:
+                    self.heat[i] = torch.zeros(n_exp + 1, dtype=torch.int64, device=self.device)
         self.moe_merged: Dict[int, torch.Tensor] = {}
         self._merge_shared_experts()
         self._step_max_kvlen = None
         self._step_segments = None            # host view of an eager step's segments: (slot, pos0, rows)
         self.ep = None                        # ExpertParallel, set by the engine for MoE models under TP
+        self.ep_listed: Dict[int, object] = {}   # ... of models of listed layers, by their layers' number of experts
 
     def _count_experts(self, i: int, ids) -> None:
         h = self.heat.get(i)
@@ -621,16 +623,53 @@ class Executor:
         return self._sum_ranks(o, w[p + "out_proj"])
 
     def _mix_gqa(self, h, run, mv, groups, nsplit):
-        """Grouped-query attention over operand rows h: prompt segments on the flash kernel, the others split over the keys."""
+        """Grouped-query attention over operand rows h."""
+        p, d = f"l{run.layer}.", self.run_dims[run.index]
+        proj = self.ops.linear(h, self.w[p + "in_proj"], out_f32=True)
+        o = torch.empty(h.shape[0], d.heads, d.hp, dtype=self.dtype, device=self.device)
+        self._gqa_rows(proj, run, mv, groups, nsplit, o)
+        return self._sum_ranks(o.view(o.shape[0], -1), self.w[p + "out_proj"])
+
+    def _gqa_rows(self, proj, run, mv, groups, nsplit, o):
+        """From the fused projection to the heads' outputs o [T, heads, hp] (rows may lie apart): prompt segments on the flash kernel, the
+        others split over the keys."""
         w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{run.layer}.", self.run_dims[run.index]
         kc, vc = self.k_cache[run.index], self.v_cache[run.index]
-        proj = ops.linear(h, w[p + "in_proj"], out_f32=True)
-        q = ops.gqa_prep(proj, d, w.get(p + "in_bias"), w[p + "inv_freq"], mv["slot"], mv["pos"], self.block_table, kc, vc, kvb, self.cfg.eps)
-        o = torch.empty_like(q)
+        norms = {"norms": (w[p + "q_norm"], w[p + "k_norm"])} if d.row_norm else {}
+        q = ops.gqa_prep(proj, d, w.get(p + "in_bias"), w[p + "inv_freq"], mv["slot"], mv["pos"], self.block_table, kc, vc, kvb, self.cfg.eps,
+                         **norms)
+        mix = {}
+        if d.maps == 2 or d.gate_off >= 0:
+            mix = dict(lam=w.get(p + "lam"), eps=self.cfg.eps, gate=proj[:, d.gate_off:d.gate_off + d.heads * d.vw] if d.gate_off >= 0 else None)
         for g in groups:
             segs = tuple(mv[k][g.seg_lo:g.seg_hi] for k in ("sslot", "srow0", "snrows", "spos0"))
-            ops.gqa_attention(q, d, kc, vc, w.get(p + "sink"), g, mv["slot"], mv["kvlen"], segs, self.block_table, kvb, nsplit, o)
-        return self._sum_ranks(o.view(o.shape[0], -1), w[p + "out_proj"])
+            ops.gqa_attention(q, d, kc, vc, w.get(p + "sink"), g, mv["slot"], mv["kvlen"], segs, self.block_table, kvb, nsplit, o, **mix)
+
+    def _parallel_block(self, x, h, run, mv, groups, nsplit, next_w, next_b):
+        """x <- x + (mixer(h) + ff(h)): the projections of the mixer, its output gates and the router are one product of h; with a dense
+        feed-forward the two output projections are one as well, over [heads | activation]. The pass that adds the sums (and the rows of
+        the chosen experts) makes the operand of the next run, which it returns."""
+        c, w, ops, p, l, d = self.cfg, self.w, self.ops, f"l{run.layer}.", self.cfg.layers[run.layer], self.run_dims[run.index]
+        T, Ko, out_proj = h.shape[0], d.heads * d.hp, w[p + "out_proj"]
+        proj = ops.linear(h, w[p + "in_proj"], out_f32=True)
+        both = ops.empty(T, out_proj.shape[1], dtype=self.dtype, device=self.device) if ops.name == "cuda" else torch.empty(T, out_proj.shape[1])
+        self._gqa_rows(proj, run, mv, groups, nsplit, both[:, :Ko].unflatten(1, (d.heads, d.hp)))
+        if l.ff and not l.experts:
+            gu = w[p + "gate_up"]
+            if isinstance(gu, torch.Tensor):
+                ops.linear(h, gu, swiglu=True, out=both[:, Ko:])
+            else:                                                     # packed weights: their kernels write dense rows
+                both[:, Ko:] = ops.linear(h, gu, swiglu=True)
+        y, pairs = ops.linear(both, out_proj, out_f32=True), None
+        if l.experts:
+            ids, wts = ops.moe_route(proj[:, d.router_off:d.router_off + l.experts], None, 1, l.top, l.groups, l.keep_groups, l.route_scale)
+            self._count_experts(run.layer, ids)
+            gu, dn, ep = w[p + "experts_gate_up"], w[p + "experts_down"], self.ep_listed.get(l.experts)
+            if ep is not None and T > ops.moe_pair_rows:
+                ep.moe(ops, h, ids, wts, gu, dn, acc=y)
+            else:
+                pairs = (ops.expert_rows(h, ids, gu, dn), wts)
+        return ops.add_layer_norm(x, y, c.hidden, c.eps, next_w, next_b, pairs)
 
     def _mix_cdelta(self, h, run, mv, groups, commit):
         """Delta rule with a decay per channel over operand rows h; verify rows keep their projections for the replay."""
@@ -647,8 +686,8 @@ class Executor:
                                mv["sslot"], mv["srow0"], mv["snrows"], self.cfg.eps, commit)
 
     def _layers_listed(self, x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit):
-        """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), with `pre_norm` also a norm ahead of the mixer and the feed-forward: x is
-        the 32-bit residual stream (updated in place), xb its copy in the GEMM operand type. The pass over the rows that adds a
+        """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), with `pre_norm` also a norm ahead of the mixer and the feed-forward; or
+        `parallel` blocks. x is the 32-bit residual stream (updated in place), xb its copy in the GEMM operand type. The pass over the rows that adds a
         sublayer's output also makes the operand of whatever comes next. `loop_rows` [T, 2 width]: operand of the product that opens
         a pass of the loop, the embedding output in its right half. Returns the last copy of x."""
         c, w, ops = self.cfg, self.w, self.ops
@@ -662,35 +701,39 @@ class Executor:
 
         def after(j):
             """Operand that run j starts from: (weight of a norm, buffer)."""
-            if j < len(self.runs) and self.runs[j].enter is not None:
+            if j < len(self.runs) and self.runs[j].enter is not None and c.loop_input:
                 return None, loop_rows[:, :W]
             return (w[f"l{self.runs[j].layer}.pre_norm"] if c.pre_norm and j < len(self.runs) else None), None
 
         for run in self.runs:
             i, l = run.layer, c.layers[run.layer]
             p = f"l{i}."
-            if run.enter is not None:
+            if run.enter is not None and c.loop_input:
                 y = ops.linear(loop_rows, w["loop_in"], out_f32=True)
                 xb = ops.add_normed(x, y, None, c.hidden, c.eps, bias=w["loop_step"][run.enter], next_w=w.get(p + "pre_norm"))
             elif run.index == 0 and c.pre_norm:
-                xb = ops.norm_rows(x, None, w[p + "pre_norm"], c.hidden, c.eps)
-            if l.mixer == "latent":
-                y = self._mix_latent(xb, run, mv, groups, nsplit, gathered)
-            elif l.mixer == "gqa":
-                y = self._mix_gqa(xb, run, mv, groups, nsplit)
+                xb = ops.norm_rows(x, None, w[p + "pre_norm"], c.hidden, c.eps, **({"bias": w[p + "pre_norm_bias"]} if c.parallel else {}))
+            if c.parallel:
+                q = f"l{self.runs[run.index + 1].layer}." if run.index + 1 < len(self.runs) else "none."
+                xb = self._parallel_block(x, xb, run, mv, groups, nsplit, w.get(q + "pre_norm"), w.get(q + "pre_norm_bias"))
             else:
-                y = self._mix_cdelta(xb, run, mv, groups, commit)
-            nxt, buf = (w.get(p + "ffn_pre_norm"), None) if l.ff else after(run.index + 1)
-            xb = ops.add_normed(x, y, w[p + "mix_norm"], c.hidden, c.eps, bias=w.get(p + "out_bias"), next_w=nxt, out=buf)
-            if l.ff:
-                act = ops.linear(xb, w[p + "gate_up"], swiglu=True) if l.act == "swiglu" else ops.linear(xb, w[p + "up"], act=l.act)
-                nxt, buf = after(run.index + 1)
-                xb = ops.add_normed(x, self._sum_ranks(act, w[p + "down"]), w[p + "ffn_norm"], c.hidden, c.eps, next_w=nxt, out=buf)
+                if l.mixer == "latent":
+                    y = self._mix_latent(xb, run, mv, groups, nsplit, gathered)
+                elif l.mixer == "gqa":
+                    y = self._mix_gqa(xb, run, mv, groups, nsplit)
+                else:
+                    y = self._mix_cdelta(xb, run, mv, groups, commit)
+                nxt, buf = (w.get(p + "ffn_pre_norm"), None) if l.ff else after(run.index + 1)
+                xb = ops.add_normed(x, y, w[p + "mix_norm"], c.hidden, c.eps, bias=w.get(p + "out_bias"), next_w=nxt, out=buf)
+                if l.ff:
+                    act = ops.linear(xb, w[p + "gate_up"], swiglu=True) if l.act == "swiglu" else ops.linear(xb, w[p + "up"], act=l.act)
+                    nxt, buf = after(run.index + 1)
+                    xb = ops.add_normed(x, self._sum_ranks(act, w[p + "down"]), w[p + "ffn_norm"], c.hidden, c.eps, next_w=nxt, out=buf)
             if i in c.tap_layers and run.index == last_run[i]:
                 self.taps.append(x[:, :c.hidden].to(self.dtype, copy=True) if c.pre_norm or xb is x else xb[:, :c.hidden])
             if self.dump_layers:
                 self._dump_layer(i, x[:, :c.hidden], False, T)
-        return xb
+        return x if xb is None else xb
 
     def _layers(self, x, mv, T, nseg, max_seg_rows, nsplit, commit, tv=None):
         c, w, ops = self.cfg, self.w, self.ops
@@ -866,8 +909,8 @@ class Executor:
         c, w, ops = self.cfg, self.w, self.ops
         if nlog == 0:
             return None, None
-        if c.out_norm:
-            rows = ops.norm_rows(x, mv["lrow"], w["final_norm"], c.hidden, c.eps)
+        if c.layers:
+            rows = ops.norm_rows(x, mv["lrow"], w["final_norm"], c.hidden, c.eps, **({"bias": w["final_norm_bias"]} if c.parallel else {}))
             logits = ops.linear(rows, w["lm_head"], out_f32=True)
             if c.logit_softcap:
                 logits = ops.softcap(logits, c.logit_softcap)
@@ -892,13 +935,13 @@ class Executor:
     def _run(self, T, nseg, nlog, max_seg_rows, nsplit, commit, greedy, x_add=None, tree=False):
         mv = self._meta_views(T, nseg, nlog)
         self._last_meta = (mv, max_seg_rows)
-        if self.cfg.out_norm:
+        if self.cfg.layers:
             c, w = self.cfg, self.w
             assert x_add is None and not tree, "models of listed layers: no injected rows, no verify trees"
-            loop_rows = torch.empty(T, 2 * w["embed"].shape[1], dtype=self.dtype, device=self.device) if c.loop else None
+            loop_rows = torch.empty(T, 2 * w["embed"].shape[1], dtype=self.dtype, device=self.device) if c.loop and c.loop_input else None
             x, xb = self.ops.embed_grams(w["embed"], w.get("bigram"), mv["tok"], mv["slot"], mv["pos"], self.block_table,
                                          self.tok_pages, self.ecfg.kv_block, c.embed_scale, c.gram_buckets, c.gram_mul_prev,
-                                         c.gram_mul_cur, **({"out": loop_rows} if c.loop else {}))
+                                         c.gram_mul_cur, **({"out": loop_rows} if loop_rows is not None else {}))
             self.last_hidden = self._layers_listed(x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit)[:, :c.hidden]
             return self._head(x, mv, nlog, greedy)
         x = self.ops.embed(self.w["embed"], mv["tok"])

@@ -52,7 +52,7 @@ def _take(w, index: torch.Tensor):
     raise TypeError(f"{type(w).__name__} rows cannot be regrouped")
 
 
-_LISTED_TOP = {"embed": "embed", "bigram": "bigram", "final_norm": "final.norm", "lm_head": "head", "loop_in": "loop.in",
+_LISTED_TOP = {"embed": "embed", "bigram": "bigram", "final_norm": "final.norm", "final_norm_bias": "final.norm.b", "lm_head": "head", "loop_in": "loop.in",
                "loop_step": "loop.step"}
 _LISTED_SUB = {
     "zototar": {"mix_norm": "norm1", "ffn_norm": "norm2", "q_a": "mix.dq", "q_a_norm": "mix.dq.norm", "q_b": "mix.uq", "kv_a": "mix.dkv",
@@ -61,27 +61,40 @@ _LISTED_SUB = {
                 "out_bias": "mix.o.b", "gnorm_w": "mix.norm", "gate": "mlp.gate", "up": "mlp.up", "down": "mlp.down",
                 **{n: f"mix.{n}" for n in ("q", "k", "v", "b", "sink", "A_log", "dt_bias", "a1", "a2", "g1", "g2")},
                 **{n + "_bias": f"mix.{n}.b" for n in "qk"}, **{n + "_conv": f"mix.{n}.conv" for n in "qkv"}},
+    # experts are stored one by one: {} is the expert's number; several names are joined by rows
+    "rakizen": {"pre_norm": "norm1", "pre_norm_bias": "norm1.b", "out_proj": "mix.o", "q_norm": "mix.q.norm", "k_norm": "mix.k.norm",
+                **{n: f"mix.{n}" for n in ("q", "k", "v", "g", "lq1", "lk1", "lq2", "lk2")},
+                **{n: f"mlp.{n}" for n in ("gate", "up", "down", "router")}, "experts_gate_up": ("mlp.e{}.gate", "mlp.e{}.up"),
+                "experts_down": ("mlp.e{}.down",)},
 }
 
 
 def _load_listed(st: SafeTensors, cfg: ModelConfig, dtype) -> Dict[str, torch.Tensor]:
     """A checkpoint of a model of listed layers under engine names; every tensor's shape is checked against the configuration.
     Widths that only the tensors tell (the low ranks of channel-delta layers) are filled into it."""
-    sub = _LISTED_SUB["zototar" if any(l.mixer == "latent" for l in cfg.layers) else "dofunex"]
+    sub = _LISTED_SUB["rakizen" if cfg.parallel else "zototar" if any(l.mixer == "latent" for l in cfg.layers) else "dofunex"]
     for i, l in enumerate(cfg.layers):
         if l.mixer == "cdelta":
             for field, base in (("decay_rank", "a1"), ("gate_rank", "g1")):
                 if not getattr(l, field) and st.has(f"l{i}.{sub[base]}"):
                     setattr(l, field, int(st.get(f"l{i}.{sub[base]}").shape[0]))
     w: Dict[str, torch.Tensor] = {}
-    for name, shape in weight_shapes(cfg).items():
-        layer, _, base = name.rpartition(".")
-        src = f"{layer}.{sub[base]}" if layer else _LISTED_TOP[base]
+
+    def read(src, shape):
         if not st.has(src):
             raise KeyError(f"{src} is missing from the checkpoint")
         t = st.get(src)
         if tuple(t.shape) != tuple(shape):
             raise ValueError(f"{src}: shape {tuple(t.shape)}, the configuration says {tuple(shape)}")
+        return t
+    for name, shape in weight_shapes(cfg).items():
+        layer, _, base = name.rpartition(".")
+        src = sub[base] if layer else _LISTED_TOP[base]
+        if isinstance(src, tuple):                                    # a stack of experts
+            one = (shape[1] // len(src), *shape[2:])
+            t = torch.stack([torch.cat([read(f"{layer}.{s.format(e)}", one) for s in src]) for e in range(shape[0])])
+        else:
+            t = read(f"{layer}.{src}" if layer else src, shape)
         w[name] = t.float() if keeps_f32(cfg, name) else t.to(dtype)
     return w
 

@@ -28,7 +28,10 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
     """A layer of a model that lists its layers (`LayerSpec`): norms on the sublayers' outputs and, with `pre_norm`, inputs."""
     l, h, p = cfg.layers[i], cfg.hidden, f"l{i}."
     out: Dict[str, tuple] = {p + "pre_norm": (h,)} if cfg.pre_norm else {}
-    out[p + "mix_norm"] = (h,)
+    if cfg.parallel:
+        out[p + "pre_norm_bias"] = (h,)
+    else:
+        out[p + "mix_norm"] = (h,)
     if l.mixer == "latent":
         out.update({p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,), p + "q_b": (l.heads * l.dim, l.q_rank)})
         if l.kv_from is None:
@@ -38,12 +41,19 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
         out[p + "v_b"] = (l.heads * l.vdim, l.kv_rank)
         out[p + "out_proj"] = (h, l.heads * l.vdim)
     elif l.mixer == "gqa":
-        for n, heads, d in (("q", l.heads, l.dim), ("k", l.kv_heads, l.dim)) + (() if l.key_values else (("v", l.kv_heads, l.vdim),)):
+        kd = l.maps * l.dim
+        for n, heads, d in (("q", l.heads, kd), ("k", l.kv_heads, kd)) + (() if l.key_values else (("v", l.kv_heads, l.vdim),)):
             out[p + n] = (heads * d, h)
             if l.bias:
                 out[p + n + "_bias"] = (heads * d,)
         if l.sink:
             out[p + "sink"] = (l.heads,)
+        if l.row_norm:
+            out.update({p + "q_norm": (l.heads * kd,), p + "k_norm": (l.kv_heads * kd,)})
+        if l.maps == 2:
+            out.update({p + n: (l.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        if l.out_gate:
+            out[p + "g"] = (l.heads * l.vdim, h)
         out[p + "out_proj"] = (h, l.heads * l.vdim)
         if l.bias:
             out[p + "out_bias"] = (h,)
@@ -55,10 +65,13 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
         out.update({p + "b": (l.heads, h), p + "A_log": (l.heads,), p + "dt_bias": (l.heads * l.dim,), p + "gnorm_w": (l.vdim,),
                     p + "a1": (l.decay_rank, h), p + "a2": (l.heads * l.dim, l.decay_rank), p + "g1": (l.gate_rank, h),
                     p + "g2": (nv, l.gate_rank), p + "out_proj": (h, nv)})
-    if l.ff:
-        if cfg.pre_norm:
-            out[p + "ffn_pre_norm"] = (h,)
-        out[p + "ffn_norm"] = (h,)
+    if l.experts:
+        out.update({p + "router": (l.experts, h), p + "experts_gate_up": (l.experts, 2 * l.ff, h), p + "experts_down": (l.experts, h, l.ff)})
+    elif l.ff:
+        if not cfg.parallel:
+            if cfg.pre_norm:
+                out[p + "ffn_pre_norm"] = (h,)
+            out[p + "ffn_norm"] = (h,)
         if l.act == "swiglu":
             out[p + "gate"] = (l.ff, h)
         out.update({p + "up": (l.ff, h), p + "down": (h, l.ff)})
@@ -117,7 +130,9 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
         out["lm_head"] = (cfg.vocab, cfg.hidden)
     if cfg.gram_buckets:
         out["bigram"] = (cfg.gram_buckets + 1, cfg.hidden)
-    if cfg.loop:
+    if cfg.parallel:
+        out["final_norm_bias"] = (cfg.hidden,)
+    if cfg.loop and cfg.loop_input:
         out["loop_in"] = (cfg.hidden, 2 * cfg.hidden)
         out["loop_step"] = (cfg.loop[2], cfg.hidden)
     for i in range(cfg.n_layers):
@@ -126,12 +141,12 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
 
 
 _F32_NAMES = ("A_log", "dt_bias", "router_bias")
-_F32_LISTED = ("norm", "gnorm_w", "_bias", "sink", "_conv", "loop_step")     # ... of models of listed layers
+_F32_LISTED = ("norm", "gnorm_w", "_bias", "sink", "_conv", "loop_step", "lq1", "lk1", "lq2", "lk2")     # ... of models of listed layers
 
 
 def keeps_f32(cfg: ModelConfig, name: str) -> bool:
     """Small tensors that enter 32-bit arithmetic and stay in 32 bits whatever the engine computes in."""
-    return name.endswith(_F32_NAMES) or (cfg.out_norm and name.endswith(_F32_LISTED))
+    return name.endswith(_F32_NAMES) or (bool(cfg.layers) and name.endswith(_F32_LISTED))
 
 
 def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="cpu", std: float = 0.02, post=None) -> Weights:
@@ -144,9 +159,9 @@ def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="c
     w: Weights = {}
     for name, shape in weight_shapes(cfg).items():
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32) * std
-        if name.endswith("gnorm_w") or (cfg.out_norm and name.endswith("norm")):
+        if name.endswith("gnorm_w") or (cfg.layers and name.endswith("norm")):
             t = t + 1.0
-        if cfg.out_norm and name.endswith("_conv"):
+        if cfg.layers and name.endswith("_conv"):
             t = t / std * shape[1] ** -0.5
         t = t if keeps_f32(cfg, name) else t.to(dtype)
         w[name] = post(name, t) if post is not None else t
@@ -303,7 +318,9 @@ def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
 @dataclass(frozen=True)
 class GqaDims:
     """Sizes of one grouped-query attention layer as its kernels see them. Cache rows and attention operands have heads of `hp`
-    columns, zeros beyond `dim`: 64 / 128 / 256 are what the tensor-core kernels take, wider heads run on the CUDA cores."""
+    columns, zeros beyond the true widths: 64 / 128 / 256 are what the tensor-core kernels take, wider heads run on the CUDA cores.
+    With two maps a cached key row holds both maps' keys side by side and every head brings two queries, each with zeros in the other
+    map's columns: differential attention is grouped-query attention over `maps * heads` queries, and values are read once for both."""
 
     heads: int
     kv_heads: int
@@ -313,6 +330,37 @@ class GqaDims:
     rot_dims: int
     v_off: int        # column of the projection where the values start (the keys' column when they are the values)
     qk_norm: bool
+    vdim: int = 0     # value width, 0 = dim
+    maps: int = 1
+    row_norm: bool = False
+    softcap: float = 0.0
+    window: int = 0
+    chunk: int = 0
+    diff: float = 0.0
+    gate_off: int = -1      # column of the projection where the output gates start, -1 = none
+    router_off: int = -1    # ... and the router's logits
+
+    @property
+    def vw(self) -> int:
+        return self.vdim or self.dim
+
+    @property
+    def queries(self) -> int:
+        """Query heads of the attention kernels."""
+        return self.maps * self.heads
+
+    @property
+    def plain(self) -> bool:
+        """No mechanism beyond what a causal grouped-query attention over one key and value width has."""
+        return self.maps == 1 and not self.row_norm and self.vw == self.dim
+
+    @property
+    def reach(self) -> int:
+        """Keys that a row can see, 0 = all."""
+        return self.window or self.chunk
+
+    def first_visible(self, pos: int) -> int:
+        return max(0, pos - self.window + 1) if self.window else pos - pos % self.chunk if self.chunk else 0
 
 
 def head_width(d: int) -> int:
@@ -321,9 +369,13 @@ def head_width(d: int) -> int:
 
 def gqa_dims(cfg: ModelConfig, i: int) -> GqaDims:
     l = cfg.layers[i]
-    assert l.dim == l.vdim, "keys and values of one width"
-    return GqaDims(l.heads, l.kv_heads, l.dim, head_width(l.dim), l.scale, l.rot_dims,
-                   (l.heads + (0 if l.key_values else l.kv_heads)) * l.dim, l.qk_norm)
+    kd = l.maps * l.dim
+    assert l.dim == l.vdim or not l.key_values, "values that are the keys have their width"
+    v_off = (l.heads + (0 if l.key_values else l.kv_heads)) * kd
+    g_off = v_off + l.kv_heads * l.vdim
+    r_off = g_off + (l.heads * l.vdim if l.out_gate else 0)
+    return GqaDims(l.heads, l.kv_heads, l.dim, head_width(max(kd, l.vdim)), l.scale, l.rot_dims, v_off, l.qk_norm, l.vdim, l.maps,
+                   l.row_norm, l.softcap, l.window, l.chunk, l.diff, g_off if l.out_gate else -1, r_off if l.experts else -1)
 
 
 def rope_frequencies(l) -> torch.Tensor:
@@ -401,18 +453,27 @@ def _pack_latent(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> 
 
 
 def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
-    """* in_proj  rows = [q | k (| v)] of all heads at their true width; in_bias the same
-    * out_proj [width, heads * hp]"""
+    """* in_proj  rows = [q | k (| v) (| output gates) (| router)] of all heads at their true width; in_bias the same
+    * out_proj [width, heads * hp]; in a parallel block with a dense feed-forward [width, heads * hp + ff]: both sublayers end in one
+      product over their joined operands
+    * lam      [1] weight of the second map"""
     l, p, d = cfg.layers[i], f"l{i}.", gqa_dims(cfg, i)
     names = ("q", "k") if l.key_values else ("q", "k", "v")
-    rows = torch.cat([w[p + n] for n in names])
+    rows = torch.cat([w[p + n] for n in names] + ([w[p + "g"]] if l.out_gate else []) + ([w[p + "router"]] if l.experts else []))
     out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     if l.bias:
         out[p + "in_bias"] = _pad(torch.cat([w[p + n + "_bias"].float() for n in names]), round_up(rows.shape[0], 8))
         out[p + "out_bias"] = _pad(w[p + "out_bias"].float(), W)
     if l.sink:
         out[p + "sink"] = w[p + "sink"].float().contiguous()
+    if l.row_norm:
+        out[p + "q_norm"], out[p + "k_norm"] = w[p + "q_norm"].float().contiguous(), w[p + "k_norm"].float().contiguous()
+    if l.maps == 2:
+        dot = lambda a, b: torch.exp((w[p + a].float() * w[p + b].float()).sum())
+        out[p + "lam"] = (dot("lq1", "lk1") - dot("lq2", "lk2") + l.diff).view(1)
     out[p + "out_proj"] = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp).view(W, -1)
+    if cfg.parallel and l.ff and not l.experts:
+        out[p + "out_proj"] = torch.cat([out[p + "out_proj"], _pad(w[p + "down"], W, round_up(l.ff, 64))], 1)
     out[p + "inv_freq"] = rope_frequencies(l).to(rows.device)
 
 
@@ -444,15 +505,27 @@ def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
                     "final_norm": vec("final_norm", cfg.logit_scale)}
     if cfg.gram_buckets:
         out["bigram"] = _pad(w["bigram"], cfg.gram_buckets + 1, W)
-    if cfg.loop:
+    if cfg.parallel:
+        out["final_norm_bias"] = vec("final_norm_bias")
+    if cfg.loop and cfg.loop_input:
         out["loop_in"] = _pad(w["loop_in"].view(cfg.hidden, 2, cfg.hidden), W, 2, W).view(W, 2 * W)
         out["loop_step"] = _pad(w["loop_step"].float(), cfg.loop[2], W)
     for i, l in enumerate(cfg.layers):
         p = f"l{i}."
         _PACK[l.mixer](cfg, w, i, W, out)
-        out[p + "mix_norm"] = vec(p + "mix_norm", cfg.residual_mult)
         if cfg.pre_norm:
             out[p + "pre_norm"] = vec(p + "pre_norm")
+        if cfg.parallel:
+            out[p + "pre_norm_bias"] = vec(p + "pre_norm_bias")
+            if l.experts:
+                F = round_up(l.ff, 64)
+                gu = _pad(w[p + "experts_gate_up"].view(l.experts, 2, l.ff, cfg.hidden), l.experts, 2, F, W)
+                out[p + "experts_gate_up"] = gu.view(l.experts, 2 * F, W)
+                out[p + "experts_down"] = _pad(w[p + "experts_down"], l.experts, W, F)
+            elif l.ff:
+                out[p + "gate_up"] = torch.cat([_pad(w[p + n], round_up(l.ff, 64), W) for n in ("gate", "up")])
+            continue
+        out[p + "mix_norm"] = vec(p + "mix_norm", cfg.residual_mult)
         if l.ff:
             F = round_up(l.ff, 64)
             up = _pad(w[p + "up"], F, W)

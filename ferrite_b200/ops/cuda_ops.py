@@ -167,8 +167,7 @@ class CudaOps(CudaLatent, CudaMixers, CudaExtras):
         """`act`: activation of the epilogue ("relu2": squared relu), not together with SwiGLU."""
         if self.dtype == torch.float32:
             assert norm_w is None and res is None, "fp32 linears have an activation epilogue only"
-            y = self.linear_f32(x, w, act, out)
-            return self.silu_mul_f32(y) if swiglu else y
+            return self.silu_mul_f32(self.linear_f32(x, w), out) if swiglu else self.linear_f32(x, w, act, out)
         if act is not None and not isinstance(w, torch.Tensor):
             assert act == "relu2" and not swiglu and not out_f32
             return self.relu2(self.linear(x, w, norm_w=norm_w, eps=eps, res=res))      # packed weights: a pass of its own

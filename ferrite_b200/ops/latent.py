@@ -78,8 +78,25 @@ class TorchLatent:
             return out
         return h.to(self.dtype)
 
-    def norm_rows(self, x, idx, w, width, eps):
-        return self._rms(x if idx is None else x[idx.long()], w, width, eps).to(self.dtype)
+    def norm_rows(self, x, idx, w, width, eps, bias=None):
+        """rms(x) * w; with a bias the layer norm (x - mean) / deviation * w + bias."""
+        x = x if idx is None else x[idx.long()]
+        return (self._rms(x, w, width, eps) if bias is None else self._layer_norm(x, w, bias, width, eps)).to(self.dtype)
+
+    @staticmethod
+    def _layer_norm(x, w, b, width, eps):
+        d = x[..., :width] - x[..., :width].mean(-1, keepdim=True)
+        h = torch.zeros_like(x)
+        h[..., :width] = d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w[:width] + b[:width]
+        return h
+
+    def add_layer_norm(self, x, y, width, eps, next_w=None, next_b=None, pairs=None):
+        """x += y in place, with `pairs` = (rows [T * top, width], weights [T, top]) also the weighted sum of a token's rows. Returns the
+        next GEMM operand, the layer norm of x (None with next_w None)."""
+        x += y.float()
+        if pairs is not None:
+            x += (pairs[0].view(x.shape[0], -1, x.shape[1]).float() * pairs[1][:, :, None]).sum(1)
+        return None if next_w is None else self._layer_norm(x, next_w, next_b, width, eps).to(self.dtype)
 
     def latent_prep(self, proj, d, q_norm, kv_norm, row_slot, row_pos, block_table, cache, kv_block, eps):
         """Both latents of a token from the fused projection: returns the normalised query latent, writes the normalised key /
@@ -119,11 +136,17 @@ class CudaLatent:
         self.C.add_normed(x, xb, y, w, width, eps, bias, next_w)
         return x if xb is None else xb
 
-    def norm_rows(self, x, idx, w, width, eps):
+    def norm_rows(self, x, idx, w, width, eps, bias=None):
         out = self.empty(x.shape[0] if idx is None else idx.numel(), x.shape[1], dtype=self.dtype, device=self.device)
         self.launches += 1
-        self.C.norm_rows(out, x, idx, w, width, eps)
+        self.C.norm_rows(out, x, idx, w, bias, width, eps)
         return out
+
+    def add_layer_norm(self, x, y, width, eps, next_w=None, next_b=None, pairs=None):
+        xb = None if next_w is None else self.empty(*x.shape, dtype=self.dtype, device=self.device)
+        self.launches += 1
+        self.C.add_layer_norm(x, xb, y, *(pairs or (None, None)), next_w, next_b, width, eps)
+        return xb
 
     def latent_prep(self, proj, d, q_norm, kv_norm, row_slot, row_pos, block_table, cache, kv_block, eps):
         cq = self.empty(proj.shape[0], d.qr, dtype=self.dtype, device=self.device)
@@ -174,8 +197,8 @@ class CudaLatent:
         self.C.softcap(logits, cap)
         return logits
 
-    def silu_mul_f32(self, gu):
-        y = self.empty(gu.shape[0], gu.shape[1] // 2, dtype=torch.float32, device=self.device)
+    def silu_mul_f32(self, gu, out=None):
+        y = out if out is not None else self.empty(gu.shape[0], gu.shape[1] // 2, dtype=torch.float32, device=self.device)
         self.launches += 1
         self.C.silu_mul_f32(y, gu)
         return y

@@ -1,6 +1,7 @@
-"""Mixers of the models whose layers are listed one by one, beside latent attention (`ops/latent.py`): grouped-query attention with
-rotated and then normed queries and keys, values that may be the projected keys, and a sink ("gqa"), and the gated delta rule with
-one decay per key channel ("cdelta"). `TorchMixers` states each op in plain PyTorch for the fp32 CPU engine, `CudaMixers` runs the
+"""Mixers of the models whose layers are listed one by one, beside latent attention (`ops/latent.py`): grouped-query attention ("gqa")
+with rotated queries and keys, normed per head after the rotation or over the whole row before it, values that may be the projected
+keys, a sink, softcapped scores, sliding windows or chunks, one softmax map per head or the difference of two, gated outputs; and the
+gated delta rule with one decay per key channel ("cdelta"). Routed feed-forwards are here too. `TorchMixers` states each op in plain PyTorch for the fp32 CPU engine, `CudaMixers` runs the
 kernels of `csrc/gqa.cu`, `csrc/cdelta.cu` and `csrc/cdelta_chunk.cu` and the shared attention kernels; both have the same signatures
 and work on the same caches and states.
 
@@ -16,13 +17,17 @@ UNIT_EPS = 1e-6       # inside the root of the delta rule's unit queries and key
 
 
 class TorchMixers:
-    def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps):
-        """Biases, rotation and norm of a step's queries and keys; keys and values into their pages. Returns q [T, heads, hp]."""
-        T = proj.shape[0]
-        p = proj.float() if bias is None else proj.float() + bias
-        q = p[:, :d.heads * d.dim].reshape(T, d.heads, d.dim)
-        k = p[:, d.heads * d.dim:(d.heads + d.kv_heads) * d.dim].reshape(T, d.kv_heads, d.dim)
-        v = p[:, d.v_off:d.v_off + d.kv_heads * d.dim].reshape(T, d.kv_heads, d.dim)
+    def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps, norms=None):
+        """Biases, norms over whole rows (`norms`: their weights for q and k), rotation and norms per head of a step's queries and keys;
+        keys and values into their pages. Returns q [T, maps * heads, hp]."""
+        T, M = proj.shape[0], d.maps
+        p = proj.float() if bias is None else proj.float() + bias[:proj.shape[1]]
+        nq, nk = d.heads * M * d.dim, d.kv_heads * M * d.dim
+        q, k = p[:, :nq], p[:, nq:nq + nk]
+        if d.row_norm:
+            q, k = (x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w for x, w in zip((q, k), norms))
+        q, k = q.reshape(T, d.heads * M, d.dim), k.reshape(T, d.kv_heads * M, d.dim)
+        v = p[:, d.v_off:d.v_off + d.kv_heads * d.vw].reshape(T, d.kv_heads, d.vw)
         ang = row_pos.double()[:, None] * inv_freq[None, :]
         c, s = ang.cos().float()[:, None], ang.sin().float()[:, None]
 
@@ -30,24 +35,48 @@ class TorchMixers:
             a, b = x[..., 0:d.rot_dims:2], x[..., 1:d.rot_dims:2]
             x = torch.cat([torch.stack([a * c - b * s, b * c + a * s], -1).flatten(-2), x[..., d.rot_dims:]], -1)
             return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) if d.qk_norm else x
-        pad = lambda x: F.pad(x, (0, d.hp - d.dim))
+        pad = lambda x: F.pad(x, (0, d.hp - x.shape[-1]))
         page, off = block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block
-        k_cache[page, off] = pad(turn(k)).to(k_cache.dtype)
+        k_cache[page, off] = pad(turn(k).reshape(T, d.kv_heads, M * d.dim)).to(k_cache.dtype)
         v_cache[page, off] = pad(v).to(v_cache.dtype)
-        return pad(turn(q)).to(self.dtype)
+        q = turn(q)
+        if M == 2:                                                    # the other map's columns of a query are zeros
+            q = torch.stack([F.pad(q[:, 0::2], (0, d.dim)), F.pad(q[:, 1::2], (d.dim, 0))], 2).flatten(1, 2)
+        return pad(q).to(self.dtype)
 
-    def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out):
-        """Causal attention of the rows of `group` over the cache; q, out [T, heads, hp], row tables of all T rows."""
-        own = [h // (d.heads // d.kv_heads) for h in range(d.heads)]
+    def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out, lam=None,
+                      gate=None, eps=0.0):
+        """Causal attention of the rows of `group` over what the layer's mask leaves of the cache; q [T, maps * heads, hp], out
+        [T, heads, hp], row tables of all T rows. Two maps: `lam` [1] weighs the second. `gate` [T, heads * vdim]: logits of the
+        outputs' sigmoid gates."""
+        own = [h // (d.queries // d.kv_heads) for h in range(d.queries)]
         for r in range(group.row_lo, group.row_hi):
             n, s = int(row_kvlen[r]), int(row_slot[r])
+            lo = d.first_visible(n - 1)
             pages = block_table[s, :(n + kv_block - 1) // kv_block].long()
-            k = k_cache[pages].flatten(0, 1)[:n, own].float()
-            v = v_cache[pages].flatten(0, 1)[:n, own].float()
+            k = k_cache[pages].flatten(0, 1)[lo:n, own].float()
+            v = v_cache[pages].flatten(0, 1)[lo:n, own].float()
             sc = torch.einsum("hd,jhd->hj", q[r].float(), k) * d.scale
+            if d.softcap:
+                sc = d.softcap * torch.tanh(sc / d.softcap)
             if sink is not None:
                 sc = torch.cat([sc, sink[:, None]], 1)
-            out[r] = torch.einsum("hj,jhd->hd", torch.softmax(sc, -1)[:, :n], v).to(out.dtype)
+            o = torch.einsum("hj,jhd->hd", torch.softmax(sc, -1)[:, :n - lo], v)
+            if d.maps == 2:
+                o = o[0::2] - lam * o[1::2]
+                o = o / torch.sqrt(o.pow(2).sum(-1, keepdim=True) / d.vw + eps) * (1 - d.diff)
+            if gate is not None:
+                o[:, :d.vw] *= torch.sigmoid(gate[r].float()).view(d.heads, d.vw)
+            out[r] = o.to(out.dtype)
+        return out
+
+    def expert_rows(self, h, ids, w_gu, w_down):
+        """Rows of a token's experts, one per (token, pick): [T * top, width] fp32."""
+        T, K = ids.shape
+        out = torch.empty(T * K, w_down.shape[1], dtype=torch.float32, device=h.device)
+        for p, e in enumerate(ids.reshape(-1).tolist()):
+            g, u = (w_gu[e].float() @ h[p // K].float()).chunk(2)
+            out[p] = w_down[e].float() @ (F.silu(g) * u).to(self.dtype).float()
         return out
 
     def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
@@ -85,36 +114,64 @@ class TorchMixers:
 
 
 class CudaMixers:
-    def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps):
-        q = self.empty(proj.shape[0], d.heads, d.hp, dtype=self.dtype, device=self.device)
+    def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps, norms=None):
+        q = self.empty(proj.shape[0], d.queries, d.hp, dtype=self.dtype, device=self.device)
         self.launches += 1
+        if not d.plain:
+            assert bias is None and not d.qk_norm, "row norms and two maps: no biases, no norms per head"
+            self.C.gqa_row_prep(q, k_cache, v_cache, proj, *(norms or (None, None)), inv_freq, row_slot, row_pos, block_table, kv_block,
+                                [d.heads, d.maps, d.dim, d.vw, d.rot_dims, d.v_off], eps, self.status_word)
+            return q
         self.C.gqa_prep(q, k_cache, v_cache, proj, bias, inv_freq, row_slot, row_pos, block_table, kv_block, d.dim, d.rot_dims, d.v_off,
                         d.qk_norm, eps, self.status_word)
         return q
 
-    def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out):
+    def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out, lam=None,
+                      gate=None, eps=0.0):
         """Prompt groups go to the tcgen05 flash kernel (softmax weights as value + remainder); the others are split over their keys on
         the mma.sync kernel. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
-        key splits; what is left of it is what fills the GPU."""
-        a, b = group.row_lo, group.row_hi
+        key splits; what is left of it is what fills the GPU and what the layer's mask leaves of the keys. The difference of two maps and
+        the output gate ride on the merge of the splits, or follow the flash kernel in a pass of their own. Rows of `out` may lie apart."""
+        a, b, nq = group.row_lo, group.row_hi, d.queries
+        mixed = d.maps == 2 or gate is not None
+        bounds = dict(window=d.window, chunk=d.chunk, softcap=d.softcap)
+        mix = (lam, None if gate is None else gate[a:b], 1.0 - d.diff, d.maps, d.vw, eps)
         tc = self.dtype == torch.bfloat16 and d.hp in (64, 128, 256)
         if group.prompt and tc and kv_block % 64 == 0:
             self.launches += 1
             flat = q.view(q.shape[0], -1)
-            rc = self.C.attn_prefill_tc(out, flat, k_cache, v_cache, flat, segs[0], segs[1], segs[2], segs[3], block_table, kv_block,
-                                        group.max_rows, d.heads, d.kv_heads, d.hp, False, self.status_word, scale=d.scale, exact_p=True, sink=sink)
+            rows = self.empty(q.shape[0], nq, d.hp, dtype=torch.float32, device=self.device) if mixed else out
+            rc = self.C.attn_prefill_tc(rows, flat, k_cache, v_cache, flat, segs[0], segs[1], segs[2], segs[3], block_table, kv_block,
+                                        group.max_rows, nq, d.kv_heads, d.hp, False, self.status_word, scale=d.scale, exact_p=True, sink=sink,
+                                        **bounds)
             assert rc == 0, "prompt attention: shape outside the tensor-core kernel"
+            if mixed:
+                self.launches += 1
+                self.C.head_mix(out[a:b], rows[a:b], *mix)
             return out
-        mma = tc and d.heads // d.kv_heads <= 64
-        per_group = max(1, 64 // max(1, d.heads // d.kv_heads))
-        ctas = (group.seg_hi - group.seg_lo) * -(-group.max_rows // per_group) * d.kv_heads if mma else (b - a) * d.heads
+        group_heads = nq // d.kv_heads
+        mma = tc and group_heads <= 64
+        per_group = max(1, 64 // max(1, group_heads))
+        ctas = (group.seg_hi - group.seg_lo) * -(-group.max_rows // per_group) * d.kv_heads if mma else (b - a) * nq
         nsplit = max(1, min(nsplit, (4 if mma else 8) * self.sm_count // max(1, ctas)))
-        o_part = self.empty((b - a) * d.heads * nsplit * d.hp, dtype=torch.float32, device=self.device)
-        ml_part = self.empty((b - a) * d.heads * nsplit * 2, dtype=torch.float32, device=self.device)
-        self.launches += 2 if mma or nsplit > 1 else 1
+        if d.reach:
+            nsplit = min(nsplit, -(-(d.reach + group.max_rows) // 32))
+        o_part = self.empty((b - a) * nq * nsplit * d.hp, dtype=torch.float32, device=self.device)
+        ml_part = self.empty((b - a) * nq * nsplit * 2, dtype=torch.float32, device=self.device)
+        self.launches += 2 if mma or mixed or nsplit > 1 else 1
         self.C.gqa_attn(out[a:b], o_part, ml_part, q[a:b], k_cache, v_cache, sink, segs[0], segs[1], segs[2], group.max_rows, row_slot[a:b],
-                        row_kvlen[a:b], block_table, kv_block, a, nsplit, d.scale, not mma, self.status_word)
+                        row_kvlen[a:b], block_table, kv_block, a, nsplit, d.scale, not mma, self.status_word, **bounds,
+                        **(dict(zip(("lam", "gate", "mix_scale", "maps", "vdim", "eps"), mix)) if mixed else {}))
         return out
+
+    def expert_rows(self, h, ids, w_gu, w_down):
+        """One row of the expert's feed-forward per (token, pick)."""
+        pairs = ids.numel()
+        act = self.empty(pairs, w_down.shape[2], dtype=self.dtype, device=self.device)
+        yp = self.empty(pairs, h.shape[1], dtype=torch.float32, device=self.device)
+        self.launches += 2
+        self.C.expert_rows(yp, act, h, w_gu, w_down, ids)
+        return yp
 
     def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
         """A few rows: both low-rank products in one launch, then one launch per group for the whole mixer. Prompt groups: two GEMMs,

@@ -42,7 +42,7 @@ class TorchOps(TorchLatent, TorchMixers, TorchExtras):
         wf = w.float() + 1.0 if centred else w.float()
         return (xf * r * wf).to(self.dtype), x
 
-    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, act=None):
+    def linear(self, x, w, norm_w=None, eps=1e-6, res=None, swiglu=False, out_f32=False, out=None, act=None):
         """y = x W^T with optional RMSNorm(1+w) prologue, SwiGLU (W = [gate|up]), activation or residual epilogue."""
         if hasattr(w, "dense"):
             w = w.dense                      # quantised weight: the oracle multiplies by its dequantised values
@@ -57,6 +57,9 @@ class TorchOps(TorchLatent, TorchMixers, TorchExtras):
         y = TORCH_ACTS[act](y)
         if res is not None:
             y = y + res.float()
+        if out is not None:
+            out.copy_(y)
+            return out
         return y if out_f32 else y.to(self.dtype)
 
     def silu_mul(self, gu):

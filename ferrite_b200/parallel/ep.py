@@ -16,7 +16,7 @@ import torch.distributed as dist
 
 
 class ExpertParallel:
-    def __init__(self, tp, device, n_experts: int, hidden: int, cap_rows: int, spin_limit: int = 0):
+    def __init__(self, tp, device, n_experts: int, hidden: int, cap_rows: int, spin_limit: int = 0, status=None):
         self.tp = tp
         self.world = tp.world if tp is not None else 1
         self.rank = tp.rank if tp is not None else 0
@@ -45,7 +45,7 @@ class ExpertParallel:
         if self.world > 1:
             dist.barrier(tp.group)
         self.ctr = torch.zeros(4, dtype=torch.int32, device=self.device)
-        self.status = tp.status if (tp is not None and tp.fused) else torch.zeros(1, dtype=torch.int32, device=self.device)
+        self.status = status if status is not None else tp.status if (tp is not None and tp.fused) else torch.zeros(1, dtype=torch.int32, device=self.device)
         sm = torch.cuda.get_device_properties(self.device).multi_processor_count
         self.handle = C.make_ep_comm(ptrs, self.rank, n_experts, hidden, cap_rows, self.ctr, self.status, spin_limit, sm)
 
@@ -54,19 +54,20 @@ class ExpertParallel:
             raise RuntimeError(f"expert-parallel rank {self.rank}: status {int(self.status.item())} "
                                "(2 = a peer wait ran out, 5 = receive buffer capacity exceeded)")
 
-    def moe(self, ops, h, ids, wts, w_gu, w_down, shared=None, shared_gate=None, res=None):
+    def moe(self, ops, h, ids, wts, w_gu, w_down, shared=None, shared_gate=None, res=None, acc=None):
         """out[t] = res[t] + shared[t] * sigmoid(shared_gate[t]) + sum_k wts[t, k] * expert_{ids[t, k]}(h[t]) for this
-        rank's token rows; w_gu / w_down hold the experts this rank owns."""
+        rank's token rows; w_gu / w_down hold the experts this rank owns. `acc` (fp32 rows): the experts' sum is added to it instead."""
         self.calls += 1
         T, K = ids.shape
         inter = w_down.shape[2]
         if self.fused:
+            assert T * K <= self.cap_rows or self.world > 1, f"{T * K} (token, expert) pairs, room for {self.cap_rows}"
             if self._act is None or self._act.numel() < self.cap_rows * inter:
                 self._act = torch.empty(self.cap_rows * inter, dtype=h.dtype, device=self.device)
             need = T * K + 3 * self.n_experts + 8
             if self._plan is None or self._plan.numel() < need:
                 self._plan = torch.empty(max(need, 4096), dtype=torch.int32, device=self.device)
-            out = torch.empty(T, self.hidden, dtype=h.dtype, device=self.device)
+            out = acc if acc is not None else torch.empty(T, self.hidden, dtype=h.dtype, device=self.device)
             sg = None if shared_gate is None else shared_gate.reshape(-1).float().contiguous()
             self.C.ep_moe(self.handle, out, h.contiguous(), ids.contiguous(), wts.contiguous(), w_gu, w_down, shared, sg,
                           res, self._act, self._plan)
