@@ -77,11 +77,11 @@ class Engine:
         if cfg.layers:
             weights = pack_listed(cfg.shard(world), weights)
         is_t = lambda v: isinstance(v, torch.Tensor)
+        # routed layers of listed models stay in 16 bits where a router's logits come out of the product, and in their experts
+        routed = {f"l{i}.{n}" for i, l in enumerate(cfg.layers) if l.experts for n in ("in_proj", "experts_gate_up", "experts_down")}
         if self.ecfg.weight_dtype in ("nvfp4", "nvfp4-a16", "nvfp4-w4a4"):
             from ..ops.qweight import quantize_experts, quantize_weight
             big = ("in_proj", "out_proj", "gate_up", "up", "down", "lm_head")
-            # routed layers of listed models stay in 16 bits where a router's logits come out of the product, and in their experts
-            routed = {f"l{i}.{n}" for i, l in enumerate(cfg.layers) if l.experts for n in ("in_proj", "experts_gate_up", "experts_down")}
             for k in list(weights.keys()):
                 if not is_t(weights[k]) or k in routed:
                     continue
@@ -95,7 +95,7 @@ class Engine:
             from ..ops.qweight import quantize_weight
             big = ("in_proj", "out_proj", "gate_up", "up", "down")
             for k in list(weights.keys()):
-                if is_t(weights[k]) and k.split(".")[-1] in big and weights[k].dim() == 2:
+                if is_t(weights[k]) and k.split(".")[-1] in big and weights[k].dim() == 2 and k not in routed:
                     weights[k] = quantize_weight(weights[k], "fp8b", keep_dense=True, dense_dtype=self.dtype)
         elif self.ecfg.weight_dtype in ("exl3", "exl3-4", "exl3-3", "exl3-5"):
             # synthetic EXL3 weights of the architecture's shapes (random bit streams are valid tensors): what a

@@ -66,7 +66,7 @@ def route(cfg: ModelConfig, logits: torch.Tensor, bias: Optional[torch.Tensor]):
     n, e = sb.shape
     g = cfg.n_groups
     grp = sb.view(n, g, e // g)
-    gscore = grp.topk(2, -1).values.sum(-1)
+    gscore = grp.topk(min(2, e // g), -1).values.sum(-1)
     _, gi = torch.sort(gscore, dim=-1, descending=True, stable=True)
     gmask = torch.zeros(n, g, dtype=torch.bool)
     gmask.scatter_(1, gi[:, :cfg.topk_groups], True)
@@ -209,6 +209,8 @@ class RefModel:
         """Grouped-query attention of listed layers; run r's keys and values are its own."""
         l, w, p = self.cfg.layers[i], self.w, f"l{i}."
         proj = {n: w[p + n] @ x + (w[p + n + "_bias"] if l.bias else 0.0) for n in ("q", "k") + (() if l.key_values else ("v",))}
+        if l.row_norm:
+            proj.update({n: rmsnorm(proj[n], w[p + n + "_norm"], self.cfg.eps, False) for n in "qk"})
         ang = st.pos * rope_frequencies(l)
         c, s = ang.cos().float(), ang.sin().float()
 
@@ -217,14 +219,27 @@ class RefModel:
             a, b = z[:, 0:l.rot_dims:2].clone(), z[:, 1:l.rot_dims:2].clone()
             z[:, 0:l.rot_dims:2], z[:, 1:l.rot_dims:2] = a * c - b * s, b * c + a * s
             return z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + self.cfg.eps) if l.qk_norm else z
-        q, k = turned(proj["q"].view(l.heads, l.dim)), proj["k"].view(l.kv_heads, l.dim)
+        H, M = l.heads, l.maps
+        q, k = turned(proj["q"].view(H * M, l.dim)), proj["k"].view(l.kv_heads * M, l.dim)
         st.run.setdefault(("k", r), []).append(turned(k))
         st.run.setdefault(("v", r), []).append(k if l.key_values else proj["v"].view(l.kv_heads, l.vdim))
-        own = torch.arange(l.heads) // (l.heads // l.kv_heads)
-        K, V = torch.stack(st.run["k", r])[:, own], torch.stack(st.run["v", r])[:, own]
-        e = torch.exp(torch.einsum("hd,thd->ht", q, K) * l.scale)
-        pr = e / (e.sum(-1, keepdim=True) + (torch.exp(w[p + "sink"])[:, None] if l.sink else 0.0))
-        return w[p + "out_proj"] @ torch.einsum("ht,thd->hd", pr, V).reshape(-1) + (w[p + "out_bias"] if l.bias else 0.0)
+        own = torch.arange(H) // (H // l.kv_heads)
+        first = max(0, st.pos - l.window + 1) if l.window else st.pos - st.pos % l.chunk if l.chunk else 0
+        K, V = torch.stack(st.run["k", r][first:]), torch.stack(st.run["v", r][first:])[:, own]
+        maps = []
+        for m in range(M):
+            sc = torch.einsum("hd,thd->ht", q[m::M], K[:, m::M][:, own]) * l.scale
+            e = torch.exp(l.softcap * torch.tanh(sc / l.softcap) if l.softcap else sc)
+            pr = e / (e.sum(-1, keepdim=True) + (torch.exp(w[p + "sink"])[:, None] if l.sink else 0.0))
+            maps.append(torch.einsum("ht,thd->hd", pr, V))
+        o = maps[0]
+        if M == 2:
+            lam = torch.exp(w[p + "lq1"] @ w[p + "lk1"]) - torch.exp(w[p + "lq2"] @ w[p + "lk2"]) + l.diff
+            o = o - lam * maps[1]
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + self.cfg.eps) * (1 - l.diff)
+        if l.out_gate:
+            o = o * torch.sigmoid(w[p + "g"] @ x).view(H, l.vdim)
+        return w[p + "out_proj"] @ o.reshape(-1) + (w[p + "out_bias"] if l.bias else 0.0)
 
     def _cdelta(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
         """Delta rule with a decay per key channel; run r's state and convolution inputs are its own."""
@@ -244,6 +259,30 @@ class RefModel:
         S = st.run["rec", r] = S + k[:, :, None] * u[:, None, :]
         o = rmsnorm(torch.einsum("hdv,hd->hv", S, q), w[p + "gnorm_w"], self.cfg.eps, False)
         return w[p + "out_proj"] @ (o * torch.sigmoid(w[p + "g2"] @ (w[p + "g1"] @ x)).view(H, V)).reshape(-1)
+
+    def _experts(self, i: int, h: torch.Tensor) -> torch.Tensor:
+        """Routed feed-forward of listed layers."""
+        l, w, p = self.cfg.layers[i], self.w, f"l{i}."
+        rc = ModelConfig(router="sigmoid_group", top_k=l.top, n_groups=l.groups, topk_groups=l.keep_groups, route_scale=l.route_scale)
+        idx, wt = route(rc, (w[p + "router"] @ h)[None], None)
+        return sum(g * (w[p + "experts_down"][e] @ swiglu(w[p + "experts_gate_up"][e] @ h)) for e, g in zip(idx[0].tolist(), wt[0].tolist()))
+
+    def _token_parallel(self, t: int, st: RefState, tap: list) -> torch.Tensor:
+        """One token through a model of parallel blocks: the row before the final norm."""
+        c, w = self.cfg, self.w
+        x = w["embed"][t] * c.embed_scale
+        for run in c.layer_runs:
+            i, l, p = run.layer, c.layers[run.layer], f"l{run.layer}."
+            h = F.layer_norm(x, x.shape, w[p + "pre_norm"], w[p + "pre_norm_bias"], c.eps)
+            y = self._gqa(run.index, i, h, st)
+            if l.experts:
+                y = y + self._experts(i, h)
+            elif l.ff:
+                y = y + w[p + "down"] @ (F.silu(w[p + "gate"] @ h) * (w[p + "up"] @ h))
+            x = x + y
+            if i in c.tap_layers and not any(q.layer == i and q.index > run.index for q in c.layer_runs):
+                tap.append(x.clone())
+        return x
 
     def _token_out_norm(self, t: int, st: RefState, tap: list) -> torch.Tensor:
         """One token through a model with norms on the sublayers' outputs: the row before the final norm."""
@@ -292,10 +331,13 @@ class RefModel:
         head = w["embed"] if c.tie_embeddings else w["lm_head"]
         for t in list(tokens):
             tap = []
-            if c.out_norm:
-                x = self._token_out_norm(int(t), st, tap)
+            if c.layers:
+                x = (self._token_parallel if c.parallel else self._token_out_norm)(int(t), st, tap)
                 st.pos += 1
-                y = head @ rmsnorm(x, w["final_norm"], c.eps, False) * c.logit_scale
+                if c.parallel:
+                    y = head @ F.layer_norm(x, x.shape, w["final_norm"], w["final_norm_bias"], c.eps) * c.logit_scale
+                else:
+                    y = head @ rmsnorm(x, w["final_norm"], c.eps, False) * c.logit_scale
                 logits.append(c.logit_softcap * torch.tanh(y / c.logit_softcap) if c.logit_softcap else y)
                 taps.append(tap)
                 continue

@@ -30,7 +30,7 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
     out: Dict[str, tuple] = {p + "pre_norm": (h,)} if cfg.pre_norm else {}
     if cfg.parallel:
         out[p + "pre_norm_bias"] = (h,)
-    else:
+    if cfg.out_norm:
         out[p + "mix_norm"] = (h,)
     if l.mixer == "latent":
         out.update({p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,), p + "q_b": (l.heads * l.dim, l.q_rank)})
@@ -506,7 +506,7 @@ def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
     if cfg.gram_buckets:
         out["bigram"] = _pad(w["bigram"], cfg.gram_buckets + 1, W)
     if cfg.parallel:
-        out["final_norm_bias"] = vec("final_norm_bias")
+        out["final_norm_bias"] = vec("final_norm_bias", cfg.logit_scale)
     if cfg.loop and cfg.loop_input:
         out["loop_in"] = _pad(w["loop_in"].view(cfg.hidden, 2, cfg.hidden), W, 2, W).view(W, 2 * W)
         out["loop_step"] = _pad(w["loop_step"].float(), cfg.loop[2], W)

@@ -155,3 +155,10 @@ def forward(cfg, weights, ids, dtype=torch.float64):
         x = x + y
         after.append(x)
     return layer_norm(x, w["final.norm"], w["final.norm.b"], eps) @ w["head"].t(), after
+
+
+def greedy(cfg, weights, prompt, n):
+    ids = list(prompt)
+    for _ in range(n):
+        ids.append(int(forward(cfg, weights, ids)[0][-1].argmax()))
+    return ids[len(prompt):]
