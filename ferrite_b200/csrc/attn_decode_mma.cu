@@ -66,7 +66,7 @@ __device__ __forceinline__ void dm_e4m3x16_to_bf16(const uint4& c, uint4& lo, ui
 // applied to the scores (K) and to P (V) instead of to every element.
 // PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (16 bits of mantissa instead of 8).
 // BND: rows see a window or a chunk of the keys up to their own, scores are softcapped (cap_log2 = cap * log2 e; scale_log2 then leads to
-// the argument of tanh_of_2log2); the splits share the keys that some row of the CTA sees.
+// the argument of the tanh); the splits share the keys that some row of the CTA sees.
 template <int HD, bool KV8, bool PX, bool BND>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, const __nv_bfloat16* __restrict__ q,
@@ -230,7 +230,7 @@ attn_decode_mma_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, 
           float sv = s[nt][e];
           if (KV8) sv *= tsc[((lane & 3) * 2 + nt * 8 + (e & 1)) * 2];
           sv *= scale_log2;
-          if (BND && cap_log2 > 0.f) sv = cap_log2 * tanh_of_2log2(sv);
+          if (BND && cap_log2 > 0.f) sv = cap_log2 * tanh_exp(sv);
           const float v = vis ? sv : -INFINITY;
           s[nt][e] = v;
           mx[h] = fmaxf(mx[h], v);
@@ -330,7 +330,7 @@ extern "C" int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, cons
   if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
   constexpr float LOG2E = 1.4426950408889634f;
   const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
-  const float scale_log2 = LOG2E * raw_scale * (cap > 0.f ? 2.f / cap : 1.f);
+  const float scale_log2 = cap > 0.f ? raw_scale / cap : raw_scale * LOG2E;
 #define FB_DM(HDV, K8, PXV, BNDV)                                                                                              \
   {                                                                                                                 \
     const size_t smem = K8 ? (size_t)(DM_BM + 2 * DM_BKV) * (HDV + 8) * 2 + (size_t)4 * DM_BKV * HDV + 4 * DM_BKV * 4 * 2 \

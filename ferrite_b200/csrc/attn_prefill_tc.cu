@@ -77,7 +77,7 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // PX: the softmax weights enter the PV product as a bf16 value plus its bf16 remainder (two TS products per k step, a second
 // P buffer in TMEM), which keeps 16 bits of their mantissa instead of 8.
 // BND: rows see a window or a chunk of the keys, scores are softcapped (cap_log2 = cap * log2 e, scale_log2 then leads to the argument of
-// tanh_of_2log2). Key tiles that no row of the CTA sees are skipped; out_f32: rows of floats.
+// the tanh, which is a polynomial where all scores of a warp's tile are below the cap). Key tiles that no row of the CTA sees are skipped; out_f32: rows of floats.
 template <int HD, bool PX, bool BND>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
@@ -279,10 +279,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         mbar_arrive(&s_empty[s]);
         const int t0 = (tile0 + j) * FT_BKV + half * HC;
         const bool need_mask = t0 + HC - 1 > pos0 + q0 || (BND && t0 < klo_last);
+        const bool capped = BND && cap_log2 > 0.f;
+        if (capped) {
+          float am = 0.f;
+#pragma unroll
+          for (int c = 0; c < HC; ++c) {
+            const float x = __uint_as_float(sr[c]) * scale_log2;
+            sr[c] = __float_as_uint(x);
+            am = fmaxf(am, fabsf(x));
+          }
+          if (__any_sync(0xffffffffu, am > 1.f)) {
+#pragma unroll
+            for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(cap_log2 * tanh_exp(__uint_as_float(sr[c])));
+          } else {
+#pragma unroll
+            for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(cap_log2 * tanh_poly(__uint_as_float(sr[c])));
+          }
+        }
 #pragma unroll
         for (int c = 0; c < HC; ++c) {
-          float v = __uint_as_float(sr[c]) * scale_log2;
-          if (BND && cap_log2 > 0.f) v = cap_log2 * tanh_of_2log2(v);
+          float v = __uint_as_float(sr[c]);
+          if (!capped) v *= scale_log2;
           if (need_mask && (t0 + c > qpos || (BND && t0 + c < klo))) v = -INFINITY;
           sr[c] = __float_as_uint(v);
           mx = fmaxf(mx, v);
@@ -430,7 +447,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if (ldo % 8) return -20;
   constexpr float LOG2E = 1.4426950408889634f;
   const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
-  const float scale_log2 = LOG2E * raw_scale * (cap > 0.f ? 2.f / cap : 1.f);
+  const float scale_log2 = cap > 0.f ? raw_scale / cap : raw_scale * LOG2E;
 #define FB_FT(HDV, PXV, BNDV)                                                                                                 \
   {                                                                                                                \
     const size_t smem = (size_t)(FT_BQ + ((HDV == 256 ? 3 : 4) + (HDV == 256 ? 2 : 3)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \

@@ -694,7 +694,12 @@ void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cach
               (!sink || sink->numel() == heads), "gqa_attn: layouts");
   const float* sk = (const float*)cptr(sink);
   if (!cuda_cores) {
-    check(fb_attn_decode_mma(nullptr, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+    const int rc = fb_attn_decode_keys(o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                                       seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), row_kvlen.data_ptr<int>(),
+                                       block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block, (int)seg_slot.numel(), (int)max_rows,
+                                       rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, (int)row_first, status.data_ptr<int>(), cur_stream());
+    if (rc != -20) check(rc, "attn_decode_keys");
+    else check(fb_attn_decode_mma(nullptr, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                              nullptr, nullptr, 0, seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(),
                              row_kvlen.data_ptr<int>(), nullptr, nullptr, block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block,
                              (int)seg_slot.numel(), (int)max_rows, rows, heads, kvh, hd, (int)nsplit, 0, (float)scale, 1, kbp, (int)row_first,

@@ -85,10 +85,9 @@ gqa_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ 
 // head. proj row = [heads x maps x dim | kv_heads x maps x dim | .. v_off: kv_heads x vdim]. A key row takes a head's maps side by side; a
 // query goes to [row][head][map][hp] with zeros in the other map's columns, so that one product with the key row gives its map's score.
 // One CTA per row: sums of squares over the row, then one warp per head.
-constexpr int GR_WARPS = 8;
-
-template <typename T>
-__global__ void __launch_bounds__(GR_WARPS * 32)
+// Positions, pages and angles do not come from the kernel before this one, so they are read while it drains.
+template <typename T, bool EVEN>
+__global__ void __launch_bounds__(512)
 gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ proj, long ldp,
                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, const double* __restrict__ inv_freq,
                     const int* __restrict__ row_slot, const int* __restrict__ row_pos, const int* __restrict__ block_table, int max_blocks,
@@ -98,19 +97,7 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
   pdl_launch_dependents();
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nq = heads * maps * dim, nk = kv_heads * maps * dim;
-  pdl_wait();
-  const float* pr = proj + (size_t)row * ldp;
   const int pos = row_pos[row];
-  float rq = 1.f, rk = 1.f;
-  if (q_norm) {
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq; i += blockDim.x) sq = fmaf(pr[i], pr[i], sq);
-    for (int i = threadIdx.x; i < nk; i += blockDim.x) sk = fmaf(pr[nq + i], pr[nq + i], sk);
-    sq = block_sum(sq, red);
-    sk = block_sum(sk, red);
-    rq = 1.f / sqrtf(sq / (float)nq + eps);
-    rk = 1.f / sqrtf(sk / (float)nk + eps);
-  }
   for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
     constexpr double TURN = 6.283185307179586476925;
     double a = (double)pos * inv_freq[i];
@@ -119,15 +106,46 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
     sincosf((float)a, &s, &c);
     gr_turn[i] = make_float2(c, s);
   }
-  __syncthreads();
   const int blk = block_table[(size_t)row_slot[row] * max_blocks + pos / kv_block];
   if (blk < 0 && threadIdx.x == 0) set_status(status, ST_BOUNDS);
+  pdl_wait();
+  const float* pr = proj + (size_t)row * ldp;
+  float rq = 1.f, rk = 1.f;
+  if (q_norm) {
+    auto squares = [&](const float* x, int n) {
+      float s = 0.f;
+      if (EVEN) {
+        for (int i = 2 * threadIdx.x; i < n; i += 2 * blockDim.x) {
+          const float2 v = *reinterpret_cast<const float2*>(x + i);
+          s = fmaf(v.x, v.x, fmaf(v.y, v.y, s));
+        }
+      } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) s = fmaf(x[i], x[i], s);
+      }
+      return s;
+    };
+    const float sq = squares(pr, nq), sk = squares(pr + nq, nk);
+    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
+    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+  } else {
+    __syncthreads();
+  }
   const size_t page_row = blk < 0 ? 0 : ((size_t)blk * kv_block + pos % kv_block) * kv_heads;
   // columns d, d + 1 of one map: src[0 .. dim), rotated; e counts from the map's first column and may leave it on either side
   auto pair = [&](const float* src, const float* w, float r, int e) {
     float2 x = make_float2(0.f, 0.f);
-    if (e >= 0 && e < dim) x.x = w ? src[e] * r * w[e] : src[e];
-    if (e + 1 >= 0 && e + 1 < dim) x.y = w ? src[e + 1] * r * w[e + 1] : src[e + 1];
+    if (EVEN) {                                             // both columns are inside or neither is
+      if (e >= 0 && e < dim) {
+        x = *reinterpret_cast<const float2*>(src + e);
+        if (w) {
+          const float2 ww = *reinterpret_cast<const float2*>(w + e);
+          x.x *= r * ww.x; x.y *= r * ww.y;
+        }
+      }
+    } else {
+      if (e >= 0 && e < dim) x.x = w ? src[e] * r * w[e] : src[e];
+      if (e + 1 >= 0 && e + 1 < dim) x.y = w ? src[e + 1] * r * w[e + 1] : src[e + 1];
+    }
     if (e >= 0 && e < rot) {                                // rot is even, and so is e wherever something is rotated
       const float2 t = gr_turn[e >> 1];
       x = make_float2(x.x * t.x - x.y * t.y, x.y * t.x + x.x * t.y);
@@ -135,7 +153,7 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
     return x;
   };
   const int units = heads * maps + 2 * kv_heads;
-  for (int u = warp; u < units; u += GR_WARPS) {
+  for (int u = warp; u < units; u += blockDim.x >> 5) {
     if (u < heads * maps) {
       const float* src = pr + u * dim;
       const float* w = q_norm ? q_norm + u * dim : nullptr;
@@ -164,7 +182,12 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
       if (blk < 0) continue;
       const float* src = pr + v_off + g * vdim;
       T* dst = v_cache + (page_row + g) * hp;
-      for (int d = 2 * lane; d < hp; d += 64) Elem<T>::store2(dst + d, d < vdim ? src[d] : 0.f, d + 1 < vdim ? src[d + 1] : 0.f);
+      for (int d = 2 * lane; d < hp; d += 64) {
+        float2 x = make_float2(0.f, 0.f);
+        if (EVEN && d < vdim) x = *reinterpret_cast<const float2*>(src + d);
+        else if (d < vdim) x = make_float2(src[d], d + 1 < vdim ? src[d + 1] : 0.f);
+        Elem<T>::store2(dst + d, x.x, x.y);
+      }
     }
   }
 }
@@ -181,13 +204,18 @@ extern "C" int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const 
   if (dim < 1 || vdim < 1 || maps < 1 || maps > 2 || maps * dim > hp || vdim > hp || hp % 64 || rot % 2 || rot > dim || (rot && !inv_freq) ||
       (rot && maps == 2 && dim % 2) || (!q_norm) != (!k_norm)) return -1;
   const size_t smem = (size_t)(rot / 2 + 1) * sizeof(float2);
+  const int threads = heads * maps + 2 * kv_heads > 16 ? 512 : 256;
   auto go = [&](auto kern, auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    return (int)launch_pdl(kern, dim3(rows), dim3(GR_WARPS * 32), smem, s, (T*)q_out, (T*)k_cache, (T*)v_cache, proj, ldp, q_norm, k_norm,
+    return (int)launch_pdl(kern, dim3(rows), dim3(threads), smem, s, (T*)q_out, (T*)k_cache, (T*)v_cache, proj, ldp, q_norm, k_norm,
                            inv_freq, row_slot, row_pos, block_table, max_blocks, kv_block, heads, kv_heads, maps, dim, vdim, hp, rot, v_off, eps,
                            status);
   };
-  return f32 ? go(gqa_row_prep_kernel<float>, (float*)0) : go(gqa_row_prep_kernel<__nv_bfloat16>, (__nv_bfloat16*)0);
+  using B = __nv_bfloat16;
+  const bool even = dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && v_off % 2 == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)q_norm | (uintptr_t)k_norm) & 7) == 0;
+  if (even) return f32 ? go(gqa_row_prep_kernel<float, true>, (float*)0) : go(gqa_row_prep_kernel<B, true>, (B*)0);
+  return f32 ? go(gqa_row_prep_kernel<float, false>, (float*)0) : go(gqa_row_prep_kernel<B, false>, (B*)0);
 }
 
 extern "C" int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* bias,

@@ -129,7 +129,7 @@ class CudaMixers:
     def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out, lam=None,
                       gate=None, eps=0.0):
         """Prompt groups go to the tcgen05 flash kernel (softmax weights as value + remainder); the others are split over their keys on
-        the mma.sync kernel. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
+        the mma.sync kernels, over the warps of a CTA as well where a segment brings at most 16 (row, head) pairs per key head. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
         key splits; what is left of it is what fills the GPU and what the layer's mask leaves of the keys. The difference of two maps and
         the output gate ride on the merge of the splits, or follow the flash kernel in a pass of their own. Rows of `out` may lie apart."""
         a, b, nq = group.row_lo, group.row_hi, d.queries
@@ -151,11 +151,12 @@ class CudaMixers:
             return out
         group_heads = nq // d.kv_heads
         mma = tc and group_heads <= 64
+        keys = mma and d.hp <= 128 and group.max_rows * group_heads <= 16 and kv_block % 64 == 0
         per_group = max(1, 64 // max(1, group_heads))
         ctas = (group.seg_hi - group.seg_lo) * -(-group.max_rows // per_group) * d.kv_heads if mma else (b - a) * nq
-        nsplit = max(1, min(nsplit, (4 if mma else 8) * self.sm_count // max(1, ctas)))
+        nsplit = max(1, min(nsplit, ((3 if d.hp == 128 else 5) if keys else 4 if mma else 8) * self.sm_count // max(1, ctas)))
         if d.reach:
-            nsplit = min(nsplit, -(-(d.reach + group.max_rows) // 32))
+            nsplit = min(nsplit, -(-(d.reach + group.max_rows) // 64) + 1 if keys else -(-(d.reach + group.max_rows) // 32))
         o_part = self.empty((b - a) * nq * nsplit * d.hp, dtype=torch.float32, device=self.device)
         ml_part = self.empty((b - a) * nq * nsplit * 2, dtype=torch.float32, device=self.device)
         self.launches += 2 if mma or mixed or nsplit > 1 else 1

@@ -1,19 +1,21 @@
 """Designs of listed layers, each beside the framework's closest other model of the same width, heads and parameter count, with
 random weights: Zototar (latent attention without positions) beside the dense MLA model, Dofunex (delta rules with a decay per
-channel, every fourth layer attention) beside the dense Gated DeltaNet hybrid.
+channel, every fourth layer attention) beside the dense Gated DeltaNet hybrid, Rakizen (parallel blocks, windows and chunks, two maps in every
+fourth layer) beside the sequential grouped-query attention model, dense or routed.
 
-`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()` /
-`kernels_dofunex()` time every kernel of the first beside the kernel that does the same job for the second and give both as fractions
-of their rooflines. They print nothing and return plain dictionaries; `bench.py --design ...` and `microbench latent|cdelta` print them.
+`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()`, `kernels_dofunex()` and
+`kernels_rakizen()` time every kernel of the first beside the kernel that does the same job for the second and give both as fractions of their
+rooflines. They print nothing and return plain dictionaries; `bench.py --design ...` and `microbench latent|cdelta|parallel` print them.
 """
 from __future__ import annotations
 
 import statistics
+from dataclasses import replace
 from typing import Dict, List
 
 import torch
 
-from ..config import EngineConfig, ModelConfig, dofunex, zototar
+from ..config import EngineConfig, ModelConfig, dofunex, rakizen, zototar
 from .microbench import Timer, graph_time, peaks, rnd
 
 SIZES = {       # name: width, heads, query latent, feed-forward width, layers
@@ -45,12 +47,34 @@ def pair_dofunex(size: str):
     return a, ModelConfig(inter=max(256, round(spare / (3 * w * n) / 256) * 256), **kw)
 
 
+def pair_rakizen(size: str):
+    """(Rakizen model, sequential model of grouped-query attention layers) of one size, equal in width, heads, feed-forward and, by the dense
+    width, parameters; routed feed-forwards in every layer of both or in none."""
+    w, h, kv, ff, n, experts, top, groups, keep = SIZES_RAKIZEN[size]
+    routed = dict(experts=experts, top=top, groups=groups, keep=keep, expert_ff=ff) if experts else {}
+    a = rakizen(w, n, h, kv, ff, VOCAB, moe_every=1, name=f"rakizen-{size}", **routed)
+    kw = dict(name=f"gqa-{size}", hidden=w, n_layers=n, full_attn_every=1, head_dim=DIM, n_q=h, n_kv=kv, rotary_dim=DIM, attn_gate=False, vocab=VOCAB,
+              tie_embeddings=False)
+    if experts:
+        return a, ModelConfig(inter=ff, n_experts=experts, top_k=top, expert_inter=ff, router="sigmoid_group", n_groups=groups, topk_groups=keep,
+                              route_scale=1.5, **kw)
+    spare = a.param_count() - ModelConfig(inter=0, **kw).param_count()
+    return a, ModelConfig(inter=max(256, round(spare / (3 * w * n) / 128) * 128), **kw)
+
+
+SIZES_RAKIZEN = {       # name: width, heads, key / value heads, (expert's) feed-forward width, layers, experts, per token, groups, kept groups
+    "2k": (2048, 16, 4, 6144, 16, 0, 0, 1, 1),
+    "4k": (4096, 32, 8, 12288, 8, 0, 0, 1, 1),
+    "2k-moe": (2048, 16, 4, 1024, 12, 64, 6, 8, 4),
+}
 SIZES_DOFUNEX = {       # name: width, heads, key / value heads of the attention layers, feed-forward width, layers
     "2k": (2048, 16, 4, 6144, 16),
     "4k": (4096, 32, 8, 11008, 8),
     "5k": (5120, 40, 8, 17408, 8),
 }
 DESIGNS = {"zototar": (pair, "mla_dense", "dense MLA model of equal width, heads, latent and parameter count", "2k,4k,7k"),
+           "rakizen": (pair_rakizen, "gqa_sequential", "sequential grouped-query attention model of equal width, heads and parameter count (routed "
+                       "feed-forwards in the moe size)", "2k,4k,2k-moe"),
            "dofunex": (pair_dofunex, "hybrid_dense", "dense Gated DeltaNet hybrid of equal width, heads and parameter count", "2k,4k,5k")}
 
 
@@ -339,5 +363,132 @@ def kernels_dofunex(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     gout = rnd(T, H * D)
     add(f"gated head norm, {T} rows", (lambda j: ops.C.gated_norm_sigmoid(gout, y, gate, w["gnorm_w"], 1e-6), T * H * D * 10.0, 0.0, 1), "gated_norm",
         (lambda j: ops.gated_norm(y.view(T, H * D), pg, 3 * H * D, gw, H, D, 1e-6), T * H * D * 8.0, 0.0, 1))
+    assert ops.status() == 0
+    return acc.rows
+
+
+def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, ctx: int = 4096, prompt: int = 2048, size: int = 1024) -> List[Dict]:
+    """Rakizen's kernels beside those of the sequential grouped-query attention model (heads of 128 columns; two maps of 64 over values of 128
+    in half the heads). Bounded rows see `size` keys; the like kernel of few rows gets a cache of that many."""
+    from ..models.weights import GqaDims
+    from ..ops.cuda_ops import CudaOps
+    from ..ops.latent import SegGroup
+    ops, acc = CudaOps(dev), _Rows(dev)
+    add = acc.add
+    D, kvb, H, G = DIM, 64, heads, kv_heads
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    inv, inv64 = torch.rand(D // 2, device=dev), torch.rand(D // 2, device=dev, dtype=torch.float64)
+    one = GqaDims(H, G, D, D, D ** -0.5, D, (H + G) * D, False, D, 1, True, 50.0, size)
+    two = GqaDims(H // 2, G // 2, D // 2, D, (D // 2) ** -0.5, 0, (H + G) * D // 2, False, D, 2, False, 50.0, 0, size, 0.6, (H + G) * D // 2 + G * D // 2)
+    nw, lam = rnd(D), torch.full((1,), 0.7, device=dev)
+    for m in (1, 16, prompt):
+        bufs = max(1, min(8, (400 << 20) // (m * width * 4)))
+        x0, y0 = [f32(m, width) for _ in range(bufs)], [f32(m, width) for _ in range(bufs)]
+        xb, yb = [rnd(m, width) for _ in range(bufs)], [rnd(m, width) for _ in range(bufs)]
+        w32, w16 = torch.ones(width, device=dev), rnd(width)
+        add(f"add_layer_norm (add, next norm), {m} rows", (lambda j: ops.add_layer_norm(x0[j], y0[j], width, 1e-6, w32, w32), m * width * 14.0, 0.0, bufs),
+            "rmsnorm + residual", (lambda j: ops.rmsnorm(xb[j], w16, 1e-6, True, res=yb[j]), m * width * 8.0, 0.0, bufs))
+        nb, many = max(1, m // kvb), m > kvb
+        slot = torch.zeros(m, dtype=torch.int32, device=dev) if many else torch.arange(m, dtype=torch.int32, device=dev)
+        pos = torch.arange(m, dtype=torch.int32, device=dev) if many else torch.zeros(m, dtype=torch.int32, device=dev)
+        bt = torch.arange((1 if many else m) * nb, dtype=torch.int32, device=dev).view(-1, nb)
+        kc, vc = rnd(bt.numel(), kvb, G, D), rnd(bt.numel(), kvb, G, D)
+        kc2, vc2 = rnd(bt.numel(), kvb, G // 2, D), rnd(bt.numel(), kvb, G // 2, D)
+        pb = 8 if many else 32
+        proj, norms = [f32(m, (H + 2 * G) * D) for _ in range(pb)], (f32(H * D), f32(G * D))
+        pq = [rnd(m, (H + 2 * G) * D) for _ in range(pb)]
+        like = ("attn_prep", (lambda j: ops.attn_prep(pq[j], nw, nw, inv, slot, pos, bt, kc, vc, kvb, H, G, D, D, False, 1e-6),
+                              m * D * (H + 2 * G) * 4.0, 0.0, pb))
+        add(f"gqa_row_prep, row norms and rotation, {m} rows, {H} / {G} heads",
+            (lambda j: ops.gqa_prep(proj[j], one, None, inv64, slot, pos, bt, kc, vc, kvb, 1e-6, norms=norms), m * D * (H + 2 * G) * 6.0, 0.0, pb), *like)
+        half = D * (H // 2 + G)                              # projected columns: H / 2 heads of two maps of D / 2, G / 2 keys and values of D
+        add(f"gqa_row_prep, two maps, {m} rows, {H // 2} / {G // 2} heads",
+            (lambda j: ops.gqa_prep(proj[j], two, None, inv64[:0], slot, pos, bt, kc2, vc2, kvb, 1e-6), m * (half * 4.0 + D * (H + G) * 2.0), 0.0, pb), *like)
+        rows, gate, o = f32(m, H, D), f32(m, H // 2 * D), rnd(m, H // 2, D)
+        if many:
+            add(f"head_mix (difference, norm, gate), {m} rows", (lambda j: ops.C.head_mix(o, rows, lam, gate, 0.4, 2, D, 1e-6), m * H * D * 7.0, 0.0, 1),
+                "gated_norm", (lambda j: ops.gated_norm(rows.view(m, H * D), pq[0], 0, nw, H, D, 1e-6), m * H * D * 8.0, 0.0, 1))
+        del x0, y0, xb, yb, proj, pq, rows
+    for m in (1, 4, 16):
+        nb, nbl = ctx // kvb, size // kvb
+        bufs = max(1, min(32, (400 << 20) // (m * size * G * D * 4)))
+        kc, vc = [rnd(m * nb, kvb, G, D) for _ in range(min(bufs, 8))], [rnd(m * nb, kvb, G, D) for _ in range(min(bufs, 8))]
+        kl, vl = [rnd(m * nbl, kvb, G, D) for _ in range(bufs)], [rnd(m * nbl, kvb, G, D) for _ in range(bufs)]
+        bt, slot = torch.arange(m * nb, dtype=torch.int32, device=dev).view(m, nb), torch.arange(m, dtype=torch.int32, device=dev)
+        btl = torch.arange(m * nbl, dtype=torch.int32, device=dev).view(m, nbl)
+        kvlen, lenl, ones = (torch.full((m,), v, dtype=torch.int32, device=dev) for v in (ctx, size, 1))
+        q, out, out2, pj, gate = rnd(m, H, D), rnd(m, H, D), rnd(m, H // 2, D), rnd(m, H * D), f32(m, H // 2 * D)
+        grp = SegGroup(0, m, 0, m, 1)
+        work = (m * size * G * D * 4.0, 4.0 * m * H * size * D, bufs)
+        like = ("attention + combine", (lambda j: ops.attention(q, pj, kl[j], vl[j], slot, lenl, btl, kvb, H, G, D, False, nsplit=16,
+                                                                segs=(slot, slot, ones, 1)), *work))
+        nk = len(kc)
+        add(f"decode attention + merge, softcap, window of {size}, {m} rows",
+            (lambda j: ops.gqa_attention(q, one, kc[j % nk], vc[j % nk], None, grp, slot, kvlen, (slot, slot, ones), bt, kvb, 64, out), work[0], work[1], nk), *like)
+        c2, v2 = [c.view(-1, kvb, G // 2, D) for c in kc], [c.view(-1, kvb, G // 2, D) for c in vc]
+        work2 = (m * size * G // 2 * D * 4.0, m * H * size * D * 3.0, nk)
+        add(f"decode attention + merge, two maps, gate, chunk of {size}, {m} rows",
+            (lambda j: ops.gqa_attention(q, two, c2[j % nk], v2[j % nk], None, grp, slot, kvlen, (slot, slot, ones), bt, kvb, 64, out2, lam=lam, gate=gate,
+                                         eps=1e-6), *work2), *like)
+        del kc, vc, kl, vl, c2, v2
+    T, nb = prompt, prompt // kvb
+    perm = torch.randperm(nb, device=dev).to(torch.int32).view(1, nb)
+    kc, vc, q, out, pj = rnd(nb, kvb, G, D), rnd(nb, kvb, G, D), rnd(T, H, D), rnd(T, H, D), rnd(T, H * D)
+    k2, v2, o2, gate = rnd(nb, kvb, G // 2, D), rnd(nb, kvb, G // 2, D), rnd(T, H // 2, D), f32(T, H // 2 * D)
+    s0 = (i32([0]), i32([0]), i32([T]), i32([0]))
+    rslot, rlen = torch.zeros(T, dtype=torch.int32, device=dev), torch.arange(1, T + 1, dtype=torch.int32, device=dev)
+    grp = SegGroup(0, 1, 0, T, T, True)
+    like = ("prompt attention, bf16 weights", (lambda j: ops.attention_prefill(q, pj, kc, vc, *s0, perm, kvb, H, G, D, False, T), 0.0,
+                                               T * (T + 1) / 2.0 * H * 4 * D, 1))
+    for sz in (size, T):
+        one, two = replace(one, window=sz), replace(two, chunk=sz)
+        seen1, seen2 = sum(min(t + 1, sz) for t in range(T)), sum(t % sz + 1 for t in range(T))
+        add(f"prompt attention, softcap, window of {sz}, {T} rows",
+            (lambda j: ops.gqa_attention(q, one, kc, vc, None, grp, rslot, rlen, s0, perm, kvb, 1, out), 0.0, seen1 * H * 4.0 * D, 1), *like)
+        add(f"prompt attention and head_mix, two maps, gate, chunk of {sz}, {T} rows",
+            (lambda j: ops.gqa_attention(q, two, k2, v2, None, grp, rslot, rlen, s0, perm, kvb, 1, o2, lam=lam, gate=gate, eps=1e-6), 0.0,
+             seen2 * H * 3.0 * D, 1), *like)
+    del kc, vc, k2, v2
+    # products: both output projections at once, beside the two of the sequential model; in_proj with fp32 sums
+    ff = 3 * width
+    for m in (1, 4, 16, prompt):
+        both, o, a, res = rnd(m, H * D + ff), rnd(m, H * D), rnd(m, ff), rnd(m, width)
+        wj = [rnd(width, H * D + ff, scale=0.02) for _ in range(4)]
+        wo, wd = [rnd(width, H * D, scale=0.02) for _ in range(4)], [rnd(width, ff, scale=0.02) for _ in range(4)]
+        work = (width * (H * D + ff) * 2.0 + m * ((H * D + ff) * 2.0 + width * 4.0), 2.0 * m * width * (H * D + ff), 4)
+        add(f"joint output projection, fp32 sums, {m} rows, {H * D} + {ff} -> {width}", (lambda j: ops.linear(both, wj[j], out_f32=True), *work),
+            "two linears + residual", (lambda j: ops.linear(a, wd[j], res=ops.linear(o, wo[j], res=res)), *work))
+        del wj, wo, wd
+        wi, x = [rnd((H + 2 * G) * D, width, scale=0.02) for _ in range(8)], rnd(m, width)
+        n = (H + 2 * G) * D
+        add(f"input projection, fp32 sums, {m} rows, {width} -> {n}",
+            (lambda j: ops.linear(x, wi[j], out_f32=True), n * width * 2.0 + m * (width * 2.0 + n * 4.0), 2.0 * m * n * width, 8), "linear, norm in front",
+            (lambda j: ops.linear(x, wi[j], norm_w=res[0], eps=1e-6), n * width * 2.0 + m * (width * 2.0 + n * 2.0), 2.0 * m * n * width, 8))
+        del wi
+    # routed feed-forward: 64 experts of 1024, six per token, four of eight groups
+    E, K, F, W = 64, 6, 1024, 2048
+    gu, dn = rnd(E, 2 * F, W, scale=0.02), rnd(E, W, F, scale=0.02)
+    for m in (1, 4, 16):
+        h, x, y, res = rnd(m, W), f32(m, W), f32(m, W), rnd(m, W)
+        picks = [ops.moe_route(f32(m, E), None, 1, K, 8, 4, 1.5) for _ in range(16)]
+        used = sum(len(set(ids.reshape(-1).tolist())) for ids, _ in picks) / 16
+        w32 = torch.ones(W, device=dev)
+        work = (used * 3.0 * F * W * 2, 6.0 * m * K * F * W, 16)
+        add(f"expert rows + add_layer_norm, {m} rows",
+            (lambda j: ops.add_layer_norm(x, y, W, 1e-6, w32, w32, (ops.expert_rows(h, picks[j][0], gu, dn), picks[j][1])), *work),
+            "moe_experts (pairs, combine)", (lambda j: ops.moe_experts(h, *picks[j], gu, dn, 0, E, None, None, res), *work))
+    from ..parallel.ep import ExpertParallel
+    h, y, res = rnd(T, W), f32(T, W), rnd(T, W)
+    ids, wts = ops.moe_route(f32(T, E), None, 1, K, 8, 4, 1.5)
+    ep = ExpertParallel(None, torch.device(dev), E, W, T * K, status=ops.status_word)
+    work = (E * 3.0 * F * W * 2, 6.0 * T * K * F * W, 1)
+    add(f"grouped experts added in fp32, {T} rows", (lambda j: ep.moe(ops, h, ids, wts, gu, dn, acc=y), *work), "grouped experts + residual",
+        (lambda j: ep.moe(ops, h, ids, wts, gu, dn, res=res), *work))
+    for grp_n, keep in ((8, 4), (16, 5)):
+        z, zl = f32(T, 48 if grp_n == 16 else E), f32(T, E)
+        n = z.shape[1]
+        add(f"router, {n} experts, {keep} of {grp_n} groups, {T} rows", (lambda j: ops.moe_route(z, None, 1, K, grp_n, keep, 1.5), T * (n + 2 * K) * 4.0, 0.0, 1),
+            "router, 4 of 8 groups", (lambda j: ops.moe_route(zl, None, 1, K, 8, 4, 1.5), T * (E + 2 * K) * 4.0, 0.0, 1))
     assert ops.status() == 0
     return acc.rows
