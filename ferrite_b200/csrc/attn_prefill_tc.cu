@@ -282,27 +282,50 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const bool capped = BND && cap_log2 > 0.f;
         if (capped) {
           float am = 0.f;
+          const uint64_t scale2 = f2_pack(scale_log2, scale_log2), cap2 = f2_pack(cap_log2, cap_log2);
+          uint64_t x[HC / 2];
 #pragma unroll
-          for (int c = 0; c < HC; ++c) {
-            const float x = __uint_as_float(sr[c]) * scale_log2;
-            sr[c] = __float_as_uint(x);
-            am = fmaxf(am, fabsf(x));
+          for (int c = 0; c < HC / 2; ++c) {
+            x[c] = f2_mul(f2_pack(__uint_as_float(sr[2 * c]), __uint_as_float(sr[2 * c + 1])), scale2);
+            const float2 v = f2_unpack(x[c]);
+            am = fmaxf(am, fmaxf(fabsf(v.x), fabsf(v.y)));
           }
           if (__any_sync(0xffffffffu, am > 1.f)) {
 #pragma unroll
-            for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(cap_log2 * tanh_exp(__uint_as_float(sr[c])));
+            for (int c = 0; c < HC / 2; ++c) {
+              const float2 v = f2_unpack(x[c]);
+              sr[2 * c] = __float_as_uint(cap_log2 * tanh_exp(v.x));
+              sr[2 * c + 1] = __float_as_uint(cap_log2 * tanh_exp(v.y));
+            }
           } else {
 #pragma unroll
-            for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(cap_log2 * tanh_poly(__uint_as_float(sr[c])));
+            for (int c = 0; c < HC / 2; ++c) {
+              const float2 v = f2_unpack(f2_mul(f2_mul(x[c], cap2), f2_tanh_ratio(x[c])));
+              sr[2 * c] = __float_as_uint(v.x);
+              sr[2 * c + 1] = __float_as_uint(v.y);
+            }
           }
         }
+        if constexpr (BND) {
+          if (!capped) {
 #pragma unroll
-        for (int c = 0; c < HC; ++c) {
-          float v = __uint_as_float(sr[c]);
-          if (!capped) v *= scale_log2;
-          if (need_mask && (t0 + c > qpos || (BND && t0 + c < klo))) v = -INFINITY;
-          sr[c] = __float_as_uint(v);
-          mx = fmaxf(mx, v);
+            for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) * scale_log2);
+          }
+          if (need_mask) {
+#pragma unroll
+            for (int c = 0; c < HC; ++c)
+              if (t0 + c > qpos || t0 + c < klo) sr[c] = __float_as_uint(-INFINITY);
+          }
+#pragma unroll
+          for (int c = 0; c < HC; ++c) mx = fmaxf(mx, __uint_as_float(sr[c]));
+        } else {
+#pragma unroll
+          for (int c = 0; c < HC; ++c) {
+            float v = __uint_as_float(sr[c]) * scale_log2;
+            if (need_mask && t0 + c > qpos) v = -INFINITY;
+            sr[c] = __float_as_uint(v);
+            mx = fmaxf(mx, v);
+          }
         }
       } else {
         fail_s[s] = 1;
@@ -342,14 +365,29 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const float mr = (m_ref == -INFINITY) ? 0.f : m_ref;
       uint32_t pr[HC / 2], px[PX ? HC / 2 : 1];
       float sum = 0.f;
+      uint64_t sum2 = f2_pack(0.f, 0.f);
 #pragma unroll
       for (int c = 0; c < HC / 2; ++c) {
+        if constexpr (BND) {                                  // the same two keys at a time
+          const float2 d = f2_unpack(f2_add(f2_pack(__uint_as_float(sr[2 * c]), __uint_as_float(sr[2 * c + 1])), f2_pack(-mr, -mr)));
+          const float p0 = fast_exp2(d.x), p1 = fast_exp2(d.y);
+          const uint64_t pp = f2_pack(p0, p1);
+          sum2 = f2_add(sum2, pp);
+          pr[c] = pack_bf2(p0, p1);
+          const float2 rest = f2_unpack(f2_add(pp, f2_pack(-bf_lo(pr[c]), -bf_hi(pr[c]))));
+          px[c] = pack_bf2(rest.x, rest.y);
+          continue;
+        }
         const float p0 = fast_exp2(__uint_as_float(sr[2 * c]) - mr);
         const float p1 = fast_exp2(__uint_as_float(sr[2 * c + 1]) - mr);
         sum += p0 + p1;
         __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);     // .x (low half) = even key
         pr[c] = *reinterpret_cast<uint32_t*>(&h);
         if constexpr (PX) px[c] = pack_bf2(p0 - bf_lo(pr[c]), p1 - bf_hi(pr[c]));
+      }
+      if constexpr (BND) {
+        const float2 v = f2_unpack(sum2);
+        sum = v.x + v.y;
       }
       l += sum;
       tmem_st16(tmem + lane_addr + COL_P + s * (FT_BKV / 2) + half * (HC / 2), pr);

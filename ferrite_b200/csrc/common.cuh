@@ -53,17 +53,43 @@ __device__ __forceinline__ float tanh_exp(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.885390081777927f));
   return 1.f - __fdividef(2.f, e + 1.f);
 }
-// tanh(x) for |x| <= 1 on the FMA pipe: x P(x^2), P a weighted least-squares fit of tanh(sqrt u) / sqrt u over [0, 1] with seven terms;
+// Two fp32 lanes in one register pair (sm_100: one instruction for both)
+__device__ __forceinline__ uint64_t f2_pack(float a, float b) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+  return v;
+}
+__device__ __forceinline__ float2 f2_unpack(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t f2_add(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+// tanh(x) / x of two |x| <= 1 on the FMA pipe: P(x^2), P a weighted least-squares fit of tanh(sqrt u) / sqrt u over [0, 1] with seven terms;
 // within 2.1e-7 of the value
-__device__ __forceinline__ float tanh_poly(float x) {
-  const float u = x * x;
-  float p = fmaf(0.00104102225f, u, -0.00620337809f);
-  p = fmaf(p, u, 0.0202899799f);
-  p = fmaf(p, u, -0.0534570292f);
-  p = fmaf(p, u, 0.13325204f);
-  p = fmaf(p, u, -0.333328396f);
-  p = fmaf(p, u, 1.f);
-  return x * p;
+__device__ __forceinline__ uint64_t f2_tanh_ratio(uint64_t x) {
+  const uint64_t u = f2_mul(x, x);
+  auto both = [](float c) { return f2_pack(c, c); };
+  uint64_t p = f2_fma(both(0.00104102225f), u, both(-0.00620337809f));
+  p = f2_fma(p, u, both(0.0202899799f));
+  p = f2_fma(p, u, both(-0.0534570292f));
+  p = f2_fma(p, u, both(0.13325204f));
+  p = f2_fma(p, u, both(-0.333328396f));
+  return f2_fma(p, u, both(1.f));
 }
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
