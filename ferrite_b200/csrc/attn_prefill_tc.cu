@@ -78,8 +78,15 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // P buffer in TMEM), which keeps 16 bits of their mantissa instead of 8.
 // BND: rows see a window or a chunk of the keys, scores are softcapped (cap_log2 = cap * log2 e, scale_log2 then leads to the argument of
 // the tanh, which is a polynomial where all scores of a warp's tile are below the cap). Key tiles that no row of the CTA sees are skipped; out_f32: rows of floats.
+// Two CTAs share an SM where heads have up to 128 columns (`ft_pair`), so that one's waits hide behind the other's arithmetic: fewer K / V
+// buffers, and P and its remainder take the place of the scores they came from (all of them are in registers by then), so that 256 TMEM
+// columns do. The scores of tile j + 2 then wait for PV(j), which read that place, instead of for the softmax threads.
+constexpr bool ft_pair(int hd, bool bnd) { return bnd && hd <= 128; }
+constexpr int ft_k_stages(int hd, bool bnd) { return ft_pair(hd, bnd) ? (hd == 128 ? 2 : 3) : hd == 256 ? 3 : 4; }
+constexpr int ft_v_stages(int hd, bool bnd) { return ft_pair(hd, bnd) ? (hd == 128 ? 2 : 3) : hd == 256 ? 2 : 3; }
+
 template <int HD, bool PX, bool BND>
-__global__ void __launch_bounds__(FT_THREADS, 1)
+__global__ void __launch_bounds__(FT_THREADS, ft_pair(HD, BND) ? 2 : 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
                        const __nv_bfloat16* __restrict__ proj, long proj_stride, const int* __restrict__ seg_slot,
@@ -91,11 +98,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
   constexpr int Q_BYTES = NCH * Q_CH, KV_BYTES = NCH * KV_CH;
-  constexpr uint32_t COL_O = 0, COL_S = HD, COL_P = HD + 2 * FT_BKV;   // TMEM columns: O | S0 S1 | P0 P1 | remainders
-  constexpr uint32_t TMEM_COLS = 512;
+  constexpr bool PAIR = ft_pair(HD, BND);
+  // TMEM columns: O | S0 S1 | P0 P1 | remainders; PAIR: O | S0 S1, P and remainder in the place of their S
+  constexpr uint32_t COL_O = 0, COL_S = HD, COL_P = PAIR ? COL_S : HD + 2 * FT_BKV;
+  constexpr uint32_t P_STEP = PAIR ? FT_BKV : FT_BKV / 2, REM = PAIR ? FT_BKV / 2 : FT_BKV;   // between P buffers; from P to its remainder
+  constexpr uint32_t TMEM_COLS = PAIR ? 256 : 512;
   // K runs three tiles ahead at head_dim 256 (S(j+1) is issued a whole tile before PV(j), so with two K buffers a K
   // load had one tile period to arrive and its latency set the pace), four below; V two / three.
-  constexpr int KS = HD == 256 ? 3 : 4, VS = HD == 256 ? 2 : 3;
+  constexpr int KS = ft_k_stages(HD, BND), VS = ft_v_stages(HD, BND);
   // All shared state lives in the dynamic allocation (no static shared memory), so the tile area starts at the
   // 1024-byte aligned base: [Q][K x KS][V x VS][row maxima 2 KB][barriers][flags]
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -117,8 +127,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   int* abort_p = reinterpret_cast<int*>(tmem_base_p + 1);
   int* fail_s = abort_p + 1;                                // [3]: a softmax wait ran out (tile parity; [2]: after the loop)
 
-  const int seg = blockIdx.z, qh = blockIdx.y;
-  const int qt = (int)gridDim.x - 1 - (int)blockIdx.x;      // long (late) query tiles first
+  // all heads of the long (late) query tiles first, so that the last CTAs to start are short ones
+  const int seg = blockIdx.z, qh = blockIdx.x;
+  const int qt = (int)gridDim.y - 1 - (int)blockIdx.y;
   pdl_launch_dependents();
   pdl_wait();
   const int n = seg_nrows[seg];
@@ -140,7 +151,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     fail_s[0] = fail_s[1] = fail_s[2] = 0;
     mbar_init(q_full, 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], 256); mbar_init(&p_full[i], 256); mbar_init(&p_empty[i], 1);
+      mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], 8); mbar_init(&p_full[i], 8); mbar_init(&p_empty[i], 1);
     }
     for (int i = 0; i < KS; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
     for (int i = 0; i < VS; ++i) { mbar_init(&v_full[i], 1); mbar_init(&v_empty[i], 1); }
@@ -213,7 +224,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       auto issue_s = [&](int j) -> bool {
         const int s = j & 1, st = j % KS;
         if (!mbar_wait_or_flag(&k_full[st], (j / KS) & 1, abort_flag)) return false;
-        if (j >= 2 && !mbar_wait_or_flag(&s_empty[s], ((j >> 1) - 1) & 1, abort_flag)) return false;
+        if (j >= 2 && !mbar_wait_or_flag(PAIR ? &p_empty[s] : &s_empty[s], ((j >> 1) - 1) & 1, abort_flag)) return false;
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < HD / 16; ++kk) {
@@ -234,12 +245,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < FT_BKV / 16; ++kk)
-          tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + s * (FT_BKV / 2) + kk * 8,
+          tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + s * P_STEP + kk * 8,
                         umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
         if (PX) {
 #pragma unroll
           for (int kk = 0; kk < FT_BKV / 16; ++kk)
-            tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + FT_BKV + s * (FT_BKV / 2) + kk * 8,
+            tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + REM + s * P_STEP + kk * 8,
                           umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, 1u);
         }
         tc_commit(&v_empty[st]);
@@ -276,7 +287,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld32(tmem + lane_addr + COL_S + s * FT_BKV + half * HC, sr);
         tmem_ld_wait();
         tc_fence_before();
-        mbar_arrive(&s_empty[s]);
+        if (!PAIR) {                                          // one arrival per softmax warp: its loads are done
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&s_empty[s]);
+        }
         const int t0 = (tile0 + j) * FT_BKV + half * HC;
         const bool need_mask = t0 + HC - 1 > pos0 + q0 || (BND && t0 < klo_last);
         const bool capped = BND && cap_log2 > 0.f;
@@ -390,11 +404,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         sum = v.x + v.y;
       }
       l += sum;
-      tmem_st16(tmem + lane_addr + COL_P + s * (FT_BKV / 2) + half * (HC / 2), pr);
-      if constexpr (PX) tmem_st16(tmem + lane_addr + COL_P + FT_BKV + s * (FT_BKV / 2) + half * (HC / 2), px);
+      tmem_st16(tmem + lane_addr + COL_P + s * P_STEP + half * (HC / 2), pr);
+      if constexpr (PX) tmem_st16(tmem + lane_addr + COL_P + REM + s * P_STEP + half * (HC / 2), px);
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(&p_full[s]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[s]);
     }
     // final hand-over: the row sum of the other half, and agreement on whether the output is complete
     bool ok = !broke && !late_fail;
@@ -478,7 +493,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, FT_BQ))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
-  dim3 grid((max_rows + FT_BQ - 1) / FT_BQ, nq, nseg);
+  dim3 grid(nq, (max_rows + FT_BQ - 1) / FT_BQ, nseg);
   if ((kb || out_f32) && (!exact_p || gated)) return -20;
   if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
   if (ldo == 0) ldo = (long)nq * hd;
@@ -488,7 +503,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   const float scale_log2 = cap > 0.f ? raw_scale / cap : raw_scale * LOG2E;
 #define FB_FT(HDV, PXV, BNDV)                                                                                                 \
   {                                                                                                                \
-    const size_t smem = (size_t)(FT_BQ + ((HDV == 256 ? 3 : 4) + (HDV == 256 ? 2 : 3)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
+    const size_t smem = (size_t)(FT_BQ + (ft_k_stages(HDV, BNDV) + ft_v_stages(HDV, BNDV)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
     auto kern = attn_prefill_tc_kernel<HDV, PXV, BNDV>;                                                                       \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
     if (e != cudaSuccess) return (int)e;                                                                           \

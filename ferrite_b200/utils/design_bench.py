@@ -441,6 +441,12 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     grp = SegGroup(0, 1, 0, T, T, True)
     like = ("prompt attention, bf16 weights", (lambda j: ops.attention_prefill(q, pj, kc, vc, *s0, perm, kvb, H, G, D, False, T), 0.0,
                                                T * (T + 1) / 2.0 * H * 4 * D, 1))
+    # rows see the keys of their chunk as rows of separate prompts of that length see theirs
+    n = T // size
+    parts = (torch.arange(n, dtype=torch.int32, device=dev), torch.arange(0, T, size, dtype=torch.int32, device=dev), i32([size] * n), i32([0] * n))
+    like_chunks = (f"prompt attention, bf16 weights, {n} prompts of {size}",
+                   (lambda j: ops.attention_prefill(q, pj, kc, vc, *parts, perm.view(n, -1), kvb, H, G, D, False, size), 0.0,
+                    n * size * (size + 1) / 2.0 * H * 4 * D, 1))
     for sz in (size, T):
         one, two = replace(one, window=sz), replace(two, chunk=sz)
         seen1, seen2 = sum(min(t + 1, sz) for t in range(T)), sum(t % sz + 1 for t in range(T))
@@ -448,7 +454,7 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
             (lambda j: ops.gqa_attention(q, one, kc, vc, None, grp, rslot, rlen, s0, perm, kvb, 1, out), 0.0, seen1 * H * 4.0 * D, 1), *like)
         add(f"prompt attention and head_mix, two maps, gate, chunk of {sz}, {T} rows",
             (lambda j: ops.gqa_attention(q, two, k2, v2, None, grp, rslot, rlen, s0, perm, kvb, 1, o2, lam=lam, gate=gate, eps=1e-6), 0.0,
-             seen2 * H * 3.0 * D, 1), *like)
+             seen2 * H * 3.0 * D, 1), *(like if sz == T else like_chunks))
     del kc, vc, k2, v2
     # products: both output projections at once, beside the two of the sequential model; in_proj with fp32 sums
     ff = 3 * width
