@@ -358,11 +358,11 @@ def rakizen_config(v: dict) -> ModelConfig:
         kind, m, ff = e["type"], e["mixer"], e.get("mlp")
         if kind not in ("attention", "attention_2"):
             raise ValueError(f"layer {i}: mixer type {kind!r} is neither attention nor attention_2")
-        size = int(m["mask"]["size"])
-        if size < 1 or float(m["softcap"]) <= 0:
-            raise ValueError(f"layer {i}: mask size {size} and softcap {m['softcap']} must be positive")
+        size, cap = int(m["mask"]["size"]), float(m.get("softcap") or 0.0)
+        if size < 1 or cap < 0:
+            raise ValueError(f"layer {i}: mask size {size} or softcap {cap} out of range")
         kw = dict(mixer="gqa", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                  scale=float(m["scale"]), softcap=float(m["softcap"]), act="swiglu")
+                  scale=float(m["scale"]), softcap=cap, act="swiglu")
         if kw["heads"] % kw["kv_heads"]:
             raise ValueError(f"layer {i}: {kw['heads']} heads do not divide over {kw['kv_heads']} key heads")
         if kind == "attention":
@@ -378,7 +378,7 @@ def rakizen_config(v: dict) -> ModelConfig:
             r = ff["router"]
             g = r.get("groups") or {"count": 1, "keep": 1}
             kw.update(ff=int(ff["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=int(g["count"]),
-                      keep_groups=int(g["keep"]), route_scale=float(r["scale"]))
+                      keep_groups=int(g["keep"]), route_scale=float(r.get("scale", 1.0)))
             if kw["experts"] % kw["groups"] or not 1 <= kw["keep_groups"] <= kw["groups"]:
                 raise ValueError(f"layer {i}: {kw['experts']} experts in {kw['groups']} groups, of which {kw['keep_groups']} are kept")
             if not 1 <= kw["top"] <= kw["experts"] // kw["groups"] * kw["keep_groups"]:

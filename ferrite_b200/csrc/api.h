@@ -12,6 +12,16 @@ typedef struct KeyBounds {
   float cap;
 } KeyBounds;
 
+// What follows the two softmax maps of a head: difference (lam: weight of the second, device), norm over vdim with eps, scale, and the sigmoid
+// of gate (rows of heads * vdim fp32 logits ldg apart, or null).
+typedef struct HeadMix {
+  const float* lam;
+  const float* gate;
+  long ldg;
+  float scale, eps;
+  int vdim;
+} HeadMix;
+
 #ifdef __cplusplus
 extern "C" {
 #endif
@@ -132,7 +142,7 @@ int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void
                        long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                        const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg, int max_rows,
                        long q_rows, long cache_rows, int nq, int nkv, int hd, int gated, float scale, int exact_p,
-                       long kv_stride, const float* sink, const KeyBounds* kb, long ldo, int out_f32, int* status, cudaStream_t s);
+                       long kv_stride, const float* sink, const KeyBounds* kb, long ldo, int out_f32, const HeadMix* mix, int* status, cudaStream_t s);
 
 // ---- gdn.cu ----
 int fb_gdn_conv(void* out, const void* proj, long proj_stride, const void* conv_w, const void* conv_state,

@@ -85,7 +85,10 @@ constexpr bool ft_pair(int hd, bool bnd) { return bnd && hd <= 128; }
 constexpr int ft_k_stages(int hd, bool bnd) { return ft_pair(hd, bnd) ? (hd == 128 ? 2 : 3) : hd == 256 ? 3 : 4; }
 constexpr int ft_v_stages(int hd, bool bnd) { return ft_pair(hd, bnd) ? (hd == 128 ? 2 : 3) : hd == 256 ? 2 : 3; }
 
-template <int HD, bool PX, bool BND>
+// DUAL: two softmax maps per head over shared values (a key row holds both maps' keys, a query has zeros in the other's columns). A CTA takes
+// both maps of 64 query rows, map 0 in lanes 0..63 and map 1 in lanes 64..127, and ends with the difference of the two, its norm over vdim,
+// the scale and the output gate: the maps' own rows never leave the SM.
+template <int HD, bool PX, bool BND, bool DUAL>
 __global__ void __launch_bounds__(FT_THREADS, ft_pair(HD, BND) ? 2 : 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
@@ -93,7 +96,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                        const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows,
                        const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
                        int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink, int window, int chunk,
-                       float cap_log2, long ldo, int out_f32, int* status) {
+                       float cap_log2, long ldo, int out_f32, const HeadMix mix, int* status) {
   constexpr int NCH = HD / 64;                     // 64-element (128-byte) chunks of the head dim
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
@@ -133,17 +136,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   pdl_launch_dependents();
   pdl_wait();
   const int n = seg_nrows[seg];
-  const int q0 = qt * FT_BQ;
+  constexpr int QR = DUAL ? FT_BQ / 2 : FT_BQ;              // query rows of the CTA
+  const int q0 = qt * QR;
   if (q0 >= n) return;                                      // uniform for the CTA, before any barrier or allocation
   if (smem_u32(smem_raw) & 1023u) {                         // the swizzled tiles need the 1024-byte base
     if (threadIdx.x == 0) set_status(status, ST_BOUNDS);
     return;
   }
   const int row0 = seg_row0[seg], pos0 = seg_pos0[seg], slot = seg_slot[seg];
-  const int kvh = qh / (nq / nkv);
+  const int kvh = (DUAL ? 2 * qh : qh) / (nq / nkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile0 = BND ? first_key(pos0 + q0, window, chunk) / FT_BKV : 0;   // first key tile that a row of the CTA sees
-  const int nt = (pos0 + min(q0 + FT_BQ, n) + FT_BKV - 1) / FT_BKV - tile0;   // key tiles up to the one the last query row ends in
+  const int nt = (pos0 + min(q0 + QR, n) + FT_BKV - 1) / FT_BKV - tile0;   // key tiles up to the one the last query row ends in
   volatile int* abort_flag = abort_p;
 
   if (threadIdx.x == 0) {
@@ -172,7 +176,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
       mbar_expect_tx(q_full, Q_BYTES);
 #pragma unroll
-      for (int c = 0; c < NCH; ++c) tma_load_2d(sQ + c * Q_CH, &tmQ, q_full, qh * HD + c * 64, row0 + q0);
+      for (int c = 0; c < NCH; ++c) {
+        if constexpr (DUAL) {
+          tma_load_2d(sQ + c * Q_CH, &tmQ, q_full, 2 * qh * HD + c * 64, row0 + q0);
+          tma_load_2d(sQ + c * Q_CH + Q_CH / 2, &tmQ, q_full, (2 * qh + 1) * HD + c * 64, row0 + q0);
+        } else {
+          tma_load_2d(sQ + c * Q_CH, &tmQ, q_full, qh * HD + c * 64, row0 + q0);
+        }
+      }
       const int* bt = block_table + (size_t)slot * max_blocks;
       int k_armed = 0, v_armed = 0;                           // tiles whose K / V loads were issued
       bool ok = true;
@@ -268,9 +279,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int half = (warp - 2) >> 2;
     const int row = quad * 32 + lane;
     const uint32_t lane_addr = (uint32_t)(quad * 32) << 16;
-    const int qpos = pos0 + q0 + row;
+    const int qpos = pos0 + q0 + (DUAL ? row % QR : row);
     const int klo = BND ? first_key(qpos, window, chunk) : 0;
-    const int klo_last = BND ? first_key(pos0 + q0 + FT_BQ - 1, window, chunk) : 0;
+    const int klo_last = BND ? first_key(pos0 + q0 + QR - 1, window, chunk) : 0;
     constexpr int HC = FT_BKV / 2;                          // keys per thread and tile
     constexpr int OC = HD / 2;                              // O columns per thread (rescale, epilogue)
     float m_ref = -INFINITY, l = 0.f;
@@ -425,37 +436,95 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       float lt = l + l_s[half ^ 1][row];
       if (sink) lt += exp2f(sink[qh] * 1.4426950408889634f - m_ref);
       const float inv = lt > 0.f ? 1.f / lt : 0.f;
-      const bool valid = q0 + row < n;
-      const size_t grow = (size_t)(row0 + q0 + row);
-      __nv_bfloat16* dst = out + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
-      float* dst32 = reinterpret_cast<float*>(out) + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
-      const __nv_bfloat16* gate = proj + grow * proj_stride + (size_t)qh * 2 * HD + HD + half * OC;
+      if constexpr (DUAL) {
+        // map 1 hands its rows over through the (now idle) key tiles; map 0 finishes them
+        constexpr int LDX = HD + 4;
+        const int qr = row % QR;
+        float* xs = reinterpret_cast<float*>(sK) + (size_t)qr * LDX + half * OC;
+        float (*ss_s)[FT_BQ] = mx_s[(nt & 1) ^ 1];            // everyone is past the last tile's maxima
+        if (row >= QR) {
 #pragma unroll 1
-      for (int c0 = 0; c0 < OC; c0 += 32) {
-        uint32_t o[32];
-        tmem_ld32(tmem + lane_addr + COL_O + half * OC + c0, o);
-        tmem_ld_wait();
-        if (BND && valid && out_f32) {
+          for (int c0 = 0; c0 < OC; c0 += 32) {
+            uint32_t o[32];
+            tmem_ld32(tmem + lane_addr + COL_O + half * OC + c0, o);
+            tmem_ld_wait();
 #pragma unroll
-          for (int v4 = 0; v4 < 8; ++v4)
-            *reinterpret_cast<float4*>(dst32 + c0 + v4 * 4) =
-                make_float4(__uint_as_float(o[v4 * 4]) * inv, __uint_as_float(o[v4 * 4 + 1]) * inv, __uint_as_float(o[v4 * 4 + 2]) * inv,
-                            __uint_as_float(o[v4 * 4 + 3]) * inv);
-        } else if (valid) {
+            for (int c = 0; c < 32; c += 4)
+              *reinterpret_cast<float4*>(xs + c0 + c) = make_float4(__uint_as_float(o[c]) * inv, __uint_as_float(o[c + 1]) * inv,
+                                                                    __uint_as_float(o[c + 2]) * inv, __uint_as_float(o[c + 3]) * inv);
+          }
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (row < QR) {
+          const float lam = mix.lam[0];
+          float ss = 0.f;
+#pragma unroll 1
+          for (int c0 = 0; c0 < OC; c0 += 32) {
+            uint32_t o[32];
+            tmem_ld32(tmem + lane_addr + COL_O + half * OC + c0, o);
+            tmem_ld_wait();
 #pragma unroll
-          for (int v4 = 0; v4 < 4; ++v4) {
-            uint32_t w[4];
-            uint4 g4 = make_uint4(0, 0, 0, 0);
-            if (gated) g4 = *reinterpret_cast<const uint4*>(gate + c0 + v4 * 8);
-            const uint32_t gu[4] = {g4.x, g4.y, g4.z, g4.w};
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              float a = __uint_as_float(o[v4 * 8 + 2 * e]) * inv, b = __uint_as_float(o[v4 * 8 + 2 * e + 1]) * inv;
-              if (gated) { a *= sigmoidf_(bf_lo(gu[e])); b *= sigmoidf_(bf_hi(gu[e])); }
-              __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-              w[e] = *reinterpret_cast<uint32_t*>(&h);
+            for (int c = 0; c < 32; c += 4) {
+              float4 v = *reinterpret_cast<const float4*>(xs + c0 + c);
+              v.x = __uint_as_float(o[c]) * inv - lam * v.x; v.y = __uint_as_float(o[c + 1]) * inv - lam * v.y;
+              v.z = __uint_as_float(o[c + 2]) * inv - lam * v.z; v.w = __uint_as_float(o[c + 3]) * inv - lam * v.w;
+              ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+              *reinterpret_cast<float4*>(xs + c0 + c) = v;
             }
-            *reinterpret_cast<uint4*>(dst + c0 + v4 * 8) = make_uint4(w[0], w[1], w[2], w[3]);
+          }
+          ss_s[half][qr] = ss;
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        // all threads together, columns of a row side by side
+        const float* xall = reinterpret_cast<const float*>(sK);
+        const int rows_here = min(QR, n - q0);
+        for (int i = threadIdx.x - 64; i < rows_here * (HD / 4); i += 256) {
+          const int xr = i / (HD / 4), d = i % (HD / 4) * 4;
+          const float r = mix.scale / sqrtf((ss_s[0][xr] + ss_s[1][xr]) / (float)mix.vdim + mix.eps);
+          const size_t grow = (size_t)(row0 + q0 + xr);
+          const float4 x = *reinterpret_cast<const float4*>(xall + (size_t)xr * LDX + d);
+          float v[4] = {x.x * r, x.y * r, x.z * r, x.w * r};
+          if (mix.gate) {
+            const float* gate = mix.gate + grow * mix.ldg + (size_t)qh * mix.vdim + d;
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (d + e < mix.vdim) v[e] *= sigmoidf_(gate[e]);
+          }
+          *reinterpret_cast<uint2*>(out + grow * (size_t)ldo + (size_t)qh * HD + d) = make_uint2(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]));
+        }
+      } else {
+        const bool valid = q0 + row < n;
+        const size_t grow = (size_t)(row0 + q0 + row);
+        __nv_bfloat16* dst = out + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
+        float* dst32 = reinterpret_cast<float*>(out) + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
+        const __nv_bfloat16* gate = proj + grow * proj_stride + (size_t)qh * 2 * HD + HD + half * OC;
+#pragma unroll 1
+        for (int c0 = 0; c0 < OC; c0 += 32) {
+          uint32_t o[32];
+          tmem_ld32(tmem + lane_addr + COL_O + half * OC + c0, o);
+          tmem_ld_wait();
+          if (BND && valid && out_f32) {
+#pragma unroll
+            for (int v4 = 0; v4 < 8; ++v4)
+              *reinterpret_cast<float4*>(dst32 + c0 + v4 * 4) =
+                  make_float4(__uint_as_float(o[v4 * 4]) * inv, __uint_as_float(o[v4 * 4 + 1]) * inv, __uint_as_float(o[v4 * 4 + 2]) * inv,
+                              __uint_as_float(o[v4 * 4 + 3]) * inv);
+          } else if (valid) {
+#pragma unroll
+            for (int v4 = 0; v4 < 4; ++v4) {
+              uint32_t w[4];
+              uint4 g4 = make_uint4(0, 0, 0, 0);
+              if (gated) g4 = *reinterpret_cast<const uint4*>(gate + c0 + v4 * 8);
+              const uint32_t gu[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                float a = __uint_as_float(o[v4 * 8 + 2 * e]) * inv, b = __uint_as_float(o[v4 * 8 + 2 * e + 1]) * inv;
+                if (gated) { a *= sigmoidf_(bf_lo(gu[e])); b *= sigmoidf_(bf_hi(gu[e])); }
+                __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+                w[e] = *reinterpret_cast<uint32_t*>(&h);
+              }
+              *reinterpret_cast<uint4*>(dst + c0 + v4 * 8) = make_uint4(w[0], w[1], w[2], w[3]);
+            }
           }
         }
       }
@@ -476,47 +545,52 @@ using namespace fb;
 // q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block] rows of nkv*hd bf16, kv_stride elements
 // apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; sink: a number per q head
 // that joins the softmax denominator, or null; kb: window, chunk and softcap, or null (only with exact_p and a bounded call: fp32 rows,
-// out_f32); ldo: elements between rows of out (0: dense); same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
+// out_f32); mix: what follows two maps per head (nq counts both maps' queries, out has nq / 2 heads), or null; ldo: elements between rows of out (0: dense); same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
 extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                                   long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                                   const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg,
                                   int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int gated,
                                   float scale, int exact_p, long kv_stride, const float* sink, const KeyBounds* kb, long ldo,
-                                  int out_f32, int* status, cudaStream_t s) {
+                                  int out_f32, const HeadMix* mix, int* status, cudaStream_t s) {
   if (nseg <= 0 || max_rows <= 0) return 0;
   if (nq % nkv) return -1;
   if ((hd != 64 && hd != 128 && hd != 256) || kv_block % FT_BKV) return -20;
   if (kv_stride == 0) kv_stride = (long)nkv * hd;
   if (kv_stride % 8) return -20;
+  const int heads = mix ? nq / 2 : nq, q_rows_cta = mix ? FT_BQ / 2 : FT_BQ;
   CUtensorMap tmQ, tmK, tmV;
   int rc;
-  if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, FT_BQ))) return rc;
+  if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, q_rows_cta))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
-  dim3 grid(nq, (max_rows + FT_BQ - 1) / FT_BQ, nseg);
-  if ((kb || out_f32) && (!exact_p || gated)) return -20;
+  dim3 grid(heads, (max_rows + q_rows_cta - 1) / q_rows_cta, nseg);
+  const HeadMix no_mix{};
+  if ((kb || out_f32 || mix) && (!exact_p || gated)) return -20;
+  if (mix && (nq % 2 || (nq / nkv) % 2 || !mix->lam || mix->vdim < 1 || mix->vdim > hd || sink || out_f32)) return -1;
   if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
-  if (ldo == 0) ldo = (long)nq * hd;
+  if (ldo == 0) ldo = (long)heads * hd;
   if (ldo % 8) return -20;
   constexpr float LOG2E = 1.4426950408889634f;
   const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
   const float scale_log2 = cap > 0.f ? raw_scale / cap : raw_scale * LOG2E;
-#define FB_FT(HDV, PXV, BNDV)                                                                                                 \
+#define FB_FT(HDV, PXV, BNDV, DUALV)                                                                                              \
   {                                                                                                                \
     const size_t smem = (size_t)(FT_BQ + (ft_k_stages(HDV, BNDV) + ft_v_stages(HDV, BNDV)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
-    auto kern = attn_prefill_tc_kernel<HDV, PXV, BNDV>;                                                                       \
+    auto kern = attn_prefill_tc_kernel<HDV, PXV, BNDV, DUALV>;                                                                     \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
     if (e != cudaSuccess) return (int)e;                                                                           \
     launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
-               gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, status);                                                                   \
+               gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, mix ? *mix : no_mix, status);                                                                   \
   }
-  if (kb || out_f32) {
-    if (hd == 256) FB_FT(256, true, true) else if (hd == 128) FB_FT(128, true, true) else FB_FT(64, true, true)
+  if (mix) {
+    if (hd == 256) FB_FT(256, true, true, true) else if (hd == 128) FB_FT(128, true, true, true) else FB_FT(64, true, true, true)
+  } else if (kb || out_f32) {
+    if (hd == 256) FB_FT(256, true, true, false) else if (hd == 128) FB_FT(128, true, true, false) else FB_FT(64, true, true, false)
   } else if (exact_p) {
-    if (hd == 256) FB_FT(256, true, false) else if (hd == 128) FB_FT(128, true, false) else FB_FT(64, true, false)
+    if (hd == 256) FB_FT(256, true, false, false) else if (hd == 128) FB_FT(128, true, false, false) else FB_FT(64, true, false, false)
   } else {
-    if (hd == 256) FB_FT(256, false, false) else if (hd == 128) FB_FT(128, false, false) else FB_FT(64, false, false)
+    if (hd == 256) FB_FT(256, false, false, false) else if (hd == 128) FB_FT(128, false, false, false) else FB_FT(64, false, false, false)
   }
 #undef FB_FT
   return (int)cudaGetLastError();

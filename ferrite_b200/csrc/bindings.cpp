@@ -280,7 +280,8 @@ void attn_prefill(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Tensor p
 int64_t attn_prefill_tc(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, Tensor seg_slot, Tensor seg_row0,
                         Tensor seg_nrows, Tensor seg_pos0, Tensor block_table, int64_t kv_block, int64_t max_rows,
                         int64_t nq, int64_t nkv, int64_t hd, bool gated, c10::optional<Tensor> status, double scale,
-                        bool exact_p, c10::optional<Tensor> sink, int64_t window, int64_t chunk, double softcap) {
+                        bool exact_p, c10::optional<Tensor> sink, int64_t window, int64_t chunk, double softcap,
+                        c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t vdim, double eps) {
   // caches: [pages, kv_block, nkv, hd] with dense rows; the rows may lie further apart (k and v side by side in one buffer)
   const long kv_stride = (long)k_cache.stride(1);
   TORCH_CHECK(q.is_contiguous() && v_cache.sizes() == k_cache.sizes() && v_cache.strides() == k_cache.strides() &&
@@ -288,6 +289,11 @@ int64_t attn_prefill_tc(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Te
               "attn_prefill_tc: layouts");
   TORCH_CHECK(out.dim() == 2 || (out.stride(2) == 1 && out.stride(1) == hd), "attn_prefill_tc: out rows");
   const KeyBounds kb{(int)window, (int)chunk, (float)softcap};
+  TORCH_CHECK(!lam || (out.dim() == 3 && out.size(1) * 2 == nq && lam->scalar_type() == torch::kFloat32 &&
+              (!gate || (gate->scalar_type() == torch::kFloat32 && gate->stride(1) == 1 && gate->size(0) == out.size(0) &&
+              gate->size(1) == out.size(1) * vdim))), "attn_prefill_tc: two maps");
+  const HeadMix mix{lam ? lam->data_ptr<float>() : nullptr, gate ? gate->data_ptr<float>() : nullptr, gate ? (long)gate->stride(0) : 0,
+                    (float)mix_scale, (float)eps, (int)vdim};
   int rc = fb_attn_prefill_tc(out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), proj.data_ptr(),
                               (long)proj.stride(0), seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(),
                               seg_nrows.data_ptr<int>(), seg_pos0.data_ptr<int>(), block_table.data_ptr<int>(),
@@ -295,7 +301,8 @@ int64_t attn_prefill_tc(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Te
                               (long)q.size(0), (long)(k_cache.size(0) * k_cache.size(1)), (int)nq, (int)nkv, (int)hd,
                               gated ? 1 : 0, (float)scale, exact_p ? 1 : 0, kv_stride, (const float*)cptr(sink),
                               window || chunk || softcap != 0.0 ? &kb : nullptr, (long)out.stride(0),
-                              out.scalar_type() == torch::kFloat32 ? 1 : 0, (int*)mptr(status), cur_stream());
+                              out.scalar_type() == torch::kFloat32 ? 1 : 0, lam ? &mix : nullptr, (int*)mptr(status),
+                              cur_stream());
   if (rc == -20) return rc;                     // shape outside this kernel: the caller takes the mma.sync kernel
   check(rc, "attn_prefill_tc");
   return 0;
@@ -425,7 +432,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("seg_slot"), py::arg("seg_row0"), py::arg("seg_nrows"), py::arg("seg_pos0"), py::arg("block_table"),
         py::arg("kv_block"), py::arg("max_rows"), py::arg("nq"), py::arg("nkv"), py::arg("hd"), py::arg("gated"), py::arg("status"),
         py::arg("scale") = 0.0, py::arg("exact_p") = false, py::arg("sink") = py::none(), py::arg("window") = 0,
-        py::arg("chunk") = 0, py::arg("softcap") = 0.0);
+        py::arg("chunk") = 0, py::arg("softcap") = 0.0, py::arg("lam") = py::none(), py::arg("gate") = py::none(), py::arg("mix_scale") = 1.0,
+        py::arg("vdim") = 0, py::arg("eps") = 0.0);
   m.def("attn_decode_mma", &attn_decode_mma);
   m.def("gdn_conv", &gdn_conv);
   m.def("gdn_rec", &gdn_rec);

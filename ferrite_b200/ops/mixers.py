@@ -131,7 +131,7 @@ class CudaMixers:
         """Prompt groups go to the tcgen05 flash kernel (softmax weights as value + remainder); the others are split over their keys on
         the mma.sync kernels, over the warps of a CTA as well where a segment brings at most 16 (row, head) pairs per key head. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
         key splits; what is left of it is what fills the GPU and what the layer's mask leaves of the keys. The difference of two maps and
-        the output gate ride on the merge of the splits, or follow the flash kernel in a pass of their own. Rows of `out` may lie apart."""
+        the output gate ride on the merge of the splits and on the flash kernel (a gate over single maps follows that in a pass of its own). Rows of `out` may lie apart."""
         a, b, nq = group.row_lo, group.row_hi, d.queries
         mixed = d.maps == 2 or gate is not None
         bounds = dict(window=d.window, chunk=d.chunk, softcap=d.softcap)
@@ -140,6 +140,12 @@ class CudaMixers:
         if group.prompt and tc and kv_block % 64 == 0:
             self.launches += 1
             flat = q.view(q.shape[0], -1)
+            if d.maps == 2:                                           # both maps of a head in one CTA, which joins them
+                rc = self.C.attn_prefill_tc(out, flat, k_cache, v_cache, flat, segs[0], segs[1], segs[2], segs[3], block_table, kv_block,
+                                            group.max_rows, nq, d.kv_heads, d.hp, False, self.status_word, scale=d.scale, exact_p=True,
+                                            lam=lam, gate=gate, mix_scale=1.0 - d.diff, vdim=d.vw, eps=eps, **bounds)
+                assert rc == 0, "prompt attention: shape outside the tensor-core kernel"
+                return out
             rows = self.empty(q.shape[0], nq, d.hp, dtype=torch.float32, device=self.device) if mixed else out
             rc = self.C.attn_prefill_tc(rows, flat, k_cache, v_cache, flat, segs[0], segs[1], segs[2], segs[3], block_table, kv_block,
                                         group.max_rows, nq, d.kv_heads, d.hp, False, self.status_word, scale=d.scale, exact_p=True, sink=sink,

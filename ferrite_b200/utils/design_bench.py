@@ -452,7 +452,7 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
         seen1, seen2 = sum(min(t + 1, sz) for t in range(T)), sum(t % sz + 1 for t in range(T))
         add(f"prompt attention, softcap, window of {sz}, {T} rows",
             (lambda j: ops.gqa_attention(q, one, kc, vc, None, grp, rslot, rlen, s0, perm, kvb, 1, out), 0.0, seen1 * H * 4.0 * D, 1), *like)
-        add(f"prompt attention and head_mix, two maps, gate, chunk of {sz}, {T} rows",
+        add(f"prompt attention, two maps, difference, gate, chunk of {sz}, {T} rows",
             (lambda j: ops.gqa_attention(q, two, k2, v2, None, grp, rslot, rlen, s0, perm, kvb, 1, o2, lam=lam, gate=gate, eps=1e-6), 0.0,
              seen2 * H * 3.0 * D, 1), *(like if sz == T else like_chunks))
     del kc, vc, k2, v2

@@ -69,12 +69,15 @@ def test_configuration_is_read_and_refused(tmp_path):
     assert c.parallel and c.pre_norm and not c.out_norm and not c.loop_input and c.n_attn == 8 and len(c.layer_runs) == 8
     assert [r.layer for r in c.layer_runs] == plain.order(CASES["ragged"])
     assert read(dict(CASES["bare"], loop=None)).loop is None
+    free = copy.deepcopy(CASES["bare"])
+    free["layers"][0]["mixer"]["softcap"] = None
+    assert read(free).layers[0].softcap == 0.0
     for change, what in (((lambda c: c.update(architecture="Rakizan")), "architecture"),
                          ((lambda c: c["layers"][1].update(type="conv")), "type"),
                          ((lambda c: c["layers"][0]["mlp"].update(kind="routed")), "kind"),
                          ((lambda c: c["layers"][0]["mixer"].update(kv_heads=4)), "heads"),
                          ((lambda c: c["layers"][0]["mixer"]["mask"].update(size=0)), "mask"),
-                         ((lambda c: c["layers"][1]["mixer"].update(softcap=0.0)), "softcap"),
+                         ((lambda c: c["layers"][1]["mixer"].update(softcap=-1.0)), "softcap"),
                          ((lambda c: c["layers"][0]["mixer"]["rot"].update(dims=42)), "rotated"),
                          ((lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(count=5)), "groups"),
                          ((lambda c: c["layers"][1]["mlp"]["router"].update(top=9)), "experts per token"),
