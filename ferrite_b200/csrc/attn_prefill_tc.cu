@@ -96,7 +96,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                        const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows,
                        const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
                        int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink, int window, int chunk,
-                       float cap_log2, long ldo, int out_f32, const HeadMix mix, int* status) {
+                       float cap_log2, long ldo, int out_f32, const HeadMix mix, int head_groups, int* status) {
   constexpr int NCH = HD / 64;                     // 64-element (128-byte) chunks of the head dim
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
@@ -130,11 +130,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   int* abort_p = reinterpret_cast<int*>(tmem_base_p + 1);
   int* fail_s = abort_p + 1;                                // [3]: a softmax wait ran out (tile parity; [2]: after the loop)
 
-  // all heads of the long (late) query tiles first, so that the last CTAs to start are short ones
-  const int seg = blockIdx.z, qh = blockIdx.x;
+  // the long (late) query tiles of a group of heads first, so that the last CTAs to start are short ones; one group after another keeps
+  // the keys and values in use few enough for L2
+  const int seg = blockIdx.z / head_groups, qh = blockIdx.z % head_groups * gridDim.x + blockIdx.x;
   const int qt = (int)gridDim.y - 1 - (int)blockIdx.y;
   pdl_launch_dependents();
   pdl_wait();
+  if (qh >= (DUAL ? nq / 2 : nq)) return;
   const int n = seg_nrows[seg];
   constexpr int QR = DUAL ? FT_BQ / 2 : FT_BQ;              // query rows of the CTA
   const int q0 = qt * QR;
@@ -563,7 +565,12 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, q_rows_cta))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
-  dim3 grid(heads, (max_rows + q_rows_cta - 1) / q_rows_cta, nseg);
+  // up to four waves of CTAs are one group; more go in groups of about two waves, whole sets of query heads that share keys
+  const int q_tiles = (max_rows + q_rows_cta - 1) / q_rows_cta, share = heads / nkv > 0 ? heads / nkv : 1;
+  const int slots = 148 * (ft_pair(hd, kb || out_f32 || mix) ? 2 : 1);
+  const int few = (2 * slots / q_tiles + share) / share * share;
+  const int group = (long)heads * q_tiles <= 4 * slots || few > heads ? heads : few, head_groups = (heads + group - 1) / group;
+  dim3 grid(group, q_tiles, nseg * head_groups);
   const HeadMix no_mix{};
   if ((kb || out_f32 || mix) && (!exact_p || gated)) return -20;
   if (mix && (nq % 2 || (nq / nkv) % 2 || !mix->lam || mix->vdim < 1 || mix->vdim > hd || sink || out_f32)) return -1;
@@ -581,7 +588,7 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
     if (e != cudaSuccess) return (int)e;                                                                           \
     launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
-               gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, mix ? *mix : no_mix, status);                                                                   \
+               gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, mix ? *mix : no_mix, head_groups, status);                                                                   \
   }
   if (mix) {
     if (hd == 256) FB_FT(256, true, true, true) else if (hd == 128) FB_FT(128, true, true, true) else FB_FT(64, true, true, true)

@@ -375,6 +375,15 @@ def test_expert_counters(monkeypatch, tmp_path):
     assert {i: sum(v) for i, v in heat.items()} == {1: 2 * 10 * 2, 3: 10 * 2} and all(len(v) == 7 for v in heat.values())
 
 
+def test_index_checks_cover_the_ops(monkeypatch):
+    monkeypatch.setenv("FB_DEBUG_BOUNDS", "1")
+    eng = Engine(tiny_rakizen(), None, EngineConfig(n_slots=1, max_ctx=64), device="cpu")
+    eng.forward([Segment(0, 0, list(range(10)), "last")])
+    assert {"embed_grams", "gqa_prep", "gqa_attention", "expert_rows"} <= set(eng.bounds.checked)
+    with pytest.raises(IndexError, match="experts of the layer"):
+        eng.ex.ops.expert_rows(torch.zeros(1, 192), i32([[6]]), torch.zeros(6, 128, 192), torch.zeros(6, 192, 64))
+
+
 def test_reference_model_agrees():
     cfg = tiny_rakizen()
     w = init_weights(cfg, seed=4, std=0.1)
