@@ -509,12 +509,12 @@ def rakizen(width: int, n_layers: int, heads: int, kv_heads: int, ff: int, vocab
             loop: Optional[List[int]] = None, name: str = "rakizen") -> ModelConfig:
     """A Rakizen model in which every `every`-th layer takes the difference of two maps (half the heads, twice the value width), the
     others a window; with `experts`, every `moe_every`-th layer has a routed feed-forward."""
-    common = dict(mixer="gqa", act="swiglu", softcap=50.0)
+    common = dict(mixer="gqa", act="swiglu", softcap=30.0)
     win = LayerSpec(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, window=window, row_norm=True, rot_dims=dim,
-                    rot_base=1e6, ff=ff, **common)
+                    rot_base=5e5, ff=ff, **common)
     two = LayerSpec(heads=heads // 2, kv_heads=max(1, kv_heads // 2), dim=dim // 2, vdim=dim, scale=(dim // 2) ** -0.5, chunk=chunk, maps=2,
-                    diff=0.6, out_gate=True, ff=ff, **common)
-    moe = dict(ff=expert_ff, experts=experts, top=top, groups=groups, keep_groups=keep, route_scale=1.5) if experts else {}
+                    diff=0.5, out_gate=True, ff=ff, **common)
+    moe = dict(ff=expert_ff, experts=experts, top=top, groups=groups, keep_groups=keep, route_scale=2.0) if experts else {}
     layers = [dataclasses.replace(two if i % every == every - 1 else win, **(moe if i % moe_every == moe_every - 1 else {})) for i in range(n_layers)]
     return ModelConfig(name=name, hidden=width, inter=ff, n_layers=n_layers, n_q=heads, n_kv=kv_heads, head_dim=dim, eps=1e-6, vocab=vocab,
                        attn_gate=False, tie_embeddings=False, layers=layers, pre_norm=True, parallel=True, loop=loop, loop_input=False)

@@ -57,7 +57,7 @@ def pair_rakizen(size: str):
               tie_embeddings=False)
     if experts:
         return a, ModelConfig(inter=ff, n_experts=experts, top_k=top, expert_inter=ff, router="sigmoid_group", n_groups=groups, topk_groups=keep,
-                              route_scale=1.5, **kw)
+                              route_scale=2.0, **kw)
     spare = a.param_count() - ModelConfig(inter=0, **kw).param_count()
     return a, ModelConfig(inter=max(256, round(spare / (3 * w * n) / 128) * 128), **kw)
 
@@ -379,8 +379,8 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
     f32 = lambda *s: torch.randn(*s, device=dev)
     inv, inv64 = torch.rand(D // 2, device=dev), torch.rand(D // 2, device=dev, dtype=torch.float64)
-    one = GqaDims(H, G, D, D, D ** -0.5, D, (H + G) * D, False, D, 1, True, 50.0, size)
-    two = GqaDims(H // 2, G // 2, D // 2, D, (D // 2) ** -0.5, 0, (H + G) * D // 2, False, D, 2, False, 50.0, 0, size, 0.6, (H + G) * D // 2 + G * D // 2)
+    one = GqaDims(H, G, D, D, D ** -0.5, D, (H + G) * D, False, D, 1, True, 30.0, size)
+    two = GqaDims(H // 2, G // 2, D // 2, D, (D // 2) ** -0.5, 0, (H + G) * D // 2, False, D, 2, False, 30.0, 0, size, 0.5, (H + G) * D // 2 + G * D // 2)
     nw, lam = rnd(D), torch.full((1,), 0.7, device=dev)
     for m in (1, 16, prompt):
         bufs = max(1, min(8, (400 << 20) // (m * width * 4)))
@@ -477,7 +477,7 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     gu, dn = rnd(E, 2 * F, W, scale=0.02), rnd(E, W, F, scale=0.02)
     for m in (1, 4, 16):
         h, x, y, res = rnd(m, W), f32(m, W), f32(m, W), rnd(m, W)
-        picks = [ops.moe_route(f32(m, E), None, 1, K, 8, 4, 1.5) for _ in range(16)]
+        picks = [ops.moe_route(f32(m, E), None, 1, K, 8, 4, 2.0) for _ in range(16)]
         used = sum(len(set(ids.reshape(-1).tolist())) for ids, _ in picks) / 16
         w32 = torch.ones(W, device=dev)
         work = (used * 3.0 * F * W * 2, 6.0 * m * K * F * W, 16)
@@ -486,7 +486,7 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
             "moe_experts (pairs, combine)", (lambda j: ops.moe_experts(h, *picks[j], gu, dn, 0, E, None, None, res), *work))
     from ..parallel.ep import ExpertParallel
     h, y, res = rnd(T, W), f32(T, W), rnd(T, W)
-    ids, wts = ops.moe_route(f32(T, E), None, 1, K, 8, 4, 1.5)
+    ids, wts = ops.moe_route(f32(T, E), None, 1, K, 8, 4, 2.0)
     ep = ExpertParallel(None, torch.device(dev), E, W, T * K, status=ops.status_word)
     work = (E * 3.0 * F * W * 2, 6.0 * T * K * F * W, 1)
     add(f"grouped experts added in fp32, {T} rows", (lambda j: ep.moe(ops, h, ids, wts, gu, dn, acc=y), *work), "grouped experts + residual",
@@ -494,7 +494,7 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
     for grp_n, keep in ((8, 4), (16, 5)):
         z, zl = f32(T, 48 if grp_n == 16 else E), f32(T, E)
         n = z.shape[1]
-        add(f"router, {n} experts, {keep} of {grp_n} groups, {T} rows", (lambda j: ops.moe_route(z, None, 1, K, grp_n, keep, 1.5), T * (n + 2 * K) * 4.0, 0.0, 1),
-            "router, 4 of 8 groups", (lambda j: ops.moe_route(zl, None, 1, K, 8, 4, 1.5), T * (E + 2 * K) * 4.0, 0.0, 1))
+        add(f"router, {n} experts, {keep} of {grp_n} groups, {T} rows", (lambda j: ops.moe_route(z, None, 1, K, grp_n, keep, 2.0), T * (n + 2 * K) * 4.0, 0.0, 1),
+            "router, 4 of 8 groups", (lambda j: ops.moe_route(zl, None, 1, K, 8, 4, 2.0), T * (E + 2 * K) * 4.0, 0.0, 1))
     assert ops.status() == 0
     return acc.rows

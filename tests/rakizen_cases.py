@@ -9,7 +9,7 @@ def dense(ff):
     return {"kind": "dense", "ff": ff}
 
 
-def moe(experts, top, groups, keep, ff, scale=1.5):
+def moe(experts, top, groups, keep, ff, scale=1.3):
     return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale, "groups": {"count": groups, "keep": keep}}}
 
 

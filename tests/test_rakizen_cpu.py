@@ -265,7 +265,7 @@ def test_every_part_shows_in_the_logits(models):
                    lambda c: c["layers"][0]["mixer"]["mask"].update(size=18), lambda c: c["layers"][1]["mixer"]["mask"].update(size=34),
                    lambda c: c["layers"][2]["mixer"]["mask"].update(size=71), lambda c: c["layers"][3]["mixer"]["mask"].update(size=89),
                    lambda c: c["layers"][0]["mixer"].update(softcap=12.0), lambda c: c["layers"][3]["mixer"].update(softcap=18.0),
-                   lambda c: c["layers"][1]["mixer"].update(diff=0.41), lambda c: c["layers"][1]["mlp"]["router"].update(scale=1.51),
+                   lambda c: c["layers"][1]["mixer"].update(diff=0.41), lambda c: c["layers"][1]["mlp"]["router"].update(scale=1.32),
                    lambda c: c["layers"][3]["mlp"]["router"]["groups"].update(keep=4), lambda c: c["layers"][3]["mlp"]["router"].update(top=3),
                    lambda c: c["norm"].update(eps=2e-3)):
         other = copy.deepcopy(cfg)
