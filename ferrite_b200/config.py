@@ -20,46 +20,56 @@ class LayerSpec:
     """One layer of a model that lists its layers one by one (`ModelConfig.layers`): the mixer, its sizes and the
     feed-forward behind it. Layers of one model may differ in all of them."""
 
-    # "latent": attention over a cached low-rank latent, no positions. "gqa": grouped-query attention over cached keys and
-    # values. "cdelta": gated delta rule with one decay per key channel (recurrent state, no cache)
+    # "latent": attention over a cached low-rank latent, without positions or with one rotated key part beside the latent. "gqa":
+    # grouped-query attention over cached keys and values. "cdelta": gated delta rule with one decay per key channel (recurrent state,
+    # no cache). "ssm": state-space duality (Mamba-2): a state per head with one decay, inputs convolved
     mixer: str = "latent"
     heads: int = 1
-    dim: int = 0                    # query / key width of a head
+    dim: int = 0                    # query / key width of a head (latent with rotation: its unrotated part; ssm: width of the state)
     vdim: int = 0                   # value width of a head
-    q_rank: int = 0                 # the queries come out of a normalised latent of this width
+    q_rank: int = 0                 # the queries come out of a normalised latent of this width (0: straight out of the input)
     kv_rank: int = 0                # width of the cached latent
     scale: float = 1.0              # scores are (q . k) * scale
-    kv_from: Optional[int] = None   # use the latents that this (earlier) layer caches instead of own ones
+    kv_from: Optional[int] = None   # use the latents (gqa: keys and values) that this (earlier) layer caches instead of own ones
     ff: int = 0                     # feed-forward width, 0 = the layer has none
-    act: str = "relu2"              # its activation; "swiglu": silu(gate) * up
-    experts: int = 0                # the feed-forward is a mixture of this many swiglu experts of width `ff` ...
+    # its activation; "swiglu": silu(gate) * up; "clamped_glu": with g = min(gate, limit) and u = up clamped to +- limit,
+    # g * sigmoid(1.702 g) * (u + 1)
+    act: str = "relu2"
+    limit: float = 0.0
+    experts: int = 0                # the feed-forward is a mixture of this many experts (swiglu or clamped_glu) of width `ff` ...
     top: int = 0                    # ... of which a token takes the `top` best (sigmoid scores) ...
     groups: int = 1                 # ... among the best `keep_groups` of `groups` groups of neighbours ...
     keep_groups: int = 1
     route_scale: float = 1.0        # ... weighted by their share of the chosen scores times this
-    kv_heads: int = 0               # gqa, cdelta: key / value (cdelta: query / key) heads, each serving heads / kv_heads heads
+    router: str = "sigmoid"         # "softmax": the largest logits, weighted by the softmax over the chosen ones (no groups)
+    shared_ff: int = 0              # width of an expert that every token takes as well, times the sigmoid of a product; 0 = none
+    shared_limit: float = 0.0       # ... and its limit
+    kv_heads: int = 0               # gqa, cdelta, ssm: key / value (cdelta: query / key; ssm: input / output) heads, each serving heads / kv_heads heads
     bias: bool = False              # gqa: biases on the query, key and output projections
     sink: bool = False              # gqa: a learned number per head in every softmax denominator
     key_values: bool = False        # gqa: the values are the projected keys, before rotation and norm
     qk_norm: bool = False           # gqa: queries and keys divided by their root mean square after the rotation
     row_norm: bool = False          # gqa: RMS norms with weights over a whole row of queries and of keys, before the rotation
     softcap: float = 0.0            # gqa: scores <- cap * tanh(scores / cap), 0 = off
-    window: int = 0                 # gqa: a row sees itself and the window - 1 positions before it, 0 = all of them
+    window: int = 0                 # gqa, latent: a row sees itself and the window - 1 positions before it, 0 = all of them
+    pool: int = 0                   # gqa, window: blocks of this many positions that lie before the window are seen as their mean key and value
     chunk: int = 0                  # gqa: a row sees the positions of its own chunk of this many, counted from 0
     maps: int = 1                   # gqa: 2 = differential: two softmax maps per head over shared values, their weighted difference
     diff: float = 0.0               # gqa, two maps: constant of the difference's weight; 1 - diff scales its normed rows
     out_gate: bool = False          # gqa: the heads' outputs are multiplied by the sigmoid of a projection of the mixer's input
-    rot_dims: int = 0               # gqa: rotated columns of a head, pairs (0, 1), (2, 3), ...
+    rot_dims: int = 0               # gqa: rotated columns of a head, pairs (0, 1), (2, 3), ...; latent: width of the rotated part
+    rot_half: bool = False          # gqa: pairs (i, i + rot_dims / 2) instead
     rot_base: float = 1e4
     rot_scaling: Optional[dict] = None   # long wavelengths stretched: factor, low, high, original
-    conv: int = 0                   # cdelta: taps of the short convolutions
+    conv: int = 0                   # cdelta, ssm: taps of the short convolutions
+    norm_groups: int = 1            # ssm: parts of the gated output, each normed by its own root mean square
     decay_rank: int = 0             # cdelta: width between the two decay projections (0: the checkpoint says)
     gate_rank: int = 0              # cdelta: ... and between the two output gate projections
 
     @property
     def cached(self) -> bool:
         """The layer keeps rows of its own in the page pool."""
-        return self.mixer != "cdelta" and self.kv_from is None
+        return self.mixer not in ("cdelta", "ssm") and self.kv_from is None
 
 
 @dataclass(frozen=True)
@@ -117,6 +127,9 @@ class ModelConfig:
     layers: List[LayerSpec] = field(default_factory=list)
     out_norm: bool = False          # x + norm(f(x)): norms on the sublayers' outputs, a 32-bit residual stream, plain norm weights
     pre_norm: bool = False          # ... and norms on the sublayers' inputs as well: x + norm(f(norm(x)))
+    layer_norm: bool = False        # ... and these norms take the mean off (weights, no biases)
+    canon: int = 0                  # what a sublayer reads is h + causal convolution of h with this many taps per channel, 0 = h
+    depth_average: bool = False     # after a layer, x becomes a weighted sum of the embedding output and all layers' results so far
     parallel: bool = False          # x + (mixer(norm(x)) + f(norm(x))): one layer norm (with bias) ahead of both sublayers, none behind
     residual_mult: float = 1.0      # x + residual_mult * norm(f(..))
     loop: Optional[List[int]] = None     # [start, stop, times]: layers start .. stop - 1 run `times` times in a row
@@ -196,18 +209,22 @@ class ModelConfig:
             n += 2 * h * h if self.loop and self.loop_input else 0
             for l in self.layers:
                 if l.mixer == "gqa":
-                    n += h * (l.maps * l.dim * (l.heads + l.kv_heads) + l.vdim * ((2 if l.out_gate else 1) * l.heads + (0 if l.key_values else l.kv_heads)))
+                    own = l.kv_heads if l.kv_from is None else 0
+                    n += h * (l.maps * l.dim * (l.heads + own) + l.vdim * ((2 if l.out_gate else 1) * l.heads + (0 if l.key_values else own)))
                 elif l.mixer == "cdelta":
                     n += h * (2 * l.kv_heads * l.dim + 2 * l.heads * l.vdim + l.heads) + (2 * l.kv_heads * l.dim + l.heads * l.vdim) * l.conv
                     n += l.decay_rank * (h + l.heads * l.dim) + l.gate_rank * (h + l.heads * l.vdim)
+                elif l.mixer == "ssm":
+                    n += h * (3 * l.heads * l.vdim + 2 * l.kv_heads * l.dim + l.heads) + (l.heads * l.vdim + 2 * l.kv_heads * l.dim) * l.conv
+                else:
+                    qd = l.heads * (l.dim + l.rot_dims)
+                    n += (h * l.q_rank + l.q_rank * qd if l.q_rank else h * qd) + l.heads * (l.dim + l.vdim) * l.kv_rank + l.heads * l.vdim * h
+                    n += h * (l.kv_rank + l.rot_dims) if l.kv_from is None else 0
+                n += h * self.canon * (2 if l.ff else 1)
                 if l.experts:
-                    n += l.experts * (h + 3 * h * l.ff)
-                    continue
-                if l.mixer != "latent":
+                    n += l.experts * (h + 3 * h * l.ff) + (h * (3 * l.shared_ff + 1) if l.shared_ff else 0)
+                else:
                     n += (3 if l.act == "swiglu" else 2) * h * l.ff
-                    continue
-                n += h * l.q_rank + l.q_rank * l.heads * l.dim + l.heads * (l.dim + l.vdim) * l.kv_rank + l.heads * l.vdim * h
-                n += (h * l.kv_rank if l.kv_from is None else 0) + 2 * h * l.ff
             return n
         for i, kind in enumerate(self.layer_kinds):
             if kind == "gdn":
@@ -232,8 +249,8 @@ class ModelConfig:
         if world == 1:
             return c
         if self.layers:
-            if self.parallel:
-                raise ValueError("models of parallel blocks run on one rank: their query and key norms span all heads")
+            if self.parallel or self.canon or any(l.row_norm or l.mixer == "ssm" for l in self.layers):
+                raise ValueError("models of parallel blocks, convolved inputs or norms that span all heads run on one rank")
             assert all(l.heads % world == 0 and l.kv_heads % world == 0 and l.ff % world == 0 for l in self.layers), \
                 f"heads and feed-forward widths must divide over {world} ranks"
             c.layers = [dataclasses.replace(l, heads=l.heads // world, kv_heads=l.kv_heads // world, ff=l.ff // world) for l in self.layers]
@@ -396,7 +413,62 @@ def rakizen_config(v: dict) -> ModelConfig:
         loop=[int(lp[k]) for k in ("start", "stop", "times")] if lp else None, loop_input=False)
 
 
-ARCHITECTURES = {"Zototar": zototar_config, "Dofunex": dofunex_config, "Rakizen": rakizen_config}
+def pironex_config(v: dict) -> ModelConfig:
+    """A Pironex config.json: layer norms on both sides of every sublayer, convolved inputs, a learned average over depth; "attention" over a
+    window and the means of the blocks before it (keys optionally another layer's), "latent_attention" with a rotated key part under a
+    window, "mamba2"; routed feed-forwards of clamped gated units with a shared expert; logits over the embedding table."""
+    layers: List[LayerSpec] = []
+    for i, e in enumerate(v["layers"]):
+        kind, m, ff = e["type"], e["mixer"], e.get("mlp")
+        kw = dict(heads=int(m["heads"]), vdim=int(m["vdim"]))
+        if kind in ("attention", "latent_attention"):
+            rot, mask = m.get("rot") or {}, m["mask"]
+            kw.update(dim=int(m["dim"]), scale=float(m["scale"]), window=int(mask["size"]), rot_dims=int(rot.get("dims", 0)),
+                      rot_base=float(rot.get("base", 1e4)))
+            if kw["window"] < 1 or kw["rot_dims"] % 2:
+                raise ValueError(f"layer {i}: mask size {kw['window']} or {kw['rot_dims']} rotated dimensions out of range")
+        if kind == "attention":
+            kw.update(mixer="gqa", kv_heads=int(m["kv_heads"]), row_norm=True, rot_half=True, softcap=float(m.get("softcap") or 0.0),
+                      pool=int(mask.get("pool") or 0))
+            src = m.get("kv_from")
+            if kw["heads"] % kw["kv_heads"]:
+                raise ValueError(f"layer {i}: {kw['heads']} heads do not divide over {kw['kv_heads']} key heads")
+            if kw["rot_dims"] > kw["dim"] or kw["softcap"] < 0 or kw["pool"] < 0:
+                raise ValueError(f"layer {i}: {kw['rot_dims']} rotated dimensions of {kw['dim']}, softcap or pool out of range")
+            if src is not None:
+                o = layers[int(src)] if 0 <= int(src) < i else None
+                if o is None or o.mixer != "gqa" or o.kv_from is not None or (o.kv_heads, o.dim, o.vdim) != (kw["kv_heads"], kw["dim"], kw["vdim"]):
+                    raise ValueError(f"layer {i}: kv_from {src} must name an earlier attention layer with keys of its own and the same key heads and widths")
+                kw["kv_from"] = int(src)
+        elif kind == "latent_attention":
+            kw.update(mixer="latent", kv_rank=int(m["kv_rank"]))
+            if kw["rot_dims"] != int(m["rot_dim"]):
+                raise ValueError(f"layer {i}: the rotated part has rot_dim {m['rot_dim']} dimensions, not {kw['rot_dims']}")
+        elif kind == "mamba2":
+            kw.update(mixer="ssm", dim=int(m["state"]), kv_heads=int(m["groups"]), conv=int(m["conv"]), norm_groups=int(m["norm_groups"]))
+            if kw["heads"] % kw["kv_heads"] or kw["heads"] * kw["vdim"] % kw["norm_groups"]:
+                raise ValueError(f"layer {i}: {kw['heads']} heads over {kw['kv_heads']} groups, {kw['norm_groups']} norm groups")
+        else:
+            raise ValueError(f"layer {i}: mixer type {kind!r} is none of attention, latent_attention, mamba2")
+        if ff:
+            if ff["kind"] != "moe":
+                raise ValueError(f"layer {i}: feed-forward kind {ff['kind']!r} is not moe")
+            r, sh = ff["router"], ff.get("shared")
+            kw.update(ff=int(ff["expert"]["ff"]), limit=float(ff["expert"]["limit"]), act="clamped_glu", router="softmax", experts=int(r["experts"]),
+                      top=int(r["top"]))
+            if not 1 <= kw["top"] <= kw["experts"]:
+                raise ValueError(f"layer {i}: {kw['top']} of {kw['experts']} experts per token")
+            if sh:
+                kw.update(shared_ff=int(sh["ff"]), shared_limit=float(sh["limit"]))
+        layers.append(LayerSpec(**kw))
+    return ModelConfig(
+        name="pironex", hidden=int(v["width"]), inter=max([l.ff for l in layers] + [0]), n_layers=len(layers), n_q=layers[0].heads,
+        n_kv=max(1, layers[0].kv_heads), head_dim=layers[0].dim, eps=float(v["norm"]["eps"]), vocab=int(v["vocab"]), attn_gate=False,
+        tie_embeddings=True, layers=layers, out_norm=True, pre_norm=True, layer_norm=True, canon=int((v.get("canon") or {}).get("taps", 0)),
+        depth_average=True, embed_scale=float((v.get("embedding") or {}).get("scale", 1.0)))
+
+
+ARCHITECTURES = {"Zototar": zototar_config, "Dofunex": dofunex_config, "Rakizen": rakizen_config, "Pironex": pironex_config}
 
 
 # ---- presets: the five benchmark configurations ----------------------------------------------------
@@ -534,7 +606,42 @@ def rakizen_7b() -> ModelConfig:
     return rakizen(4096, 32, 32, 8, 12288, 129280, name="rakizen-7b")
 
 
+def pironex(width: int, n_layers: int, heads: int, kv_heads: int, vocab: int, dim: int = 128, kv_rank: int = 512, rot_dim: int = 64,
+            state: int = 128, groups: int = 1, ssm_heads: int = 0, ssm_vdim: int = 64, window: int = 1024, pool: int = 16, experts: int = 64,
+            top: int = 6, expert_ff: int = 1024, shared_ff: int = 1024, name: str = "pironex") -> ModelConfig:
+    """A Pironex model that repeats latent attention, pooled attention (every second one with the keys of the one before it), and two
+    state-space layers."""
+    ff = dict(ff=expert_ff, act="clamped_glu", limit=7.0, experts=experts, top=top, router="softmax", shared_ff=shared_ff, shared_limit=7.0)
+    lat = LayerSpec(mixer="latent", heads=heads, dim=dim, vdim=dim, kv_rank=kv_rank, rot_dims=rot_dim, rot_base=1e4, window=window,
+                    scale=(dim + rot_dim) ** -0.5, **ff)
+    att = LayerSpec(mixer="gqa", heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, row_norm=True, rot_half=True, rot_dims=dim // 2,
+                    rot_base=1e6, softcap=50.0, window=window, pool=pool, **ff)
+    ssm = LayerSpec(mixer="ssm", heads=ssm_heads or 2 * width // ssm_vdim, vdim=ssm_vdim, dim=state, kv_heads=groups, conv=4, norm_groups=groups, **ff)
+    layers = [dataclasses.replace((lat, att, ssm, ssm)[i % 4]) for i in range(n_layers)]
+    for i in range(5, n_layers, 8):
+        layers[i].kv_from = i - 4
+    return ModelConfig(name=name, hidden=width, inter=expert_ff, n_layers=n_layers, n_q=heads, n_kv=kv_heads, head_dim=dim, eps=1e-5, vocab=vocab,
+                       attn_gate=False, tie_embeddings=True, layers=layers, out_norm=True, pre_norm=True, layer_norm=True, canon=4, depth_average=True,
+                       embed_scale=width ** 0.5)
+
+
+def tiny_pironex() -> ModelConfig:
+    """6-layer plumbing model of the pooled-attention / state-space family: unequal layers, sizes off the kernels' tile grid."""
+    c = pironex(136, 6, 4, 2, 300, dim=40, kv_rank=72, rot_dim=20, state=24, groups=2, ssm_heads=4, ssm_vdim=36, window=24, pool=5, experts=6, top=2,
+                expert_ff=44, shared_ff=60, name="tiny-pironex")
+    c.layers[3] = dataclasses.replace(c.layers[3], heads=6, kv_heads=3, vdim=20, dim=40, conv=3, norm_groups=4, ff=0, experts=0, top=0, shared_ff=0)
+    c.layers[4] = dataclasses.replace(c.layers[4], heads=3, dim=24, vdim=56, kv_rank=136, rot_dims=8, window=70)
+    c.layers[5] = dataclasses.replace(c.layers[5], pool=7, window=31, softcap=0.0)
+    return c
+
+
+def pironex_moe() -> ModelConfig:
+    """24-layer Pironex model of width 2048, 64 experts of 1024 with 6 per token and a shared one."""
+    return pironex(2048, 24, 16, 4, 129280, name="pironex-moe")
+
+
 PRESETS = {
+    "tiny-pironex": tiny_pironex, "pironex-moe": pironex_moe,
     "tiny-rakizen": tiny_rakizen, "rakizen-7b": rakizen_7b,
     "tiny-dofunex": tiny_dofunex, "dofunex-7b": dofunex_7b,
     "tiny-zototar": tiny_zototar, "zototar-7b": zototar_7b,

@@ -92,6 +92,14 @@ __device__ __forceinline__ uint64_t f2_tanh_ratio(uint64_t x) {
   return f2_fma(p, u, both(1.f));
 }
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + __expf(-x)); }
+// gate of a gated unit: silu(g) * u, or with a limit the clamped form min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u) + 1)
+__device__ __forceinline__ float glu_act(float g, float u, float limit) {
+  if (limit > 0.f) {
+    g = fminf(g, limit);
+    return g * sigmoidf_(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+  return siluf_(g) * u;
+}
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(__expf(x)); }
 
 // activation a linear's epilogue may apply to its fp32 sums

@@ -139,12 +139,12 @@ extern "C" int fb_ag_gemm(void* Y, const void* W, const void* res, int M, int N,
 }
 
 // ---- grouped GEMM over expert-sorted rows (mixture of experts, prompt-sized) ------------------------------------
-// Y[r][N] = X[r][K] W[e(r)][N or 2N][K]^T (+ SwiGLU) for the rows r of every expert e: rows are contiguous per
+// Y[r][N] = X[r][K] W[e(r)][N or 2N][K]^T (+ SwiGLU, or with a limit clamped gated units) for the rows r of every expert e: rows are contiguous per
 // expert, `row_base` / `tile_start` are device-side prefix sums (experts + 1 entries) so the call needs no host
 // synchronisation. `max_rows` bounds the rows (the tensor map's extent). Counterpart of the reference's segmented
 // prompt GEMM over sorted (token, expert) pairs (`ggq_mmq_moe*`, `kernels/k-gguf/src/mmq.rs:522`).
 extern "C" int fb_gemm_grouped(void* Y, const void* X, const void* W, const int* tile_start, const int* row_base,
-                               int experts, int max_rows, int N, int K, long ldx, long ldy, int mode, int* status,
+                               int experts, int max_rows, int N, int K, long ldx, long ldy, int mode, float limit, int* status,
                                int sm_count, cudaStream_t s) {
   if (experts <= 0 || max_rows <= 0) return 0;
   if (K % 8 || ldx % 8 || ldy % 8) return -1;
@@ -156,7 +156,7 @@ extern "C" int fb_gemm_grouped(void* Y, const void* X, const void* W, const int*
   const int w_rows = a.dual ? 2 * N : N;
   a.gr.tile_start = tile_start; a.gr.row_base = row_base; a.gr.experts = experts; a.gr.w_rows = w_rows;
   a.gr.uniform_rows = 0;
-  a.Y = Y; a.res = nullptr; a.workspace = nullptr; a.counters = nullptr; a.status = status; a.ldy = ldy;
+  a.Y = Y; a.res = nullptr; a.workspace = nullptr; a.counters = nullptr; a.status = status; a.ldy = ldy; a.limit = limit;
   a.M = max_rows;
   p.grid = sm_count;                               // the real tile count is only known on the device
   CUtensorMap tmA, tmB;

@@ -72,6 +72,7 @@ struct GemmArgs {
   // so the shared-memory layout, the descriptors and their k advance are those of the bf16 path. The epilogue
   // multiplies by a per-token-row and a per-output-feature scale (either may be null).
   int fp8;
+  float limit;              // dual: limit of clamped gated units, 0 = SwiGLU
   const float* scale_m;     // [M]
   const float* scale_n;     // [N] (SwiGLU: [2N], gate features then up features)
   int act;                  // epilogue activation of the plain (not dual) form
@@ -537,7 +538,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 x *= a.scale_n[n + j];
                 if (a.dual) u *= a.scale_n[a.N + n + j];
               }
-              v[j] = a.dual ? siluf_(x) * u : epilogue_act(x, a.act);
+              v[j] = a.dual ? glu_act(x, u, a.limit) : epilogue_act(x, a.act);
             }
             if (n + 32 <= a.N) {
               if (a.res) {
@@ -591,7 +592,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 if (m < a.M) {
                   const float sc = (a.scale_m ? a.scale_m[m] : 1.f);
                   float x = __uint_as_float(r0[j]) * sc * (a.scale_n ? a.scale_n[n] : 1.f);
-                  if (a.dual) x = siluf_(x) * (__uint_as_float(r1[j]) * sc * (a.scale_n ? a.scale_n[a.N + n] : 1.f));
+                  if (a.dual) x = glu_act(x, __uint_as_float(r1[j]) * sc * (a.scale_n ? a.scale_n[a.N + n] : 1.f), a.limit);
                   else x = epilogue_act(x, a.act);
                   if (a.res) x += bf2f(a.res[(size_t)m * a.ldy + n]);
                   if (a.out_f32) reinterpret_cast<float*>(a.Y)[(size_t)m * a.ldy + n] = x;
@@ -639,7 +640,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 const float sc = (a.scale_m ? a.scale_m[m] : 1.f);
                 g *= sc * (a.scale_n ? a.scale_n[n] : 1.f);
                 if (a.dual) u *= sc * (a.scale_n ? a.scale_n[a.N + n] : 1.f);
-                float x = a.dual ? siluf_(g) * u : epilogue_act(g, a.act);
+                float x = a.dual ? glu_act(g, u, a.limit) : epilogue_act(g, a.act);
                 if (a.res) x += bf2f(a.res[(size_t)m * a.ldy + n]);
                 if (a.out_f32) reinterpret_cast<float*>(a.Y)[(size_t)m * a.ldy + n] = x;
                 else Yb[(size_t)m * a.ldy + n] = f2bf(x);
@@ -738,7 +739,7 @@ struct GemmPlan { GemmArgs a; int grid; size_t smem; };
 
 static int plan_gemm(GemmPlan& p, int M, int N, int K, int mode, int split_k, int sm_count, int fp8 = 0) {
   GemmArgs& a = p.a;
-  a.fp8 = fp8; a.scale_m = nullptr; a.scale_n = nullptr; a.out_f32 = 0; a.act = ACT_NONE;
+  a.fp8 = fp8; a.scale_m = nullptr; a.scale_n = nullptr; a.out_f32 = 0; a.act = ACT_NONE; a.limit = 0.f;
   a.M = M; a.N = N; a.K = K;
   a.dual = mode == 1;
   a.swap = M <= 64;

@@ -10,10 +10,10 @@ extern "C" long fb_gemm_workspace_bytes(int M, int N, int split_k) {
   return tiles * split_k * 2L * bn * GM_BM * (long)sizeof(float);
 }
 
-// mode bit 0: SwiGLU over gate|up rows; bit 2: squared relu; bit 1: Y is fp32 (residual stays bf16 with the same leading dimension)
-extern "C" int fb_gemm_bf16(void* Y, const void* X, const void* W, const void* res, int M, int N, int K, long ldx,
-                            long ldy, int mode, int split_k, float* workspace, int* counters, int* status,
-                            int sm_count, cudaStream_t s) {
+// mode bit 0: SwiGLU over gate|up rows (with a limit, clamped gated units); bit 2: squared relu; bit 1: Y is fp32 (residual stays bf16 with the same leading dimension)
+extern "C" int fb_gemm_bf16_glu(void* Y, const void* X, const void* W, const void* res, int M, int N, int K, long ldx,
+                                long ldy, int mode, float limit, int split_k, float* workspace, int* counters, int* status,
+                                int sm_count, cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
   const int out_f32 = (mode >> 1) & 1, act = (mode & 4) ? ACT_RELU2 : ACT_NONE;
   mode &= 1;
@@ -25,7 +25,7 @@ extern "C" int fb_gemm_bf16(void* Y, const void* X, const void* W, const void* r
   GemmArgs& a = p.a;
   if (a.split_k > 1 && (!workspace || !counters)) return -6;
   a.Y = Y; a.res = (const __nv_bfloat16*)res; a.workspace = workspace; a.counters = counters; a.status = status;
-  a.ldy = ldy; a.out_f32 = out_f32; a.act = act;
+  a.ldy = ldy; a.out_f32 = out_f32; a.act = act; a.limit = limit;
   const int w_rows = a.dual ? 2 * N : N;
   CUtensorMap tmA, tmB;
   if (a.swap) {
@@ -46,6 +46,12 @@ extern "C" int fb_gemm_bf16(void* Y, const void* X, const void* W, const void* r
   }
   gemm_bf16_tc_kernel<0><<<p.grid, GM_THREADS, p.smem, s>>>(tmA, tmB, a);
   return (int)cudaGetLastError();
+}
+
+extern "C" int fb_gemm_bf16(void* Y, const void* X, const void* W, const void* res, int M, int N, int K, long ldx,
+                            long ldy, int mode, int split_k, float* workspace, int* counters, int* status,
+                            int sm_count, cudaStream_t s) {
+  return fb_gemm_bf16_glu(Y, X, W, res, M, N, K, ldx, ldy, mode, 0.f, split_k, workspace, counters, status, sm_count, s);
 }
 
 // ---- FP8 (e4m3) operands ----------------------------------------------------------------------------------

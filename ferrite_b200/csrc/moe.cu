@@ -15,6 +15,7 @@ namespace fb {
 constexpr int RT_MAXPL = 32;      // experts per lane (up to 1024 experts)
 
 // mode 0: softmax over all experts, top-k, renormalise, * scale.
+// mode 2: top-k of the logits, weights = softmax over the chosen ones * scale.
 // mode 1: scores = sigmoid(logit); choose by score + bias inside the best `topk_groups` of `n_groups` groups
 //         (group score = sum of its two best biased scores); weights = chosen scores / sum * scale.
 __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float* __restrict__ wts,
@@ -42,6 +43,9 @@ __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float*
     for (int j = 0; j < per; ++j) { sc[j] = sc[j] == -INFINITY ? 0.f : __expf(sc[j] - mx); sum += sc[j]; }
     sum = warp_sum(sum);
     for (int j = 0; j < per; ++j) { sc[j] /= sum; sel[j] = (lane * per + j < n_exp) ? sc[j] : -INFINITY; }
+  } else if (mode == 2) {
+    mx = warp_max(mx);
+    for (int j = 0; j < per; ++j) { sel[j] = sc[j]; sc[j] = expf(sc[j] - mx); }      // the largest logit is always chosen
   } else {
     for (int j = 0; j < per; ++j) {
       int e = lane * per + j;
@@ -130,21 +134,33 @@ __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float*
 // Pair GEMVs. Weight rows are bf16; a CTA handles 16 output rows of one (token, expert) pair.
 constexpr int MOE_THREADS = 256;
 
-// act[p][j] = silu(Wg[e][j] . x[t]) * (Wu[e][j] . x[t]);  W_gu[e] = [2*inter][hidden] (gate rows then up rows)
+// One more expert that lies apart from the stack: entry n_exp of the ids, of a width and a limit of its own.
+struct SharedExpert {
+  const void* w_gu;      // [2 * inter][hidden], or null
+  const void* w_down;    // [hidden][inter]
+  int id, inter;
+  float limit;
+};
+
+// act[p][j] = silu(Wg[e][j] . x[t]) * (Wu[e][j] . x[t]) (or the clamped form);  W_gu[e] = [2*inter][hidden] (gate rows then up rows). Rows of
+// act are ld_act elements apart.
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(__nv_bfloat16* __restrict__ act, const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w_gu,
-                   const int* __restrict__ ids, int top_k, int hidden, int inter, int e_lo, int e_hi) {
+                   const int* __restrict__ ids, int top_k, int hidden, int inter, int e_lo, int e_hi, int ld_act, float limit,
+                   const SharedExpert sh) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) __nv_bfloat16 xs_moe[];
   pdl_wait();                                                // ids come from the router kernel before this one
   const int p = blockIdx.y, e = ids[p];
-  if (e < e_lo || e >= e_hi) return;                         // another rank owns this expert
+  const bool shared = sh.w_gu && e == sh.id;
+  if (!shared && (e < e_lo || e >= e_hi)) return;            // another rank owns this expert
+  if (shared) { inter = sh.inter; limit = sh.limit; }
   const int t = p / top_k;
   for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x)
     reinterpret_cast<uint4*>(xs_moe)[i] = reinterpret_cast<const uint4*>(x + (size_t)t * hidden)[i];
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const __nv_bfloat16* we = w_gu + (size_t)(e - e_lo) * 2 * inter * hidden;
+  const __nv_bfloat16* we = shared ? (const __nv_bfloat16*)sh.w_gu : w_gu + (size_t)(e - e_lo) * 2 * inter * hidden;
   // the warp's two outputs run together: four weight rows stream at once, twice unrolled (8 loads of 16 bytes in flight)
   const int j0 = blockIdx.x * 16 + warp * 2;
   if (j0 >= inter) return;
@@ -176,29 +192,31 @@ moe_gate_up_kernel(__nv_bfloat16* __restrict__ act, const __nv_bfloat16* __restr
   }
   g0 = warp_sum(g0); u0 = warp_sum(u0); g1 = warp_sum(g1); u1 = warp_sum(u1);
   if (lane == 0) {
-    act[(size_t)p * inter + j0] = f2bf(siluf_(g0) * u0);
-    if (j0 + 1 < inter) act[(size_t)p * inter + j0 + 1] = f2bf(siluf_(g1) * u1);
+    act[(size_t)p * ld_act + j0] = f2bf(glu_act(g0, u0, limit));
+    if (j0 + 1 < inter) act[(size_t)p * ld_act + j0 + 1] = f2bf(glu_act(g1, u1, limit));
   }
 }
 
 // yp[p][n] = Wd[e][n] . act[p];  W_down[e] = [hidden][inter]; fp32 out (zero for pairs of other ranks)
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_down_kernel(float* __restrict__ yp, const __nv_bfloat16* __restrict__ act, const __nv_bfloat16* __restrict__ w_down,
-                const int* __restrict__ ids, int hidden, int inter, int e_lo, int e_hi) {
+                const int* __restrict__ ids, int hidden, int inter, int e_lo, int e_hi, int ld_act, const SharedExpert sh) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) __nv_bfloat16 as_moe[];
   pdl_wait();
   const int p = blockIdx.y, e = ids[p];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n0 = blockIdx.x * 16 + warp * 2;
-  if (e < e_lo || e >= e_hi) {
+  const bool shared = sh.w_gu && e == sh.id;
+  if (shared) inter = sh.inter;
+  if (!shared && (e < e_lo || e >= e_hi)) {
     if (lane == 0) for (int r = 0; r < 2; ++r) if (n0 + r < hidden) yp[(size_t)p * hidden + n0 + r] = 0.f;
     return;
   }
   for (int i = threadIdx.x; i < inter / 8; i += blockDim.x)
-    reinterpret_cast<uint4*>(as_moe)[i] = reinterpret_cast<const uint4*>(act + (size_t)p * inter)[i];
+    reinterpret_cast<uint4*>(as_moe)[i] = reinterpret_cast<const uint4*>(act + (size_t)p * ld_act)[i];
   __syncthreads();
-  const __nv_bfloat16* we = w_down + (size_t)(e - e_lo) * hidden * inter;
+  const __nv_bfloat16* we = shared ? (const __nv_bfloat16*)sh.w_down : w_down + (size_t)(e - e_lo) * hidden * inter;
   if (n0 >= hidden) return;
   const int n1 = min(n0 + 1, hidden - 1);
   const __nv_bfloat16* w0 = we + (size_t)n0 * inter;
@@ -221,19 +239,23 @@ moe_down_kernel(float* __restrict__ yp, const __nv_bfloat16* __restrict__ act, c
   }
 }
 
-// The same in 32 bits, one warp per output: GU: out[p][j] = silu(W[e][j] . x[t]) * (W[e][N + j] . x[t]), else out[p][j] = W[e][j] . x[p]
+// The same in 32 bits, one warp per output: GU: out[p][j] = silu(W[e][j] . x[t]) * (W[e][N + j] . x[t]), else out[p][j] = W[e][j] . x[p];
+// rows of the activations ld_act floats apart
 template <bool GU>
 __global__ void __launch_bounds__(256) expert_f32_kernel(float* __restrict__ out, const float* __restrict__ x, const float* __restrict__ w,
-                                                         const int* __restrict__ ids, int p0, int top_k, int K, int N, int n_exp) {
+                                                         const int* __restrict__ ids, int p0, int top_k, int K, int N, int n_exp, int ld_act,
+                                                         float limit, const SharedExpert sh) {
   pdl_launch_dependents();
   pdl_wait();
   const int p = p0 + blockIdx.y, e = ids[p], lane = threadIdx.x & 31;
   const int j = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const bool shared = sh.w_gu && e == sh.id;
+  if (shared) { if (GU) N = sh.inter; else K = sh.inter; limit = sh.limit; }
   if (j >= N) return;
   float a = 0.f, b = 0.f;
-  if (e >= 0 && e < n_exp) {
-    const float* xr = x + (size_t)(GU ? p / top_k : p) * K;
-    const float* w0 = w + ((size_t)e * (GU ? 2 : 1) * N + j) * K;
+  if (shared || (e >= 0 && e < n_exp)) {
+    const float* xr = GU ? x + (size_t)(p / top_k) * K : x + (size_t)p * ld_act;
+    const float* w0 = (shared ? (const float*)(GU ? sh.w_gu : sh.w_down) : w + (size_t)e * (GU ? 2 : 1) * N * K) + (size_t)j * K;
     for (int k = lane * 4; k < K; k += 128) {
       const float4 xv = *reinterpret_cast<const float4*>(xr + k), v = *reinterpret_cast<const float4*>(w0 + k);
       a = fmaf(xv.x, v.x, fmaf(xv.y, v.y, fmaf(xv.z, v.z, fmaf(xv.w, v.w, a))));
@@ -245,7 +267,15 @@ __global__ void __launch_bounds__(256) expert_f32_kernel(float* __restrict__ out
   }
   a = warp_sum(a);
   if (GU) b = warp_sum(b);
-  if (lane == 0) out[(size_t)p * N + j] = GU ? a / (1.f + expf(-a)) * b : a;
+  if (lane != 0) return;
+  if (!GU) {
+    out[(size_t)p * N + j] = a;
+  } else if (limit > 0.f) {
+    a = fminf(a, limit);
+    out[(size_t)p * ld_act + j] = a / (1.f + expf(-1.702f * a)) * (fminf(fmaxf(b, -limit), limit) + 1.f);
+  } else {
+    out[(size_t)p * ld_act + j] = a / (1.f + expf(-a)) * b;
+  }
 }
 
 // out[t] = (res[t]) + sum_k wts[t][k] * yp[t*K + k]  (pick order) + shared[t] * gate[t]; fp32 or bf16 out
@@ -287,19 +317,40 @@ extern "C" int fb_moe_route(int* ids, float* wts, const float* logits, const flo
                          n_groups, topk_groups, scale, ld, shared_col, shared_id, lane_groups);
 }
 
-// The pair products in 32 bits: act and yp as fb_moe_gate_up / fb_moe_down leave them; ids outside [0, n_exp) give zero rows.
+// The pair products in 32 bits: act and yp as fb_moe_gate_up / fb_moe_down leave them; ids outside [0, n_exp) give zero rows, but for the
+// shared expert's (shared_gu not null), which is id n_exp.
 extern "C" int fb_expert_rows_f32(float* yp, float* act, const float* x, const float* w_gu, const float* w_down, const int* ids, int pairs,
-                                  int top_k, int hidden, int inter, int n_exp, cudaStream_t s) {
+                                  int top_k, int hidden, int inter, int n_exp, int ld_act, float limit, const float* shared_gu,
+                                  const float* shared_down, int shared_inter, float shared_limit, cudaStream_t s) {
   if (pairs <= 0) return 0;
-  if (hidden % 4 || inter % 4) return -1;
+  const int widest = shared_gu && shared_inter > inter ? shared_inter : inter;
+  if (hidden % 4 || inter % 4 || (shared_gu && shared_inter % 4) || ld_act % 4 || ld_act < widest) return -1;
+  const SharedExpert sh{shared_gu, shared_down, n_exp, shared_inter, shared_limit};
   for (int p0 = 0; p0 < pairs; p0 += 32768) {              // grid.y; a multiple of top_k is not needed: pairs are counted from 0
     const int n = pairs - p0 < 32768 ? pairs - p0 : 32768;
-    int rc = (int)launch_pdl(expert_f32_kernel<true>, dim3((inter + 7) / 8, n), dim3(256), 0, s, act, x, w_gu, ids, p0, top_k, hidden, inter, n_exp);
+    int rc = (int)launch_pdl(expert_f32_kernel<true>, dim3((widest + 7) / 8, n), dim3(256), 0, s, act, x, w_gu, ids, p0, top_k, hidden, inter, n_exp,
+                             ld_act, limit, sh);
     if (!rc) rc = (int)launch_pdl(expert_f32_kernel<false>, dim3((hidden + 7) / 8, n), dim3(256), 0, s, yp, (const float*)act, w_down, ids, p0,
-                                  top_k, inter, hidden, n_exp);
+                                  top_k, inter, hidden, n_exp, ld_act, limit, sh);
     if (rc) return rc;
   }
   return 0;
+}
+
+// Pair GEMVs of few rows, both products: clamped gated units with a limit, and the shared expert (id n_exp) where shared_gu is not null
+extern "C" int fb_expert_rows(float* yp, void* act, const void* x, const void* w_gu, const void* w_down, const int* ids, int pairs, int top_k,
+                              int hidden, int inter, int n_exp, int ld_act, float limit, const void* shared_gu, const void* shared_down,
+                              int shared_inter, float shared_limit, cudaStream_t s) {
+  if (pairs <= 0) return 0;
+  const int widest = shared_gu && shared_inter > inter ? shared_inter : inter;
+  if (hidden % 8 || inter % 8 || (shared_gu && shared_inter % 8) || ld_act % 8 || ld_act < widest || pairs > 65535) return -1;
+  const SharedExpert sh{shared_gu, shared_down, n_exp, shared_inter, shared_limit};
+  const int rc = (int)launch_pdl(moe_gate_up_kernel, dim3((widest + 15) / 16, pairs), dim3(MOE_THREADS), (size_t)hidden * 2, s,
+                                 (__nv_bfloat16*)act, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w_gu, ids, top_k, hidden, inter, 0, n_exp,
+                                 ld_act, limit, sh);
+  if (rc) return rc;
+  return (int)launch_pdl(moe_down_kernel, dim3((hidden + 15) / 16, pairs), dim3(MOE_THREADS), (size_t)widest * 2, s, yp,
+                         (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, ids, hidden, inter, 0, n_exp, ld_act, sh);
 }
 
 extern "C" int fb_moe_gate_up(void* act, const void* x, const void* w_gu, const int* ids, int pairs, int top_k,
@@ -308,7 +359,7 @@ extern "C" int fb_moe_gate_up(void* act, const void* x, const void* w_gu, const 
   if (hidden % 8) return -1;
   return (int)launch_pdl(moe_gate_up_kernel, dim3((inter + 15) / 16, pairs), dim3(MOE_THREADS), (size_t)hidden * 2, s,
                          (__nv_bfloat16*)act, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w_gu, ids, top_k, hidden,
-                         inter, e_lo, e_hi);
+                         inter, e_lo, e_hi, inter, 0.f, SharedExpert{});
 }
 
 extern "C" int fb_moe_down(float* yp, const void* act, const void* w_down, const int* ids, int pairs, int hidden,
@@ -316,7 +367,7 @@ extern "C" int fb_moe_down(float* yp, const void* act, const void* w_down, const
   if (pairs <= 0) return 0;
   if (inter % 8) return -1;
   return (int)launch_pdl(moe_down_kernel, dim3((hidden + 15) / 16, pairs), dim3(MOE_THREADS), (size_t)inter * 2, s, yp,
-                         (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, ids, hidden, inter, e_lo, e_hi);
+                         (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, ids, hidden, inter, e_lo, e_hi, inter, SharedExpert{});
 }
 
 extern "C" int fb_moe_combine(void* out, const float* yp, const float* wts, const void* shared, const float* shared_gate,

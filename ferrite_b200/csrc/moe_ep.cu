@@ -168,12 +168,12 @@ __global__ void ep_signal_kernel(EpComm c) {
 
 // ---- 6. combine ------------------------------------------------------------------------------------------------
 // grid = local tokens; out[t] = res[t] + shared[t] * sigmoid(gate[t]) + sum_k wts[t][k] * result_row(t, k), pick order
-// With `acc` the sum is added to its fp32 rows instead of being written to out.
+// With `acc` the sum is added to its fp32 rows (`add` 0: written to them) instead of being written to out. Gates gate_ld floats apart.
 __global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16* __restrict__ out, float* __restrict__ acc32,
                                                          const int* __restrict__ ids, const float* __restrict__ wts,
                                                          const int* __restrict__ pos, const int* __restrict__ send_off,
                                                          const __nv_bfloat16* __restrict__ shared,
-                                                         const float* __restrict__ shared_gate,
+                                                         const float* __restrict__ shared_gate, long gate_ld, int add,
                                                          const __nv_bfloat16* __restrict__ res, int rows, int top_k) {
   __shared__ int fail_s;
   const int t = blockIdx.x;
@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16
   __syncthreads();
   const int H = c.hidden;
   if (!fail_s && t < rows) {
-    const float g = shared ? (shared_gate ? sigmoidf_(shared_gate[t]) : 1.f) : 0.f;
+    const float g = shared ? (shared_gate ? sigmoidf_(shared_gate[t * gate_ld]) : 1.f) : 0.f;
     for (int i = threadIdx.x; i < H / 8; i += blockDim.x) {
       float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
       for (int k = 0; k < top_k; ++k) {
@@ -213,7 +213,7 @@ __global__ void __launch_bounds__(256) ep_combine_kernel(EpComm c, __nv_bfloat16
       }
       if (acc32) {
         float4* a = reinterpret_cast<float4*>(acc32 + (size_t)t * H + i * 8);
-        const float4 a0 = a[0], a1 = a[1];
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), a0 = add ? a[0] : zero, a1 = add ? a[1] : zero;
         a[0] = make_float4(a0.x + acc[0], a0.y + acc[1], a0.z + acc[2], a0.w + acc[3]);
         a[1] = make_float4(a1.x + acc[4], a1.y + acc[5], a1.z + acc[6], a1.w + acc[7]);
         continue;
@@ -258,9 +258,9 @@ extern "C" long fb_ep_out_offset(int n_experts, int hidden, long cap_rows) { ret
 
 // One expert-parallel MoE block over this rank's `rows` tokens. `act` is scratch [cap_rows][inter] bf16; `plan` is int
 // scratch of rows * top_k + 3 * n_experts + 8 entries. w_gu / w_down hold only the experts this rank owns. out_f32: `out` holds
-// fp32 rows to which the experts' sum is added.
-extern "C" int fb_ep_moe(void* out, int out_f32, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
-                         const void* shared, const float* shared_gate, const void* res, void* act, int* plan, int rows,
+// fp32 rows, 1: to which the experts' sum is added, 2: which take it. limit: of clamped gated units (0: SwiGLU).
+extern "C" int fb_ep_moe(void* out, int out_f32, float limit, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
+                         const void* shared, const float* shared_gate, long gate_ld, const void* res, void* act, int* plan, int rows,
                          int top_k, int n_experts, int hidden, int inter, long cap_rows, const void* const* peers, int rank,
                          int world, uint32_t* ctr, int* status, unsigned spin_limit, int sm_count, cudaStream_t s) {
   if (world < 1 || world > EP_MAX_RANKS || n_experts > EP_MAX_EXPERTS || n_experts % world || hidden % 8 || inter % 8)
@@ -284,14 +284,14 @@ extern "C" int fb_ep_moe(void* out, int out_f32, const void* x, const int* ids, 
   if (e != cudaSuccess) return (int)e;
   const char* local = reinterpret_cast<const char*>(peers[rank]);
   int rc = fb_gemm_grouped(act, local + l.recv_off, w_gu, tile_start, row_base, c.per_rank, (int)cap_rows, inter, hidden,
-                           hidden, inter, 1, status, sm_count, s);
+                           hidden, inter, 1, limit, status, sm_count, s);
   if (rc) return rc;
   rc = fb_gemm_grouped(const_cast<char*>(local) + l.out_off, act, w_down, tile_start, row_base, c.per_rank, (int)cap_rows,
-                       hidden, inter, inter, hidden, 0, status, sm_count, s);
+                       hidden, inter, inter, hidden, 0, 0.f, status, sm_count, s);
   if (rc) return rc;
   ep_signal_kernel<<<1, 32, 0, s>>>(c);
   ep_combine_kernel<<<rows > 0 ? rows : 1, 256, 0, s>>>(c, (__nv_bfloat16*)out, out_f32 ? (float*)out : nullptr, ids, wts, pos, send_off,
-                                                        (const __nv_bfloat16*)shared, shared_gate,
+                                                        (const __nv_bfloat16*)shared, shared_gate, gate_ld, out_f32 == 1,
                                                         (const __nv_bfloat16*)res, rows, top_k);
   return (int)cudaGetLastError();
 }

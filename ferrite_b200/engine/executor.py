@@ -23,7 +23,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from ..config import EngineConfig, ModelConfig
-from ..models.weights import Weights, delta_dims, gqa_dims, latent_dims
+from ..models.weights import Weights, delta_dims, gqa_dims, latent_dims, ssm_dims
 from ..ops.latent import SegGroup, seg_groups
 from ..ops.qweight import QWeight
 
@@ -178,6 +178,8 @@ class Executor:
         # models of listed layers: caches and states belong to runs of layers (a looped layer has one per pass)
         self.runs = c.layer_runs if c.layers else []
         self.run_dims: Dict[int, object] = {}
+        self.kv_run: Dict[int, int] = {}         # gqa runs: the run whose cache they read
+        self.pools: Dict[Tuple[int, int], Tuple[torch.Tensor, torch.Tensor]] = {}   # (run, block length): mean keys and values, paged
         for r in self.runs:
             l, zeros = c.layers[r.layer], lambda *s, t=dt: torch.zeros(*s, dtype=t, device=dev)
             if l.mixer == "latent":
@@ -188,12 +190,28 @@ class Executor:
                     self.v_cache[r.index] = zeros(n_blocks, 0)
             elif l.mixer == "gqa":
                 d = self.run_dims[r.index] = gqa_dims(c, r.layer)
-                self.k_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
-                self.v_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
+                self.kv_run[r.index] = r.index if d.source < 0 else max(q.index for q in self.runs[:r.index] if q.layer == d.source)
+                if d.source < 0:
+                    self.k_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
+                    self.v_cache[r.index] = zeros(n_blocks, ecfg.kv_block, d.kv_heads, d.hp)
+                if d.pool:
+                    per_page = -(-ecfg.kv_block // d.pool)       # blocks that end in a page, at most
+                    self.pools.setdefault((self.kv_run[r.index], d.pool), tuple(zeros(n_blocks, per_page, d.kv_heads, d.hp) for _ in "kv"))
+            elif l.mixer == "ssm":
+                d = self.run_dims[r.index] = ssm_dims(c, r.layer)
+                self.rec_state[r.index] = zeros(ecfg.n_slots, d.heads, d.state, d.vdim, t=torch.float32)
+                self.conv_state[r.index] = zeros(ecfg.n_slots, d.conv - 1, d.channels)
             else:
                 d = self.run_dims[r.index] = delta_dims(c, r.layer)
                 self.rec_state[r.index] = zeros(ecfg.n_slots, d.heads, d.dim, d.vdim, t=torch.float32)
                 self.conv_state[r.index] = zeros(ecfg.n_slots, d.conv - 1, d.channels)
+        # convolved operands: the last inputs of every sublayer, one tensor for all of them
+        self.canon_at: Dict[Tuple[int, str], int] = {}
+        if c.canon > 1:
+            for r in self.runs:
+                for what in ("mix", "ffn")[:2 if c.layers[r.layer].ff else 1]:
+                    self.canon_at[r.index, what] = len(self.canon_at)
+            self.conv_state["canon"] = torch.zeros(ecfg.n_slots, len(self.canon_at), c.canon - 1, weights["embed"].shape[1], dtype=dt, device=dev)
         # the token at every cached position, paged like the latents: the token before a segment (bigram embeddings) is read
         # from here, so it follows the pages through parking, forks, resumed prefixes and rejected drafts
         self.tok_pages = torch.zeros(n_blocks, ecfg.kv_block, dtype=torch.int32, device=dev) if c.gram_buckets else None
@@ -334,7 +352,9 @@ class Executor:
             item = torch.empty(0, dtype=self.dtype).element_size()
             dims = [(gqa_dims if c.layers[r.layer].mixer == "gqa" else latent_dims)(c, r.layer) for r in c.layer_runs if c.layers[r.layer].cached]
             row = sum(2 * d.kv_heads * d.hp if hasattr(d, "kv_heads") else d.lat for d in dims)
-            return e.kv_block * (item * row + (4 if c.gram_buckets else 0))
+            means = {(i if l.kv_from is None else l.kv_from, l.pool): gqa_dims(c, i) for i, l in enumerate(c.layers) if l.pool}
+            pooled = sum(2 * -(-e.kv_block // d.pool) * d.kv_heads * d.hp for d in means.values())
+            return e.kv_block * (item * row + (4 if c.gram_buckets else 0)) + item * pooled
         return per * max(1, self.cfg.n_attn)
 
     # ---- block tables -----------------------------------------------------------------------------
@@ -410,6 +430,9 @@ class Executor:
             self.v_cache[i][d] = self.v_cache[i][s]
             if i in self.kv_scale:
                 self.kv_scale[i][d] = self.kv_scale[i][s]
+        for means in self.pools.values():
+            for t in means:
+                t[d] = t[s]
         if self.tok_pages is not None:
             self.tok_pages[d] = self.tok_pages[s]
 
@@ -599,48 +622,61 @@ class Executor:
         w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{run.layer}.", self.run_dims[run.index]
         cache, T = self.k_cache[d.source], xb.shape[0]
         proj = ops.linear(xb, w[p + "in_proj"], out_f32=True)
-        cq = ops.latent_prep(proj, d, w[p + "q_a_norm"], w.get(p + "kv_a_norm"), mv["slot"], mv["pos"], self.block_table, cache, kvb,
-                             self.cfg.eps)
-        q = ops.linear(cq, w[p + "q_b"])
+        if d.q_rank:
+            cq = ops.latent_prep(proj, d, w[p + "q_a_norm"], w.get(p + "kv_a_norm"), mv["slot"], mv["pos"], self.block_table, cache, kvb,
+                                 self.cfg.eps)
+            q = ops.linear(cq, w[p + "q_b"])
+        else:
+            q = ops.latent_rot_prep(proj, d, w[p + "kv_a_norm"], w[p + "inv_freq"], mv["slot"], mv["pos"], self.block_table, cache, kvb,
+                                    self.cfg.eps).view(T, -1)
         o = None
+        rows = lambda: torch.empty(T, d.heads * d.vp, dtype=q.dtype, device=q.device)
         for g in groups:
             segs = tuple(mv[k][g.seg_lo:g.seg_hi] for k in ("sslot", "srow0", "snrows", "spos0"))
-            if g.prompt and d.hp <= 256:
-                o = torch.empty_like(q) if o is None else o
-                key = (d.source, g.row_lo)
+            if g.prompt and d.hp <= 256 and self.dtype == torch.bfloat16:
+                o = rows() if o is None else o
+                key = (d.source, g.row_lo, d.window)
                 if key not in gathered:                  # shared by the layers that share the latents
-                    gathered[key] = ops.latent_rows(cache, g, kvb)
+                    gathered[key] = ops.latent_rows(cache, g, kvb, d.window)
                 ops.latent_attention_prompt(q, gathered[key], w[p + "kv_up"], d, g, segs, kvb, o)
                 continue
             a, b = g.row_lo, g.row_hi
             qabs = ops.head_linear(q[a:b].view(b - a, d.heads, d.hp), w[p + "k_abs"])
-            ol = ops.latent_attention(qabs, cache, g, mv["slot"][a:b], mv["kvlen"][a:b], segs, self.block_table, kvb, d.scale, nsplit)
+            ol = ops.latent_attention(qabs, cache, g, mv["slot"][a:b], mv["kvlen"][a:b], segs, self.block_table, kvb, d.scale, nsplit,
+                                      vlat=d.vlat, window=d.window)
             if a == 0 and b == T:
                 o = ops.head_linear(ol, w[p + "v_up"]).reshape(T, -1)
             else:
-                o = torch.empty_like(q) if o is None else o
-                ops.head_linear(ol, w[p + "v_up"], out=o[a:b].view(b - a, d.heads, d.hp))
+                o = rows() if o is None else o
+                ops.head_linear(ol, w[p + "v_up"], out=o[a:b].view(b - a, d.heads, d.vp))
         return self._sum_ranks(o, w[p + "out_proj"])
 
-    def _mix_gqa(self, h, run, mv, groups, nsplit):
+    def _mix_gqa(self, h, run, mv, groups, nsplit, gathered):
         """Grouped-query attention over operand rows h."""
         p, d = f"l{run.layer}.", self.run_dims[run.index]
         proj = self.ops.linear(h, self.w[p + "in_proj"], out_f32=True)
         o = torch.empty(h.shape[0], d.heads, d.hp, dtype=self.dtype, device=self.device)
-        self._gqa_rows(proj, run, mv, groups, nsplit, o)
+        self._gqa_rows(proj, run, mv, groups, nsplit, o, gathered)
         return self._sum_ranks(o.view(o.shape[0], -1), self.w[p + "out_proj"])
 
-    def _gqa_rows(self, proj, run, mv, groups, nsplit, o):
+    def _gqa_rows(self, proj, run, mv, groups, nsplit, o, gathered=None):
         """From the fused projection to the heads' outputs o [T, heads, hp] (rows may lie apart): prompt segments on the flash kernel, the
-        others split over the keys."""
+        others split over the keys. `gathered`: what this step's layers have made of the caches so far."""
         w, ops, kvb, p, d = self.w, self.ops, self.ecfg.kv_block, f"l{run.layer}.", self.run_dims[run.index]
-        kc, vc = self.k_cache[run.index], self.v_cache[run.index]
-        norms = {"norms": (w[p + "q_norm"], w[p + "k_norm"])} if d.row_norm else {}
+        src = self.kv_run[run.index]
+        kc, vc = self.k_cache[src], self.v_cache[src]
+        norms = {"norms": (w[p + "q_norm"], w.get(p + "k_norm"))} if d.row_norm else {}
         q = ops.gqa_prep(proj, d, w.get(p + "in_bias"), w[p + "inv_freq"], mv["slot"], mv["pos"], self.block_table, kc, vc, kvb, self.cfg.eps,
                          **norms)
         mix = {}
         if d.maps == 2 or d.gate_off >= 0:
             mix = dict(lam=w.get(p + "lam"), eps=self.cfg.eps, gate=proj[:, d.gate_off:d.gate_off + d.heads * d.vw] if d.gate_off >= 0 else None)
+        if d.pool:
+            mix["pooled"] = self.pools[src, d.pool]
+            if (src, d.pool) not in gathered:            # once per step: layers that share keys share their means
+                gathered[src, d.pool] = True
+                max_rows = max(g.max_rows for g in groups)
+                ops.pool_keys(d, kc, vc, mix["pooled"], mv["sslot"], mv["spos0"], mv["snrows"], max_rows, self.block_table, kvb)
         for g in groups:
             segs = tuple(mv[k][g.seg_lo:g.seg_hi] for k in ("sslot", "srow0", "snrows", "spos0"))
             ops.gqa_attention(q, d, kc, vc, w.get(p + "sink"), g, mv["slot"], mv["kvlen"], segs, self.block_table, kvb, nsplit, o, **mix)
@@ -679,22 +715,110 @@ class Executor:
             self.verify_proj[run.index] = proj
         return self._sum_ranks(self._cdelta(proj, run, mv, groups, commit), w[p + "out_proj"])
 
+    def _mix_ssm(self, h, run, mv, groups, commit):
+        """State-space recurrence over operand rows h; verify rows keep their projections for the replay."""
+        proj = self.ops.linear(h, self.w[f"l{run.layer}.in_proj"])
+        if not commit:
+            self.verify_proj[run.index] = proj
+        return self._sum_ranks(self._ssm(proj, run, mv, groups, commit), self.w[f"l{run.layer}.out_proj"])
+
+    def _ssm(self, proj, run, mv, groups, commit):
+        p, r = f"l{run.layer}.", run.index
+        names = ("conv", "conv_bias", "A", "dt_bias", "skip", "gnorm_w")
+        return self.ops.ssm(proj, self.run_dims[r], {n: self.w[p + n] for n in names}, self.rec_state[r], self.conv_state[r], groups,
+                            mv["sslot"], mv["srow0"], mv["snrows"], mv["slot"], mv["pos"], self.cfg.eps, commit)
+
+    def _experts_listed(self, h, run):
+        """Routed feed-forward of operand rows h -> (32-bit sums or None, (expert rows, weights) or None): what the next residual add
+        takes. Few rows: the shared expert is one more pick of every token; prompt rows: it joins the combine of the grouped products."""
+        l, w, ops, p = self.cfg.layers[run.layer], self.w, self.ops, f"l{run.layer}."
+        logits, ep = ops.linear(h, w[p + "router"], out_f32=True), self.ep_listed.get(l.experts)
+        gu, dn, n = w[p + "experts_gate_up"], w[p + "experts_down"], l.experts
+        mode = 2 if l.router == "softmax" else 1
+        if ep is None or h.shape[0] <= ops.moe_pair_rows:
+            shared = dict(shared_col=n, shared_id=n) if l.shared_ff else {}
+            ids, wts = ops.moe_route(logits, None, mode, l.top, l.groups, l.keep_groups, l.route_scale, n_exp=n, **shared)
+            self._count_experts(run.layer, ids)
+            stacks = (w[p + "shared_gate_up"], w[p + "shared_down"], l.shared_limit) if l.shared_ff else None
+            return None, (ops.expert_rows(h, ids, gu, dn, l.limit, stacks), wts)
+        ids, wts = ops.moe_route(logits, None, mode, l.top, l.groups, l.keep_groups, l.route_scale, n_exp=n)
+        self._count_experts(run.layer, ids)
+        y, shared, gate = torch.empty(h.shape[0], h.shape[1], dtype=torch.float32, device=self.device), None, None
+        if l.shared_ff:
+            shared = ops.linear(ops.glu(h, w[p + "shared_gate_up"][0], l.shared_limit), w[p + "shared_down"][0])
+            gate = logits[:, n]
+        ep.moe(ops, h, ids, wts, gu, dn, shared, gate, acc=y, add=False, limit=l.limit)
+        return y, None
+
     def _cdelta(self, proj, run, mv, groups, commit):
         p, r = f"l{run.layer}.", run.index
         names = ("decay_up", "gate_up_lr", "conv", "A_log", "dt_bias", "gnorm_w")
         return self.ops.cdelta(proj, self.run_dims[r], {n: self.w[p + n] for n in names}, self.rec_state[r], self.conv_state[r], groups,
                                mv["sslot"], mv["srow0"], mv["snrows"], self.cfg.eps, commit)
 
-    def _layers_listed(self, x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit):
+    def _conv_operand(self, x_in, x, y, post, nxt, mv, single, commit, at=None, name=None, pairs=None, average=None):
+        """Designs of layer norms and convolved operands: x = x_in + norm(y) (weights `post`), its average over depth, the next sublayer's
+        operand (norm weights `nxt`, convolution `name`, whose inputs before this step lie at `at`)."""
+        c, w, ops = self.cfg, self.w, self.ops
+        kw, tails = {}, None
+        if nxt is not None and c.canon:
+            tails = self.conv_state["canon"][:, self.canon_at[at]] if c.canon > 1 else torch.empty(1, 0, x.shape[1], device=x.device, dtype=self.dtype)
+            kw = dict(conv=(w[name], tails), row_slot=mv["slot"], row_pos=mv["pos"], single=single, commit=commit)
+        xb, h = ops.add_conv_normed(x_in, x, y, None if post is None else w[post], c.hidden, c.eps, None if nxt is None else w[nxt],
+                                    pairs=pairs, average=average, **kw)
+        if kw and c.canon > 1:
+            if not commit:
+                self.verify_proj[at] = h
+            elif not single:
+                ops.conv_tail(tails, h, mv["sslot"], mv["srow0"], mv["snrows"])
+        return xb
+
+    def _layers_conv(self, x0, xs, mv, groups, max_seg_rows, nsplit, commit):
+        """x <- x + norm(mixer(conv(norm(x)))), x <- x + norm(ff(conv(norm(x)))), then the average over depth. x0: the embedding output,
+        xs: the results of the layers (xs[0] is x0) with `depth_average`. Returns the residual stream behind the last layer."""
+        c = self.cfg
+        gathered: Dict[tuple, object] = {}
+        x = torch.empty_like(x0)
+        single = max_seg_rows == 1
+        step = lambda x_in, y, post, nxt, at, name, **kw: self._conv_operand(x_in, x, y, post, nxt, mv, single, commit, at, name, **kw)
+        xb = step(x0, None, None, f"l{self.runs[0].layer}.pre_norm", (0, "mix"), f"l{self.runs[0].layer}.mix_canon")
+        x_in, last_run = x0, {r.layer: r.index for r in self.runs}
+        for run in self.runs:
+            i, l, p, r = run.layer, c.layers[run.layer], f"l{run.layer}.", run.index
+            if l.mixer == "latent":
+                y = self._mix_latent(xb, run, mv, groups, nsplit, gathered)
+            elif l.mixer == "gqa":
+                y = self._mix_gqa(xb, run, mv, groups, nsplit, gathered)
+            else:
+                y = self._mix_ssm(xb, run, mv, groups, commit)
+            pairs, post = None, p + "mix_norm"
+            if l.ff:
+                xb = step(x_in, y, post, p + "ffn_pre_norm", (r, "ffn"), p + "ffn_canon")
+                y, pairs = self._experts_listed(xb, run)
+                x_in, post = x, p + "ffn_norm"
+            q = f"l{self.runs[r + 1].layer}." if r + 1 < len(self.runs) else None
+            xb = step(x_in, y, post, None if q is None else q + "pre_norm", (r + 1, "mix"), None if q is None else q + "mix_canon", pairs=pairs,
+                      average=(xs, r + 1, self.w[p + "dwa"]) if c.depth_average else None)
+            x_in = x
+            if i in c.tap_layers and r == last_run[i]:
+                self.taps.append(x[:, :c.hidden].to(self.dtype, copy=True))
+            if self.dump_layers:
+                self._dump_layer(i, x[:, :c.hidden], False, x.shape[0])
+        return x
+
+    def _layers_listed(self, x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit, xs=None):
         """x <- x + norm(mixer(x)), x <- x + norm(ff(x)), with `pre_norm` also a norm ahead of the mixer and the feed-forward; or
         `parallel` blocks. x is the 32-bit residual stream (updated in place), xb its copy in the GEMM operand type. The pass over the rows that adds a
         sublayer's output also makes the operand of whatever comes next. `loop_rows` [T, 2 width]: operand of the product that opens
-        a pass of the loop, the embedding output in its right half. Returns the last copy of x."""
+        a pass of the loop, the embedding output in its right half. Returns the stream behind the last layer and its last copy."""
         c, w, ops = self.cfg, self.w, self.ops
         self.taps = []
         kinds = {l.mixer for l in c.layers}
         groups = seg_groups(self._step_segments if ops.name == "cuda" and (self.dtype == torch.bfloat16 or "cdelta" in kinds) else None, nseg, T,
-                            max_seg_rows, FLASH_MIN_ROWS, self.block_table, self.ecfg.kv_block, self.device, "latent" in kinds)
+                            max_seg_rows, FLASH_MIN_ROWS, self.block_table, self.ecfg.kv_block, self.device)
+        if c.canon or c.layer_norm:
+            x = self._layers_conv(x, xs, mv, groups, max_seg_rows, nsplit, commit)
+            return x, x
         gathered: Dict[tuple, torch.Tensor] = {}
         W = x.shape[1]
         last_run = {r.layer: r.index for r in self.runs}
@@ -720,7 +844,7 @@ class Executor:
                 if l.mixer == "latent":
                     y = self._mix_latent(xb, run, mv, groups, nsplit, gathered)
                 elif l.mixer == "gqa":
-                    y = self._mix_gqa(xb, run, mv, groups, nsplit)
+                    y = self._mix_gqa(xb, run, mv, groups, nsplit, gathered)
                 else:
                     y = self._mix_cdelta(xb, run, mv, groups, commit)
                 nxt, buf = (w.get(p + "ffn_pre_norm"), None) if l.ff else after(run.index + 1)
@@ -733,7 +857,7 @@ class Executor:
                 self.taps.append(x[:, :c.hidden].to(self.dtype, copy=True) if c.pre_norm or xb is x else xb[:, :c.hidden])
             if self.dump_layers:
                 self._dump_layer(i, x[:, :c.hidden], False, T)
-        return x if xb is None else xb
+        return x, (x if xb is None else xb)
 
     def _layers(self, x, mv, T, nseg, max_seg_rows, nsplit, commit, tv=None):
         c, w, ops = self.cfg, self.w, self.ops
@@ -910,7 +1034,8 @@ class Executor:
         if nlog == 0:
             return None, None
         if c.layers:
-            rows = ops.norm_rows(x, mv["lrow"], w["final_norm"], c.hidden, c.eps, **({"bias": w["final_norm_bias"]} if c.parallel else {}))
+            rows = ops.norm_rows(x, mv["lrow"], w["final_norm"], c.hidden, c.eps,
+                                 **({"bias": w["final_norm_bias"]} if c.parallel else {"mean": True} if c.layer_norm else {}))
             logits = ops.linear(rows, w["lm_head"], out_f32=True)
             if c.logit_softcap:
                 logits = ops.softcap(logits, c.logit_softcap)
@@ -938,11 +1063,15 @@ class Executor:
         if self.cfg.layers:
             c, w = self.cfg, self.w
             assert x_add is None and not tree, "models of listed layers: no injected rows, no verify trees"
-            loop_rows = torch.empty(T, 2 * w["embed"].shape[1], dtype=self.dtype, device=self.device) if c.loop and c.loop_input else None
+            W = w["embed"].shape[1]
+            loop_rows = torch.empty(T, 2 * W, dtype=self.dtype, device=self.device) if c.loop and c.loop_input else None
+            xs = torch.empty(len(self.runs) + 1, T, W, dtype=torch.float32, device=self.device) if c.depth_average else None
             x, xb = self.ops.embed_grams(w["embed"], w.get("bigram"), mv["tok"], mv["slot"], mv["pos"], self.block_table,
                                          self.tok_pages, self.ecfg.kv_block, c.embed_scale, c.gram_buckets, c.gram_mul_prev,
-                                         c.gram_mul_cur, **({"out": loop_rows} if loop_rows is not None else {}))
-            self.last_hidden = self._layers_listed(x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit)[:, :c.hidden]
+                                         c.gram_mul_cur, **({"out": loop_rows} if loop_rows is not None else {}),
+                                         **({"x": xs[0]} if xs is not None else {}))
+            x, last = self._layers_listed(x, xb, loop_rows, mv, T, nseg, max_seg_rows, nsplit, commit, xs)
+            self.last_hidden = last[:, :c.hidden]
             return self._head(x, mv, nlog, greedy)
         x = self.ops.embed(self.w["embed"], mv["tok"])
         if x_add is not None and self.input_rows:
@@ -979,7 +1108,7 @@ class Executor:
         mv["snrows"].copy_(torch.tensor(list(keep), dtype=torch.int32), non_blocking=False)
         mr = max(max(keep), 1)
         if (self._last_graph_key is not None and self.profile is None
-                and ((self._replay_fused(mr) and "gdn" in self.kinds) or "cdelta" in self.kinds)):
+                and ((self._replay_fused(mr) and "gdn" in self.kinds) or {"cdelta", "ssm"} & set(self.kinds) or self.canon_at)):
             # The verify step ran as a CUDA graph, so the projections it saved sit in that graph's buffers: the replay
             # (one fused launch per GDN layer, the kept counts are device data) is captured once per forward graph and
             # replayed with it. Eager verify steps allocate fresh projections every time and replay eagerly.
@@ -1001,9 +1130,12 @@ class Executor:
     def _replay_layers(self, mv, mr: int) -> None:
         c, w, ops = self.cfg, self.w, self.ops
         for run in self.runs:
-            if c.layers[run.layer].mixer == "cdelta":
+            mixer = c.layers[run.layer].mixer
+            if mixer in ("cdelta", "ssm"):
                 proj = self.verify_proj[run.index]
-                self._cdelta(proj, run, mv, [SegGroup(0, mv["sslot"].numel(), 0, proj.shape[0], mr)], True)
+                (self._cdelta if mixer == "cdelta" else self._ssm)(proj, run, mv, [SegGroup(0, mv["sslot"].numel(), 0, proj.shape[0], mr)], True)
+        for at, j in self.canon_at.items():
+            ops.conv_tail(self.conv_state["canon"][:, j], self.verify_proj[at], mv["sslot"], mv["srow0"], mv["snrows"])
         for i, kind in enumerate(self.kinds):
             if kind != "gdn":
                 continue
@@ -1097,7 +1229,7 @@ class Executor:
                      and self.profile is None and x_add is None and not self.dump_layers)
         tree = batch.tree
         if tree:
-            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and not {"mla", "latent", "gqa", "cdelta"} & set(self.kinds), \
+            assert not batch.commit and max_seg_rows <= TREE_MAX_ROWS and not {"mla", "latent", "gqa", "cdelta", "ssm"} & set(self.kinds), \
                 "verify trees: commit=False, at most TREE_MAX_ROWS rows per segment, attention / GDN layers"
             assert self.tp is None or self.tp.world == 1 or not self.tp.sp_ready(T)
         logit_rows = self._upload(batch)

@@ -66,13 +66,19 @@ _LISTED_SUB = {
                 **{n: f"mix.{n}" for n in ("q", "k", "v", "g", "lq1", "lk1", "lq2", "lk2")},
                 **{n: f"mlp.{n}" for n in ("gate", "up", "down", "router")}, "experts_gate_up": ("mlp.e{}.gate", "mlp.e{}.up"),
                 "experts_down": ("mlp.e{}.down",)},
+    "pironex": {"pre_norm": "norm1", "mix_norm": "norm1b", "ffn_pre_norm": "norm2", "ffn_norm": "norm2b", "mix_canon": "canon1", "ffn_canon": "canon2",
+                "dwa": "dwa", "out_proj": "mix.o", "q_norm": "mix.q.norm", "k_norm": "mix.k.norm", "kv_a": "mix.dkv", "kv_a_norm": "mix.dkv.norm",
+                "k_b": "mix.uk", "v_b": "mix.uv", "xbc_conv": "mix.conv", "xbc_bias": "mix.conv.b", "skip": "mix.D", "gnorm_w": "mix.norm",
+                **{n: f"mix.{n}" for n in ("q", "k", "v", "in", "A_log", "dt_bias")}, "router": "mlp.router",
+                "experts_gate_up": ("mlp.e{}.gate", "mlp.e{}.up"), "experts_down": ("mlp.e{}.down",),
+                "shared_gate": "mlp.shared.sg", "shared_gate_up": ("mlp.shared.gate", "mlp.shared.up"), "shared_down": ("mlp.shared.down",)},
 }
 
 
 def _load_listed(st: SafeTensors, cfg: ModelConfig, dtype) -> Dict[str, torch.Tensor]:
     """A checkpoint of a model of listed layers under engine names; every tensor's shape is checked against the configuration.
     Widths that only the tensors tell (the low ranks of channel-delta layers) are filled into it."""
-    sub = _LISTED_SUB["rakizen" if cfg.parallel else "zototar" if any(l.mixer == "latent" for l in cfg.layers) else "dofunex"]
+    sub = _LISTED_SUB["pironex" if cfg.canon or cfg.depth_average else "rakizen" if cfg.parallel else "zototar" if any(l.mixer == "latent" for l in cfg.layers) else "dofunex"]
     for i, l in enumerate(cfg.layers):
         if l.mixer == "cdelta":
             for field, base in (("decay_rank", "a1"), ("gate_rank", "g1")):

@@ -33,23 +33,26 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
     if cfg.out_norm:
         out[p + "mix_norm"] = (h,)
     if l.mixer == "latent":
-        out.update({p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,), p + "q_b": (l.heads * l.dim, l.q_rank)})
+        if l.q_rank:
+            out.update({p + "q_a": (l.q_rank, h), p + "q_a_norm": (l.q_rank,), p + "q_b": (l.heads * l.dim, l.q_rank)})
+        else:
+            out[p + "q"] = (l.heads * (l.dim + l.rot_dims), h)
         if l.kv_from is None:
-            out[p + "kv_a"] = (l.kv_rank, h)
+            out[p + "kv_a"] = (l.kv_rank + l.rot_dims, h)
             out[p + "kv_a_norm"] = (l.kv_rank,)
         out[p + "k_b"] = (l.heads * l.dim, l.kv_rank)
         out[p + "v_b"] = (l.heads * l.vdim, l.kv_rank)
         out[p + "out_proj"] = (h, l.heads * l.vdim)
     elif l.mixer == "gqa":
-        kd = l.maps * l.dim
-        for n, heads, d in (("q", l.heads, kd), ("k", l.kv_heads, kd)) + (() if l.key_values else (("v", l.kv_heads, l.vdim),)):
+        kd, own = l.maps * l.dim, l.kv_from is None
+        for n, heads, d in (("q", l.heads, kd),) + ((("k", l.kv_heads, kd),) if own else ()) + ((("v", l.kv_heads, l.vdim),) if own and not l.key_values else ()):
             out[p + n] = (heads * d, h)
             if l.bias:
                 out[p + n + "_bias"] = (heads * d,)
         if l.sink:
             out[p + "sink"] = (l.heads,)
         if l.row_norm:
-            out.update({p + "q_norm": (l.heads * kd,), p + "k_norm": (l.kv_heads * kd,)})
+            out.update({p + "q_norm": (l.heads * kd,), **({p + "k_norm": (l.kv_heads * kd,)} if own else {})})
         if l.maps == 2:
             out.update({p + n: (l.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
         if l.out_gate:
@@ -57,6 +60,10 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
         out[p + "out_proj"] = (h, l.heads * l.vdim)
         if l.bias:
             out[p + "out_bias"] = (h,)
+    elif l.mixer == "ssm":
+        nv, ch = l.heads * l.vdim, l.heads * l.vdim + 2 * l.kv_heads * l.dim
+        out.update({p + "in": (nv + ch + l.heads, h), p + "xbc_conv": (ch, l.conv), p + "xbc_bias": (ch,), p + "A_log": (l.heads,), p + "dt_bias": (l.heads,),
+                    p + "skip": (l.heads,), p + "gnorm_w": (nv,), p + "out_proj": (h, nv)})
     else:
         nk, nv = l.kv_heads * l.dim, l.heads * l.vdim
         for n, rows in (("q", nk), ("k", nk), ("v", nv)):
@@ -65,13 +72,21 @@ def listed_weight_shapes(cfg: ModelConfig, i: int) -> Dict[str, tuple]:
         out.update({p + "b": (l.heads, h), p + "A_log": (l.heads,), p + "dt_bias": (l.heads * l.dim,), p + "gnorm_w": (l.vdim,),
                     p + "a1": (l.decay_rank, h), p + "a2": (l.heads * l.dim, l.decay_rank), p + "g1": (l.gate_rank, h),
                     p + "g2": (nv, l.gate_rank), p + "out_proj": (h, nv)})
+    if cfg.canon:
+        out[p + "mix_canon"] = (h, cfg.canon)
+        if l.ff:
+            out[p + "ffn_canon"] = (h, cfg.canon)
+    if cfg.depth_average:
+        out[p + "dwa"] = (i + 2,)
+    if l.ff and not cfg.parallel:
+        if cfg.pre_norm:
+            out[p + "ffn_pre_norm"] = (h,)
+        out[p + "ffn_norm"] = (h,)
     if l.experts:
         out.update({p + "router": (l.experts, h), p + "experts_gate_up": (l.experts, 2 * l.ff, h), p + "experts_down": (l.experts, h, l.ff)})
+        if l.shared_ff:
+            out.update({p + "shared_gate": (1, h), p + "shared_gate_up": (1, 2 * l.shared_ff, h), p + "shared_down": (1, h, l.shared_ff)})
     elif l.ff:
-        if not cfg.parallel:
-            if cfg.pre_norm:
-                out[p + "ffn_pre_norm"] = (h,)
-            out[p + "ffn_norm"] = (h,)
         if l.act == "swiglu":
             out[p + "gate"] = (l.ff, h)
         out.update({p + "up": (l.ff, h), p + "down": (h, l.ff)})
@@ -141,7 +156,7 @@ def weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
 
 
 _F32_NAMES = ("A_log", "dt_bias", "router_bias")
-_F32_LISTED = ("norm", "gnorm_w", "_bias", "sink", "_conv", "loop_step", "lq1", "lk1", "lq2", "lk2")     # ... of models of listed layers
+_F32_LISTED = ("norm", "gnorm_w", "_bias", "sink", "_conv", "_canon", "dwa", "skip", "loop_step", "lq1", "lk1", "lq2", "lk2")     # ... of models of listed layers
 
 
 def keeps_f32(cfg: ModelConfig, name: str) -> bool:
@@ -161,8 +176,10 @@ def init_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="c
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32) * std
         if name.endswith("gnorm_w") or (cfg.layers and name.endswith("norm")):
             t = t + 1.0
-        if cfg.layers and name.endswith("_conv"):
+        if cfg.layers and name.endswith(("_conv", "_canon")):
             t = t / std * shape[1] ** -0.5
+        if name.endswith("dwa"):
+            t[-1] += 1.0
         t = t if keeps_f32(cfg, name) else t.to(dtype)
         w[name] = post(name, t) if post is not None else t
     return w
@@ -294,17 +311,29 @@ class LatentDims:
     q_rank: int
     kv_rank: int
     qr: int           # padded q_rank
-    lat: int          # padded kv_rank = cache row
-    hp: int           # padded head width, keys and values alike
+    lat: int          # padded kv_rank + rot = cache row: the latent, then the rotated key part
+    hp: int           # padded head width of the keys (unrotated part, then rotated part)
     scale: float
     source: int       # layer whose cache holds the latents
+    vp: int = 0       # ... of the values
+    vlat: int = 0     # columns of a cache row that the few-row kernel gathers as values (kv_rank at least)
+    dim: int = 0      # unrotated width of a key
+    rot: int = 0      # rotated width
+    window: int = 0   # a row sees itself and the window - 1 positions before it, 0 = all of them
+
+    def __post_init__(self):
+        object.__setattr__(self, "vp", self.vp or self.hp)
+        object.__setattr__(self, "vlat", self.vlat or self.lat)
 
 
 def latent_dims(cfg: ModelConfig, i: int) -> LatentDims:
     l = cfg.layers[i]
-    hp = head_width(max(l.dim, l.vdim))
-    return LatentDims(l.heads, l.q_rank, l.kv_rank, round_up(l.q_rank, 64), round_up(l.kv_rank, 64), hp, l.scale,
-                      i if l.kv_from is None else l.kv_from)
+    kd = l.dim + l.rot_dims
+    # 192 / 128 are one form of the prompt kernel, else it takes keys and values of one width
+    hp, vp = (192, 128) if 128 < kd <= 192 and l.vdim <= 128 else 2 * (head_width(max(kd, l.vdim)),)
+    lat, vlat = round_up(l.kv_rank + l.rot_dims, 64), round_up(l.kv_rank, 64)
+    return LatentDims(l.heads, l.q_rank, l.kv_rank, round_up(l.q_rank, 64), lat, hp, l.scale, i if l.kv_from is None else l.kv_from, vp,
+                      vlat if lat == 576 else lat, l.dim, l.rot_dims, l.window)
 
 
 def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
@@ -339,6 +368,9 @@ class GqaDims:
     diff: float = 0.0
     gate_off: int = -1      # column of the projection where the output gates start, -1 = none
     router_off: int = -1    # ... and the router's logits
+    rot_half: bool = False  # rotated pairs are (i, i + rot_dims / 2)
+    pool: int = 0           # blocks of this many positions before the window are seen as their means
+    source: int = -1        # layer whose cache holds keys and values, -1 = the layer itself
 
     @property
     def vw(self) -> int:
@@ -352,15 +384,19 @@ class GqaDims:
     @property
     def plain(self) -> bool:
         """No mechanism beyond what a causal grouped-query attention over one key and value width has."""
-        return self.maps == 1 and not self.row_norm and self.vw == self.dim
+        return self.maps == 1 and not self.row_norm and self.vw == self.dim and not self.rot_half
 
     @property
     def reach(self) -> int:
-        """Keys that a row can see, 0 = all."""
-        return self.window or self.chunk
+        """Keys that a row can see, 0 = no bound."""
+        return 0 if self.pool else self.window or self.chunk
 
     def first_visible(self, pos: int) -> int:
         return max(0, pos - self.window + 1) if self.window else pos - pos % self.chunk if self.chunk else 0
+
+    def blocks_visible(self, pos: int) -> int:
+        """Pooled blocks that the row at `pos` sees: those that end before its window."""
+        return max(0, pos - self.window + 1) // self.pool if self.pool else 0
 
 
 def head_width(d: int) -> int:
@@ -375,7 +411,8 @@ def gqa_dims(cfg: ModelConfig, i: int) -> GqaDims:
     g_off = v_off + l.kv_heads * l.vdim
     r_off = g_off + (l.heads * l.vdim if l.out_gate else 0)
     return GqaDims(l.heads, l.kv_heads, l.dim, head_width(max(kd, l.vdim)), l.scale, l.rot_dims, v_off, l.qk_norm, l.vdim, l.maps,
-                   l.row_norm, l.softcap, l.window, l.chunk, l.diff, g_off if l.out_gate else -1, r_off if l.experts else -1)
+                   l.row_norm, l.softcap, l.window, l.chunk, l.diff, g_off if l.out_gate else -1, r_off if l.experts and cfg.parallel else -1,
+                   l.rot_half, l.pool, -1 if l.kv_from is None else l.kv_from)
 
 
 def rope_frequencies(l) -> torch.Tensor:
@@ -427,29 +464,69 @@ def delta_dims(cfg: ModelConfig, i: int) -> DeltaDims:
                      round_up(l.heads * l.vdim, 64))
 
 
+@dataclass(frozen=True)
+class SsmDims:
+    """Sizes of one state-space layer as its kernels see them: columns of the projection [z | x | B | C | dt]; the state of a head is
+    [state][vdim]."""
+
+    heads: int
+    groups: int
+    state: int
+    vdim: int
+    conv: int
+    norm_groups: int
+    ko: int           # padded heads * vdim
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """Columns that pass the short convolution: x | B | C."""
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def dt_off(self) -> int:
+        return self.inner + self.channels
+
+
+def ssm_dims(cfg: ModelConfig, i: int) -> SsmDims:
+    l = cfg.layers[i]
+    return SsmDims(l.heads, l.kv_heads, l.dim, l.vdim, l.conv, l.norm_groups, round_up(l.heads * l.vdim, 64))
+
+
 def _pack_latent(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
-    """* in_proj  rows = [q_a | kv_a]           one product for both latents of a token
+    """* in_proj  rows = [q_a | kv_a]           one product for both latents of a token; without a query latent [q | kv_a] at true widths
     * q_b      [heads * hp, qr]              per head zero-padded rows, so queries come out at the padded width
-    * kv_up    [2 * heads * hp, lat]         key rows of every head, then value rows: expands latents for prompt rows
-    * k_abs    [heads, lat, hp]              W_uk^T per head: folds the key projection into a decode row's query
-    * v_up     [heads, hp, lat]              W_uv per head (a view of kv_up): latent-space outputs to values
-    * out_proj [width, heads * hp]"""
+    * kv_up    [heads * (hp + vp), lat]      key rows of every head, then value rows: expands latents for prompt rows. The rotated part
+                                             of a cache row passes to every head's keys through ones
+    * k_abs    [heads, lat, hp]              W_uk^T per head (and the same ones): folds the key projection into a decode row's query
+    * v_up     [heads, vp, vlat]             W_uv per head: latent-space outputs to values
+    * out_proj [width, heads * vp]"""
     l, p, d = cfg.layers[i], f"l{i}.", latent_dims(cfg, i)
-    parts = [_pad(w[p + "q_a"], d.qr, W)]
-    out[p + "q_a_norm"] = _pad(w[p + "q_a_norm"].float(), d.qr)
+    if l.q_rank:
+        parts = [_pad(w[p + "q_a"], d.qr, W)]
+        out[p + "q_a_norm"] = _pad(w[p + "q_a_norm"].float(), d.qr)
+        q_b = _pad(w[p + "q_b"].view(l.heads, l.dim, l.q_rank), l.heads, d.hp, d.qr)
+        out[p + "q_b"] = q_b.view(l.heads * d.hp, d.qr)
+    else:
+        parts = [_pad(w[p + "q"], w[p + "q"].shape[0], W)]
+        out[p + "inv_freq"] = rope_frequencies(l).to(w[p + "q"].device)
     if l.kv_from is None:
-        parts.append(_pad(w[p + "kv_a"], d.lat, W))
+        parts.append(_pad(w[p + "kv_a"], d.lat if l.q_rank else l.kv_rank + l.rot_dims, W))
         out[p + "kv_a_norm"] = _pad(w[p + "kv_a_norm"].float(), d.lat)
-    out[p + "in_proj"] = torch.cat(parts)
-    q_b = _pad(w[p + "q_b"].view(l.heads, l.dim, l.q_rank), l.heads, d.hp, d.qr)
-    out[p + "q_b"] = q_b.view(l.heads * d.hp, d.qr)
+    rows = torch.cat(parts)
+    out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     k = _pad(w[p + "k_b"].view(l.heads, l.dim, l.kv_rank), l.heads, d.hp, d.lat)
-    v = _pad(w[p + "v_b"].view(l.heads, l.vdim, l.kv_rank), l.heads, d.hp, d.lat)
+    for j in range(l.rot_dims):
+        k[:, l.dim + j, l.kv_rank + j] = 1.0
+    v = _pad(w[p + "v_b"].view(l.heads, l.vdim, l.kv_rank), l.heads, d.vp, d.lat)
     out[p + "kv_up"] = torch.cat([k.view(-1, d.lat), v.view(-1, d.lat)])
     out[p + "k_abs"] = k.transpose(1, 2).contiguous()
-    out[p + "v_up"] = out[p + "kv_up"][l.heads * d.hp:].view(l.heads, d.hp, d.lat)
-    o = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.hp)
-    out[p + "out_proj"] = o.view(W, l.heads * d.hp)
+    out[p + "v_up"] = out[p + "kv_up"][l.heads * d.hp:].view(l.heads, d.vp, d.lat)[..., :d.vlat].contiguous()
+    o = _pad(w[p + "out_proj"].view(cfg.hidden, l.heads, l.vdim), W, l.heads, d.vp)
+    out[p + "out_proj"] = o.view(W, l.heads * d.vp)
 
 
 def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
@@ -458,8 +535,8 @@ def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> Non
       product over their joined operands
     * lam      [1] weight of the second map"""
     l, p, d = cfg.layers[i], f"l{i}.", gqa_dims(cfg, i)
-    names = ("q", "k") if l.key_values else ("q", "k", "v")
-    rows = torch.cat([w[p + n] for n in names] + ([w[p + "g"]] if l.out_gate else []) + ([w[p + "router"]] if l.experts else []))
+    names = ("q",) if l.kv_from is not None else ("q", "k") if l.key_values else ("q", "k", "v")
+    rows = torch.cat([w[p + n] for n in names] + ([w[p + "g"]] if l.out_gate else []) + ([w[p + "router"]] if l.experts and cfg.parallel else []))
     out[p + "in_proj"] = _pad(rows, round_up(rows.shape[0], 8), W)
     if l.bias:
         out[p + "in_bias"] = _pad(torch.cat([w[p + n + "_bias"].float() for n in names]), round_up(rows.shape[0], 8))
@@ -467,7 +544,8 @@ def _pack_gqa(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> Non
     if l.sink:
         out[p + "sink"] = w[p + "sink"].float().contiguous()
     if l.row_norm:
-        out[p + "q_norm"], out[p + "k_norm"] = w[p + "q_norm"].float().contiguous(), w[p + "k_norm"].float().contiguous()
+        for n in ("q_norm", "k_norm") if l.kv_from is None else ("q_norm",):
+            out[p + n] = w[p + n].float().contiguous()
     if l.maps == 2:
         dot = lambda a, b: torch.exp((w[p + a].float() * w[p + b].float()).sum())
         out[p + "lam"] = (dot("lq1", "lk1") - dot("lq2", "lk2") + l.diff).view(1)
@@ -492,7 +570,37 @@ def _pack_cdelta(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> 
     out[p + "out_proj"] = _pad(w[p + "out_proj"], W, d.ko)
 
 
-_PACK = {"latent": _pack_latent, "gqa": _pack_gqa, "cdelta": _pack_cdelta}
+def _pack_ssm(cfg: ModelConfig, w: Weights, i: int, W: int, out: Weights) -> None:
+    """* in_proj  rows = [z | x | B | C | dt]
+    * conv     [taps, channels], conv_bias; A [heads] = -exp(A_log)
+    * out_proj [width, ko]"""
+    l, p, d = cfg.layers[i], f"l{i}.", ssm_dims(cfg, i)
+    out[p + "in_proj"] = _pad(w[p + "in"], round_up(w[p + "in"].shape[0], 8), W)
+    out[p + "conv"] = w[p + "xbc_conv"].float().t().contiguous()
+    out[p + "conv_bias"] = w[p + "xbc_bias"].float().contiguous()
+    out[p + "A"] = -torch.exp(w[p + "A_log"].float())
+    for n in ("dt_bias", "skip", "gnorm_w"):
+        out[p + n] = w[p + n].float().contiguous()
+    out[p + "out_proj"] = _pad(w[p + "out_proj"], W, d.ko)
+
+
+def _pack_experts(cfg: ModelConfig, w: Weights, p: str, l, W: int, out: Weights) -> None:
+    """* experts_gate_up [experts, 2 F, width], experts_down [experts, width, F]; shared_gate_up, shared_down the same of the shared expert
+    * router  rows = [router | shared expert's gate], unless the router rides on another product"""
+    def stack(name, n, ff):
+        F = round_up(ff, 64)
+        gu = _pad(w[f"{p}{name}_gate_up"].view(n, 2, ff, cfg.hidden), n, 2, F, W)
+        out[f"{p}{name}_gate_up"] = gu.view(n, 2 * F, W)
+        out[f"{p}{name}_down"] = _pad(w[f"{p}{name}_down"], n, W, F)
+    stack("experts", l.experts, l.ff)
+    if l.shared_ff:
+        stack("shared", 1, l.shared_ff)
+    if not cfg.parallel:
+        rows = torch.cat([w[p + "router"]] + ([w[p + "shared_gate"]] if l.shared_ff else []))
+        out[p + "router"] = _pad(rows, round_up(rows.shape[0], 8), W)
+
+
+_PACK = {"latent": _pack_latent, "gqa": _pack_gqa, "cdelta": _pack_cdelta, "ssm": _pack_ssm}
 
 
 def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
@@ -501,8 +609,8 @@ def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
     them."""
     W = round_up(cfg.hidden, 64)
     vec = lambda n, f=1.0: _pad(w[n].float() * f, W)
-    out: Weights = {"embed": _pad(w["embed"], cfg.vocab, W), "lm_head": _pad(w["lm_head"], w["lm_head"].shape[0], W),
-                    "final_norm": vec("final_norm", cfg.logit_scale)}
+    out: Weights = {"embed": _pad(w["embed"], cfg.vocab, W), "final_norm": vec("final_norm", cfg.logit_scale)}
+    out["lm_head"] = out["embed"] if cfg.tie_embeddings else _pad(w["lm_head"], w["lm_head"].shape[0], W)
     if cfg.gram_buckets:
         out["bigram"] = _pad(w["bigram"], cfg.gram_buckets + 1, W)
     if cfg.parallel:
@@ -518,22 +626,26 @@ def pack_listed(cfg: ModelConfig, w: Weights) -> Weights:
         if cfg.parallel:
             out[p + "pre_norm_bias"] = vec(p + "pre_norm_bias")
             if l.experts:
-                F = round_up(l.ff, 64)
-                gu = _pad(w[p + "experts_gate_up"].view(l.experts, 2, l.ff, cfg.hidden), l.experts, 2, F, W)
-                out[p + "experts_gate_up"] = gu.view(l.experts, 2 * F, W)
-                out[p + "experts_down"] = _pad(w[p + "experts_down"], l.experts, W, F)
+                _pack_experts(cfg, w, p, l, W, out)
             elif l.ff:
                 out[p + "gate_up"] = torch.cat([_pad(w[p + n], round_up(l.ff, 64), W) for n in ("gate", "up")])
             continue
         out[p + "mix_norm"] = vec(p + "mix_norm", cfg.residual_mult)
+        for n in (("mix_canon", "ffn_canon") if l.ff else ("mix_canon",)) if cfg.canon else ():
+            out[p + n] = _pad(w[p + n].float().t(), cfg.canon, W)                          # [taps, width]
+        if cfg.depth_average:
+            out[p + "dwa"] = w[p + "dwa"].float().contiguous()
         if l.ff:
             F = round_up(l.ff, 64)
-            up = _pad(w[p + "up"], F, W)
-            if l.act == "swiglu":
-                out[p + "gate_up"] = torch.cat([_pad(w[p + "gate"], F, W), up])
+            if l.experts:
+                _pack_experts(cfg, w, p, l, W, out)
             else:
-                out[p + "up"] = up
-            out[p + "down"] = _pad(w[p + "down"], W, F)
+                up = _pad(w[p + "up"], F, W)
+                if l.act == "swiglu":
+                    out[p + "gate_up"] = torch.cat([_pad(w[p + "gate"], F, W), up])
+                else:
+                    out[p + "up"] = up
+                out[p + "down"] = _pad(w[p + "down"], W, F)
             out[p + "ffn_norm"] = vec(p + "ffn_norm", cfg.residual_mult)
             if cfg.pre_norm:
                 out[p + "ffn_pre_norm"] = vec(p + "ffn_pre_norm")

@@ -19,33 +19,50 @@ UNIT_EPS = 1e-6       # inside the root of the delta rule's unit queries and key
 class TorchMixers:
     def gqa_prep(self, proj, d, bias, inv_freq, row_slot, row_pos, block_table, k_cache, v_cache, kv_block, eps, norms=None):
         """Biases, norms over whole rows (`norms`: their weights for q and k), rotation and norms per head of a step's queries and keys;
-        keys and values into their pages. Returns q [T, maps * heads, hp]."""
-        T, M = proj.shape[0], d.maps
+        keys and values into their pages (a layer with another one's keys projects queries only). Returns q [T, maps * heads, hp]."""
+        T, M, own = proj.shape[0], d.maps, d.source < 0
         p = proj.float() if bias is None else proj.float() + bias[:proj.shape[1]]
         nq, nk = d.heads * M * d.dim, d.kv_heads * M * d.dim
-        q, k = p[:, :nq], p[:, nq:nq + nk]
+        q, k = p[:, :nq], p[:, nq:nq + nk] if own else None
         if d.row_norm:
-            q, k = (x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w for x, w in zip((q, k), norms))
-        q, k = q.reshape(T, d.heads * M, d.dim), k.reshape(T, d.kv_heads * M, d.dim)
-        v = p[:, d.v_off:d.v_off + d.kv_heads * d.vw].reshape(T, d.kv_heads, d.vw)
+            q, k = (None if x is None else x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w for x, w in zip((q, k), norms))
+        q = q.reshape(T, d.heads * M, d.dim)
         ang = row_pos.double()[:, None] * inv_freq[None, :]
         c, s = ang.cos().float()[:, None], ang.sin().float()[:, None]
 
         def turn(x):
-            a, b = x[..., 0:d.rot_dims:2], x[..., 1:d.rot_dims:2]
-            x = torch.cat([torch.stack([a * c - b * s, b * c + a * s], -1).flatten(-2), x[..., d.rot_dims:]], -1)
+            if d.rot_half:
+                a, b = x[..., :d.rot_dims // 2], x[..., d.rot_dims // 2:d.rot_dims]
+                x = torch.cat([a * c - b * s, b * c + a * s, x[..., d.rot_dims:]], -1)
+            else:
+                a, b = x[..., 0:d.rot_dims:2], x[..., 1:d.rot_dims:2]
+                x = torch.cat([torch.stack([a * c - b * s, b * c + a * s], -1).flatten(-2), x[..., d.rot_dims:]], -1)
             return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) if d.qk_norm else x
         pad = lambda x: F.pad(x, (0, d.hp - x.shape[-1]))
-        page, off = block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block
-        k_cache[page, off] = pad(turn(k).reshape(T, d.kv_heads, M * d.dim)).to(k_cache.dtype)
-        v_cache[page, off] = pad(v).to(v_cache.dtype)
+        if own:
+            v = p[:, d.v_off:d.v_off + d.kv_heads * d.vw].reshape(T, d.kv_heads, d.vw)
+            page, off = block_table[row_slot.long(), row_pos.long() // kv_block].long(), row_pos.long() % kv_block
+            k_cache[page, off] = pad(turn(k.reshape(T, d.kv_heads * M, d.dim)).reshape(T, d.kv_heads, M * d.dim)).to(k_cache.dtype)
+            v_cache[page, off] = pad(v).to(v_cache.dtype)
         q = turn(q)
         if M == 2:                                                    # the other map's columns of a query are zeros
             q = torch.stack([F.pad(q[:, 0::2], (0, d.dim)), F.pad(q[:, 1::2], (d.dim, 0))], 2).flatten(1, 2)
         return pad(q).to(self.dtype)
 
+    def pool_keys(self, d, k_cache, v_cache, pooled, seg_slot, seg_pos0, seg_nrows, max_rows, block_table, kv_block):
+        """Means of the cached keys and values of every block of `pool` positions whose last one is in the step. A mean lies in the page of
+        the block's last position, at that position's number of whole blocks in the page."""
+        P = d.pool
+        for s in range(len(seg_slot)):
+            p0, n, slot = int(seg_pos0[s]), int(seg_nrows[s]), int(seg_slot[s])
+            for e in range((p0 + P) // P * P - 1, p0 + n, P):
+                at = torch.arange(e - P + 1, e + 1)
+                page, off = block_table[slot, at // kv_block].long(), at % kv_block
+                for cache, means in zip((k_cache, v_cache), pooled):
+                    means[int(page[-1]), e % kv_block // P] = cache[page, off].float().mean(0).to(means.dtype)
+
     def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out, lam=None,
-                      gate=None, eps=0.0):
+                      gate=None, eps=0.0, pooled=None):
         """Causal attention of the rows of `group` over what the layer's mask leaves of the cache; q [T, maps * heads, hp], out
         [T, heads, hp], row tables of all T rows. Two maps: `lam` [1] weighs the second. `gate` [T, heads * vdim]: logits of the
         outputs' sigmoid gates."""
@@ -56,12 +73,16 @@ class TorchMixers:
             pages = block_table[s, :(n + kv_block - 1) // kv_block].long()
             k = k_cache[pages].flatten(0, 1)[lo:n, own].float()
             v = v_cache[pages].flatten(0, 1)[lo:n, own].float()
+            if d.pool:
+                end = torch.arange(d.blocks_visible(n - 1)) * d.pool + d.pool - 1
+                bp = block_table[s, end // kv_block].long()
+                k, v = (torch.cat([m[bp, end % kv_block // d.pool][:, own].float(), x]) for m, x in zip(pooled, (k, v)))
             sc = torch.einsum("hd,jhd->hj", q[r].float(), k) * d.scale
             if d.softcap:
                 sc = d.softcap * torch.tanh(sc / d.softcap)
             if sink is not None:
                 sc = torch.cat([sc, sink[:, None]], 1)
-            o = torch.einsum("hj,jhd->hd", torch.softmax(sc, -1)[:, :n - lo], v)
+            o = torch.einsum("hj,jhd->hd", torch.softmax(sc, -1)[:, :len(k)], v)
             if d.maps == 2:
                 o = o[0::2] - lam * o[1::2]
                 o = o / torch.sqrt(o.pow(2).sum(-1, keepdim=True) / d.vw + eps) * (1 - d.diff)
@@ -70,14 +91,49 @@ class TorchMixers:
             out[r] = o.to(out.dtype)
         return out
 
-    def expert_rows(self, h, ids, w_gu, w_down):
-        """Rows of a token's experts, one per (token, pick): [T * top, width] fp32."""
+    def expert_rows(self, h, ids, w_gu, w_down, limit=0.0, shared=None):
+        """Rows of a token's experts, one per (token, pick): [T * top, width] fp32. `limit`: clamped gated units instead of swiglu; `shared` =
+        (gate | up, down, limit): the expert one past the last."""
         T, K = ids.shape
         out = torch.empty(T * K, w_down.shape[1], dtype=torch.float32, device=h.device)
         for p, e in enumerate(ids.reshape(-1).tolist()):
-            g, u = (w_gu[e].float() @ h[p // K].float()).chunk(2)
-            out[p] = w_down[e].float() @ (F.silu(g) * u).to(self.dtype).float()
+            gu, dn, lim = (w_gu[e], w_down[e], limit) if e < w_down.shape[0] else (shared[0][0], shared[1][0], shared[2])
+            a = self.glu_act(gu.float() @ h[p // K].float(), lim)
+            out[p] = dn.float() @ a.to(self.dtype).float()
         return out
+
+    @staticmethod
+    def glu_act(gu, limit):
+        g, u = gu.chunk(2, -1)
+        if not limit:
+            return F.silu(g) * u
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+    def ssm(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, row_slot, row_pos, eps, commit=True):
+        """Rows of the projection [z | x | B | C | dt] through the state-space recurrence of one layer -> [T, ko]. `w`: the layer's tensors by
+        name."""
+        T, H, G, N, V = proj.shape[0], d.heads, d.groups, d.state, d.vdim
+        c = self.conv_rows(proj[:, d.inner:d.dt_off], w["conv"], conv_state, row_slot, row_pos, bias=w["conv_bias"], silu=True).float()
+        dt = F.softplus(proj[:, d.dt_off:d.dt_off + H].float() + w["dt_bias"], threshold=80.0)
+        a = torch.exp(w["A"] * dt)
+        own = [h // (H // G) for h in range(H)]
+        x = c[:, :d.inner].reshape(T, H, V)
+        B, C = (c[:, d.inner + j * G * N:d.inner + (j + 1) * G * N].reshape(T, G, N)[:, own] for j in (0, 1))
+        y = torch.zeros(T, d.ko, dtype=torch.float32, device=proj.device)
+        for s in range(len(seg_slot)):
+            n, r0, slot = int(seg_nrows[s]), int(seg_row0[s]), int(seg_slot[s])
+            S = rec_state[slot].clone()
+            for t in range(r0, r0 + n):
+                S = S * a[t][:, None, None] + dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
+                y[t, :d.inner] = (torch.einsum("hnv,hn->hv", S, C[t]) + w["skip"][:, None] * x[t]).flatten()
+            if commit and n > 0:
+                rec_state[slot] = S
+        if commit:
+            self.conv_tail(conv_state, proj[:, d.inner:d.dt_off], seg_slot, seg_row0, seg_nrows)
+        g = (y[:, :d.inner] * F.silu(proj[:, :d.inner].float())).reshape(T, d.norm_groups, -1)
+        y[:, :d.inner] = (g / torch.sqrt(g.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * w["gnorm_w"]
+        return y.to(self.dtype)
 
     def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
         """Rows of the fused projection through the delta rule of one layer -> [T, ko]. `w`: the layer's tensors by name."""

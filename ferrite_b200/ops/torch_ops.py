@@ -320,7 +320,14 @@ class TorchOps(TorchLatent, TorchMixers, TorchExtras):
         return y
 
     # ---- mixture of experts ---------------------------------------------------------------------------
-    def moe_route(self, logits, bias, mode, top_k, n_groups, topk_groups, scale):
+    def moe_route(self, logits, bias, mode, top_k, n_groups, topk_groups, scale, n_exp=0, shared_col=-1, shared_id=-1):
+        if mode == 2:                        # softmax over the chosen logits; the shared expert as one more pick
+            val, idx = torch.sort(logits[:, :n_exp or logits.shape[1]].float(), dim=-1, descending=True, stable=True)
+            idx, wts = idx[:, :top_k], torch.softmax(val[:, :top_k], -1) * scale
+            if shared_id >= 0:
+                idx = torch.cat([idx, torch.full_like(idx[:, :1], shared_id)], 1)
+                wts = torch.cat([wts, torch.sigmoid(logits[:, shared_col:shared_col + 1].float())], 1)
+            return idx.to(torch.int32), wts
         from ..config import ModelConfig
         from ..models.ref import route
         c = ModelConfig(router="softmax" if mode == 0 else "sigmoid_group", top_k=top_k, n_groups=n_groups,
