@@ -22,6 +22,16 @@ typedef struct HeadMix {
   int vdim;
 } HeadMix;
 
+// Means of blocks of `size` positions that a row under a window sees beside it: the blocks that end before the window. Few rows: mean rows
+// [page][per page][kv heads][hd], at the page of a block's last position; prompts: gathered rows, those of segment i from start[i] on, `rows` in all.
+typedef struct PoolKeys {
+  const void* k;
+  const void* v;
+  int size;
+  const int* start;
+  long rows;
+} PoolKeys;
+
 #ifdef __cplusplus
 extern "C" {
 #endif
@@ -47,6 +57,8 @@ int fb_gemv_bf16(void* Y, const void* X, const void* W, const void* norm_w, cons
 // ---- gemm_tcgen05.cu ----
 // Y[M][N] = X[M][K] * W[N][K]^T (+ res), or SwiGLU over W = [gate rows | up rows] (2N rows). bf16 in/out,
 // fp32 accumulation in TMEM. workspace/counters are needed only when split_k > 1.
+int fb_gemm_bf16_glu(void* Y, const void* X, const void* W, const void* res, int M, int N, int K, long ldx, long ldy,
+                     int mode, float limit, int split_k, float* workspace, int* counters, int* status, int sm_count, cudaStream_t s);
 int fb_gemm_bf16(void* Y, const void* X, const void* W, const void* res, int M, int N, int K, long ldx, long ldy,
                  int mode, int split_k, float* workspace, int* counters, int* status, int sm_count, cudaStream_t s);
 long fb_gemm_workspace_bytes(int M, int N, int split_k);
@@ -110,8 +122,8 @@ int fb_attn_decode_mma(void* out, float* o_part, float* ml_part, const void* q, 
                        int nkv, int hd, int nsplit, int gated, float scale, int exact_p, const KeyBounds* kb, int row_first, cudaStream_t s);
 int fb_attn_decode_keys(float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache, const int* seg_slot,
                         const int* seg_row0, const int* seg_nrows, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block,
-                        int nseg, int max_rows, int rows, int nq, int nkv, int hd, int nsplit, float scale, const KeyBounds* kb, int row_first,
-                        int* status, cudaStream_t s);
+                        int nseg, int max_rows, int rows, int nq, int nkv, int hd, int nsplit, float scale, const KeyBounds* kb, const PoolKeys* pool,
+                        int row_first, int* status, cudaStream_t s);
 // 4-bit KV cache: codes [..][hd/2] bytes, scales [..][2 * hd/32] fp32 per (token, kv head) row (K groups, V groups)
 int fb_attn_prep_q4(void* q_out, void* k_cache4, void* v_cache4, float* kv_scale, const void* proj, long proj_stride,
                     const void* q_norm, const void* k_norm, const float* inv_freq, const int* row_slot, const int* row_pos,
@@ -141,8 +153,9 @@ int fb_kv_dequant_qn(void* k_out, void* v_out, const void* k_cache, const void* 
 int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                        long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                        const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg, int max_rows,
-                       long q_rows, long cache_rows, int nq, int nkv, int hd, int gated, float scale, int exact_p,
-                       long kv_stride, const float* sink, const KeyBounds* kb, long ldo, int out_f32, const HeadMix* mix, int* status, cudaStream_t s);
+                       long q_rows, long cache_rows, int nq, int nkv, int hd, int hdv, int gated, float scale, int exact_p,
+                       long kv_stride, const float* sink, const KeyBounds* kb, const PoolKeys* pool, long ldo, int out_f32, const HeadMix* mix,
+                       int* status, cudaStream_t s);
 
 // ---- gdn.cu ----
 int fb_gdn_conv(void* out, const void* proj, long proj_stride, const void* conv_w, const void* conv_state,

@@ -103,7 +103,11 @@ int fb_moe_down_fp4(float* yp, const void* act, const void* wq, const void* ws, 
                     int hidden, int inter, int e_lo, int e_hi, cudaStream_t s);
 int fb_nvfp4_dequant(void* out, const void* wq, const void* ws, float gscale, long elements, cudaStream_t s);
 int fb_expert_rows_f32(float* yp, float* act, const float* x, const float* w_gu, const float* w_down, const int* ids, int pairs, int top_k,
-                       int hidden, int inter, int n_exp, cudaStream_t s);
+                       int hidden, int inter, int n_exp, int ld_act, float limit, const float* shared_gu, const float* shared_down,
+                       int shared_inter, float shared_limit, cudaStream_t s);
+int fb_expert_rows(float* yp, void* act, const void* x, const void* w_gu, const void* w_down, const int* ids, int pairs, int top_k, int hidden,
+                   int inter, int n_exp, int ld_act, float limit, const void* shared_gu, const void* shared_down, int shared_inter,
+                   float shared_limit, cudaStream_t s);
 int fb_moe_combine(void* out, const float* yp, const float* wts, const void* shared, const float* shared_gate,
                    const void* res, int rows, int top_k, int hidden, int out_f32, cudaStream_t s);
 
@@ -118,7 +122,7 @@ int fb_ag_gemm(void* Y, const void* W, const void* res, int M, int N, int K, lon
                unsigned spin_limit, int sm_count, cudaStream_t s);
 
 int fb_gemm_grouped(void* Y, const void* X, const void* W, const int* tile_start, const int* row_base, int experts,
-                    int max_rows, int N, int K, long ldx, long ldy, int mode, int* status, int sm_count, cudaStream_t s);
+                    int max_rows, int N, int K, long ldx, long ldy, int mode, float limit, int* status, int sm_count, cudaStream_t s);
 
 // Y[g] = X[g] W[g]^T for `groups` problems of one shape: X [groups * rows][K], W [groups][N][K], Y [groups * rows][N]
 int fb_gemm_batched(void* Y, const void* X, const void* W, int groups, int rows, int N, int K, int* status, int sm_count,
@@ -131,8 +135,8 @@ int fb_head_linear(void* y, const void* x, const void* W, int T, int heads, int 
 long fb_ep_workspace_bytes(int n_experts, int hidden, long cap_rows);
 long fb_ep_recv_offset(int n_experts, int hidden, long cap_rows);
 long fb_ep_out_offset(int n_experts, int hidden, long cap_rows);
-int fb_ep_moe(void* out, int out_f32, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
-              const void* shared, const float* shared_gate, const void* res, void* act, int* plan, int rows, int top_k,
+int fb_ep_moe(void* out, int out_f32, float limit, const void* x, const int* ids, const float* wts, const void* w_gu, const void* w_down,
+              const void* shared, const float* shared_gate, long gate_ld, const void* res, void* act, int* plan, int rows, int top_k,
               int n_experts, int hidden, int inter, long cap_rows, const void* const* peers, int rank, int world,
               uint32_t* ctr, int* status, unsigned spin_limit, int sm_count, cudaStream_t s);
 
@@ -168,8 +172,8 @@ int fb_embed_grams(float* x, void* xb, int copies, const void* table, const void
                    long buckets, long mul_prev, long mul_cur, int f32, int* status, cudaStream_t s);
 int fb_add_normed(float* x, void* xb, int xb_f32, long ldb, const void* y, int y_f32, const float* bias, const float* w,
                   const float* next_w, int rows, int width, int ld, long ldy, float eps, cudaStream_t s);
-int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int rows, int width, int ld, float eps, int f32,
-                 cudaStream_t s);
+int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int mean, int rows, int width, int ld, float eps,
+                 int f32, cudaStream_t s);
 int fb_add_layer_norm(float* x, void* xb, int f32, const void* y, int y_f32, long ldy, const float* yp, const float* wts, int top,
                       const float* next_w, const float* next_b, int rows, int width, int ld, float eps, cudaStream_t s);
 int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const float* q_norm, const float* kv_norm,
@@ -178,15 +182,16 @@ int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp, const flo
 int fb_softcap(float* y, int rows, int n, long ld, float cap, cudaStream_t s);
 int fb_relu2(void* y, const void* x, long ldx, int rows, int n, cudaStream_t s);
 int fb_latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
-                   const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat, int nsplit,
-                   float scale, int f32, int* status, cudaStream_t s);
+                   const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat, int vl,
+                   int window, int nsplit, float scale, int f32, int* status, cudaStream_t s);
 int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
                   const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen, const int* block_table,
-                  int max_blocks, int kv_block, int rows, int row_base, int heads, int lat, int nsplit, float scale, int* status,
-                  cudaStream_t s);
+                  int max_blocks, int kv_block, int rows, int row_base, int heads, int lat, int vl, int window, int nsplit, float scale,
+                  int* status, cudaStream_t s);
 int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache, const float* sink,
                 const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
-                int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb, long ldo, int f32, int* status, cudaStream_t s);
+                int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb, const PoolKeys* pool, long ldo, int f32, int* status,
+                cudaStream_t s);
 int fb_attn_merge(void* out, long ldo, const float* o_part, const float* ml_part, const float* sink, int rows, int heads, int nsplit, int hd,
                   cudaStream_t s);
 int fb_attn_merge_mix(void* out, long ldo, const float* o_part, const float* ml_part, const float* lam, const float* gate, long ldg,
@@ -200,7 +205,7 @@ int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, lo
                 int kv_heads, int dim, int hp, int rot, int v_off, int norm, float eps, int f32, int* status, cudaStream_t s);
 int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* q_norm, const float* k_norm,
                     const double* inv_freq, const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block,
-                    int rows, int heads, int kv_heads, int maps, int dim, int vdim, int hp, int rot, int v_off, float eps, int f32, int* status,
+                    int rows, int heads, int kv_heads, int maps, int dim, int vdim, int hp, int rot, int v_off, int half, float eps, int f32, int* status,
                     cudaStream_t s);
 
 // ---- cdelta.cu, cdelta_chunk.cu ----

@@ -5,6 +5,9 @@
 // where scores are softcapped. Here M is 16 pairs and a 64-key tile is cut over the four warps, 16 keys each: every warp keeps a softmax of
 // its own (maximum, sum, unnormalised output), the four are joined once at the end. K and V stream through two cp.async stages.
 //
+// POOL: the means of the blocks before a row's window come first in the list of keys that the splits share, in tiles of their own (a tile of
+// means is gathered row by row, since they lie in the pages of their blocks' last positions).
+//
 // grid (segments x row groups, kv heads, key splits). Rows see the keys up to their own, of a window or a chunk (`first_key`), scores may be
 // softcapped, softmax weights enter the PV product as a bf16 value plus its bf16 remainder. A CTA leaves the record of its split
 // (unnormalised o, maximum, sum) for the merges of `latent.cu`; the order of the joins is fixed, so results do not depend on scheduling.
@@ -35,13 +38,14 @@ __device__ __forceinline__ void dk_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <int HD>
+template <int HD, bool POOL>
 __global__ void __launch_bounds__(DK_THREADS)
 attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part, const __nv_bfloat16* __restrict__ q,
                         const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ seg_slot,
                         const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows, const int* __restrict__ row_kvlen,
                         const int* __restrict__ block_table, int max_blocks, int kv_block, int nq, int nkv, int nsplit, int groups_per_seg,
-                        int row_first, float scale_log2, int window, int chunk, float cap_log2, int* status) {
+                        int row_first, float scale_log2, int window, int chunk, float cap_log2, const __nv_bfloat16* __restrict__ k_mean,
+                        const __nv_bfloat16* __restrict__ v_mean, int pool, int* status) {
   constexpr int LD = HD + 8;                    // padded row (elements): conflict-free ldmatrix
   constexpr int CPR = HD / 8;                   // 16-byte pieces per row
   extern __shared__ __align__(16) unsigned char dk_smem[];
@@ -61,9 +65,12 @@ attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part,
   // rows of a segment follow one another: the last one sees the latest key, the first one the earliest
   const int kv_end = row_kvlen[row0 + rows_here - 1];
   const int first_lo = first_key(row_kvlen[row0] - 1, window, chunk), kv_lo = first_lo / DK_KEYS * DK_KEYS;
-  int per = (kv_end - kv_lo + nsplit - 1) / nsplit;
+  // list of keys: place u < shift is mean u (those of the last row's blocks), the others are token u - shift + kv_lo
+  const int nb = POOL ? first_key(kv_end - 1, window, 0) / pool : 0, shift = POOL ? (nb + DK_KEYS - 1) / DK_KEYS * DK_KEYS : 0;
+  const int at0 = POOL ? 0 : kv_lo, list_end = POOL ? shift + kv_end - kv_lo : kv_end;
+  int per = (list_end - at0 + nsplit - 1) / nsplit;
   per = (per + DK_KEYS - 1) / DK_KEYS * DK_KEYS;
-  const int lo = kv_lo + split * per, hi = min(kv_end, lo + per);
+  const int lo = at0 + split * per, hi = min(list_end, lo + per);
   // (row, head) pair m of this CTA -> its record
   auto record = [&](int m) { return ((size_t)(row0 + m / G) * nq + kvh * G + m % G) * nsplit + split; };
   if (lo >= hi) {                               // an empty split: the merge skips it
@@ -76,9 +83,26 @@ attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part,
     dk_cp16(sQ + m * LD + cc * 8, q + ((size_t)(row0 + (ok ? m / G : 0)) * nq + kvh * G + (ok ? m % G : 0)) * HD + cc * 8, ok);
   }
   auto load_tile = [&](int t0, int stage) {     // a tile lies in one page: both start on multiples of 64 keys
+    if constexpr (POOL) {
+      if (t0 < shift) {
+        const int per_page = (kv_block + pool - 1) / pool;
+#pragma unroll 4
+        for (int i = 0; i < DK_KEYS * CPR / DK_THREADS; ++i) {
+          const int c = tid + i * DK_THREADS, r = c / CPR, cc = c % CPR, e = (t0 + r) * pool + pool - 1;
+          const int blk = t0 + r < nb ? bt[e / kv_block] : -1;
+          if (blk < 0 && t0 + r < nb) set_status(status, ST_BOUNDS);
+          const size_t off = blk < 0 ? 0 : (((size_t)blk * per_page + e % kv_block / pool) * nkv + kvh) * HD + cc * 8;
+          dk_cp16(sK + (stage * DK_KEYS + r) * LD + cc * 8, k_mean + off, blk >= 0);
+          dk_cp16(sV + (stage * DK_KEYS + r) * LD + cc * 8, v_mean + off, blk >= 0);
+        }
+        dk_commit();
+        return;
+      }
+      t0 += kv_lo - shift;
+    }
     const int blk = bt[t0 / kv_block];
     if (blk < 0 && tid == 0) set_status(status, ST_BOUNDS);
-    const int live = blk < 0 ? 0 : min(DK_KEYS, hi - t0);
+    const int live = blk < 0 ? 0 : min(DK_KEYS, (POOL ? min(kv_end, hi + kv_lo - shift) : hi) - t0);
     const size_t base = blk < 0 ? 0 : (((size_t)blk * kv_block + t0 % kv_block) * nkv + kvh) * HD;
     const size_t ld = (size_t)nkv * HD;
 #pragma unroll
@@ -112,7 +136,9 @@ attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part,
     else dk_wait<0>();
     __syncthreads();
     const int t0 = lo + tile * DK_KEYS + warp * 16;          // this warp's 16 keys
-    if (t0 < hi && t0 + 15 >= first_lo) {
+    const bool means = POOL && t0 < shift;
+    const int off = POOL && !means ? kv_lo - shift : 0;      // from the place in the list to the token
+    if (t0 < hi && (means || t0 + off + 15 >= first_lo)) {
       const __nv_bfloat16* K = sK + (stage * DK_KEYS + warp * 16) * LD;
       const __nv_bfloat16* V = sV + (stage * DK_KEYS + warp * 16) * LD;
       float s[2][4] = {};
@@ -138,7 +164,11 @@ attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part,
             const int t = kbase + nt * 8 + e;
             float v = s[nt][2 * h + e] * scale_log2;
             if (cap_log2 > 0.f) v = cap_log2 * tanh_exp(v);
-            if (t >= kvl[h] || t < klo[h] || t >= hi) v = -INFINITY;
+            if constexpr (POOL) {
+              if (t >= hi || (means ? (t + 1) * pool > klo[h] : t + off >= kvl[h] || t + off < klo[h])) v = -INFINITY;
+            } else {
+              if (t >= kvl[h] || t < klo[h] || t >= hi) v = -INFINITY;
+            }
             s[nt][2 * h + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -216,16 +246,17 @@ attn_decode_keys_kernel(float* __restrict__ o_part, float* __restrict__ ml_part,
 using namespace fb;
 
 // Records of key splits as fb_attn_decode_mma leaves them (o_part [rows][nq][nsplit][hd], ml_part two floats each); scale of the scores; kb:
-// window, chunk and softcap, or null. Returns -20 for shapes it does not take: heads of 64 or 128 columns, max_rows * (nq / nkv) <= 16, pages
-// of a multiple of 64 keys.
+// window, chunk and softcap, or null; pool: means of the blocks before the window, or null. Returns -20 for shapes it does not take: heads of 64
+// or 128 columns, max_rows * (nq / nkv) <= 16 (with means: nq / nkv <= 16), pages of a multiple of 64 keys.
 extern "C" int fb_attn_decode_keys(float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache, const int* seg_slot,
                                    const int* seg_row0, const int* seg_nrows, const int* row_kvlen, const int* block_table, int max_blocks,
                                    int kv_block, int nseg, int max_rows, int rows, int nq, int nkv, int hd, int nsplit, float scale,
-                                   const KeyBounds* kb, int row_first, int* status, cudaStream_t s) {
+                                   const KeyBounds* kb, const PoolKeys* pool, int row_first, int* status, cudaStream_t s) {
   if (nseg <= 0 || rows <= 0) return 0;
   if (nkv <= 0 || nq % nkv || nsplit < 1) return -1;
   const int G = nq / nkv;
-  if ((hd != 64 && hd != 128) || (long)max_rows * G > DK_M || kv_block % DK_KEYS) return -20;
+  if ((hd != 64 && hd != 128) || (pool ? G : (long)max_rows * G) > DK_M || kv_block % DK_KEYS) return -20;
+  if (pool && (pool->size < 1 || !kb || !kb->window)) return -1;
   if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
   constexpr float LOG2E = 1.4426950408889634f;
   const float cap = kb ? kb->cap : 0.f;
@@ -238,7 +269,9 @@ extern "C" int fb_attn_decode_keys(float* o_part, float* ml_part, const void* q,
     return (int)launch_pdl(kern, grid, dim3(DK_THREADS), smem, s, o_part, ml_part, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache,
                            (const __nv_bfloat16*)v_cache, seg_slot, seg_row0, seg_nrows, row_kvlen, block_table, max_blocks, kv_block, nq, nkv,
                            nsplit, gps, row_first, cap > 0.f ? scale / cap : scale * LOG2E, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E,
+                           pool ? (const __nv_bfloat16*)pool->k : nullptr, pool ? (const __nv_bfloat16*)pool->v : nullptr, pool ? pool->size : 0,
                            status);
   };
-  return hd == 64 ? go(attn_decode_keys_kernel<64>) : go(attn_decode_keys_kernel<128>);
+  if (pool) return hd == 64 ? go(attn_decode_keys_kernel<64, true>) : go(attn_decode_keys_kernel<128, true>);
+  return hd == 64 ? go(attn_decode_keys_kernel<64, false>) : go(attn_decode_keys_kernel<128, false>);
 }

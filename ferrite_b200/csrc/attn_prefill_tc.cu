@@ -88,22 +88,26 @@ constexpr int ft_v_stages(int hd, bool bnd) { return ft_pair(hd, bnd) ? (hd == 1
 // DUAL: two softmax maps per head over shared values (a key row holds both maps' keys, a query has zeros in the other's columns). A CTA takes
 // both maps of 64 query rows, map 0 in lanes 0..63 and map 1 in lanes 64..127, and ends with the difference of the two, its norm over vdim,
 // the scale and the output gate: the maps' own rows never leave the SM.
-template <int HD, bool PX, bool BND, bool DUAL>
+//
+// HD, HV: columns of a head's keys and values. POOL: the means of the blocks before a row's window are keys as well; the CTA's first tiles are
+// those of the means that its last row sees, out of a buffer where a segment's means lie side by side from row pool_start[seg] on.
+template <int HD, int HV, bool PX, bool BND, bool DUAL, bool POOL>
 __global__ void __launch_bounds__(FT_THREADS, ft_pair(HD, BND) ? 2 : 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                       const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
+                       const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmKp,
+                       const __grid_constant__ CUtensorMap tmVp, const int* __restrict__ pool_start, int pool, __nv_bfloat16* __restrict__ out,
                        const __nv_bfloat16* __restrict__ proj, long proj_stride, const int* __restrict__ seg_slot,
                        const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows,
                        const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
                        int kv_block, int nq, int nkv, int gated, float scale_log2, const float* __restrict__ sink, int window, int chunk,
                        float cap_log2, long ldo, int out_f32, const HeadMix mix, int head_groups, int* status) {
-  constexpr int NCH = HD / 64;                     // 64-element (128-byte) chunks of the head dim
+  constexpr int NCH = HD / 64, VCH = HV / 64;      // 64-element (128-byte) chunks of the head dims
   constexpr int Q_CH = FT_BQ * 128;                // bytes of one Q chunk box (128 rows x 128 B)
   constexpr int KV_CH = FT_BKV * 128;              // bytes of one K / V chunk box (64 rows x 128 B)
-  constexpr int Q_BYTES = NCH * Q_CH, KV_BYTES = NCH * KV_CH;
+  constexpr int Q_BYTES = NCH * Q_CH, K_BYTES = NCH * KV_CH, V_BYTES = VCH * KV_CH;
   constexpr bool PAIR = ft_pair(HD, BND);
   // TMEM columns: O | S0 S1 | P0 P1 | remainders; PAIR: O | S0 S1, P and remainder in the place of their S
-  constexpr uint32_t COL_O = 0, COL_S = HD, COL_P = PAIR ? COL_S : HD + 2 * FT_BKV;
+  constexpr uint32_t COL_O = 0, COL_S = HV, COL_P = PAIR ? COL_S : HV + 2 * FT_BKV;
   constexpr uint32_t P_STEP = PAIR ? FT_BKV : FT_BKV / 2, REM = PAIR ? FT_BKV / 2 : FT_BKV;   // between P buffers; from P to its remainder
   constexpr uint32_t TMEM_COLS = PAIR ? 256 : 512;
   // K runs three tiles ahead at head_dim 256 (S(j+1) is issued a whole tile before PV(j), so with two K buffers a K
@@ -113,10 +117,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   // 1024-byte aligned base: [Q][K x KS][V x VS][row maxima 2 KB][barriers][flags]
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* sQ = smem_raw;
-  unsigned char* sK = sQ + Q_BYTES;                         // [KS][KV_BYTES]
-  unsigned char* sV = sK + KS * KV_BYTES;                   // [VS][KV_BYTES]
-  float (*mx_s)[2][FT_BQ] = reinterpret_cast<float (*)[2][FT_BQ]>(sV + VS * KV_BYTES);   // [2][2][128] by tile parity
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + VS * KV_BYTES + 2 * 2 * FT_BQ * 4);
+  unsigned char* sK = sQ + Q_BYTES;                         // [KS][K_BYTES]
+  unsigned char* sV = sK + KS * K_BYTES;                    // [VS][V_BYTES]
+  float (*mx_s)[2][FT_BQ] = reinterpret_cast<float (*)[2][FT_BQ]>(sV + VS * V_BYTES);   // [2][2][128] by tile parity
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + VS * V_BYTES + 2 * 2 * FT_BQ * 4);
   uint64_t* q_full = bars;
   uint64_t* s_full = bars + 2;                              // [2]
   uint64_t* s_empty = bars + 4;                             // [2]
@@ -149,7 +153,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int kvh = (DUAL ? 2 * qh : qh) / (nq / nkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile0 = BND ? first_key(pos0 + q0, window, chunk) / FT_BKV : 0;   // first key tile that a row of the CTA sees
-  const int nt = (pos0 + min(q0 + QR, n) + FT_BKV - 1) / FT_BKV - tile0;   // key tiles up to the one the last query row ends in
+  const int last_pos = pos0 + min(q0 + QR, n) - 1;
+  const int np = POOL ? (first_key(last_pos, window, 0) / pool + FT_BKV - 1) / FT_BKV : 0;   // tiles of means
+  const int nt = np + last_pos / FT_BKV + 1 - tile0;        // ... and key tiles up to the one the last query row ends in
   volatile int* abort_flag = abort_p;
 
   if (threadIdx.x == 0) {
@@ -190,7 +196,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       int k_armed = 0, v_armed = 0;                           // tiles whose K / V loads were issued
       bool ok = true;
       auto tile_row = [&](int j) -> int {
-        const int t0 = (tile0 + j) * FT_BKV;
+        if (POOL && j < np) return pool_start[seg] + j * FT_BKV;
+        const int t0 = (tile0 + j - np) * FT_BKV;
         const int blk = bt[t0 / kv_block];
         return blk < 0 ? -1 : blk * kv_block + t0 % kv_block;
       };
@@ -198,9 +205,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const int st = j % KS, krow = tile_row(j);
         if (krow < 0) { set_status(status, ST_BOUNDS); return false; }
         if (j >= KS && !mbar_wait_or_flag(&k_empty[st], ((j / KS) - 1) & 1, abort_flag)) { set_status(status, ST_MBAR_TIMEOUT); return false; }
-        mbar_expect_tx(&k_full[st], KV_BYTES);
+        mbar_expect_tx(&k_full[st], K_BYTES);
+        const CUtensorMap* tm = POOL && j < np ? &tmKp : &tmK;
 #pragma unroll
-        for (int c = 0; c < NCH; ++c) tma_load_2d(sK + st * KV_BYTES + c * KV_CH, &tmK, &k_full[st], kvh * HD + c * 64, krow);
+        for (int c = 0; c < NCH; ++c) tma_load_2d(sK + st * K_BYTES + c * KV_CH, tm, &k_full[st], kvh * HD + c * 64, krow);
         k_armed = j + 1;
         return true;
       };
@@ -208,9 +216,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const int st = j % VS, krow = tile_row(j);
         if (krow < 0) { set_status(status, ST_BOUNDS); return false; }
         if (j >= VS && !mbar_wait_or_flag(&v_empty[st], ((j / VS) - 1) & 1, abort_flag)) { set_status(status, ST_MBAR_TIMEOUT); return false; }
-        mbar_expect_tx(&v_full[st], KV_BYTES);
+        mbar_expect_tx(&v_full[st], V_BYTES);
+        const CUtensorMap* tm = POOL && j < np ? &tmVp : &tmV;
 #pragma unroll
-        for (int c = 0; c < NCH; ++c) tma_load_2d(sV + st * KV_BYTES + c * KV_CH, &tmV, &v_full[st], kvh * HD + c * 64, krow);
+        for (int c = 0; c < VCH; ++c) tma_load_2d(sV + st * V_BYTES + c * KV_CH, tm, &v_full[st], kvh * HV + c * 64, krow);
         v_armed = j + 1;
         return true;
       };
@@ -231,7 +240,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     if (lane == 0) {
       // ---- MMA issuer ---------------------------------------------------------------------------------------
       constexpr uint32_t idesc_s = umma_idesc(1, 1, FT_BQ, FT_BKV);
-      constexpr uint32_t idesc_pv = umma_idesc(1, 1, FT_BQ, HD) | (1u << 16);     // B read MN-major
+      constexpr uint32_t idesc_pv = umma_idesc(1, 1, FT_BQ, HV) | (1u << 16);     // B read MN-major
       const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV);
       bool ok = mbar_wait_or_flag(q_full, 0, abort_flag);
       auto issue_s = [&](int j) -> bool {
@@ -243,7 +252,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int kk = 0; kk < HD / 16; ++kk) {
           const uint32_t off = (uint32_t)(kk & 3) * 32u;
           tc_mma_f16(tmem + COL_S + s * FT_BKV, umma_desc_k128(aQ + (kk >> 2) * Q_CH + off),
-                     umma_desc_k128(aK + st * KV_BYTES + (kk >> 2) * KV_CH + off), idesc_s, kk > 0 ? 1u : 0u);
+                     umma_desc_k128(aK + st * K_BYTES + (kk >> 2) * KV_CH + off), idesc_s, kk > 0 ? 1u : 0u);
         }
         tc_commit(&s_full[s]);
         tc_commit(&k_empty[st]);
@@ -259,12 +268,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
         for (int kk = 0; kk < FT_BKV / 16; ++kk)
           tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + s * P_STEP + kk * 8,
-                        umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
+                        umma_desc_mn128(aV + st * V_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
         if (PX) {
 #pragma unroll
           for (int kk = 0; kk < FT_BKV / 16; ++kk)
             tc_mma_f16_ts(tmem + COL_O, tmem + COL_P + REM + s * P_STEP + kk * 8,
-                          umma_desc_mn128(aV + st * KV_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, 1u);
+                          umma_desc_mn128(aV + st * V_BYTES + kk * 16 * 128, KV_CH, 1024), idesc_pv, 1u);
         }
         tc_commit(&v_empty[st]);
         tc_commit(&p_empty[s]);
@@ -285,7 +294,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int klo = BND ? first_key(qpos, window, chunk) : 0;
     const int klo_last = BND ? first_key(pos0 + q0 + QR - 1, window, chunk) : 0;
     constexpr int HC = FT_BKV / 2;                          // keys per thread and tile
-    constexpr int OC = HD / 2;                              // O columns per thread (rescale, epilogue)
+    constexpr int OC = HV / 2;                              // O columns per thread (rescale, epilogue)
     float m_ref = -INFINITY, l = 0.f;
     bool broke = false;
     bool late_fail = false;                                 // a wait after the barrier ran out: reported at the next one
@@ -304,8 +313,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           __syncwarp();
           if (lane == 0) mbar_arrive(&s_empty[s]);
         }
-        const int t0 = (tile0 + j) * FT_BKV + half * HC;
-        const bool need_mask = t0 + HC - 1 > pos0 + q0 || (BND && t0 < klo_last);
+        const bool means = POOL && j < np;                    // keys of the tile are means: number t0 + c
+        const int t0 = (means ? j : tile0 + j - np) * FT_BKV + half * HC;
+        const bool need_mask = means || t0 + HC - 1 > pos0 + q0 || (BND && t0 < klo_last);
         const bool capped = BND && cap_log2 > 0.f;
         if (capped) {
           float am = 0.f;
@@ -338,7 +348,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
             for (int c = 0; c < HC; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) * scale_log2);
           }
-          if (need_mask) {
+          if (means) {
+#pragma unroll
+            for (int c = 0; c < HC; ++c)
+              if ((t0 + c + 1) * pool > klo) sr[c] = __float_as_uint(-INFINITY);
+          } else if (need_mask) {
 #pragma unroll
             for (int c = 0; c < HC; ++c)
               if (t0 + c > qpos || t0 + c < klo) sr[c] = __float_as_uint(-INFINITY);
@@ -497,8 +511,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       } else {
         const bool valid = q0 + row < n;
         const size_t grow = (size_t)(row0 + q0 + row);
-        __nv_bfloat16* dst = out + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
-        float* dst32 = reinterpret_cast<float*>(out) + grow * (size_t)ldo + (size_t)qh * HD + half * OC;
+        __nv_bfloat16* dst = out + grow * (size_t)ldo + (size_t)qh * HV + half * OC;
+        float* dst32 = reinterpret_cast<float*>(out) + grow * (size_t)ldo + (size_t)qh * HV + half * OC;
         const __nv_bfloat16* gate = proj + grow * proj_stride + (size_t)qh * 2 * HD + HD + half * OC;
 #pragma unroll 1
         for (int c0 = 0; c0 < OC; c0 += 32) {
@@ -546,25 +560,35 @@ using namespace fb;
 
 // q: [q_rows][nq*hd] bf16 (post norm / RoPE); caches: [cache_rows = blocks*kv_block] rows of nkv*hd bf16, kv_stride elements
 // apart (0: dense); scale: of the scores (0: 1 / sqrt(hd)); exact_p: softmax weights as value + remainder; sink: a number per q head
-// that joins the softmax denominator, or null; kb: window, chunk and softcap, or null (only with exact_p and a bounded call: fp32 rows,
+// that joins the softmax denominator, or null; hdv: columns of a head's values (0: hd; 128 beside 192 of the keys); pool: gathered means of the
+// blocks before the window, or null; kb: window, chunk and softcap, or null (only with exact_p and a bounded call: fp32 rows,
 // out_f32); mix: what follows two maps per head (nq counts both maps' queries, out has nq / 2 heads), or null; ldo: elements between rows of out (0: dense); same outputs as fb_attn_prefill. Returns -20 when the shape is outside what this kernel takes (the caller uses fb_attn_prefill).
 extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache, const void* v_cache, const void* proj,
                                   long proj_stride, const int* seg_slot, const int* seg_row0, const int* seg_nrows,
                                   const int* seg_pos0, const int* block_table, int max_blocks, int kv_block, int nseg,
-                                  int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int gated,
-                                  float scale, int exact_p, long kv_stride, const float* sink, const KeyBounds* kb, long ldo,
-                                  int out_f32, const HeadMix* mix, int* status, cudaStream_t s) {
+                                  int max_rows, long q_rows, long cache_rows, int nq, int nkv, int hd, int hdv, int gated,
+                                  float scale, int exact_p, long kv_stride, const float* sink, const KeyBounds* kb, const PoolKeys* pool,
+                                  long ldo, int out_f32, const HeadMix* mix, int* status, cudaStream_t s) {
   if (nseg <= 0 || max_rows <= 0) return 0;
   if (nq % nkv) return -1;
-  if ((hd != 64 && hd != 128 && hd != 256) || kv_block % FT_BKV) return -20;
-  if (kv_stride == 0) kv_stride = (long)nkv * hd;
+  if (hdv == 0) hdv = hd;
+  const bool wide = hd == 192 && hdv == 128;
+  if ((!wide && ((hd != 64 && hd != 128 && hd != 256) || hdv != hd)) || kv_block % FT_BKV) return -20;
+  if (kv_stride == 0) kv_stride = wide ? -1 : (long)nkv * hd;          // keys and values of different widths lie in one buffer
+  if (kv_stride < 0 || (wide && (mix || pool || gated || out_f32 || sink || !exact_p))) return -20;
+  if (pool && (pool->size < 1 || !pool->start || pool->rows < 0 || !kb || !kb->window || mix || out_f32)) return -1;
   if (kv_stride % 8) return -20;
   const int heads = mix ? nq / 2 : nq, q_rows_cta = mix ? FT_BQ / 2 : FT_BQ;
-  CUtensorMap tmQ, tmK, tmV;
+  CUtensorMap tmQ, tmK, tmV, tmKp, tmVp;
   int rc;
   if ((rc = make_tmap_bf16_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)nq * hd, (uint64_t)nq * hd, q_rows_cta))) return rc;
   if ((rc = make_tmap_bf16_2d(&tmK, k_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
-  if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hd, (uint64_t)kv_stride, FT_BKV))) return rc;
+  if ((rc = make_tmap_bf16_2d(&tmV, v_cache, (uint64_t)cache_rows, (uint64_t)nkv * hdv, (uint64_t)kv_stride, FT_BKV))) return rc;
+  tmKp = tmK; tmVp = tmV;
+  if (pool && pool->rows > 0) {
+    if ((rc = make_tmap_bf16_2d(&tmKp, pool->k, (uint64_t)pool->rows, (uint64_t)nkv * hd, (uint64_t)nkv * hd, FT_BKV))) return rc;
+    if ((rc = make_tmap_bf16_2d(&tmVp, pool->v, (uint64_t)pool->rows, (uint64_t)nkv * hd, (uint64_t)nkv * hd, FT_BKV))) return rc;
+  }
   // up to four waves of CTAs are one group; more go in groups of about two waves, whole sets of query heads that share keys
   const int q_tiles = (max_rows + q_rows_cta - 1) / q_rows_cta, share = heads / nkv > 0 ? heads / nkv : 1;
   const int slots = 148 * (ft_pair(hd, kb || out_f32 || mix) ? 2 : 1);
@@ -575,29 +599,39 @@ extern "C" int fb_attn_prefill_tc(void* out, const void* q, const void* k_cache,
   if ((kb || out_f32 || mix) && (!exact_p || gated)) return -20;
   if (mix && (nq % 2 || (nq / nkv) % 2 || !mix->lam || mix->vdim < 1 || mix->vdim > hd || sink || out_f32)) return -1;
   if (kb && (kb->window < 0 || kb->chunk < 0 || (kb->window && kb->chunk) || kb->cap < 0.f)) return -1;
-  if (ldo == 0) ldo = (long)heads * hd;
+  if (ldo == 0) ldo = (long)heads * hdv;
   if (ldo % 8) return -20;
   constexpr float LOG2E = 1.4426950408889634f;
   const float cap = kb ? kb->cap : 0.f, raw_scale = scale != 0.f ? scale : 1.f / sqrtf((float)hd);
   const float scale_log2 = cap > 0.f ? raw_scale / cap : raw_scale * LOG2E;
-#define FB_FT(HDV, PXV, BNDV, DUALV)                                                                                              \
+#define FB_FT(HDK, HVV, PXV, BNDV, DUALV, POOLV)                                                                   \
   {                                                                                                                \
-    const size_t smem = (size_t)(FT_BQ + (ft_k_stages(HDV, BNDV) + ft_v_stages(HDV, BNDV)) * FT_BKV) * HDV * 2 + 2048 + 512;                                             \
-    auto kern = attn_prefill_tc_kernel<HDV, PXV, BNDV, DUALV>;                                                                     \
+    const size_t smem = (size_t)(FT_BQ + ft_k_stages(HDK, BNDV) * FT_BKV) * HDK * 2 +                              \
+                        (size_t)ft_v_stages(HDK, BNDV) * FT_BKV * HVV * 2 + 2048 + 512;                            \
+    auto kern = attn_prefill_tc_kernel<HDK, HVV, PXV, BNDV, DUALV, POOLV>;                                         \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
     if (e != cudaSuccess) return (int)e;                                                                           \
-    launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
+    launch_pdl(kern, grid, dim3(FT_THREADS), smem, s, tmQ, tmK, tmV, tmKp, tmVp, pool ? pool->start : nullptr, pool ? pool->size : 1, (__nv_bfloat16*)out, (const __nv_bfloat16*)proj, \
                proj_stride, seg_slot, seg_row0, seg_nrows, seg_pos0, block_table, max_blocks, kv_block, nq, nkv,   \
                gated, scale_log2, sink, kb ? kb->window : 0, kb ? kb->chunk : 0, cap * LOG2E, ldo, out_f32, mix ? *mix : no_mix, head_groups, status);                                                                   \
   }
-  if (mix) {
-    if (hd == 256) FB_FT(256, true, true, true) else if (hd == 128) FB_FT(128, true, true, true) else FB_FT(64, true, true, true)
+  if (wide) {
+    FB_FT(192, 128, true, true, false, false)
+  } else if (pool) {
+    if (hd == 256) FB_FT(256, 256, true, true, false, true) else if (hd == 128) FB_FT(128, 128, true, true, false, true)
+    else FB_FT(64, 64, true, true, false, true)
+  } else if (mix) {
+    if (hd == 256) FB_FT(256, 256, true, true, true, false) else if (hd == 128) FB_FT(128, 128, true, true, true, false)
+    else FB_FT(64, 64, true, true, true, false)
   } else if (kb || out_f32) {
-    if (hd == 256) FB_FT(256, true, true, false) else if (hd == 128) FB_FT(128, true, true, false) else FB_FT(64, true, true, false)
+    if (hd == 256) FB_FT(256, 256, true, true, false, false) else if (hd == 128) FB_FT(128, 128, true, true, false, false)
+    else FB_FT(64, 64, true, true, false, false)
   } else if (exact_p) {
-    if (hd == 256) FB_FT(256, true, false, false) else if (hd == 128) FB_FT(128, true, false, false) else FB_FT(64, true, false, false)
+    if (hd == 256) FB_FT(256, 256, true, false, false, false) else if (hd == 128) FB_FT(128, 128, true, false, false, false)
+    else FB_FT(64, 64, true, false, false, false)
   } else {
-    if (hd == 256) FB_FT(256, false, false, false) else if (hd == 128) FB_FT(128, false, false, false) else FB_FT(64, false, false, false)
+    if (hd == 256) FB_FT(256, 256, false, false, false, false) else if (hd == 128) FB_FT(128, 128, false, false, false, false)
+    else FB_FT(64, 64, false, false, false, false)
   }
 #undef FB_FT
   return (int)cudaGetLastError();

@@ -281,13 +281,21 @@ int64_t attn_prefill_tc(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Te
                         Tensor seg_nrows, Tensor seg_pos0, Tensor block_table, int64_t kv_block, int64_t max_rows,
                         int64_t nq, int64_t nkv, int64_t hd, bool gated, c10::optional<Tensor> status, double scale,
                         bool exact_p, c10::optional<Tensor> sink, int64_t window, int64_t chunk, double softcap,
-                        c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t vdim, double eps) {
-  // caches: [pages, kv_block, nkv, hd] with dense rows; the rows may lie further apart (k and v side by side in one buffer)
-  const long kv_stride = (long)k_cache.stride(1);
-  TORCH_CHECK(q.is_contiguous() && v_cache.sizes() == k_cache.sizes() && v_cache.strides() == k_cache.strides() &&
+                        c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t vdim, double eps,
+                        c10::optional<Tensor> k_mean, c10::optional<Tensor> v_mean, c10::optional<Tensor> mean_start, int64_t pool) {
+  // caches: [pages, kv_block, nkv, hd] with dense rows; the rows may lie further apart (k and v side by side in one buffer, of their own widths)
+  const long kv_stride = (long)k_cache.stride(1), hdv = (long)v_cache.size(3);
+  TORCH_CHECK(q.is_contiguous() && v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == k_cache.size(1) && v_cache.size(2) == k_cache.size(2) &&
+              v_cache.stride(0) == k_cache.stride(0) && v_cache.stride(1) == kv_stride && v_cache.stride(3) == 1 && v_cache.stride(2) == hdv &&
               k_cache.stride(3) == 1 && k_cache.stride(2) == hd && k_cache.stride(0) == kv_block * kv_stride,
               "attn_prefill_tc: layouts");
-  TORCH_CHECK(out.dim() == 2 || (out.stride(2) == 1 && out.stride(1) == hd), "attn_prefill_tc: out rows");
+  TORCH_CHECK(out.dim() == 2 || (out.stride(2) == 1 && out.stride(1) == hdv), "attn_prefill_tc: out rows");
+  // means of the blocks before the window: rows [n, nkv, hd] of every segment from row mean_start[segment] on
+  TORCH_CHECK(pool == 0 || (k_mean && v_mean && mean_start && k_mean->is_contiguous() && v_mean->is_contiguous() && k_mean->sizes() == v_mean->sizes() &&
+              k_mean->numel() == k_mean->size(0) * nkv * hd && k_mean->scalar_type() == q.scalar_type() && v_mean->scalar_type() == q.scalar_type() &&
+              mean_start->numel() >= seg_slot.numel() && mean_start->scalar_type() == torch::kInt32), "attn_prefill_tc: means");
+  const PoolKeys pk{pool ? k_mean->data_ptr() : nullptr, pool ? v_mean->data_ptr() : nullptr, (int)pool,
+                    pool ? mean_start->data_ptr<int>() : nullptr, pool ? (long)k_mean->size(0) : 0};
   const KeyBounds kb{(int)window, (int)chunk, (float)softcap};
   TORCH_CHECK(!lam || (out.dim() == 3 && out.size(1) * 2 == nq && lam->scalar_type() == torch::kFloat32 &&
               (!gate || (gate->scalar_type() == torch::kFloat32 && gate->stride(1) == 1 && gate->size(0) == out.size(0) &&
@@ -298,9 +306,9 @@ int64_t attn_prefill_tc(Tensor out, Tensor q, Tensor k_cache, Tensor v_cache, Te
                               (long)proj.stride(0), seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(),
                               seg_nrows.data_ptr<int>(), seg_pos0.data_ptr<int>(), block_table.data_ptr<int>(),
                               (int)block_table.size(1), (int)kv_block, (int)seg_slot.numel(), (int)max_rows,
-                              (long)q.size(0), (long)(k_cache.size(0) * k_cache.size(1)), (int)nq, (int)nkv, (int)hd,
+                              (long)q.size(0), (long)(k_cache.size(0) * k_cache.size(1)), (int)nq, (int)nkv, (int)hd, (int)hdv,
                               gated ? 1 : 0, (float)scale, exact_p ? 1 : 0, kv_stride, (const float*)cptr(sink),
-                              window || chunk || softcap != 0.0 ? &kb : nullptr, (long)out.stride(0),
+                              window || chunk || softcap != 0.0 ? &kb : nullptr, pool ? &pk : nullptr, (long)out.stride(0),
                               out.scalar_type() == torch::kFloat32 ? 1 : 0, lam ? &mix : nullptr, (int*)mptr(status),
                               cur_stream());
   if (rc == -20) return rc;                     // shape outside this kernel: the caller takes the mma.sync kernel
@@ -410,6 +418,7 @@ void kv_move_rows(Tensor k, c10::optional<Tensor> v, c10::optional<Tensor> sc, T
 }  // namespace
 
 void register_ext(pybind11::module_& m);
+void register_listed(pybind11::module_& m);
 void register_host(pybind11::module_& m);
 void register_oracle(pybind11::module_& m);
 void register_gguf_host(pybind11::module_& m);
@@ -433,7 +442,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("kv_block"), py::arg("max_rows"), py::arg("nq"), py::arg("nkv"), py::arg("hd"), py::arg("gated"), py::arg("status"),
         py::arg("scale") = 0.0, py::arg("exact_p") = false, py::arg("sink") = py::none(), py::arg("window") = 0,
         py::arg("chunk") = 0, py::arg("softcap") = 0.0, py::arg("lam") = py::none(), py::arg("gate") = py::none(), py::arg("mix_scale") = 1.0,
-        py::arg("vdim") = 0, py::arg("eps") = 0.0);
+        py::arg("vdim") = 0, py::arg("eps") = 0.0, py::arg("k_mean") = py::none(), py::arg("v_mean") = py::none(),
+        py::arg("mean_start") = py::none(), py::arg("pool") = 0);
   m.def("attn_decode_mma", &attn_decode_mma);
   m.def("gdn_conv", &gdn_conv);
   m.def("gdn_rec", &gdn_rec);
@@ -453,6 +463,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("chain_accept", &chain_accept);
   m.def("kv_move_rows", &kv_move_rows);
   register_ext(m);
+  register_listed(m);
   register_host(m);
   register_oracle(m);
   register_gguf_host(m);

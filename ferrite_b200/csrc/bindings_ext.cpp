@@ -360,13 +360,14 @@ int is_f32(const Tensor& t) {
 
 void ep_moe(const EpHandle& c, Tensor out, Tensor x, Tensor ids, Tensor wts, Tensor w_gu, Tensor w_down,
             c10::optional<Tensor> shared, c10::optional<Tensor> shared_gate, c10::optional<Tensor> res, Tensor act,
-            Tensor plan) {
+            Tensor plan, double limit, bool add) {
   int rows = (int)x.size(0), top_k = (int)ids.size(1), inter = (int)w_down.size(2);
   TORCH_CHECK(plan.numel() >= (int64_t)rows * top_k + 3 * c.n_experts + 8, "ep_moe: plan scratch too small");
   TORCH_CHECK(act.numel() >= c.cap_rows * inter, "ep_moe: activation scratch too small");
-  check(fb_ep_moe(out.data_ptr(), is_f32(out), x.data_ptr(), ids.data_ptr<int>(), wts.data_ptr<float>(), w_gu.data_ptr(),
+  TORCH_CHECK(!shared_gate || (is_f32(*shared_gate) && shared_gate->dim() == 1 && shared_gate->size(0) == rows), "ep_moe: gates of the shared expert");
+  check(fb_ep_moe(out.data_ptr(), is_f32(out) ? (add ? 1 : 2) : 0, (float)limit, x.data_ptr(), ids.data_ptr<int>(), wts.data_ptr<float>(), w_gu.data_ptr(),
                   w_down.data_ptr(), cptr(shared), shared_gate.has_value() ? shared_gate->data_ptr<float>() : nullptr,
-                  cptr(res), act.data_ptr(), plan.data_ptr<int>(), rows, top_k, c.n_experts, c.hidden, inter, c.cap_rows,
+                  shared_gate.has_value() ? (long)shared_gate->stride(0) : 0, cptr(res), act.data_ptr(), plan.data_ptr<int>(), rows, top_k, c.n_experts, c.hidden, inter, c.cap_rows,
                   c.peers.data(), c.rank, c.world, (uint32_t*)c.ctr.data_ptr(), c.status.data_ptr<int>(), c.spin_limit,
                   c.sm, cur_stream()), "ep_moe");
 }
@@ -375,7 +376,7 @@ void gemm_grouped(Tensor Y, Tensor X, Tensor W, Tensor tile_start, Tensor row_ba
   int experts = (int)W.size(0);
   int N = (int)(mode == 1 ? W.size(1) / 2 : W.size(1));
   check(fb_gemm_grouped(Y.data_ptr(), X.data_ptr(), W.data_ptr(), tile_start.data_ptr<int>(), row_base.data_ptr<int>(),
-                        experts, (int)X.size(0), N, (int)X.size(1), (long)X.stride(0), (long)Y.stride(0), (int)mode,
+                        experts, (int)X.size(0), N, (int)X.size(1), (long)X.stride(0), (long)Y.stride(0), (int)mode, 0.f,
                         status.data_ptr<int>(), 0, cur_stream()), "gemm_grouped");
 }
 
@@ -618,23 +619,26 @@ void gqa_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::option
                     (int)v_off, norm ? 1 : 0, (float)eps, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_prep");
 }
 
-// sizes: heads, maps, dim, vdim, rotated columns, first column of the values
-void gqa_row_prep(Tensor q, Tensor k_cache, Tensor v_cache, Tensor proj, c10::optional<Tensor> q_norm, c10::optional<Tensor> k_norm, Tensor inv_freq,
+// sizes: heads, maps, dim, vdim, rotated columns, first column of the values, 1 for pairs half the rotated columns apart. Without caches only
+// queries are made.
+void gqa_row_prep(Tensor q, c10::optional<Tensor> k_cache, c10::optional<Tensor> v_cache, Tensor proj, c10::optional<Tensor> q_norm, c10::optional<Tensor> k_norm, Tensor inv_freq,
                   Tensor row_slot, Tensor row_pos, Tensor block_table, int64_t kv_block, std::vector<int64_t> sizes, double eps, Tensor status) {
-  TORCH_CHECK(sizes.size() == 6, "gqa_row_prep: six sizes");
+  TORCH_CHECK(sizes.size() == 7, "gqa_row_prep: seven sizes");
   const int64_t heads = sizes[0], maps = sizes[1], dim = sizes[2], vdim = sizes[3], rot = sizes[4], v_off = sizes[5];
-  const int64_t kvh = k_cache.size(2), hp = q.size(2);
-  TORCH_CHECK(q.is_contiguous() && q.size(1) == heads * maps && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.sizes() == v_cache.sizes() &&
-              k_cache.size(3) == hp && k_cache.size(1) == kv_block && is_f32(proj) && proj.stride(1) == 1 && proj.size(0) == q.size(0) &&
-              q.scalar_type() == k_cache.scalar_type() && q.scalar_type() == v_cache.scalar_type() && v_off >= (heads + kvh) * maps * dim &&
-              proj.size(1) >= v_off + kvh * vdim && inv_freq.scalar_type() == torch::kFloat64 && inv_freq.numel() * 2 >= rot &&
+  const int64_t kvh = k_cache ? k_cache->size(2) : 0, hp = q.size(2);
+  TORCH_CHECK(k_cache.has_value() == v_cache.has_value() && (!k_cache || (k_cache->is_contiguous() && v_cache->is_contiguous() &&
+              k_cache->sizes() == v_cache->sizes() && k_cache->size(3) == hp && k_cache->size(1) == kv_block &&
+              q.scalar_type() == k_cache->scalar_type() && q.scalar_type() == v_cache->scalar_type() && v_off >= (heads + kvh) * maps * dim &&
+              proj.size(1) >= v_off + kvh * vdim)), "gqa_row_prep: caches");
+  TORCH_CHECK(q.is_contiguous() && q.size(1) == heads * maps && is_f32(proj) && proj.stride(1) == 1 && proj.size(0) == q.size(0) &&
+              proj.size(1) >= heads * maps * dim && inv_freq.scalar_type() == torch::kFloat64 && inv_freq.numel() * 2 >= rot &&
               (!q_norm || (is_f32(*q_norm) && q_norm->numel() == heads * maps * dim)) &&
               (!k_norm || (is_f32(*k_norm) && k_norm->numel() == kvh * maps * dim)), "gqa_row_prep: layouts");
-  check(fb_gqa_row_prep(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), proj.data_ptr<float>(), (long)proj.stride(0),
+  check(fb_gqa_row_prep(q.data_ptr(), optr(k_cache), optr(v_cache), proj.data_ptr<float>(), (long)proj.stride(0),
                         (const float*)cptr(q_norm), (const float*)cptr(k_norm), inv_freq.data_ptr<double>(), row_slot.data_ptr<int>(),
                         row_pos.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block, (int)q.size(0), (int)heads,
-                        (int)kvh, (int)maps, (int)dim, (int)vdim, (int)hp, (int)rot, (int)v_off, (float)eps, is_f32(q), status.data_ptr<int>(),
-                        cur_stream()), "gqa_row_prep");
+                        (int)kvh, (int)maps, (int)dim, (int)vdim, (int)hp, (int)rot, (int)v_off, (int)sizes[6], (float)eps, is_f32(q),
+                        status.data_ptr<int>(), cur_stream()), "gqa_row_prep");
 }
 
 // Two maps per head, output gates: out [rows, heads, hd] from in [rows, heads * maps, hd]
@@ -648,23 +652,28 @@ void head_mix(Tensor out, Tensor in, c10::optional<Tensor> lam, c10::optional<Te
                     is_f32(out), cur_stream()), "head_mix");
 }
 
-// Rows of every (token, pick)'s expert: x [rows, hidden], w_gu [experts, 2 inter, hidden], w_down [experts, hidden, inter]
-void expert_rows(Tensor yp, Tensor act, Tensor x, Tensor w_gu, Tensor w_down, Tensor ids) {
+// Rows of every (token, pick)'s expert: x [rows, hidden], w_gu [experts, 2 inter, hidden], w_down [experts, hidden, inter]; limit: of clamped
+// gated units (0: swiglu); shared_gu [2 inter', hidden], shared_down [hidden, inter']: the expert one past the last
+void expert_rows(Tensor yp, Tensor act, Tensor x, Tensor w_gu, Tensor w_down, Tensor ids, double limit, c10::optional<Tensor> shared_gu,
+                 c10::optional<Tensor> shared_down, double shared_limit) {
   const int pairs = (int)ids.numel(), top = (int)ids.size(1), hidden = (int)x.size(1), inter = (int)w_down.size(2), ne = (int)w_down.size(0);
   TORCH_CHECK(x.is_contiguous() && w_gu.is_contiguous() && w_down.is_contiguous() && ids.is_contiguous() && yp.is_contiguous() &&
-              act.is_contiguous() && is_f32(yp) && yp.size(0) == pairs && yp.size(1) == hidden && act.size(0) == pairs && act.size(1) == inter &&
+              act.is_contiguous() && is_f32(yp) && yp.size(0) == pairs && yp.size(1) == hidden && act.size(0) == pairs && act.size(1) >= inter &&
               w_gu.size(0) == ne && w_gu.size(1) == 2 * inter && w_gu.size(2) == hidden && w_down.size(1) == hidden &&
               act.scalar_type() == x.scalar_type() && w_gu.scalar_type() == x.scalar_type() && w_down.scalar_type() == x.scalar_type() &&
               ids.size(0) == x.size(0), "expert_rows: layouts");
+  const int si = shared_down ? (int)shared_down->size(1) : 0, lda = (int)act.size(1);
+  TORCH_CHECK(shared_gu.has_value() == shared_down.has_value() && (!shared_gu || (shared_gu->is_contiguous() && shared_down->is_contiguous() &&
+              shared_gu->size(0) == 2 * si && shared_gu->size(1) == hidden && shared_down->size(0) == hidden && lda >= si &&
+              shared_gu->scalar_type() == x.scalar_type() && shared_down->scalar_type() == x.scalar_type())), "expert_rows: shared expert");
   if (is_f32(x)) {
     check(fb_expert_rows_f32(yp.data_ptr<float>(), act.data_ptr<float>(), x.data_ptr<float>(), w_gu.data_ptr<float>(), w_down.data_ptr<float>(),
-                             ids.data_ptr<int>(), pairs, top, hidden, inter, ne, cur_stream()), "expert_rows_f32");
+                             ids.data_ptr<int>(), pairs, top, hidden, inter, ne, lda, (float)limit, (const float*)cptr(shared_gu),
+                             (const float*)cptr(shared_down), si, (float)shared_limit, cur_stream()), "expert_rows_f32");
     return;
   }
-  check(fb_moe_gate_up(act.data_ptr(), x.data_ptr(), w_gu.data_ptr(), ids.data_ptr<int>(), pairs, top, hidden, inter, 0, ne, cur_stream()),
-        "moe_gate_up");
-  check(fb_moe_down(yp.data_ptr<float>(), act.data_ptr(), w_down.data_ptr(), ids.data_ptr<int>(), pairs, hidden, inter, 0, ne, cur_stream()),
-        "moe_down");
+  check(fb_expert_rows(yp.data_ptr<float>(), act.data_ptr(), x.data_ptr(), w_gu.data_ptr(), w_down.data_ptr(), ids.data_ptr<int>(), pairs, top, hidden,
+                       inter, ne, lda, (float)limit, cptr(shared_gu), cptr(shared_down), si, (float)shared_limit, cur_stream()), "expert_rows");
 }
 
 // Few rows of grouped-query attention: q [rows, queries, hd], out [rows, heads, hd] (rows may lie apart; queries = maps * heads); with lam or
@@ -673,7 +682,8 @@ void expert_rows(Tensor yp, Tensor act, Tensor x, Tensor w_gu, Tensor w_down, Te
 void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cache, Tensor v_cache, c10::optional<Tensor> sink,
               Tensor seg_slot, Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, Tensor row_slot, Tensor row_kvlen, Tensor block_table,
               int64_t kv_block, int64_t row_first, int64_t nsplit, double scale, bool cuda_cores, Tensor status, int64_t window, int64_t chunk,
-              double softcap, c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t maps, int64_t vdim, double eps) {
+              double softcap, c10::optional<Tensor> lam, c10::optional<Tensor> gate, double mix_scale, int64_t maps, int64_t vdim, double eps,
+              c10::optional<Tensor> k_mean, c10::optional<Tensor> v_mean, int64_t pool) {
   const int rows = (int)q.size(0), heads = (int)q.size(1), hd = (int)q.size(2), kvh = (int)k_cache.size(2);
   const long recs = (long)rows * heads * nsplit;
   const bool mixed = lam.has_value() || gate.has_value();
@@ -693,11 +703,18 @@ void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cach
               o_part.numel() >= recs * hd && ml_part.numel() >= recs * 2 && row_slot.numel() == rows && row_kvlen.numel() == rows &&
               (!sink || sink->numel() == heads), "gqa_attn: layouts");
   const float* sk = (const float*)cptr(sink);
+  const PoolKeys pk{cptr(k_mean), cptr(v_mean), (int)pool, nullptr, 0};
+  const PoolKeys* pkp = pool ? &pk : nullptr;
+  if (pool)
+    for (const auto& m : {k_mean, v_mean})
+      TORCH_CHECK(m && m->is_contiguous() && m->scalar_type() == q.scalar_type() && m->size(0) == k_cache.size(0) &&
+                  m->size(1) == (kv_block + pool - 1) / pool && m->size(2) == kvh && m->size(3) == hd, "gqa_attn: means");
   if (!cuda_cores) {
     const int rc = fb_attn_decode_keys(o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                                        seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), row_kvlen.data_ptr<int>(),
                                        block_table.data_ptr<int>(), (int)block_table.size(1), (int)kv_block, (int)seg_slot.numel(), (int)max_rows,
-                                       rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, (int)row_first, status.data_ptr<int>(), cur_stream());
+                                       rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, pkp, (int)row_first, status.data_ptr<int>(), cur_stream());
+    TORCH_CHECK(rc != -20 || !pool, "gqa_attn: means outside the tensor-core kernel's shapes");
     if (rc != -20) check(rc, "attn_decode_keys");
     else check(fb_attn_decode_mma(nullptr, o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                              nullptr, nullptr, 0, seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(),
@@ -711,7 +728,7 @@ void gqa_attn(Tensor out, Tensor o_part, Tensor ml_part, Tensor q, Tensor k_cach
   }
   check(fb_gqa_attn(mixed ? nullptr : out.data_ptr(), o_part.data_ptr<float>(), ml_part.data_ptr<float>(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                     sk, row_slot.data_ptr<int>(), row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
-                    (int)kv_block, rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, ldo, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_attn");
+                    (int)kv_block, rows, heads, kvh, hd, (int)nsplit, (float)scale, kbp, pkp, ldo, is_f32(q), status.data_ptr<int>(), cur_stream()), "gqa_attn");
   if (mixed) finish();
 }
 
@@ -797,10 +814,10 @@ void gated_norm_sigmoid(Tensor out, Tensor y, Tensor z, Tensor w, double eps) {
                               w.data_ptr<float>(), (int)y.size(0), heads, dv, (float)eps, is_f32(out), cur_stream()), "gated_norm_sigmoid");
 }
 
-void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, c10::optional<Tensor> bias, int64_t width, double eps) {
+void norm_rows(Tensor out, Tensor x, c10::optional<Tensor> idx, Tensor w, c10::optional<Tensor> bias, int64_t width, double eps, bool mean) {
   TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && out.size(1) == x.size(1) && w.numel() == x.size(1) && is_f32(w) &&
               (!bias || (bias->numel() == x.size(1) && is_f32(*bias))), "norm_rows: layouts");
-  check(fb_norm_rows(out.data_ptr(), x.data_ptr<float>(), (const int*)cptr(idx), w.data_ptr<float>(), (const float*)cptr(bias), (int)out.size(0), (int)width,
+  check(fb_norm_rows(out.data_ptr(), x.data_ptr<float>(), (const int*)cptr(idx), w.data_ptr<float>(), (const float*)cptr(bias), mean, (int)out.size(0), (int)width,
                      (int)x.size(1), (float)eps, is_f32(out), cur_stream()), "norm_rows");
 }
 
@@ -826,25 +843,26 @@ void relu2(Tensor y, Tensor x) {
 }
 
 void latent_attn(Tensor out, c10::optional<Tensor> o_part, c10::optional<Tensor> ml_part, Tensor q, Tensor cache, Tensor row_slot,
-                 Tensor row_kvlen, Tensor block_table, int64_t kv_block, int64_t nsplit, double scale, Tensor status) {
+                 Tensor row_kvlen, Tensor block_table, int64_t kv_block, int64_t nsplit, double scale, Tensor status, int64_t window) {
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && cache.is_contiguous() && cache.size(-1) == q.size(2) &&
               (nsplit == 1 || (o_part && ml_part)), "latent_attn: layouts");
+  TORCH_CHECK(out.size(2) <= q.size(2) && out.size(0) == q.size(0) && out.size(1) == q.size(1), "latent_attn: out");
   check(fb_latent_attn(out.data_ptr(), (float*)optr(o_part), (float*)optr(ml_part), q.data_ptr(), cache.data_ptr(),
                        row_slot.data_ptr<int>(), row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
-                       (int)kv_block, (int)q.size(0), (int)q.size(1), (int)q.size(2), (int)nsplit, (float)scale, is_f32(q),
-                       status.data_ptr<int>(), cur_stream()), "latent_attn");
+                       (int)kv_block, (int)q.size(0), (int)q.size(1), (int)q.size(2), (int)out.size(2), (int)window, (int)nsplit, (float)scale,
+                       is_f32(q), status.data_ptr<int>(), cur_stream()), "latent_attn");
 }
 
 int64_t latent_mma(Tensor out, c10::optional<Tensor> o_part, c10::optional<Tensor> ml_part, Tensor q, Tensor cache, Tensor seg_slot,
                    Tensor seg_row0, Tensor seg_nrows, int64_t max_rows, Tensor row_kvlen, Tensor block_table, int64_t kv_block,
-                   int64_t row_base, int64_t nsplit, double scale, Tensor status) {
+                   int64_t row_base, int64_t nsplit, double scale, Tensor status, int64_t window) {
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && cache.is_contiguous() && cache.size(-1) == q.size(2) &&
               !is_f32(q) && (nsplit == 1 || (o_part && ml_part)), "latent_mma: layouts");
   const int rc = fb_latent_mma(out.data_ptr(), (float*)optr(o_part), (float*)optr(ml_part), q.data_ptr(), cache.data_ptr(),
                                seg_slot.data_ptr<int>(), seg_row0.data_ptr<int>(), seg_nrows.data_ptr<int>(), (int)seg_slot.numel(),
                                (int)max_rows, row_kvlen.data_ptr<int>(), block_table.data_ptr<int>(), (int)block_table.size(1),
-                               (int)kv_block, (int)q.size(0), (int)row_base, (int)q.size(1), (int)q.size(2), (int)nsplit,
-                               (float)scale, status.data_ptr<int>(), cur_stream());
+                               (int)kv_block, (int)q.size(0), (int)row_base, (int)q.size(1), (int)q.size(2), (int)out.size(2),
+                               (int)window, (int)nsplit, (float)scale, status.data_ptr<int>(), cur_stream());
   if (rc == -20) return rc;                     // shape outside this kernel: the caller takes the CUDA-core kernel
   check(rc, "latent_mma");
   return 0;
@@ -935,12 +953,18 @@ void register_ext(pybind11::module_& m) {
   m.def("mla_attn", &mla_attn);
   m.def("embed_grams", &embed_grams);
   m.def("add_normed", &add_normed);
-  m.def("norm_rows", &norm_rows);
+  m.def("norm_rows", &norm_rows, pybind11::arg("out"), pybind11::arg("x"), pybind11::arg("idx"), pybind11::arg("w"), pybind11::arg("bias"),
+        pybind11::arg("width"), pybind11::arg("eps"), pybind11::arg("mean") = false);
   m.def("latent_prep", &latent_prep);
   m.def("softcap", &softcap);
   m.def("relu2", &relu2);
-  m.def("latent_attn", &latent_attn);
-  m.def("latent_mma", &latent_mma);
+  m.def("latent_attn", &latent_attn, pybind11::arg("out"), pybind11::arg("o_part"), pybind11::arg("ml_part"), pybind11::arg("q"), pybind11::arg("cache"),
+        pybind11::arg("row_slot"), pybind11::arg("row_kvlen"), pybind11::arg("block_table"), pybind11::arg("kv_block"), pybind11::arg("nsplit"),
+        pybind11::arg("scale"), pybind11::arg("status"), pybind11::arg("window") = 0);
+  m.def("latent_mma", &latent_mma, pybind11::arg("out"), pybind11::arg("o_part"), pybind11::arg("ml_part"), pybind11::arg("q"), pybind11::arg("cache"),
+        pybind11::arg("seg_slot"), pybind11::arg("seg_row0"), pybind11::arg("seg_nrows"), pybind11::arg("max_rows"), pybind11::arg("row_kvlen"),
+        pybind11::arg("block_table"), pybind11::arg("kv_block"), pybind11::arg("row_base"), pybind11::arg("nsplit"), pybind11::arg("scale"),
+        pybind11::arg("status"), pybind11::arg("window") = 0);
   m.def("gemm_f32", &gemm_f32);
   m.def("silu_mul_f32", &silu_mul_f32);
   m.def("gqa_prep", &gqa_prep);
@@ -949,10 +973,12 @@ void register_ext(pybind11::module_& m) {
         pybind11::arg("row_kvlen"), pybind11::arg("block_table"), pybind11::arg("kv_block"), pybind11::arg("row_first"), pybind11::arg("nsplit"), pybind11::arg("scale"),
         pybind11::arg("cuda_cores"), pybind11::arg("status"), pybind11::arg("window") = 0, pybind11::arg("chunk") = 0, pybind11::arg("softcap") = 0.0,
         pybind11::arg("lam") = pybind11::none(), pybind11::arg("gate") = pybind11::none(), pybind11::arg("mix_scale") = 1.0, pybind11::arg("maps") = 1, pybind11::arg("vdim") = 0,
-        pybind11::arg("eps") = 0.0);
+        pybind11::arg("eps") = 0.0, pybind11::arg("k_mean") = pybind11::none(), pybind11::arg("v_mean") = pybind11::none(), pybind11::arg("pool") = 0);
   m.def("gqa_row_prep", &gqa_row_prep);
   m.def("head_mix", &head_mix);
-  m.def("expert_rows", &expert_rows);
+  m.def("expert_rows", &expert_rows, pybind11::arg("yp"), pybind11::arg("act"), pybind11::arg("x"), pybind11::arg("w_gu"), pybind11::arg("w_down"),
+        pybind11::arg("ids"), pybind11::arg("limit") = 0.0, pybind11::arg("shared_gu") = pybind11::none(), pybind11::arg("shared_down") = pybind11::none(),
+        pybind11::arg("shared_limit") = 0.0);
   m.def("add_layer_norm", &add_layer_norm);
   m.def("cd_lowrank", &cd_lowrank);
   m.def("cd_step", &cd_step);
@@ -970,7 +996,9 @@ void register_ext(pybind11::module_& m) {
   pybind11::class_<EpHandle>(m, "EpHandle");
   m.def("make_ep_comm", &make_ep_comm);
   m.def("ep_workspace_bytes", [](int64_t e, int64_t h, int64_t cap) { return (int64_t)fb_ep_workspace_bytes((int)e, (int)h, cap); });
-  m.def("ep_moe", &ep_moe);
+  m.def("ep_moe", &ep_moe, pybind11::arg("comm"), pybind11::arg("out"), pybind11::arg("x"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("w_gu"),
+        pybind11::arg("w_down"), pybind11::arg("shared"), pybind11::arg("shared_gate"), pybind11::arg("res"), pybind11::arg("act"), pybind11::arg("plan"),
+        pybind11::arg("limit") = 0.0, pybind11::arg("add") = true);
   m.def("gemm_grouped", &gemm_grouped);
   m.def("gemm_batched", &gemm_batched);
   m.def("head_linear", &head_linear);

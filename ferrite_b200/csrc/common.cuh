@@ -433,6 +433,13 @@ __device__ __forceinline__ void multimem_red_add_u32(uint32_t* mc_ptr, uint32_t 
 
 // ---- programmatic dependent launch ----------------------------------------------------------------------
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// A pointer to what the kernel before this one wrote, for use after pdl_wait. Loads through `const __restrict__` parameters count as loads of
+// memory that never changes during the kernel, which the compiler may move ahead of the wait; behind this they cannot be.
+template <typename T>
+__device__ __forceinline__ T* after_wait(T* p) {
+  asm volatile("" : "+l"(p)::"memory");
+  return p;
+}
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
 }  // namespace fb

@@ -41,6 +41,7 @@ __global__ void add_conv_normed_kernel(const float* __restrict__ x_in, float* __
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  x_in = after_wait(x_in); y = after_wait(y); yp = after_wait(yp); wts = after_wait(wts);
   const size_t row = blockIdx.x;
   const float* xi = x_in + row * ld;
   float sum = 0.f;
@@ -118,6 +119,7 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(T* __restrict__ out, lon
   __shared__ int before[CR_ROWS], slots[CR_ROWS];            // rows of the step that precede a row, up to taps - 1
   pdl_launch_dependents();
   pdl_wait();
+  x = after_wait(x); tails = after_wait(tails);
   const int r0 = blockIdx.y * CR_ROWS, here = min(CR_ROWS, rows - r0);
   if (threadIdx.x < here) {
     const int r = r0 + threadIdx.x, s = row_slot[r], p = row_pos[r];
@@ -179,6 +181,7 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(T* __restrict__ tails, l
                                                         const int* __restrict__ seg_nrows) {
   pdl_launch_dependents();
   pdl_wait();
+  x = after_wait(x);
   const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y, n = seg_nrows[s], K = taps - 1;
   if (c >= C || n <= 0) return;
   T* t = tails + seg_slot[s] * tail_step + c;

@@ -26,6 +26,7 @@ gqa_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ 
   pdl_launch_dependents();
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
+  proj = after_wait(proj);
   const int pos = row_pos[row];
   for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
     constexpr double TURN = 6.283185307179586476925;
@@ -84,9 +85,10 @@ gqa_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ 
 // The form with norms over whole rows of queries and of keys (weights, before the rotation), a value width of its own and two maps per
 // head. proj row = [heads x maps x dim | kv_heads x maps x dim | .. v_off: kv_heads x vdim]. A key row takes a head's maps side by side; a
 // query goes to [row][head][map][hp] with zeros in the other map's columns, so that one product with the key row gives its map's score.
+// HALF: the rotated pairs are (i, i + rot / 2). Without caches only queries are made (the layer reads another layer's keys).
 // One CTA per row: sums of squares over the row, then one warp per head.
 // Positions, pages and angles do not come from the kernel before this one, so they are read while it drains.
-template <typename T, bool EVEN>
+template <typename T, bool EVEN, bool HALF>
 __global__ void __launch_bounds__(512)
 gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ proj, long ldp,
                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, const double* __restrict__ inv_freq,
@@ -109,6 +111,7 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
   const int blk = block_table[(size_t)row_slot[row] * max_blocks + pos / kv_block];
   if (blk < 0 && threadIdx.x == 0) set_status(status, ST_BOUNDS);
   pdl_wait();
+  proj = after_wait(proj);
   const float* pr = proj + (size_t)row * ldp;
   float rq = 1.f, rk = 1.f;
   if (q_norm) {
@@ -124,9 +127,9 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
       }
       return s;
     };
-    const float sq = squares(pr, nq), sk = squares(pr + nq, nk);
+    const float sq = squares(pr, nq), sk = k_cache ? squares(pr + nq, nk) : 0.f;
     rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
-    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+    if (k_cache) rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
   } else {
     __syncthreads();
   }
@@ -146,13 +149,27 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
       if (e >= 0 && e < dim) x.x = w ? src[e] * r * w[e] : src[e];
       if (e + 1 >= 0 && e + 1 < dim) x.y = w ? src[e + 1] * r * w[e + 1] : src[e + 1];
     }
+    if constexpr (HALF) {                                   // the other column of a pair lies rot / 2 further or back
+      const int hr = rot / 2;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int c = e + k;
+        if (c < 0 || c >= rot) continue;
+        const int o = c < hr ? c + hr : c - hr;
+        const float z = w ? src[o] * r * w[o] : src[o];
+        const float2 t = gr_turn[c < hr ? c : o];
+        float& v = k ? x.y : x.x;
+        v = c < hr ? v * t.x - z * t.y : v * t.x + z * t.y;
+      }
+      return x;
+    }
     if (e >= 0 && e < rot) {                                // rot is even, and so is e wherever something is rotated
       const float2 t = gr_turn[e >> 1];
       x = make_float2(x.x * t.x - x.y * t.y, x.y * t.x + x.x * t.y);
     }
     return x;
   };
-  const int units = heads * maps + 2 * kv_heads;
+  const int units = heads * maps + (k_cache ? 2 * kv_heads : 0);
   for (int u = warp; u < units; u += blockDim.x >> 5) {
     if (u < heads * maps) {
       const float* src = pr + u * dim;
@@ -192,17 +209,109 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
   }
 }
 
+// ---- pooled blocks ------------------------------------------------------------------------------------------------------
+// The mean of the cached keys (values) of every block of `pool` positions whose last one, e, is in the step: into the page of e, at row
+// (e % kv_block) / pool of its mean rows [per_page][kv_heads][hp]. grid (blocks that can end in a segment, kv heads, segments); half of the
+// CTA takes the keys, half the values.
+constexpr int PK_THREADS = 128;
+
+template <typename T>
+__global__ void __launch_bounds__(PK_THREADS) pool_keys_kernel(T* __restrict__ k_mean, T* __restrict__ v_mean, const T* __restrict__ k_cache,
+                                                               const T* __restrict__ v_cache, const int* __restrict__ seg_slot,
+                                                               const int* __restrict__ seg_pos0, const int* __restrict__ seg_nrows,
+                                                               const int* __restrict__ block_table, int max_blocks, int kv_block, int kv_heads, int hp,
+                                                               int pool, int per_page, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  k_cache = after_wait(k_cache); v_cache = after_wait(v_cache);
+  const int seg = blockIdx.z, h = blockIdx.y, p0 = seg_pos0[seg], n = seg_nrows[seg];
+  const int e = (p0 / pool + 1 + blockIdx.x) * pool - 1;                 // last position of the block
+  if (e >= p0 + n) return;
+  const int* bt = block_table + (size_t)seg_slot[seg] * max_blocks;
+  const bool keys = threadIdx.x < PK_THREADS / 2;
+  const T* cache = keys ? k_cache : v_cache;
+  const int own = bt[e / kv_block];
+  if (own < 0) { if (threadIdx.x == 0) set_status(status, ST_BOUNDS); return; }
+  T* dst = (keys ? k_mean : v_mean) + (((size_t)own * per_page + e % kv_block / pool) * kv_heads + h) * hp;
+  const float inv = 1.f / (float)pool;
+  for (int d = (threadIdx.x % (PK_THREADS / 2)) * 4; d < hp; d += PK_THREADS / 2 * 4) {
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int t = e - pool + 1; t <= e; ++t) {
+      const int blk = bt[t / kv_block];
+      if (blk < 0) { set_status(status, ST_BOUNDS); continue; }
+      const float4 v = Elem<T>::load4(cache + (((size_t)blk * kv_block + t % kv_block) * kv_heads + h) * hp + d);
+      s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+    }
+    Elem<T>::store4(dst + d, make_float4(s.x * inv, s.y * inv, s.z * inv, s.w * inv));
+  }
+}
+
+// Mean rows of the blocks that a prompt's rows see, side by side: out rows [start[seg], start[seg] + count[seg]) of segment seg, zeros up to
+// start[seg + 1]; grid (rows of out). A row is `width` elements of keys and as many of values.
+__global__ void __launch_bounds__(128) pool_gather_kernel(__nv_bfloat16* __restrict__ k_out, __nv_bfloat16* __restrict__ v_out,
+                                                          const __nv_bfloat16* __restrict__ k_mean, const __nv_bfloat16* __restrict__ v_mean,
+                                                          const int* __restrict__ seg_slot, const int* __restrict__ start, const int* __restrict__ count,
+                                                          int nseg, const int* __restrict__ block_table, int max_blocks, int kv_block, int width,
+                                                          int pool, int per_page, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  k_mean = after_wait(k_mean); v_mean = after_wait(v_mean);
+  const int row = blockIdx.x;
+  int seg = 0;
+  while (seg + 1 < nseg && start[seg + 1] <= row) ++seg;
+  const int b = row - start[seg], e = b * pool + pool - 1;
+  int blk = -1;
+  if (b < count[seg]) {
+    blk = block_table[(size_t)seg_slot[seg] * max_blocks + e / kv_block];
+    if (blk < 0 && threadIdx.x == 0) set_status(status, ST_BOUNDS);
+  }
+  const size_t src = blk < 0 ? 0 : ((size_t)blk * per_page + e % kv_block / pool) * width, dst = (size_t)row * width;
+  for (int i = threadIdx.x * 8; i < width; i += 128 * 8) {
+    const uint4 z = make_uint4(0, 0, 0, 0);
+    *reinterpret_cast<uint4*>(k_out + dst + i) = blk < 0 ? z : *reinterpret_cast<const uint4*>(k_mean + src + i);
+    *reinterpret_cast<uint4*>(v_out + dst + i) = blk < 0 ? z : *reinterpret_cast<const uint4*>(v_mean + src + i);
+  }
+}
+
 }  // namespace fb
 
 using namespace fb;
 
+// Caches [page][kv_block][kv_heads][hp], means [page][per_page][kv_heads][hp]
+extern "C" int fb_pool_keys(void* k_mean, void* v_mean, const void* k_cache, const void* v_cache, const int* seg_slot, const int* seg_pos0,
+                            const int* seg_nrows, int nseg, int max_rows, const int* block_table, int max_blocks, int kv_block, int kv_heads, int hp,
+                            int pool, int f32, int* status, cudaStream_t s) {
+  if (nseg <= 0 || max_rows <= 0) return 0;
+  if (pool < 1 || hp % 4 || kv_heads < 1 || kv_heads > 65535 || nseg > 65535) return -1;
+  const dim3 grid((max_rows - 1) / pool + 1, kv_heads, nseg);
+  const int per_page = (kv_block + pool - 1) / pool;
+  auto go = [&](auto kern, auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    return (int)launch_pdl(kern, grid, dim3(PK_THREADS), 0, s, (T*)k_mean, (T*)v_mean, (const T*)k_cache, (const T*)v_cache, seg_slot, seg_pos0,
+                           seg_nrows, block_table, max_blocks, kv_block, kv_heads, hp, pool, per_page, status);
+  };
+  return f32 ? go(pool_keys_kernel<float>, (float*)0) : go(pool_keys_kernel<__nv_bfloat16>, (__nv_bfloat16*)0);
+}
+
+extern "C" int fb_pool_gather(void* k_out, void* v_out, const void* k_mean, const void* v_mean, const int* seg_slot, const int* start,
+                              const int* count, int nseg, int rows, const int* block_table, int max_blocks, int kv_block, int width, int pool,
+                              int* status, cudaStream_t s) {
+  if (nseg <= 0 || rows <= 0) return 0;
+  if (pool < 1 || width % 8) return -1;
+  return (int)launch_pdl(pool_gather_kernel, dim3(rows), dim3(128), 0, s, (__nv_bfloat16*)k_out, (__nv_bfloat16*)v_out, (const __nv_bfloat16*)k_mean,
+                         (const __nv_bfloat16*)v_mean, seg_slot, start, count, nseg, block_table, max_blocks, kv_block, width, pool,
+                         (kv_block + pool - 1) / pool, status);
+}
+
 extern "C" int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* q_norm,
                                const float* k_norm, const double* inv_freq, const int* row_slot, const int* row_pos, const int* block_table,
                                int max_blocks, int kv_block, int rows, int heads, int kv_heads, int maps, int dim, int vdim, int hp, int rot,
-                               int v_off, float eps, int f32, int* status, cudaStream_t s) {
+                               int v_off, int half, float eps, int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
+  if (!k_cache != !v_cache || (half && maps != 1)) return -1;
   if (dim < 1 || vdim < 1 || maps < 1 || maps > 2 || maps * dim > hp || vdim > hp || hp % 64 || rot % 2 || rot > dim || (rot && !inv_freq) ||
-      (rot && maps == 2 && dim % 2) || (!q_norm) != (!k_norm)) return -1;
+      (rot && maps == 2 && dim % 2) || (k_cache && (!q_norm) != (!k_norm))) return -1;
   const size_t smem = (size_t)(rot / 2 + 1) * sizeof(float2);
   const int threads = heads * maps + 2 * kv_heads > 16 ? 512 : 256;
   auto go = [&](auto kern, auto* tag) {
@@ -214,8 +323,12 @@ extern "C" int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const 
   using B = __nv_bfloat16;
   const bool even = dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && v_off % 2 == 0 &&
                     (((uintptr_t)proj | (uintptr_t)q_norm | (uintptr_t)k_norm) & 7) == 0;
-  if (even) return f32 ? go(gqa_row_prep_kernel<float, true>, (float*)0) : go(gqa_row_prep_kernel<B, true>, (B*)0);
-  return f32 ? go(gqa_row_prep_kernel<float, false>, (float*)0) : go(gqa_row_prep_kernel<B, false>, (B*)0);
+  if (half) {
+    if (even) return f32 ? go(gqa_row_prep_kernel<float, true, true>, (float*)0) : go(gqa_row_prep_kernel<B, true, true>, (B*)0);
+    return f32 ? go(gqa_row_prep_kernel<float, false, true>, (float*)0) : go(gqa_row_prep_kernel<B, false, true>, (B*)0);
+  }
+  if (even) return f32 ? go(gqa_row_prep_kernel<float, true, false>, (float*)0) : go(gqa_row_prep_kernel<B, true, false>, (B*)0);
+  return f32 ? go(gqa_row_prep_kernel<float, false, false>, (float*)0) : go(gqa_row_prep_kernel<B, false, false>, (B*)0);
 }
 
 extern "C" int fb_gqa_prep(void* q_out, void* k_cache, void* v_cache, const float* proj, long ldp, const float* bias,

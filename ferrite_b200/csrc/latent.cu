@@ -94,6 +94,7 @@ __global__ void add_normed_kernel(float* __restrict__ x, T* __restrict__ xb, lon
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  y = after_wait(y);
   const size_t row = blockIdx.x;
   const S* yr = y + row * ldy;
   float ss = 0.f;
@@ -136,6 +137,7 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const float* __restrict__ 
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  x = after_wait(x);
   const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * ld;
   const float r = row_rscale<float>(xr, ld, width, eps, red);
   for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
@@ -168,7 +170,7 @@ template <typename T>
 __device__ __forceinline__ void ln_store(T* out, const float* row, float2 st, const float* w, const float* b, int ld) {
   for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
     float4 v = *reinterpret_cast<const float4*>(row + i);
-    const float4 ww = *reinterpret_cast<const float4*>(w + i), bb = *reinterpret_cast<const float4*>(b + i);
+    const float4 ww = *reinterpret_cast<const float4*>(w + i), bb = b ? *reinterpret_cast<const float4*>(b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     v.x = (v.x - st.x) * st.y * ww.x + bb.x; v.y = (v.y - st.x) * st.y * ww.y + bb.y;
     v.z = (v.z - st.x) * st.y * ww.z + bb.z; v.w = (v.w - st.x) * st.y * ww.w + bb.w;
     Elem<T>::store4(out + i, v);
@@ -184,6 +186,7 @@ __global__ void add_layer_norm_kernel(float* __restrict__ x, T* __restrict__ xb,
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  y = after_wait(y); yp = after_wait(yp); wts = after_wait(wts);
   const size_t row = blockIdx.x;
   const S* yr = y + row * ldy;
   float* xr = x + row * ld;
@@ -214,6 +217,7 @@ __global__ void layer_norm_rows_kernel(T* __restrict__ out, const float* __restr
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  x = after_wait(x);
   const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * ld;
   float sum = 0.f;
   for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
@@ -236,6 +240,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ cq, T*
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  proj = after_wait(proj);
   const size_t row = blockIdx.x;
   const float* pr = proj + row * ldp;
   float r = row_rscale<float>(pr, qr, q_rank, eps, red);
@@ -260,6 +265,59 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ cq, T*
   }
 }
 
+// The form with a rotated key part: proj row = [heads x (dim | rot) | latent (kv_rank) | key part (rot)], fp32. Queries go to [row][head][hp] with
+// their last rot columns rotated (pairs (0, 1), (2, 3), ..), the normed latent and the rotated key part to the token's cache row, zeros beyond.
+// Angles are formed and reduced to one turn in double.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rot_prep_kernel(T* __restrict__ q_out, T* __restrict__ cache, const float* __restrict__ proj, long ldp,
+                                                              const float* __restrict__ kv_norm, const double* __restrict__ inv_freq,
+                                                              const int* __restrict__ row_slot, const int* __restrict__ row_pos,
+                                                              const int* __restrict__ block_table, int max_blocks, int kv_block, int heads, int dim,
+                                                              int rot, int hp, int kv_rank, int lat, float eps, int* status) {
+  extern __shared__ float2 lr_turn[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  const size_t row = blockIdx.x;
+  const int pos = row_pos[row];
+  for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+    constexpr double TURN = 6.283185307179586476925;
+    double a = (double)pos * inv_freq[i];
+    a -= TURN * rint(a / TURN);
+    float s, c;
+    sincosf((float)a, &s, &c);
+    lr_turn[i] = make_float2(c, s);
+  }
+  const int blk = block_table[(size_t)row_slot[row] * max_blocks + pos / kv_block];
+  pdl_wait();
+  proj = after_wait(proj);
+  const float* pr = proj + row * ldp;
+  const int kd = dim + rot;
+  const float* pc = pr + (size_t)heads * kd;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss = fmaf(pc[i], pc[i], ss);
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)kv_rank + eps);      // (its barriers publish the angles)
+  auto turned = [&](const float* src, int e) {               // column e of a rotated part
+    const float2 t = lr_turn[e >> 1];
+    const float u = src[e & ~1], v = src[e | 1];
+    return e & 1 ? v * t.x + u * t.y : u * t.x - v * t.y;
+  };
+  if (blk < 0) {
+    if (threadIdx.x == 0) set_status(status, ST_BOUNDS);
+  } else {
+    T* dst = cache + ((size_t)blk * kv_block + pos % kv_block) * lat;
+    for (int i = threadIdx.x; i < lat; i += blockDim.x)
+      dst[i] = Elem<T>::from(i < kv_rank ? pc[i] * r * kv_norm[i] : i < kv_rank + rot ? turned(pc + kv_rank, i - kv_rank) : 0.f);
+  }
+  for (int i = 2 * threadIdx.x; i < heads * hp; i += 2 * blockDim.x) {
+    const int h = i / hp, d = i % hp;
+    const float* src = pr + h * kd;
+    float o[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) o[e] = d + e < dim ? src[d + e] : d + e < kd ? turned(src + dim, d + e - dim) : 0.f;
+    Elem<T>::store2(q_out + row * (size_t)heads * hp + i, o[0], o[1]);
+  }
+}
+
 __global__ void softcap_kernel(float* __restrict__ y, long ld, int n, float cap) {
   pdl_launch_dependents();
   pdl_wait();
@@ -281,7 +339,8 @@ __global__ void relu2_kernel(__nv_bfloat16* __restrict__ y, const __nv_bfloat16*
 // lat = 64 nl with nl <= NJ. One split writes the normalised output itself, more leave partials for the merge. KV: cache rows are
 // [kv_heads][lat] of keys with the values in v_cache (else one latent row, keys and values alike); sink: a number per head that
 // joins the denominator; window / chunk bound the keys a row sees, cap > 0 softcaps the scores (scale_log2 is then scale / cap).
-// `records`: one split leaves its partial as well. Rows of out are ldo elements apart.
+// `records`: one split leaves its partial as well. Rows of out are ldo elements apart and have vl columns per head (latents: the first ones of
+// a cache row). pool > 0 (KV): the means of the blocks before the window come first in the list of keys.
 constexpr int LA_WARPS = 4;
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -294,20 +353,24 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
                                                                     const int* __restrict__ block_table, int max_blocks,
                                                                     int kv_block, int heads, int kv_heads, int lat, int nsplit,
                                                                     float scale_log2, int window, int chunk, float cap, long ldo, int records,
+                                                                    int vl, const T* __restrict__ k_mean, const T* __restrict__ v_mean, int pool,
                                                                     int* status) {
   extern __shared__ float so[];                            // [warps][lat]
   __shared__ float sml[LA_WARPS][2];
   pdl_launch_dependents();
   pdl_wait();
+  q = after_wait(q); cache = after_wait(cache); v_cache = after_wait(v_cache); k_mean = after_wait(k_mean); v_mean = after_wait(v_mean);
   const int nl = lat / 64;
   const int row = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kvlen = row_kvlen[row];
   const int* bt = block_table + (size_t)row_slot[row] * max_blocks;
-  const int kv_lo = KV ? first_key(kvlen - 1, window, chunk) : 0;
-  int per = (kvlen - kv_lo + nsplit - 1) / nsplit;
+  const int kv_lo = first_key(kvlen - 1, window, chunk);
+  // list of keys: nb means, then the tokens from kv_lo on
+  const int nb = KV && pool > 0 ? kv_lo / pool : 0, keys = nb + kvlen - kv_lo, per_page = KV && pool > 0 ? (kv_block + pool - 1) / pool : 1;
+  int per = (keys + nsplit - 1) / nsplit;
   per = (per + 31) / 32 * 32;
-  const int lo = kv_lo + split * per, hi = min(kvlen, lo + per);
+  const int lo = split * per, hi = min(keys, lo + per);
   const T* qr = q + ((size_t)row * heads + h) * lat;
   float2 qf[NJ], o[NJ];
 #pragma unroll
@@ -317,12 +380,14 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
     qf[j].x *= scale_log2; qf[j].y *= scale_log2;
   }
   float m = -INFINITY, l = 0.f;
-  for (int t = lo + warp; t < hi; t += LA_WARPS) {
+  for (int u = lo + warp; u < hi; u += LA_WARPS) {
+    const bool mean = u < nb;
+    const int t = mean ? u * pool + pool - 1 : u - nb + kv_lo;
     const int blk = bt[t / kv_block];
     if (blk < 0) { if (lane == 0) set_status(status, ST_BOUNDS); break; }
-    size_t at = (size_t)blk * kv_block + t % kv_block;
+    size_t at = mean ? (size_t)blk * per_page + t % kv_block / pool : (size_t)blk * kv_block + t % kv_block;
     if constexpr (KV) at = at * kv_heads + h / (heads / kv_heads);
-    const T* kr = cache + at * lat + 2 * lane;
+    const T* kr = (mean ? k_mean : cache) + at * lat + 2 * lane;
     float2 k[NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) k[j] = j < nl ? Elem<T>::load2(kr + 64 * j) : make_float2(0.f, 0.f);
@@ -335,7 +400,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
     const float a = exp2f(m - mn), p = exp2f(s - mn);
     l = l * a + p;
     if constexpr (KV) {
-      const T* vr = v_cache + at * lat + 2 * lane;
+      const T* vr = (mean ? v_mean : v_cache) + at * lat + 2 * lane;
 #pragma unroll
       for (int j = 0; j < NJ; ++j) k[j] = j < nl ? Elem<T>::load2(vr + 64 * j) : make_float2(0.f, 0.f);
     }
@@ -360,12 +425,12 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(T* __restric
   const float den = Ls + (sink && nsplit == 1 ? exp2f(sink[h] * LOG2E - M) : 0.f);
   const bool final_rows = nsplit == 1 && !records;
   const float inv = final_rows ? (den > 0.f ? 1.f / den : 0.f) : 1.f;
-  for (int d = threadIdx.x; d < lat; d += blockDim.x) {
+  for (int d = threadIdx.x; d < vl; d += blockDim.x) {
     float acc = 0.f;
 #pragma unroll
     for (int w = 0; w < LA_WARPS; ++w) acc += so[(size_t)w * lat + d] * f[w];
-    if (final_rows) out[(size_t)row * ldo + (size_t)h * lat + d] = Elem<T>::from(acc * inv);
-    else o_part[pidx * lat + d] = acc;
+    if (final_rows) out[(size_t)row * ldo + (size_t)h * vl + d] = Elem<T>::from(acc * inv);
+    else o_part[pidx * vl + d] = acc;
   }
   if (!final_rows && threadIdx.x == 0) { ml_part[pidx * 2] = M; ml_part[pidx * 2 + 1] = Ls; }
 }
@@ -382,6 +447,7 @@ __global__ void __launch_bounds__(128 * LG_GROUPS) latent_merge_kernel(T* __rest
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  o_part = after_wait(o_part); ml_part = after_wait(ml_part);
   const size_t rh = (size_t)blockIdx.x * heads + blockIdx.y, pbase = rh * nsplit;
   const int tid = threadIdx.x, grp = tid / 128, col = (tid % 128) * 4;
   float M = -INFINITY, Ls = 0.f;
@@ -436,6 +502,7 @@ __global__ void __launch_bounds__(MX_THREADS) attn_merge_mix_kernel(T* __restric
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  o_part = after_wait(o_part); ml_part = after_wait(ml_part); gate = after_wait(gate);
   const int tid = threadIdx.x, map = tid / PER, t = tid % PER, warp = tid >> 5, lane = tid & 31;
   const size_t row = blockIdx.x;
   const int h = blockIdx.y;
@@ -501,6 +568,7 @@ __global__ void __launch_bounds__(256) head_mix_kernel(T* __restrict__ out, long
                                                        float eps) {
   pdl_launch_dependents();
   pdl_wait();
+  in = after_wait(in); gate = after_wait(gate);
   const size_t row = blockIdx.x;
   const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (h >= heads) return;
@@ -544,7 +612,9 @@ __global__ void __launch_bounds__(256) head_mix_kernel(T* __restrict__ out, long
 // transposed: warp = all 64 M rows x lat / 8 columns. The softmax weights go through shared memory as a bf16 value plus its bf16
 // remainder, two products each, so they keep 16 bits of mantissa instead of 8; scores, maxima, exponentials and row sums are
 // 32-bit.
-constexpr int LM_M = 64, LM_KEYS = 64, LM_THREADS = 256, LM_LDP = LM_KEYS + 8;
+// A cache row has 64 NJ columns; values are its first 64 VJ (the rest is a key part). M is 64, or 32 where rows are so wide that two key
+// tiles and 64 queries do not fit.
+constexpr int LM_KEYS = 64, LM_THREADS = 256, LM_LDP = LM_KEYS + 8;
 
 __device__ __forceinline__ void lm_cp16(void* smem, const void* gmem, bool valid) {
   const int sz = valid ? 16 : 0;
@@ -566,6 +636,7 @@ __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], ui
 
 template <int NJ>
 struct Lm {
+  static constexpr int LM_M = NJ <= 8 ? 64 : 32, VJ = NJ <= 8 ? NJ : 8;
   static constexpr int LAT = NJ * 64, LD = LAT + 8;
   static constexpr size_t SMEM = (size_t)(LM_M + 2 * LM_KEYS) * LD * 2 + (size_t)2 * LM_M * LM_LDP * 2 + 6 * LM_M * 4;
 };
@@ -576,8 +647,8 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
                   const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache, const int* __restrict__ seg_slot,
                   const int* __restrict__ seg_row0, const int* __restrict__ seg_nrows, const int* __restrict__ row_kvlen,
                   const int* __restrict__ block_table, int max_blocks, int kv_block, int heads, int row_base, int tiles_per_seg,
-                  int nsplit, float scale_log2, int* status) {
-  constexpr int LAT = Lm<NJ>::LAT, LD = Lm<NJ>::LD, CPR = LAT / 8;
+                  int nsplit, float scale_log2, int window, int* status) {
+  constexpr int LAT = Lm<NJ>::LAT, LD = Lm<NJ>::LD, CPR = LAT / 8, LM_M = Lm<NJ>::LM_M, MT = LM_M / 16, VJ = Lm<NJ>::VJ, VL = VJ * 64;
   extern __shared__ __align__(16) unsigned char lm_smem[];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [M][LD]
   __nv_bfloat16* sK = sQ + LM_M * LD;                                      // [2][KEYS][LD]
@@ -594,9 +665,10 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
   const int row0 = seg_row0[seg];
   const int* bt = block_table + (size_t)seg_slot[seg] * max_blocks;
   const int kv_end = row_kvlen[row0 + (m0 + valid_m - 1) / heads - row_base];          // rows of a segment see ever more keys
-  int per = (kv_end + nsplit - 1) / nsplit;
+  const int kv_lo = first_key(row_kvlen[row0 + m0 / heads - row_base] - 1, window, 0) / LM_KEYS * LM_KEYS;
+  int per = (kv_end - kv_lo + nsplit - 1) / nsplit;
   per = (per + LM_KEYS - 1) / LM_KEYS * LM_KEYS;
-  const int lo = split * per, hi = min(kv_end, lo + per);
+  const int lo = kv_lo + split * per, hi = min(kv_end, lo + per);
   // (row, head) flat index of an M row in q / out, which start at row row_base of the step
   const size_t flat0 = (size_t)(row0 - row_base) * heads + m0;
   if (lo >= hi) {
@@ -632,18 +704,19 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
   const int mw = few ? warp & 1 : warp & 3, nw = few ? warp >> 1 : warp >> 2, kgroups = few ? 4 : 2;
   const int npairs = few ? 1 : 2, key0 = nw * 16 * npairs;
   const int r_lo = mw * 16 + lane / 4;                       // this thread's two M rows: r_lo, r_lo + 8
-  int kvl[2];
+  int kvl[2], klo[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int m = r_lo + 8 * h;
     kvl[h] = m < valid_m ? row_kvlen[row0 + (m0 + m) / heads - row_base] : 0;
+    klo[h] = m < valid_m ? first_key(kvl[h] - 1, window, 0) : 0;
   }
   float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
-  float o[4][NJ][4];
+  float o[MT][VJ][4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+  for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int j = 0; j < NJ; ++j) { o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f; }
+    for (int j = 0; j < VJ; ++j) { o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f; }
   const int ntiles = (hi - lo + LM_KEYS - 1) / LM_KEYS;
   const bool score_on = mw * 16 < valid_m;
 
@@ -686,7 +759,7 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = kbase + nt * 8 + (e & 1), h = e >> 1;
-          const float v = (nt < 2 * npairs && t < kvl[h] && t < hi) ? s[nt][e] * scale_log2 : -INFINITY;
+          const float v = (nt < 2 * npairs && t < kvl[h] && t >= klo[h] && t < hi) ? s[nt][e] * scale_log2 : -INFINITY;
           s[nt][e] = v;
           mx[h] = fmaxf(mx[h], v);
         }
@@ -724,20 +797,20 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
     }
     __syncthreads();
 #pragma unroll
-    for (int mt = 0; mt < 4; ++mt) {
+    for (int mt = 0; mt < MT; ++mt) {
       if (mt * 16 >= valid_m) break;
       const float f0 = sfac[mt * 16 + lane / 4], f1 = sfac[mt * 16 + lane / 4 + 8];
       if (!__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) continue;
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) { o[mt][j][0] *= f0; o[mt][j][1] *= f0; o[mt][j][2] *= f1; o[mt][j][3] *= f1; }
+      for (int j = 0; j < VJ; ++j) { o[mt][j][0] *= f0; o[mt][j][1] *= f0; o[mt][j][2] *= f1; o[mt][j][3] *= f1; }
     }
 #pragma unroll
     for (int kp = 0; kp < 2; ++kp) {
-      uint32_t b[NJ][4];                                     // 8 columns x 32 keys each: two k steps
+      uint32_t b[VJ][4];                                     // 8 columns x 32 keys each: two k steps
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) lm_ldsm_t(b[j], K + (kp * 32 + lane) * LD + (warp * NJ + j) * 8);
+      for (int j = 0; j < VJ; ++j) lm_ldsm_t(b[j], K + (kp * 32 + lane) * LD + (warp * VJ + j) * 8);
 #pragma unroll
-      for (int mt = 0; mt < 4; ++mt) {
+      for (int mt = 0; mt < MT; ++mt) {
         if (mt * 16 >= valid_m) break;
 #pragma unroll
         for (int k2 = 0; k2 < 2; ++k2) {
@@ -746,7 +819,7 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
             uint32_t a[4];
             lm_ldsm(a, sP + (part * LM_M + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LM_LDP + (kp * 2 + k2) * 16 + (lane >> 4) * 8);
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) lm_mma(o[mt][j], a, b[j][2 * k2], b[j][2 * k2 + 1]);
+            for (int j = 0; j < VJ; ++j) lm_mma(o[mt][j], a, b[j][2 * k2], b[j][2 * k2 + 1]);
           }
         }
       }
@@ -778,19 +851,19 @@ latent_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ o_part, f
   }
   __syncthreads();
 #pragma unroll
-  for (int mt = 0; mt < 4; ++mt)
+  for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int r = mt * 16 + lane / 4 + 8 * h;
       if (r >= valid_m) continue;
       const float inv = nsplit == 1 ? sinv[r] : 1.f;
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int d = (warp * NJ + j) * 8 + (lane & 3) * 2;
+      for (int j = 0; j < VJ; ++j) {
+        const int d = (warp * VJ + j) * 8 + (lane & 3) * 2;
         if (nsplit == 1)
-          *reinterpret_cast<uint32_t*>(out + (flat0 + r) * LAT + d) = pack_bf2(o[mt][j][2 * h] * inv, o[mt][j][2 * h + 1] * inv);
+          *reinterpret_cast<uint32_t*>(out + (flat0 + r) * VL + d) = pack_bf2(o[mt][j][2 * h] * inv, o[mt][j][2 * h + 1] * inv);
         else
-          *reinterpret_cast<float2*>(o_part + ((flat0 + r) * nsplit + split) * LAT + d) = make_float2(o[mt][j][2 * h], o[mt][j][2 * h + 1]);
+          *reinterpret_cast<float2*>(o_part + ((flat0 + r) * nsplit + split) * VL + d) = make_float2(o[mt][j][2 * h], o[mt][j][2 * h + 1]);
       }
     }
 }
@@ -883,13 +956,13 @@ static int row_smem(Kern kern, size_t smem) {
   return smem > 40 * 1024 ? (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : 0;
 }
 
-// b: bias of a layer norm, or null for the root mean square norm
-extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int rows, int width, int ld, float eps,
-                            int f32, cudaStream_t s) {
+// mean: layer norm (b: its bias, or null), else the root mean square norm
+extern "C" int fb_norm_rows(void* out, const float* x, const int* idx, const float* w, const float* b, int mean, int rows, int width, int ld,
+                            float eps, int f32, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (ld % 4 || ld > 49152) return -1;
   const dim3 g(rows), t(row_threads(ld));
-  if (b) {
+  if (b || mean) {
     auto go = [&](auto kern, auto* o) {
       if (const int e = row_smem(kern, (size_t)ld * 4)) return e;
       return (int)launch_pdl(kern, g, t, (size_t)ld * 4, s, o, x, idx, w, b, width, ld, eps);
@@ -929,6 +1002,20 @@ extern "C" int fb_latent_prep(void* cq, void* cache, const float* proj, long ldp
                          block_table, max_blocks, kv_block, q_rank, qr, kv_rank, lat, eps, status);
 }
 
+// proj: rows of heads * (dim + rot) + kv_rank + rot floats, ldp apart; kv_norm: kv_rank floats; lat >= kv_rank + rot, hp >= dim + rot
+extern "C" int fb_latent_rot_prep(void* q_out, void* cache, const float* proj, long ldp, const float* kv_norm, const double* inv_freq,
+                                  const int* row_slot, const int* row_pos, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
+                                  int dim, int rot, int hp, int kv_rank, int lat, float eps, int f32, int* status, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (rot % 2 || rot < 0 || dim < 0 || dim + rot > hp || hp % 2 || kv_rank < 1 || kv_rank + rot > lat) return -1;
+  auto go = [&](auto kern, auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    return (int)launch_pdl(kern, dim3(rows), dim3(256), (size_t)(rot / 2 + 1) * sizeof(float2), s, (T*)q_out, (T*)cache, proj, ldp, kv_norm, inv_freq,
+                           row_slot, row_pos, block_table, max_blocks, kv_block, heads, dim, rot, hp, kv_rank, lat, eps, status);
+  };
+  return f32 ? go(latent_rot_prep_kernel<float>, (float*)0) : go(latent_rot_prep_kernel<bf16>, (bf16*)0);
+}
+
 extern "C" int fb_softcap(float* y, int rows, int n, long ld, float cap, cudaStream_t s) {
   if (rows <= 0 || n <= 0) return 0;
   if (rows > 65535) return -1;
@@ -952,18 +1039,19 @@ static int latent_merge(void* out, long ldo, const float* o_part, const float* m
 template <typename T, bool KV>
 static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const void* v_cache, const float* sink,
                        const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads,
-                       int kv_heads, int lat, int nsplit, float scale, const KeyBounds* kb, long ldo, bool records, int* status,
-                       cudaStream_t s) {
+                       int kv_heads, int lat, int vl, int nsplit, float scale, const KeyBounds* kb, const PoolKeys* pool, long ldo, bool records,
+                       int* status, cudaStream_t s) {
   const KeyBounds none{0, 0, 0.f};
   const KeyBounds& b = kb ? *kb : none;
-  if (b.window < 0 || b.chunk < 0 || (b.window && b.chunk) || b.cap < 0.f) return -1;
+  if (b.window < 0 || b.chunk < 0 || (b.window && b.chunk) || b.cap < 0.f || (pool && (pool->size < 1 || !b.window))) return -1;
   const float scale_log2 = b.cap > 0.f ? scale / b.cap : scale * LOG2E;
   const dim3 grid(rows, heads, nsplit);
   const size_t smem = (size_t)LA_WARPS * lat * 4;
   auto go = [&](auto kern) {
     return (int)launch_pdl(kern, grid, dim3(LA_WARPS * 32), smem, s, (T*)out, o_part, ml_part, (const T*)q, (const T*)cache,
                            (const T*)v_cache, sink, row_slot, row_kvlen, block_table, max_blocks, kv_block, heads, kv_heads, lat, nsplit,
-                           scale_log2, b.window, b.chunk, b.cap, ldo, records ? 1 : 0, status);
+                           scale_log2, b.window, b.chunk, b.cap, ldo, records ? 1 : 0, vl, pool ? (const T*)pool->k : nullptr,
+                           pool ? (const T*)pool->v : nullptr, pool ? pool->size : 0, status);
   };
   int rc;
   if (lat <= 128) rc = go(latent_attn_kernel<T, 2, KV>);
@@ -971,35 +1059,37 @@ static int latent_attn(void* out, float* o_part, float* ml_part, const void* q, 
   else if (lat <= 512) rc = go(latent_attn_kernel<T, 8, KV>);
   else rc = go(latent_attn_kernel<T, 16, KV>);
   if (rc || nsplit == 1 || records) return rc;
-  return latent_merge<T>(out, ldo, o_part, ml_part, sink, rows, heads, nsplit, lat, s);
+  return latent_merge<T>(out, ldo, o_part, ml_part, sink, rows, heads, nsplit, vl, s);
 }
 
-// out [rows][heads][lat]; partials (nsplit > 1): o_part rows * heads * nsplit * lat floats, ml_part two per record
+// out [rows][heads][vl] (the first vl columns of the rows; 64 | vl); window: keys that a row sees, 0 = all; partials (nsplit > 1): o_part rows * heads * nsplit * lat floats, ml_part two per record
 extern "C" int fb_latent_attn(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* row_slot,
                               const int* row_kvlen, const int* block_table, int max_blocks, int kv_block, int rows, int heads, int lat,
-                              int nsplit, float scale, int f32, int* status, cudaStream_t s) {
+                              int vl, int window, int nsplit, float scale, int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
+  if (vl % 64 || vl > lat || window < 0) return -1;
+  const KeyBounds kb{window, 0, 0.f};
   if (lat % 64 || lat > 1024 || heads > 65535 || nsplit < 1 || nsplit > 4096) return -1;
-  const long ldo = (long)heads * lat;
+  const long ldo = (long)heads * vl;
   return f32 ? latent_attn<float, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
-                                         kv_block, rows, heads, 1, lat, nsplit, scale, nullptr, ldo, false, status, s)
+                                         kv_block, rows, heads, 1, lat, vl, nsplit, scale, &kb, nullptr, ldo, false, status, s)
              : latent_attn<bf16, false>(out, o_part, ml_part, q, cache, nullptr, nullptr, row_slot, row_kvlen, block_table, max_blocks,
-                                        kv_block, rows, heads, 1, lat, nsplit, scale, nullptr, ldo, false, status, s);
+                                        kv_block, rows, heads, 1, lat, vl, nsplit, scale, &kb, nullptr, ldo, false, status, s);
 }
 
 // The same over separate keys and values: caches [page][kv_block][kv_heads][hd], q / out [rows][heads][hd] (rows of out ldo elements
-// apart); sink: heads floats or null; kb: window, chunk, softcap, or null; out null: the records of the splits stay for the caller
+// apart); sink: heads floats or null; kb: window, chunk, softcap, or null; pool: means of the blocks before the window, or null; out null: the records of the splits stay for the caller
 extern "C" int fb_gqa_attn(void* out, float* o_part, float* ml_part, const void* q, const void* k_cache, const void* v_cache,
                            const float* sink, const int* row_slot, const int* row_kvlen, const int* block_table, int max_blocks,
-                           int kv_block, int rows, int heads, int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb, long ldo,
-                           int f32, int* status, cudaStream_t s) {
+                           int kv_block, int rows, int heads, int kv_heads, int hd, int nsplit, float scale, const KeyBounds* kb,
+                           const PoolKeys* pool, long ldo, int f32, int* status, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (hd % 64 || hd > 1024 || heads > 65535 || kv_heads <= 0 || heads % kv_heads || nsplit < 1 || nsplit > 4096) return -1;
   if (ldo % 4 || (!out && sink)) return -1;
   return f32 ? latent_attn<float, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
-                                        kv_block, rows, heads, kv_heads, hd, nsplit, scale, kb, ldo, !out, status, s)
+                                        kv_block, rows, heads, kv_heads, hd, hd, nsplit, scale, kb, pool, ldo, !out, status, s)
              : latent_attn<bf16, true>(out, o_part, ml_part, q, k_cache, v_cache, sink, row_slot, row_kvlen, block_table, max_blocks,
-                                       kv_block, rows, heads, kv_heads, hd, nsplit, scale, kb, ldo, !out, status, s);
+                                       kv_block, rows, heads, kv_heads, hd, hd, nsplit, scale, kb, pool, ldo, !out, status, s);
 }
 
 // Merge of key splits alone (records as fb_attn_decode_mma leaves them), sink: heads floats or null
@@ -1040,16 +1130,16 @@ extern "C" int fb_head_mix(void* out, long ldo, const float* in, const float* la
   return maps == 2 ? go(head_mix_kernel<bf16, 2>, (bf16*)out) : go(head_mix_kernel<bf16, 1>, (bf16*)out);
 }
 
-// The same on tensor cores for bf16, lat <= 512 and pages of a multiple of 64 keys (-20 otherwise). Rows come in
+// The same on tensor cores for bf16, lat <= 512 with vl = lat, or 576 with vl = 512, and pages of a multiple of 64 keys (-20 otherwise). Rows come in
 // segments (consecutive rows of one slot); seg_row0 counts the rows of the step, of which q / out / row_kvlen hold those from row_base on.
 extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const void* q, const void* cache, const int* seg_slot,
                              const int* seg_row0, const int* seg_nrows, int nseg, int max_rows, const int* row_kvlen,
                              const int* block_table, int max_blocks, int kv_block, int rows, int row_base, int heads, int lat,
-                             int nsplit, float scale, int* status, cudaStream_t s) {
+                             int vl, int window, int nsplit, float scale, int* status, cudaStream_t s) {
   if (rows <= 0 || nseg <= 0) return 0;
-  if (lat % 64 || lat > 512 || kv_block % LM_KEYS) return -20;
-  if (nsplit < 1 || nsplit > 4096) return -1;
-  const int tps = (max_rows * heads + LM_M - 1) / LM_M;
+  if (lat % 64 || lat > 576 || vl != (lat <= 512 ? lat : 512) || kv_block % LM_KEYS) return -20;
+  if (nsplit < 1 || nsplit > 4096 || window < 0) return -1;
+  const int m_tile = lat <= 512 ? 64 : 32, tps = (max_rows * heads + m_tile - 1) / m_tile;
   const dim3 grid(nseg * tps, nsplit);
   const float sl = scale * 1.4426950408889634f;
   int rc = 0;
@@ -1060,13 +1150,13 @@ extern "C" int fb_latent_mma(void* out, float* o_part, float* ml_part, const voi
     if (e != cudaSuccess) return (int)e;                                                                                       \
     rc = (int)launch_pdl(kern, grid, dim3(LM_THREADS), Lm<NJ>::SMEM, s, (bf16*)out, o_part, ml_part, (const bf16*)q,           \
                          (const bf16*)cache, seg_slot, seg_row0, seg_nrows, row_kvlen, block_table, max_blocks, kv_block, heads, \
-                         row_base, tps, nsplit, sl, status);                                                                   \
+                         row_base, tps, nsplit, sl, window, status);                                                           \
     break;                                                                                                                     \
   }
-  switch (lat / 64) { FB_LM(1) FB_LM(2) FB_LM(3) FB_LM(4) FB_LM(5) FB_LM(6) FB_LM(7) FB_LM(8) }
+  switch (lat / 64) { FB_LM(1) FB_LM(2) FB_LM(3) FB_LM(4) FB_LM(5) FB_LM(6) FB_LM(7) FB_LM(8) FB_LM(9) }
 #undef FB_LM
   if (rc || nsplit == 1) return rc;
-  return latent_merge<bf16>(out, (long)heads * lat, o_part, ml_part, nullptr, rows, heads, nsplit, lat, s);
+  return latent_merge<bf16>(out, (long)heads * vl, o_part, ml_part, nullptr, rows, heads, nsplit, vl, s);
 }
 
 // y [batch][M][N] = act(x [batch][M][K] w [batch][N][K]^T); row strides ldx / ldy, batch strides x_bs / w_bs / y_bs (elements)

@@ -24,6 +24,7 @@ __global__ void __launch_bounds__(32) route_kernel(int* __restrict__ ids, float*
                                                    float scale, int ld, int shared_col, int shared_id, int lane_groups) {
   pdl_launch_dependents();
   pdl_wait();
+  logits = after_wait(logits);
   const int row = blockIdx.x, lane = threadIdx.x;
   const float* lp = logits + (size_t)row * ld;
   // `shared_id` >= 0: the always-on shared expert rides along as pick number top_k (expert id shared_id of the stack),
@@ -151,6 +152,7 @@ moe_gate_up_kernel(__nv_bfloat16* __restrict__ act, const __nv_bfloat16* __restr
   pdl_launch_dependents();
   extern __shared__ __align__(16) __nv_bfloat16 xs_moe[];
   pdl_wait();                                                // ids come from the router kernel before this one
+  ids = after_wait(ids); x = after_wait(x);
   const int p = blockIdx.y, e = ids[p];
   const bool shared = sh.w_gu && e == sh.id;
   if (!shared && (e < e_lo || e >= e_hi)) return;            // another rank owns this expert
@@ -204,6 +206,7 @@ moe_down_kernel(float* __restrict__ yp, const __nv_bfloat16* __restrict__ act, c
   pdl_launch_dependents();
   extern __shared__ __align__(16) __nv_bfloat16 as_moe[];
   pdl_wait();
+  ids = after_wait(ids); act = after_wait(act);
   const int p = blockIdx.y, e = ids[p];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n0 = blockIdx.x * 16 + warp * 2;
@@ -247,6 +250,7 @@ __global__ void __launch_bounds__(256) expert_f32_kernel(float* __restrict__ out
                                                          float limit, const SharedExpert sh) {
   pdl_launch_dependents();
   pdl_wait();
+  ids = after_wait(ids); x = after_wait(x);
   const int p = p0 + blockIdx.y, e = ids[p], lane = threadIdx.x & 31;
   const int j = blockIdx.x * 8 + (threadIdx.x >> 5);
   const bool shared = sh.w_gu && e == sh.id;

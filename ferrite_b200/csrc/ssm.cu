@@ -33,6 +33,7 @@ __global__ void __launch_bounds__(SS_THREADS) ssm_step_kernel(float* __restrict_
   const int g = h / (heads / groups), inner = heads * V, ch = inner + 2 * groups * N, vals = SS_COLS + 2 * N;
   const float a_h = A[h], db = dt_bias[h], sk = skip[h];
   pdl_wait();
+  proj = after_wait(proj); tails = after_wait(tails);
   const int slot = seg_slot[blockIdx.x], row0 = seg_row0[blockIdx.x], n = seg_nrows[blockIdx.x];
   if (n <= 0) return;
   const int q = tid & 3, ng = tid >> 2, v = v0 + 4 * q;      // this thread's columns v .. v + 3, rows ng, ng + 32, ...
@@ -123,6 +124,7 @@ __global__ void __launch_bounds__(256) group_norm_gated_kernel(T* __restrict__ o
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
+  y = after_wait(y); proj = after_wait(proj);
   const size_t row = blockIdx.x;
   const int part = blockIdx.y, size = inner / parts, c0 = part * size;
   float ss = 0.f;

@@ -72,6 +72,7 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
   float* wt = reinterpret_cast<float*>(sX + SD_Q * SD_LDX);  // [64]
   pdl_launch_dependents();
   pdl_wait();
+  xbc = after_wait(xbc); proj = after_wait(proj);
   const int c = blockIdx.x, h = blockIdx.y / d.VT, v0 = blockIdx.y % d.VT * SD_V, seg = blockIdx.z;
   const int n = seg_nrows[seg] - c * SD_Q;
   if (n <= 0) return;
@@ -157,6 +158,7 @@ __global__ void __launch_bounds__(256) ssd_scan_kernel(float* __restrict__ state
                                                        const int* __restrict__ seg_slot, const int* __restrict__ seg_nrows, SdDims d, int chunks) {
   pdl_launch_dependents();
   pdl_wait();
+  ends = after_wait(ends);
   const int i = blockIdx.x * 256 + threadIdx.x, h = blockIdx.y, seg = blockIdx.z, size = d.N * d.V;
   const int nc = (seg_nrows[seg] + SD_Q - 1) / SD_Q;
   if (i >= size || nc <= 0) return;
@@ -193,6 +195,7 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
   float4* info = reinterpret_cast<float4*>(sS + 2 * d.NP * SD_LDX);      // [64]
   pdl_launch_dependents();
   pdl_wait();
+  states = after_wait(states); rowinfo = after_wait(rowinfo); xbc = after_wait(xbc);
   const int c = blockIdx.x, h = blockIdx.y / d.VT, v0 = blockIdx.y % d.VT * SD_V, seg = blockIdx.z;
   const int n = seg_nrows[seg] - c * SD_Q;
   if (n <= 0) return;

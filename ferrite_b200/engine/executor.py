@@ -1133,7 +1133,8 @@ class Executor:
             mixer = c.layers[run.layer].mixer
             if mixer in ("cdelta", "ssm"):
                 proj = self.verify_proj[run.index]
-                (self._cdelta if mixer == "cdelta" else self._ssm)(proj, run, mv, [SegGroup(0, mv["sslot"].numel(), 0, proj.shape[0], mr)], True)
+                # (a segment may keep none of its rows, so the tails move on by the counts: never the form of one row per segment)
+                (self._cdelta if mixer == "cdelta" else self._ssm)(proj, run, mv, [SegGroup(0, mv["sslot"].numel(), 0, proj.shape[0], max(mr, 2))], True)
         for at, j in self.canon_at.items():
             ops.conv_tail(self.conv_state["canon"][:, j], self.verify_proj[at], mv["sslot"], mv["srow0"], mv["snrows"])
         for i, kind in enumerate(self.kinds):

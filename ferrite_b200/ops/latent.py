@@ -236,9 +236,10 @@ class TorchLatent:
 
 
 class CudaLatent:
-    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur, out=None):
-        x = self.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=self.device)
-        xb = out if out is not None else None if self.dtype == torch.float32 else self.empty(*x.shape, dtype=self.dtype, device=self.device)
+    def embed_grams(self, table, grams, ids, row_slot, row_pos, block_table, tok_pages, kv_block, scale, buckets, mul_prev, mul_cur, out=None,
+                    x=None):
+        own, x = x, x if x is not None else self.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=self.device)
+        xb = out if out is not None else None if self.dtype == torch.float32 or own is not None else self.empty(*x.shape, dtype=self.dtype, device=self.device)
         self.launches += 1
         self.C.embed_grams(x, xb, table, grams, ids, row_slot, row_pos, block_table, kv_block, tok_pages, scale, buckets, mul_prev, mul_cur,
                            self.status_word)
@@ -252,11 +253,46 @@ class CudaLatent:
         self.C.add_normed(x, xb, y, w, width, eps, bias, next_w)
         return x if xb is None else xb
 
-    def norm_rows(self, x, idx, w, width, eps, bias=None):
+    def norm_rows(self, x, idx, w, width, eps, bias=None, mean=False):
         out = self.empty(x.shape[0] if idx is None else idx.numel(), x.shape[1], dtype=self.dtype, device=self.device)
         self.launches += 1
-        self.C.norm_rows(out, x, idx, w, bias, width, eps)
+        self.C.norm_rows(out, x, idx, w, bias, width, eps, mean)
         return out
+
+    def add_conv_normed(self, x_in, x, y, w, width, eps, next_w, pairs=None, average=None, conv=None, row_slot=None, row_pos=None, single=False,
+                        commit=True):
+        """One pass over the rows; the convolution rides on it where every segment is one row (`single`), else it is a pass of its own."""
+        rows, f32 = x.shape, self.dtype == torch.float32
+        fused = conv is not None and single
+        h = out = None
+        if next_w is not None and not (fused and commit):
+            h = self.empty(*rows, dtype=self.dtype, device=self.device)
+        if fused:
+            out = self.empty(*rows, dtype=self.dtype, device=self.device)
+        xs, place, dwa = average or (None, 0, None)
+        self.launches += 1
+        self.C.add_conv_normed(x_in, x, y, *(pairs or (None, None)), w, xs, place, dwa, next_w, h, out, *(conv if fused else (None, None)),
+                               row_slot if fused else None, commit, width, eps, f32)
+        if conv is not None and not fused:
+            out = self.conv_rows(h, conv[0], conv[1], row_slot, row_pos, residual=True)
+        return (h if conv is None else out), h
+
+    def conv_rows(self, x, w, tails, row_slot, row_pos, bias=None, silu=False, residual=False):
+        out = self.empty(*x.shape, dtype=self.dtype, device=self.device)
+        self.launches += 1
+        self.C.conv_rows(out, x, w, tails, row_slot, row_pos, bias, silu, residual)
+        return out
+
+    def conv_tail(self, tails, x, seg_slot, seg_row0, seg_nrows):
+        self.launches += 1
+        self.C.conv_tail(tails, x, seg_slot, seg_row0, seg_nrows)
+
+    def latent_rot_prep(self, proj, d, kv_norm, inv_freq, row_slot, row_pos, block_table, cache, kv_block, eps):
+        q = self.empty(proj.shape[0], d.heads, d.hp, dtype=self.dtype, device=self.device)
+        self.launches += 1
+        self.C.latent_rot_prep(q, cache, proj, kv_norm, inv_freq, row_slot, row_pos, block_table, kv_block, d.dim, d.rot, d.kv_rank, eps,
+                               self.status_word)
+        return q
 
     def add_layer_norm(self, x, y, width, eps, next_w=None, next_b=None, pairs=None):
         xb = None if next_w is None else self.empty(*x.shape, dtype=self.dtype, device=self.device)
@@ -271,25 +307,29 @@ class CudaLatent:
                            self.status_word)
         return cq
 
-    def latent_attention(self, qabs, cache, group, row_slot, row_kvlen, segs, block_table, kv_block, scale, nsplit=1):
+    def latent_attention(self, qabs, cache, group, row_slot, row_kvlen, segs, block_table, kv_block, scale, nsplit=1, vlat=0, window=0):
         """Rows of one slot form a segment (`segs` = slots, first rows, row counts), so its rows and heads share every pass over
-        the latents on the tensor cores; fp32 and latents wider than 512 take the CUDA-core kernel. `nsplit` bounds the key
-        splits; what is left of it is what fills the GPU."""
+        the latents on the tensor cores; fp32 and cache rows wider than 576 take the CUDA-core kernel. `nsplit` bounds the key
+        splits; what is left of it is what fills the GPU and what the window leaves of the keys."""
         rows, heads, lat = qabs.shape
-        mma = qabs.dtype == torch.bfloat16 and lat <= 512
-        ctas = rows * heads if not mma else max(1, (group.seg_hi - group.seg_lo) * ((group.max_rows * heads + 63) // 64))
+        vlat = vlat or lat
+        mma = qabs.dtype == torch.bfloat16 and (lat <= 512 or (lat == 576 and vlat == 512)) and kv_block % 64 == 0
+        tile = 64 if lat <= 512 else 32
+        ctas = rows * heads if not mma else max(1, (group.seg_hi - group.seg_lo) * ((group.max_rows * heads + tile - 1) // tile))
         per_sm = 8 if not mma else 2 if lat <= 192 else 1          # CTAs; a tile of wide latents fills an SM's shared memory
         nsplit = max(1, min(nsplit, per_sm * self.sm_count // ctas))
-        out = self.empty(rows, heads, lat, dtype=qabs.dtype, device=self.device)
+        if window:
+            nsplit = min(nsplit, -(-(window + group.max_rows) // 64) + 1)
+        out = self.empty(rows, heads, vlat, dtype=qabs.dtype, device=self.device)
         o_part = ml_part = None
         if nsplit > 1:
-            o_part = self.empty(rows * heads * nsplit * lat, dtype=torch.float32, device=self.device)
+            o_part = self.empty(rows * heads * nsplit * vlat, dtype=torch.float32, device=self.device)
             ml_part = self.empty(rows * heads * nsplit * 2, dtype=torch.float32, device=self.device)
         self.launches += 1 if nsplit == 1 else 2
         if mma and self.C.latent_mma(out, o_part, ml_part, qabs, cache, segs[0], segs[1], segs[2], group.max_rows, row_kvlen,
-                                     block_table, kv_block, group.row_lo, nsplit, scale, self.status_word) == 0:
+                                     block_table, kv_block, group.row_lo, nsplit, scale, self.status_word, window) == 0:
             return out
-        self.C.latent_attn(out, o_part, ml_part, qabs, cache, row_slot, row_kvlen, block_table, kv_block, nsplit, scale, self.status_word)
+        self.C.latent_attn(out, o_part, ml_part, qabs, cache, row_slot, row_kvlen, block_table, kv_block, nsplit, scale, self.status_word, window)
         return out
 
     def latent_rows(self, cache, group, kv_block, window=0):
@@ -314,6 +354,15 @@ class CudaLatent:
         self.launches += 1
         self.C.softcap(logits, cap)
         return logits
+
+    def glu(self, x, w, limit):
+        """Clamped gated units of x w^T, w = [gate rows | up rows], more rows than the row kernels take."""
+        M, N = x.shape[0], w.shape[0] // 2
+        y = self.empty(M, N, dtype=self.dtype, device=self.device)
+        assert self.dtype == torch.bfloat16 and N % 8 == 0 and M > 64, "glu: prompt rows in bf16"
+        self.launches += 1
+        self.C.gemm_glu(y, x, w, limit, 1, None, None, self.status_word)
+        return y
 
     def silu_mul_f32(self, gu, out=None):
         y = out if out is not None else self.empty(gu.shape[0], gu.shape[1] // 2, dtype=torch.float32, device=self.device)

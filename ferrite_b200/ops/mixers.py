@@ -175,15 +175,31 @@ class CudaMixers:
         self.launches += 1
         if not d.plain:
             assert bias is None and not d.qk_norm, "row norms and two maps: no biases, no norms per head"
-            self.C.gqa_row_prep(q, k_cache, v_cache, proj, *(norms or (None, None)), inv_freq, row_slot, row_pos, block_table, kv_block,
-                                [d.heads, d.maps, d.dim, d.vw, d.rot_dims, d.v_off], eps, self.status_word)
+            caches = (k_cache, v_cache) if d.source < 0 else (None, None)
+            self.C.gqa_row_prep(q, *caches, proj, *(norms or (None, None)), inv_freq, row_slot, row_pos, block_table, kv_block,
+                                [d.heads, d.maps, d.dim, d.vw, d.rot_dims, d.v_off, int(d.rot_half)], eps, self.status_word)
             return q
+        assert d.source < 0, "keys of another layer: row norms only"
         self.C.gqa_prep(q, k_cache, v_cache, proj, bias, inv_freq, row_slot, row_pos, block_table, kv_block, d.dim, d.rot_dims, d.v_off,
                         d.qk_norm, eps, self.status_word)
         return q
 
+    def pool_keys(self, d, k_cache, v_cache, pooled, seg_slot, seg_pos0, seg_nrows, max_rows, block_table, kv_block):
+        self.launches += 1
+        self.C.pool_keys(*pooled, k_cache, v_cache, seg_slot, seg_pos0, seg_nrows, max_rows, block_table, kv_block, d.pool, self.status_word)
+
+    def _pooled_rows(self, d, pooled, group, seg_slot, block_table, kv_block):
+        """Means of the blocks that a prompt group's rows see, side by side: (keys, values, first row of every segment)."""
+        count, start = group.pooled(d.window, d.pool)
+        tables = torch.tensor([start[:-1], count], dtype=torch.int32).pin_memory().to(self.device, non_blocking=True)
+        k, v = (self.empty(max(64, start[-1]), d.kv_heads, d.hp, dtype=self.dtype, device=self.device) for _ in "kv")
+        if start[-1]:
+            self.launches += 1
+            self.C.pool_gather(k[:start[-1]], v[:start[-1]], *pooled, seg_slot, tables[0], tables[1], block_table, kv_block, d.pool, self.status_word)
+        return k, v, tables[0]
+
     def gqa_attention(self, q, d, k_cache, v_cache, sink, group, row_slot, row_kvlen, segs, block_table, kv_block, nsplit, out, lam=None,
-                      gate=None, eps=0.0):
+                      gate=None, eps=0.0, pooled=None):
         """Prompt groups go to the tcgen05 flash kernel (softmax weights as value + remainder); the others are split over their keys on
         the mma.sync kernels, over the warps of a CTA as well where a segment brings at most 16 (row, head) pairs per key head. 32-bit runs, heads wider than 256 and pages off the 64 grid take the CUDA-core kernel. `nsplit` bounds the
         key splits; what is left of it is what fills the GPU and what the layer's mask leaves of the keys. The difference of two maps and
@@ -194,6 +210,10 @@ class CudaMixers:
         mix = (lam, None if gate is None else gate[a:b], 1.0 - d.diff, d.maps, d.vw, eps)
         tc = self.dtype == torch.bfloat16 and d.hp in (64, 128, 256)
         if group.prompt and tc and kv_block % 64 == 0:
+            if d.pool:
+                assert not mixed and sink is None, "pooled windows: single maps without gates and sinks"
+                k, v, start = self._pooled_rows(d, pooled, group, segs[0], block_table, kv_block)
+                bounds.update(k_mean=k, v_mean=v, mean_start=start, pool=d.pool)
             self.launches += 1
             flat = q.view(q.shape[0], -1)
             if d.maps == 2:                                           # both maps of a head in one CTA, which joins them
@@ -213,8 +233,14 @@ class CudaMixers:
             return out
         group_heads = nq // d.kv_heads
         mma = tc and group_heads <= 64
-        keys = mma and d.hp <= 128 and group.max_rows * group_heads <= 16 and kv_block % 64 == 0
-        per_group = max(1, 64 // max(1, group_heads))
+        keys = mma and d.hp <= 128 and (1 if d.pool else group.max_rows) * group_heads <= 16 and kv_block % 64 == 0
+        per_group = max(1, (16 if d.pool else 64) // max(1, group_heads))
+        if d.pool:
+            assert not mixed and sink is None, "pooled windows: single maps without gates and sinks"
+            mma = keys
+            bounds.update(k_mean=pooled[0], v_mean=pooled[1], pool=d.pool)
+            seen = block_table.shape[1] * kv_block if nsplit >= 64 else nsplit * 64      # context that nsplit stands for
+            nsplit = min(nsplit, -(-(d.window + group.max_rows) // 64) + 2 + -(-seen // (64 * d.pool)))
         ctas = (group.seg_hi - group.seg_lo) * -(-group.max_rows // per_group) * d.kv_heads if mma else (b - a) * nq
         nsplit = max(1, min(nsplit, ((3 if d.hp == 128 else 5) if keys else 4 if mma else 8) * self.sm_count // max(1, ctas)))
         if d.reach:
@@ -227,14 +253,43 @@ class CudaMixers:
                         **(dict(zip(("lam", "gate", "mix_scale", "maps", "vdim", "eps"), mix)) if mixed else {}))
         return out
 
-    def expert_rows(self, h, ids, w_gu, w_down):
+    def expert_rows(self, h, ids, w_gu, w_down, limit=0.0, shared=None):
         """One row of the expert's feed-forward per (token, pick)."""
         pairs = ids.numel()
-        act = self.empty(pairs, w_down.shape[2], dtype=self.dtype, device=self.device)
+        sgu, sdn, slim = (shared[0][0], shared[1][0], shared[2]) if shared is not None else (None, None, 0.0)
+        act = self.empty(pairs, max(w_down.shape[2], 0 if sdn is None else sdn.shape[1]), dtype=self.dtype, device=self.device)
         yp = self.empty(pairs, h.shape[1], dtype=torch.float32, device=self.device)
         self.launches += 2
-        self.C.expert_rows(yp, act, h, w_gu, w_down, ids)
+        self.C.expert_rows(yp, act, h, w_gu, w_down, ids, limit, sgu, sdn, slim)
         return yp
+
+    def ssm(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, row_slot, row_pos, eps, commit=True):
+        """Few rows: one launch per group from the projection to the heads' outputs. Prompt groups: convolutions, then the chunked form. The
+        gated norm is one launch over all rows; with one row per segment it also moves the convolution's tails on."""
+        T = proj.shape[0]
+        sizes = [d.heads, d.groups, d.state, d.vdim, d.conv]
+        y = self.empty(T, d.inner, dtype=torch.float32, device=self.device)
+        out = self.empty(T, d.ko, dtype=self.dtype, device=self.device)
+        par = (w["A"], w["dt_bias"], w["skip"])
+        xbc = proj[:, d.inner:d.dt_off]
+        conv = None
+        for g in groups:
+            segs = tuple(t[g.seg_lo:g.seg_hi] for t in (seg_slot, seg_row0, seg_nrows))
+            if g.prompt and commit and self.dtype == torch.bfloat16 and d.state <= 256:
+                if conv is None:
+                    conv = self.conv_rows(xbc, w["conv"], conv_state, row_slot, row_pos, bias=w["conv_bias"], silu=True)
+                nb = self.C.ssd_chunk_scratch_bytes(T, g.seg_hi - g.seg_lo, g.max_rows, d.heads, d.state, d.vdim)
+                self.launches += 3
+                self.C.ssd_chunk(y, rec_state, self.scratch("ssd_chunk", nb // 4, torch.float32), conv, proj, *par, *segs, g.max_rows, sizes)
+            else:
+                self.launches += 1
+                self.C.ssm_step(y, rec_state, conv_state, proj, w["conv"], w["conv_bias"], *par, *segs, sizes, commit)
+        single = commit and d.conv > 1 and all(g.max_rows == 1 for g in groups) and seg_slot.numel() == T
+        self.launches += 1
+        self.C.group_norm_gated(out, y, proj, w["gnorm_w"], d.norm_groups, eps, conv_state if single else None, row_slot if single else None)
+        if commit and not single:
+            self.conv_tail(conv_state, xbc, seg_slot, seg_row0, seg_nrows)
+        return out
 
     def cdelta(self, proj, d, w, rec_state, conv_state, groups, seg_slot, seg_row0, seg_nrows, eps, commit=True):
         """A few rows: both low-rank products in one launch, then one launch per group for the whole mixer. Prompt groups: two GEMMs,

@@ -54,9 +54,10 @@ class ExpertParallel:
             raise RuntimeError(f"expert-parallel rank {self.rank}: status {int(self.status.item())} "
                                "(2 = a peer wait ran out, 5 = receive buffer capacity exceeded)")
 
-    def moe(self, ops, h, ids, wts, w_gu, w_down, shared=None, shared_gate=None, res=None, acc=None):
+    def moe(self, ops, h, ids, wts, w_gu, w_down, shared=None, shared_gate=None, res=None, acc=None, add=True, limit=0.0):
         """out[t] = res[t] + shared[t] * sigmoid(shared_gate[t]) + sum_k wts[t, k] * expert_{ids[t, k]}(h[t]) for this
-        rank's token rows; w_gu / w_down hold the experts this rank owns. `acc` (fp32 rows): the experts' sum is added to it instead."""
+        rank's token rows; w_gu / w_down hold the experts this rank owns. `acc` (fp32 rows): the sum is added to it, or with `add` off
+        written to it, instead. `limit`: the experts are clamped gated units."""
         self.calls += 1
         T, K = ids.shape
         inter = w_down.shape[2]
@@ -68,9 +69,11 @@ class ExpertParallel:
             if self._plan is None or self._plan.numel() < need:
                 self._plan = torch.empty(max(need, 4096), dtype=torch.int32, device=self.device)
             out = acc if acc is not None else torch.empty(T, self.hidden, dtype=h.dtype, device=self.device)
-            sg = None if shared_gate is None else shared_gate.reshape(-1).float().contiguous()
+            sg = shared_gate
+            if sg is not None and (sg.dim() != 1 or sg.dtype != torch.float32):
+                sg = sg.reshape(-1).float().contiguous()
             self.C.ep_moe(self.handle, out, h.contiguous(), ids.contiguous(), wts.contiguous(), w_gu, w_down, shared, sg,
-                          res, self._act, self._plan)
+                          res, self._act, self._plan, limit, add)
             ops.launches += 7
             return out
         # process-group statement of the same block
