@@ -514,7 +514,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     sub = ap.add_subparsers(dest="cmd", required=True)
 
     def common(p, max_tokens: int):
-        p.add_argument("--preset", default="tiny", help="tiny | tiny-mla | tiny-zototar | tiny-dofunex | tiny-rakizen | 27b | moe80b | mla671b | zototar-7b | dofunex-7b | rakizen-7b | drafter")
+        p.add_argument("--preset", default="tiny", help="tiny | tiny-mla | tiny-zototar | tiny-dofunex | tiny-rakizen | tiny-pironex | 27b | moe80b | mla671b | zototar-7b | dofunex-7b | rakizen-7b | pironex-moe | drafter")
         p.add_argument("--model", default="", help="checkpoint directory (config.json + safetensors, or a .gguf)")
         p.add_argument("--layers", type=int, default=0)
         p.add_argument("--weights", default="bf16")

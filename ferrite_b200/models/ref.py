@@ -194,8 +194,10 @@ class RefModel:
         return w[p + "out_proj"] @ o.reshape(-1)
 
     def _latent(self, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
-        """Position-free latent attention; a layer with `kv_from` reads the rows that layer appended for this token."""
+        """Latent attention; a layer with `kv_from` reads the rows that layer appended for this token."""
         l, w, p, eps = self.cfg.layers[i], self.w, f"l{i}.", self.cfg.eps
+        if not l.q_rank:
+            return self._latent_rotated(i, x, st)
         q = (w[p + "q_b"] @ rmsnorm(w[p + "q_a"] @ x, w[p + "q_a_norm"], eps, False)).view(l.heads, l.dim)
         if l.kv_from is None:
             st.k[i].append(rmsnorm(w[p + "kv_a"] @ x, w[p + "kv_a_norm"], eps, False))
@@ -205,27 +207,68 @@ class RefModel:
         pr = torch.softmax(torch.einsum("hd,thd->ht", q, k) * l.scale, -1)
         return w[p + "out_proj"] @ torch.einsum("ht,thv->hv", pr, v).reshape(-1)
 
-    def _gqa(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
-        """Grouped-query attention of listed layers; run r's keys and values are its own."""
+    def _latent_rotated(self, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """Latent attention under a window with one rotated key part for all heads beside the latent."""
+        l, w, p, R = self.cfg.layers[i], self.w, f"l{i}.", self.cfg.layers[i].rot_dims
+        ang = st.pos * rope_frequencies(l)
+        c, s = ang.cos().float(), ang.sin().float()
+        turned = lambda z: torch.stack([z[..., 0::2] * c - z[..., 1::2] * s, z[..., 1::2] * c + z[..., 0::2] * s], -1).flatten(-2)
+        q, kva = (w[p + "q"] @ x).view(l.heads, l.dim + R), w[p + "kv_a"] @ x
+        st.k[i].append(rmsnorm(kva[:l.kv_rank], w[p + "kv_a_norm"], self.cfg.eps, False))
+        st.v[i].append(turned(kva[l.kv_rank:]))
+        first = max(0, st.pos - l.window + 1) if l.window else 0
+        lat, kr = torch.stack(st.k[i][first:]), torch.stack(st.v[i][first:])
+        k, v = (lat @ w[p + "k_b"].t()).view(-1, l.heads, l.dim), (lat @ w[p + "v_b"].t()).view(-1, l.heads, l.vdim)
+        sc = torch.einsum("hd,thd->ht", q[:, :l.dim], k) + torch.einsum("hd,td->ht", turned(q[:, l.dim:]), kr)
+        return w[p + "out_proj"] @ torch.einsum("ht,thv->hv", torch.softmax(sc * l.scale, -1), v).reshape(-1)
+
+    def _ssm(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """State-space recurrence with one decay per head; run r's state and convolution inputs are its own."""
         l, w, p = self.cfg.layers[i], self.w, f"l{i}."
-        proj = {n: w[p + n] @ x + (w[p + n + "_bias"] if l.bias else 0.0) for n in ("q", "k") + (() if l.key_values else ("v",))}
+        H, V, N, G = l.heads, l.vdim, l.dim, l.kv_heads
+        z, xbc, dt = torch.split(w[p + "in"] @ x, [H * V, H * V + 2 * G * N, H])
+        buf = st.run.setdefault(("xbc", r), [])
+        buf.append(xbc)
+        c = F.silu(sum(b * w[p + "xbc_conv"][:, l.conv - 1 - j] for j, b in enumerate(reversed(buf[-l.conv:]))) + w[p + "xbc_bias"])
+        xs, B, C = torch.split(c, [H * V, G * N, G * N])
+        own = torch.arange(H) // (H // G)
+        xs, B, C, dt = xs.view(H, V), B.view(G, N)[own], C.view(G, N)[own], softplus(dt + w[p + "dt_bias"])
+        S = st.run.get(("rec", r), torch.zeros(H, N, V)) * torch.exp(-torch.exp(w[p + "A_log"]) * dt)[:, None, None]
+        S = st.run["rec", r] = S + (dt[:, None] * B)[:, :, None] * xs[:, None, :]
+        y = (torch.einsum("hnv,hn->hv", S, C) + w[p + "skip"][:, None] * xs).reshape(-1) * F.silu(z)
+        y = (y.view(l.norm_groups, -1) * torch.rsqrt(y.view(l.norm_groups, -1).pow(2).mean(-1, keepdim=True) + self.cfg.eps)).reshape(-1)
+        return w[p + "out_proj"] @ (y * w[p + "gnorm_w"])
+
+    def _gqa(self, r: int, i: int, x: torch.Tensor, st: RefState) -> torch.Tensor:
+        """Grouped-query attention of listed layers; run r's keys and values are its own, or those of the layer it names."""
+        l, w, p = self.cfg.layers[i], self.w, f"l{i}."
+        own_kv = l.kv_from is None
+        proj = {n: w[p + n] @ x + (w[p + n + "_bias"] if l.bias else 0.0)
+                for n in ("q",) + (("k",) if own_kv else ()) + (("v",) if own_kv and not l.key_values else ())}
         if l.row_norm:
-            proj.update({n: rmsnorm(proj[n], w[p + n + "_norm"], self.cfg.eps, False) for n in "qk"})
+            proj.update({n: rmsnorm(proj[n], w[p + n + "_norm"], self.cfg.eps, False) for n in "qk" if n in proj})
         ang = st.pos * rope_frequencies(l)
         c, s = ang.cos().float(), ang.sin().float()
 
         def turned(z):
-            z = z.clone()
-            a, b = z[:, 0:l.rot_dims:2].clone(), z[:, 1:l.rot_dims:2].clone()
-            z[:, 0:l.rot_dims:2], z[:, 1:l.rot_dims:2] = a * c - b * s, b * c + a * s
+            z, half = z.clone(), l.rot_dims // 2
+            u, v = (slice(0, half), slice(half, l.rot_dims)) if l.rot_half else (slice(0, l.rot_dims, 2), slice(1, l.rot_dims, 2))
+            a, b = z[:, u].clone(), z[:, v].clone()
+            z[:, u], z[:, v] = a * c - b * s, b * c + a * s
             return z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + self.cfg.eps) if l.qk_norm else z
         H, M = l.heads, l.maps
-        q, k = turned(proj["q"].view(H * M, l.dim)), proj["k"].view(l.kv_heads * M, l.dim)
-        st.run.setdefault(("k", r), []).append(turned(k))
-        st.run.setdefault(("v", r), []).append(k if l.key_values else proj["v"].view(l.kv_heads, l.vdim))
+        q = turned(proj["q"].view(H * M, l.dim))
+        if own_kv:
+            k = proj["k"].view(l.kv_heads * M, l.dim)
+            st.run.setdefault(("k", r), []).append(turned(k))
+            st.run.setdefault(("v", r), []).append(k if l.key_values else proj["v"].view(l.kv_heads, l.vdim))
+        else:
+            r = max(x.index for x in self.cfg.layer_runs[:r] if x.layer == l.kv_from)
         own = torch.arange(H) // (H // l.kv_heads)
         first = max(0, st.pos - l.window + 1) if l.window else st.pos - st.pos % l.chunk if l.chunk else 0
-        K, V = torch.stack(st.run["k", r][first:]), torch.stack(st.run["v", r][first:])[:, own]
+        blocks = [slice(b * l.pool, (b + 1) * l.pool) for b in range(first // l.pool)] if l.pool else []
+        seen = lambda rows: torch.stack([torch.stack(rows[b]).mean(0) for b in blocks] + rows[first:])
+        K, V = seen(st.run["k", r]), seen(st.run["v", r])[:, own]
         maps = []
         for m in range(M):
             sc = torch.einsum("hd,thd->ht", q[m::M], K[:, m::M][:, own]) * l.scale
@@ -263,9 +306,48 @@ class RefModel:
     def _experts(self, i: int, h: torch.Tensor) -> torch.Tensor:
         """Routed feed-forward of listed layers."""
         l, w, p = self.cfg.layers[i], self.w, f"l{i}."
+        if l.act == "clamped_glu":
+            def expert(gate_up, down, limit):
+                g, u = (gate_up @ h).chunk(2)
+                g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+                return down @ (g * torch.sigmoid(1.702 * g) * (u + 1))
+            val, idx = torch.sort(w[p + "router"] @ h, descending=True, stable=True)
+            out = sum(g * expert(w[p + "experts_gate_up"][e], w[p + "experts_down"][e], l.limit)
+                      for e, g in zip(idx[:l.top].tolist(), torch.softmax(val[:l.top], -1)))
+            if l.shared_ff:
+                out = out + torch.sigmoid(w[p + "shared_gate"] @ h) * expert(w[p + "shared_gate_up"][0], w[p + "shared_down"][0], l.shared_limit)
+            return out
         rc = ModelConfig(router="sigmoid_group", top_k=l.top, n_groups=l.groups, topk_groups=l.keep_groups, route_scale=l.route_scale)
         idx, wt = route(rc, (w[p + "router"] @ h)[None], None)
         return sum(g * (w[p + "experts_down"][e] @ swiglu(w[p + "experts_gate_up"][e] @ h)) for e, g in zip(idx[0].tolist(), wt[0].tolist()))
+
+    def _token_conv(self, t: int, st: RefState, tap: list) -> torch.Tensor:
+        """One token through a model of layer norms, convolved operands and averages over depth: the row before the final norm."""
+        c, w = self.cfg, self.w
+        x = w["embed"][t] * c.embed_scale
+        xs = [x]
+        norm = lambda z, name: F.layer_norm(z, z.shape, w[name], None, c.eps)
+
+        def operand(name, conv, key):
+            h = norm(x, name)
+            if not c.canon:
+                return h
+            buf = st.run.setdefault(key, [])
+            buf.append(h)
+            return h + sum(b * w[conv][:, c.canon - 1 - j] for j, b in enumerate(reversed(buf[-c.canon:])))
+        for run in c.layer_runs:
+            i, l, p, r = run.layer, c.layers[run.layer], f"l{run.layer}.", run.index
+            h = operand(p + "pre_norm", p + "mix_canon", ("mix", r))
+            y = self._latent(i, h, st) if l.mixer == "latent" else (self._gqa if l.mixer == "gqa" else self._ssm)(r, i, h, st)
+            x = x + norm(y, p + "mix_norm")
+            if l.ff:
+                x = x + norm(self._experts(i, operand(p + "ffn_pre_norm", p + "ffn_canon", ("ffn", r))), p + "ffn_norm")
+            if c.depth_average:
+                xs.append(x)
+                x = sum(g * z for g, z in zip(w[p + "dwa"], xs))
+            if i in c.tap_layers:
+                tap.append(x.clone())
+        return x
 
     def _token_parallel(self, t: int, st: RefState, tap: list) -> torch.Tensor:
         """One token through a model of parallel blocks: the row before the final norm."""
@@ -332,10 +414,10 @@ class RefModel:
         for t in list(tokens):
             tap = []
             if c.layers:
-                x = (self._token_parallel if c.parallel else self._token_out_norm)(int(t), st, tap)
+                x = (self._token_parallel if c.parallel else self._token_conv if c.layer_norm else self._token_out_norm)(int(t), st, tap)
                 st.pos += 1
-                if c.parallel:
-                    y = head @ F.layer_norm(x, x.shape, w["final_norm"], w["final_norm_bias"], c.eps) * c.logit_scale
+                if c.parallel or c.layer_norm:
+                    y = head @ F.layer_norm(x, x.shape, w["final_norm"], w.get("final_norm_bias"), c.eps) * c.logit_scale
                 else:
                     y = head @ rmsnorm(x, w["final_norm"], c.eps, False) * c.logit_scale
                 logits.append(c.logit_softcap * torch.tanh(y / c.logit_softcap) if c.logit_softcap else y)

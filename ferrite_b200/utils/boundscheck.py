@@ -42,7 +42,7 @@ def _special(ex, op: str, param: str, bound: Dict[str, Any]) -> Optional[Tuple[i
     if op in ("moe_experts",) and param == "ids":
         return 0, max(1, ex.full_cfg.n_experts) + 1, "experts (+ the shared expert's stack entry)"
     if op == "expert_rows" and param == "ids":
-        return 0, int(bound["w_down"].shape[0]), "experts of the layer"
+        return 0, int(bound["w_down"].shape[0]) + (1 if bound.get("shared") is not None else 0), "experts of the layer"
     if param == "row_parent":
         return -1, 1 << 30, "tree rows"
     return None
