@@ -100,12 +100,12 @@ def main():
     ap.add_argument("--model", default="27b", choices=["27b", "moe80b", "mla671b"],
                     help="27b: the headline model. moe80b (80B-A3B hybrid MoE, fits one GPU with --dtype nvfp4) and mla671b "
                          "(needs --layers on one GPU) measure the same plain decode + 2K prefill on the MoE families")
-    ap.add_argument("--design", default="", choices=["", "zototar", "dofunex", "rakizen"],
+    ap.add_argument("--design", default="", choices=["", "zototar", "dofunex", "rakizen", "pironex"],
                     help="instead of the headline workload, prefill and decode throughput of a design of listed layers beside the closest "
                          "other model of equal size (random weights; zototar: the dense MLA model, dofunex: the dense Gated DeltaNet hybrid, "
-                         "rakizen: the sequential grouped-query attention model), "
+                         "rakizen: the sequential grouped-query attention model, pironex: the routed Gated DeltaNet hybrid), "
                          "at the sizes of --sizes; one JSON line")
-    ap.add_argument("--sizes", default="", help="with --design: sizes to measure (model widths; zototar 2k,4k,7k, dofunex 2k,4k,5k, rakizen 2k,4k,2k-moe)")
+    ap.add_argument("--sizes", default="", help="with --design: sizes to measure (model widths; zototar 2k,4k,7k, dofunex 2k,4k,5k, rakizen 2k,4k,2k-moe, pironex 1k,2k,4k)")
     ap.add_argument("--fused-layers", default="auto", choices=["auto", "on", "off"],
                     help="plain decode rows: one persistent kernel per layer (auto = when tensor parallel)")
     ap.add_argument("--no-extras", action="store_true", help="only the headline decode measurement and the 2K prefill")

@@ -16,98 +16,168 @@ namespace fb {
 
 using bf16 = __nv_bfloat16;
 
-// mean and 1 / deviation of a row of `width` true columns (zeros up to ld) that waits in shared memory
-__device__ __forceinline__ float2 cr_stats(const float* row, float sum, int width, int ld, float eps, float* red) {
-  const float mean = block_sum(sum, red) / (float)width;
-  float ss = 0.f;
-  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-    const float4 v = *reinterpret_cast<const float4*>(row + i);
-    const float d[4] = {v.x - mean, v.y - mean, v.z - mean, v.w - mean};
+// Count, mean and sum of squared deviations of a part of a row; parts are joined pairwise, so nothing cancels.
+struct RowStats { float n, mean, m2; };
+__device__ __forceinline__ RowStats cr_join(RowStats a, RowStats b) {
+  const float n = a.n + b.n, f = n > 0.f ? b.n / n : 0.f, d = b.mean - a.mean;
+  return {n, fmaf(d, f, a.mean), a.m2 + b.m2 + d * d * a.n * f};
+}
+__device__ __forceinline__ RowStats cr_warp(RowStats s) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-      if (i + e < width) ss = fmaf(d[e], d[e], ss);
+  for (int o = 16; o > 0; o >>= 1)
+    s = cr_join(s, {__shfl_xor_sync(0xffffffffu, s.n, o), __shfl_xor_sync(0xffffffffu, s.mean, o), __shfl_xor_sync(0xffffffffu, s.m2, o)});
+  return s;
+}
+// (mean, 1 / deviation) of the row whose columns i + e < width, i = 4 (threadIdx.x + k blockDim.x), the threads hold in v[k]
+template <int NV>
+__device__ __forceinline__ float2 cr_stats(const float4 (&v)[NV], int width, float eps, RowStats* red) {
+  RowStats s{0.f, 0.f, 0.f};
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int left = width - 4 * (threadIdx.x + k * blockDim.x);
+    const float c[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+    RowStats t{0.f, 0.f, 0.f};
+    if (left >= 4) {
+      t.n = 4.f;
+      t.mean = 0.25f * ((c[0] + c[1]) + (c[2] + c[3]));
+#pragma unroll
+      for (int e = 0; e < 4; ++e) t.m2 = fmaf(c[e] - t.mean, c[e] - t.mean, t.m2);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 3; ++e)
+        if (e < left) t = cr_join(t, {1.f, c[e], 0.f});
+    }
+    s = k == 0 ? t : cr_join(s, t);
   }
-  return make_float2(mean, 1.f / sqrtf(block_sum(ss, red) / (float)width + eps));
+  s = cr_warp(s);
+  const int lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  __syncthreads();
+  if (lane == 0) red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  s = cr_warp(lane < warps ? red[lane] : RowStats{0.f, 0.f, 0.f});
+  return make_float2(s.mean, 1.f / sqrtf(s.m2 / (float)width + eps));
 }
 
-template <typename T>
-__global__ void add_conv_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, const float* __restrict__ y, long ldy,
-                                       const float* __restrict__ yp, const float* __restrict__ wts, int top, const float* __restrict__ w,
-                                       float* __restrict__ xs, long xs_step, int place, const float* __restrict__ dwa,
-                                       const float* __restrict__ next_w, T* __restrict__ h_out, T* __restrict__ xb, const float* __restrict__ cw,
-                                       int taps, T* __restrict__ tails, long tail_step, const int* __restrict__ row_slot, int commit, int width,
-                                       int ld, float eps) {
-  extern __shared__ __align__(16) float cr_row[];
-  __shared__ float red[32];
+// NV: groups of four columns per thread, the whole row in registers. CONV: the convolution rides on the pass (one row per segment). What does
+// not come from the kernel before this one (weights) is read while that drains, what no norm has to wait for (results, tails) before the norms.
+constexpr int cn_threads(int nv) { return nv == 16 ? 1024 : 512; }
+
+template <typename T, int NV, bool CONV>
+__global__ void __launch_bounds__(cn_threads(NV), NV == 1 && !CONV ? 2 : 1)
+add_conv_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, const float* __restrict__ y, long ldy, const float* __restrict__ yp,
+                       const float* __restrict__ wts, int top, const float* __restrict__ w, float* __restrict__ xs, long xs_step, int place,
+                       const float* __restrict__ dwa, const float* __restrict__ next_w, T* __restrict__ h_out, T* __restrict__ xb,
+                       const float* __restrict__ cw, int taps, T* __restrict__ tails, long tail_step, const int* __restrict__ row_slot, int commit,
+                       int width, int ld, float eps) {
+  constexpr bool EARLY = NV == 1 && CONV;
+  constexpr int PART = 4;                                    // expert rows, results and taps read at a time
+  __shared__ RowStats red[32];
   pdl_launch_dependents();
+  const size_t row = blockIdx.x;
+  auto col = [&](int k) { return 4 * (threadIdx.x + k * (int)blockDim.x); };
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto load = [&](const float* p, int i) { return i < ld ? *reinterpret_cast<const float4*>(p + i) : zero; };
+  auto axpy = [](float4& a, float g, const float4& b) {
+    a.x = fmaf(g, b.x, a.x); a.y = fmaf(g, b.y, a.y); a.z = fmaf(g, b.z, a.z); a.w = fmaf(g, b.w, a.w);
+  };
+  float4 w_own = zero, next_own = zero, conv_own[EARLY ? PART : 1];
+  if (EARLY) {
+    if (w) w_own = load(w, col(0));
+    if (next_w) next_own = load(next_w, col(0));
+#pragma unroll
+    for (int j = 0; j < PART; ++j) conv_own[EARLY ? j : 0] = j < taps && taps <= PART ? load(cw + (size_t)j * ld, col(0)) : zero;
+  }
+  const float last = xs ? dwa[place] : 1.f;
+  const int slot = CONV ? row_slot[row] : 0;
   pdl_wait();
   x_in = after_wait(x_in); y = after_wait(y); yp = after_wait(yp); wts = after_wait(wts);
-  const size_t row = blockIdx.x;
-  const float* xi = x_in + row * ld;
-  float sum = 0.f;
+  float4 v[NV], f[NV], past[NV];
+  T* tail = CONV ? tails + slot * tail_step : nullptr;
+  float4 tail_own[EARLY ? PART - 1 : 1];
+  if (EARLY && next_w) {
+#pragma unroll
+    for (int j = 0; j < PART - 1; ++j)
+      tail_own[EARLY ? j : 0] = j + 1 < taps && taps <= PART && col(0) < ld ? Elem<T>::load4(tail + (size_t)j * ld + col(0)) : zero;
+  }
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = col(k);
+    v[k] = load(x_in + row * ld, i);
+    f[k] = w && y ? load(y + row * ldy, i) : zero;
+    past[k] = zero;
+    for (int p0 = 0; p0 < top; p0 += PART) {
+      float g[PART];
+      float4 e[PART];
+#pragma unroll
+      for (int j = 0; j < PART; ++j) {
+        const size_t r = row * top + p0 + j;
+        g[j] = p0 + j < top ? wts[r] : 0.f;
+        e[j] = p0 + j < top ? load(yp + r * ld, i) : zero;
+      }
+#pragma unroll
+      for (int j = 0; j < PART; ++j) axpy(f[k], g[j], e[j]);
+    }
+    if (xs && i < ld) {                                      // earlier results
+      const float* xr = xs + row * ld + i;
+      for (int j0 = 0; j0 < place; j0 += PART) {
+        float4 r[PART];
+#pragma unroll
+        for (int j = 0; j < PART; ++j) r[j] = j0 + j < place ? *reinterpret_cast<const float4*>(xr + (j0 + j) * xs_step) : zero;
+#pragma unroll
+        for (int j = 0; j < PART; ++j) axpy(past[k], j0 + j < place ? dwa[j0 + j] : 0.f, r[j]);
+      }
+    }
+  }
   if (w) {                                                   // the sublayer's output, its norm, the residual sum
-    for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-      float4 s = y ? *reinterpret_cast<const float4*>(y + row * ldy + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int k = 0; k < top; ++k) {
-        const float g = wts[row * top + k];
-        const float4 e = *reinterpret_cast<const float4*>(yp + (row * top + k) * ld + i);
-        s.x = fmaf(g, e.x, s.x); s.y = fmaf(g, e.y, s.y); s.z = fmaf(g, e.z, s.z); s.w = fmaf(g, e.w, s.w);
-      }
-      *reinterpret_cast<float4*>(cr_row + i) = s;
-      sum += (s.x + s.y) + (s.z + s.w);
-    }
-    const float2 st = cr_stats(cr_row, sum, width, ld, eps, red);
-    sum = 0.f;
-    const float last = xs ? dwa[place] : 1.f;
-    for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-      const float4 f = *reinterpret_cast<const float4*>(cr_row + i), ww = *reinterpret_cast<const float4*>(w + i);
-      float4 v = *reinterpret_cast<const float4*>(xi + i);
-      v.x += (f.x - st.x) * st.y * ww.x; v.y += (f.y - st.x) * st.y * ww.y;
-      v.z += (f.z - st.x) * st.y * ww.z; v.w += (f.w - st.x) * st.y * ww.w;
+    const float2 st = cr_stats<NV>(f, width, eps, red);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = col(k);
+      const float4 ww = EARLY ? w_own : load(w, i);
+      v[k].x += (f[k].x - st.x) * st.y * ww.x; v[k].y += (f[k].y - st.x) * st.y * ww.y;
+      v[k].z += (f[k].z - st.x) * st.y * ww.z; v[k].w += (f[k].w - st.x) * st.y * ww.w;
+      if (i >= ld) continue;
       if (xs) {                                              // this layer's result, then the sum over depth
-        *reinterpret_cast<float4*>(xs + place * xs_step + row * ld + i) = v;
-        v.x *= last; v.y *= last; v.z *= last; v.w *= last;
-#pragma unroll 4
-        for (int j = 0; j < place; ++j) {
-          const float g = dwa[j];
-          const float4 r = *reinterpret_cast<const float4*>(xs + j * xs_step + row * ld + i);
-          v.x = fmaf(g, r.x, v.x); v.y = fmaf(g, r.y, v.y); v.z = fmaf(g, r.z, v.z); v.w = fmaf(g, r.w, v.w);
-        }
+        *reinterpret_cast<float4*>(xs + place * xs_step + row * ld + i) = v[k];
+        axpy(past[k], last, v[k]);
+        v[k] = past[k];
       }
-      *reinterpret_cast<float4*>(x + row * ld + i) = v;
-      *reinterpret_cast<float4*>(cr_row + i) = v;
-      sum += (v.x + v.y) + (v.z + v.w);
-    }
-  } else {
-    for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-      const float4 v = *reinterpret_cast<const float4*>(xi + i);
-      *reinterpret_cast<float4*>(cr_row + i) = v;
-      sum += (v.x + v.y) + (v.z + v.w);
+      *reinterpret_cast<float4*>(x + row * ld + i) = v[k];
     }
   }
   if (!next_w) return;
-  const float2 st = cr_stats(cr_row, sum, width, ld, eps, red);
-  T* tail = xb ? tails + row_slot[row] * tail_step : nullptr;
-  for (int i = threadIdx.x * 4; i < ld; i += blockDim.x * 4) {
-    const float4 v = *reinterpret_cast<const float4*>(cr_row + i), ww = *reinterpret_cast<const float4*>(next_w + i);
-    T h4[4] = {Elem<T>::from((v.x - st.x) * st.y * ww.x), Elem<T>::from((v.y - st.x) * st.y * ww.y),
-               Elem<T>::from((v.z - st.x) * st.y * ww.z), Elem<T>::from((v.w - st.x) * st.y * ww.w)};
+  const float2 st = cr_stats<NV>(v, width, eps, red);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = col(k);
+    if (i >= ld) continue;
+    const float4 nw = EARLY ? next_own : load(next_w, i);
+    T h4[4] = {Elem<T>::from((v[k].x - st.x) * st.y * nw.x), Elem<T>::from((v[k].y - st.x) * st.y * nw.y),
+               Elem<T>::from((v[k].z - st.x) * st.y * nw.z), Elem<T>::from((v[k].w - st.x) * st.y * nw.w)};
     const float4 h = make_float4(Elem<T>::to(h4[0]), Elem<T>::to(h4[1]), Elem<T>::to(h4[2]), Elem<T>::to(h4[3]));
     if (h_out) Elem<T>::store4(h_out + row * ld + i, h);
-    if (!xb) continue;
-    const float4 c = *reinterpret_cast<const float4*>(cw + (size_t)(taps - 1) * ld + i);
-    float4 o = make_float4(fmaf(c.x, h.x, h.x), fmaf(c.y, h.y, h.y), fmaf(c.z, h.z, h.z), fmaf(c.w, h.w, h.w));
-    for (int j = 0; j + 1 < taps; ++j) {
-      const float4 p = Elem<T>::load4(tail + (size_t)j * ld + i), g = *reinterpret_cast<const float4*>(cw + (size_t)j * ld + i);
-      o.x = fmaf(g.x, p.x, o.x); o.y = fmaf(g.y, p.y, o.y); o.z = fmaf(g.z, p.z, o.z); o.w = fmaf(g.w, p.w, o.w);
-      if (commit && j > 0) Elem<T>::store4(tail + (size_t)(j - 1) * ld + i, p);
+    if constexpr (CONV) {
+      float4 o = h;
+      auto tap = [&](int j, const float4& c, const float4& p) {
+        o.x = fmaf(c.x, p.x, o.x); o.y = fmaf(c.y, p.y, o.y); o.z = fmaf(c.z, p.z, o.z); o.w = fmaf(c.w, p.w, o.w);
+        if (commit && j > 0) Elem<T>::store4(tail + (size_t)(j - 1) * ld + i, p);
+      };
+      if (EARLY && taps <= PART) {
+#pragma unroll
+        for (int j = 0; j < PART; ++j)
+          if (j < taps) tap(j, conv_own[EARLY ? j : 0], j + 1 < taps ? tail_own[EARLY && j < PART - 1 ? j : 0] : h);
+      } else {
+        for (int j = 0; j < taps; ++j) {
+          const float4 p = j + 1 < taps ? Elem<T>::load4(tail + (size_t)j * ld + i) : h;
+          tap(j, *reinterpret_cast<const float4*>(cw + (size_t)j * ld + i), p);
+        }
+      }
+      Elem<T>::store4(xb + row * ld + i, o);
     }
-    if (commit && taps > 1) Elem<T>::store4(tail + (size_t)(taps - 2) * ld + i, h);
-    Elem<T>::store4(xb + row * ld + i, o);
   }
 }
 
-// grid (column blocks, strips of CR_ROWS rows). A row's predecessors are those of the step while slot and position go on, the tail's beyond.
+// TAPS: taps known at compile time, 0 = any. grid (column blocks, strips of CR_ROWS rows). A row's predecessors are those of the step while slot and position go on, the tail's beyond.
 constexpr int CR_ROWS = 8;
 
 template <typename T, int VEC, int TAPS>
@@ -139,39 +209,69 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(T* __restrict__ out, lon
       v[0] = Elem<T>::to(*p);
     }
   };
-  float wt[TAPS ? TAPS : 1][VEC], bs[VEC];
-  if constexpr (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) wt[j][e] = w[(size_t)j * C + c0 + e];
-  }
+  float bs[VEC];
 #pragma unroll
   for (int e = 0; e < VEC; ++e) bs[e] = bias ? bias[c0 + e] : 0.f;
-  for (int i = 0; i < here; ++i) {
-    const int r = r0 + i, n = before[i];
-    float acc[VEC], cur[VEC];
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) acc[e] = bs[e];
-#pragma unroll
-    for (int j = 0; j < taps; ++j) {                         // tap j meets the row taps - 1 - j back
-      const int back = taps - 1 - j;
-      float v[VEC];
-      load(back <= n ? x + (size_t)(r - back) * ldx + c0 : tails + slots[i] * tail_step + (size_t)(taps - 1 - (back - n)) * C + c0, v);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(TAPS ? wt[TAPS ? j : 0][e] : w[(size_t)j * C + c0 + e], v[e], acc[e]);
-      if (back == 0) {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) cur[e] = v[e];
-      }
-    }
+  auto finish = [&](int r, float (&acc)[VEC], const float (&cur)[VEC]) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-      if (silu) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+      if (silu) acc[e] = acc[e] / (1.f + __expf(-acc[e]));
       if (residual) acc[e] += cur[e];
     }
     if constexpr (VEC == 4) Elem<T>::store4(out + (size_t)r * ldo + c0, make_float4(acc[0], acc[1], acc[2], acc[3]));
     else out[(size_t)r * ldo + c0] = Elem<T>::from(acc[0]);
+  };
+  if constexpr (TAPS > 0) {
+    // all rows of the strip and the TAPS - 1 before it are read at once, those of another segment or of a tail replaced where one starts
+    using Raw = std::conditional_t<VEC == 1, T, std::conditional_t<sizeof(T) == 4, float4, uint2>>;      // VEC values as they lie in memory
+    float wt[TAPS][VEC];
+    Raw in[TAPS - 1 + CR_ROWS];
+    auto fetch = [](const T* p) { return *reinterpret_cast<const Raw*>(p); };
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) wt[j][e] = w[(size_t)j * C + c0 + e];
+#pragma unroll
+    for (int j = 0; j < TAPS - 1 + CR_ROWS; ++j) {
+      const int r = r0 + j - (TAPS - 1);
+      if (r >= 0 && r < rows) in[j] = fetch(x + (size_t)r * ldx + c0);
+    }
+#pragma unroll
+    for (int i = 0; i < CR_ROWS; ++i) {
+      if (i >= here) break;
+      const int n = before[i];
+      if (n < TAPS - 1) {                                    // close behind a segment's start: the rows before it are the tail's
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int back = TAPS - 1 - j;
+          if (back > n) in[i + j] = fetch(tails + slots[i] * tail_step + (size_t)(TAPS - 1 - (back - n)) * C + c0);
+        }
+      }
+      float acc[VEC], cur[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = bs[e];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        load(reinterpret_cast<const T*>(&in[i + j]), cur);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wt[j][e], cur[e], acc[e]);
+      }
+      finish(r0 + i, acc, cur);
+    }
+  } else {
+    for (int i = 0; i < here; ++i) {
+      const int r = r0 + i, n = before[i];
+      float acc[VEC], cur[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = bs[e];
+      for (int j = 0; j < taps; ++j) {                       // tap j meets the row taps - 1 - j back
+        const int back = taps - 1 - j;
+        load(back <= n ? x + (size_t)(r - back) * ldx + c0 : tails + slots[i] * tail_step + (size_t)(taps - 1 - (back - n)) * C + c0, cur);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(w[(size_t)j * C + c0 + e], cur[e], acc[e]);
+      }
+      finish(r, acc, cur);
+    }
   }
 }
 
@@ -204,18 +304,21 @@ extern "C" int fb_add_conv_normed(const float* x_in, float* x, const float* y, l
   if (rows <= 0) return 0;
   if (ld % 4 || ldy % 4 || ld > 49152 || width < 1 || width > ld || (top && (!yp || !wts)) || (w && !y && !top) || (xs && (!dwa || !w || place < 0)) ||
       (next_w && !h_out && !xb) || (xb && (!cw || taps < 1 || !row_slot || (taps > 1 && (!tails || tail_step % 4))))) return -1;
-  const size_t smem = (size_t)ld * 4;
-  const dim3 g(rows), b(ld >= 4096 ? 512 : ld >= 1024 ? 256 : 128);
+  const int quads = ld / 4;
+  int nv = 1;
+  while (nv < 16 && quads > cn_threads(nv) * nv) nv *= 2;
+  if (quads > cn_threads(nv) * nv) return -1;
+  const dim3 g(rows), b(((quads + nv - 1) / nv + 31) / 32 * 32);
   auto go = [&](auto kern, auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    if (smem > 40 * 1024) {
-      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) return (int)e;
-    }
-    return (int)launch_pdl(kern, g, b, smem, s, x_in, x, y, ldy, yp, wts, top, w, xs, xs_step, place, dwa, next_w, (T*)h_out, (T*)xb, cw, taps,
+    return (int)launch_pdl(kern, g, b, 0, s, x_in, x, y, ldy, yp, wts, top, w, xs, xs_step, place, dwa, next_w, (T*)h_out, (T*)xb, cw, taps,
                            (T*)tails, tail_step, row_slot, commit, width, ld, eps);
   };
-  return f32 ? go(add_conv_normed_kernel<float>, (float*)0) : go(add_conv_normed_kernel<bf16>, (bf16*)0);
+#define FB_CN2(NV, CONV) (f32 ? go(add_conv_normed_kernel<float, NV, CONV>, (float*)0) : go(add_conv_normed_kernel<bf16, NV, CONV>, (bf16*)0))
+#define FB_CN(NV) (xb ? FB_CN2(NV, true) : FB_CN2(NV, false))
+  return nv == 1 ? FB_CN(1) : nv == 2 ? FB_CN(2) : nv == 4 ? FB_CN(4) : nv == 8 ? FB_CN(8) : FB_CN(16);
+#undef FB_CN
+#undef FB_CN2
 }
 
 // out [rows][C] (ldo elements apart) from x (ldx), w [taps][C]; bias: C floats or null

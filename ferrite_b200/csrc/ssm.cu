@@ -113,38 +113,58 @@ __global__ void __launch_bounds__(SS_THREADS) ssm_step_kernel(float* __restrict_
   }
 }
 
-// out = y * silu(z), each of `parts` equal parts of the row divided by its root mean square, times w; grid (rows, parts). With `tails` (one row
-// per segment) the row's inputs join its slot's tail as well: nobody reads the old one any more.
-template <typename T>
-__global__ void __launch_bounds__(256) group_norm_gated_kernel(T* __restrict__ out, long ldo, const float* __restrict__ y, long ldy,
-                                                               const T* __restrict__ proj, long ldp, const float* __restrict__ w, int inner, int parts,
-                                                               int ko, float eps, T* __restrict__ tails, long tail_step, int taps, int ch,
-                                                               const int* __restrict__ row_slot) {
-  extern __shared__ float gn_s[];
+// out = y * silu(z), each of `parts` equal parts of the row divided by its root mean square, times w; grid (rows, parts (+ tail blocks)). With
+// `tails` (one row per segment) CTAs behind the parts move the slot's tail on by the row's inputs: nobody reads the old one any more.
+// VEC: four columns at a time.
+constexpr int GN_THREADS = 256, GN_TAIL = 1024;              // channels of a tail per CTA
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(GN_THREADS) group_norm_gated_kernel(T* __restrict__ out, long ldo, const float* __restrict__ y, long ldy,
+                                                                      const T* __restrict__ proj, long ldp, const float* __restrict__ w, int inner,
+                                                                      int parts, int ko, float eps, T* __restrict__ tails, long tail_step, int taps,
+                                                                      int ch, const int* __restrict__ row_slot) {
+  extern __shared__ __align__(16) float gn_s[];
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   y = after_wait(y); proj = after_wait(proj);
   const size_t row = blockIdx.x;
   const int part = blockIdx.y, size = inner / parts, c0 = part * size;
+  if (part >= parts) {                                       // a piece of the tail
+    const int lo = (part - parts) * GN_TAIL, hi = min(ch, lo + GN_TAIL);
+    T* t = tails + row_slot[row] * tail_step;
+    for (int j0 = 0; j0 + 1 < taps; ++j0)
+#pragma unroll
+      for (int k = 0; k < GN_TAIL / GN_THREADS; ++k) {
+        const int c = lo + k * GN_THREADS + threadIdx.x;
+        if (c < hi) t[(size_t)j0 * ch + c] = j0 + 2 < taps ? t[(size_t)(j0 + 1) * ch + c] : proj[row * ldp + inner + c];
+      }
+    return;
+  }
   float ss = 0.f;
-  for (int i = threadIdx.x; i < size; i += blockDim.x) {
-    const float z = Elem<T>::to(proj[row * ldp + c0 + i]);
-    const float v = y[row * ldy + c0 + i] * (z / (1.f + __expf(-z)));
-    gn_s[i] = v;
-    ss = fmaf(v, v, ss);
+  for (int i = threadIdx.x * VEC; i < size; i += GN_THREADS * VEC) {
+    if constexpr (VEC == 4) {
+      const float4 z = Elem<T>::load4(proj + row * ldp + c0 + i), a = *reinterpret_cast<const float4*>(y + row * ldy + c0 + i);
+      const float4 v = make_float4(a.x * siluf_(z.x), a.y * siluf_(z.y), a.z * siluf_(z.z), a.w * siluf_(z.w));
+      *reinterpret_cast<float4*>(gn_s + i) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    } else {
+      const float v = y[row * ldy + c0 + i] * siluf_(Elem<T>::to(proj[row * ldp + c0 + i]));
+      gn_s[i] = v;
+      ss = fmaf(v, v, ss);
+    }
   }
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)size + eps);
-  for (int i = threadIdx.x; i < size; i += blockDim.x) out[row * ldo + c0 + i] = Elem<T>::from(gn_s[i] * r * w[c0 + i]);
-  if (part == parts - 1)
-    for (int i = inner + threadIdx.x; i < ko; i += blockDim.x) out[row * ldo + i] = Elem<T>::from(0.f);
-  if (!tails) return;
-  const int per = (ch + parts - 1) / parts, hi = min(ch, (part + 1) * per);
-  for (int c = part * per + threadIdx.x; c < hi; c += blockDim.x) {
-    T* t = tails + row_slot[row] * tail_step + c;
-    for (int j = 0; j + 2 < taps; ++j) t[(size_t)j * ch] = t[(size_t)(j + 1) * ch];
-    t[(size_t)(taps - 2) * ch] = proj[row * ldp + inner + c];
+  for (int i = threadIdx.x * VEC; i < size; i += GN_THREADS * VEC) {
+    if constexpr (VEC == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(gn_s + i), ww = *reinterpret_cast<const float4*>(w + c0 + i);
+      Elem<T>::store4(out + row * ldo + c0 + i, make_float4(v.x * r * ww.x, v.y * r * ww.y, v.z * r * ww.z, v.w * r * ww.w));
+    } else {
+      out[row * ldo + c0 + i] = Elem<T>::from(gn_s[i] * r * w[c0 + i]);
+    }
   }
+  if (part == parts - 1)
+    for (int i = inner + threadIdx.x; i < ko; i += GN_THREADS) out[row * ldo + i] = Elem<T>::from(0.f);
 }
 
 }  // namespace fb
@@ -177,15 +197,19 @@ extern "C" int fb_group_norm_gated(void* out, long ldo, const float* y, long ldy
                                    cudaStream_t s) {
   if (rows <= 0) return 0;
   if (parts < 1 || inner % parts || ko < inner || parts > 65535 || (long)inner / parts > 49152 || (tails && (taps < 2 || !row_slot))) return -1;
-  const size_t smem = (size_t)(inner / parts) * 4;
+  const int size = inner / parts, blocks = parts + (tails ? (ch + GN_TAIL - 1) / GN_TAIL : 0);
+  const size_t smem = (size_t)size * 4, item = f32 ? 4 : 2;
+  const bool vec = size % 4 == 0 && ldo % 4 == 0 && ldy % 4 == 0 && ldp % 4 == 0 && (((uintptr_t)y | (uintptr_t)w) & 15) == 0 &&
+                   (((uintptr_t)out | (uintptr_t)proj) & (4 * item - 1)) == 0;
   auto go = [&](auto kern, auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     if (smem > 40 * 1024) {
       const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
     }
-    return (int)launch_pdl(kern, dim3(rows, parts), dim3(inner / parts >= 512 ? 256 : 128), smem, s, (T*)out, ldo, y, ldy, (const T*)proj, ldp, w, inner,
+    return (int)launch_pdl(kern, dim3(rows, blocks), dim3(GN_THREADS), smem, s, (T*)out, ldo, y, ldy, (const T*)proj, ldp, w, inner,
                            parts, ko, eps, (T*)tails, tail_step, taps, ch, row_slot);
   };
-  return f32 ? go(group_norm_gated_kernel<float>, (float*)0) : go(group_norm_gated_kernel<bf16>, (bf16*)0);
+  if (vec) return f32 ? go(group_norm_gated_kernel<float, 4>, (float*)0) : go(group_norm_gated_kernel<bf16, 4>, (bf16*)0);
+  return f32 ? go(group_norm_gated_kernel<float, 1>, (float*)0) : go(group_norm_gated_kernel<bf16, 1>, (bf16*)0);
 }

@@ -18,7 +18,13 @@ namespace fb {
 
 using bf16 = __nv_bfloat16;
 
-constexpr int SD_Q = 64, SD_THREADS = 128, SD_V = 64, SD_LDX = SD_V + 8;
+constexpr int SD_Q = 64, SD_THREADS = 256, SD_V = 64, SD_LDX = SD_V + 8;
+
+__device__ __forceinline__ void sd_cp16(void* smem, const void* gmem, bool valid) {
+  const int sz = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem)), "l"(gmem), "r"(sz) : "memory");
+}
+__device__ __forceinline__ void sd_cp_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 __device__ __forceinline__ void sd_ldsm(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -39,15 +45,16 @@ struct SdDims {
   int inner, ch;
 };
 
-// rows x cols of a row-major source (ld elements apart) into smem rows of lds elements, zeros beyond; VEC: 8 elements at a time
+// rows x cols of a row-major source (ld elements apart) into smem rows of lds elements, zeros beyond; VEC: 8 elements at a time, without
+// waiting (sd_cp_wait does)
 template <bool VEC>
 __device__ __forceinline__ void sd_load(bf16* dst, int lds, const bf16* src, long ld, int rows, int cols, int cols_pad) {
   if (VEC) {
     const int per = cols_pad / 8;
     for (int i = threadIdx.x; i < SD_Q * per; i += SD_THREADS) {
       const int r = i / per, c = i % per * 8;
-      *reinterpret_cast<uint4*>(dst + r * lds + c) =
-          r < rows && c < cols ? *reinterpret_cast<const uint4*>(src + (size_t)r * ld + c) : make_uint4(0, 0, 0, 0);
+      const bool ok = r < rows && c < cols;
+      sd_cp16(dst + r * lds + c, src + (ok ? (size_t)r * ld + c : 0), ok);
     }
   } else {
     for (int i = threadIdx.x; i < SD_Q * cols_pad; i += SD_THREADS) {
@@ -77,6 +84,9 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
   const int n = seg_nrows[seg] - c * SD_Q;
   if (n <= 0) return;
   const int here = min(SD_Q, n), row0 = seg_row0[seg] + c * SD_Q, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bf16* rows = xbc + (size_t)row0 * d.ch;
+  sd_load<VEC>(sX, SD_LDX, rows + h * d.V + v0, d.ch, here, min(SD_V, d.V - v0), SD_V);
+  sd_load<VEC>(sH, LDN, rows + d.inner + h / (d.heads / d.groups) * d.N, d.ch, here, d.N, d.NP);
   if (warp == 0) {
     float dt[2];
     double a[2];
@@ -107,9 +117,7 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
     }
     if (v0 == 0 && lane == 0) ends[((size_t)seg * chunks + c) * d.heads + h] = expf((float)end);
   }
-  const bf16* rows = xbc + (size_t)row0 * d.ch;
-  sd_load<VEC>(sX, SD_LDX, rows + h * d.V + v0, d.ch, here, min(SD_V, d.V - v0), SD_V);
-  sd_load<VEC>(sH, LDN, rows + d.inner + h / (d.heads / d.groups) * d.N, d.ch, here, d.N, d.NP);
+  if (VEC) sd_cp_wait();
   __syncthreads();
   for (int i = threadIdx.x; i < SD_Q * d.NP / 2; i += SD_THREADS) {
     const int t = i / (d.NP / 2), at = t * LDN + i % (d.NP / 2) * 2;
@@ -121,8 +129,10 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
   }
   __syncthreads();
   float* out = states + (((size_t)seg * chunks + c) * d.heads + h) * d.N * d.V;
-  for (int m0 = warp * 16; m0 < d.NP; m0 += 64) {
-    float acc[8][4] = {};
+  // warps 0 .. 3 take the first 32 columns of the tile, warps 4 .. 7 the others
+  const int vh = warp / 4 * 32;
+  for (int m0 = warp % 4 * 16; m0 < d.NP; m0 += 64) {
+    float acc[4][4] = {};
 #pragma unroll
     for (int k0 = 0; k0 < SD_Q; k0 += 16) {
       uint32_t ah[4], al[4];
@@ -130,9 +140,9 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
       sd_ldsm_t(ah, sH + at);
       sd_ldsm_t(al, sL + at);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
+      for (int np = 0; np < 2; ++np) {
         uint32_t b[4];
-        sd_ldsm_t(b, sX + (k0 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + np * 16 + (lane >> 4) * 8);
+        sd_ldsm_t(b, sX + (k0 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + vh + np * 16 + (lane >> 4) * 8);
         sd_mma(acc[2 * np], ah, b[0], b[1]);
         sd_mma(acc[2 * np + 1], ah, b[2], b[3]);
         sd_mma(acc[2 * np], al, b[0], b[1]);
@@ -140,10 +150,10 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_state_kernel(float* __restrict
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = m0 + lane / 4 + (e >> 1) * 8, v = v0 + i * 8 + (lane & 3) * 2 + (e & 1);
+        const int r = m0 + lane / 4 + (e >> 1) * 8, v = v0 + vh + i * 8 + (lane & 3) * 2 + (e & 1);
         if (VEC) {
           if ((e & 1) == 0 && r < d.N && v < d.V) *reinterpret_cast<float2*>(out + (size_t)r * d.V + v) = make_float2(acc[i][e], acc[i][e + 1]);
         } else if (r < d.N && v < d.V) {
@@ -224,16 +234,17 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
   }
   for (int t = threadIdx.x; t < SD_Q; t += SD_THREADS)
     info[t] = t < here ? rowinfo[(size_t)(row0 + t) * d.heads + h] : make_float4(0.f, 0.f, 0.f, 0.f);
+  if (VEC) sd_cp_wait();
   __syncthreads();
-  // warp: rows 16 warp .. + 15 against the keys up to its last row
-  const int t0 = warp * 16, r_lo = t0 + lane / 4;
-  float sc[8][4] = {}, inter[8][4] = {}, acc[8][4] = {};
+  // warp: 16 rows against the rows up to its last one, half of the tile's columns
+  const int tw = warp % 4, t0 = tw * 16, r_lo = t0 + lane / 4, vh = warp / 4 * 32;
+  float sc[8][4] = {}, inter[4][4] = {}, acc[4][4] = {};
   for (int ks = 0; ks < d.NP / 16; ++ks) {
     uint32_t a[4];
     sd_ldsm(a, sC + (t0 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDN + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      if (j > warp) break;
+      if (j > tw) break;
       uint32_t b[4];
       sd_ldsm(b, sB + (j * 16 + (lane >> 4) * 8 + (lane & 7)) * LDN + ks * 16 + ((lane >> 3) & 1) * 8);
       sd_mma(sc[2 * j], a, b[0], b[1]);
@@ -242,9 +253,9 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
 #pragma unroll
     for (int part = 0; part < 2; ++part)
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
+      for (int np = 0; np < 2; ++np) {
         uint32_t b[4];
-        sd_ldsm_t(b, sS + (part * d.NP + ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + np * 16 + (lane >> 4) * 8);
+        sd_ldsm_t(b, sS + (part * d.NP + ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + vh + np * 16 + (lane >> 4) * 8);
         sd_mma(inter[2 * np], a, b[0], b[1]);
         sd_mma(inter[2 * np + 1], a, b[2], b[3]);
       }
@@ -252,7 +263,7 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
   const float4 it[2] = {info[r_lo], info[r_lo + 8]};
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
-    if (j > warp) break;
+    if (j > tw) break;
     uint32_t ah[4], al[4];
 #pragma unroll
     for (int half = 0; half < 2; ++half)
@@ -270,9 +281,9 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
         al[half * 2 + hr] = pack_bf2(p[0] - bf_lo(v), p[1] - bf_hi(v));
       }
 #pragma unroll
-    for (int np = 0; np < 4; ++np) {
+    for (int np = 0; np < 2; ++np) {
       uint32_t b[4];
-      sd_ldsm_t(b, sX + (j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + np * 16 + (lane >> 4) * 8);
+      sd_ldsm_t(b, sX + (j * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * SD_LDX + vh + np * 16 + (lane >> 4) * 8);
       sd_mma(acc[2 * np], ah, b[0], b[1]);
       sd_mma(acc[2 * np + 1], ah, b[2], b[3]);
       sd_mma(acc[2 * np], al, b[0], b[1]);
@@ -287,8 +298,8 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_out_kernel(float* __restrict__
     const float dec = __expf(it[hr].x + it[hr].y);
     float* dst = y + (size_t)(row0 + t) * ldy + (size_t)h * d.V;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int v = i * 8 + (lane & 3) * 2;
+    for (int i = 0; i < 4; ++i) {
+      const int v = vh + i * 8 + (lane & 3) * 2;
       float o[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) o[e] = fmaf(dec, inter[i][2 * hr + e], acc[i][2 * hr + e]) + sk * bf2f(sX[t * SD_LDX + v + e]);

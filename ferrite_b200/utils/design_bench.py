@@ -1,11 +1,13 @@
 """Designs of listed layers, each beside the framework's closest other model of the same width, heads and parameter count, with
 random weights: Zototar (latent attention without positions) beside the dense MLA model, Dofunex (delta rules with a decay per
 channel, every fourth layer attention) beside the dense Gated DeltaNet hybrid, Rakizen (parallel blocks, windows and chunks, two maps in every
-fourth layer) beside the sequential grouped-query attention model, dense or routed.
+fourth layer) beside the sequential grouped-query attention model, dense or routed, Pironex (latent attention, pooled windows, state-space layers,
+routed feed-forwards with a shared expert) beside the routed Gated DeltaNet hybrid.
 
-`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()`, `kernels_dofunex()` and
-`kernels_rakizen()` time every kernel of the first beside the kernel that does the same job for the second and give both as fractions of their
-rooflines. They print nothing and return plain dictionaries; `bench.py --design ...` and `microbench latent|cdelta|parallel` print them.
+`models()` measures prefill and decode throughput through the engine (CUDA graphs for decode steps), `kernels()`, `kernels_dofunex()`,
+`kernels_rakizen()` and `kernels_pironex()` time every kernel of the first beside the kernel that does the same job for the second and give both as
+fractions of their rooflines. They print nothing and return plain dictionaries; `bench.py --design ...` and `microbench
+latent|cdelta|parallel|pooled` print them.
 """
 from __future__ import annotations
 
@@ -15,7 +17,7 @@ from typing import Dict, List
 
 import torch
 
-from ..config import EngineConfig, ModelConfig, dofunex, rakizen, zototar
+from ..config import EngineConfig, ModelConfig, dofunex, pironex, rakizen, zototar
 from .microbench import Timer, graph_time, peaks, rnd
 
 SIZES = {       # name: width, heads, query latent, feed-forward width, layers
@@ -62,6 +64,22 @@ def pair_rakizen(size: str):
     return a, ModelConfig(inter=max(256, round(spare / (3 * w * n) / 128) * 128), **kw)
 
 
+def pair_pironex(size: str):
+    """(Pironex model, routed hybrid of Gated DeltaNet and gated attention layers) of one size: equal width, heads, layers, experts and shared
+    expert; every second layer of the hybrid is attention, as every second of the other reads keys."""
+    w, h, kv, n, experts, top, ff = SIZES_PIRONEX[size]
+    a = pironex(w, n, h, kv, VOCAB, dim=DIM, experts=experts, top=top, expert_ff=ff, shared_ff=ff, name=f"pironex-{size}")
+    b = ModelConfig(name=f"hybrid-moe-{size}", hidden=w, inter=ff, n_layers=n, full_attn_every=2, head_dim=DIM, n_q=h, n_kv=kv, rotary_dim=DIM // 2,
+                    lin_k_heads=h, lin_v_heads=h, lin_dk=DIM, lin_dv=DIM, vocab=VOCAB, tie_embeddings=True, n_experts=experts, top_k=top,
+                    expert_inter=ff, n_shared=1, router="softmax")
+    return a, b
+
+
+SIZES_PIRONEX = {       # name: width, heads, key / value heads, layers, experts, per token, their width
+    "1k": (1024, 8, 2, 16, 32, 4, 512),
+    "2k": (2048, 16, 4, 12, 64, 6, 1024),
+    "4k": (4096, 32, 8, 8, 32, 4, 1536),
+}
 SIZES_RAKIZEN = {       # name: width, heads, key / value heads, (expert's) feed-forward width, layers, experts, per token, groups, kept groups
     "2k": (2048, 16, 4, 6144, 16, 0, 0, 1, 1),
     "4k": (4096, 32, 8, 12288, 8, 0, 0, 1, 1),
@@ -75,6 +93,7 @@ SIZES_DOFUNEX = {       # name: width, heads, key / value heads of the attention
 DESIGNS = {"zototar": (pair, "mla_dense", "dense MLA model of equal width, heads, latent and parameter count", "2k,4k,7k"),
            "rakizen": (pair_rakizen, "gqa_sequential", "sequential grouped-query attention model of equal width, heads and parameter count (routed "
                        "feed-forwards in the moe size)", "2k,4k,2k-moe"),
+           "pironex": (pair_pironex, "hybrid_moe", "routed Gated DeltaNet hybrid of equal width, heads, layers and experts", "1k,2k,4k"),
            "dofunex": (pair_dofunex, "hybrid_dense", "dense Gated DeltaNet hybrid of equal width, heads and parameter count", "2k,4k,5k")}
 
 
@@ -248,7 +267,7 @@ def kernels(dev, heads: int = 32, width: int = 4096, ctx: int = 4096, prompt: in
     kv = ops.linear(ops.latent_rows(c0, grp, kvb), kv_up).view(-1, kvb, 2, heads, D)
 
     def flash(exact):
-        return lambda j: ops.C.attn_prefill_tc(out, q0, kv[:, :, 0], kv[:, :, 1], q0, grp.own, s0[1], s0[2], s0[3], grp.table, kvb, T, heads,
+        return lambda j: ops.C.attn_prefill_tc(out, q0, kv[:, :, 0], kv[:, :, 1], q0, grp.own, s0[1], s0[2], s0[3], grp.context()[1], kvb, T, heads,
                                                heads, D, False, ops.status_word, scale=0.088, exact_p=exact)
     add(f"flash, softmax weights as value + remainder, {T} rows, {heads} heads of {D}", (flash(True), 0.0, tri * heads * 4 * D, 1),
         "flash, bf16 softmax weights", (flash(False), 0.0, tri * heads * 4 * D, 1))
@@ -496,5 +515,182 @@ def kernels_rakizen(dev, heads: int = 32, kv_heads: int = 8, width: int = 4096, 
         n = z.shape[1]
         add(f"router, {n} experts, {keep} of {grp_n} groups, {T} rows", (lambda j: ops.moe_route(z, None, 1, K, grp_n, keep, 2.0), T * (n + 2 * K) * 4.0, 0.0, 1),
             "router, 4 of 8 groups", (lambda j: ops.moe_route(zl, None, 1, K, 8, 4, 2.0), T * (E + 2 * K) * 4.0, 0.0, 1))
+    assert ops.status() == 0
+    return acc.rows
+
+
+def kernels_pironex(dev, heads: int = 16, kv_heads: int = 4, width: int = 2048, ctx: int = 4096, prompt: int = 2048, size: int = 1024,
+                    pool: int = 16) -> List[Dict]:
+    """Pironex's kernels beside those of the routed Gated DeltaNet hybrid and, for its latent attention, of the MLA model. Bounded rows see `size`
+    keys and the means before them; the like kernel of few rows gets a cache of as many keys."""
+    from ..models.weights import GqaDims, LatentDims, SsmDims
+    from ..ops.cuda_ops import CudaOps
+    from ..ops.latent import SegGroup
+    from ..parallel.ep import ExpertParallel
+    ops, acc = CudaOps(dev), _Rows(dev)
+    add = acc.add
+    D, L, R, kvb, H, G, W, T = DIM, KV_RANK, ROPE, 64, heads, kv_heads, width, prompt
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    full = lambda m, v: torch.full((m,), v, dtype=torch.int32, device=dev)
+    inv, inv64 = torch.rand(D // 2, device=dev), torch.rand(D // 2, device=dev, dtype=torch.float64)
+    att = GqaDims(H, G, D, D, D ** -0.5, D // 2, (H + G) * D, False, D, row_norm=True, softcap=50.0, window=size, rot_half=True, pool=pool)
+    lat = LatentDims(H, 0, L, 0, L + R, D + R, (D + R) ** -0.5, 0, D, L, D, R, size)
+    E, K, F = 64, 6, 1024
+    for m in (1, 16, T):
+        many, n = m > 64, 3
+        slot = torch.zeros(m, dtype=torch.int32, device=dev) if many else torch.arange(m, dtype=torch.int32, device=dev)
+        pos = torch.arange(m, dtype=torch.int32, device=dev) if many else torch.zeros(m, dtype=torch.int32, device=dev)
+        bufs = max(1, min(8, (400 << 20) // (m * W * 4)))
+        x, y = [f32(m, W) for _ in range(bufs)], [f32(m, W) for _ in range(bufs)]
+        xb, yb = [rnd(m, W) for _ in range(bufs)], [rnd(m, W) for _ in range(bufs)]
+        w32, w16, cw, tails = torch.ones(W, device=dev), rnd(W), f32(4, W), rnd(64, n, W)
+        place, xs = 8, [f32(10, m, W) for _ in range(max(1, bufs // 4))]
+        dwa, one = torch.rand(place + 1, device=dev), dict(conv=(cw, tails), row_slot=slot, row_pos=pos, single=not many)
+        like = ("rmsnorm + residual", (lambda j: ops.rmsnorm(xb[j], w16, 1e-6, True, res=yb[j]), m * W * 8.0, 0.0, bufs))
+        conv_bytes = m * W * (4.0 if many else 14.0)               # the convolution's own pass, or the tails of every row
+        add(f"seam: norm of y, add, norm, convolution, {m} rows", (lambda j: ops.add_conv_normed(x[j], x[j], y[j], w32, W, 1e-6, w32, **one),
+                                                                  m * W * 14.0 + conv_bytes, 0.0, bufs), *like)
+        add(f"seam with an average over {place + 1} results, {m} rows",
+            (lambda j: ops.add_conv_normed(x[j], x[j], y[j], w32, W, 1e-6, w32, average=(xs[j % len(xs)], place, dwa), **one),
+             m * W * (14.0 + 4.0 * place + 4.0) + conv_bytes, 0.0, bufs), *like)
+        nb = max(1, m // kvb)
+        bt = torch.arange((1 if many else m) * nb, dtype=torch.int32, device=dev).view(-1, nb)
+        kc, vc, pb = rnd(bt.numel(), kvb, G, D), rnd(bt.numel(), kvb, G, D), 8 if many else 32
+        means = tuple(rnd(bt.numel(), kvb // pool, G, D) for _ in "kv")
+        proj, norms, pq = [f32(m, (H + 2 * G) * D) for _ in range(pb)], (f32(H * D), f32(G * D)), [rnd(m, (2 * H + 2 * G) * D) for _ in range(pb)]
+        nw, segs = rnd(D), (i32([0]), i32([0]), i32([m])) if many else (slot, slot * 0, full(m, 1))
+
+        def prep(j):
+            ops.gqa_prep(proj[j], att, None, inv64, slot, pos, bt, kc, vc, kvb, 1e-6, norms=norms)
+            ops.pool_keys(att, kc, vc, means, *segs, m if many else 1, bt, kvb)
+        attn_prep = ("attn_prep", (lambda j: ops.attn_prep(pq[j], nw, nw, inv, slot, pos, bt, kc, vc, kvb, H, G, D, D // 2, True, 1e-6),
+                                   m * D * (H + 2 * G) * 4.0, 0.0, pb))
+        add(f"gqa_row_prep + pool_keys, {m} rows, {H} / {G} heads", (prep, m * D * ((H + 2 * G) * 6.0 + (4.0 * G if many else 0.0)), 0.0, pb), *attn_prep)
+        pl, cl, kn = [f32(m, H * (D + R) + L + R) for _ in range(pb)], rnd(bt.numel(), kvb, L + R), torch.ones(L + R, device=dev)
+        qq, kva, k16, inv_r = rnd(m, H * (D + R)), [rnd(m, L + R) for _ in range(pb)], rnd(L), torch.rand(R // 2, device=dev)
+        add(f"latent_rot_prep, {m} rows", (lambda j: ops.latent_rot_prep(pl[j], lat, kn, inv64[:R // 2], slot, pos, bt, cl, kvb, 1e-6),
+                                           m * (H * (D + R) + L + R) * 6.0, 0.0, pb),
+            "mla_prep", (lambda j: ops.mla_prep(qq, kva[j], k16, None, inv_r, slot, pos, bt, cl, kvb, H, D, L, R, 1e-6, absorb=False),
+                         m * ((L + R) * 4.0 + H * R * 4.0), 0.0, pb))
+        del x, y, xb, yb, xs, proj, pq, pl
+    blocks = (ctx - size) // pool
+    for m in (1, 4, 16):
+        nb, seen = ctx // kvb, (size + blocks + kvb - 1) // kvb * kvb
+        nbl = seen // kvb
+        bufs = max(1, min(32, (400 << 20) // (m * seen * G * D * 4)))
+        nk = min(bufs, 8)
+        kc, vc = [rnd(m * nb, kvb, G, D) for _ in range(nk)], [rnd(m * nb, kvb, G, D) for _ in range(nk)]
+        means = [tuple(rnd(m * nb, kvb // pool, G, D) for _ in "kv") for _ in range(nk)]
+        kl, vl = [rnd(m * nbl, kvb, G, D) for _ in range(bufs)], [rnd(m * nbl, kvb, G, D) for _ in range(bufs)]
+        slot, ones, full_len, like_len = torch.arange(m, dtype=torch.int32, device=dev), full(m, 1), full(m, ctx), full(m, seen)
+        bt, btl = torch.arange(m * nb, dtype=torch.int32, device=dev).view(m, nb), torch.arange(m * nbl, dtype=torch.int32, device=dev).view(m, nbl)
+        q, out, pj, grp = rnd(m, H, D), rnd(m, H, D), rnd(m, 2 * H * D), SegGroup(0, m, 0, m, 1)
+        work = (m * (size + blocks) * G * D * 4.0, 4.0 * m * H * (size + blocks) * D)
+        add(f"decode attention + merge, window of {size} and {blocks} means, {m} rows",
+            (lambda j: ops.gqa_attention(q, att, kc[j], vc[j], None, grp, slot, full_len, (slot, slot, ones), bt, kvb, 64, out, pooled=means[j]), *work, nk),
+            f"attention + combine, {seen} keys",
+            (lambda j: ops.attention(q, pj, kl[j], vl[j], slot, like_len, btl, kvb, H, G, D, True, nsplit=32, segs=(slot, slot, ones, 1)), *work, bufs))
+        del kc, vc, means, kl, vl
+        nbl = size // kvb
+        bufs = max(1, min(16, (400 << 20) // (m * ctx * (L + R) * 2)))
+        c0, c1 = [rnd(m * nb, kvb, L + R) for _ in range(bufs)], [rnd(m * nbl, kvb, L + R) for _ in range(2 * bufs)]
+        btl = torch.arange(m * nbl, dtype=torch.int32, device=dev).view(m, nbl)
+        qa, short = rnd(m, H, L + R), full(m, size)
+        work = (m * size * (L + R) * 2.0, 2.0 * m * H * size * (2 * L + R))
+        add(f"latent_mma + merge, window of {size} in {ctx}, {m} rows",
+            (lambda j: ops.latent_attention(qa, c0[j], grp, slot, full_len, (slot, slot, ones), bt, kvb, 0.07, 64, vlat=L, window=size), *work, bufs),
+            f"mla_attn + combine, {size} keys", (lambda j: ops.mla_attention(qa, c1[j], slot, short, btl, kvb, H, L, R, 0.07, nsplit=16), *work, 2 * bufs))
+        del c0, c1
+    # prompt attention
+    nb = T // kvb
+    perm = torch.randperm(nb, device=dev).to(torch.int32).view(1, nb)
+    s0, rslot, rlen = (i32([0]), i32([0]), i32([T]), i32([0])), torch.zeros(T, dtype=torch.int32, device=dev), torch.arange(1, T + 1, dtype=torch.int32, device=dev)
+    kc, vc, q, out, pj = rnd(nb, kvb, G, D), rnd(nb, kvb, G, D), rnd(T, H, D), rnd(T, H, D), rnd(T, 2 * H * D)
+    grp = SegGroup(0, 1, 0, T, T, True)
+    grp.segments, grp.block_table, grp.kv_block = [(0, 0, T)], perm, kvb
+    start, rows = i32([0]), (T - size) // pool
+    km, vm = rnd(max(64, (rows + 63) // 64 * 64), G, D), rnd(max(64, (rows + 63) // 64 * 64), G, D)
+    seen = sum(min(t + 1, size) + max(0, t + 1 - size) // pool for t in range(T))
+    like = ("prompt attention, bf16 weights", (lambda j: ops.attention_prefill(q, pj, kc, vc, *s0, perm, kvb, H, G, D, True, T), 0.0,
+                                               T * (T + 1) / 2.0 * H * 4 * D, 1))
+    add(f"prompt attention, softcap, window of {size} and means, {T} rows",
+        (lambda j: ops.C.attn_prefill_tc(out, q.view(T, -1), kc, vc, q.view(T, -1), s0[0], s0[1], s0[2], s0[3], perm, kvb, T, H, G, D, False,
+                                         ops.status_word, scale=D ** -0.5, exact_p=True, window=size, softcap=50.0, k_mean=km, v_mean=vm,
+                                         mean_start=start, pool=pool), 0.0, seen * H * 4.0 * D, 1), *like)
+    c0, kv_up, kv_b = rnd(nb, kvb, L + R), rnd(H * (2 * D + R), L + R, scale=L ** -0.5), rnd(2 * H * D, L, scale=L ** -0.5)
+    q1, ol, qabs = rnd(T, H * (D + R)), rnd(T, H * D), rnd(T, H, L + R)
+    lat_seen, lat_all = sum(min(t + 1, size) for t in range(T)), T * (T + 1) / 2.0
+    up0, up1 = 2.0 * T * (L * 2 * D) * H, 2.0 * T * L * 2 * H * D
+    add(f"latent prompt attention (gather, expansion, flash), window of {size}, {T} rows",
+        (lambda j: ops.latent_attention_prompt(q1, ops.latent_rows(c0, grp, kvb, size), kv_up, lat, grp, s0, kvb, ol), 0.0,
+         up0 + lat_seen * H * 2.0 * (2 * D + R), 1), "mla prompt attention (gather, GEMM, packing, flash)",
+        (lambda j: ops.mla_attention_prefill(q1, qabs, c0, kv_b, [(0, 0, T)], s0[1], s0[2], s0[3], perm, kvb, H, D, D, L, R), 0.0,
+         up1 + lat_all * H * 2.0 * (2 * D + R), 1))
+    # recurrences: 2 W / 64 heads of 64 with a state of 128, beside W / 128 heads of 128 x 128
+    SH, SV, SN = 2 * W // 64, 64, 128
+    d = SsmDims(SH, 1, SN, SV, 4, 1, SH * SV)
+    w = dict(conv=f32(4, d.channels), conv_bias=f32(d.channels), A=-torch.rand(SH, device=dev), dt_bias=f32(SH) - 2, skip=f32(SH), gnorm_w=f32(d.inner))
+    cw, A, dtb, gw = rnd(3 * H * D, 4), f32(H), f32(H), rnd(D)
+    ld = (d.dt_off + SH + 7) // 8 * 8
+    for m in (1, 4, 16):
+        bufs = max(2, min(64, (400 << 20) // (m * SH * SN * SV * 4)))
+        rec, tail, rec2, tail2 = ([f32(m, SH, SN, SV) for _ in range(bufs)], [rnd(m, 3, d.channels) for _ in range(bufs)],
+                                  [f32(m, H, D, D) for _ in range(2 * bufs)], [rnd(m, 3, 3 * H * D) for _ in range(2 * bufs)])
+        proj, pg, slot, ones = rnd(m, ld), rnd(m, 4 * H * D + 2 * H), torch.arange(m, dtype=torch.int32, device=dev), full(m, 1)
+        grp1 = [SegGroup(0, m, 0, m, 1)]
+        add(f"ssm_step + gated norm, {m} rows, {SH} heads of {SN} x {SV}",
+            (lambda j: ops.ssm(proj, d, w, rec[j], tail[j], grp1, slot, slot, ones, slot, slot, 1e-6), m * (SH * SN * SV * 8.0 + ld * 8.0), 0.0, bufs),
+            f"gdn_step, {H} heads of {D} x {D}",
+            (lambda j: ops.gdn_step(pg, cw, rec2[j], tail2[j], A, dtb, gw, slot, slot, ones, H, H, D, D, 1e-6), m * (H * D * D * 8.0 + H * D * 20.0), 0.0, 2 * bufs))
+        del rec, rec2
+    rec, tail, rec2, tail2 = f32(1, SH, SN, SV), rnd(1, 3, d.channels), f32(1, H, D, D), rnd(1, 3, 3 * H * D)
+    proj, pg, pos = rnd(T, ld), rnd(T, 4 * H * D + 2 * H), rlen - 1
+    # per 64-row chunk and head: C B^T, its product with x, C with the state, and the chunk's state
+    fl = T / 64 * SH * (2.0 * 64 * 64 * SN + 2 * 64 * 64 * SV + 4 * 64 * SN * SV)
+    fl2 = T / 64 * H * (4 * 64 * 64 * D + 64 * 64 * 64 / 3 + 6 * 64 * D * D + 4 * 64 * 64 * D)
+    one, grp1 = (i32([0]), i32([0]), i32([T])), [SegGroup(0, 1, 0, T, T, True)]
+    gdn = (lambda: ops.gdn_rec(ops.gdn_conv(pg, cw, tail2, *one, 3 * H * D, T), pg, rec2, tail2, A, dtb, *one, H, H, D, D, 1e-6, chunked=True, max_rows=T))
+    add(f"state-space layer (convolutions, three chunk kernels, gated norm, tail), {T} rows",
+        (lambda j: ops.ssm(proj, d, w, rec, tail, grp1, *one, rslot, pos, 1e-6), T * (ld * 2.0 + d.inner * 2.0), fl, 1),
+        "gdn_conv + gdn_chunk + gated_norm", (lambda j: ops.gated_norm(gdn(), pg, 3 * H * D, gw, H, D, 1e-6), T * H * D * 10.0, fl2, 1))
+    xbc = proj[:, d.inner:d.dt_off]
+    add(f"conv_rows, {T} rows of {d.channels}",
+        (lambda j: ops.conv_rows(xbc, w["conv"], tail, rslot, pos, bias=w["conv_bias"], silu=True), T * d.channels * 4.0, 0.0, 1), "gdn_conv",
+        (lambda j: ops.gdn_conv(pg, cw, tail2, *one, 3 * H * D, T), T * 3 * H * D * 4.0, 0.0, 1))
+    ys, conv = f32(T, d.inner), ops.conv_rows(xbc, w["conv"], tail, rslot, pos, bias=w["conv_bias"], silu=True)
+    scratch = ops.scratch("ssd_chunk", ops.C.ssd_chunk_scratch_bytes(T, 1, T, SH, SN, SV) // 4, torch.float32)
+    sizes = [SH, 1, SN, SV, 4]
+    qkv = ops.gdn_conv(pg, cw, tail2, *one, 3 * H * D, T)
+    add(f"ssd_chunk (states, scan, outputs), {T} rows", (lambda j: ops.C.ssd_chunk(ys, rec, scratch, conv, proj, w["A"], w["dt_bias"], w["skip"], *one, T, sizes),
+                                                       T * d.channels * 2.0 + T * d.inner * 4.0, fl, 1), "gdn_chunk",
+        (lambda j: ops.gdn_rec(qkv, pg, rec2, tail2, A, dtb, *one, H, H, D, D, 1e-6, chunked=True, max_rows=T), T * H * D * 10.0, fl2, 1))
+    yg, go = f32(T, H * D), rnd(T, d.ko)
+    add(f"gated norm of whole rows, {T} rows of {d.inner}", (lambda j: ops.C.group_norm_gated(go, ys, proj, w["gnorm_w"], 1, 1e-6, None, None),
+                                                            T * d.inner * 8.0, 0.0, 1), "gated_norm",
+        (lambda j: ops.gated_norm(yg, pg, 3 * H * D, gw, H, D, 1e-6), T * H * D * 8.0, 0.0, 1))
+    # routed feed-forward with a shared expert
+    gu, dn = rnd(E + 1, 2 * F, W, scale=0.02), rnd(E + 1, W, F, scale=0.02)
+    sh = (rnd(1, 2 * F, W, scale=0.02), rnd(1, W, F, scale=0.02), 7.0)
+    for m in (1, 4, 16):
+        h, x, res, w32 = rnd(m, W), f32(m, W), rnd(m, W), torch.ones(W, device=dev)
+        z = [f32(m, E + 8) for _ in range(16)]
+        picks = [ops.moe_route(v, None, 2, K, 1, 1, 1.0, n_exp=E, shared_col=E, shared_id=E) for v in z]
+        used = sum(len(set(ids.reshape(-1).tolist())) for ids, _ in picks) / 16
+        work = (used * 3.0 * F * W * 2, 6.0 * m * (K + 1) * F * W, 16)
+        add(f"expert rows, shared one included, + seam, {m} rows",
+            (lambda j: ops.add_conv_normed(x, x, None, w32, W, 1e-6, w32, pairs=(ops.expert_rows(h, picks[j][0], gu[:E], dn[:E], 7.0, sh), picks[j][1])), *work),
+            "moe_experts (pairs, combine)", (lambda j: ops.moe_experts(h, *picks[j], gu, dn, 0, E + 1, None, None, res), *work))
+        add(f"router by logits, {E} experts, {m} rows", (lambda j: ops.moe_route(z[j], None, 2, K, 1, 1, 1.0, n_exp=E, shared_col=E, shared_id=E),
+                                                        m * (E + 2 * K) * 4.0, 0.0, 16), "router, softmax",
+            (lambda j: ops.moe_route(z[j], None, 0, K, 1, 1, 1.0, n_exp=E, shared_col=E, shared_id=E), m * (E + 2 * K) * 4.0, 0.0, 16))
+    h, y, res, z = rnd(T, W), f32(T, W), rnd(T, W), f32(T, E + 8)
+    ids, wts = ops.moe_route(z, None, 2, K, 1, 1, 1.0, n_exp=E)
+    ep = ExpertParallel(None, torch.device(dev), E, W, T * K, status=ops.status_word)
+    work = ((E + 1) * 3.0 * F * W * 2, 6.0 * T * (K + 1) * F * W, 1)
+    add(f"clamped experts and shared expert, {T} rows",
+        (lambda j: ep.moe(ops, h, ids, wts, gu[:E], dn[:E], ops.linear(ops.glu(h, sh[0][0], 7.0), sh[1][0]), z[:, E], acc=y, add=False, limit=7.0), *work),
+        "swiglu experts and shared expert",
+        (lambda j: ep.moe(ops, h, ids, wts, gu[:E], dn[:E], ops.linear(ops.linear(h, sh[0][0], swiglu=True), sh[1][0]), z[:, E], res=res), *work))
     assert ops.status() == 0
     return acc.rows

@@ -159,7 +159,7 @@ def graph_time(t, chain, reps):
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("what", choices=["gemv", "gemm", "layer", "attn_decode", "attn_prefill", "gdn", "moe", "exl3",
-                                     "head_linear", "ffn_fp4", "select", "latent", "cdelta", "parallel"])
+                                     "head_linear", "ffn_fp4", "select", "latent", "cdelta", "parallel", "pooled"])
     ap.add_argument("--heads", type=int, default=32, help="latent: heads")
     ap.add_argument("--width", type=int, default=4096, help="latent: model width")
     ap.add_argument("--kv", default="bf16", help="attn_decode: cache form (bf16 | fp8 | int6 | int4)")
@@ -270,6 +270,11 @@ def main():
         # the Rakizen kernels beside the sequential grouped-query attention model's
         from .design_bench import kernels_rakizen
         for r in kernels_rakizen(dev, a.heads, max(2, a.heads // 4), a.width, a.ctx):
+            print(json.dumps(r), flush=True)
+    elif a.what == "pooled":
+        # the Pironex kernels beside those of the routed Gated DeltaNet hybrid and the MLA model
+        from .design_bench import kernels_pironex
+        for r in kernels_pironex(dev, a.heads, max(2, a.heads // 4), a.width, a.ctx):
             print(json.dumps(r), flush=True)
     elif a.what == "ffn_fp4":
         # dense FFN block of the 27B model on prompt rows, NVFP4 weights and activations: gate|up + SwiGLU + down with the
