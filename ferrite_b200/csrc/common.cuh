@@ -433,6 +433,8 @@ __device__ __forceinline__ void multimem_red_add_u32(uint32_t* mc_ptr, uint32_t 
 
 // ---- programmatic dependent launch ----------------------------------------------------------------------
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// Ask L2 for a line. Reads nothing into the kernel, so it may come before pdl_wait for anything: L2 is where writes meet.
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 // A pointer to what the kernel before this one wrote, for use after pdl_wait. Loads through `const __restrict__` parameters count as loads of
 // memory that never changes during the kernel, which the compiler may move ahead of the wait; behind this they cannot be.
 template <typename T>

@@ -28,27 +28,24 @@ __device__ __forceinline__ RowStats cr_warp(RowStats s) {
     s = cr_join(s, {__shfl_xor_sync(0xffffffffu, s.n, o), __shfl_xor_sync(0xffffffffu, s.mean, o), __shfl_xor_sync(0xffffffffu, s.m2, o)});
   return s;
 }
-// (mean, 1 / deviation) of the row whose columns i + e < width, i = 4 (threadIdx.x + k blockDim.x), the threads hold in v[k]
-template <int NV>
-__device__ __forceinline__ float2 cr_stats(const float4 (&v)[NV], int width, float eps, RowStats* red) {
-  RowStats s{0.f, 0.f, 0.f};
+// ... of four columns, of which `left` are inside the row's true width
+__device__ __forceinline__ RowStats cr_quad(const float4& v, int left) {
+  const float c[4] = {v.x, v.y, v.z, v.w};
+  RowStats t{0.f, 0.f, 0.f};
+  if (left >= 4) {
+    t.n = 4.f;
+    t.mean = 0.25f * ((c[0] + c[1]) + (c[2] + c[3]));
 #pragma unroll
-  for (int k = 0; k < NV; ++k) {
-    const int left = width - 4 * (threadIdx.x + k * blockDim.x);
-    const float c[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
-    RowStats t{0.f, 0.f, 0.f};
-    if (left >= 4) {
-      t.n = 4.f;
-      t.mean = 0.25f * ((c[0] + c[1]) + (c[2] + c[3]));
+    for (int e = 0; e < 4; ++e) t.m2 = fmaf(c[e] - t.mean, c[e] - t.mean, t.m2);
+  } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) t.m2 = fmaf(c[e] - t.mean, c[e] - t.mean, t.m2);
-    } else {
-#pragma unroll
-      for (int e = 0; e < 3; ++e)
-        if (e < left) t = cr_join(t, {1.f, c[e], 0.f});
-    }
-    s = k == 0 ? t : cr_join(s, t);
+    for (int e = 0; e < 3; ++e)
+      if (e < left) t = cr_join(t, {1.f, c[e], 0.f});
   }
+  return t;
+}
+// (mean, 1 / deviation) of what all threads of the CTA hold
+__device__ __forceinline__ float2 cr_block(RowStats s, int width, float eps, RowStats* red) {
   s = cr_warp(s);
   const int lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   __syncthreads();
@@ -57,19 +54,95 @@ __device__ __forceinline__ float2 cr_stats(const float4 (&v)[NV], int width, flo
   s = cr_warp(lane < warps ? red[lane] : RowStats{0.f, 0.f, 0.f});
   return make_float2(s.mean, 1.f / sqrtf(s.m2 / (float)width + eps));
 }
+// columns i + e < width, i = 4 (threadIdx.x + k blockDim.x), in v[k]
+template <int NV>
+__device__ __forceinline__ float2 cr_stats(const float4 (&v)[NV], int width, float eps, RowStats* red) {
+  RowStats s = cr_quad(v[0], width - 4 * (int)threadIdx.x);
+#pragma unroll
+  for (int k = 1; k < NV; ++k) s = cr_join(s, cr_quad(v[k], width - 4 * (int)(threadIdx.x + k * blockDim.x)));
+  return cr_block(s, width, eps, red);
+}
 
-// NV: groups of four columns per thread, the whole row in registers. CONV: the convolution rides on the pass (one row per segment). What does
-// not come from the kernel before this one (weights) is read while that drains, what no norm has to wait for (results, tails) before the norms.
+// The pass of steps whose segments have several rows: many small CTAs, the row waits in shared memory between the norms (every thread reads what
+// it wrote itself), so that one CTA's barriers hide behind another's loads.
+constexpr int CN_ROW_THREADS = 256;
+
+__device__ __forceinline__ float2 cr_row_stats(const float* row, int width, int ld, float eps, RowStats* red) {
+  RowStats s{0.f, 0.f, 0.f};
+  for (int i = threadIdx.x * 4; i < ld; i += CN_ROW_THREADS * 4) {
+    s = cr_join(s, cr_quad(*reinterpret_cast<const float4*>(row + i), width - i));
+  }
+  return cr_block(s, width, eps, red);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(CN_ROW_THREADS)
+add_rows_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, const float* __restrict__ y, long ldy, const float* __restrict__ yp,
+                       const float* __restrict__ wts, int top, const float* __restrict__ w, float* __restrict__ xs, long xs_step, int place,
+                       const float* __restrict__ dwa, const float* __restrict__ next_w, T* __restrict__ h_out, int width, int ld, float eps) {
+  extern __shared__ __align__(16) float cr_row[];
+  __shared__ RowStats red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  x_in = after_wait(x_in); y = after_wait(y); yp = after_wait(yp); wts = after_wait(wts);
+  const size_t row = blockIdx.x;
+  const float* xi = x_in + row * ld;
+  if (w) {
+    for (int i = threadIdx.x * 4; i < ld; i += CN_ROW_THREADS * 4) {
+      float4 s = y ? *reinterpret_cast<const float4*>(y + row * ldy + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = 0; k < top; ++k) {
+        const float g = wts[row * top + k];
+        const float4 e = *reinterpret_cast<const float4*>(yp + (row * top + k) * ld + i);
+        s.x = fmaf(g, e.x, s.x); s.y = fmaf(g, e.y, s.y); s.z = fmaf(g, e.z, s.z); s.w = fmaf(g, e.w, s.w);
+      }
+      *reinterpret_cast<float4*>(cr_row + i) = s;
+    }
+    const float2 st = cr_row_stats(cr_row, width, ld, eps, red);
+    const float last = xs ? dwa[place] : 1.f;
+    for (int i = threadIdx.x * 4; i < ld; i += CN_ROW_THREADS * 4) {
+      const float4 f = *reinterpret_cast<const float4*>(cr_row + i), ww = *reinterpret_cast<const float4*>(w + i);
+      float4 v = *reinterpret_cast<const float4*>(xi + i);
+      v.x += (f.x - st.x) * st.y * ww.x; v.y += (f.y - st.x) * st.y * ww.y;
+      v.z += (f.z - st.x) * st.y * ww.z; v.w += (f.w - st.x) * st.y * ww.w;
+      if (xs) {                                              // this layer's result, then the sum over depth
+        *reinterpret_cast<float4*>(xs + place * xs_step + row * ld + i) = v;
+        v.x *= last; v.y *= last; v.z *= last; v.w *= last;
+#pragma unroll 4
+        for (int j = 0; j < place; ++j) {
+          const float g = dwa[j];
+          const float4 r = *reinterpret_cast<const float4*>(xs + j * xs_step + row * ld + i);
+          v.x = fmaf(g, r.x, v.x); v.y = fmaf(g, r.y, v.y); v.z = fmaf(g, r.z, v.z); v.w = fmaf(g, r.w, v.w);
+        }
+      }
+      *reinterpret_cast<float4*>(x + row * ld + i) = v;
+      *reinterpret_cast<float4*>(cr_row + i) = v;
+    }
+  } else {
+    for (int i = threadIdx.x * 4; i < ld; i += CN_ROW_THREADS * 4)
+      *reinterpret_cast<float4*>(cr_row + i) = *reinterpret_cast<const float4*>(xi + i);
+  }
+  if (!next_w) return;
+  const float2 st = cr_row_stats(cr_row, width, ld, eps, red);
+  for (int i = threadIdx.x * 4; i < ld; i += CN_ROW_THREADS * 4) {
+    const float4 v = *reinterpret_cast<const float4*>(cr_row + i), ww = *reinterpret_cast<const float4*>(next_w + i);
+    Elem<T>::store4(h_out + row * ld + i, make_float4((v.x - st.x) * st.y * ww.x, (v.y - st.x) * st.y * ww.y, (v.z - st.x) * st.y * ww.z,
+                                                      (v.w - st.x) * st.y * ww.w));
+  }
+}
+
+// The pass of steps whose segments are one row each, with the convolution on it. NV: groups of four columns per thread, the whole row in
+// registers. What does not come from the kernel before this one (weights) is read while that drains, what no norm has to wait for (results,
+// tails) before the norms.
 constexpr int cn_threads(int nv) { return nv == 16 ? 1024 : 512; }
 
-template <typename T, int NV, bool CONV>
-__global__ void __launch_bounds__(cn_threads(NV), NV == 1 && !CONV ? 2 : 1)
+template <typename T, int NV>
+__global__ void __launch_bounds__(cn_threads(NV))
 add_conv_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, const float* __restrict__ y, long ldy, const float* __restrict__ yp,
                        const float* __restrict__ wts, int top, const float* __restrict__ w, float* __restrict__ xs, long xs_step, int place,
                        const float* __restrict__ dwa, const float* __restrict__ next_w, T* __restrict__ h_out, T* __restrict__ xb,
                        const float* __restrict__ cw, int taps, T* __restrict__ tails, long tail_step, const int* __restrict__ row_slot, int commit,
                        int width, int ld, float eps) {
-  constexpr bool EARLY = NV == 1 && CONV;
+  constexpr bool EARLY = NV == 1;
   constexpr int PART = 4;                                    // expert rows, results and taps read at a time
   __shared__ RowStats red[32];
   pdl_launch_dependents();
@@ -88,11 +161,27 @@ add_conv_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, co
     for (int j = 0; j < PART; ++j) conv_own[EARLY ? j : 0] = j < taps && taps <= PART ? load(cw + (size_t)j * ld, col(0)) : zero;
   }
   const float last = xs ? dwa[place] : 1.f;
-  const int slot = CONV ? row_slot[row] : 0;
+  const int slot = row_slot[row];
+  T* tail = tails + slot * tail_step;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {                             // lines that nobody has touched since the last step
+    const int i = col(k);
+    if (i >= ld) break;
+    if (i % 32 == 0) {
+      if (!EARLY) {
+        if (w) prefetch_l2(w + i);
+        if (next_w) prefetch_l2(next_w + i);
+        for (int j = 0; j < taps; ++j) prefetch_l2(cw + (size_t)j * ld + i);
+      }
+      if (xs)
+        for (int j = 0; j < place; ++j) prefetch_l2(xs + j * xs_step + row * ld + i);
+    }
+    if (i % (128 / (int)sizeof(T)) == 0)
+      for (int j = 0; j + 1 < taps; ++j) prefetch_l2(tail + (size_t)j * ld + i);
+  }
   pdl_wait();
   x_in = after_wait(x_in); y = after_wait(y); yp = after_wait(yp); wts = after_wait(wts);
   float4 v[NV], f[NV], past[NV];
-  T* tail = CONV ? tails + slot * tail_step : nullptr;
   float4 tail_own[EARLY ? PART - 1 : 1];
   if (EARLY && next_w) {
 #pragma unroll
@@ -156,24 +245,22 @@ add_conv_normed_kernel(const float* __restrict__ x_in, float* __restrict__ x, co
                Elem<T>::from((v[k].z - st.x) * st.y * nw.z), Elem<T>::from((v[k].w - st.x) * st.y * nw.w)};
     const float4 h = make_float4(Elem<T>::to(h4[0]), Elem<T>::to(h4[1]), Elem<T>::to(h4[2]), Elem<T>::to(h4[3]));
     if (h_out) Elem<T>::store4(h_out + row * ld + i, h);
-    if constexpr (CONV) {
-      float4 o = h;
-      auto tap = [&](int j, const float4& c, const float4& p) {
-        o.x = fmaf(c.x, p.x, o.x); o.y = fmaf(c.y, p.y, o.y); o.z = fmaf(c.z, p.z, o.z); o.w = fmaf(c.w, p.w, o.w);
-        if (commit && j > 0) Elem<T>::store4(tail + (size_t)(j - 1) * ld + i, p);
-      };
-      if (EARLY && taps <= PART) {
+    float4 o = h;
+    auto tap = [&](int j, const float4& c, const float4& p) {
+      o.x = fmaf(c.x, p.x, o.x); o.y = fmaf(c.y, p.y, o.y); o.z = fmaf(c.z, p.z, o.z); o.w = fmaf(c.w, p.w, o.w);
+      if (commit && j > 0) Elem<T>::store4(tail + (size_t)(j - 1) * ld + i, p);
+    };
+    if (EARLY && taps <= PART) {
 #pragma unroll
-        for (int j = 0; j < PART; ++j)
-          if (j < taps) tap(j, conv_own[EARLY ? j : 0], j + 1 < taps ? tail_own[EARLY && j < PART - 1 ? j : 0] : h);
-      } else {
-        for (int j = 0; j < taps; ++j) {
-          const float4 p = j + 1 < taps ? Elem<T>::load4(tail + (size_t)j * ld + i) : h;
-          tap(j, *reinterpret_cast<const float4*>(cw + (size_t)j * ld + i), p);
-        }
+      for (int j = 0; j < PART; ++j)
+        if (j < taps) tap(j, conv_own[EARLY ? j : 0], j + 1 < taps ? tail_own[EARLY && j < PART - 1 ? j : 0] : h);
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const float4 p = j + 1 < taps ? Elem<T>::load4(tail + (size_t)j * ld + i) : h;
+        tap(j, *reinterpret_cast<const float4*>(cw + (size_t)j * ld + i), p);
       }
-      Elem<T>::store4(xb + row * ld + i, o);
     }
+    Elem<T>::store4(xb + row * ld + i, o);
   }
 }
 
@@ -304,6 +391,19 @@ extern "C" int fb_add_conv_normed(const float* x_in, float* x, const float* y, l
   if (rows <= 0) return 0;
   if (ld % 4 || ldy % 4 || ld > 49152 || width < 1 || width > ld || (top && (!yp || !wts)) || (w && !y && !top) || (xs && (!dwa || !w || place < 0)) ||
       (next_w && !h_out && !xb) || (xb && (!cw || taps < 1 || !row_slot || (taps > 1 && (!tails || tail_step % 4))))) return -1;
+  if (!xb) {
+    const size_t smem = (size_t)ld * 4;
+    auto go = [&](auto kern, auto* tag) {
+      using T = std::remove_pointer_t<decltype(tag)>;
+      if (smem > 40 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+      }
+      return (int)launch_pdl(kern, dim3(rows), dim3(CN_ROW_THREADS), smem, s, x_in, x, y, ldy, yp, wts, top, w, xs, xs_step, place, dwa, next_w,
+                             (T*)h_out, width, ld, eps);
+    };
+    return f32 ? go(add_rows_normed_kernel<float>, (float*)0) : go(add_rows_normed_kernel<bf16>, (bf16*)0);
+  }
   const int quads = ld / 4;
   int nv = 1;
   while (nv < 16 && quads > cn_threads(nv) * nv) nv *= 2;
@@ -314,11 +414,9 @@ extern "C" int fb_add_conv_normed(const float* x_in, float* x, const float* y, l
     return (int)launch_pdl(kern, g, b, 0, s, x_in, x, y, ldy, yp, wts, top, w, xs, xs_step, place, dwa, next_w, (T*)h_out, (T*)xb, cw, taps,
                            (T*)tails, tail_step, row_slot, commit, width, ld, eps);
   };
-#define FB_CN2(NV, CONV) (f32 ? go(add_conv_normed_kernel<float, NV, CONV>, (float*)0) : go(add_conv_normed_kernel<bf16, NV, CONV>, (bf16*)0))
-#define FB_CN(NV) (xb ? FB_CN2(NV, true) : FB_CN2(NV, false))
+#define FB_CN(NV) (f32 ? go(add_conv_normed_kernel<float, NV>, (float*)0) : go(add_conv_normed_kernel<bf16, NV>, (bf16*)0))
   return nv == 1 ? FB_CN(1) : nv == 2 ? FB_CN(2) : nv == 4 ? FB_CN(4) : nv == 8 ? FB_CN(8) : FB_CN(16);
 #undef FB_CN
-#undef FB_CN2
 }
 
 // out [rows][C] (ldo elements apart) from x (ldx), w [taps][C]; bias: C floats or null

@@ -86,7 +86,7 @@ gqa_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ 
 // head. proj row = [heads x maps x dim | kv_heads x maps x dim | .. v_off: kv_heads x vdim]. A key row takes a head's maps side by side; a
 // query goes to [row][head][map][hp] with zeros in the other map's columns, so that one product with the key row gives its map's score.
 // HALF: the rotated pairs are (i, i + rot / 2). Without caches only queries are made (the layer reads another layer's keys).
-// One CTA per row: sums of squares over the row, then one warp per head.
+// One CTA per row: sums of squares over the row, then one warp per head; of a few rows several CTAs, which form the same sums and share the heads.
 // Positions, pages and angles do not come from the kernel before this one, so they are read while it drains.
 template <typename T, bool EVEN, bool HALF>
 __global__ void __launch_bounds__(512)
@@ -170,7 +170,7 @@ gqa_row_prep_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restric
     return x;
   };
   const int units = heads * maps + (k_cache ? 2 * kv_heads : 0);
-  for (int u = warp; u < units; u += blockDim.x >> 5) {
+  for (int u = blockIdx.y * (blockDim.x >> 5) + warp; u < units; u += gridDim.y * (blockDim.x >> 5)) {
     if (u < heads * maps) {
       const float* src = pr + u * dim;
       const float* w = q_norm ? q_norm + u * dim : nullptr;
@@ -313,10 +313,10 @@ extern "C" int fb_gqa_row_prep(void* q_out, void* k_cache, void* v_cache, const 
   if (dim < 1 || vdim < 1 || maps < 1 || maps > 2 || maps * dim > hp || vdim > hp || hp % 64 || rot % 2 || rot > dim || (rot && !inv_freq) ||
       (rot && maps == 2 && dim % 2) || (k_cache && (!q_norm) != (!k_norm))) return -1;
   const size_t smem = (size_t)(rot / 2 + 1) * sizeof(float2);
-  const int threads = heads * maps + 2 * kv_heads > 16 ? 512 : 256;
+  const int units = heads * maps + 2 * kv_heads, threads = units > 16 ? 512 : 256, share = rows <= 16 ? (units * 32 + threads - 1) / threads : 1;
   auto go = [&](auto kern, auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    return (int)launch_pdl(kern, dim3(rows), dim3(threads), smem, s, (T*)q_out, (T*)k_cache, (T*)v_cache, proj, ldp, q_norm, k_norm,
+    return (int)launch_pdl(kern, dim3(rows, share), dim3(threads), smem, s, (T*)q_out, (T*)k_cache, (T*)v_cache, proj, ldp, q_norm, k_norm,
                            inv_freq, row_slot, row_pos, block_table, max_blocks, kv_block, heads, kv_heads, maps, dim, vdim, hp, rot, v_off, eps,
                            status);
   };

@@ -268,6 +268,9 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ cq, T*
 // The form with a rotated key part: proj row = [heads x (dim | rot) | latent (kv_rank) | key part (rot)], fp32. Queries go to [row][head][hp] with
 // their last rot columns rotated (pairs (0, 1), (2, 3), ..), the normed latent and the rotated key part to the token's cache row, zeros beyond.
 // Angles are formed and reduced to one turn in double.
+// grid (rows, 1 + groups of LR_HEADS heads): the first CTA of a row makes its cache row, the others heads of its query.
+constexpr int LR_HEADS = 8;
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rot_prep_kernel(T* __restrict__ q_out, T* __restrict__ cache, const float* __restrict__ proj, long ldp,
                                                               const float* __restrict__ kv_norm, const double* __restrict__ inv_freq,
@@ -292,29 +295,35 @@ __global__ void __launch_bounds__(256) latent_rot_prep_kernel(T* __restrict__ q_
   proj = after_wait(proj);
   const float* pr = proj + row * ldp;
   const int kd = dim + rot;
-  const float* pc = pr + (size_t)heads * kd;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss = fmaf(pc[i], pc[i], ss);
-  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)kv_rank + eps);      // (its barriers publish the angles)
   auto turned = [&](const float* src, int e) {               // column e of a rotated part
     const float2 t = lr_turn[e >> 1];
     const float u = src[e & ~1], v = src[e | 1];
     return e & 1 ? v * t.x + u * t.y : u * t.x - v * t.y;
   };
-  if (blk < 0) {
-    if (threadIdx.x == 0) set_status(status, ST_BOUNDS);
-  } else {
+  if (blockIdx.y == 0) {
+    const float* pc = pr + (size_t)heads * kd;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss = fmaf(pc[i], pc[i], ss);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)kv_rank + eps);    // (its barriers publish the angles)
+    if (blk < 0) {
+      if (threadIdx.x == 0) set_status(status, ST_BOUNDS);
+      return;
+    }
     T* dst = cache + ((size_t)blk * kv_block + pos % kv_block) * lat;
     for (int i = threadIdx.x; i < lat; i += blockDim.x)
       dst[i] = Elem<T>::from(i < kv_rank ? pc[i] * r * kv_norm[i] : i < kv_rank + rot ? turned(pc + kv_rank, i - kv_rank) : 0.f);
+    return;
   }
-  for (int i = 2 * threadIdx.x; i < heads * hp; i += 2 * blockDim.x) {
-    const int h = i / hp, d = i % hp;
-    const float* src = pr + h * kd;
+  __syncthreads();
+  const int h = (blockIdx.y - 1) * LR_HEADS + (threadIdx.x >> 5);            // one warp per head
+  if (h >= heads) return;
+  const float* src = pr + h * kd;
+  T* dst = q_out + (row * heads + h) * (size_t)hp;
+  for (int d = 2 * (threadIdx.x & 31); d < hp; d += 64) {
     float o[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) o[e] = d + e < dim ? src[d + e] : d + e < kd ? turned(src + dim, d + e - dim) : 0.f;
-    Elem<T>::store2(q_out + row * (size_t)heads * hp + i, o[0], o[1]);
+    Elem<T>::store2(dst + d, o[0], o[1]);
   }
 }
 
@@ -1010,7 +1019,8 @@ extern "C" int fb_latent_rot_prep(void* q_out, void* cache, const float* proj, l
   if (rot % 2 || rot < 0 || dim < 0 || dim + rot > hp || hp % 2 || kv_rank < 1 || kv_rank + rot > lat) return -1;
   auto go = [&](auto kern, auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    return (int)launch_pdl(kern, dim3(rows), dim3(256), (size_t)(rot / 2 + 1) * sizeof(float2), s, (T*)q_out, (T*)cache, proj, ldp, kv_norm, inv_freq,
+    return (int)launch_pdl(kern, dim3(rows, 1 + (heads + LR_HEADS - 1) / LR_HEADS), dim3(LR_HEADS * 32), (size_t)(rot / 2 + 1) * sizeof(float2), s,
+                           (T*)q_out, (T*)cache, proj, ldp, kv_norm, inv_freq,
                            row_slot, row_pos, block_table, max_blocks, kv_block, heads, dim, rot, hp, kv_rank, lat, eps, status);
   };
   return f32 ? go(latent_rot_prep_kernel<float>, (float*)0) : go(latent_rot_prep_kernel<bf16>, (bf16*)0);
