@@ -62,7 +62,7 @@ class LayerSpec:
     rot_base: float = 1e4
     rot_scaling: Optional[dict] = None   # long wavelengths stretched: factor, low, high, original
     conv: int = 0                   # cdelta, ssm: taps of the short convolutions
-    norm_groups: int = 1            # ssm: parts of the gated output, each normed by its own root mean square
+    norm_groups: int = 1            # ssm: equal parts of the gated output with an RMS norm each
     decay_rank: int = 0             # cdelta: width between the two decay projections (0: the checkpoint says)
     gate_rank: int = 0              # cdelta: ... and between the two output gate projections
 

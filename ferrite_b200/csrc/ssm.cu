@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(SS_THREADS) ssm_step_kernel(float* __restrict_
   }
 }
 
-// out = y * silu(z), each of `parts` equal parts of the row divided by its root mean square, times w; grid (rows, parts (+ tail blocks)). With
+// out = y * silu(z), an RMS norm over each of `parts` equal parts of the row, times w; grid (rows, parts (+ tail blocks)). With
 // `tails` (one row per segment) CTAs behind the parts move the slot's tail on by the row's inputs: nobody reads the old one any more.
 // VEC: four columns at a time.
 constexpr int GN_THREADS = 256, GN_TAIL = 1024;              // channels of a tail per CTA

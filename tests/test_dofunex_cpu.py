@@ -454,7 +454,7 @@ def test_command_line_generates(models, capsys):
 def test_two_ranks_equal_one():
     import torch.multiprocessing as mp
 
-    from test_tp_cpu import _free_port, _worker
+    from test_tp_cpu import _free_port, _worker, gather
     cfg = tiny_dofunex()
     prompt = torch.randint(0, cfg.vocab, (70,), generator=torch.Generator().manual_seed(6)).tolist()
     eng = Engine(cfg, init_weights(cfg, seed=0), EngineConfig(n_slots=1, max_ctx=128), device="cpu")
@@ -465,7 +465,7 @@ def test_two_ranks_equal_one():
     procs = [ctx.Process(target=_worker, args=(r, 2, port, prompt, q, "tiny-dofunex")) for r in range(2)]
     for p in procs:
         p.start()
-    outs = sorted([q.get(timeout=180) for _ in range(2)], key=lambda t: t[0])
+    outs = gather(q, 2)
     for p in procs:
         p.join(timeout=60)
     for rank, logits, ids, l2 in outs:

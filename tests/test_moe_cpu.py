@@ -77,7 +77,7 @@ def _worker(rank, world, port, q, plen=20):
         cfg = tiny_moe("softmax")
         eng = Engine(cfg, weights(cfg), EngineConfig(n_slots=1, max_ctx=128), device="cpu", tp=tp)
         logits, _, _ = eng.forward([Segment(0, 0, prompt_of(cfg, plen), "all")])
-        q.put((rank, logits))
+        q.put((rank, logits.numpy()))       # by value: a tensor's shared storage is gone once its process has ended
         dist.destroy_process_group()
     except Exception as e:  # noqa: BLE001
         q.put((rank, repr(e)))
@@ -101,7 +101,7 @@ def test_expert_parallel_two_ranks(plen):
         p.join(timeout=60)
     for rank, logits in outs:
         assert not isinstance(logits, str), logits
-        assert torch.allclose(logits, want, atol=5e-5, rtol=1e-4), rank
+        assert torch.allclose(torch.from_numpy(logits), want, atol=5e-5, rtol=1e-4), rank
 
 
 def test_expert_heat_counters(tmp_path, monkeypatch):

@@ -34,8 +34,15 @@ def _worker(rank, world, port, prompt, q, preset="tiny"):
     eng = Engine(cfg, w, EngineConfig(n_slots=1, max_ctx=128), device="cpu", tp=tp)
     logits, picks, _ = eng.forward([Segment(0, 0, prompt, "all")])
     l2, p2, _ = eng.forward([Segment(0, len(prompt), [int(picks[0][-1])], "last")])
-    q.put((rank, logits, picks[0], l2))
+    # arrays travel by value; a tensor's shared storage is gone once its process has ended
+    q.put((rank, logits.numpy(), picks[0].numpy(), l2.numpy()))
     dist.destroy_process_group()
+
+
+def gather(q, world):
+    """What the ranks' workers put, by rank, as tensors."""
+    outs = sorted([q.get(timeout=180) for _ in range(world)], key=lambda t: t[0])
+    return [(o[0], *(torch.from_numpy(x) for x in o[1:])) for o in outs]
 
 
 @pytest.mark.parametrize("world,plen", [(2, 24), (2, 97)])
@@ -54,7 +61,7 @@ def test_tp_matches_single_rank(world, plen):
     procs = [ctx.Process(target=_worker, args=(r, world, port, prompt, q)) for r in range(world)]
     for p in procs:
         p.start()
-    outs = sorted([q.get(timeout=120) for _ in range(world)], key=lambda t: t[0])
+    outs = gather(q, world)
     for p in procs:
         p.join(timeout=60)
     for rank, logits, ids, l2 in outs:
@@ -81,7 +88,7 @@ def test_moe_latent_attention_model_under_tp2(plen):
     procs = [ctx.Process(target=_worker, args=(r, 2, port, prompt, q, "tiny-mla")) for r in range(2)]
     for p in procs:
         p.start()
-    outs = sorted([q.get(timeout=180) for _ in range(2)], key=lambda t: t[0])
+    outs = gather(q, 2)
     for p in procs:
         p.join(timeout=60)
     for rank, logits, ids, l2 in outs:

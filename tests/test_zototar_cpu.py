@@ -326,7 +326,7 @@ def test_trace_replay(models, tmp_path, monkeypatch, capsys):
 def test_two_ranks_equal_one():
     import torch.multiprocessing as mp
 
-    from test_tp_cpu import _free_port, _worker
+    from test_tp_cpu import _free_port, _worker, gather
     cfg = tiny_zototar()
     prompt = torch.randint(0, cfg.vocab, (70,), generator=torch.Generator().manual_seed(6)).tolist()
     eng = Engine(cfg, init_weights(cfg, seed=0), EngineConfig(n_slots=1, max_ctx=128), device="cpu")
@@ -337,7 +337,7 @@ def test_two_ranks_equal_one():
     procs = [ctx.Process(target=_worker, args=(r, 2, port, prompt, q, "tiny-zototar")) for r in range(2)]
     for p in procs:
         p.start()
-    outs = sorted([q.get(timeout=180) for _ in range(2)], key=lambda t: t[0])
+    outs = gather(q, 2)
     for p in procs:
         p.join(timeout=60)
     for rank, logits, ids, l2 in outs:
